@@ -1,13 +1,15 @@
 """In-tree native builds.
 
-Two shared libraries are produced under ``oxibonsai_b200/_lib``:
+Three shared libraries are produced under ``oxibonsai_b200/_lib``:
 
 * ``libbonsai_host.so`` - C++17 host library (GGUF, codecs, CPU oracle, runtime data structures),
   compiled with g++.
 * ``libbonsai_cuda.so`` - every CUDA kernel and native launcher, compiled by nvcc for
   ``sm_100a`` only (``-gencode arch=compute_100a,code=sm_100a``); nvcc cross-compiles without a GPU.
+* ``libbonsai_layered.so`` - the kernels of the layer-list decoders (``csrc/layered``) with the sampler and the tcgen05 GEMM
+  they share with the other models: what serving such a model needs, and no more.
 
-Both expose a plain C ABI and are loaded with ctypes (``oxibonsai_b200._native``), so neither the
+All expose a plain C ABI and are loaded with ctypes (``oxibonsai_b200._native``), so neither the
 build nor the import depends on torch's extension machinery.  A content hash of the sources is
 stored beside each library; a library is rebuilt only when its hash is stale.
 """
@@ -32,10 +34,8 @@ NVCC_FLAGS = ["-std=c++17", "-O3", "-lineinfo", "-shared", "-Xcompiler", "-fPIC"
 
 
 def _sources(kind: str) -> list[Path]:
-    if kind == "host":
-        pats = ["capi_*.cpp", "core/*.cpp", "cpu/*.cpp", "runtime/*.cpp"]
-    else:
-        pats = ["cuda/*.cu", "comm/*.cu"]
+    pats = {"host": ["capi_*.cpp", "core/*.cpp", "cpu/*.cpp", "runtime/*.cpp"], "cuda": ["cuda/*.cu", "comm/*.cu"],
+            "layered": ["layered/*.cu", "cuda/sampler.cu", "cuda/bitgemm_prefill.cu"]}[kind]
     out: list[Path] = []
     for p in pats:
         out += sorted(CSRC.glob(p))
@@ -45,17 +45,15 @@ def _sources(kind: str) -> list[Path]:
 def _digest(kind: str, flags: list[str]) -> str:
     h = hashlib.sha256()
     h.update(" ".join(flags).encode())
-    for p in sorted(CSRC.rglob("*")):
-        if p.suffix in (".cpp", ".hpp", ".h", ".cu", ".cuh"):
-            if kind == "host" and p.suffix in (".cu", ".cuh"):
-                continue
-            h.update(p.relative_to(CSRC).as_posix().encode())
-            h.update(p.read_bytes())
+    headers = (".hpp", ".h") if kind == "host" else (".hpp", ".h", ".cuh")
+    for p in sorted(set(_sources(kind)) | {q for q in CSRC.rglob("*") if q.suffix in headers}):
+        h.update(p.relative_to(CSRC).as_posix().encode())
+        h.update(p.read_bytes())
     return h.hexdigest()
 
 
 def lib_path(kind: str) -> Path:
-    return LIB / ("libbonsai_host.so" if kind == "host" else "libbonsai_cuda.so")
+    return LIB / f"libbonsai_{kind}.so"
 
 
 def is_stale(kind: str) -> bool:
@@ -80,7 +78,7 @@ def _headers_digest(kind: str, flags: list[str]) -> str:
 
 
 def build(kind: str, force: bool = False, verbose: bool = False) -> Path:
-    """Builds one library (``"host"`` or ``"cuda"``) if its sources changed; returns its path.
+    """Builds one library (``"host"``, ``"cuda"`` or ``"layered"``) if its sources changed; returns its path.
 
     Each translation unit is compiled to an object under ``_lib/obj`` (skipped when neither it nor
     any header changed) and the objects are linked into the shared library.
@@ -104,7 +102,7 @@ def build(kind: str, force: bool = False, verbose: bool = False) -> Path:
         if cc is None:
             raise RuntimeError("nvcc not found; cannot build the CUDA library")
     cflags = [f for f in flags if f != "-shared"]
-    if kind == "cuda" and verbose:
+    if kind != "host" and verbose:
         cflags += ["-Xptxas", "-v"]
     hd = _headers_digest(kind, cflags)
 
@@ -176,12 +174,12 @@ def sanitizer_runtimes() -> list[str]:
 
 
 def build_all(force: bool = False, verbose: bool = False) -> dict[str, Path]:
-    return {k: build(k, force=force, verbose=verbose) for k in ("host", "cuda")}
+    return {k: build(k, force=force, verbose=verbose) for k in ("host", "cuda", "layered")}
 
 
 if __name__ == "__main__":
     force = "--force" in sys.argv
     verbose = "-v" in sys.argv
-    kinds = [a for a in sys.argv[1:] if a in ("host", "cuda")] or ["host", "cuda"]
+    kinds = [a for a in sys.argv[1:] if a in ("host", "cuda", "layered")] or ["host", "cuda", "layered"]
     for k in kinds:
         print(k, "->", build(k, force=force, verbose=verbose))

@@ -1,9 +1,9 @@
-"""ctypes loaders for the two in-tree native libraries.
+"""ctypes loaders for the in-tree native libraries.
 
-``host()`` returns ``libbonsai_host.so`` (C++: GGUF, codecs, CPU oracle, runtime structures) and
-``cuda()`` returns ``libbonsai_cuda.so`` (sm_100a kernels and native launchers).  Libraries are
-built on first use when missing or stale and a compiler is present.  ``cuda()`` raises when the
-library cannot be loaded: GPU code paths never fall back silently to PyTorch ops.
+``host()`` returns ``libbonsai_host.so`` (C++: GGUF, codecs, CPU oracle, runtime structures),
+``cuda()`` returns ``libbonsai_cuda.so`` (sm_100a kernels and native launchers) and ``layered()``
+``libbonsai_layered.so`` (kernels of the layer-list decoders).  Libraries are built on first use when
+missing or stale and a compiler is present.  ``cuda()`` and ``layered()`` raise when the library cannot be loaded: GPU code paths never fall back silently to PyTorch ops.
 """
 from __future__ import annotations
 
@@ -15,6 +15,7 @@ from . import _build
 _lock = threading.Lock()
 _host = None
 _cuda = None
+_layered = None
 
 
 class NativeError(RuntimeError):
@@ -39,7 +40,7 @@ def _load(kind: str) -> C.CDLL:
             # on the file lock and find the library fresh when they get it.
             import fcntl
             _build.LIB.mkdir(exist_ok=True)
-            with open(_build.LIB / f".{kind}.lock", "w") as lock:
+            with open(_build.LIB / ".build.lock", "w") as lock:      # the CUDA libraries share object files
                 fcntl.flock(lock, fcntl.LOCK_EX)
                 try:
                     if _build.is_stale(kind):
@@ -71,6 +72,15 @@ def cuda() -> C.CDLL:
                 lib = _load("cuda")
                 _cuda = lib
     return _cuda
+
+
+def layered() -> C.CDLL:
+    global _layered
+    if _layered is None:
+        with _lock:
+            if _layered is None:
+                _layered = _load("layered")
+    return _layered
 
 
 def check(rc: int) -> int:

@@ -28,6 +28,7 @@
 // kept in the same order ("paired-K" layout), which every producer of a prefill activation writes
 // (norm_to_f16_paired_kernel, the SwiGLU epilogue here, the prefill attention output).
 #include <cuda.h>
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 
 #include "common.cuh"
@@ -61,7 +62,9 @@ struct PfParams {
   __half* out_f16;         // [T][out_ld]  (epi 2: SwiGLU, paired-K order; epi 3: plain f16 store)
   int* status;
   int n_rows, K, T, epi, out_ld;
-  int dense;               // 1: A is a dense f16 matrix fetched by TMA (natural K order), no expansion
+  int dense;               // 1: A is a dense f16 / bf16 matrix fetched by TMA (natural K order), no expansion
+  int bf16;                // dense operands are bf16 (both) instead of f16
+  float glu_limit, glu_alpha, glu_offset;   // epi 4
   int streamk;             // 1: ranges cut anywhere in (tile, pair) space, partial tiles meet in the workspace
   float* ws_part;          // [2 * grid][TOK][128] partial accumulators
   int* ws_count;           // [tiles] arrival counters, zero between launches
@@ -123,7 +126,13 @@ __device__ __forceinline__ float pf_residual(const PfParams& p, int tok, int row
 
 // epilogue for one accumulator value; every lane of the warp calls it (epi 2 exchanges gate / up between lanes)
 __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, int tok, int row, int a, bool row_ok) {
-  if (p.epi == 2) {
+  if (p.epi == 4) {
+    // clamped gated unit: min(g, limit) * sigmoid(alpha g) * (clamp(u, -limit, limit) + offset), stored as bf16
+    const float u = fminf(fmaxf(__shfl_xor_sync(0xffffffffu, v, 1), -p.glu_limit), p.glu_limit), g = fminf(v, p.glu_limit);
+    if (row_ok && tok < p.T && (a & 1) == 0)
+      reinterpret_cast<__nv_bfloat16*>(p.out_f16)[(size_t)tok * p.out_ld + (row >> 1)] =
+          __float2bfloat16_rn(g / (1.0f + expf(-p.glu_alpha * g)) * (u + p.glu_offset));
+  } else if (p.epi == 2) {
     float other = __shfl_xor_sync(0xffffffffu, v, 1);
     if (row_ok && tok < p.T && (a & 1) == 0)
       p.out_f16[(size_t)tok * p.out_ld + paired_k(row >> 1)] = __float2half_rn(v / (1.0f + __expf(-v)) * other);
@@ -235,7 +244,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
     if (failed && lane == 0) atomicExch(p.status, 1);
   } else if (warp >= kPfMmaWarp && warp < kPfMmaWarp + NISS) {
     // ------------------------------- MMA issuers ------------------------------------------------
-    constexpr uint32_t idesc = tc::idesc_f32acc(tc::FMT_F16, tc::FMT_F16, 128, TOK);
+    const uint32_t idesc = p.bf16 ? tc::idesc_f32acc(tc::FMT_BF16, tc::FMT_BF16, 128, TOK) : tc::idesc_f32acc(tc::FMT_F16, tc::FMT_F16, 128, TOK);
     const int mw = warp - kPfMmaWarp;
     int pair = pair0, seg = 0;
     bool fresh = true;   // this issuer's next MMA starts its accumulator of the segment: overwrite instead of accumulate
@@ -521,12 +530,13 @@ __global__ void norm_to_f16_paired_kernel(const float* __restrict__ x, int x_ld,
 
 }  // namespace bonsai
 
-static bool make_map_f16(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer, uint64_t ld_elems, uint32_t box_rows) {
+static bool make_map_f16(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer, uint64_t ld_elems, uint32_t box_rows,
+                         CUtensorMapDataType type = CU_TENSOR_MAP_DATA_TYPE_FLOAT16) {
   cuuint64_t dims[2] = {(cuuint64_t)inner, (cuuint64_t)outer};
   cuuint64_t strides[1] = {(cuuint64_t)ld_elems * 2};
   cuuint32_t box[2] = {64, box_rows};
   cuuint32_t estr[2] = {1, 1};
-  return cuTensorMapEncodeTiled(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+  return cuTensorMapEncodeTiled(map, type, 2, const_cast<void*>(base), dims, strides, box, estr,
                                 CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                                 CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
@@ -592,9 +602,26 @@ int bonsai_bitgemm_prefill_ws(const void* codes, const void* scales, const void*
     amap = xmap;
   }
   PfParams p{(const uint32_t*)codes, (const __half*)scales, out_f32, residual, (__half*)out_f16, status, n_rows, K, T, epi, out_ld,
-             dense_w != nullptr ? 1 : 0, 0, nullptr, nullptr};
+             dense_w != nullptr ? 1 : 0, 0, 0.0f, 0.0f, 0.0f, 0, nullptr, nullptr};
   return tok == 64 ? launch_prefill<64>(xmap, amap, p, sms, ws, ws_bytes, balance, stream)
                    : launch_prefill<256>(xmap, amap, p, sms, ws, ws_bytes, balance, stream);
+}
+
+// Dense bf16 operands: W [n_rows][K] (K a multiple of 128), x [T][x_ld], f32 accumulation.  epi 0: out_f32 = W x; 4: out_bf16 =
+// clamped gated unit over interleaved gate / up rows (n_rows / 2 columns).  Workspace and status as above.
+int bonsai_dense_gemm_bf16(const void* w, int n_rows, int K, const void* x, int x_ld, int T, float* out_f32, void* out_bf16, int out_ld, int epi,
+                           float limit, float alpha, float offset, int* status, void* ws, size_t ws_bytes, int sms, cudaStream_t stream) {
+  using namespace bonsai;
+  if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && epi != 4)) return BONSAI_CUDA_BAD_ARG;
+  if ((epi == 0 && out_f32 == nullptr) || (epi == 4 && (out_bf16 == nullptr || n_rows % 2 != 0)) || status == nullptr) return BONSAI_CUDA_BAD_ARG;
+  const int tok = T <= 64 ? 64 : 256;
+  CUtensorMap xmap, amap;
+  if (!make_map_f16(&xmap, x, K, T, x_ld, tok, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
+      !make_map_f16(&amap, w, K, n_rows, K, 128, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
+    return BONSAI_CUDA_BAD_ARG;
+  PfParams p{nullptr, nullptr, out_f32, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, 1, limit, alpha, offset, 0, nullptr, nullptr};
+  return tok == 64 ? launch_prefill<64>(xmap, amap, p, sms, ws, ws_bytes, 1, stream)
+                   : launch_prefill<256>(xmap, amap, p, sms, ws, ws_bytes, 1, stream);
 }
 
 int bonsai_bitgemm_prefill(const void* codes, const void* scales, const void* x_f16, int x_ld, float* out_f32,

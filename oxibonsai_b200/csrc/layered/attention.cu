@@ -1,0 +1,621 @@
+// Attention of the layer-list decoders over a paged cache whose rows are both key and value.
+//
+// The design's values are its un-normalised keys, so one cache row per token and kv head serves both products: the row holds
+// the projected key, and a float beside it the reciprocal root mean square of the key norm.  The norm's weight and the score
+// scale are folded into the query (q' = norm(q) * w_q * w_k * scale), the key's root mean square multiplies the score of its
+// column.  That halves the cache traffic of separate K and V rows, and a tile is staged once for S = Q K^T and O = P K.
+//
+//   score(i, j) = q'_i . k_j * rk_j - slope_h (i - j)      j <= i and (i - j < window or j < keep)
+//   out         = softmax(score) K * sigmoid(gate_h)
+//
+// Rows of a batch are tokens: a row has a position and a slot (its sequence's block-table row).  `append_kernel` writes the
+// rows' keys; `prompt_kernel` handles portions of prompts (tiles of 64 query rows = tokens x heads of one kv group);
+// `decode_kernel` single tokens, whose append it does itself; `f32_kernel` is the 32-bit mode for both.
+// Only the page tiles that a window can see are visited: the kept first tokens and the window's range.
+#include <cooperative_groups.h>
+
+#include "layered/layered.cuh"
+
+namespace bonsai {
+namespace lay {
+
+struct Attn {
+  const float* proj;        // [T][ld]: q heads at q_col, k heads at k_col, one gate per head at g_col
+  const float* q_norm;      // [dim]
+  const float* k_norm;      // [dim]
+  const float* slopes;      // [heads]
+  const int* pos;           // [T]
+  const int* slots;         // [T]
+  const int* block_table;   // [slots][max_pages]
+  void* pool;               // [pages][kv_heads][page_size][HD], bf16 (f32 in the 32-bit mode), columns past dim zero
+  float* krms;              // [pages][kv_heads][page_size]
+  void* out;                // [T][ldo], head h at h * dim
+  int ld, q_col, k_col, g_col, ldo;
+  int heads, kv_heads, dim, max_pages, pshift;   // page size 1 << pshift
+  int window, keep;         // window <= 0: no window
+  float eps, scale;
+};
+
+// first visible position outside the kept ones for a query at `p`
+__device__ __forceinline__ int window_lo(const Attn& a, int p) { return a.window > 0 ? max(0, p - a.window + 1) : 0; }
+__device__ __forceinline__ bool sees(const Attn& a, int i, int j) { return j <= i && (a.window <= 0 || i - j < a.window || j < a.keep); }
+__device__ __forceinline__ size_t cache_row(const Attn& a, const int* bt, int kvh, int t) {
+  return ((((size_t)bt[t >> a.pshift] * a.kv_heads + kvh) << a.pshift)) + (t & ((1 << a.pshift) - 1));
+}
+
+// A warp writes one key row and its reciprocal root mean square.
+template <int HD, typename C>
+__device__ __forceinline__ void append_row(const Attn& a, const float* k, size_t row, int lane) {
+  C* dst = static_cast<C*>(a.pool) + row * HD;
+  float ss = 0.0f;
+#pragma unroll
+  for (int d = lane; d < HD; d += 32) {
+    const float v = d < a.dim ? k[d] : 0.0f;
+    store_act(dst + d, v);
+    ss += v * v;
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) a.krms[row] = 1.0f / sqrtf(ss / (float)a.dim + a.eps);
+}
+
+// grid (row groups of 4 x kv head): one warp per (row of the list, kv head)
+template <int HD, typename C>
+__global__ void append_kernel(Attn a, int first, int count) {
+  pdl_wait();
+  pdl_trigger();
+  const int lane = threadIdx.x & 31, i = blockIdx.x * 4 + (threadIdx.x >> 5), kvh = blockIdx.y;
+  if (i >= count) return;
+  const int t = first + i;
+  if (a.pos[t] >= (a.max_pages << a.pshift)) return;
+  const int* bt = a.block_table + (size_t)a.slots[t] * a.max_pages;
+  append_row<HD, C>(a, a.proj + (size_t)t * a.ld + a.k_col + kvh * a.dim, cache_row(a, bt, kvh, a.pos[t]), lane);
+}
+
+// A warp normalises one query head and leaves q' * log2(e) in dst (columns past dim zero): scores are base-2 logarithms.
+template <int HD>
+__device__ __forceinline__ void load_query(const Attn& a, const float* q, bf16* dst, int lane) {
+  float v[HD / 32], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < HD / 32; ++i) {
+    const int d = lane + 32 * i;
+    v[i] = d < a.dim ? q[d] : 0.0f;
+    ss += v[i] * v[i];
+  }
+  ss = warp_sum(ss);
+  const float f = a.scale * kLog2e / sqrtf(ss / (float)a.dim + a.eps);
+#pragma unroll
+  for (int i = 0; i < HD / 32; ++i) {
+    const int d = lane + 32 * i;
+    dst[d] = __float2bfloat16_rn(d < a.dim ? v[i] * f * a.q_norm[d] * a.k_norm[d] : 0.0f);
+  }
+}
+
+// ---- portions of prompts ------------------------------------------------------------------------------------------------------
+// entries[e] = {first row, tokens, slot, first position}; tiles[i] = {entry, first token of the tile}.  A tile holds
+// 64 / G tokens x the G query heads of one kv head.
+template <int HD>
+__global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries, const int2* tiles) {
+  constexpr int LD = HD + 8;
+  constexpr bool kQReg = HD <= 128;   // query fragments stay in registers (else they are re-read from shared memory)
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  bf16* sQ = reinterpret_cast<bf16*>(smem_raw);
+  bf16* sK = sQ + 64 * LD;            // two stages of [64][LD]
+  float* sR = reinterpret_cast<float*>(sK + 2 * 64 * LD);   // two stages of 64 key factors
+  const int kvh = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int G = a.heads / a.kv_heads, tpt = 64 / G;
+  pdl_wait();
+  pdl_trigger();
+  const int2 tl = tiles[gridDim.y - 1 - blockIdx.y];
+  const int4 en = entries[tl.x];
+  const int q0 = tl.y, ntok = min(tpt, en.y - q0), rows = ntok * G;
+  const int pfirst = en.w + q0, plast = pfirst + ntok - 1;
+  const int lo = window_lo(a, pfirst), hi = plast + 1;
+  const int* bt = a.block_table + (size_t)en.z * a.max_pages;
+  const bf16* pool = static_cast<const bf16*>(a.pool);
+
+  auto fetch = [&](int kb, int st) {
+    bf16* dst = sK + st * 64 * LD;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < 64 * (HD / 8); i += 128) {
+      const int r = i / (HD / 8), c = (i % (HD / 8)) * 8, t = kb + r;
+      const bool ok = t < hi;
+      cp_async16(dst + r * LD + c, pool + (ok ? cache_row(a, bt, kvh, t) * HD + c : 0), ok);
+    }
+    if (threadIdx.x < 64) sR[st * 64 + threadIdx.x] = kb + threadIdx.x < hi ? a.krms[cache_row(a, bt, kvh, kb + threadIdx.x)] : 0.0f;
+  };
+  // key tiles: those that hold kept tokens, then those of the window's range
+  auto next = [&](int kb) {
+    kb += 64;
+    if (kb >= a.keep && kb + 64 <= lo) kb = lo & ~63;
+    return kb;
+  };
+  int kb = next(-64);
+  fetch(kb, 0);
+  cp_async_commit();
+  for (int r = warp * 16; r < warp * 16 + 16; ++r) {
+    if (r < rows) {
+      load_query<HD>(a, a.proj + (size_t)(en.x + q0 + r / G) * a.ld + a.q_col + (kvh * G + r % G) * a.dim, sQ + r * LD, lane);
+    } else {
+      for (int d = lane; d < HD; d += 32) sQ[r * LD + d] = __float2bfloat16_rn(0.0f);
+    }
+  }
+  __syncwarp();
+  uint32_t qf[kQReg ? HD / 16 : 1][4];
+  if (kQReg) {
+#pragma unroll
+    for (int ks = 0; ks < (kQReg ? HD / 16 : 1); ++ks) ldsm4(qf[ks], frag_a(sQ, LD, warp * 16, ks * 16, lane));
+  }
+  float o[HD / 8][4];
+#pragma unroll
+  for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+  int row[2], qpos[2], head[2];
+  float slope[2];
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    row[e] = warp * 16 + (lane >> 2) + 8 * e;
+    qpos[e] = row[e] < rows ? pfirst + row[e] / G : -1;      // rows past the tile see nothing
+    head[e] = kvh * G + row[e] % G;
+    slope[e] = a.slopes[head[e]] * kLog2e;
+  }
+  const int wfirst = pfirst + warp * 16 / G, wlast = min(plast, pfirst + (warp * 16 + 15) / G);   // positions of this warp's rows
+  const bool wlive = warp * 16 + 15 < rows;
+  for (int it = 0; kb < hi; ++it) {
+    const int nx = next(kb);
+    if (nx < hi) fetch(nx, (it + 1) & 1);
+    cp_async_commit();
+    cp_async_wait<1>();
+    __syncthreads();
+    const bf16* k = sK + (it & 1) * 64 * LD;
+    const float* kr = sR + (it & 1) * 64;
+    float s[8][4];
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.0f;
+#pragma unroll
+    for (int ks = 0; ks < HD / 16; ++ks) {
+      uint32_t qt[4];
+      if (!kQReg) ldsm4(qt, frag_a(sQ, LD, warp * 16, ks * 16, lane));
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        uint32_t b[4];
+        ldsm4(b, frag_b_rows(k, LD, np * 16, ks * 16, lane));
+        mma_bf16(s[2 * np], kQReg ? qf[kQReg ? ks : 0] : qt, b[0], b[1]);
+        mma_bf16(s[2 * np + 1], kQReg ? qf[kQReg ? ks : 0] : qt, b[2], b[3]);
+      }
+    }
+    const bool whole = wlive && kb + 63 <= wfirst && (a.window <= 0 || wlast - kb < a.window || kb + 63 < a.keep);
+    float nm[2] = {mx[0], mx[1]};
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) {
+      const int c = nt * 8 + (lane & 3) * 2;
+      const float2 f = *reinterpret_cast<const float2*>(kr + c);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = e >> 1, j = kb + c + (e & 1);
+        s[nt][e] = s[nt][e] * ((e & 1) ? f.y : f.x) - slope[r] * (float)(qpos[r] - j);
+        if (!whole && !sees(a, qpos[r], j)) s[nt][e] = -INFINITY;
+        nm[r] = fmaxf(nm[r], s[nt][e]);
+      }
+    }
+    float base[2], resc[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      nm[r] = fmaxf(nm[r], __shfl_xor_sync(0xffffffffu, nm[r], 1));
+      nm[r] = fmaxf(nm[r], __shfl_xor_sync(0xffffffffu, nm[r], 2));
+      base[r] = nm[r] == -INFINITY ? 0.0f : nm[r];           // nothing visible yet: every term is ex2(-inf) = 0
+      resc[r] = ex2(mx[r] - base[r]);
+      mx[r] = nm[r];
+      l[r] *= resc[r];
+    }
+    uint32_t p[8][2];
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) {
+      float v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        v[e] = ex2(s[nt][e] - base[e >> 1]);
+        l[e >> 1] += v[e];
+      }
+      p[nt][0] = pack_bf16(v[0], v[1]);
+      p[nt][1] = pack_bf16(v[2], v[3]);
+    }
+#pragma unroll
+    for (int i = 0; i < HD / 8; ++i) {
+      o[i][0] *= resc[0]; o[i][1] *= resc[0];
+      o[i][2] *= resc[1]; o[i][3] *= resc[1];
+    }
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks) {
+      const uint32_t pa[4] = {p[2 * ks][0], p[2 * ks][1], p[2 * ks + 1][0], p[2 * ks + 1][1]};
+#pragma unroll
+      for (int np = 0; np < HD / 16; ++np) {
+        uint32_t b[4];
+        ldsm4_t(b, frag_b_cols(k, LD, ks * 16, np * 16, lane));
+        mma_bf16(o[2 * np], pa, b[0], b[1]);
+        mma_bf16(o[2 * np + 1], pa, b[2], b[3]);
+      }
+    }
+    __syncthreads();   // every warp is done with this stage before it is refilled
+    kb = nx;
+  }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+    if (row[r] >= rows) continue;
+    const size_t t = en.x + q0 + row[r] / G;
+    const float f = sigmoid(a.proj[t * a.ld + a.g_col + head[r]]) / l[r];   // the query's own position is always visible
+    bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + head[r] * a.dim;
+#pragma unroll
+    for (int nt = 0; nt < HD / 8; ++nt) {
+      const int d = nt * 8 + (lane & 3) * 2;
+      if (d < a.dim) dst[d] = __float2bfloat16_rn(o[nt][2 * r] * f);
+      if (d + 1 < a.dim) dst[d + 1] = __float2bfloat16_rn(o[nt][2 * r + 1] * f);
+    }
+  }
+}
+
+// ---- single tokens --------------------------------------------------------------------------------------------------------------
+// grid (kv heads x groups of 16 query heads, splits, rows); the splits of one row form a cluster and meet in distributed
+// shared memory.  A warp walks 16-token tiles of the visible range; the split that holds the row's own position appends its
+// key before it reads it.
+template <int HD>
+__global__ void __launch_bounds__(256) decode_kernel(Attn a) {
+  constexpr int LD = HD + 8, NW = 8;
+  constexpr int kTile = 16 * LD;      // elements of a tile
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                    // [16][LD]
+  float* res = reinterpret_cast<float*>(sQ + kTile);               // this CTA's merged rows [16][HD + 2]
+  bf16* tiles = reinterpret_cast<bf16*>(res + 16 * (HD + 2));      // [warp][2][16][LD], later the warps' partial rows
+  float* part = reinterpret_cast<float*>(tiles);                   // [warp][16][HD + 2]
+  namespace cg = cooperative_groups;
+  cg::cluster_group cluster = cg::this_cluster();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int G = a.heads / a.kv_heads, mg = (G + 15) / 16;
+  const int kvh = blockIdx.x / mg, h0 = (blockIdx.x % mg) * 16, nh = min(16, G - h0);
+  const int split = blockIdx.y, nsplit = gridDim.y;
+  // the row's place and the keys of earlier positions are older than the kernel before this one
+  const int t = blockIdx.z;
+  const int pos = a.pos[t];
+  if (pos >= (a.max_pages << a.pshift)) {    // no page can hold it: the whole cluster leaves
+    pdl_wait();
+    pdl_trigger();
+    return;
+  }
+  const int* bt = a.block_table + (size_t)a.slots[t] * a.max_pages;
+  const bf16* pool = static_cast<const bf16*>(a.pool);
+  const int lo16 = window_lo(a, pos) >> 4, end16 = (pos >> 4) + 1;
+  const int nkeep = a.window > 0 ? min((a.keep + 15) >> 4, lo16) : 0;     // tiles of kept tokens before the window's first tile
+  const int ntiles = nkeep + end16 - lo16;
+  const int per = (ntiles + nsplit - 1) / nsplit;
+  const int b0 = split * per, b1 = min(ntiles, b0 + per);
+  const bool owner = b1 == ntiles && b0 < b1;                            // holds the last tile: the row's own position
+  bf16* wt = tiles + warp * 2 * kTile;
+  auto first_token = [&](int j) { return (j < nkeep ? j : lo16 + j - nkeep) << 4; };
+  float2 kf[2], kn[2];   // key factors of this lane's columns: current and next tile
+  auto issue = [&](int j, int buf) {
+    const int tb = first_token(j);
+#pragma unroll 4
+    for (int i = lane; i < 16 * (HD / 8); i += 32) {
+      const int r = i / (HD / 8), c = (i % (HD / 8)) * 8;
+      const bool ok = tb + r <= pos;
+      cp_async16(wt + buf * kTile + r * LD + c, pool + (ok ? cache_row(a, bt, kvh, tb + r) * HD + c : 0), ok);
+    }
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      const int j0 = tb + nt * 8 + (lane & 3) * 2;
+      kn[nt].x = j0 <= pos ? __ldcg(a.krms + cache_row(a, bt, kvh, j0)) : 0.0f;
+      kn[nt].y = j0 + 1 <= pos ? __ldcg(a.krms + cache_row(a, bt, kvh, j0 + 1)) : 0.0f;
+    }
+  };
+  const bool early = b0 + warp < b1 && !(owner && b0 + warp == b1 - 1);
+  if (early) issue(b0 + warp, 0);
+  pdl_wait();
+  pdl_trigger();
+  const float* prow = a.proj + (size_t)t * a.ld;
+  for (int r = warp; r < 16 + (owner ? 1 : 0); r += NW) {
+    if (r < nh) load_query<HD>(a, prow + a.q_col + (kvh * G + h0 + r) * a.dim, sQ + r * LD, lane);
+    else if (r < 16)
+      for (int d = lane; d < HD; d += 32) sQ[r * LD + d] = __float2bfloat16_rn(0.0f);
+    else {
+      append_row<HD, bf16>(a, prow + a.k_col + kvh * a.dim, cache_row(a, bt, kvh, pos), lane);
+      __threadfence();
+    }
+  }
+  __syncthreads();
+  float o[HD / 8][4];
+#pragma unroll
+  for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+  const int g = lane >> 2;
+  float slope[2];
+#pragma unroll
+  for (int r = 0; r < 2; ++r) slope[r] = a.slopes[kvh * G + h0 + min(g + 8 * r, nh - 1)] * kLog2e;
+  if (b0 + warp < b1 && !early) issue(b0 + warp, 0);
+  cp_async_commit();
+  int buf = 0;
+  for (int j = b0 + warp; j < b1; j += NW, buf ^= 1) {
+    kf[0] = kn[0];
+    kf[1] = kn[1];
+    if (j + NW < b1) issue(j + NW, buf ^ 1);
+    cp_async_commit();
+    cp_async_wait<1>();
+    __syncwarp();
+    const bf16* k = wt + buf * kTile;
+    const int tb = first_token(j);
+    float s[2][4] = {};
+#pragma unroll
+    for (int ks = 0; ks < HD / 16; ++ks) {
+      uint32_t q[4], b[4];
+      ldsm4(q, frag_a(sQ, LD, 0, ks * 16, lane));
+      ldsm4(b, frag_b_rows(k, LD, 0, ks * 16, lane));
+      mma_bf16(s[0], q, b[0], b[1]);
+      mma_bf16(s[1], q, b[2], b[3]);
+    }
+    float nm[2] = {mx[0], mx[1]}, base[2], resc[2];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j1 = tb + nt * 8 + (lane & 3) * 2 + (e & 1);
+        s[nt][e] = s[nt][e] * ((e & 1) ? kf[nt].y : kf[nt].x) - slope[e >> 1] * (float)(pos - j1);
+        if (!sees(a, pos, j1)) s[nt][e] = -INFINITY;
+        nm[e >> 1] = fmaxf(nm[e >> 1], s[nt][e]);
+      }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      nm[r] = fmaxf(nm[r], __shfl_xor_sync(0xffffffffu, nm[r], 1));
+      nm[r] = fmaxf(nm[r], __shfl_xor_sync(0xffffffffu, nm[r], 2));
+      base[r] = nm[r] == -INFINITY ? 0.0f : nm[r];
+      resc[r] = ex2(mx[r] - base[r]);
+      mx[r] = nm[r];
+      l[r] *= resc[r];
+    }
+    uint32_t pa[4];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      float v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        v[e] = ex2(s[nt][e] - base[e >> 1]);
+        l[e >> 1] += v[e];
+      }
+      pa[2 * nt] = pack_bf16(v[0], v[1]);
+      pa[2 * nt + 1] = pack_bf16(v[2], v[3]);
+    }
+#pragma unroll
+    for (int i = 0; i < HD / 8; ++i) {
+      o[i][0] *= resc[0]; o[i][1] *= resc[0];
+      o[i][2] *= resc[1]; o[i][3] *= resc[1];
+    }
+#pragma unroll
+    for (int np = 0; np < HD / 16; ++np) {
+      uint32_t b[4];
+      ldsm4_t(b, frag_b_cols(k, LD, 0, np * 16, lane));
+      mma_bf16(o[2 * np], pa, b[0], b[1]);
+      mma_bf16(o[2 * np + 1], pa, b[2], b[3]);
+    }
+    __syncwarp();
+  }
+  cp_async_wait<0>();
+  __syncthreads();     // the tiles are free: the warps' partial rows take their place
+  constexpr int ST = HD + 2;
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+    if (g + 8 * r >= nh) continue;
+    float* dst = part + (warp * 16 + g + 8 * r) * ST;
+#pragma unroll
+    for (int nt = 0; nt < HD / 8; ++nt) {
+      dst[nt * 8 + (lane & 3) * 2] = o[nt][2 * r];
+      dst[nt * 8 + (lane & 3) * 2 + 1] = o[nt][2 * r + 1];
+    }
+    if ((lane & 3) == 0) {
+      dst[HD] = mx[r];
+      dst[HD + 1] = l[r];
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nh * HD; i += 256) {
+    const int r = i / HD, d = i % HD;
+    float M = -INFINITY, acc = 0.0f, L = 0.0f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) M = fmaxf(M, part[(w * 16 + r) * ST + HD]);
+#pragma unroll
+    for (int w = 0; w < NW; ++w) {
+      const float* src = part + (w * 16 + r) * ST;
+      const float f = src[HD] == -INFINITY ? 0.0f : ex2(src[HD] - M);
+      acc += f * src[d];
+      L += f * src[HD + 1];
+    }
+    res[r * ST + d] = acc;
+    if (d == 0) {
+      res[r * ST + HD] = M;
+      res[r * ST + HD + 1] = L;
+    }
+  }
+  if (nsplit > 1) cluster.sync();
+  else __syncthreads();
+  // every CTA of the cluster finishes its share of the outputs
+  for (int i = split * 256 + threadIdx.x; i < nh * a.dim; i += nsplit * 256) {
+    const int r = i / a.dim, d = i % a.dim;
+    float M = -INFINITY, acc = 0.0f, L = 0.0f;
+    for (int s = 0; s < nsplit; ++s) M = fmaxf(M, (nsplit > 1 ? cluster.map_shared_rank(res, s) : res)[r * ST + HD]);
+    for (int s = 0; s < nsplit; ++s) {
+      const float* src = (nsplit > 1 ? cluster.map_shared_rank(res, s) : res) + r * ST;
+      const float f = src[HD] == -INFINITY ? 0.0f : ex2(src[HD] - M);
+      acc += f * src[d];
+      L += f * src[HD + 1];
+    }
+    const int h = kvh * G + h0 + r;
+    static_cast<bf16*>(a.out)[(size_t)t * a.ldo + h * a.dim + d] = __float2bfloat16_rn(acc / L * sigmoid(prow[a.g_col + h]));
+  }
+  if (nsplit > 1) cluster.sync();   // nobody leaves while its rows are being read
+}
+
+// ---- 32-bit mode ------------------------------------------------------------------------------------------------------------------
+// grid (heads, rows): four warps take the visible keys in turn, exact f32 products and exponentials
+template <int HD>
+__global__ void __launch_bounds__(128) f32_kernel(Attn a) {
+  __shared__ float sm[4][HD + 2];
+  pdl_wait();
+  pdl_trigger();
+  const int h = blockIdx.x, t = blockIdx.y, kvh = h / (a.heads / a.kv_heads);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int pos = a.pos[t];
+  if (pos >= (a.max_pages << a.pshift)) return;
+  const int* bt = a.block_table + (size_t)a.slots[t] * a.max_pages;
+  const float* pool = static_cast<const float*>(a.pool);
+  const float* qr = a.proj + (size_t)t * a.ld + a.q_col + h * a.dim;
+  float q[HD / 32], o[HD / 32], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < HD / 32; ++i) {
+    const int d = lane + 32 * i;
+    q[i] = d < a.dim ? qr[d] : 0.0f;
+    o[i] = 0.0f;
+    ss += q[i] * q[i];
+  }
+  const float rq = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+#pragma unroll
+  for (int i = 0; i < HD / 32; ++i) {
+    const int d = lane + 32 * i;
+    q[i] = d < a.dim ? q[i] * rq * a.q_norm[d] * a.k_norm[d] : 0.0f;
+  }
+  const float slope = a.slopes[h];
+  float m = -INFINITY, l = 0.0f;
+  const int lo = window_lo(a, pos), nkeep = min(a.window > 0 ? a.keep : 0, lo);
+  for (int i = warp; i < nkeep + pos + 1 - lo; i += 4) {
+    const int j = i < nkeep ? i : lo + i - nkeep;
+    const size_t row = cache_row(a, bt, kvh, j);
+    float k[HD / 32], s = 0.0f;
+#pragma unroll
+    for (int c = 0; c < HD / 32; ++c) {
+      k[c] = pool[row * HD + lane + 32 * c];
+      s = fmaf(q[c], k[c], s);
+    }
+    s = warp_sum(s) * a.krms[row] * a.scale - slope * (float)(pos - j);
+    const float nm = fmaxf(m, s), f = expf(m - nm), p = expf(s - nm);
+    m = nm;
+    l = l * f + p;
+#pragma unroll
+    for (int c = 0; c < HD / 32; ++c) o[c] = o[c] * f + p * k[c];
+  }
+#pragma unroll
+  for (int c = 0; c < HD / 32; ++c) sm[warp][lane + 32 * c] = o[c];
+  if (lane == 0) {
+    sm[warp][HD] = m;
+    sm[warp][HD + 1] = l;
+  }
+  __syncthreads();
+  float M = -INFINITY, L = 0.0f;
+  for (int w = 0; w < 4; ++w) M = fmaxf(M, sm[w][HD]);
+  for (int w = 0; w < 4; ++w) L += expf(sm[w][HD] - M) * sm[w][HD + 1];
+  const float f = sigmoid(a.proj[(size_t)t * a.ld + a.g_col + h]) / L;
+  for (int d = threadIdx.x; d < a.dim; d += 128) {
+    float acc = 0.0f;
+    for (int w = 0; w < 4; ++w) acc += expf(sm[w][HD] - M) * sm[w][d];
+    static_cast<float*>(a.out)[(size_t)t * a.ldo + h * a.dim + d] = acc * f;
+  }
+}
+
+template <int HD>
+static int run_append(const Attn& a, int first, int count, int f32, cudaStream_t stream) {
+  const dim3 grid((count + 3) / 4, a.kv_heads);
+  return f32 ? launch(append_kernel<HD, float>, grid, 128, 0, stream, 1, 0, a, first, count)
+             : launch(append_kernel<HD, bf16>, grid, 128, 0, stream, 1, 0, a, first, count);
+}
+template <int HD>
+static int run_prompt(const Attn& a, const int* entries, const int* tiles, int ntiles, cudaStream_t stream) {
+  const size_t smem = (size_t)3 * 64 * (HD + 8) * sizeof(bf16) + 128 * sizeof(float);
+  cudaFuncSetAttribute(prompt_kernel<HD>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
+  return launch(prompt_kernel<HD>, dim3(a.kv_heads, ntiles), 128, smem, stream, 1, 0, a, (const int4*)entries, (const int2*)tiles);
+}
+template <int HD>
+static int run_decode(const Attn& a, int nrows, int nsplit, cudaStream_t stream) {
+  const int mg = (a.heads / a.kv_heads + 15) / 16;
+  const size_t smem = (size_t)16 * (HD + 8) * sizeof(bf16) * (1 + 16) + (size_t)16 * (HD + 2) * sizeof(float);
+  return launch(decode_kernel<HD>, dim3(a.kv_heads * mg, nsplit, nrows), 256, smem, stream, nsplit, 1, a);
+}
+template <int HD>
+static int run_f32(const Attn& a, int T, cudaStream_t stream) {
+  return launch(f32_kernel<HD>, dim3(a.heads, T), 128, 0, stream, 1, 0, a);
+}
+
+static int padded_dim(int dim) {
+  const int sizes[] = {32, 64, 96, 128, 192, 256};
+  for (int s : sizes)
+    if (dim <= s) return s;
+  return 0;
+}
+
+static bool fill(Attn& a, const void* const* ptrs, const int* ints, const float* floats) {
+  a.proj = (const float*)ptrs[0]; a.q_norm = (const float*)ptrs[1]; a.k_norm = (const float*)ptrs[2]; a.slopes = (const float*)ptrs[3];
+  a.pos = (const int*)ptrs[4]; a.slots = (const int*)ptrs[5]; a.block_table = (const int*)ptrs[6]; a.pool = const_cast<void*>(ptrs[7]);
+  a.krms = (float*)ptrs[8]; a.out = const_cast<void*>(ptrs[9]);
+  a.ld = ints[0]; a.q_col = ints[1]; a.k_col = ints[2]; a.g_col = ints[3]; a.ldo = ints[4]; a.heads = ints[5]; a.kv_heads = ints[6];
+  a.dim = ints[7]; a.max_pages = ints[8];
+  for (a.pshift = 0; (2 << a.pshift) <= ints[9]; ++a.pshift) {} a.window = ints[10]; a.keep = ints[11];
+  a.eps = floats[0]; a.scale = floats[1];
+  return a.heads >= 1 && a.kv_heads >= 1 && a.heads % a.kv_heads == 0 && a.heads / a.kv_heads <= 64 && a.dim >= 1 && padded_dim(a.dim) > 0 &&
+         a.pshift >= 4 && (1 << a.pshift) == ints[9] && a.keep >= 0;
+}
+
+#define BONSAI_BY_DIM(CALL)                                  \
+  switch (padded_dim(a.dim)) {                               \
+    case 32: { constexpr int HD = 32; return CALL; }         \
+    case 64: { constexpr int HD = 64; return CALL; }         \
+    case 96: { constexpr int HD = 96; return CALL; }         \
+    case 128: { constexpr int HD = 128; return CALL; }       \
+    case 192: { constexpr int HD = 192; return CALL; }       \
+    case 256: { constexpr int HD = 256; return CALL; }       \
+    default: return BONSAI_CUDA_BAD_ARG;                     \
+  }
+
+}  // namespace lay
+}  // namespace bonsai
+
+extern "C" {
+
+// elements of a cache row for a head size (0: not supported)
+int bonsai_lay_attn_row(int dim) { return dim < 1 ? 0 : bonsai::lay::padded_dim(dim); }
+
+// Arguments of all launches: ptrs = {proj, q_norm, k_norm, slopes, pos, slots, block_table, pool, krms, out}, ints = {ld,
+// q_col, k_col, g_col, ldo, heads, kv_heads, dim, max_pages, page_size, window, keep}, floats = {eps, scale}.
+
+// Writes the keys of rows first .. first + count - 1.
+int bonsai_lay_attn_append(const void* const* ptrs, const int* ints, const float* floats, int first, int count, int f32, cudaStream_t stream) {
+  using namespace bonsai::lay;
+  Attn a;
+  if (!fill(a, ptrs, ints, floats) || count < 1 || first < 0) return BONSAI_CUDA_BAD_ARG;
+  BONSAI_BY_DIM((run_append<HD>(a, first, count, f32, stream)))
+}
+
+// entries int4 [..] {first row, tokens, slot, first position}, tiles int2 [ntiles] {entry, first token}; a tile has
+// 64 / (heads / kv_heads) tokens.  The rows' keys must have been appended.
+int bonsai_lay_attn_prompt(const void* const* ptrs, const int* ints, const float* floats, const int* entries, const int* tiles, int ntiles,
+                           cudaStream_t stream) {
+  using namespace bonsai::lay;
+  Attn a;
+  if (!fill(a, ptrs, ints, floats) || ntiles < 1 || ntiles > 65535) return BONSAI_CUDA_BAD_ARG;
+  BONSAI_BY_DIM((run_prompt<HD>(a, entries, tiles, ntiles, stream)))
+}
+
+// One token in each of the rows 0 .. nrows - 1, its key appended here.
+int bonsai_lay_attn_decode(const void* const* ptrs, const int* ints, const float* floats, int nrows, int nsplit, cudaStream_t stream) {
+  using namespace bonsai::lay;
+  Attn a;
+  if (!fill(a, ptrs, ints, floats) || nrows < 1 || nrows > 65535 || (nsplit != 1 && nsplit != 2 && nsplit != 4 && nsplit != 8)) return BONSAI_CUDA_BAD_ARG;
+  BONSAI_BY_DIM((run_decode<HD>(a, nrows, nsplit, stream)))
+}
+
+// All T rows, 32-bit throughout; the rows' keys must have been appended.
+int bonsai_lay_attn_f32(const void* const* ptrs, const int* ints, const float* floats, int T, cudaStream_t stream) {
+  using namespace bonsai::lay;
+  Attn a;
+  if (!fill(a, ptrs, ints, floats) || T < 1 || T > 65535) return BONSAI_CUDA_BAD_ARG;
+  BONSAI_BY_DIM((run_f32<HD>(a, T, stream)))
+}
+
+}  // extern "C"

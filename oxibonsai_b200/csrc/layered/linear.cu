@@ -1,0 +1,178 @@
+// Projections with dense bf16 weights: out[t][n] = sum_k x[t][k] W[n][k].
+//
+// `few_rows_kernel` serves decode batches and short portions (up to 32 rows): the weights are streamed once, a warp's lane
+// loads 16 contiguous bytes of a weight row and uses them directly as `mma.sync.m16n8k16` A registers.  That is the
+// fragment layout up to a permutation of k inside every 32 inputs, and the activations are loaded through the same
+// permutation (16 contiguous bytes of an activation row as the B registers), so neither operand passes through shared
+// memory.  The eight warps of a CTA split K and meet in shared memory once.  More rows go to the tcgen05 GEMM
+// (cuda/bitgemm_prefill.cu, dense bf16 operands).
+//
+// `f32_kernel` is the 32-bit mode: f32 activations, the same bf16 weights (exact in f32), f32 FMA throughout.
+//
+// Epilogues: 0 = f32 store, 1 = clamped gated unit over interleaved gate / up rows:
+//   g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(alpha g) * (u + up_offset).
+#include "layered/layered.cuh"
+
+namespace bonsai {
+namespace lay {
+
+struct Glu {
+  float limit, alpha, up_offset;
+};
+
+__device__ __forceinline__ float glu(const Glu& a, float g, float u) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return g * sigmoid(a.alpha * g) * (u + a.up_offset);
+}
+
+constexpr int kWarps = 8;
+
+template <int NT>   // 8-row groups of activations
+__global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __restrict__ W, int n, int kp, const bf16* x, int ldx, int T,
+                                                              float* out, bf16* out16, int ldo, int epi, Glu act) {
+  constexpr int LD = 8 * NT + 1;
+  __shared__ float red[kWarps][16][LD];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t4 = lane & 3;
+  const int row0 = blockIdx.x * 16;
+  const bf16* w0 = W + (size_t)min(row0 + g, n - 1) * kp + 8 * t4;
+  const bf16* w1 = W + (size_t)min(row0 + g + 8, n - 1) * kp + 8 * t4;
+  const int chunks = kp >> 7;   // 128 inputs each
+  uint4 a[4], b[4];
+  auto load_w = [&](int c) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      a[i] = __ldcs(reinterpret_cast<const uint4*>(w0 + c * 128 + i * 32));
+      b[i] = __ldcs(reinterpret_cast<const uint4*>(w1 + c * 128 + i * 32));
+    }
+  };
+  if (warp < chunks) load_w(warp);   // weights depend on no earlier kernel
+  pdl_wait();
+  pdl_trigger();
+  const bf16* xr[NT];
+#pragma unroll
+  for (int j = 0; j < NT; ++j) xr[j] = x + (size_t)min(8 * j + g, T - 1) * ldx + 8 * t4;
+  float acc[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
+  for (int c = warp; c < chunks; c += kWarps) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const uint32_t lo[4] = {a[i].x, b[i].x, a[i].y, b[i].y}, hi[4] = {a[i].z, b[i].z, a[i].w, b[i].w};
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const uint4 v = *reinterpret_cast<const uint4*>(xr[j] + c * 128 + i * 32);
+        mma_bf16(acc[j], lo, v.x, v.y);
+        mma_bf16(acc[j], hi, v.z, v.w);
+      }
+    }
+    if (c + kWarps < chunks) load_w(c + kWarps);
+  }
+#pragma unroll
+  for (int j = 0; j < NT; ++j) {
+    red[warp][g][8 * j + 2 * t4] = acc[j][0];
+    red[warp][g][8 * j + 2 * t4 + 1] = acc[j][1];
+    red[warp][g + 8][8 * j + 2 * t4] = acc[j][2];
+    red[warp][g + 8][8 * j + 2 * t4 + 1] = acc[j][3];
+  }
+  __syncthreads();
+  if (epi == 0) {
+    for (int i = threadIdx.x; i < 16 * T; i += kWarps * 32) {
+      const int r = i & 15, t = i >> 4;
+      float v = 0.0f;
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) v += red[w][r][t];
+      if (row0 + r < n) out[(size_t)t * ldo + row0 + r] = v;
+    }
+  } else {
+    for (int i = threadIdx.x; i < 8 * T; i += kWarps * 32) {
+      const int r = i & 7, t = i >> 3;
+      float gv = 0.0f, uv = 0.0f;
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) {
+        gv += red[w][2 * r][t];
+        uv += red[w][2 * r + 1][t];
+      }
+      if (row0 + 2 * r + 1 < n) out16[(size_t)t * ldo + (row0 >> 1) + r] = __float2bfloat16_rn(glu(act, gv, uv));
+    }
+  }
+}
+
+// 64 weight rows x 64 activation rows per CTA, 256 threads with 4 x 4 outputs each
+__global__ void __launch_bounds__(256) f32_kernel(const bf16* __restrict__ W, int n, int k, int kp, const float* x, int ldx, int T,
+                                                  float* out, int ldo, int epi, Glu act) {
+  __shared__ float sw[16][68], sx[16][68];
+  pdl_wait();
+  pdl_trigger();
+  const int n0 = blockIdx.x * 64, t0 = blockIdx.y * 64;
+  const int tn = threadIdx.x & 15, tt = threadIdx.x >> 4;
+  float acc[4][4] = {};   // [activation row][weight row]
+  for (int k0 = 0; k0 < k; k0 += 16) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int idx = threadIdx.x + i * 256, r = idx >> 4, c = idx & 15;
+      const bool kin = k0 + c < k;
+      sw[c][r] = kin && n0 + r < n ? __bfloat162float(W[(size_t)(n0 + r) * kp + k0 + c]) : 0.0f;
+      sx[c][r] = kin && t0 + r < T ? x[(size_t)(t0 + r) * ldx + k0 + c] : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < 16; ++c) {
+      float wv[4], xv[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        wv[i] = sw[c][tn * 4 + i];
+        xv[i] = sx[c][tt * 4 + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xv[i], wv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = t0 + tt * 4 + i;
+    if (t >= T) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = n0 + tn * 4 + j;
+      if (epi == 0) {
+        if (r < n) out[(size_t)t * ldo + r] = acc[i][j];
+      } else if ((j & 1) == 0 && r + 1 < n) {
+        out[(size_t)t * ldo + (r >> 1)] = glu(act, acc[i][j], acc[i][j + 1]);
+      }
+    }
+  }
+}
+
+}  // namespace lay
+}  // namespace bonsai
+
+extern "C" {
+
+// W bf16 [n][kp] (kp a multiple of 128, columns past the layer's width zero), x bf16 [T][ldx] (ldx >= kp, finite in the
+// padding), T <= 32.  epi 0: out f32 [T][ldo]; epi 1: out16 bf16 [T][ldo] of n / 2 columns.
+int bonsai_lay_linear_few(const void* W, int n, int kp, const void* x, int ldx, int T, float* out, void* out16, int ldo, int epi, float limit,
+                          float alpha, float up_offset, cudaStream_t stream) {
+  using namespace bonsai::lay;
+  if (n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || T < 1 || T > 32 || epi < 0 || epi > 1) return BONSAI_CUDA_BAD_ARG;
+  if ((epi == 0 && out == nullptr) || (epi == 1 && (out16 == nullptr || n % 2 != 0))) return BONSAI_CUDA_BAD_ARG;
+  const Glu act{limit, alpha, up_offset};
+  const dim3 grid((n + 15) / 16);
+#define BONSAI_FEW(NT) \
+  launch(few_rows_kernel<NT>, grid, kWarps * 32, 0, stream, 1, 0, (const bf16*)W, n, kp, (const bf16*)x, ldx, T, out, (bf16*)out16, ldo, epi, act)
+  return T <= 8 ? BONSAI_FEW(1) : (T <= 16 ? BONSAI_FEW(2) : BONSAI_FEW(4));
+#undef BONSAI_FEW
+}
+
+int bonsai_lay_linear_f32(const void* W, int n, int k, int kp, const float* x, int ldx, int T, float* out, int ldo, int epi, float limit, float alpha,
+                          float up_offset, cudaStream_t stream) {
+  using namespace bonsai::lay;
+  if (n < 1 || k < 1 || kp < k || ldx < k || T < 1 || out == nullptr || epi < 0 || epi > 1 || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
+  return launch(f32_kernel, dim3((n + 63) / 64, (T + 63) / 64), 256, 0, stream, 1, 0, (const bf16*)W, n, k, kp, x, ldx, T, out, ldo, epi,
+                Glu{limit, alpha, up_offset});
+}
+
+}  // extern "C"

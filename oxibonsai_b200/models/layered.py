@@ -1,0 +1,411 @@
+"""Decoders described layer by layer (``layered_config``): weights, mixers and the step runner.
+
+A step is a batch of rows (tokens).  Rows of single tokens (decode) come first, portions of prompts follow, each portion
+contiguous; every projection runs over all rows, a mixer runs its single-token kernel over the first group and its prompt
+kernel over the second.  A row carries its position and its slot; the slot's block-table row names the pages of its sequence
+and the state table its recurrent state row, so which pages, rows and companions a token has does not enter its arithmetic.
+
+Two modes: bf16 (tensor-core projections and attention, f32 residual stream, norms, scores, gates and recurrent state) and
+the exact mode, f32 throughout.  Decode steps of slots 0 .. n-1 are captured into CUDA graphs; mixed batches are issued
+eagerly with the same kernels.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from pathlib import Path
+from typing import Sequence
+
+import numpy as np
+import torch
+
+from ..ops import cuda_ops as K
+from ..ops import layered_ops as L
+from ..ops import nvtx
+from .layered_config import AttentionSpec, LayeredConfig, MlstmSpec
+from .paged import SharedRowCache, StatePool
+from .rope_scaling import geometric_slopes
+from .slot_state import SlotState
+
+
+def _tensor(t) -> torch.Tensor:
+    """A checkpoint tensor as a host torch tensor (bf16 kept, everything else widened to f32)."""
+    if t.dtype == "BF16":
+        return torch.from_numpy(np.array(np.frombuffer(t.data, dtype="<i2"))).view(torch.bfloat16).reshape(t.shape)
+    return torch.from_numpy(np.array(t.to_f32()))
+
+
+@dataclass
+class MlpWeights:
+    norm: torch.Tensor
+    gate_up: L.DenseWeight
+    down: L.DenseWeight
+
+
+@dataclass
+class LayerWeights:
+    norm: torch.Tensor
+    proj: L.DenseWeight              # every projection that reads the mixer's input, one matrix
+    out: L.DenseWeight
+    vectors: dict[str, torch.Tensor]
+    mlp: MlpWeights | None
+
+
+class LayeredWeights:
+    """Device-resident weights of a model directory (``model.safetensors``)."""
+
+    def __init__(self, cfg: LayeredConfig, tensors: dict[str, torch.Tensor], device):
+        shapes = cfg.tensor_shapes()
+        for n, s in shapes.items():
+            if n not in tensors:
+                raise ValueError(f"checkpoint has no tensor {n}")
+            if tuple(tensors[n].shape) != s:
+                raise ValueError(f"tensor {n} is {list(tensors[n].shape)}, expected {list(s)}")
+        self.cfg, self.device = cfg, torch.device(device)
+        m = lambda n: tensors[n].to(torch.bfloat16)
+        v = lambda n: tensors[n].float().to(self.device)
+        self.embed = L.DenseWeight([m("embed")], self.device)      # also the output head
+        self.final_norm = v("final.norm")
+        self.layers: list[LayerWeights] = []
+        for i, spec in enumerate(cfg.layer_specs):
+            p, x = f"l{i}.", f"l{i}.mix."
+            if spec.mixer.kind == "attention":
+                proj, vec = ["q", "k", "g"], ["q.norm", "k.norm"]
+            else:
+                proj, vec = ["q", "k", "v", "g", "i", "f"], ["i.b", "f.b", "norm"]
+            mlp = None
+            if spec.mlp is not None:
+                mlp = MlpWeights(v(p + "norm2"), L.DenseWeight([m(p + "mlp.gate"), m(p + "mlp.up")], self.device, interleave=True),
+                                 L.DenseWeight([m(p + "mlp.down")], self.device))
+            self.layers.append(LayerWeights(v(p + "norm1"), L.DenseWeight([m(x + n) for n in proj], self.device),
+                                            L.DenseWeight([m(x + "o")], self.device), {n: v(x + n) for n in vec}, mlp))
+        torch.cuda.synchronize(self.device)
+
+    @classmethod
+    def from_dir(cls, cfg: LayeredConfig, path, device) -> "LayeredWeights":
+        from ..convert import read_safetensors
+        return cls(cfg, {t.name: _tensor(t) for t in read_safetensors(str(Path(path) / "model.safetensors"))}, device)
+
+    @property
+    def packed_bytes(self) -> int:
+        """Bytes a decode step must stream."""
+        n = self.embed.nbytes
+        for l in self.layers:
+            n += l.proj.nbytes + l.out.nbytes + (0 if l.mlp is None else l.mlp.gate_up.nbytes + l.mlp.down.nbytes)
+        return n
+
+
+def new_row_cache(cfg: LayeredConfig, num_pages: int, page_size: int, exact: bool, device) -> SharedRowCache:
+    layers = {i: (cfg.layer_specs[i].mixer.kv_heads, L.lib().bonsai_lay_attn_row(cfg.layer_specs[i].mixer.dim)) for i in cfg.attention_layers}
+    return SharedRowCache(layers, num_pages, page_size, K.KV_F32 if exact else K.KV_BF16, torch.float32 if exact else torch.bfloat16, device)
+
+
+def new_state_pool(cfg: LayeredConfig, num_rows: int, device) -> StatePool:
+    layers = {}
+    for i in cfg.recurrent_layers:
+        m: MlstmSpec = cfg.layer_specs[i].mixer
+        d, e = L.lib().bonsai_lay_mlstm_dim(m.dim), L.lib().bonsai_lay_mlstm_vdim(m.vdim)
+        layers[i] = {"S": (m.heads, d, e), "n": (m.heads, e // 64, d), "m": (m.heads, e // 64)}
+    return StatePool(layers, num_rows, device)
+
+
+@dataclass
+class Rows:
+    """Row metadata the kernels read: one set for decode steps (row = slot), one that mixed batches fill."""
+    tokens: torch.Tensor
+    positions: torch.Tensor
+    slots: torch.Tensor
+
+
+@dataclass
+class StepShape:
+    """How a step's rows split: ``singles`` single-token rows, then ``portions`` (device address of the int4 list and of the
+    query tiles per tokens-per-tile)."""
+    rows: int
+    singles: int
+    portions: int = 0
+    entries: int = 0
+    tiles: dict[int, tuple[int, int]] | None = None      # tokens per tile -> (device address, tiles)
+
+
+class AttentionMixer:
+    def __init__(self, r: "LayeredRunner", index: int, spec: AttentionSpec):
+        self.r, self.spec, self.w, cfg = r, spec, r.w.layers[index], r.cfg
+        self.tile = 64 // spec.group
+        self.slopes = geometric_slopes(spec.heads, spec.slope_exponent).to(r.device)
+        self.out = r.act_buffer(spec.out_width)
+        q, k, g = self.w.proj.columns
+        ints = [r.proj.stride(0), q, k, g, self.out.stride(0), spec.heads, spec.kv_heads, spec.dim, r.max_pages, r.kv.page_size, spec.window,
+                spec.keep_first]
+        cache, factors = r.kv.rows[index], r.kv.factors[index]
+        self.call = {id(rows): L.MixerCall([r.proj, self.w.vectors["q.norm"], self.w.vectors["k.norm"], self.slopes, rows.positions, rows.slots,
+                                            r.block_table, cache, factors, self.out], ints, [cfg.eps, spec.scale]) for rows in (r.slot_rows, r.batch_rows)}
+
+    def splits(self, batch: int) -> int:
+        """KV splits of one row's decode attention: about a CTA per SM, and no more than there are 16-token tiles per warp."""
+        s = self.spec
+        seen = self.r.max_seq if s.window <= 0 else min(self.r.max_seq, s.window + s.keep_first + 32)
+        n, ctas = 1, batch * s.kv_heads * (-(-s.group // 16))
+        while n < 8 and ctas * n * 2 <= 160 and n * 2 * 128 <= seen + 127:
+            n *= 2
+        return n
+
+    def __call__(self, rows: Rows, st: StepShape, stream: int) -> torch.Tensor:
+        lib, a = L.lib(), self.call[id(rows)].args
+        if self.r.exact:
+            K.check(lib.bonsai_lay_attn_append(*a, 0, st.rows, 1, stream), "attn_append")
+            K.check(lib.bonsai_lay_attn_f32(*a, st.rows, stream), "attn_f32")
+            return self.out
+        if st.singles:
+            K.check(lib.bonsai_lay_attn_decode(*a, st.singles, self.splits(st.singles), stream), "attn_decode")
+        if st.portions:
+            tiles, n = st.tiles[self.tile]
+            K.check(lib.bonsai_lay_attn_append(*a, st.singles, st.rows - st.singles, 0, stream), "attn_append")
+            K.check(lib.bonsai_lay_attn_prompt(*a, st.entries, tiles, n, stream), "attn_prompt")
+        return self.out
+
+    def launches(self) -> int:
+        return 2 if self.r.exact else 1
+
+
+class MlstmMixer:
+    def __init__(self, r: "LayeredRunner", index: int, spec: MlstmSpec):
+        self.r, self.spec, self.w, cfg = r, spec, r.w.layers[index], r.cfg
+        self.out = r.act_buffer(spec.out_width)
+        q, k, v, self.g_col, i, f = self.w.proj.columns
+        s = r.states.tensors[index]
+        self.chunked = not r.exact and spec.dim <= L.lib().bonsai_lay_mlstm_chunk_dim()
+        self.fused = spec.vdim <= L.lib().bonsai_lay_mlstm_fused_vdim()
+        floats = [spec.gate_cap, cfg.eps, spec.den_eps, spec.dim ** -0.5]
+
+        def call(rows, out):
+            return L.MixerCall([r.proj, self.w.vectors["i.b"], self.w.vectors["f.b"], self.w.vectors["norm"], s["S"], s["n"], s["m"], rows.positions,
+                                rows.slots, r.state_table, out],
+                               [r.proj.stride(0), q, k, v, self.g_col, i, f, out.stride(0), spec.heads, spec.dim, spec.vdim], floats)
+        # o f32 for the gated head norm, and the finished activations of the fused single-token step
+        self.raw = {id(rows): call(rows, r.head_out) for rows in (r.slot_rows, r.batch_rows)}
+        self.done = {id(rows): call(rows, self.out) for rows in (r.slot_rows, r.batch_rows)}
+
+    def _finish(self, row0: int, count: int) -> None:
+        s = self.spec
+        L.gated_head_norm(self.r.head_out, row0, self.r.proj, self.g_col, self.w.vectors["norm"], self.r.cfg.eps, count, s.heads, s.vdim, self.out)
+
+    def __call__(self, rows: Rows, st: StepShape, stream: int) -> torch.Tensor:
+        lib = L.lib()
+        if st.singles and self.fused:
+            K.check(lib.bonsai_lay_mlstm_step(*self.done[id(rows)].args, None, st.singles, 2 if self.r.exact else 1, stream), "mlstm_step")
+        elif st.singles:
+            K.check(lib.bonsai_lay_mlstm_step(*self.raw[id(rows)].args, None, st.singles, 3, stream), "mlstm_step")
+            self._finish(0, st.singles)
+        if st.portions:
+            a = self.raw[id(rows)].args
+            if self.chunked:
+                K.check(lib.bonsai_lay_mlstm_chunk(*a, st.entries, st.portions, stream), "mlstm_chunk")
+            else:
+                K.check(lib.bonsai_lay_mlstm_step(*a, st.entries, st.portions, 0, stream), "mlstm_step")
+            self._finish(st.singles, st.rows - st.singles)
+        return self.out
+
+    def launches(self) -> int:
+        return 1 if self.fused else 2
+
+
+MIXERS = {"attention": AttentionMixer, "mlstm": MlstmMixer}
+
+
+class LayeredRunner(SlotState):
+    """Owns the activation buffers, the caches and the captured decode steps of a layer-list decoder.  Same surface as
+    ``Qwen3Runner`` where the engine and the scheduler use it."""
+
+    sample_fn = staticmethod(L.sample)
+
+    def __init__(self, weights: LayeredWeights, kv: SharedRowCache, states: StatePool, max_batch: int, max_seq: int, exact: bool = False,
+                 prefill_chunk: int = 4096):
+        self.w, self.kv, self.states, self.exact = weights, kv, states, exact
+        self.cfg, self.device = weights.cfg, weights.device
+        self.max_batch, self.max_seq = max_batch, max_seq
+        self.max_pages = -(-max_seq // kv.page_size)
+        self.capacity = max(int(prefill_chunk), 64, max_batch)         # rows of a step
+        self.prefill_capacity = self.capacity
+        cfg, dev, cap = self.cfg, self.device, self.capacity
+        f32, i32 = dict(dtype=torch.float32, device=dev), dict(dtype=torch.int32, device=dev)
+        self.init_slots(max_batch, self.max_pages, cfg.vocab, dev)
+        self.logits = torch.zeros((max_batch, cfg.vocab), **f32)
+        self.state_table = torch.zeros(max_batch, **i32)
+        self._state_row: dict[int, int] = {}
+        self.kv_pools = {kv.kvt: kv}
+        self.slot_formats = [kv.kvt] * max_batch
+        self.scratch = L.GemmScratch(dev, self.status)
+        # activations; the padding columns of the bf16 buffers stay zero for the projections that read them
+        self._acts: dict[int, torch.Tensor] = {}
+        self.x = torch.zeros((cap, cfg.width), **f32)
+        self.x16 = None if exact else self.act_buffer(cfg.width, shared=False)
+        self.normed = self.act_buffer(cfg.width, shared=False)
+        self.y = torch.zeros((cap, L.round_up(cfg.width, 4)), **f32)
+        self.proj = torch.zeros((cap, max(L.round_up(l.proj.n, 4) for l in weights.layers)), **f32)
+        widths = [cfg.layer_specs[i].mixer.out_width for i in cfg.recurrent_layers]
+        self.head_out = torch.zeros((cap, L.round_up(max(widths, default=4), 4)), **f32)
+        # row metadata: decode steps use the slot tensors as they are; a mixed batch uploads [tokens | positions | slots | lists]
+        self.slot_rows = Rows(self.tokens, self.positions, torch.arange(max_batch, **i32))
+        self._tile_sizes = sorted({64 // cfg.layer_specs[i].mixer.group for i in cfg.attention_layers})
+        self._meta = torch.zeros(3 * cap + 4 * cap + 2 * cap * len(self._tile_sizes) + cap + 16, **i32)
+        self.batch_rows = Rows(*(self._meta[i * cap:(i + 1) * cap] for i in range(3)))
+        self._host = [torch.zeros(self._meta.numel(), dtype=torch.int32).pin_memory() for _ in range(2)]
+        self._host_free = [torch.cuda.Event() for _ in range(2)]
+        self._turn = 0
+        self.mixers = [MIXERS[s.mixer.kind](self, i, s.mixer) for i, s in enumerate(cfg.layer_specs)]
+        self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
+
+    def act_buffer(self, width: int, shared: bool = True) -> torch.Tensor:
+        """Input buffer of a projection with ``width`` inputs: f32 in the exact mode, else bf16 padded to the tensor-core width.
+        One per width, so that the padding of a narrower layer never holds another layer's values."""
+        if shared and width in self._acts:
+            return self._acts[width]
+        ld = L.round_up(width, 4 if self.exact else L.K_ALIGN)
+        t = torch.zeros((self.capacity, ld), dtype=torch.float32 if self.exact else torch.bfloat16, device=self.device)
+        if shared:
+            self._acts[width] = t
+        return t
+
+    # ---- slots ------------------------------------------------------------------------------------------------------------------
+    def bind_state(self, slot: int) -> None:
+        if self.cfg.recurrent_layers and slot not in self._state_row:
+            row = self._state_row[slot] = self.states.alloc()
+            self.state_table[slot] = row
+
+    def release_state(self, slot: int) -> None:
+        row = self._state_row.pop(slot, None)
+        if row is not None:
+            self.states.release(row)
+
+    def move_state(self, src: int, dst: int) -> None:
+        self.release_state(dst)
+        if src in self._state_row:
+            self._state_row[dst] = self._state_row.pop(src)
+            self.state_table[dst].copy_(self.state_table[src], non_blocking=True)
+
+    def set_slot_format(self, slot: int, kvt: int) -> None:
+        if kvt != self.kv.kvt:
+            raise ValueError("the layer-list decoders have one cache format per engine")
+
+    # ---- one step ------------------------------------------------------------------------------------------------------------------
+    def _layers(self, rows: Rows, st: StepShape) -> None:
+        cfg, T, s = self.cfg, st.rows, K.stream()
+        x, x16 = self.x, self.x16
+        h = x if self.exact else x16
+        L.embed(self.w.embed.data, rows.tokens, T, cfg.width, x, x16)
+        for spec, w, mixer in zip(cfg.layer_specs, self.w.layers, self.mixers):
+            L.linear(w.proj, h, T, self.proj, self.scratch)
+            L.linear(w.out, mixer(rows, st, s), T, self.y, self.scratch)
+            L.norm_add(x, self.y, w.norm, cfg.eps, T, x16)
+            if spec.mlp is not None:
+                act = self.act_buffer(spec.mlp.ff)
+                L.linear(w.mlp.gate_up, h, T, act, self.scratch, (spec.mlp.limit, spec.mlp.alpha, spec.mlp.offset))
+                L.linear(w.mlp.down, act, T, self.y, self.scratch)
+                L.norm_add(x, self.y, w.mlp.norm, cfg.eps, T, x16)
+
+    def _head(self, row_list: int | None, count: int, out: torch.Tensor) -> None:
+        """Logits of ``count`` rows (device address of their indices, None = the first ones) into ``out`` [count, vocab]."""
+        L.norm_rows(self.x, row_list, count, self.w.final_norm, self.cfg.eps, self.normed)
+        L.linear(self.w.embed, self.normed, count, out, self.scratch)
+
+    def step_eager(self, batch: int, sample: bool = True, lm_head: bool = True, masked: bool = False) -> None:
+        """One token for each of the slots 0 .. batch-1 (tokens and positions are read from the slot tensors)."""
+        self._layers(self.slot_rows, StepShape(batch, batch))
+        if lm_head:
+            self._head(None, batch, self.logits)
+        if sample:
+            self.sample_rows(0, batch, masked, advance=True)
+
+    def step(self, batch: int, sample: bool = True, masked: bool = False) -> None:
+        """:meth:`step_eager` replayed from a CUDA graph captured at its first call."""
+        key = (batch, sample, masked)
+        g = self._graphs.get(key)
+        if g is None:
+            for mlp in (s.mlp for s in self.cfg.layer_specs if s.mlp is not None):
+                self.act_buffer(mlp.ff)                        # allocated outside the capture
+            g = self._graphs[key] = K.capture_graph(self.device, lambda: self.step_eager(batch, sample, masked=masked))
+        mark = nvtx.push(f"decode_step[batch={batch}]")
+        g.replay()
+        nvtx.pop(mark)
+
+    def run_batch(self, entries: Sequence[tuple[int, Sequence[int], int]], want: Sequence[Sequence[int]], device_tokens: bool = False) -> torch.Tensor:
+        """Runs portions of several sequences as one batch.  ``entries``: (slot, tokens, first position) each, the slots
+        distinct; ``want``: per entry the places among its tokens whose logits are asked for.  Returns them as f32
+        [wanted, vocab], in the order of the entries and of their places.  ``device_tokens``: single-token entries take their
+        token from ``tokens[slot]`` on the device (the host's value is ignored)."""
+        T = sum(len(e[1]) for e in entries)
+        if T == 0 or T > self.capacity:
+            raise ValueError(f"a step takes 1 to {self.capacity} tokens, got {T}")
+        if len({e[0] for e in entries}) != len(entries):
+            raise ValueError("a step takes one entry per slot")
+        order = sorted(range(len(entries)), key=lambda i: (len(entries[i][1]) != 1, i))     # single tokens first
+        cap = self.capacity
+        turn = self._turn = (self._turn + 1) % 2
+        self._host_free[turn].synchronize()                    # the copy that read this buffer has finished
+        host = self._host[turn].numpy()
+        lists, row, row0 = [], 0, [0] * len(entries)
+        for i in order:
+            slot, toks, pos0 = entries[i]
+            n = len(toks)
+            t = np.asarray(toks, dtype=np.int64)
+            if n == 0 or t.min() < 0 or t.max() >= self.cfg.vocab:
+                raise ValueError(f"entry of slot {slot}: needs tokens in [0, {self.cfg.vocab})")
+            if not 0 <= slot < self.max_batch or pos0 < 0 or pos0 + n > self.max_seq:
+                raise ValueError(f"entry of slot {slot}: {n} tokens at position {pos0} do not fit {self.max_batch} slots of {self.max_seq} tokens")
+            host[row:row + n] = t
+            host[cap + row:cap + row + n] = np.arange(pos0, pos0 + n)
+            host[2 * cap + row:2 * cap + row + n] = slot
+            if n > 1:
+                lists.append((row, n, slot, pos0))
+            row0[i] = row
+            row += n
+        singles = sum(len(e[1]) == 1 for e in entries)
+        end = -(-3 * cap // 4) * 4
+        put = lambda a: (end, end + a.size)
+        base = self._meta.data_ptr()
+        st = StepShape(T, singles, len(lists), base + 4 * end, {})
+        if lists:
+            a = np.asarray(lists, dtype=np.int32).reshape(-1)
+            lo, hi = put(a)
+            host[lo:hi] = a
+            end = hi
+            for size in self._tile_sizes:
+                a = np.asarray([(e, t) for e, (_, n, _, _) in enumerate(lists) for t in range(0, n, size)], dtype=np.int32).reshape(-1)
+                lo, hi = put(a)
+                host[lo:hi] = a
+                st.tiles[size] = (base + 4 * lo, a.size // 2)
+                end = hi
+        wanted = np.asarray([row0[i] + p for i, ps in enumerate(want) for p in ps], dtype=np.int32)
+        host[end:end + wanted.size] = wanted
+        rows_at = base + 4 * end
+        end += wanted.size
+        self._meta[:end].copy_(self._host[turn][:end], non_blocking=True)
+        self._host_free[turn].record()
+        if device_tokens and singles:
+            idx = self.batch_rows.slots[:singles].long()
+            self.batch_rows.tokens[:singles].copy_(torch.index_select(self.tokens, 0, idx))
+        mark = nvtx.push(f"batch[rows={T},singles={singles},portions={len(lists)}]")
+        self._layers(self.batch_rows, st)
+        out = torch.empty((wanted.size, self.cfg.vocab), dtype=torch.float32, device=self.device)
+        if wanted.size:
+            self._head(rows_at, wanted.size, out)
+        nvtx.pop(mark)
+        return out
+
+    def prefill(self, tokens: Sequence[int], slot: int, pos0: int = 0, chunk: int = 4096) -> None:
+        """Runs prompt ``tokens`` of the sequence in ``slot`` from position ``pos0`` on; leaves the logits of the last one in
+        ``logits[slot]``."""
+        n, chunk = len(tokens), max(1, min(chunk, self.capacity))
+        for done in range(0, n, chunk):
+            part = tokens[done:done + chunk]
+            last = done + len(part) == n
+            out = self.run_batch([(slot, part, pos0 + done)], [[len(part) - 1] if last else []])
+            if last:
+                self.logits[slot].copy_(out[0], non_blocking=True)
+
+    def kernel_launches(self, batch: int, sample: bool = True) -> int:
+        """Launches of one decode step (each is one of this library's kernels)."""
+        n = 1 + 2 + int(sample)
+        for spec, mixer in zip(self.cfg.layer_specs, self.mixers):
+            n += 3 + mixer.launches() + (3 if spec.mlp is not None else 0)
+        return n

@@ -24,6 +24,8 @@ from ..core.gguf import GgufFile, Qwen3Config
 from ..core.oracle import rope_table
 from ..ops import cuda_ops as K
 from ..ops import nvtx
+from .paged import PagePool
+from .slot_state import SlotState
 
 _QUANT_TYPES = (G.TQ2_0_G128, G.Q1_0_G128)
 
@@ -229,7 +231,7 @@ class Qwen3Weights:
         return n + self.lm_head.numel() * 2
 
 
-class PagedKvCache:
+class PagedKvCache(PagePool):
     """Page pool shared by all sequences of a rank; one K and one V pool per layer.
 
     Reference: ``PagedKvCache`` / ``BlockPool`` / ``BlockTable`` (crates/oxibonsai-model/src/paged_kv_cache.rs:33-557),
@@ -238,7 +240,8 @@ class PagedKvCache:
     """
 
     def __init__(self, cfg: Qwen3Config, kv_heads_local: int, num_pages: int, page_size: int, kvt: int, device):
-        self.kvt, self.page_size, self.num_pages = kvt, page_size, num_pages
+        super().__init__(num_pages, page_size)
+        self.kvt = kvt
         hd = cfg.head_dim
         row = {K.KV_F32: hd, K.KV_F16: hd, K.KV_Q8: hd, K.KV_Q4: hd // 2}[kvt]
         dt = K.KV_DTYPES[kvt]
@@ -250,34 +253,6 @@ class PagedKvCache:
             self.v_scale = torch.zeros(shape[:-1], dtype=torch.float32, device=device)
         else:
             self.k_scale = self.v_scale = None
-        self.free_pages = list(range(num_pages - 1, -1, -1))
-        self.refcount = [0] * num_pages        # pages may be shared between sequences and the prefix cache
-        self.on_exhausted = None               # optional callback(n_missing) that may free pages (prefix-cache eviction)
-
-    def alloc(self, n: int) -> list[int]:
-        if n > len(self.free_pages) and self.on_exhausted is not None:
-            self.on_exhausted(n - len(self.free_pages))
-        if n > len(self.free_pages):
-            raise MemoryError(f"KV cache exhausted: need {n} pages, {len(self.free_pages)} free")
-        pages = [self.free_pages.pop() for _ in range(n)]
-        for p in pages:
-            self.refcount[p] = 1
-        return pages
-
-    def retain(self, pages: list[int]) -> None:
-        for p in pages:
-            self.refcount[p] += 1
-
-    def release(self, pages: list[int]) -> None:
-        for p in reversed(pages):
-            self.refcount[p] -= 1
-            if self.refcount[p] <= 0:
-                self.refcount[p] = 0
-                self.free_pages.append(p)
-
-    @property
-    def utilization(self) -> float:
-        return 1.0 - len(self.free_pages) / max(1, self.num_pages)
 
     @property
     def nbytes(self) -> int:
@@ -287,7 +262,7 @@ class PagedKvCache:
         return n
 
 
-class Qwen3Runner:
+class Qwen3Runner(SlotState):
     """Owns the activation buffers and the native step runner for a fixed maximum batch."""
 
     def __init__(self, weights: Qwen3Weights, kv: PagedKvCache, max_batch: int, max_seq: int, nsplit: int | None = None,
@@ -322,13 +297,7 @@ class Qwen3Runner:
         B = max_batch
         f32 = dict(dtype=torch.float32, device=dev)
         i32 = dict(dtype=torch.int32, device=dev)
-        # [status word, token of slot 0, token of slot 1, ...]: one device-to-host copy brings the sampled tokens and the
-        # word in which a kernel records an expired bounded wait (copy pipeline, tensor-parallel peer)
-        self.ctl = torch.zeros(B + 1, **i32)
-        self.status = self.ctl[:1]
-        self.tokens = self.ctl[1:]
-        self.positions = torch.zeros(B, **i32)
-        self.block_table = torch.zeros((B, self.max_pages), **i32)
+        self.init_slots(B, self.max_pages, cfg.vocab, dev)
         self.h = torch.zeros((B, cfg.hidden), **f32)
         self.qkv = torch.zeros((B, (nq + 2 * nkv) * hd), **f32)
         self.q = torch.zeros((B, nq, hd), **f32)
@@ -345,14 +314,7 @@ class Qwen3Runner:
             self.partial = torch.zeros((B, cfg.hidden), **f32)
         self.ws_acc = torch.zeros((B, nq, self.nsplit, hd), **f32)
         self.ws_ml = torch.zeros((B, nq, self.nsplit, 2), **f32)
-        self.temps = torch.zeros(B, **f32)
-        self.topks = torch.zeros(B, **i32)
-        self.topps = torch.ones(B, **f32)
-        self.rng = torch.full((B,), 42, dtype=torch.int64, device=dev)
         self.out_tokens = torch.zeros(B, **i32)
-        # per-slot vocabulary masks of constrained decoding (bit set = token allowed), read by the sampler of a masked step
-        self.mask_words = (cfg.vocab + 31) // 32
-        self.allow_mask = torch.full((B, self.mask_words), -1, **i32)
         self.attn_counters = torch.zeros(B * max(1, nkv), **i32)
         cos, sin = rope_table(hd, max_seq, cfg.rope_base)
         self.rope_cos = torch.from_numpy(cos).to(dev)
@@ -414,16 +376,6 @@ class Qwen3Runner:
     def _push_slot_formats(self) -> None:
         arr = (C.c_int * len(self.slot_formats))(*self.slot_formats)
         K.check(K.lib().bonsai_runner_set_slot_formats(self._native, arr, len(self.slot_formats)), "runner_set_slot_formats")
-
-    def check_status(self, value: int | None = None) -> None:
-        """Raises when a kernel of an earlier step recorded an expired wait (``value``: the status word as already read by
-        the caller, else it is read here)."""
-        v = int(self.status.item()) if value is None else int(value)
-        if v:
-            self.status.zero_()
-            what = {2: "a tensor-parallel peer did not deliver its partial sums", 3: "a tensor-parallel peer did not reach a barrier",
-                    4: "a tensor-parallel peer did not enter an all-reduce", 5: "the weight copy pipeline of a GEMV stalled"}.get(v, "a bounded wait expired")
-            raise K.CudaKernelError(f"decode step reported status {v}: {what}")
 
     def __del__(self):
         try:

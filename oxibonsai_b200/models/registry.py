@@ -5,15 +5,21 @@ Reference: crates/oxibonsai-model/src/model_registry.rs:39-80 (variant from ``(l
 (``ModelSpec``, ``CapabilityProfile``), model_config_builder.rs:71- (``ModelConfigBuilder``) and gguf_loader.rs:19-509
 (validation, memory budget, chunked tensor iteration).  The shapes the B200 benchmarks use (36 x 4096, 36 x 2560,
 28 x 2048 - the published Qwen3 8B / 4B / 1.7B shapes) are recognised too.
+
+Designs without a GGUF form are model directories (``config.json`` + ``model.safetensors``): ``ARCHITECTURES`` maps the
+configuration's "architecture" to its reader.
 """
 from __future__ import annotations
 
+import json
 from dataclasses import dataclass, field, replace
 from enum import Enum
-from typing import Iterator
+from pathlib import Path
+from typing import Callable, Iterator
 
 from ..core import gguf as G
 from ..core.gguf import GgufFile, Qwen3Config
+from .layered_config import LayeredConfig, LayeredConfigError, keripel_config
 
 
 class ModelVariant(Enum):
@@ -227,3 +233,48 @@ def memory_budget_check(f: GgufFile, available_bytes: int, context: int = 4096, 
     weights = sum(G.data_size(t.type, t.n_elements) for t in f.tensors)
     kv = int(context * batch * cfg.layers * 2 * cfg.kv_heads * cfg.head_dim * kv_bytes_per_elem)
     return {"weights": weights, "kv_cache": kv, "total": weights + kv, "available": available_bytes, "fits": weights + kv <= available_bytes}
+
+
+# ---- designs described by a config.json ------------------------------------------------------------------------------------------
+# "architecture" of a model directory's config.json -> reader of that design's configuration
+ARCHITECTURES: dict[str, Callable[[dict, str], LayeredConfig]] = {"Keripel": keripel_config}
+
+
+def is_model_dir(path) -> bool:
+    """True for a directory with a ``config.json`` that names one of the registered designs."""
+    f = Path(path) / "config.json"
+    if not f.is_file():
+        return False
+    try:
+        return json.loads(f.read_text(encoding="utf-8")).get("architecture") in ARCHITECTURES
+    except (ValueError, AttributeError):
+        return False
+
+
+def load_model_dir_config(path) -> LayeredConfig:
+    """Reads the ``config.json`` of a model directory with the reader its "architecture" selects."""
+    f = Path(path) / "config.json"
+    raw = json.loads(f.read_text(encoding="utf-8"))
+    arch = raw.get("architecture") if isinstance(raw, dict) else None
+    if arch not in ARCHITECTURES:
+        raise LayeredConfigError(f"{f}: unknown architecture {arch!r}; registered: {sorted(ARCHITECTURES)}")
+    return ARCHITECTURES[arch](raw, Path(path).resolve().name)
+
+
+def validate_model_dir(path) -> GgufValidation:
+    """Checks that a model directory's tensors are those its configuration asks for, with their shapes."""
+    from ..convert import read_safetensors
+    try:
+        want = load_model_dir_config(path).tensor_shapes()
+        have = {t.name: t.shape for t in read_safetensors(str(Path(path) / "model.safetensors"))}
+    except (OSError, ValueError) as e:
+        return GgufValidation(False, [str(e)])
+    v = GgufValidation(True)
+    for n, shape in want.items():
+        if n not in have:
+            v.errors.append(f"missing tensor {n}")
+        elif tuple(have[n]) != shape:
+            v.errors.append(f"{n} is {list(have[n])}, expected {list(shape)}")
+    v.warnings += [f"unused tensor {n}" for n in have if n not in want]
+    v.ok = not v.errors
+    return v

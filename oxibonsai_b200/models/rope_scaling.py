@@ -181,6 +181,12 @@ def alibi_slopes(n_heads: int) -> torch.Tensor:
     return torch.tensor(pow2(closest) + extra, dtype=torch.float32)
 
 
+def geometric_slopes(n_heads: int, exponent: float = 8.0) -> torch.Tensor:
+    """``2^(-exponent (h + 1) / n_heads)`` for every head count (:func:`alibi_slopes` interleaves two such series where the head
+    count is not a power of two)."""
+    return torch.tensor([2.0 ** (-exponent * (h + 1) / n_heads) for h in range(n_heads)], dtype=torch.float32)
+
+
 class AliBiBias:
     def __init__(self, n_heads: int):
         self.slopes = alibi_slopes(n_heads)

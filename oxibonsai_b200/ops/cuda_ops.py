@@ -12,7 +12,7 @@ import torch
 from .. import _native
 
 EPI_STORE, EPI_RESID, EPI_SWIGLU = 0, 1, 2
-KV_F32, KV_F16, KV_Q8, KV_Q4 = 0, 1, 2, 3
+KV_F32, KV_F16, KV_Q8, KV_Q4, KV_BF16 = 0, 1, 2, 3, 4
 KV_DTYPES = {KV_F32: torch.float32, KV_F16: torch.float16, KV_Q8: torch.int8, KV_Q4: torch.uint8}
 
 _vp, _i, _f, _u64 = C.c_void_p, C.c_int, C.c_float, C.c_uint64
@@ -408,12 +408,13 @@ def attn_decode_qkv(qkv, q_norm, k_norm, eps, rope_cos, rope_sin, positions, blo
 
 
 def sample(logits: torch.Tensor, temps=None, topks=None, topps=None, rng=None, positions=None, advance=False,
-           allow_mask=None, out=None) -> torch.Tensor:
-    """Samples one token per row of ``logits`` ([batch, vocab] f32).  ``temps=None`` means greedy."""
+           allow_mask=None, out=None, library: C.CDLL | None = None) -> torch.Tensor:
+    """Samples one token per row of ``logits`` ([batch, vocab] f32).  ``temps=None`` means greedy.  ``library``: another native
+    library that holds the sampler (its signature declared)."""
     batch, vocab = logits.shape
     if out is None:
         out = torch.empty(batch, dtype=torch.int32, device=logits.device)
-    check(lib().bonsai_sample(logits.data_ptr(), batch, vocab, logits.stride(0), ptr(temps), ptr(topks), ptr(topps), ptr(rng),
+    check((library or lib()).bonsai_sample(logits.data_ptr(), batch, vocab, logits.stride(0), ptr(temps), ptr(topks), ptr(topps), ptr(rng),
                               out.data_ptr(), ptr(positions), int(advance and positions is not None), ptr(allow_mask),
                               0 if allow_mask is None else allow_mask.shape[1], stream()), "sample")
     return out

@@ -1,0 +1,155 @@
+"""Torch-facing wrappers of the layer-list decoder kernels in ``libbonsai_layered.so`` (csrc/layered, the sampler and the
+tcgen05 GEMM).  Every function launches on torch's current stream; there is no PyTorch fallback."""
+from __future__ import annotations
+
+import ctypes as C
+
+import torch
+
+from .. import _native
+from . import cuda_ops as K
+
+_vp, _i, _f = C.c_void_p, C.c_int, C.c_float
+_SIG = {
+    "bonsai_lay_embed": [_vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp],
+    "bonsai_lay_norm_add": [_vp, _vp, _i, _vp, _f, _i, _i, _vp, _i, _vp],
+    "bonsai_lay_norm_rows": [_vp, _vp, _vp, _f, _i, _i, _vp, _i, _i, _vp],
+    "bonsai_lay_gated_head_norm": [_vp, _i, _vp, _i, _vp, _f, _i, _i, _i, _vp, _i, _i, _vp],
+    "bonsai_lay_linear_few": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _vp],
+    "bonsai_lay_linear_f32": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
+    "bonsai_dense_gemm_bf16": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _vp, _vp, C.c_size_t, _i, _vp],
+    "bonsai_bitgemm_prefill_ws_bytes": [],
+    "bonsai_lay_attn_row": [_i],
+    "bonsai_lay_attn_append": [_vp, _vp, _vp, _i, _i, _i, _vp],
+    "bonsai_lay_attn_prompt": [_vp, _vp, _vp, _vp, _vp, _i, _vp],
+    "bonsai_lay_attn_decode": [_vp, _vp, _vp, _i, _i, _vp],
+    "bonsai_lay_attn_f32": [_vp, _vp, _vp, _i, _vp],
+    "bonsai_lay_mlstm_dim": [_i],
+    "bonsai_lay_mlstm_vdim": [_i],
+    "bonsai_lay_mlstm_chunk_dim": [],
+    "bonsai_lay_mlstm_fused_vdim": [],
+    "bonsai_lay_mlstm_step": [_vp, _vp, _vp, _vp, _i, _i, _vp],
+    "bonsai_lay_mlstm_chunk": [_vp, _vp, _vp, _vp, _i, _vp],
+    "bonsai_sample": K._SIG["bonsai_sample"],
+}
+_lib = None
+FEW_ROWS = 32               # rows up to which a projection goes to the weight-streaming kernel
+K_ALIGN = 128               # inputs of a bf16 projection are padded to a multiple of this
+
+
+def lib() -> C.CDLL:
+    global _lib
+    if _lib is None:
+        l = _native.layered()
+        for name, args in _SIG.items():
+            fn = getattr(l, name)
+            fn.argtypes = args
+            fn.restype = C.c_size_t if name.endswith("ws_bytes") else C.c_int
+        _lib = l
+    return _lib
+
+
+def round_up(n: int, m: int) -> int:
+    return -(-n // m) * m
+
+
+class DenseWeight:
+    """bf16 matrix [n, kp] on the device: ``k`` inputs, zero columns up to a multiple of 128.  ``columns[i]`` is the first
+    output of part i; parts start at multiples of four outputs (zero rows in between)."""
+
+    def __init__(self, parts: list[torch.Tensor], device, interleave: bool = False):
+        self.k = parts[0].shape[1]
+        assert all(p.shape[1] == self.k and p.dtype == torch.bfloat16 for p in parts)
+        self.kp = round_up(self.k, K_ALIGN)
+        if interleave:                       # rows 2j, 2j + 1 = row j of the two parts (the gated epilogue's order)
+            a, b = parts
+            self.columns, rows = [0, 1], [torch.stack([a, b], dim=1).reshape(-1, self.k)]
+            self.n = 2 * a.shape[0]
+        else:
+            self.columns, rows, n = [], [], 0
+            for p in parts:
+                self.columns.append(n)
+                pad = round_up(p.shape[0], 4) - p.shape[0] if len(parts) > 1 else 0
+                rows += [p, torch.zeros((pad, self.k), dtype=torch.bfloat16)]
+                n += p.shape[0] + pad
+            self.n = n
+        m = torch.zeros((self.n, self.kp), dtype=torch.bfloat16)
+        m[:, : self.k] = torch.cat(rows)
+        self.data = m.to(device)
+
+    @property
+    def nbytes(self) -> int:
+        return self.data.numel() * 2
+
+
+class GemmScratch:
+    """Workspace and status word of the tcgen05 GEMM for one stream."""
+
+    def __init__(self, device, status: torch.Tensor):
+        self.ws = torch.zeros(int(lib().bonsai_bitgemm_prefill_ws_bytes()), dtype=torch.uint8, device=device)
+        self.status = status
+        self.sms = torch.cuda.get_device_properties(device).multi_processor_count
+
+
+def linear(w: DenseWeight, x: torch.Tensor, T: int, out: torch.Tensor, scratch: GemmScratch, glu: tuple[float, float, float] | None = None) -> None:
+    """out[:T] = x[:T] W^T.  bf16 ``x`` (row stride >= kp, finite in the padding): tensor cores, f32 ``out`` (bf16 with
+    ``glu``); f32 ``x``: 32-bit throughout.  ``glu`` = (limit, alpha, offset): gated unit over interleaved rows."""
+    l, s = lib(), K.stream()
+    lim, alpha, off = glu if glu is not None else (0.0, 0.0, 0.0)
+    if x.dtype == torch.float32:
+        K.check(l.bonsai_lay_linear_f32(w.data.data_ptr(), w.n, w.k, w.kp, x.data_ptr(), x.stride(0), T, out.data_ptr(), out.stride(0),
+                                        int(glu is not None), lim, alpha, off, s), "linear_f32")
+        return
+    assert x.dtype == torch.bfloat16 and out.dtype == (torch.float32 if glu is None else torch.bfloat16)
+    f32, b16 = (out.data_ptr(), None) if glu is None else (None, out.data_ptr())
+    if T <= FEW_ROWS:
+        K.check(l.bonsai_lay_linear_few(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), int(glu is not None),
+                                        lim, alpha, off, s), "linear_few")
+    else:
+        K.check(l.bonsai_dense_gemm_bf16(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0),
+                                         0 if glu is None else 4, lim, alpha, off, scratch.status.data_ptr(), scratch.ws.data_ptr(),
+                                         scratch.ws.numel(), scratch.sms, s), "dense_gemm_bf16")
+
+
+def embed(table: torch.Tensor, tokens: torch.Tensor, T: int, width: int, x: torch.Tensor, x16: torch.Tensor | None) -> None:
+    K.check(lib().bonsai_lay_embed(table.data_ptr(), table.stride(0), tokens.data_ptr(), T, width, x.data_ptr(), K.ptr(x16),
+                                   0 if x16 is None else x16.stride(0), K.stream()), "embed")
+
+
+def norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, T: int, x16: torch.Tensor | None) -> None:
+    """x += rmsnorm(y) * w over the first T rows; ``x16`` receives the bf16 copy."""
+    K.check(lib().bonsai_lay_norm_add(x.data_ptr(), y.data_ptr(), y.stride(0), w.data_ptr(), eps, T, x.shape[1], K.ptr(x16),
+                                      0 if x16 is None else x16.stride(0), K.stream()), "norm_add")
+
+
+def norm_rows(x: torch.Tensor, rows: int | None, count: int, w: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+    """out[i] = rmsnorm(x[rows[i]]) * w (``rows``: device address of int32 indices, None = 0 .. count - 1)."""
+    K.check(lib().bonsai_lay_norm_rows(x.data_ptr(), rows, w.data_ptr(), eps, count, x.shape[1], out.data_ptr(), out.stride(0),
+                                       int(out.dtype == torch.float32), K.stream()), "norm_rows")
+
+
+def gated_head_norm(o: torch.Tensor, row0: int, gate: torch.Tensor, gate_col: int, w: torch.Tensor, eps: float, T: int, heads: int, vdim: int,
+                    out: torch.Tensor) -> None:
+    """out[row] = o / rms(o per head) * w * sigmoid(gate) for rows row0 .. row0 + T - 1 of all three."""
+    K.check(lib().bonsai_lay_gated_head_norm(o.data_ptr() + 4 * row0 * o.stride(0), o.stride(0), gate.data_ptr() + 4 * (row0 * gate.stride(0) + gate_col),
+                                             gate.stride(0), w.data_ptr(), eps, T, heads, vdim,
+                                             out.data_ptr() + out.element_size() * row0 * out.stride(0), out.stride(0),
+                                             int(out.dtype == torch.float32), K.stream()), "gated_head_norm")
+
+
+class MixerCall:
+    """The argument blocks (pointers, sizes, constants) of one mixer's launches; the tensors must outlive it."""
+
+    def __init__(self, ptrs: list[torch.Tensor], ints: list[int], floats: list[float]):
+        self._keep = ptrs
+        self.ptrs = (_vp * len(ptrs))(*[t.data_ptr() for t in ptrs])
+        self.ints = (_i * len(ints))(*ints)
+        self.floats = (_f * len(floats))(*floats)
+
+    @property
+    def args(self):
+        return self.ptrs, self.ints, self.floats
+
+
+def sample(logits: torch.Tensor, *a, **kw) -> torch.Tensor:
+    return K.sample(logits, *a, library=lib(), **kw)

@@ -22,7 +22,8 @@ from ..models.qwen3 import PagedKvCache, Qwen3Runner, Qwen3Weights
 from ..ops import cuda_ops as K
 from .presets import SamplingParams, SamplingPreset
 
-KV_NAMES = {"f32": K.KV_F32, "fp32": K.KV_F32, "f16": K.KV_F16, "fp16": K.KV_F16, "q8": K.KV_Q8, "int8": K.KV_Q8, "q4": K.KV_Q4, "int4": K.KV_Q4}
+KV_NAMES = {"f32": K.KV_F32, "fp32": K.KV_F32, "f16": K.KV_F16, "fp16": K.KV_F16, "q8": K.KV_Q8, "int8": K.KV_Q8, "q4": K.KV_Q4, "int4": K.KV_Q4,
+            "bf16": K.KV_BF16}
 
 
 @dataclass
@@ -47,32 +48,24 @@ class GenerationStats:
 class InferenceEngine:
     """Single-process engine for one GPU (or one tensor-parallel rank)."""
 
+    eos_token = EOS_TOKEN
+    supports_prefix_cache = True
+
     def __init__(self, model_path: str, max_seq_len: int = 4096, max_batch: int = 1, kv_dtype: str = "f16",
                  device: str | torch.device = "cuda:0", sampling: SamplingParams | None = None, page_size: int = 64,
                  kv_pages: int | None = None, tp_rank: int = 0, tp_size: int = 1, warmup: bool = True, exact: bool | None = None,
                  repack_cache: str | None = None, prefill_chunk: int | None = None):
         if not torch.cuda.is_available():
-            raise RuntimeError("InferenceEngine needs a CUDA device; use oxibonsai_b200.core.Oracle for the CPU path")
+            raise RuntimeError(f"{type(self).__name__} needs a CUDA device; use oxibonsai_b200.core.Oracle for the CPU path")
         self.device = torch.device(device)
         torch.cuda.set_device(self.device)
-        K.lib()  # fail loudly if the native kernels are missing
         self.model_path = str(model_path)
-        self.gguf = GgufFile.open(self.model_path)
-        self.config: Qwen3Config = self.gguf.config()
         self.max_seq_len = int(max_seq_len)
         self.max_batch = int(max_batch)
         self.sampling = (sampling or SamplingPreset.BALANCED.params()).validate()
         self.kvt = KV_NAMES[kv_dtype.lower()]
-        t0 = time.perf_counter()
         # exact = f32 activations end to end (the token-stream gate); default: exact only with an f32 KV cache
         self.exact = (self.kvt == K.KV_F32) if exact is None else bool(exact)
-        # directory of the repacked-weight cache (None = decode and repack the GGUF tensors on every start)
-        self.repack_cache = repack_cache if repack_cache is not None else os.environ.get("OXIBONSAI_REPACK_CACHE") or None
-        self.weights = Qwen3Weights(self.gguf, self.device, tp_rank, tp_size, decode_layout=not self.exact,
-                                    cache_dir=self.repack_cache, source_path=self.model_path)
-        pages_per_seq = (self.max_seq_len + page_size - 1) // page_size
-        self.kv = PagedKvCache(self.config, self.weights.kv_heads_local, kv_pages or pages_per_seq * self.max_batch, page_size,
-                               self.kvt, self.device)
         # Tokens per prompt chunk of the batched prefill path (the activation buffers are sized for it).  Larger chunks fill
         # the GPU better in the projections with few row tiles (QKV / attention output: 48 / 32 row tiles x one column block
         # per 256 tokens on 148 SMs): time to first token of a 4096-token prompt on the 8B shape 0.148 s at 1024, 0.132 s at
@@ -80,8 +73,11 @@ class InferenceEngine:
         self.prefill_chunk = int(prefill_chunk or os.environ.get("OXIBONSAI_PREFILL_CHUNK") or 4096)
         if self.prefill_chunk < 64 or self.prefill_chunk % 64:
             raise ValueError("prefill_chunk must be a multiple of 64")
-        self.runner = Qwen3Runner(self.weights, self.kv, self.max_batch, self.max_seq_len, fast=not self.exact,
-                                  prefill_chunk=self.prefill_chunk)
+        # directory of the repacked-weight cache (None = decode and repack the GGUF tensors on every start)
+        self.repack_cache = repack_cache if repack_cache is not None else os.environ.get("OXIBONSAI_REPACK_CACHE") or None
+        t0 = time.perf_counter()
+        pages_per_seq = (self.max_seq_len + page_size - 1) // page_size
+        self._load_model(kv_pages or pages_per_seq * self.max_batch, page_size, tp_rank, tp_size)
         self.load_seconds = time.perf_counter() - t0
         # pinned staging for the per-step host <-> device traffic
         self._tok_host = torch.zeros(self.max_batch, dtype=torch.int32).pin_memory()
@@ -97,6 +93,19 @@ class InferenceEngine:
             self.warmup()
 
     # ---- construction helpers -------------------------------------------------------------------
+    def _load_model(self, kv_pages: int, page_size: int, tp_rank: int, tp_size: int) -> None:
+        """Loads the checkpoint: sets ``config``, ``weights``, ``kv`` and ``runner``."""
+        K.lib()  # fail loudly if the native kernels are missing
+        if self.kvt == K.KV_BF16:
+            raise ValueError("bf16 pages belong to the layer-list decoders; use f32, f16, q8 or q4")
+        self.gguf = GgufFile.open(self.model_path)
+        self.config: Qwen3Config = self.gguf.config()
+        self.weights = Qwen3Weights(self.gguf, self.device, tp_rank, tp_size, decode_layout=not self.exact,
+                                    cache_dir=self.repack_cache, source_path=self.model_path)
+        self.kv = PagedKvCache(self.config, self.weights.kv_heads_local, kv_pages, page_size, self.kvt, self.device)
+        self.runner = Qwen3Runner(self.weights, self.kv, self.max_batch, self.max_seq_len, fast=not self.exact,
+                                  prefill_chunk=self.prefill_chunk)
+
     @classmethod
     def from_gguf_path(cls, path: str, **kw) -> "InferenceEngine":
         return cls(path, **kw)
@@ -126,8 +135,10 @@ class InferenceEngine:
             have.extend(self._pool_of(slot).alloc(need - len(have)))
             row = torch.tensor(have, dtype=torch.int32)
             self.runner.block_table[slot, : len(have)].copy_(row.to(self.device))
+        self.runner.bind_state(slot)
 
     def _release_slot(self, slot: int) -> None:
+        self.runner.release_state(slot)
         pages = self._slot_pages.pop(slot, [])
         self._pool_of(slot).release(pages)
         if slot in self._masked:
@@ -150,7 +161,7 @@ class InferenceEngine:
         return self.kv_formats()
 
     def kv_formats(self) -> list[str]:
-        names = {K.KV_F32: "f32", K.KV_F16: "f16", K.KV_Q8: "q8", K.KV_Q4: "q4"}
+        names = {K.KV_F32: "f32", K.KV_F16: "f16", K.KV_Q8: "q8", K.KV_Q4: "q4", K.KV_BF16: "bf16"}
         return [names[k] for k in sorted(self.runner.kv_pools)]
 
     def kv_utilization(self) -> float:
@@ -296,14 +307,13 @@ class InferenceEngine:
                 constraint.reset()
                 self.set_mask(0, constraint.allowed_mask())
             # first token: sample from the prefill logits on the device
-            K.sample(r.logits[:1], r.temps[:1], r.topks[:1], r.topps[:1], r.rng[:1], out=r.tokens[:1],
-                     allow_mask=r.allow_mask[:1] if masked else None)
+            r.sample_rows(0, 1, masked)
             tok = self._read_tokens(1)[0]
             stats.prefill_seconds = time.perf_counter() - t0
             pos = len(prompt)
             t_dec = time.perf_counter()
             for _ in range(max_new):
-                if stop_at_eos and tok == EOS_TOKEN:
+                if stop_at_eos and tok == self.eos_token:
                     break
                 stats.generated_tokens += 1
                 stats.token_times.append(time.perf_counter())
@@ -353,7 +363,7 @@ class InferenceEngine:
                 self._set_sampling(s, replace(p, seed=p.seed + s))
                 self._start_sequence(s, [int(t) for t in prompt], min(self.max_seq_len, n + max_tokens))
             lens = torch.tensor([len(q) for q in prompts], dtype=torch.int32).pin_memory().to(self.device, non_blocking=True)
-            K.sample(r.logits[:B], r.temps[:B], r.topks[:B], r.topps[:B], r.rng[:B], out=r.tokens[:B])
+            r.sample_rows(0, B)
             r.positions[:B].copy_(lens)
             out: list[list[int]] = [[] for _ in range(B)]
             done = [False] * B
@@ -363,7 +373,7 @@ class InferenceEngine:
                     if done[s]:
                         continue
                     tok = int(host[s])
-                    if stop_at_eos and tok == EOS_TOKEN:
+                    if stop_at_eos and tok == self.eos_token:
                         done[s] = True
                         continue
                     out[s].append(tok)
@@ -382,9 +392,7 @@ class InferenceEngine:
         """Binds ``slot``, prefills ``prompt`` and returns the first sampled token."""
         self._set_sampling(slot, params or self.sampling)
         self._start_sequence(slot, [int(t) for t in prompt], min(self.max_seq_len, max_total))
-        r = self.runner
-        K.sample(r.logits[slot: slot + 1], r.temps[slot: slot + 1], r.topks[slot: slot + 1], r.topps[slot: slot + 1], r.rng[slot: slot + 1],
-                 out=r.tokens[slot: slot + 1])
+        self.runner.sample_rows(slot, slot + 1)
         return self._read_tokens(1, slot)[0]
 
     def begin_sequence(self, prompt: Sequence[int], max_total: int, slot: int = 0, params: SamplingParams | None = None,
@@ -425,11 +433,9 @@ class InferenceEngine:
         the prefix cache and returns the first sampled token (restricted to ``mask`` when one is given)."""
         if self.prefix_cache is not None and slot not in self._slot_fmt:
             self.prefix_cache.insert([int(t) for t in prompt], self._slot_pages[slot])
-        r = self.runner
         if mask is not None:
             self.set_mask(slot, mask)
-        K.sample(r.logits[slot: slot + 1], r.temps[slot: slot + 1], r.topks[slot: slot + 1], r.topps[slot: slot + 1], r.rng[slot: slot + 1],
-                 out=r.tokens[slot: slot + 1], allow_mask=r.allow_mask[slot: slot + 1] if mask is not None else None)
+        self.runner.sample_rows(slot, slot + 1, mask is not None)
         return self._read_tokens(1, slot)[0]
 
     def step_batch(self, positions: Sequence[int], masks: dict | None = None) -> list[int]:
@@ -502,6 +508,7 @@ class InferenceEngine:
             r.allow_mask[src].fill_(-1)
         else:
             self._masked.discard(dst)
+        r.move_state(src, dst)
         self._slot_pages[dst] = self._slot_pages.pop(src, [])
         fmt = self._slot_fmt.pop(src, None)
         if fmt is not None:
@@ -525,6 +532,114 @@ class InferenceEngine:
                 "head_dim": c.head_dim, "intermediate": c.inter, "vocab": c.vocab, "context": c.context,
                 "weight_bytes": self.weights.packed_bytes, "kv_bytes": self.kv.nbytes, "load_seconds": self.load_seconds,
                 "weights_from_repack_cache": self.weights.from_cache}
+
+
+class LayeredEngine(InferenceEngine):
+    """Engine for model directories (``config.json`` + ``model.safetensors``) of the layer-list designs.
+
+    Sequences own pages of the attention layers' cache and one row of recurrent state.  ``kv_dtype`` "f32" selects the exact
+    mode (f32 throughout); "bf16" (or "f16", the other engines' default name for the 16-bit cache) the serving mode.  Steps may
+    mix single decoded tokens with portions of prompts (:meth:`step_mixed`, :meth:`feed`)."""
+
+    eos_token = -1                 # the designs name no end-of-sequence token
+
+    def _load_model(self, kv_pages: int, page_size: int, tp_rank: int, tp_size: int) -> None:
+        from ..models.layered import LayeredRunner, LayeredWeights, new_row_cache, new_state_pool
+        from ..models.registry import load_model_dir_config
+        if tp_size != 1:
+            raise NotImplementedError("tensor parallelism covers the Q1_0_g128 / TQ2_0_g128 runner only")
+        if self.kvt not in (K.KV_F32, K.KV_F16, K.KV_BF16):
+            raise ValueError("the layer-list decoders keep f32 or bf16 caches")
+        if self.exact != (self.kvt == K.KV_F32):
+            self.kvt = K.KV_F32 if self.exact else K.KV_BF16
+        self.config = load_model_dir_config(self.model_path)
+        self.weights = LayeredWeights.from_dir(self.config, self.model_path, self.device)
+        self.kv = new_row_cache(self.config, kv_pages, page_size, self.exact, self.device)
+        self.kvt = self.kv.kvt
+        states = new_state_pool(self.config, self.max_batch, self.device)
+        self.runner = LayeredRunner(self.weights, self.kv, states, self.max_batch, self.max_seq_len, self.exact, self.prefill_chunk)
+
+    @property
+    def supports_prefix_cache(self) -> bool:
+        return not self.config.recurrent_layers            # cached pages do not bring the recurrent state back
+
+    def enable_prefix_cache(self, max_pages: int | None = None):
+        if not self.supports_prefix_cache:
+            raise ValueError("a model with recurrent layers cannot resume from cached prompt pages")
+        return super().enable_prefix_cache(max_pages)
+
+    def enable_kv_formats(self, formats: Sequence[str] = ("q8", "q4"), pages: int | None = None) -> list[str]:
+        return self.kv_formats()                           # one format per engine
+
+    def prefill(self, prompt: Sequence[int], slot: int = 0, pos0: int = 0) -> None:
+        """Runs prompt tokens of ``slot`` from position ``pos0`` on in chunks, leaving the last one's logits in the runner."""
+        self.runner.prefill([int(t) for t in prompt], slot, pos0, self.prefill_chunk)
+
+    def begin_sequence(self, prompt: Sequence[int], max_total: int, slot: int = 0, params: SamplingParams | None = None,
+                       kv_format: str | None = None) -> int:
+        if len(prompt) == 0 or min(prompt) < 0 or max(prompt) >= self.config.vocab:      # before it shares a step with others
+            raise ValueError(f"a prompt needs tokens in [0, {self.config.vocab})")
+        return super().begin_sequence(prompt, max_total, slot, params, kv_format)
+
+    @property
+    def step_token_limit(self) -> int:
+        return self.runner.capacity
+
+    # ---- batches of portions and single tokens ----------------------------------------------------------------------------------------
+    supports_mixed_steps = True
+
+    def step_mixed(self, positions: Sequence[int], chunk: Sequence[int], slot: int, pos0: int, last: bool, masks: dict | None = None) -> list[int]:
+        """One step that decodes the sequences in slots 0..len(positions)-1 and runs ``chunk`` (prompt tokens of ``slot`` from
+        position ``pos0`` on) in the same batch.  Returns the sampled tokens of the decoded slots; with ``last`` the logits
+        after the chunk are left in ``logits[slot]`` for :meth:`finish_sequence`."""
+        B, r = len(positions), self.runner
+        for s, m in (masks or {}).items():
+            self.set_mask(s, m)
+        entries = [(s, (0,), p) for s, p in enumerate(positions)] + [(slot, [int(t) for t in chunk], pos0)]
+        if len(chunk) == 1:                    # a single token is a decode row: its token must be where the others' are
+            r.tokens[slot] = int(chunk[0])
+        out = r.run_batch(entries, [[0]] * B + [[len(chunk) - 1] if last else []], device_tokens=True)
+        r.logits[:B].copy_(out[:B], non_blocking=True)
+        if last:
+            r.logits[slot].copy_(out[B], non_blocking=True)
+        r.sample_rows(0, B, bool(masks))
+        return self._read_tokens(B)
+
+    def reserve(self, slot: int, n_tokens: int) -> None:
+        """Makes sure ``slot`` owns the pages of its first ``n_tokens`` tokens (and a state row); :meth:`close_sequence` gives
+        them back."""
+        self._bind_slot(slot, n_tokens)
+
+    def feed(self, entries: Sequence[tuple[int, Sequence[int], int]], want: Sequence[Sequence[int]]) -> torch.Tensor:
+        """Runs given tokens without sampling: ``entries`` = (slot, tokens, first position), all in one batch, from the cache
+        and state that earlier steps left; ``want`` names the places among each entry's tokens whose logits are returned
+        (f32 [wanted, vocab]).  A batch of single tokens in slots 0..n-1 is the captured decode step."""
+        r, n = self.runner, len(entries)
+        if all(len(t) == 1 and p > 0 for _, t, p in entries) and [s for s, _, _ in entries] == list(range(n)):
+            for s, t, p in entries:
+                if not 0 <= int(t[0]) < self.config.vocab or p >= self.max_seq_len:
+                    raise ValueError(f"entry of slot {s}: token {t[0]} at position {p} is out of range")
+                self._tok_host[s], self._pos_host[s] = int(t[0]), p
+            r.tokens[:n].copy_(self._tok_host[:n], non_blocking=True)
+            r.positions[:n].copy_(self._pos_host[:n], non_blocking=True)
+            r.step(n, sample=False)
+            out = r.logits[[s for s, w in enumerate(want) for _ in w]]
+        else:
+            out = r.run_batch(entries, want)
+        torch.cuda.synchronize(self.device)
+        r.check_status()
+        return out
+
+    def verify_greedy(self, tokens, pos0, slot=0):
+        raise NotImplementedError("drafted tokens cannot be taken back from a recurrent state")
+
+    verify_sampled = verify_greedy
+
+    def model_info(self) -> dict:
+        c = self.config
+        return {"name": c.name, "arch": c.arch, "layers": c.layers, "hidden": c.width, "vocab": c.vocab, "attention_layers": len(c.attention_layers),
+                "recurrent_layers": len(c.recurrent_layers), "weight_bytes": self.weights.packed_bytes, "kv_bytes": self.kv.nbytes,
+                "state_bytes": self.runner.states.nbytes, "load_seconds": self.load_seconds, "max_batch": self.max_batch}
 
 
 def layer_weight_type(gguf: GgufFile) -> int:
@@ -653,7 +768,10 @@ class GenericFormatEngine:
 
 
 def load_engine(model_path: str, **options):
-    """``InferenceEngine`` for Q1_0_g128 / TQ2_0_g128 checkpoints, ``GenericFormatEngine`` for every other weight format."""
+    """``LayeredEngine`` for model directories, ``InferenceEngine`` for Q1_0_g128 / TQ2_0_g128 checkpoints,
+    ``GenericFormatEngine`` for every other GGUF weight format."""
+    if os.path.isdir(str(model_path)):
+        return LayeredEngine(str(model_path), **options)
     from ..core import gguf as G
     with_type = layer_weight_type(GgufFile.open(str(model_path)))
     if with_type in (G.TQ2_0_G128, G.Q1_0_G128):

@@ -9,7 +9,8 @@ scheduler iteration, with a decode step of the live batch after every chunk - so
 the running streams by one chunk's time per step instead of the whole prompt's (the reference's ``ChunkedPrefill`` plans the
 chunks, crates/oxibonsai-model/src/chunked_prefill.rs:9-320, but runs them back to back).  Live sequences always occupy
 slots 0..n-1: when a sequence ends, the last live slot is moved into the hole (only its block-table row and sampler state
-move; KV pages are referenced, never copied).
+move; KV pages are referenced, never copied).  Engines with ``supports_mixed_steps`` run the chunk and the decode step as one
+batch instead of one after the other.
 """
 from __future__ import annotations
 
@@ -164,7 +165,10 @@ class BatchScheduler:
         self._deferred: Request | None = None  # popped from the queue, waiting for KV pages
         self.admissions = 0
         self.prefill_chunks = 0
-        self.eos = EOS_TOKEN if eos_token is None else eos_token
+        self.eos = getattr(engine, "eos_token", EOS_TOKEN) if eos_token is None else eos_token
+        # the engine takes a prompt chunk and the live sequences' tokens in one batch (not with steps in flight)
+        self.mixed = bool(getattr(engine, "supports_mixed_steps", False)) and not self.overlap
+        self.mixed_steps = 0
         self.queue = BoundedPriorityQueue(queue_capacity)
         self.idle_sleep = idle_sleep
         self.live: list[Request] = []          # live[i] occupies slot i
@@ -230,6 +234,8 @@ class BatchScheduler:
                 last_idle = time.monotonic()
                 if self.overlap:
                     self._step_overlapped()
+                elif self.mixed and self._pending is not None:
+                    self._step_mixed()
                 else:
                     self._step()
             except Exception as e:  # a failing step must not wedge the waiting clients
@@ -358,37 +364,58 @@ class BatchScheduler:
                 r.finish()
                 return True
             self._pending = {"r": r, "slot": slot, "done": covered}
+        if self.mixed and self.live:
+            return True                          # the chunk goes into the decode step that follows
         p = self._pending
-        r, slot = p["r"], p["slot"]
+        end = self._chunk_end()
         try:
-            if r.cancelled:
+            if p["r"].cancelled:
                 raise _Cancelled()
-            n = len(r.prompt)
-            # short remainders go in one piece; never leave a tail shorter than the engine's batched-prefill threshold
-            chunk = self.prefill_chunk_tokens * (self.prefill_chunk_boost if 4 * len(self.live) < eng.max_batch else 1)
-            end = n if n - p["done"] <= chunk + eng.prefill_min_tokens else p["done"] + chunk
-            eng.prefill(r.prompt[p["done"]:end], slot, p["done"])
-            self.prefill_chunks += 1
-            self._admit_cost = end - p["done"]
-            p["done"] = end
-            if end < n:
-                return True
+            eng.prefill(p["r"].prompt[p["done"]:end], p["slot"], p["done"])
+        except Exception as e:
+            self._drop_pending(e)
+            return True
+        return self._chunk_done(end)
+
+    def _chunk_end(self) -> int:
+        """End of the pending request's next prompt chunk: short remainders go in one piece, and no tail is shorter than the
+        engine's batched-prefill threshold."""
+        p, eng = self._pending, self.engine
+        n = len(p["r"].prompt)
+        chunk = self.prefill_chunk_tokens * (self.prefill_chunk_boost if 4 * len(self.live) < eng.max_batch else 1)
+        limit = getattr(eng, "step_token_limit", None)       # rows of one mixed step
+        if self.mixed and limit is not None:
+            chunk = max(1, min(chunk, limit - len(self.live) - eng.prefill_min_tokens))
+        return n if n - p["done"] <= chunk + eng.prefill_min_tokens else p["done"] + chunk
+
+    def _drop_pending(self, e: Exception) -> None:
+        """The pending request ends without having been admitted: cancelled, or failed with ``e``."""
+        r = self._pending["r"]
+        self.engine.close_sequence(self._pending["slot"])
+        if isinstance(e, _Cancelled):
+            r.finish_reason = "cancelled"
+        else:
+            r.error = e
+        r.finish()
+        self._pending = None
+
+    def _chunk_done(self, end: int) -> bool:
+        """Bookkeeping after a chunk of the pending prompt has run; the last one makes the request live."""
+        eng, p = self.engine, self._pending
+        r, slot = p["r"], p["slot"]
+        self.prefill_chunks += 1
+        self._admit_cost = end - p["done"]
+        p["done"] = end
+        if end < len(r.prompt):
+            return True
+        try:
             if r.constraint is not None:
                 r.constraint.reset()
                 first = eng.finish_sequence(r.prompt, slot, r.constraint.allowed_mask())
             else:
                 first = eng.finish_sequence(r.prompt, slot)
-        except _Cancelled:
-            eng.close_sequence(slot)
-            r.finish_reason = "cancelled"
-            r.finish()
-            self._pending = None
-            return True
         except Exception as e:
-            eng.close_sequence(slot)
-            r.error = e
-            r.finish()
-            self._pending = None
+            self._drop_pending(e)
             return True
         self._pending = None
         if r.logprobs is not None:               # from the prefill logits, which stay with the prefill slot
@@ -466,6 +493,27 @@ class BatchScheduler:
         masks = {s: r.constraint.allowed_mask() for s, r in enumerate(self.live) if r.constraint is not None}
         # raises when a kernel of the step recorded an expired wait
         toks = eng.step_batch(self._pos, masks) if masks else eng.step_batch(self._pos)
+        self._deliver(B, toks)
+        if self.after_step is not None:
+            self.after_step()
+
+    def _step_mixed(self) -> None:
+        """A decode step of the live sequences with the pending prompt's next chunk in the same batch."""
+        p, eng, B = self._pending, self.engine, len(self.live)
+        if p["r"].cancelled:
+            self._drop_pending(_Cancelled())
+            self._step()
+            return
+        end = self._chunk_end()
+        masks = {s: r.constraint.allowed_mask() for s, r in enumerate(self.live) if r.constraint is not None}
+        toks = eng.step_mixed(self._pos, p["r"].prompt[p["done"]:end], p["slot"], p["done"], end == len(p["r"].prompt), masks)
+        self.mixed_steps += 1
+        self._deliver(B, toks)
+        self._chunk_done(end)
+        if self.after_step is not None:
+            self.after_step()
+
+    def _deliver(self, B: int, toks: Sequence[int]) -> None:
         self.steps += 1
         for s in range(B):
             self._pos[s] += 1
@@ -473,5 +521,3 @@ class BatchScheduler:
         for s in range(B - 1, -1, -1):
             if self._emit(s, toks[s]):
                 self._retire(s)
-        if self.after_step is not None:
-            self.after_step()
