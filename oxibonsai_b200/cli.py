@@ -31,6 +31,8 @@ def tokenizer_candidates(model_path: str) -> list[Path]:
     def push(c: Path):
         if c not in out:
             out.append(c)
+    if p.is_dir():                        # a model directory brings its own
+        push(p / "tokenizer.json")
     push(parent / "tokenizer.json")
     push(parent / ".." / "tokenizer.json")
     base = strip_quant_suffix(p.stem)
@@ -90,7 +92,7 @@ def cmd_run(args) -> int:
     prompt = sys.stdin.read() if args.prompt == "-" else args.prompt
     tok = _load_tokenizer(args.model, args.tokenizer)
     eng = _engine(args)
-    ids = tok.encode(prompt) or [151644]
+    ids = tok.encode(prompt) or [151644 if eng.config.vocab > 151644 else 0]
     dec = StreamingDecoder()
     t0 = time.perf_counter()
     n = 0
@@ -148,7 +150,24 @@ def cmd_serve(args) -> int:
     return serve_main(argv)
 
 
+def model_dir_info(path: str) -> dict:
+    """:func:`model_info` of a model directory (``config.json`` + ``model.safetensors``)."""
+    from .models.registry import load_model_dir_config, validate_model_dir
+    cfg = load_model_dir_config(path)
+    v = validate_model_dir(path)
+    weights = Path(path) / "model.safetensors"
+    layers = [{"mixer": s.mixer.kind, **{k: x for k, x in vars(s.mixer).items()}, "mlp": None if s.mlp is None else dict(vars(s.mlp))} for s in cfg.layer_specs]
+    return {"path": path, "gpu_engine": "layer-list engine", "architecture": cfg.arch, "name": cfg.name, "quantization": "BF16",
+            "tensors": len(cfg.tensor_shapes()), "estimated_parameters": cfg.param_count(),
+            "file_size_bytes": os.path.getsize(weights) if weights.exists() else 0,
+            "config": {"layers": cfg.layers, "hidden": cfg.width, "vocab": cfg.vocab, "rms_eps": cfg.eps, "attention_layers": cfg.attention_layers,
+                       "recurrent_layers": cfg.recurrent_layers, "layer_list": layers},
+            "valid": v.ok, "errors": v.errors, "warnings": v.warnings}
+
+
 def model_info(path: str) -> dict:
+    if os.path.isdir(path):
+        return model_dir_info(path)
     from .core import GgufFile
     from .core.compat import build_compat_report, extract_model_card
     from .models.registry import validate_gguf
@@ -174,6 +193,12 @@ def cmd_info(args) -> int:
     info = model_info(args.model)
     if args.json:
         print(json.dumps(info, indent=2))
+    elif os.path.isdir(args.model):
+        c = info["config"]
+        print(f"# {info['name']}\narchitecture: {info['architecture']} ({c['layers']} layers x {c['hidden']}, vocab {c['vocab']}, "
+              f"{info['estimated_parameters'] / 1e6:.1f} M parameters, {info['quantization']})\nGPU engine: {info['gpu_engine']}")
+        for i, l in enumerate(c["layer_list"]):
+            print(f"  layer {i}: " + ", ".join(f"{k} {v}" for k, v in l.items() if k != "mlp") + (", no feed-forward" if l["mlp"] is None else f", feed-forward {l['mlp']['ff']}"))
     else:
         from .core import GgufFile
         from .core.compat import extract_model_card
@@ -190,7 +215,8 @@ def cmd_validate(args) -> int:
         print(f"warning: {w}")
     for e in info["errors"]:
         print(f"error: {e}")
-    print(f"{args.model}: {'OK' if info['valid'] else 'INVALID'} - GGUF v{info['gguf_version']}, {info['tensors']} tensors, {info['quantization']}, "
+    container = f"GGUF v{info['gguf_version']}" if "gguf_version" in info else "model directory"
+    print(f"{args.model}: {'OK' if info['valid'] else 'INVALID'} - {container}, {info['tensors']} tensors, {info['quantization']}, "
           f"{info['config']['layers']} layers x {info['config']['hidden']}")
     return 0 if info["valid"] else 1
 
@@ -307,8 +333,8 @@ def build_parser() -> argparse.ArgumentParser:
         p.add_argument("--seed", type=int, default=42)
         p.add_argument("--max-seq-len", type=int, default=4096)
         p.add_argument("--tokenizer")
-        p.add_argument("--kv-cache", default="f16", choices=["f32", "f16", "q8", "q4"])
-    r = sub.add_parser("run", help="run inference on a GGUF model")
+        p.add_argument("--kv-cache", default="f16", choices=["f32", "f16", "bf16", "q8", "q4"], help="cache format; a model directory takes bf16 (f16 means the same there) or f32")
+    r = sub.add_parser("run", help="run inference on a GGUF file or a model directory")
     r.add_argument("-m", "--model", required=True)
     r.add_argument("-p", "--prompt", required=True, help='prompt text, "-" for stdin')
     sampling(r, 256)
@@ -326,7 +352,7 @@ def build_parser() -> argparse.ArgumentParser:
     s.add_argument("--max-seq-len", type=int, default=4096)
     s.add_argument("--tokenizer")
     s.set_defaults(fn=cmd_serve)
-    i = sub.add_parser("info", help="display model info from a GGUF file")
+    i = sub.add_parser("info", help="display model info of a GGUF file or a model directory")
     i.add_argument("-m", "--model", required=True)
     i.add_argument("--json", action="store_true")
     i.set_defaults(fn=cmd_info)

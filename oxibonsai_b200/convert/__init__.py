@@ -88,14 +88,19 @@ def read_safetensors(path: str) -> Iterator[SafeTensor]:
         yield SafeTensor(name, e["dtype"], tuple(int(d) for d in e["shape"]), mm[base + lo: base + hi])
 
 
-def write_safetensors(path: str, tensors: dict[str, np.ndarray]) -> None:
-    """Writes float32 / float16 arrays as a safetensors file (used by tests and by the export tools)."""
+def write_safetensors(path: str, tensors: dict) -> None:
+    """Writes float32 / float16 arrays, or torch tensors (bfloat16 included), as a safetensors file (used by tests and by the
+    export tools)."""
     names = {np.dtype(np.float32): "F32", np.dtype(np.float16): "F16", np.dtype(np.int64): "I64", np.dtype(np.int32): "I32"}
     header, blobs, off = {}, [], 0
     for k, a in tensors.items():
+        dtype = None
+        if not isinstance(a, np.ndarray) and str(getattr(a, "dtype", "")) == "torch.bfloat16":
+            import torch
+            a, dtype = a.contiguous().view(torch.int16).numpy(), "BF16"
         a = np.ascontiguousarray(a)
         b = a.tobytes()
-        header[k] = {"dtype": names[a.dtype], "shape": list(a.shape), "data_offsets": [off, off + len(b)]}
+        header[k] = {"dtype": dtype or names[a.dtype], "shape": list(a.shape), "data_offsets": [off, off + len(b)]}
         blobs.append(b)
         off += len(b)
     h = json.dumps(header, separators=(",", ":")).encode()

@@ -5,6 +5,7 @@ is no PyTorch fallback: if the native library is missing the call raises.
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes as C
 
 import torch
@@ -439,11 +440,24 @@ def attn_decode_last_form() -> int:
 _capture_lock = __import__("threading").Lock()
 
 
+@contextlib.contextmanager
+def _collector_off(gc):
+    on = gc.isenabled()
+    gc.disable()
+    try:
+        yield
+    finally:
+        if on:
+            gc.enable()
+
+
 def capture_graph(device, fn) -> "torch.cuda.CUDAGraph":
     """Captures the launches of ``fn()`` on a side stream into a CUDA graph.  One capture at a time per process, and in
     thread-local capture mode: engines of several GPUs live in one process (replica serving), and another engine's thread
-    must be free to allocate, copy and synchronise while this one records."""
-    with _capture_lock:
+    must be free to allocate, copy and synchronise while this one records.  The garbage collector stays off meanwhile: freeing
+    an abandoned engine's graphs or streams is not permitted during a capture and would end it."""
+    import gc
+    with _capture_lock, _collector_off(gc):
         s = torch.cuda.Stream(device=device)
         s.wait_stream(torch.cuda.current_stream(device))
         g = torch.cuda.CUDAGraph()

@@ -50,6 +50,7 @@ class InferenceEngine:
 
     eos_token = EOS_TOKEN
     supports_prefix_cache = True
+    exact_prefills_in_chunks = False
 
     def __init__(self, model_path: str, max_seq_len: int = 4096, max_batch: int = 1, kv_dtype: str = "f16",
                  device: str | torch.device = "cuda:0", sampling: SamplingParams | None = None, page_size: int = 64,
@@ -204,7 +205,7 @@ class InferenceEngine:
         """Shares the KV pages of repeated prompt prefixes between sequences (full pages only).  The cache may hold up to
         ``max_pages`` pages (default: a quarter of the pool) and gives pages back when the pool runs dry."""
         from .prefix_cache import PrefixCache
-        if self.exact:
+        if self.exact and not self.exact_prefills_in_chunks:
             raise ValueError("the exact-f32 mode prefills token by token and does not use the prefix cache")
         self.prefix_cache = PrefixCache(self.kv.page_size, max_pages or max(1, self.kv.num_pages // 4), self.kv.retain, self.kv.release)
         self.kv.on_exhausted = lambda missing: self.prefix_cache.evict(missing)
@@ -542,6 +543,7 @@ class LayeredEngine(InferenceEngine):
     mix single decoded tokens with portions of prompts (:meth:`step_mixed`, :meth:`feed`)."""
 
     eos_token = -1                 # the designs name no end-of-sequence token
+    exact_prefills_in_chunks = True
 
     def _load_model(self, kv_pages: int, page_size: int, tp_rank: int, tp_size: int) -> None:
         from ..models.layered import LayeredRunner, LayeredWeights, new_row_cache, new_state_pool
@@ -615,7 +617,7 @@ class LayeredEngine(InferenceEngine):
         and state that earlier steps left; ``want`` names the places among each entry's tokens whose logits are returned
         (f32 [wanted, vocab]).  A batch of single tokens in slots 0..n-1 is the captured decode step."""
         r, n = self.runner, len(entries)
-        if all(len(t) == 1 and p > 0 for _, t, p in entries) and [s for s, _, _ in entries] == list(range(n)):
+        if n > 0 and all(len(t) == 1 and p > 0 for _, t, p in entries) and [s for s, _, _ in entries] == list(range(n)):
             for s, t, p in entries:
                 if not 0 <= int(t[0]) < self.config.vocab or p >= self.max_seq_len:
                     raise ValueError(f"entry of slot {s}: token {t[0]} at position {p} is out of range")

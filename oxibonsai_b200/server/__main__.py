@@ -79,7 +79,8 @@ def main(argv: list[str] | None = None) -> int:
     if hasattr(engine, "step_batch"):             # continuous batching over the engine's sequence slots
         for e in engines:
             if not e.exact and hasattr(e, "enable_prefix_cache"):
-                e.enable_prefix_cache()
+                if e.supports_prefix_cache:
+                    e.enable_prefix_cache()
                 if policy is not None:
                     e.enable_kv_formats(("f16", "q8", "q4"))      # the levels of the policy that the engine does not have yet
             scheds.append(BatchScheduler(e, eos_token=getattr(tokenizer, "eos_token_id", None), queue_capacity=cfg.queue_capacity, prefill_chunk_tokens=cfg.prefill_chunk_tokens, prefill_chunk_boost=cfg.prefill_chunk_boost,

@@ -75,8 +75,8 @@ class ServerConfig:
             errs.append("kv_policy must be one of off, adaptive, aggressive")
         if self.chat_template not in ("auto", "chatml", "qwen", "llama3", "mistral", "gemma"):
             errs.append("chat_template must be one of auto, chatml, qwen, llama3, mistral, gemma")
-        if self.kv_cache.lower() not in ("f32", "f16", "q8", "q4"):
-            errs.append("kv_cache must be one of f32, f16, q8, q4")
+        if self.kv_cache.lower() not in ("f32", "f16", "bf16", "q8", "q4"):
+            errs.append("kv_cache must be one of f32, f16, bf16, q8, q4")
         if check_paths:
             for name in ("model_path", "tokenizer_path"):
                 p = getattr(self, name)

@@ -1,0 +1,66 @@
+"""Small seeded model directories for the tests of the layer-list decoders."""
+import json
+import os
+
+import layered_oracle as O
+import torch
+
+
+def attention(heads=6, kv_heads=2, dim=40, scale=0.2, size=37, keep=3, ff=None, limit=1.1):
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale,
+                                           "mask": {"size": size, "keep_first": keep}}, "mlp": mlp(ff, limit)}
+
+
+def mlstm(heads=3, dim=24, vdim=40, cap=9.0, ff=None, limit=0.7):
+    return {"type": "mlstm", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}, "mlp": mlp(ff, limit)}
+
+
+def mlp(ff, limit):
+    return None if ff is None else {"kind": "dense", "ff": ff, "limit": limit}
+
+
+def config(layers, width=152, vocab=331, eps=1e-5):
+    return {"architecture": "Keripel", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+# every branch in one model: both mixers with and without a feed-forward, group sizes 3 and 1, odd sizes
+def mixed_config():
+    return config([attention(ff=200), mlstm(), attention(heads=4, kv_heads=4, dim=72, scale=0.11, size=100, keep=0),
+                   mlstm(heads=1, dim=100, vdim=136, cap=4.0, ff=90)])
+
+
+def write(path, cfg, weights):
+    from oxibonsai_b200.convert import write_safetensors
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    write_safetensors(os.path.join(path, "model.safetensors"), {k: v.bfloat16() for k, v in weights.items()})
+    return str(path)
+
+
+class Model:
+    """A model directory with its oracle weights."""
+
+    def __init__(self, path, cfg, seed=0, tweak=None, scale=1.0):
+        self.cfg = cfg
+        w = O.random_weights(cfg, seed, scale)
+        if tweak is not None:
+            tweak(w)
+            w = {k: v.bfloat16().float() for k, v in w.items()}
+        self.path = write(path, cfg, w)
+        self.w = {k: v.double() for k, v in w.items()}
+
+    def tokens(self, n, seed=1):
+        return torch.randint(0, self.cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+    def logits(self, tokens):
+        return O.forward(self.cfg, self.w, tokens)
+
+    def greedy(self, prompt, n):
+        """Greedy continuation and the smallest gap between the two best logits on the way."""
+        seq, gap = list(prompt), float("inf")
+        for _ in range(n):
+            top = torch.topk(self.logits(seq)[-1], 2).values
+            gap = min(gap, float(top[0] - top[1]))
+            seq.append(int(self.logits(seq)[-1].argmax()))
+        return seq[len(prompt):], gap

@@ -163,6 +163,8 @@ def random_weights(cfg, seed=0, scale=1.0):
             t = 0.5 * t - 1.0
         elif name.endswith(".f.b"):
             t = 2.0 + 1.5 * t                      # from strong forgetting to almost none
+        elif name.endswith((".i", ".f")):
+            t = t * 0.5 * scale * shape[-1] ** -0.5
         else:
             t = t * scale * shape[-1] ** -0.5
         w[name] = t.bfloat16().float()
