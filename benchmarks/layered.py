@@ -1,0 +1,332 @@
+#!/usr/bin/env python
+"""Layer-list decoders (Keripel) beside the closest existing model, the generic-format Qwen3 engine with f16 weights.
+
+    python benchmarks/layered.py kernels [--width 4096]     every kernel of the design and its counterpart, with roofline fractions
+    python benchmarks/layered.py models  [--sizes s,m]      prefill and decode throughput at equal parameter count
+
+Random weights, random tokens.  Kernels: CUDA events around a CUDA graph of repeated launches that walks through enough copies
+of its inputs to exceed L2; the roofline is the slower of bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate.
+"""
+from __future__ import annotations
+
+import argparse
+import json
+import os
+import sys
+import tempfile
+
+sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
+
+import torch
+
+from kernels import peaks, time_us
+
+F16 = 1
+
+
+def design(width: int, repeats: int, vocab: int = 32000, window: int = 1024) -> dict:
+    """``repeats`` times three recurrent layers and one attention layer with a feed-forward block."""
+    m = {"type": "mlstm", "mixer": {"heads": max(2, width // 512), "dim": 256, "vdim": 512, "gate_cap": 15.0}, "mlp": None}
+    a = {"type": "attention", "mixer": {"heads": width // 128, "kv_heads": max(1, width // 512), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                        "mask": {"size": window, "keep_first": 4}},
+         "mlp": {"kind": "dense", "ff": 3 * width, "limit": 7.0}}
+    return {"architecture": "Keripel", "layers": [m, m, m, a] * repeats, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width}
+
+
+def write_design(path: str, cfg: dict) -> int:
+    """A model directory with random bf16 weights; returns the parameter count."""
+    from oxibonsai_b200.convert import write_safetensors
+    from oxibonsai_b200.models.layered_config import keripel_config
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    g = torch.Generator(device="cuda").manual_seed(0)
+    t = {}
+    for n, s in keripel_config(cfg).tensor_shapes().items():
+        x = torch.randn(s, generator=g, device="cuda")
+        x = 1 + 0.1 * x if "norm" in n else (x if len(s) == 1 else x * s[-1] ** -0.5)
+        t[n] = x.bfloat16().cpu()
+    write_safetensors(os.path.join(path, "model.safetensors"), t)
+    return keripel_config(cfg).param_count()
+
+
+class Report:
+    def __init__(self):
+        p = peaks()
+        self.hbm, self.flops = p.get("hbm_gbs", 6650.0), p.get("bf16_tflops", 1590.0)
+        self.rows: list[dict] = []
+
+    def add(self, kernel: str, case: str, us: float, nbytes: float, flops: float = 0.0, like: str = "") -> float:
+        roof = max(nbytes / (self.hbm * 1e3), flops / (self.flops * 1e6))
+        r = {"kernel": kernel, "case": case, "us": round(us, 2), "roofline_us": round(roof, 2), "frac": round(roof / us, 4), "like": like}
+        self.rows.append(r)
+        print(json.dumps(r), flush=True)
+        return roof / us
+
+
+def bench_linear(rep: Report, width: int, iters: int, profile: bool) -> None:
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    scratch = L.GemmScratch(dev, torch.zeros(1, dtype=torch.int32, device=dev))
+    for name, n, k in (("proj", 3 * width + 16, width), ("gate_up", 6 * width, width), ("down", width, 3 * width)):
+        copies = max(2, int(400e6 / (2 * n * k)) + 1)
+        ws = []
+        for i in range(copies):
+            w = L.DenseWeight([torch.zeros(8, k, dtype=torch.bfloat16)], dev)
+            w.n, w.data = n, torch.randn(n, k, device=dev).bfloat16()
+            ws.append(w)
+        for T in (1, 8, 32, 64, 256, 4096):
+            x = torch.randn(T, k, device=dev).bfloat16()
+            glu = (7.0, 1.702, 1.0) if name == "gate_up" else None
+            out = torch.empty(T, n // 2 if glu else n, dtype=torch.bfloat16 if glu else torch.float32, device=dev)
+            it = [0]
+
+            def ours():
+                it[0] += 1
+                L.linear(ws[it[0] % copies], x, T, out, scratch, glu)
+            nbytes, flops = 2 * n * k + 2 * T * k + out.numel() * out.element_size(), 2.0 * T * n * k
+            rep.add("linear", f"{name} {n}x{k} T={T}", time_us(ours, iters, profile), nbytes, flops)
+            xf, xh = x.float(), x.half()
+            of = torch.empty(T, n, device=dev)
+
+            def like():                      # same bytes read as f16
+                it[0] += 1
+                w = ws[it[0] % copies].data
+                if T == 1:
+                    K.quant_gemv(F16, w.view(torch.uint8).view(-1), n, k, xf.view(-1), out=of.view(-1))
+                elif T <= 32:
+                    K.quant_gemv_batched(F16, w.view(torch.uint8).view(-1), n, k, xf, out=of)
+                else:
+                    K.dense_gemm_f16(w.view(torch.float16), xh, out=of, status=scratch.status)
+            rep.add("quant_gemv" if T <= 32 else "dense_gemm_f16", f"{name} {n}x{k} T={T}", time_us(like, iters, profile), 2 * n * k + 2 * T * k + 4 * T * n,
+                    flops, "linear")
+
+
+def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    nq, nkv, hd, page = width // 128, max(1, width // 512), 128, 64
+    i32 = dict(dtype=torch.int32, device=dev)
+    for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
+        npages = ctx // page
+        copies = max(2, int(300e6 / (2 * B * ctx * nkv * hd)) + 1)
+        pools = [torch.randn(B * npages, nkv, page, hd, device=dev).bfloat16() for _ in range(copies)]
+        rk = torch.ones(B * npages, nkv, page, device=dev)
+        bt = torch.arange(B * npages, **i32).view(B, npages)
+        pos, slots = torch.full((B,), ctx - 1, **i32), torch.arange(B, **i32)
+        ld = (nq + nkv) * hd + nq
+        proj = torch.randn(B, ld, device=dev)
+        w1, slopes = torch.ones(hd, device=dev), torch.full((nq,), 0.01, device=dev)
+        out = torch.zeros(B, nq * hd, dtype=torch.bfloat16, device=dev)
+        calls = [L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, p, rk, out], [ld, 0, nq * hd, (nq + nkv) * hd, nq * hd, nq, nkv, hd, npages, page, 0, 0],
+                             [1e-6, hd ** -0.5]) for p in pools]
+        it = [0]
+        split = 1
+        while split < 8 and B * nkv * split * 2 <= 160:
+            split *= 2
+
+        def ours():
+            it[0] += 1
+            K.check(L.lib().bonsai_lay_attn_decode(*calls[it[0] % copies].args, B, split, K.stream()), "attn_decode")
+        kv_row = 2 * B * ctx * nkv * hd
+        rep.add("attn_decode", f"B={B} ctx={ctx} heads={nq}/{nkv}", time_us(ours, iters, profile), kv_row, 4.0 * B * ctx * nq * hd)
+        vp = [p.view(torch.float16) for p in pools]
+        q, o = torch.randn(B, nq, hd, device=dev), torch.empty(B, nq, hd, device=dev)
+
+        def like():
+            it[0] += 1
+            K.attn_decode(q, pos, bt, nq, nkv, hd, K.KV_F16, page, vp[it[0] % copies], vp[(it[0] + 1) % copies], nsplit=16, out=o)
+        rep.add("attn_decode (f16 K and V)", f"B={B} ctx={ctx} heads={nq}/{nkv}", time_us(like, iters, profile), 2 * kv_row, 4.0 * B * ctx * nq * hd, "attn_decode")
+    T, npages = 4096, 64
+    pool, rk = torch.randn(npages, nkv, page, hd, device=dev).bfloat16(), torch.ones(npages, nkv, page, device=dev)
+    bt, pos, slots = torch.arange(npages, **i32).view(1, -1), torch.arange(T, **i32), torch.zeros(T, **i32)
+    proj, out = torch.randn(T, ld, device=dev), torch.zeros(T, nq * hd, dtype=torch.bfloat16, device=dev)
+    tpt = 64 // (nq // nkv)
+    entries = torch.tensor([0, T, 0, 0], **i32)
+    tiles = torch.tensor([[0, t] for t in range(0, T, tpt)], **i32)
+    for window in (0, 1024):
+        call = L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, pool, rk, out], [ld, 0, nq * hd, (nq + nkv) * hd, nq * hd, nq, nkv, hd, npages, page, window, 4],
+                           [1e-6, hd ** -0.5])
+
+        def ours():
+            K.check(L.lib().bonsai_lay_attn_prompt(*call.args, entries.data_ptr(), tiles.data_ptr(), len(tiles), K.stream()), "attn_prompt")
+        pairs = T * (T + 1) / 2 if not window else T * window - window * (window - 1) / 2 + 4 * (T - window)
+        rep.add("attn_prompt", f"T={T} window={window or 'all'} heads={nq}/{nkv}", time_us(ours, 10, profile), 4 * T * ld + 2 * T * nkv * hd + 2 * T * nq * hd,
+                4.0 * pairs * nq * hd)
+
+    def append():
+        K.check(L.lib().bonsai_lay_attn_append(*call.args, 0, T, 0, K.stream()), "attn_append")
+    rep.add("attn_append", f"T={T}", time_us(append, iters, profile), 6 * T * nkv * hd)
+    q, o16 = torch.randn(T, nq, hd, device=dev), torch.empty(T, nq * hd, dtype=torch.float16, device=dev)
+    kp, vp = torch.randn(npages, nkv, page, hd, device=dev).half(), torch.randn(npages, nkv, page, hd, device=dev).half()
+    rep.add("attn_prefill", f"T={T} heads={nq}/{nkv}", time_us(lambda: K.attn_prefill(q, 0, bt[0], nq, nkv, hd, K.KV_F16, page, kp, vp, out=o16), 10, profile),
+            4 * T * nq * hd + 4 * T * nkv * hd + 2 * T * nq * hd, 4.0 * T * (T + 1) / 2 * nq * hd, "attn_prompt")
+
+
+def bench_mlstm(rep: Report, width: int, iters: int, profile: bool) -> None:
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    H, d, e = max(2, width // 512), 256, 512
+    cols = [0, H * d, 2 * H * d, 2 * H * d + H * e, 2 * H * d + 2 * H * e, 2 * H * d + 2 * H * e + 4]
+    ld = cols[-1] + 8
+    i32 = dict(dtype=torch.int32, device=dev)
+    bias, norm = torch.zeros(H + 4, device=dev), torch.ones(H * e, device=dev)
+
+    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, plan_segments
+    scratch = [torch.empty(MAX_SEGMENTS * n, device=dev) for n in (H * d * e, H * d * e // 64, H * e // 64, H * e // 32)]
+
+    def call(T, rows, out, states, pos):
+        proj = torch.randn(T, ld, device=dev)
+        S, n, m = states
+        return L.MixerCall([proj, bias, bias + 4, norm, S, n, m, pos, torch.arange(rows, **i32), torch.arange(rows, **i32), out, *scratch],
+                           [ld, *cols, out.stride(0), H, d, e], [15.0, 1e-6, 1e-6, d ** -0.5])
+    state = lambda rows: (torch.zeros(rows, H, d, e, device=dev), torch.zeros(rows, H, e // 64, d, device=dev), torch.zeros(rows, H, e // 64, device=dev))
+    for B in (1, 8, 64):
+        copies = max(2, int(400e6 / (4 * B * H * d * e)) + 1)
+        out = torch.zeros(B, H * e, dtype=torch.bfloat16, device=dev)
+        calls = [call(B, B, out, state(B), torch.full((B,), 5, **i32)) for _ in range(copies)]
+        it = [0]
+
+        def step():
+            it[0] += 1
+            K.check(L.lib().bonsai_lay_mlstm_step(*calls[it[0] % copies].args, None, B, 1, K.stream()), "mlstm_step")
+        rep.add("mlstm_step", f"B={B} heads={H} {d}x{e}", time_us(step, iters, profile), 8.0 * B * H * d * e, 4.0 * B * H * d * e)
+        del calls
+    for nseq, T in ((1, 4096), (1, 512), (8, 512)):
+        rows = nseq * T
+        out = torch.zeros(rows, H * e, device=dev)
+        c = call(rows, nseq, out, state(nseq), torch.zeros(nseq, **i32))
+        entries = torch.tensor([[s * T, T, s, 0] for s in range(nseq)], **i32)
+        size = plan_segments([T] * nseq, H * e // 64, torch.cuda.get_device_properties(dev).multi_processor_count) * CHUNK
+        segs = [(s * T + x, min(size, T - x), s, int(x + size >= T)) for s in range(nseq) for x in range(0, T, size)] if size else []
+        per = len(segs) // nseq
+        sl = torch.tensor(segs or [[0] * 4], **i32)
+        pl = torch.tensor([(s, 0, s * per, per) for s in range(nseq)], **i32)
+        fn = lambda: K.check(L.lib().bonsai_lay_mlstm_chunk(*c.args, entries.data_ptr(), nseq, sl.data_ptr(), len(segs), pl.data_ptr(), K.stream()), "mlstm_chunk")
+        # the recurrence's own products (k v^T and S^T q) against one pass over q, k, v and o
+        rep.add("mlstm_chunk", f"{nseq} x {T} tokens heads={H} {d}x{e} segments={len(segs)}", time_us(fn, 10, profile), 4.0 * rows * H * (2 * d + 2 * e), 4.0 * rows * H * d * e)
+        act = torch.zeros(rows, H * e, dtype=torch.bfloat16, device=dev)
+        gate = torch.randn(rows, ld, device=dev)
+        rep.add("gated_head_norm", f"T={rows}", time_us(lambda: L.gated_head_norm(out, 0, gate, 0, norm, 1e-6, rows, H, e, act), iters, profile), 10.0 * rows * H * e)
+    for T in (1, 64, 4096):
+        x, y, w = torch.randn(T, width, device=dev), torch.randn(T, width, device=dev), torch.ones(width, device=dev)
+        x16 = torch.zeros(T, width, dtype=torch.bfloat16, device=dev)
+        rep.add("norm_add", f"T={T} width={width}", time_us(lambda: L.norm_add(x, y, w, 1e-6, T, x16), iters, profile), 14.0 * T * width)
+
+
+# ---- whole models ---------------------------------------------------------------------------------------------------------------------
+SIZES = {"s": dict(width=1024, repeats=3), "m": dict(width=2048, repeats=4), "l": dict(width=4096, repeats=4)}
+
+
+def _event_ms(fn, n: int) -> float:
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    e0.record()
+    for _ in range(n):
+        fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / n
+
+
+def measure_layered(path: str, steps: int, warmup: int, prompt: int, batches) -> dict:
+    from oxibonsai_b200.runtime import EngineBuilder
+    eng = EngineBuilder().model_path(path).preset("greedy").max_seq_len(prompt + 1024).max_batch(max(batches)).kv_cache("bf16").build()
+    r, vocab = eng.runner, eng.config.vocab
+    toks = torch.randint(0, vocab, (prompt,), generator=torch.Generator().manual_seed(1)).tolist()
+    res = {"weight_GB": round(eng.weights.packed_bytes / 1e9, 3), "launches_per_step": r.kernel_launches(1)}
+    for b in range(max(batches)):
+        eng.reserve(b, prompt + 3 * (steps + warmup) + 8)
+    for _ in range(3):
+        eng.prefill(toks, 0)
+    ms = _event_ms(lambda: eng.prefill(toks, 0), 5)
+    res[f"prefill_{prompt}_tok_s"] = round(prompt / ms * 1e3)
+    for b in range(1, max(batches)):
+        eng.prefill(toks, b)
+    for B in batches:
+        r.positions[:B].fill_(prompt)
+        for _ in range(warmup):
+            r.step(B)
+        ms = _event_ms(lambda: r.step(B), steps)
+        res[f"decode_b{B}_tok_s"], res[f"decode_b{B}_ms"] = round(B / ms * 1e3, 1), round(ms, 4)
+    r.check_status()
+    return res
+
+
+def measure_generic(path: str, steps: int, warmup: int, prompt: int, batches) -> dict:
+    from oxibonsai_b200.runtime.engine import GenericFormatEngine
+    eng = GenericFormatEngine(path, max_seq_len=prompt + 1024, max_batch=max(batches))
+    e = eng._eng
+    toks = torch.randint(0, eng.config.vocab, (prompt,), generator=torch.Generator().manual_seed(1)).tolist()
+    res = {"weight_GB": round(eng.model_info()["weight_bytes"] / 1e9, 3), "launches_per_step": e.kernel_launches_per_step(1)}
+    for b in range(max(batches)):
+        eng.begin_sequence(toks, prompt + 900, b)
+    dt = torch.tensor(toks, dtype=torch.int32, device="cuda")
+    for _ in range(3):
+        e.prefill(dt, 0, 0)
+    ms = _event_ms(lambda: e.prefill(dt, 0, 0), 5)
+    res[f"prefill_{prompt}_tok_s"] = round(prompt / ms * 1e3)
+    for b in range(1, max(batches)):
+        e.prefill(dt, 0, b)
+    for B in batches:
+        e.pos[:B].fill_(prompt)
+        for _ in range(warmup):
+            e.step(B)
+        ms = _event_ms(lambda: e.step(B), steps)
+        res[f"decode_b{B}_tok_s"], res[f"decode_b{B}_ms"] = round(B / ms * 1e3, 1), round(ms, 4)
+    return res
+
+
+def run_models(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64)) -> list[dict]:
+    from oxibonsai_b200.cli import requantize_gguf
+    from oxibonsai_b200.core import Qwen3Config, write_synthetic_gguf
+    rows = []
+    for size in sizes:
+        cfg = design(**SIZES[size])
+        width = cfg["width"]
+        with tempfile.TemporaryDirectory() as d:
+            params = write_design(os.path.join(d, "design"), cfg)
+            ours = measure_layered(os.path.join(d, "design"), steps, warmup, prompt, batches)
+        torch.cuda.empty_cache()
+        heads, kv, inter, vocab = width // 128, max(1, width // 512), 3 * width, cfg["vocab"]
+        per_layer = width * (heads + 2 * kv) * 128 + heads * 128 * width + 3 * width * inter
+        layers = max(1, round((params - vocab * width) / per_layer))
+        with tempfile.TemporaryDirectory() as d:
+            packed, path = os.path.join(d, "packed.gguf"), os.path.join(d, "generic.gguf")
+            write_synthetic_gguf(packed, Qwen3Config(hidden=width, inter=inter, layers=layers, heads=heads, kv_heads=kv, head_dim=128, vocab=vocab,
+                                                   context=8192, name="generic"), tied=True, seed=1)
+            requantize_gguf(packed, path, "f16")
+            like = measure_generic(path, steps, warmup, prompt, batches)
+        torch.cuda.empty_cache()
+        row = {"size": size, "width": width, "design_layers": len(cfg["layers"]), "generic_layers": layers, "params_M": round(params / 1e6),
+               "generic_params_M": round((layers * per_layer + vocab * width) / 1e6), "design": ours, "generic_f16": like}
+        rows.append(row)
+        print(json.dumps(row), flush=True)
+    return rows
+
+
+def main() -> None:
+    ap = argparse.ArgumentParser()
+    ap.add_argument("case", choices=["kernels", "models"])
+    ap.add_argument("--width", type=int, default=4096)
+    ap.add_argument("--only", default="linear,attention,mlstm")
+    ap.add_argument("--iters", type=int, default=40)
+    ap.add_argument("--sizes", default="s,m,l")
+    ap.add_argument("--profile", action="store_true", help="a few eager launches per case, for captures under a profiler")
+    a = ap.parse_args()
+    torch.cuda.set_device(0)
+    if a.case == "models":
+        run_models(a.sizes.split(","))
+        return
+    rep = Report()
+    for name, fn in (("linear", bench_linear), ("attention", bench_attention), ("mlstm", bench_mlstm)):
+        if name in a.only.split(","):
+            fn(rep, a.width, a.iters, a.profile)
+
+
+if __name__ == "__main__":
+    main()

@@ -126,13 +126,7 @@ __device__ __forceinline__ float pf_residual(const PfParams& p, int tok, int row
 
 // epilogue for one accumulator value; every lane of the warp calls it (epi 2 exchanges gate / up between lanes)
 __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, int tok, int row, int a, bool row_ok) {
-  if (p.epi == 4) {
-    // clamped gated unit: min(g, limit) * sigmoid(alpha g) * (clamp(u, -limit, limit) + offset), stored as bf16
-    const float u = fminf(fmaxf(__shfl_xor_sync(0xffffffffu, v, 1), -p.glu_limit), p.glu_limit), g = fminf(v, p.glu_limit);
-    if (row_ok && tok < p.T && (a & 1) == 0)
-      reinterpret_cast<__nv_bfloat16*>(p.out_f16)[(size_t)tok * p.out_ld + (row >> 1)] =
-          __float2bfloat16_rn(g / (1.0f + expf(-p.glu_alpha * g)) * (u + p.glu_offset));
-  } else if (p.epi == 2) {
+  if (p.epi == 2) {
     float other = __shfl_xor_sync(0xffffffffu, v, 1);
     if (row_ok && tok < p.T && (a & 1) == 0)
       p.out_f16[(size_t)tok * p.out_ld + paired_k(row >> 1)] = __float2half_rn(v / (1.0f + __expf(-v)) * other);
@@ -141,6 +135,30 @@ __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, 
     if (p.epi == 0) p.out_f32[o] = v;
     else if (p.epi == 1) p.out_f32[o] = res + v;
     else p.out_f16[o] = __float2half_rn(v);
+  }
+}
+
+// Epilogue 4 for CB accumulator values of one weight row, columns tok0 .. tok0 + CB - 1: the clamped gated unit over gate (even)
+// and up (odd) rows, min(g, limit) * sigmoid(alpha g) * (clamp(u, -limit, limit) + offset), stored as bf16.  The two lanes of a
+// pair split the columns: the even lane finishes even ones, the odd lane odd ones, so every lane has CB / 2 outputs and one
+// shuffle per output.
+template <int CB>
+__device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, int tok0, int row, int a, bool row_ok) {
+  const bool odd = a & 1;
+  float o[CB / 2];
+#pragma unroll
+  for (int j = 0; j < CB / 2; ++j) {
+    const float keep = odd ? v[2 * j + 1] : v[2 * j];
+    const float other = __shfl_xor_sync(0xffffffffu, odd ? v[2 * j] : v[2 * j + 1], 1);
+    const float g = fminf(odd ? other : keep, p.glu_limit);
+    const float u = fminf(fmaxf(odd ? keep : other, -p.glu_limit), p.glu_limit);
+    o[j] = __fdividef(g, 1.0f + __expf(-p.glu_alpha * g)) * (u + p.glu_offset);
+  }
+  __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out_f16) + (row >> 1);
+#pragma unroll
+  for (int j = 0; j < CB / 2; ++j) {
+    const int tok = tok0 + 2 * j + (odd ? 1 : 0);
+    if (row_ok && tok < p.T) dst[(size_t)tok * p.out_ld] = __float2bfloat16_rn(o[j]);
   }
 }
 
@@ -396,7 +414,12 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
           for (int j = 0; j < CB; ++j) rr[j] = __float_as_uint(__uint_as_float(rr[j]) + __uint_as_float(r2[j]));
         }
         if (c0 >= ncols) continue;
-        if (whole) {
+        if (whole && p.epi == 4) {
+          float v[CB];
+#pragma unroll
+          for (int j = 0; j < CB; ++j) v[j] = __uint_as_float(rr[j]);
+          pf_store_glu<CB>(p, v, tok0 + c0, row, a, row_ok);
+        } else if (whole) {
           float res[CB];
 #pragma unroll
           for (int j = 0; j < CB; ++j) res[j] = pf_residual(p, tok0 + c0 + j, row, row_ok);
@@ -472,6 +495,10 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
 #pragma unroll
                   for (int i = 0; i < 5; ++i) v[j] += i < cnt ? x[i] : 0.0f;
                 }
+                if (last && p.epi == 4) {
+                  pf_store_glu<8>(p, v, tok0 + cb, row, a, row_ok);      // columns past the last token are dropped there
+                  continue;
+                }
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                   if (last) pf_store(p, v[j], res[j], tok0 + cb + j, row, a, row_ok && cb + j < ncols);
@@ -482,7 +509,15 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
               if (!landed) failed = true;
             }
           } else {
-            for (int c = 0; c < ncols; ++c) {
+            for (int c = 0; c < ncols && p.epi == 4; c += 2) {
+              float v[2] = {0.0f, 0.0f};
+              for (int i = 0; i < nc; ++i)
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+                  if (c + j < ncols) v[j] += __ldcg(p.ws_part + (size_t)s_slots[i] * (128 * TOK) + (c + j) * 128 + a);
+              pf_store_glu<2>(p, v, tok0 + c, row, a, row_ok);
+            }
+            for (int c = 0; c < ncols && p.epi != 4; ++c) {
               float v = 0.0f;
               for (int i = 0; i < nc; ++i) v += __ldcg(p.ws_part + (size_t)s_slots[i] * (128 * TOK) + c * 128 + a);
               pf_store(p, v, pf_residual(p, tok0 + c, row, row_ok), tok0 + c, row, a, row_ok);

@@ -260,14 +260,16 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
 // grid (kv heads x groups of 16 query heads, splits, rows); the splits of one row form a cluster and meet in distributed
 // shared memory.  A warp walks 16-token tiles of the visible range; the split that holds the row's own position appends its
 // key before it reads it.
+constexpr int decode_stages(int hd) { return hd <= 128 ? 4 : 2; }   // key tiles a warp keeps in flight, one of them in use
+
 template <int HD>
 __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
-  constexpr int LD = HD + 8, NW = 8;
+  constexpr int LD = HD + 8, NW = 8, NST = decode_stages(HD);
   constexpr int kTile = 16 * LD;      // elements of a tile
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                    // [16][LD]
   float* res = reinterpret_cast<float*>(sQ + kTile);               // this CTA's merged rows [16][HD + 2]
-  bf16* tiles = reinterpret_cast<bf16*>(res + 16 * (HD + 2));      // [warp][2][16][LD], later the warps' partial rows
+  bf16* tiles = reinterpret_cast<bf16*>(res + 16 * (HD + 2));      // [warp][stage][16][LD], later the warps' partial rows
   float* part = reinterpret_cast<float*>(tiles);                   // [warp][16][HD + 2]
   namespace cg = cooperative_groups;
   cg::cluster_group cluster = cg::this_cluster();
@@ -291,26 +293,24 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
   const int per = (ntiles + nsplit - 1) / nsplit;
   const int b0 = split * per, b1 = min(ntiles, b0 + per);
   const bool owner = b1 == ntiles && b0 < b1;                            // holds the last tile: the row's own position
-  bf16* wt = tiles + warp * 2 * kTile;
+  bf16* wt = tiles + warp * NST * kTile;
+  float* wf = reinterpret_cast<float*>(tiles + NW * NST * kTile) + warp * NST * 16;   // key factors of the tiles
   auto first_token = [&](int j) { return (j < nkeep ? j : lo16 + j - nkeep) << 4; };
-  float2 kf[2], kn[2];   // key factors of this lane's columns: current and next tile
-  auto issue = [&](int j, int buf) {
+  auto issue = [&](int j, int st) {     // a tile lies in one page: its rows and factors are contiguous
     const int tb = first_token(j);
-#pragma unroll 4
-    for (int i = lane; i < 16 * (HD / 8); i += 32) {
-      const int r = i / (HD / 8), c = (i % (HD / 8)) * 8;
-      const bool ok = tb + r <= pos;
-      cp_async16(wt + buf * kTile + r * LD + c, pool + (ok ? cache_row(a, bt, kvh, tb + r) * HD + c : 0), ok);
-    }
+    const size_t row = cache_row(a, bt, kvh, tb);
 #pragma unroll
-    for (int nt = 0; nt < 2; ++nt) {
-      const int j0 = tb + nt * 8 + (lane & 3) * 2;
-      kn[nt].x = j0 <= pos ? __ldcg(a.krms + cache_row(a, bt, kvh, j0)) : 0.0f;
-      kn[nt].y = j0 + 1 <= pos ? __ldcg(a.krms + cache_row(a, bt, kvh, j0 + 1)) : 0.0f;
+    for (int i = 0; i < 16 * (HD / 8) / 32; ++i) {
+      const int idx = lane + 32 * i, r = idx / (HD / 8), c = (idx % (HD / 8)) * 8;
+      cp_async16(wt + st * kTile + r * LD + c, pool + (row + r) * HD + c, tb + r <= pos);
     }
+    if (lane < 4) cp_async16(wf + st * 16 + lane * 4, a.krms + row + lane * 4, true);
   };
-  const bool early = b0 + warp < b1 && !(owner && b0 + warp == b1 - 1);
-  if (early) issue(b0 + warp, 0);
+  const int j0 = b0 + warp;
+  auto is_new = [&](int j) { return owner && j == b1 - 1; };              // the tile that receives the row's own key
+#pragma unroll
+  for (int st = 0; st < NST - 1; ++st)
+    if (j0 + st * NW < b1 && !is_new(j0 + st * NW)) issue(j0 + st * NW, st);
   pdl_wait();
   pdl_trigger();
   const float* prow = a.proj + (size_t)t * a.ld;
@@ -332,34 +332,42 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
   float slope[2];
 #pragma unroll
   for (int r = 0; r < 2; ++r) slope[r] = a.slopes[kvh * G + h0 + min(g + 8 * r, nh - 1)] * kLog2e;
-  if (b0 + warp < b1 && !early) issue(b0 + warp, 0);
-  cp_async_commit();
-  int buf = 0;
-  for (int j = b0 + warp; j < b1; j += NW, buf ^= 1) {
-    kf[0] = kn[0];
-    kf[1] = kn[1];
-    if (j + NW < b1) issue(j + NW, buf ^ 1);
+#pragma unroll
+  for (int st = 0; st < NST - 1; ++st) {
+    if (j0 + st * NW < b1 && is_new(j0 + st * NW)) issue(j0 + st * NW, st);
     cp_async_commit();
-    cp_async_wait<1>();
+  }
+  constexpr bool kQReg = HD <= 128;
+  uint32_t qf[kQReg ? HD / 16 : 1][4];
+  if (kQReg) {
+#pragma unroll
+    for (int ks = 0; ks < (kQReg ? HD / 16 : 1); ++ks) ldsm4(qf[ks], frag_a(sQ, LD, 0, ks * 16, lane));
+  }
+  int it = 0;
+  for (int j = j0; j < b1; j += NW, ++it) {
+    cp_async_wait<NST - 2>();
     __syncwarp();
-    const bf16* k = wt + buf * kTile;
+    if (j + (NST - 1) * NW < b1) issue(j + (NST - 1) * NW, (it + NST - 1) % NST);
+    cp_async_commit();
+    const bf16* k = wt + (it % NST) * kTile;
+    const float* kf = wf + (it % NST) * 16;
     const int tb = first_token(j);
     float s[2][4] = {};
 #pragma unroll
     for (int ks = 0; ks < HD / 16; ++ks) {
       uint32_t q[4], b[4];
-      ldsm4(q, frag_a(sQ, LD, 0, ks * 16, lane));
+      if (!kQReg) ldsm4(q, frag_a(sQ, LD, 0, ks * 16, lane));
       ldsm4(b, frag_b_rows(k, LD, 0, ks * 16, lane));
-      mma_bf16(s[0], q, b[0], b[1]);
-      mma_bf16(s[1], q, b[2], b[3]);
+      mma_bf16(s[0], kQReg ? qf[kQReg ? ks : 0] : q, b[0], b[1]);
+      mma_bf16(s[1], kQReg ? qf[kQReg ? ks : 0] : q, b[2], b[3]);
     }
     float nm[2] = {mx[0], mx[1]}, base[2], resc[2];
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int j1 = tb + nt * 8 + (lane & 3) * 2 + (e & 1);
-        s[nt][e] = s[nt][e] * ((e & 1) ? kf[nt].y : kf[nt].x) - slope[e >> 1] * (float)(pos - j1);
+        const int c = nt * 8 + (lane & 3) * 2 + (e & 1), j1 = tb + c;
+        s[nt][e] = s[nt][e] * kf[c] - slope[e >> 1] * (float)(pos - j1);
         if (!sees(a, pos, j1)) s[nt][e] = -INFINITY;
         nm[e >> 1] = fmaxf(nm[e >> 1], s[nt][e]);
       }
@@ -535,7 +543,8 @@ static int run_prompt(const Attn& a, const int* entries, const int* tiles, int n
 template <int HD>
 static int run_decode(const Attn& a, int nrows, int nsplit, cudaStream_t stream) {
   const int mg = (a.heads / a.kv_heads + 15) / 16;
-  const size_t smem = (size_t)16 * (HD + 8) * sizeof(bf16) * (1 + 16) + (size_t)16 * (HD + 2) * sizeof(float);
+  const size_t smem = (size_t)16 * (HD + 8) * sizeof(bf16) * (1 + 8 * decode_stages(HD)) + (size_t)16 * (HD + 2) * sizeof(float) +
+                      (size_t)8 * decode_stages(HD) * 16 * sizeof(float);
   return launch(decode_kernel<HD>, dim3(a.kv_heads * mg, nsplit, nrows), 256, smem, stream, nsplit, 1, a);
 }
 template <int HD>

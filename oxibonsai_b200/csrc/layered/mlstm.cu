@@ -15,6 +15,11 @@
 // Gates, weights, normaliser and state are f32; the state and the weighted values enter their products as a bf16 pair
 // (value and remainder), i.e. with 16 significant bits.
 //
+// A long prompt in few sequences leaves most SMs idle, since its chunks follow one another.  It is then cut into segments:
+// every segment but the last first runs from an empty state (state products only), `combine_kernel` turns these local states
+// into the state each segment starts from - with (F, m, S, n) of a segment: m' = max(F + m_prev, m),
+// S' = e^(F + m_prev - m') S_prev + e^(m - m') S - and a second pass computes the outputs of all segments at once.
+//
 // State layout: S [row][head][DIM][VP], n [row][head][VP / 64][DIM], m [row][head][VP / 64] - every column tile keeps its own
 // copy of n and m - with DIM, VP the padded sizes; the padding stays zero.  A sequence's first token (position 0) starts from
 // zero whatever its state row holds.
@@ -39,7 +44,13 @@ struct Mlstm {
   void* out;               // finished activations [T][ldo] or o f32 [T][ldo]
   int ld, q_col, k_col, v_col, g_col, i_col, f_col, ldo;
   int heads, dim, vdim, vp;
+  int vec;                 // head rows start on 16-byte boundaries
   float cap, eps, den_eps, q_scale;
+  // segmented prompts: one state per segment, laid out like the pool's rows, and per column tile the local state's F and m
+  float* seg_S;
+  float* seg_n;
+  float* seg_m;
+  float* seg_F;
 };
 
 __device__ __forceinline__ float log_input_gate(const Mlstm& a, float raw, int h) { return a.cap * tanhf((raw + a.i_bias[h]) / a.cap); }
@@ -167,32 +178,43 @@ constexpr int kL = 64;      // tokens per chunk
 constexpr int kVT = 64;     // value columns per CTA
 constexpr int kVLD = kVT + 8;
 
+constexpr int chunk_warps(int dim) { return dim >= 256 ? 16 : 8; }
+
 template <int DIM>
 struct ChunkSmem {
-  static constexpr int LD = DIM + 8;
+  static constexpr int LD = DIM + 8, NCH = chunk_warps(DIM) / 4;
   bf16 q[kL * LD], k[kL * LD];
   bf16 v[kL * kVLD], vh[kL * kVLD], vl[kL * kVLD];   // values; weighted values: leading part and remainder
   bf16 sh[DIM * kVLD], sl[DIM * kVLD];               // state at the start of the chunk: leading part and remainder
   bf16 p[kL * kVLD];                                 // weighted scores
   float n[DIM];
-  float c[kL];          // i_s - F_s
-  float r[kL];          // F_t - m_t
-  float g[kL];          // weight of the initial state
-  float em[kL];         // e^-m_t
-  float w[kL];          // weight of token s in the final state
-  float rows[2][kL];    // row sums of p over the two key halves
+  struct alignas(16) Gates {
+    float c[kL];        // i_s - F_s
+    float r[kL];        // F_t - m_t
+    float g[kL];        // weight of the initial state
+    float em[kL];       // e^-m_t
+    float w[kL];        // weight of token s in the final state
+    float tail[4];      // decay of the state over the chunk, m and F at its end
+  } gates[2];           // this chunk's and the next one's
+  float rows[NCH][kL];  // row sums of p over the warps' key columns
   float nq[kL];         // q_t . n_0
-  float tail[2];        // decay of the state over the chunk, m at its end
 };
 
-// grid (vp / 64, heads, entries), 256 threads.  Warp w: rows (w & 3) * 16 .. + 15 of the chunk and half w >> 2 of the columns.
-template <int DIM>
-__global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries) {
+enum ChunkMode { kWhole, kLocal, kResume };
+
+// grid (vp / 64, heads, entries).  Warp w: rows (w & 3) * 16 .. + 15 of the chunk and group w >> 2 of the columns (keys and
+// values); of the state two 16-row tiles and WN 8-column tiles.
+// kWhole: entries {first row, tokens, slot, first position}, state from and to the pool.  kLocal / kResume: entries are the
+// segments {first row, tokens, slot, last of its prompt}; kLocal leaves a segment's local state in its scratch row, kResume
+// starts from the scratch row and writes the last segment's state to the pool.
+template <int DIM, int MODE>
+__global__ void __launch_bounds__(32 * chunk_warps(DIM), DIM <= 128 ? 2 : 1) chunk_kernel(Mlstm a, const int4* entries) {
   constexpr int LD = DIM + 8;
-  constexpr int MT = DIM / 16;                       // 16-row tiles of the state
-  constexpr int WM = MT >= 8 ? MT / 8 : 1;           // of which a warp holds this many,
-  constexpr int WN = MT >= 8 ? 8 : MT;               // with this many 8-column tiles each (MT = 4: half the columns)
-  static_assert(WM * WN * 8 == MT * 8, "state tiles over the warps");
+  constexpr int NW = chunk_warps(DIM), NTH = 32 * NW;
+  constexpr int CW = 256 / NW;                       // columns of a warp's group: 64 / (NW / 4)
+  constexpr int MT = DIM / 16, MG = MT / 2;          // 16-row tiles of the state, pairs of them
+  constexpr int WM = 2, WN = 8 * MG / NW;            // state tiles of a warp
+  static_assert(WN >= 2 && WN % 2 == 0 && MG * 8 == NW * WN, "state tiles over the warps");
   extern __shared__ __align__(16) uint8_t smem_raw[];
   ChunkSmem<DIM>& sm = *reinterpret_cast<ChunkSmem<DIM>*>(smem_raw);
   const int tile = blockIdx.x, ntile = gridDim.x, h = blockIdx.y, col0 = tile * kVT;
@@ -201,13 +223,14 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
   pdl_wait();
   pdl_trigger();
   const int4 en = entries[blockIdx.z];
-  const size_t shd = (size_t)a.state_rows[en.z] * a.heads + h;
-  float* gS = a.S + shd * DIM * a.vp + col0;
-  float* gn = a.n + (shd * ntile + tile) * DIM;
-  float* gm = a.m + shd * ntile + tile;
-  const bool fresh = en.w == 0;
-  auto state_row = [&](int i) { return (MT >= 8 ? warp + 8 * i : warp % MT) * 16; };
-  const int sc0 = MT >= 8 ? 0 : (warp / MT) * 32;    // first column of this warp's state tiles
+  if (MODE == kLocal && en.w) return;                // nothing resumes from the last segment's local state
+  const size_t pool = (size_t)a.state_rows[en.z] * a.heads + h, seg = (size_t)blockIdx.z * a.heads + h;
+  const size_t src = MODE == kWhole ? pool : seg, dst = MODE == kLocal ? seg : pool;
+  const float* inS = (MODE == kWhole ? a.S : a.seg_S) + src * DIM * a.vp + col0;
+  const float* in_n = (MODE == kWhole ? a.n : a.seg_n) + (src * ntile + tile) * DIM;
+  const bool fresh = MODE == kLocal || (MODE == kWhole && en.w == 0);
+  auto state_row = [&](int i) { return ((warp % MG) * 2 + i) * 16; };
+  const int sc0 = (warp / MG) * WN * 8;              // first column of this warp's state tiles
   float st[WM][WN][4];
 #pragma unroll
   for (int i = 0; i < WM; ++i)
@@ -216,39 +239,138 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         float2 v = make_float2(0.f, 0.f);
-        if (!fresh) v = *reinterpret_cast<const float2*>(gS + (size_t)(state_row(i) + g + 8 * e) * a.vp + sc0 + j * 8 + 2 * t4);
+        if (!fresh) v = *reinterpret_cast<const float2*>(inS + (size_t)(state_row(i) + g + 8 * e) * a.vp + sc0 + j * 8 + 2 * t4);
         st[i][j][2 * e] = v.x;
         st[i][j][2 * e + 1] = v.y;
       }
-  for (int d = tid; d < DIM; d += 256) sm.n[d] = fresh ? 0.0f : gn[d];
-  float m0 = fresh ? 0.0f : *gm;
+  float nv[WM][4];      // n of this warp's state rows: column 0 of an accumulator tile (lanes with t4 == 0), warps with sc0 == 0
+#pragma unroll
+  for (int i = 0; i < WM; ++i) {
+    nv[i][0] = fresh ? 0.0f : in_n[state_row(i) + g];
+    nv[i][2] = fresh ? 0.0f : in_n[state_row(i) + g + 8];
+    nv[i][1] = nv[i][3] = 0.0f;
+  }
+  // a local state has no floor at 0: its maximum starts empty
+  float m0 = MODE == kLocal ? -INFINITY : (fresh ? 0.0f : (MODE == kWhole ? a.m : a.seg_m)[src * ntile + tile]);
+  float Fsum = 0.0f;
 
-  for (int t0 = 0; t0 < en.y; t0 += kL) {
+  // One warp turns the raw gates of a chunk into its weights; it does so a chunk ahead, from values loaded earlier still.
+  constexpr int kGateWarp = 4 * (NW / 4 - 1);        // the warp with the least other work: first rows, last columns
+  float raw[2][2];                                   // this lane's two tokens: log forget gate's and log input gate's raw value
+  auto load_raw = [&](int at) {
+    const float* gp = a.proj + (size_t)(en.x + at + 2 * lane) * a.ld + h;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const bool ok = at + 2 * lane + e < en.y;
+      raw[e][0] = ok ? gp[(size_t)e * a.ld + a.f_col] : 0.0f;
+      raw[e][1] = ok ? gp[(size_t)e * a.ld + a.i_col] : 0.0f;
+    }
+  };
+  auto make_gates = [&](int at, float m0, typename ChunkSmem<DIM>::Gates& G) {
+    // scan of (F, M): F_t = f_1 + .. + f_t, M_t = max over s <= t of F_t - F_s + i_s; two tokens per lane
+    float f[2], ig[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const bool ok = at + 2 * lane + e < en.y;
+      f[e] = ok ? log_forget_gate(a, raw[e][0], h) : 0.0f;
+      ig[e] = ok ? log_input_gate(a, raw[e][1], h) : -INFINITY;
+    }
+    float F = f[0] + f[1], M = fmaxf(ig[0] + f[1], ig[1]);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float pf = __shfl_up_sync(0xffffffffu, F, o), pm = __shfl_up_sync(0xffffffffu, M, o);
+      if (lane >= o) {
+        M = fmaxf(pm + F, M);
+        F += pf;
+      }
+    }
+    float eF = __shfl_up_sync(0xffffffffu, F, 1), eM = __shfl_up_sync(0xffffffffu, M, 1);   // before this lane's tokens
+    if (lane == 0) {
+      eF = 0.0f;
+      eM = -INFINITY;
+    }
+    float Ft[2], Mt[2];
+    Ft[0] = eF + f[0];
+    Mt[0] = fmaxf(fmaxf(eM + f[0], ig[0]), Ft[0] + m0);
+    Ft[1] = F;
+    Mt[1] = fmaxf(M, Ft[1] + m0);
+    const float FL = __shfl_sync(0xffffffffu, Ft[1], 31), mL = __shfl_sync(0xffffffffu, Mt[1], 31);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int s = 2 * lane + e;
+      G.c[s] = ig[e] - Ft[e];
+      G.r[s] = Ft[e] - Mt[e];
+      G.g[s] = expf(Ft[e] + m0 - Mt[e]);
+      G.em[s] = expf(-Mt[e]);
+      G.w[s] = expf(FL - mL + ig[e] - Ft[e]);
+    }
+    if (lane == 0) {
+      G.tail[0] = expf(FL + m0 - mL);
+      G.tail[1] = mL;
+      G.tail[2] = FL;
+    }
+  };
+  if (warp == kGateWarp) {
+    load_raw(0);
+    make_gates(0, m0, sm.gates[0]);
+  }
+
+  for (int t0 = 0, it = 0; t0 < en.y; t0 += kL, ++it) {
     const int nt = min(kL, en.y - t0);
+    const bool more = t0 + kL < en.y;
+    const typename ChunkSmem<DIM>::Gates& G = sm.gates[it & 1];
     const float* base = a.proj + (size_t)(en.x + t0) * a.ld;
     // ---- stage the chunk: projections as bf16, the state as a bf16 pair, the gates ------------------------------------------------
-    for (int i = tid; i < kL * (DIM / 4); i += 256) {
-      const int r = i / (DIM / 4), d = (i % (DIM / 4)) * 4;
-      float qv[4], kv[4];
-      const float* qp = base + (size_t)r * a.ld + a.q_col + h * a.dim + d;
-      const float* kp = base + (size_t)r * a.ld + a.k_col + h * a.dim + d;
+    const float* qb = base + a.q_col + h * a.dim;
+    const float* kb = base + a.k_col + h * a.dim;
+    const float* vb = base + a.v_col + h * a.vdim + col0;
+    if (a.vec) {
+      constexpr int C4 = DIM / 4, N = kL * C4 / NTH, NB = N < 4 ? N : 4;   // float4 per thread, of which NB are in flight
+      constexpr int NVV = kL * (kVT / 4) / NTH;
+      const int d4 = a.dim >> 2, v4 = (a.vdim - col0) >> 2;
+      float4 vv[NVV];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const bool ok = r < nt && d + e < a.dim;
-        qv[e] = ok ? qp[e] * a.q_scale : 0.0f;
-        kv[e] = ok ? kp[e] : 0.0f;
+      for (int j = 0; j < NVV; ++j) {
+        const int i = tid + j * NTH, r = i >> 4, c = i & 15;
+        vv[j] = r < nt && c < v4 ? reinterpret_cast<const float4*>(vb + (size_t)r * a.ld)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
       }
-      *reinterpret_cast<uint2*>(sm.q + r * LD + d) = make_uint2(pack_bf16(qv[0], qv[1]), pack_bf16(qv[2], qv[3]));
-      *reinterpret_cast<uint2*>(sm.k + r * LD + d) = make_uint2(pack_bf16(kv[0], kv[1]), pack_bf16(kv[2], kv[3]));
-    }
-    for (int i = tid; i < kL * (kVT / 4); i += 256) {
-      const int r = i / (kVT / 4), c = (i % (kVT / 4)) * 4;
-      const float* vp = base + (size_t)r * a.ld + a.v_col + h * a.vdim + col0 + c;
-      float v[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[e] = r < nt && col0 + c + e < a.vdim ? vp[e] : 0.0f;
-      *reinterpret_cast<uint2*>(sm.v + r * kVLD + c) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+      for (int i0 = 0; i0 < N; i0 += NB) {
+        float4 qv[NB], kv[NB];
+#pragma unroll
+        for (int j = 0; j < NB; ++j) {
+          const int i = tid + (i0 + j) * NTH, r = i / C4, c = i % C4;
+          const bool ok = r < nt && c < d4;
+          if (MODE != kLocal) qv[j] = ok ? reinterpret_cast<const float4*>(qb + (size_t)r * a.ld)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+          kv[j] = ok ? reinterpret_cast<const float4*>(kb + (size_t)r * a.ld)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int j = 0; j < NB; ++j) {
+          const int i = tid + (i0 + j) * NTH, r = i / C4, c = i % C4;
+          if (MODE != kLocal)
+            *reinterpret_cast<uint2*>(sm.q + r * LD + 4 * c) =
+                make_uint2(pack_bf16(qv[j].x * a.q_scale, qv[j].y * a.q_scale), pack_bf16(qv[j].z * a.q_scale, qv[j].w * a.q_scale));
+          *reinterpret_cast<uint2*>(sm.k + r * LD + 4 * c) = make_uint2(pack_bf16(kv[j].x, kv[j].y), pack_bf16(kv[j].z, kv[j].w));
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < NVV; ++j) {
+        const int i = tid + j * NTH, r = i >> 4, c = i & 15;
+        *reinterpret_cast<uint2*>(sm.v + r * kVLD + 4 * c) = make_uint2(pack_bf16(vv[j].x, vv[j].y), pack_bf16(vv[j].z, vv[j].w));
+      }
+    } else {
+      for (int i = tid; i < kL * DIM; i += NTH) {
+        const int r = i / DIM, d = i % DIM;
+        const bool ok = r < nt && d < a.dim;
+        sm.q[r * LD + d] = __float2bfloat16_rn(ok ? qb[(size_t)r * a.ld + d] * a.q_scale : 0.0f);
+        sm.k[r * LD + d] = __float2bfloat16_rn(ok ? kb[(size_t)r * a.ld + d] : 0.0f);
+      }
+      for (int i = tid; i < kL * kVT; i += NTH) {
+        const int r = i / kVT, c = i % kVT;
+        sm.v[r * kVLD + c] = __float2bfloat16_rn(r < nt && col0 + c < a.vdim ? vb[(size_t)r * a.ld + c] : 0.0f);
+      }
     }
+    if (MODE != kLocal)
 #pragma unroll
     for (int i = 0; i < WM; ++i)
 #pragma unroll
@@ -261,69 +383,50 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
           *reinterpret_cast<__nv_bfloat162*>(sm.sh + o) = hi;
           *reinterpret_cast<uint32_t*>(sm.sl + o) = pack_bf16(x - __bfloat162float(hi.x), y - __bfloat162float(hi.y));
         }
-    if (warp == 0) {
-      // scan of (F, M): F_t = f_1 + .. + f_t, M_t = max over s <= t of F_t - F_s + i_s; two tokens per lane
-      float f[2], ig[2];
+    if (MODE != kLocal && sc0 == 0 && t4 == 0) {
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int s = 2 * lane + e;
-        const bool ok = s < nt;
-        f[e] = ok ? log_forget_gate(a, base[(size_t)s * a.ld + a.f_col + h], h) : 0.0f;
-        ig[e] = ok ? log_input_gate(a, base[(size_t)s * a.ld + a.i_col + h], h) : -INFINITY;
-      }
-      float F = f[0] + f[1], M = fmaxf(ig[0] + f[1], ig[1]);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float pf = __shfl_up_sync(0xffffffffu, F, o), pm = __shfl_up_sync(0xffffffffu, M, o);
-        if (lane >= o) {
-          M = fmaxf(pm + F, M);
-          F += pf;
-        }
-      }
-      float eF = __shfl_up_sync(0xffffffffu, F, 1), eM = __shfl_up_sync(0xffffffffu, M, 1);   // before this lane's tokens
-      if (lane == 0) {
-        eF = 0.0f;
-        eM = -INFINITY;
-      }
-      float Ft[2], Mt[2];
-      Ft[0] = eF + f[0];
-      Mt[0] = fmaxf(fmaxf(eM + f[0], ig[0]), Ft[0] + m0);
-      Ft[1] = F;
-      Mt[1] = fmaxf(M, Ft[1] + m0);
-      const float FL = __shfl_sync(0xffffffffu, Ft[1], 31), mL = __shfl_sync(0xffffffffu, Mt[1], 31);
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int s = 2 * lane + e;
-        sm.c[s] = ig[e] - Ft[e];
-        sm.r[s] = Ft[e] - Mt[e];
-        sm.g[s] = expf(Ft[e] + m0 - Mt[e]);
-        sm.em[s] = expf(-Mt[e]);
-        sm.w[s] = expf(FL - mL + ig[e] - Ft[e]);
-      }
-      if (lane == 0) {
-        sm.tail[0] = expf(FL + m0 - mL);
-        sm.tail[1] = mL;
+      for (int i = 0; i < WM; ++i) {
+        sm.n[state_row(i) + g] = nv[i][0];
+        sm.n[state_row(i) + g + 8] = nv[i][2];
       }
     }
     __syncthreads();
     // ---- weighted scores, the initial state's share, its normaliser, weighted values ---------------------------------------------
-    float s[4][4] = {}, oi[4][4] = {};
-    const bool live = ch == 0 || rg >= 2;            // the upper key half is ahead of the lower rows
+    if (more) {
+      // the next chunk's projections into L2, its raw gates into registers
+      const float* nb = base + (size_t)kL * a.ld;
+      const int left = min(kL, en.y - t0 - kL);
+      for (int i = tid; i < kL * (DIM / 32); i += NTH) {
+        const int r = i / (DIM / 32), d = i % (DIM / 32) * 32;
+        if (r < left && d < a.dim) {
+          const float* p = nb + (size_t)r * a.ld + h * a.dim + d;
+          if (MODE != kLocal) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + a.q_col));
+          asm volatile("prefetch.global.L2 [%0];" ::"l"(p + a.k_col));
+        }
+      }
+      if (tid < 2 * kL && (tid >> 1) < left && col0 + (tid & 1) * 32 < a.vdim)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(nb + (size_t)(tid >> 1) * a.ld + a.v_col + h * a.vdim + col0 + (tid & 1) * 32));
+      if (warp == kGateWarp) load_raw(t0 + kL);
+    }
+    float oi[CW / 8][4] = {};
+    if constexpr (MODE != kLocal) {
+    float s[CW / 8][4] = {};
+    const bool live = ch * CW <= rg * 16 + 15;       // else all of these keys come after the rows
 #pragma unroll 4
     for (int ks = 0; ks < MT; ++ks) {
       uint32_t q[4], b[4];
       ldsm4(q, frag_a(sm.q, LD, rg * 16, ks * 16, lane));
 #pragma unroll
-      for (int np = 0; np < 2; ++np) {
+      for (int np = 0; np < CW / 16; ++np) {
         if (live) {
-          ldsm4(b, frag_b_rows(sm.k, LD, ch * 32 + np * 16, ks * 16, lane));
+          ldsm4(b, frag_b_rows(sm.k, LD, ch * CW + np * 16, ks * 16, lane));
           mma_bf16(s[2 * np], q, b[0], b[1]);
           mma_bf16(s[2 * np + 1], q, b[2], b[3]);
         }
-        ldsm4_t(b, frag_b_cols(sm.sh, kVLD, ks * 16, ch * 32 + np * 16, lane));
+        ldsm4_t(b, frag_b_cols(sm.sh, kVLD, ks * 16, ch * CW + np * 16, lane));
         mma_bf16(oi[2 * np], q, b[0], b[1]);
         mma_bf16(oi[2 * np + 1], q, b[2], b[3]);
-        ldsm4_t(b, frag_b_cols(sm.sl, kVLD, ks * 16, ch * 32 + np * 16, lane));
+        ldsm4_t(b, frag_b_cols(sm.sl, kVLD, ks * 16, ch * CW + np * 16, lane));
         mma_bf16(oi[2 * np], q, b[0], b[1]);
         mma_bf16(oi[2 * np + 1], q, b[2], b[3]);
       }
@@ -331,13 +434,13 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int t = rg * 16 + g + 8 * e;
-      const float r = sm.r[t];
+      const float r = G.r[t];
       float sum = 0.0f;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int k0 = ch * 32 + j * 8 + 2 * t4;
-        const float x = k0 <= t ? s[j][2 * e] * expf(r + sm.c[k0]) : 0.0f;
-        const float y = k0 + 1 <= t ? s[j][2 * e + 1] * expf(r + sm.c[k0 + 1]) : 0.0f;
+      for (int j = 0; j < CW / 8; ++j) {
+        const int k0 = ch * CW + j * 8 + 2 * t4;
+        const float x = k0 <= t ? s[j][2 * e] * expf(r + G.c[k0]) : 0.0f;
+        const float y = k0 + 1 <= t ? s[j][2 * e + 1] * expf(r + G.c[k0 + 1]) : 0.0f;
         sum += x + y;
         *reinterpret_cast<uint32_t*>(sm.p + t * kVLD + k0) = pack_bf16(x, y);
       }
@@ -346,30 +449,37 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
       if (t4 == 0) sm.rows[ch][t] = sum;
     }
     {
-      const int t = tid >> 2;
+      constexpr int TPR = NTH / kL;                  // threads per row
+      const int t = tid / TPR, d0 = (tid % TPR) * 8;
       float x = 0.0f;
-      for (int d = (tid & 3) * 2; d < DIM; d += 8) {
-        const __nv_bfloat162 q = *reinterpret_cast<const __nv_bfloat162*>(sm.q + t * LD + d);
-        x += __bfloat162float(q.x) * sm.n[d] + __bfloat162float(q.y) * sm.n[d + 1];
+#pragma unroll 4
+      for (int d = d0; d < DIM; d += 8 * TPR) {
+        const uint4 q = *reinterpret_cast<const uint4*>(sm.q + t * LD + d);
+        const float4 n0 = *reinterpret_cast<const float4*>(sm.n + d), n1 = *reinterpret_cast<const float4*>(sm.n + d + 4);
+        const __nv_bfloat162* qq = reinterpret_cast<const __nv_bfloat162*>(&q);
+        const float2 q0 = __bfloat1622float2(qq[0]), q1 = __bfloat1622float2(qq[1]), q2 = __bfloat1622float2(qq[2]), q3 = __bfloat1622float2(qq[3]);
+        x += q0.x * n0.x + q0.y * n0.y + q1.x * n0.z + q1.y * n0.w + q2.x * n1.x + q2.y * n1.y + q3.x * n1.z + q3.y * n1.w;
       }
-      x += __shfl_xor_sync(0xffffffffu, x, 1);
-      x += __shfl_xor_sync(0xffffffffu, x, 2);
-      if ((tid & 3) == 0) sm.nq[t] = x;
+#pragma unroll
+      for (int o = 1; o < TPR; o <<= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+      if (tid % TPR == 0) sm.nq[t] = x;
     }
-    for (int i = tid; i < kL * (kVT / 2); i += 256) {
+    }
+    for (int i = tid; i < kL * (kVT / 2); i += NTH) {
       const int r = i / (kVT / 2), c = (i % (kVT / 2)) * 2;
       const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(sm.v + r * kVLD + c);
-      const float x = sm.w[r] * __bfloat162float(v.x), y = sm.w[r] * __bfloat162float(v.y);
+      const float x = G.w[r] * __bfloat162float(v.x), y = G.w[r] * __bfloat162float(v.y);
       const __nv_bfloat162 hi = __floats2bfloat162_rn(x, y);
       *reinterpret_cast<__nv_bfloat162*>(sm.vh + r * kVLD + c) = hi;
       *reinterpret_cast<uint32_t*>(sm.vl + r * kVLD + c) = pack_bf16(x - __bfloat162float(hi.x), y - __bfloat162float(hi.y));
     }
     __syncthreads();
+    if constexpr (MODE != kLocal) {
     // ---- outputs ---------------------------------------------------------------------------------------------------------------------
     {
-      const float g0 = sm.g[rg * 16 + g], g1 = sm.g[rg * 16 + g + 8];
+      const float g0 = G.g[rg * 16 + g], g1 = G.g[rg * 16 + g + 8];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
+      for (int j = 0; j < CW / 8; ++j) {
         oi[j][0] *= g0; oi[j][1] *= g0;
         oi[j][2] *= g1; oi[j][3] *= g1;
       }
@@ -380,8 +490,8 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
       uint32_t p[4], b[4];
       ldsm4(p, frag_a(sm.p, kVLD, rg * 16, ks * 16, lane));
 #pragma unroll
-      for (int np = 0; np < 2; ++np) {
-        ldsm4_t(b, frag_b_cols(sm.v, kVLD, ks * 16, ch * 32 + np * 16, lane));
+      for (int np = 0; np < CW / 16; ++np) {
+        ldsm4_t(b, frag_b_cols(sm.v, kVLD, ks * 16, ch * CW + np * 16, lane));
         mma_bf16(oi[2 * np], p, b[0], b[1]);
         mma_bf16(oi[2 * np + 1], p, b[2], b[3]);
       }
@@ -390,19 +500,24 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
     for (int e = 0; e < 2; ++e) {
       const int t = rg * 16 + g + 8 * e;
       if (t >= nt) continue;
-      const float nq = sm.g[t] * sm.nq[t] + sm.rows[0][t] + sm.rows[1][t];
-      const float den = 1.0f / (fmaxf(fabsf(nq), sm.em[t]) + a.den_eps);
+      float nq = G.g[t] * sm.nq[t];
+#pragma unroll
+      for (int c = 0; c < NW / 4; ++c) nq += sm.rows[c][t];
+      const float den = 1.0f / (fmaxf(fabsf(nq), G.em[t]) + a.den_eps);
       float* dst = static_cast<float*>(a.out) + (size_t)(en.x + t0 + t) * a.ldo + h * a.vdim + col0;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = ch * 32 + j * 8 + 2 * t4;
+      for (int j = 0; j < CW / 8; ++j) {
+        const int c = ch * CW + j * 8 + 2 * t4;
         if (col0 + c < a.vdim) dst[c] = oi[j][2 * e] * den;
         if (col0 + c + 1 < a.vdim) dst[c + 1] = oi[j][2 * e + 1] * den;
       }
     }
+    }
     // ---- the state at the end of the chunk ------------------------------------------------------------------------------------------
-    const float decay = sm.tail[0];
-    m0 = sm.tail[1];
+    if (more && warp == kGateWarp) make_gates(t0 + kL, G.tail[1], sm.gates[(it + 1) & 1]);
+    const float decay = G.tail[0];
+    m0 = G.tail[1];
+    Fsum += G.tail[2];
 #pragma unroll
     for (int i = 0; i < WM; ++i)
 #pragma unroll
@@ -410,10 +525,27 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[i][j][e] *= decay;
 #pragma unroll
+    for (int i = 0; i < WM; ++i) {
+      nv[i][0] *= decay;
+      nv[i][2] *= decay;
+    }
+#pragma unroll
     for (int ks = 0; ks < kL / 16; ++ks) {
       uint32_t kt[WM][4], b[4];
 #pragma unroll
       for (int i = 0; i < WM; ++i) ldsm4_t(kt[i], frag_a_cols(sm.k, LD, state_row(i), ks * 16, lane));
+      if (sc0 == 0) {        // n: the weights themselves as a column, a bf16 pair
+        const float2 w0 = *reinterpret_cast<const float2*>(G.w + ks * 16 + 2 * t4), w1 = *reinterpret_cast<const float2*>(G.w + ks * 16 + 8 + 2 * t4);
+        const __nv_bfloat162 h0 = __floats2bfloat162_rn(w0.x, w0.y), h1 = __floats2bfloat162_rn(w1.x, w1.y);
+        const uint32_t hi0 = g == 0 ? *reinterpret_cast<const uint32_t*>(&h0) : 0u, hi1 = g == 0 ? *reinterpret_cast<const uint32_t*>(&h1) : 0u;
+        const uint32_t lo0 = g == 0 ? pack_bf16(w0.x - __bfloat162float(h0.x), w0.y - __bfloat162float(h0.y)) : 0u;
+        const uint32_t lo1 = g == 0 ? pack_bf16(w1.x - __bfloat162float(h1.x), w1.y - __bfloat162float(h1.y)) : 0u;
+#pragma unroll
+        for (int i = 0; i < WM; ++i) {
+          mma_bf16(nv[i], kt[i], hi0, hi1);
+          mma_bf16(nv[i], kt[i], lo0, lo1);
+        }
+      }
 #pragma unroll
       for (int np = 0; np < WN / 2; ++np) {
         ldsm4_t(b, frag_b_cols(sm.vh, kVLD, ks * 16, sc0 + np * 16, lane));
@@ -430,24 +562,80 @@ __global__ void __launch_bounds__(256) chunk_kernel(Mlstm a, const int4* entries
         }
       }
     }
-    for (int d = tid; d < DIM; d += 256) {
-      float x = sm.n[d] * decay;
-#pragma unroll 8
-      for (int r = 0; r < kL; ++r) x += sm.w[r] * __bfloat162float(sm.k[r * LD + d]);
-      sm.n[d] = x;      // read by the next chunk only
-    }
     __syncthreads();    // the staged tiles are free
   }
+  if (MODE == kResume && !en.w) return;
+  float* outS = (MODE == kLocal ? a.seg_S : a.S) + dst * DIM * a.vp + col0;
 #pragma unroll
   for (int i = 0; i < WM; ++i)
 #pragma unroll
     for (int j = 0; j < WN; ++j)
 #pragma unroll
       for (int e = 0; e < 2; ++e)
-        *reinterpret_cast<float2*>(gS + (size_t)(state_row(i) + g + 8 * e) * a.vp + sc0 + j * 8 + 2 * t4) =
+        *reinterpret_cast<float2*>(outS + (size_t)(state_row(i) + g + 8 * e) * a.vp + sc0 + j * 8 + 2 * t4) =
             make_float2(st[i][j][2 * e], st[i][j][2 * e + 1]);
-  for (int d = tid; d < DIM; d += 256) gn[d] = sm.n[d];
-  if (tid == 0) *gm = m0;
+  float* out_n = (MODE == kLocal ? a.seg_n : a.n) + (dst * ntile + tile) * DIM;
+  if (sc0 == 0 && t4 == 0) {
+#pragma unroll
+    for (int i = 0; i < WM; ++i) {
+      out_n[state_row(i) + g] = nv[i][0];
+      out_n[state_row(i) + g + 8] = nv[i][2];
+    }
+  }
+  if (tid == 0) {
+    if (MODE == kLocal) *reinterpret_cast<float2*>(a.seg_F + 2 * (dst * ntile + tile)) = make_float2(Fsum, m0);
+    else a.m[dst * ntile + tile] = m0;
+  }
+}
+
+// Local states of the segments -> the states they start from.  grid (vp / 64 * 4, heads, prompts), 256 threads: a quarter of
+// a column tile's state rows.  prompts[e] = {slot, first position, first segment, segments}.
+template <int DIM>
+__global__ void __launch_bounds__(256) combine_kernel(Mlstm a, const int4* prompts) {
+  pdl_wait();
+  pdl_trigger();
+  const int tile = blockIdx.x >> 2, quarter = blockIdx.x & 3, ntile = gridDim.x >> 2, h = blockIdx.y;
+  const int4 pr = prompts[blockIdx.z];
+  const bool fresh = pr.y == 0;
+  const size_t pool = (size_t)a.state_rows[pr.x] * a.heads + h;
+  constexpr int N = DIM / 4 * 16 / 256;              // float4 per thread
+  const int c = (threadIdx.x & 15) * 4, r0 = quarter * (DIM / 4) + (threadIdx.x >> 4);
+  const bool vector = quarter == 0 && threadIdx.x < DIM;
+  auto at = [&](float* S, size_t row, int i) { return reinterpret_cast<float4*>(S + (row * DIM + r0 + 16 * i) * a.vp + tile * 64 + c); };
+  float4 s[N];
+#pragma unroll
+  for (int i = 0; i < N; ++i) s[i] = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *at(a.S, pool, i);
+  float n = vector && !fresh ? a.n[(pool * ntile + tile) * DIM + threadIdx.x] : 0.0f;
+  float m = fresh ? 0.0f : a.m[pool * ntile + tile];
+  for (int j = 0; j < pr.w; ++j) {
+    const size_t row = (size_t)(pr.z + j) * a.heads + h, idx = row * ntile + tile;
+    const bool last = j == pr.w - 1;                 // its scratch row holds no local state
+    float4 d[N];
+    float dn = 0.0f, fa = 0.0f, fb = 0.0f, mn = m;
+    if (!last) {
+#pragma unroll
+      for (int i = 0; i < N; ++i) d[i] = *at(a.seg_S, row, i);
+      if (vector) dn = a.seg_n[idx * DIM + threadIdx.x];
+      const float2 loc = *reinterpret_cast<const float2*>(a.seg_F + 2 * idx);   // F and m of the local state
+      mn = fmaxf(loc.x + m, loc.y);
+      fa = expf(loc.x + m - mn);
+      fb = expf(loc.y - mn);
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) *at(a.seg_S, row, i) = s[i];
+    if (vector) a.seg_n[idx * DIM + threadIdx.x] = n;
+    if (vector && threadIdx.x == 0) a.seg_m[idx] = m;
+    if (last) break;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      s[i].x = fa * s[i].x + fb * d[i].x;
+      s[i].y = fa * s[i].y + fb * d[i].y;
+      s[i].z = fa * s[i].z + fb * d[i].z;
+      s[i].w = fa * s[i].w + fb * d[i].w;
+    }
+    n = fa * n + fb * dn;
+    m = mn;
+  }
 }
 
 static int padded_state_dim(int dim) {
@@ -471,16 +659,24 @@ static int run_step(const Mlstm& a, const int* entries, int count, int mode, cud
 }
 
 template <int DIM>
-static int run_chunk(const Mlstm& a, const int* entries, int count, cudaStream_t stream) {
-  return launch(chunk_kernel<DIM>, dim3(a.vp / kVT, a.heads, count), 256, sizeof(ChunkSmem<DIM>), stream, 1, 0, a, (const int4*)entries);
+static int run_chunk(const Mlstm& a, const int* entries, int count, const int* segs, int nsegs, const int* prompts, cudaStream_t stream) {
+  const int nt = a.vp / kVT;
+  constexpr size_t smem = sizeof(ChunkSmem<DIM>);
+  if (nsegs == 0) return launch(chunk_kernel<DIM, kWhole>, dim3(nt, a.heads, count), 32 * chunk_warps(DIM), smem, stream, 1, 0, a, (const int4*)entries);
+  int rc = launch(chunk_kernel<DIM, kLocal>, dim3(nt, a.heads, nsegs), 32 * chunk_warps(DIM), smem, stream, 1, 0, a, (const int4*)segs);
+  if (rc == BONSAI_CUDA_OK) rc = launch(combine_kernel<DIM>, dim3(nt * 4, a.heads, count), 256, 0, stream, 1, 0, a, (const int4*)prompts);
+  if (rc == BONSAI_CUDA_OK) rc = launch(chunk_kernel<DIM, kResume>, dim3(nt, a.heads, nsegs), 32 * chunk_warps(DIM), smem, stream, 1, 0, a, (const int4*)segs);
+  return rc;
 }
 
 static bool fill(Mlstm& a, const void* const* ptrs, const int* ints, const float* floats) {
   a.proj = (const float*)ptrs[0]; a.i_bias = (const float*)ptrs[1]; a.f_bias = (const float*)ptrs[2]; a.norm = (const float*)ptrs[3];
   a.S = (float*)ptrs[4]; a.n = (float*)ptrs[5]; a.m = (float*)ptrs[6]; a.pos = (const int*)ptrs[7]; a.slots = (const int*)ptrs[8];
   a.state_rows = (const int*)ptrs[9]; a.out = const_cast<void*>(ptrs[10]);
+  a.seg_S = (float*)ptrs[11]; a.seg_n = (float*)ptrs[12]; a.seg_m = (float*)ptrs[13]; a.seg_F = (float*)ptrs[14];
   a.ld = ints[0]; a.q_col = ints[1]; a.k_col = ints[2]; a.v_col = ints[3]; a.g_col = ints[4]; a.i_col = ints[5]; a.f_col = ints[6];
   a.ldo = ints[7]; a.heads = ints[8]; a.dim = ints[9]; a.vdim = ints[10]; a.vp = (a.vdim + kVT - 1) / kVT * kVT;
+  a.vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && (a.ld | a.q_col | a.k_col | a.v_col) % 4 == 0 && (uintptr_t)a.proj % 16 == 0;
   a.cap = floats[0]; a.eps = floats[1]; a.den_eps = floats[2]; a.q_scale = floats[3];
   return a.heads >= 1 && a.heads <= 65535 && a.dim >= 1 && a.vdim >= 1 && padded_state_dim(a.dim) > 0;
 }
@@ -498,7 +694,10 @@ int bonsai_lay_mlstm_chunk_dim() { return 256; }
 // largest vdim whose single-token step finishes its outputs itself (one cluster per head)
 int bonsai_lay_mlstm_fused_vdim() { return 8 * bonsai::lay::kVT; }
 
-// ptrs = {proj, i_bias, f_bias, norm, S, n, m, pos, slots, state_rows, out}, ints = {ld, q_col, k_col, v_col, g_col, i_col,
+// tokens per chunk
+int bonsai_lay_mlstm_chunk_tokens() { return bonsai::lay::kL; }
+
+// ptrs = {proj, i_bias, f_bias, norm, S, n, m, pos, slots, state_rows, out, seg_S, seg_n, seg_m, seg_F}, ints = {ld, q_col, k_col, v_col, g_col, i_col,
 // f_col, ldo, heads, dim, vdim}, floats = {cap, eps, den_eps, q_scale}.
 
 // mode 0: entries (int4 {first row, tokens, slot, first position}), o f32; single tokens in rows 0 .. count - 1: mode 1 / 2
@@ -517,15 +716,19 @@ int bonsai_lay_mlstm_step(const void* const* ptrs, const int* ints, const float*
   }
 }
 
-// Portions of prompts, o f32.
-int bonsai_lay_mlstm_chunk(const void* const* ptrs, const int* ints, const float* floats, const int* entries, int count, cudaStream_t stream) {
+// Portions of prompts, o f32.  nsegs > 0: cut into the segments segs int4 [nsegs] {first row, tokens (a multiple of the chunk
+// except at a portion's end), slot, 1 for the last of its portion}, with prompts int4 [count] {slot, first position, first
+// segment, segments} and scratch for nsegs states.
+int bonsai_lay_mlstm_chunk(const void* const* ptrs, const int* ints, const float* floats, const int* entries, int count, const int* segs, int nsegs,
+                           const int* prompts, cudaStream_t stream) {
   using namespace bonsai::lay;
   Mlstm a;
-  if (!fill(a, ptrs, ints, floats) || count < 1 || count > 65535 || entries == nullptr) return BONSAI_CUDA_BAD_ARG;
+  if (!fill(a, ptrs, ints, floats) || count < 1 || count > 65535 || entries == nullptr || nsegs < 0 || nsegs > 65535) return BONSAI_CUDA_BAD_ARG;
+  if (nsegs > 0 && (segs == nullptr || prompts == nullptr || a.seg_S == nullptr)) return BONSAI_CUDA_BAD_ARG;
   switch (padded_state_dim(a.dim)) {
-    case 64: return run_chunk<64>(a, entries, count, stream);
-    case 128: return run_chunk<128>(a, entries, count, stream);
-    case 256: return run_chunk<256>(a, entries, count, stream);
+    case 64: return run_chunk<64>(a, entries, count, segs, nsegs, prompts, stream);
+    case 128: return run_chunk<128>(a, entries, count, segs, nsegs, prompts, stream);
+    case 256: return run_chunk<256>(a, entries, count, segs, nsegs, prompts, stream);
     default: return BONSAI_CUDA_BAD_ARG;
   }
 }

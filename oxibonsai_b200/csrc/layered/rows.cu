@@ -81,21 +81,48 @@ __global__ void norm_rows_kernel(const float* x, const int* rows, const float* _
   for (int c = threadIdx.x; c < width; c += blockDim.x) store_act(out + (size_t)blockIdx.x * ld + c, xr[c] * inv * w[c]);
 }
 
-// One block per (head, row): o / rms(o over the head) * w * sigmoid(gate)
+// One warp per (row, head): o / rms(o over the head) * w * sigmoid(gate)
 template <typename OUT>
-__global__ void gated_head_norm_kernel(const float* o, int ldo, const float* gate, int ldg, const float* __restrict__ w,
-                                       float eps, int vdim, OUT* out, int ld) {
-  __shared__ float s32[32];
+__global__ void __launch_bounds__(256) gated_head_norm_kernel(const float* o, int ldo, const float* gate, int ldg, const float* __restrict__ w,
+                                                              float eps, int T, int heads, int vdim, OUT* out, int ld, int vec) {
   pdl_wait();
   pdl_trigger();
-  const int h = blockIdx.x, t = blockIdx.y;
-  const float* orow = o + (size_t)t * ldo + h * vdim;
-  const float* grow = gate + (size_t)t * ldg + h * vdim;
+  const int lane = threadIdx.x & 31, item = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (item >= T * heads) return;
+  const int t = item / heads, c0 = (item % heads) * vdim;
+  const float* orow = o + (size_t)t * ldo + c0;
+  const float* grow = gate + (size_t)t * ldg + c0;
+  OUT* dst = out + (size_t)t * ld + c0;
+  w += c0;
+  if (vec) {                 // rows of float4, up to kKeep per lane
+    const int nch = vdim >> 2;
+    float4 v[kKeep], g[kKeep];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int c = lane + 32 * i;
+      v[i] = c < nch ? reinterpret_cast<const float4*>(orow)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+      g[i] = c < nch ? reinterpret_cast<const float4*>(grow)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int c = lane + 32 * i;
+      if (c < nch) {
+        const float4 ww = reinterpret_cast<const float4*>(w)[c];
+        const float y[4] = {v[i].x * inv * ww.x * sigmoid(g[i].x), v[i].y * inv * ww.y * sigmoid(g[i].y), v[i].z * inv * ww.z * sigmoid(g[i].z),
+                            v[i].w * inv * ww.w * sigmoid(g[i].w)};
+        if constexpr (sizeof(OUT) == 2) reinterpret_cast<uint2*>(dst)[c] = make_uint2(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]));
+        else reinterpret_cast<float4*>(dst)[c] = make_float4(y[0], y[1], y[2], y[3]);
+      }
+    }
+    return;
+  }
   float ss = 0.0f;
-  for (int c = threadIdx.x; c < vdim; c += blockDim.x) ss += orow[c] * orow[c];
-  const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)vdim + eps);
-  for (int c = threadIdx.x; c < vdim; c += blockDim.x)
-    store_act(out + (size_t)t * ld + h * vdim + c, orow[c] * inv * w[h * vdim + c] * sigmoid(grow[c]));
+  for (int c = lane; c < vdim; c += 32) ss += orow[c] * orow[c];
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  for (int c = lane; c < vdim; c += 32) store_act(dst + c, orow[c] * inv * w[c] * sigmoid(grow[c]));
 }
 
 static int row_threads(int width) {
@@ -135,10 +162,13 @@ int bonsai_lay_norm_rows(const float* x, const int* rows, const float* w, float 
 int bonsai_lay_gated_head_norm(const float* o, int ldo, const float* gate, int ldg, const float* w, float eps, int T, int heads, int vdim, void* out,
                                int ld, int f32_out, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (T < 1 || T > 65535 || heads < 1 || vdim < 1 || ld < heads * vdim) return BONSAI_CUDA_BAD_ARG;
-  const int th = vdim >= 256 ? 256 : (vdim > 64 ? 128 : 64);
-  if (f32_out) return launch(gated_head_norm_kernel<float>, dim3(heads, T), th, 0, stream, 1, 0, o, ldo, gate, ldg, w, eps, vdim, (float*)out, ld);
-  return launch(gated_head_norm_kernel<bf16>, dim3(heads, T), th, 0, stream, 1, 0, o, ldo, gate, ldg, w, eps, vdim, (bf16*)out, ld);
+  if (T < 1 || heads < 1 || vdim < 1 || ld < heads * vdim || (long long)T * heads >= (1ll << 30)) return BONSAI_CUDA_BAD_ARG;
+  const dim3 grid((T * heads + 7) / 8);
+  const uintptr_t at = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out);
+  const int vec = vdim % 4 == 0 && vdim <= 128 * kKeep && ldo % 4 == 0 && ldg % 4 == 0 && ld % 4 == 0 && at % 16 == 0;
+  if (f32_out)
+    return launch(gated_head_norm_kernel<float>, grid, 256, 0, stream, 1, 0, o, ldo, gate, ldg, w, eps, T, heads, vdim, (float*)out, ld, vec);
+  return launch(gated_head_norm_kernel<bf16>, grid, 256, 0, stream, 1, 0, o, ldo, gate, ldg, w, eps, T, heads, vdim, (bf16*)out, ld, vec);
 }
 
 }  // extern "C"

@@ -125,6 +125,29 @@ class StepShape:
     portions: int = 0
     entries: int = 0
     tiles: dict[int, tuple[int, int]] | None = None      # tokens per tile -> (device address, tiles)
+    segments: int = 0                                    # recurrences run the portions cut into this many segments (0: whole)
+    segment_list: int = 0
+    prompt_list: int = 0
+
+
+MAX_SEGMENTS = 24           # segment states the scratch of the recurrent layers holds
+CHUNK = 64                  # tokens per chunk of the recurrences
+
+
+def plan_segments(lengths: Sequence[int], ctas: int, sms: int) -> int:
+    """Chunks per segment for portions of ``lengths`` tokens when one segment occupies ``ctas`` CTAs, one per SM; 0 = do not
+    cut.  Segments run side by side, but their state products run twice; the constants are fitted to measured times (8 heads of
+    256 x 512: 4096 tokens 600 us whole, 443 us in 2 segments, 451 in 4, 548 in 16; 512 tokens 76 us whole, 64 us in 2)."""
+    chunks = [-(-n // CHUNK) for n in lengths]
+    best, best_cost = 0, max(chunks) * -(-ctas * len(chunks) // sms)
+    for size in range(4, max(chunks)):
+        segs = sum(-(-c // size) for c in chunks)
+        if segs > MAX_SEGMENTS:
+            continue
+        cost = 1.5 * size * -(-ctas * segs // sms) + 0.5 + 0.6 * segs
+        if cost < best_cost:
+            best, best_cost = size, cost
+    return best
 
 
 class AttentionMixer:
@@ -179,7 +202,7 @@ class MlstmMixer:
 
         def call(rows, out):
             return L.MixerCall([r.proj, self.w.vectors["i.b"], self.w.vectors["f.b"], self.w.vectors["norm"], s["S"], s["n"], s["m"], rows.positions,
-                                rows.slots, r.state_table, out],
+                                rows.slots, r.state_table, out, *r.segment_scratch],
                                [r.proj.stride(0), q, k, v, self.g_col, i, f, out.stride(0), spec.heads, spec.dim, spec.vdim], floats)
         # o f32 for the gated head norm, and the finished activations of the fused single-token step
         self.raw = {id(rows): call(rows, r.head_out) for rows in (r.slot_rows, r.batch_rows)}
@@ -199,7 +222,7 @@ class MlstmMixer:
         if st.portions:
             a = self.raw[id(rows)].args
             if self.chunked:
-                K.check(lib.bonsai_lay_mlstm_chunk(*a, st.entries, st.portions, stream), "mlstm_chunk")
+                K.check(lib.bonsai_lay_mlstm_chunk(*a, st.entries, st.portions, st.segment_list, st.segments, st.prompt_list, stream), "mlstm_chunk")
             else:
                 K.check(lib.bonsai_lay_mlstm_step(*a, st.entries, st.portions, 0, stream), "mlstm_step")
             self._finish(st.singles, st.rows - st.singles)
@@ -244,10 +267,17 @@ class LayeredRunner(SlotState):
         self.proj = torch.zeros((cap, max(L.round_up(l.proj.n, 4) for l in weights.layers)), **f32)
         widths = [cfg.layer_specs[i].mixer.out_width for i in cfg.recurrent_layers]
         self.head_out = torch.zeros((cap, L.round_up(max(widths, default=4), 4)), **f32)
+        # states of the segments a long prompt is cut into (layers run one after another and share them)
+        chunked = [] if exact else [m for m in (cfg.layer_specs[i].mixer for i in cfg.recurrent_layers) if m.dim <= L.lib().bonsai_lay_mlstm_chunk_dim()]
+        self._segment_ctas = min((m.heads * L.lib().bonsai_lay_mlstm_vdim(m.vdim) // 64 for m in chunked), default=0)
+        shapes = [(m.heads, L.lib().bonsai_lay_mlstm_dim(m.dim), L.lib().bonsai_lay_mlstm_vdim(m.vdim)) for m in chunked]
+        segs = min(MAX_SEGMENTS, cap // CHUNK) if shapes else 0
+        self.segment_scratch = [torch.empty(max(1, segs * max((f(*s) for s in shapes), default=0)), **f32) for f in
+                                (lambda h, d, e: h * d * e, lambda h, d, e: h * d * e // 64, lambda h, d, e: h * e // 64, lambda h, d, e: h * e // 32)]
         # row metadata: decode steps use the slot tensors as they are; a mixed batch uploads [tokens | positions | slots | lists]
         self.slot_rows = Rows(self.tokens, self.positions, torch.arange(max_batch, **i32))
         self._tile_sizes = sorted({64 // cfg.layer_specs[i].mixer.group for i in cfg.attention_layers})
-        self._meta = torch.zeros(3 * cap + 4 * cap + 2 * cap * len(self._tile_sizes) + cap + 16, **i32)
+        self._meta = torch.zeros(3 * cap + 4 * cap + 8 * MAX_SEGMENTS + 2 * cap * len(self._tile_sizes) + cap + 16, **i32)
         self.batch_rows = Rows(*(self._meta[i * cap:(i + 1) * cap] for i in range(3)))
         self._host = [torch.zeros(self._meta.numel(), dtype=torch.int32).pin_memory() for _ in range(2)]
         self._host_free = [torch.cuda.Event() for _ in range(2)]
@@ -369,6 +399,19 @@ class LayeredRunner(SlotState):
             lo, hi = put(a)
             host[lo:hi] = a
             end = hi
+            lengths = [n for _, n, _, _ in lists]
+            size = plan_segments(lengths, self._segment_ctas, self.scratch.sms) if self._segment_ctas else 0
+            if size:
+                segs, prompts = [], []
+                for first, n, slot, pos0 in lists:
+                    cuts = range(0, n, size * CHUNK)
+                    prompts.append((slot, pos0, len(segs), len(cuts)))
+                    segs += [(first + c, min(size * CHUNK, n - c), slot, int(c == cuts[-1])) for c in cuts]
+                a = np.asarray(segs + prompts, dtype=np.int32).reshape(-1)
+                lo, hi = put(a)
+                host[lo:hi] = a
+                st.segments, st.segment_list, st.prompt_list = len(segs), base + 4 * lo, base + 4 * (lo + 4 * len(segs))
+                end = hi
             for size in self._tile_sizes:
                 a = np.asarray([(e, t) for e, (_, n, _, _) in enumerate(lists) for t in range(0, n, size)], dtype=np.int32).reshape(-1)
                 lo, hi = put(a)

@@ -29,7 +29,8 @@ _SIG = {
     "bonsai_lay_mlstm_chunk_dim": [],
     "bonsai_lay_mlstm_fused_vdim": [],
     "bonsai_lay_mlstm_step": [_vp, _vp, _vp, _vp, _i, _i, _vp],
-    "bonsai_lay_mlstm_chunk": [_vp, _vp, _vp, _vp, _i, _vp],
+    "bonsai_lay_mlstm_chunk_tokens": [],
+    "bonsai_lay_mlstm_chunk": [_vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _vp],
     "bonsai_sample": K._SIG["bonsai_sample"],
 }
 _lib = None

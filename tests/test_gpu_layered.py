@@ -226,6 +226,27 @@ def test_state_carries_far(tmp_path, kv):
         check(feed(eng, tokens, cuts), want, kv, what=str(cuts[:3]))
 
 
+@pytest.mark.parametrize("d,e", [(20, 70), (100, 40), (200, 66)])
+def test_long_prompts_in_segments(tmp_path, d, e):
+    """Prompts long enough for the recurrence to be cut into segments, from position 0 and from a state, alone and together."""
+    from oxibonsai_b200.models.layered import plan_segments
+    m = M.Model(tmp_path / "m", M.config([M.mlstm(heads=2, dim=d, vdim=e)], vocab=70, width=64), seed=d,
+                tweak=lambda w: w["l0.mix.f.b"].copy_(torch.tensor([6.0, 1.0])))
+    eng = engine(m, "bf16", max_batch=3, max_seq=1024, chunk=2048)
+    poison(eng)
+    tokens = m.tokens(900)
+    want = m.logits(tokens)
+    assert plan_segments([900], eng.runner._segment_ctas, 148) and plan_segments([600, 700], eng.runner._segment_ctas, 148)
+    check(feed(eng, tokens, []), want, "bf16", "whole")
+    check(feed(eng, tokens, [77, 700, 2]), want, "bf16", "resumed")
+    for s, n in ((0, 600), (1, 1), (2, 900)):
+        eng.reserve(s, n)
+    eng.feed([(2, tokens[:200], 0)], [[]])
+    out = eng.feed([(0, tokens[:600], 0), (1, tokens[:1], 0), (2, tokens[200:], 200)], [list(range(600)), [0], list(range(700))])
+    check(out, torch.cat([want[:600], want[:1], want[200:]]), "bf16", "together")
+    check(eng.feed([(0, tokens[600:601], 600), (2, [5], 900)], [[0], []]), want[600:601], "bf16", "decode after")
+
+
 # ---- other sizes --------------------------------------------------------------------------------------------------------------------------
 SIZES = {
     "one head each": [M.attention(heads=1, kv_heads=1, dim=32, size=9, keep=1, ff=64), M.mlstm(heads=1, dim=16, vdim=16, cap=1.0, ff=33)],
