@@ -235,7 +235,7 @@ def _event_ms(fn, n: int) -> float:
 
 def measure_layered(path: str, steps: int, warmup: int, prompt: int, batches) -> dict:
     from oxibonsai_b200.runtime import EngineBuilder
-    eng = EngineBuilder().model_path(path).preset("greedy").max_seq_len(prompt + 1024).max_batch(max(batches)).kv_cache("bf16").build()
+    eng = EngineBuilder().model_path(path).preset("greedy").max_seq_len(prompt + 3 * (steps + warmup) + 64).max_batch(max(batches)).kv_cache("bf16").build()
     r, vocab = eng.runner, eng.config.vocab
     toks = torch.randint(0, vocab, (prompt,), generator=torch.Generator().manual_seed(1)).tolist()
     res = {"weight_GB": round(eng.weights.packed_bytes / 1e9, 3), "launches_per_step": r.kernel_launches(1)}
@@ -259,12 +259,12 @@ def measure_layered(path: str, steps: int, warmup: int, prompt: int, batches) ->
 
 def measure_generic(path: str, steps: int, warmup: int, prompt: int, batches) -> dict:
     from oxibonsai_b200.runtime.engine import GenericFormatEngine
-    eng = GenericFormatEngine(path, max_seq_len=prompt + 1024, max_batch=max(batches))
+    eng = GenericFormatEngine(path, max_seq_len=prompt + 3 * (steps + warmup) + 64, max_batch=max(batches))
     e = eng._eng
     toks = torch.randint(0, eng.config.vocab, (prompt,), generator=torch.Generator().manual_seed(1)).tolist()
     res = {"weight_GB": round(eng.model_info()["weight_bytes"] / 1e9, 3), "launches_per_step": e.kernel_launches_per_step(1)}
     for b in range(max(batches)):
-        eng.begin_sequence(toks, prompt + 900, b)
+        eng.begin_sequence(toks, prompt + 3 * (steps + warmup), b)
     dt = torch.tensor(toks, dtype=torch.int32, device="cuda")
     for _ in range(3):
         e.prefill(dt, 0, 0)
@@ -281,7 +281,7 @@ def measure_generic(path: str, steps: int, warmup: int, prompt: int, batches) ->
     return res
 
 
-def run_models(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64)) -> list[dict]:
+def run_models(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64), log=sys.stdout) -> list[dict]:
     from oxibonsai_b200.cli import requantize_gguf
     from oxibonsai_b200.core import Qwen3Config, write_synthetic_gguf
     rows = []
@@ -305,7 +305,7 @@ def run_models(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batc
         row = {"size": size, "width": width, "design_layers": len(cfg["layers"]), "generic_layers": layers, "params_M": round(params / 1e6),
                "generic_params_M": round((layers * per_layer + vocab * width) / 1e6), "design": ours, "generic_f16": like}
         rows.append(row)
-        print(json.dumps(row), flush=True)
+        print(json.dumps(row), file=log, flush=True)
     return rows
 
 

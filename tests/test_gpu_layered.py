@@ -254,6 +254,7 @@ SIZES = {
     "wide heads": [M.attention(heads=2, kv_heads=1, dim=256, scale=0.05, size=50, keep=5), M.mlstm(heads=2, dim=256, vdim=200)],
     "three quarters": [M.attention(heads=3, kv_heads=3, dim=96, scale=0.1), M.attention(heads=4, kv_heads=2, dim=192, scale=0.07, ff=31), M.mlstm(dim=128, vdim=64)],
     "long keys, many values": [M.mlstm(heads=1, dim=300, vdim=600), M.attention(heads=2, kv_heads=2, dim=17, size=300, keep=0)],
+    "nothing even": [M.mlstm(heads=3, dim=13, vdim=7, ff=21), M.attention(heads=9, kv_heads=3, dim=11, size=23, keep=2, ff=5)],
     "only recurrent": [M.mlstm(heads=2, dim=65, vdim=129, cap=30.0, ff=100)],
 }
 
@@ -261,7 +262,7 @@ SIZES = {
 @pytest.mark.parametrize("kv", ["f32", "bf16"])
 @pytest.mark.parametrize("name", SIZES)
 def test_sizes(tmp_path, name, kv):
-    m = M.Model(tmp_path / "m", M.config(SIZES[name], width=72 if name != "wide heads" else 264, vocab=97, eps=1e-6), seed=len(name))
+    m = M.Model(tmp_path / "m", M.config(SIZES[name], width={"wide heads": 264, "nothing even": 75}.get(name, 72), vocab=97, eps=1e-6), seed=len(name))
     eng = engine(m, kv, max_batch=2)
     poison(eng)
     tokens = m.tokens(140)
