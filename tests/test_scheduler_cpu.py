@@ -68,7 +68,7 @@ def _expected(prompt, n):
 
 
 def test_prompt_chunks_interleave_with_decode_steps():
-    eng = FakeEngine()
+    eng = FakeEngine(step_delay=0.01)                           # the first stream must still run when a loaded machine submits the second
     sched = BatchScheduler(eng, eos_token=-1, prefill_chunk_tokens=64)
     a = sched.submit(list(range(1, 21)), SamplingParams(), 40)
     sched.start()
