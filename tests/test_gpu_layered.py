@@ -70,7 +70,7 @@ def mixed_engine(request, mixed):
 
 # ---- projections -------------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("T", [1, 2, 8, 9, 16, 17, 32, 33, 64, 65, 300])
-@pytest.mark.parametrize("n,k", [(5, 40), (77, 152), (331, 384), (130, 1000)])
+@pytest.mark.parametrize("n,k", [(5, 40), (77, 152), (331, 384), (130, 1000), (301, 8200)])      # the last one is split along K between CTAs
 def test_linear(T, n, k):
     from oxibonsai_b200.ops import layered_ops as L
     g = torch.Generator().manual_seed(T * 1000 + n)
@@ -88,12 +88,12 @@ def test_linear(T, n, k):
         out = torch.full((T, n + 3), 7.0, device="cuda")[:, :n]
         L.linear(single, act, T, out, scratch)
         want = xd @ a.double().T
-        assert float((out.cpu().double() - want).abs().max()) < 2e-5
+        assert float((out.cpu().double() - want).abs().max()) < 2e-5 * max(1.0, k / 1000)      # f32 sums of k terms
         gl = torch.zeros(T, n, dtype=act.dtype, device="cuda")
         L.linear(pair, act, T, gl, scratch, (limit, alpha, offset))
         gg, uu = torch.clamp(want, max=limit), torch.clamp(xd @ b.double().T, -limit, limit)
         want = gg * torch.sigmoid(alpha * gg) * (uu + offset)
-        assert float((gl.cpu().double() - want).abs().max()) < (2e-5 if exact else 0.02)
+        assert float((gl.cpu().double() - want).abs().max()) < (2e-5 * max(1.0, k / 1000) if exact else 0.02)
     assert int(status.item()) == 0
 
 
