@@ -79,7 +79,7 @@ def bench_linear(rep: Report, width: int, iters: int, profile: bool) -> None:
             ws.append(w)
         for T in (1, 8, 32, 64, 256, 4096):
             x = torch.randn(T, k, device=dev).bfloat16()
-            glu = (7.0, 1.702, 1.0) if name == "gate_up" else None
+            glu = L.Glu(7.0, 1.702, 1.0) if name == "gate_up" else None
             out = torch.empty(T, n // 2 if glu else n, dtype=torch.bfloat16 if glu else torch.float32, device=dev)
             it = [0]
 
@@ -121,8 +121,8 @@ def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
         proj = torch.randn(B, ld, device=dev)
         w1, slopes = torch.ones(hd, device=dev), torch.full((nq,), 0.01, device=dev)
         out = torch.zeros(B, nq * hd, dtype=torch.bfloat16, device=dev)
-        calls = [L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, p, rk, out], [ld, 0, nq * hd, (nq + nkv) * hd, nq * hd, nq, nkv, hd, npages, page, 0, 0],
-                             [1e-6, hd ** -0.5]) for p in pools]
+        calls = [L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, p, rk, None, out],
+                             [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, 0, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0]) for p in pools]
         it = [0]
         split = 1
         while split < 8 and B * nkv * split * 2 <= 160:
@@ -148,8 +148,8 @@ def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
     entries = torch.tensor([0, T, 0, 0], **i32)
     tiles = torch.tensor([[0, t] for t in range(0, T, tpt)], **i32)
     for window in (0, 1024):
-        call = L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, pool, rk, out], [ld, 0, nq * hd, (nq + nkv) * hd, nq * hd, nq, nkv, hd, npages, page, window, 4],
-                           [1e-6, hd ** -0.5])
+        call = L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, pool, rk, None, out],
+                           [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, window, 4], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0])
 
         def ours():
             K.check(L.lib().bonsai_lay_attn_prompt(*call.args, entries.data_ptr(), tiles.data_ptr(), len(tiles), K.stream()), "attn_prompt")
@@ -211,7 +211,7 @@ def bench_mlstm(rep: Report, width: int, iters: int, profile: bool) -> None:
         rep.add("mlstm_chunk", f"{nseq} x {T} tokens heads={H} {d}x{e} segments={len(segs)}", time_us(fn, 10, profile), 4.0 * rows * H * (2 * d + 2 * e), 4.0 * rows * H * d * e)
         act = torch.zeros(rows, H * e, dtype=torch.bfloat16, device=dev)
         gate = torch.randn(rows, ld, device=dev)
-        rep.add("gated_head_norm", f"T={rows}", time_us(lambda: L.gated_head_norm(out, 0, gate, 0, norm, 1e-6, rows, H, e, act), iters, profile), 10.0 * rows * H * e)
+        rep.add("gated_head_norm", f"T={rows}", time_us(lambda: L.gated_norm(out, 0, gate, 0, norm, 1e-6, rows, H, e, act), iters, profile), 10.0 * rows * H * e)
     for T in (1, 64, 4096):
         x, y, w = torch.randn(T, width, device=dev), torch.randn(T, width, device=dev), torch.ones(width, device=dev)
         x16 = torch.zeros(T, width, dtype=torch.bfloat16, device=dev)

@@ -156,7 +156,11 @@ def model_dir_info(path: str) -> dict:
     cfg = load_model_dir_config(path)
     v = validate_model_dir(path)
     weights = Path(path) / "model.safetensors"
-    layers = [{"mixer": s.mixer.kind, **{k: x for k, x in vars(s.mixer).items()}, "mlp": None if s.mlp is None else dict(vars(s.mlp))} for s in cfg.layer_specs]
+    fields = lambda spec: {k: vars(x) if k == "rotary" and x is not None else x for k, x in vars(spec).items() if k != "parts"}
+    layers = []
+    for s in cfg.layer_specs:
+        parts = [{"prefix": b.prefix, "output_scale": b.scale, "mixer": b.spec.kind, **fields(b.spec)} for b in s.mixer.branches if b.prefix]
+        layers.append({"mixer": s.mixer.kind, **fields(s.mixer), **({"parts": parts} if parts else {}), "mlp": None if s.mlp is None else dict(vars(s.mlp))})
     return {"path": path, "gpu_engine": "layer-list engine", "architecture": cfg.arch, "name": cfg.name, "quantization": "BF16",
             "tensors": len(cfg.tensor_shapes()), "estimated_parameters": cfg.param_count(),
             "file_size_bytes": os.path.getsize(weights) if weights.exists() else 0,

@@ -134,6 +134,7 @@ __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, 
     const size_t o = (size_t)tok * p.out_ld + row;
     if (p.epi == 0) p.out_f32[o] = v;
     else if (p.epi == 1) p.out_f32[o] = res + v;
+    else if (p.epi == 5) reinterpret_cast<__nv_bfloat16*>(p.out_f16)[o] = __float2bfloat16_rn(fmaxf(v, 0.0f) * fmaxf(v, 0.0f));
     else p.out_f16[o] = __float2half_rn(v);
   }
 }
@@ -643,12 +644,12 @@ int bonsai_bitgemm_prefill_ws(const void* codes, const void* scales, const void*
 }
 
 // Dense bf16 operands: W [n_rows][K] (K a multiple of 128), x [T][x_ld], f32 accumulation.  epi 0: out_f32 = W x; 4: out_bf16 =
-// clamped gated unit over interleaved gate / up rows (n_rows / 2 columns).  Workspace and status as above.
+// clamped gated unit over interleaved gate / up rows (n_rows / 2 columns); 5: out_bf16 = relu(W x)^2.  Workspace and status as above.
 int bonsai_dense_gemm_bf16(const void* w, int n_rows, int K, const void* x, int x_ld, int T, float* out_f32, void* out_bf16, int out_ld, int epi,
                            float limit, float alpha, float offset, int* status, void* ws, size_t ws_bytes, int sms, cudaStream_t stream) {
   using namespace bonsai;
-  if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && epi != 4)) return BONSAI_CUDA_BAD_ARG;
-  if ((epi == 0 && out_f32 == nullptr) || (epi == 4 && (out_bf16 == nullptr || n_rows % 2 != 0)) || status == nullptr) return BONSAI_CUDA_BAD_ARG;
+  if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && epi != 4 && epi != 5)) return BONSAI_CUDA_BAD_ARG;
+  if ((epi == 0 && out_f32 == nullptr) || (epi != 0 && out_bf16 == nullptr) || (epi == 4 && n_rows % 2 != 0) || status == nullptr) return BONSAI_CUDA_BAD_ARG;
   const int tok = T <= 64 ? 64 : 256;
   CUtensorMap xmap, amap;
   if (!make_map_f16(&xmap, x, K, T, x_ld, tok, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||

@@ -1,12 +1,16 @@
-// Attention of the layer-list decoders over a paged cache whose rows are both key and value.
+// Attention of the layer-list decoders over a paged cache.  Queries and keys are divided by their root mean square; everything
+// else is a parameter that a design may leave out:
 //
-// The design's values are its un-normalised keys, so one cache row per token and kv head serves both products: the row holds
-// the projected key, and a float beside it the reciprocal root mean square of the key norm.  The norm's weight and the score
-// scale are folded into the query (q' = norm(q) * w_q * w_k * scale), the key's root mean square multiplies the score of its
-// column.  That halves the cache traffic of separate K and V rows, and a tile is staged once for S = Q K^T and O = P K.
+//   score(i, j) = cap(q'_i . k'_j) - slope_h (i - j)       j <= i and (i - j < window or j < keep)
+//   out         = softmax(score) V * sigmoid(gate_h) * out_scale
 //
-//   score(i, j) = q'_i . k_j * rk_j - slope_h (i - j)      j <= i and (i - j < window or j < keep)
-//   out         = softmax(score) K * sigmoid(gate_h)
+// with q' = norm(q) [* w_q * w_k] * scale [* (1 + coef ln(floor((i + 1) / every) + 1))] and cap(s) = s or c tanh(s / c).
+//
+// Two kinds of cache rows (template parameter SEP):
+//  * one row per token that is both key and value (designs whose values are the un-normalised keys): the row holds the projected
+//    key, a float beside it the reciprocal root mean square, which multiplies the scores of its column.  Half the cache traffic
+//    of separate rows, and a tile is staged once for S = Q K^T and O = P K;
+//  * SEP: a row of normalised keys and a row of values, both padded to the same row length.
 //
 // Rows of a batch are tokens: a row has a position and a slot (its sequence's block-table row).  `append_kernel` writes the
 // rows' keys; `prompt_kernel` handles portions of prompts (tiles of 64 query rows = tokens x heads of one kv group);
@@ -21,20 +25,33 @@ namespace lay {
 
 struct Attn {
   const float* proj;        // [T][ld]: q heads at q_col, k heads at k_col, one gate per head at g_col
-  const float* q_norm;      // [dim]
+  const float* q_norm;      // [dim]; null: no norm weights
   const float* k_norm;      // [dim]
-  const float* slopes;      // [heads]
+  const float* slopes;      // [heads]; null: no distance bias
   const int* pos;           // [T]
   const int* slots;         // [T]
   const int* block_table;   // [slots][max_pages]
   void* pool;               // [pages][kv_heads][page_size][HD], bf16 (f32 in the 32-bit mode), columns past dim zero
-  float* krms;              // [pages][kv_heads][page_size]
-  void* out;                // [T][ldo], head h at h * dim
-  int ld, q_col, k_col, g_col, ldo;
-  int heads, kv_heads, dim, max_pages, pshift;   // page size 1 << pshift
+  float* krms;              // [pages][kv_heads][page_size]; SEP: unused
+  void* vpool;              // SEP: value rows, laid out like the pool
+  void* out;                // [T][ldo], head h at h * vdim
+  int ld, q_col, k_col, v_col, g_col, ldo;       // g_col < 0: no gate
+  int heads, kv_heads, dim, vdim, max_pages, pshift;   // page size 1 << pshift
   int window, keep;         // window <= 0: no window
-  float eps, scale;
+  float eps, scale, out_scale;
+  float softcap;            // <= 0: scores are not capped
+  float temp_coef, temp_every;   // query temperature; coef 0: none
 };
+
+__device__ __forceinline__ float temperature(const Attn& a, int pos) {
+  return a.temp_coef == 0.0f ? 1.0f : 1.0f + a.temp_coef * logf(floorf((float)(pos + 1) / a.temp_every) + 1.0f);
+}
+__device__ __forceinline__ float gate(const Attn& a, size_t t, int head) {
+  return a.g_col < 0 ? a.out_scale : a.out_scale * sigmoid(a.proj[t * a.ld + a.g_col + head]);
+}
+// Scores arrive as base-2 logarithms, or with a cap as x = 2 log2(e) score / cap: cap * tanh(score / cap) * log2(e) from one
+// exponential, tanh(y) = 1 - 2 / (e^2y + 1).
+__device__ __forceinline__ float cap_score(float x, float cap_log2e) { return cap_log2e - __fdividef(2.0f * cap_log2e, ex2(x) + 1.0f); }
 
 // first visible position outside the kept ones for a query at `p`
 __device__ __forceinline__ int window_lo(const Attn& a, int p) { return a.window > 0 ? max(0, p - a.window + 1) : 0; }
@@ -43,10 +60,27 @@ __device__ __forceinline__ size_t cache_row(const Attn& a, const int* bt, int kv
   return ((((size_t)bt[t >> a.pshift] * a.kv_heads + kvh) << a.pshift)) + (t & ((1 << a.pshift) - 1));
 }
 
-// A warp writes one key row and its reciprocal root mean square.
-template <int HD, typename C>
-__device__ __forceinline__ void append_row(const Attn& a, const float* k, size_t row, int lane) {
+// A warp writes one token's row of kv head kvh: the key and its reciprocal root mean square, or the normalised key and the value.
+template <int HD, bool SEP, typename C>
+__device__ __forceinline__ void append_row(const Attn& a, const float* proj, int kvh, size_t row, int lane) {
   C* dst = static_cast<C*>(a.pool) + row * HD;
+  const float* k = proj + a.k_col + kvh * a.dim;
+  if constexpr (SEP) {
+    const float* v = proj + a.v_col + kvh * a.vdim;
+    C* vdst = static_cast<C*>(a.vpool) + row * HD;
+    float x[HD / 32], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < HD / 32; ++i) {
+      const int d = lane + 32 * i;
+      x[i] = d < a.dim ? k[d] : 0.0f;
+      store_act(vdst + d, d < a.vdim ? v[d] : 0.0f);
+      ss += x[i] * x[i];
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+#pragma unroll
+    for (int i = 0; i < HD / 32; ++i) store_act(dst + lane + 32 * i, x[i] * inv);
+    return;
+  }
   float ss = 0.0f;
 #pragma unroll
   for (int d = lane; d < HD; d += 32) {
@@ -59,7 +93,7 @@ __device__ __forceinline__ void append_row(const Attn& a, const float* k, size_t
 }
 
 // grid (row groups of 4 x kv head): one warp per (row of the list, kv head)
-template <int HD, typename C>
+template <int HD, bool SEP, typename C>
 __global__ void append_kernel(Attn a, int first, int count) {
   pdl_wait();
   pdl_trigger();
@@ -68,12 +102,13 @@ __global__ void append_kernel(Attn a, int first, int count) {
   const int t = first + i;
   if (a.pos[t] >= (a.max_pages << a.pshift)) return;
   const int* bt = a.block_table + (size_t)a.slots[t] * a.max_pages;
-  append_row<HD, C>(a, a.proj + (size_t)t * a.ld + a.k_col + kvh * a.dim, cache_row(a, bt, kvh, a.pos[t]), lane);
+  append_row<HD, SEP, C>(a, a.proj + (size_t)t * a.ld, kvh, cache_row(a, bt, kvh, a.pos[t]), lane);
 }
 
-// A warp normalises one query head and leaves q' * log2(e) in dst (columns past dim zero): scores are base-2 logarithms.
+// A warp normalises one query head and leaves q' * log2(e) in dst (columns past dim zero): scores are base-2 logarithms; with
+// a cap, q' * 2 log2(e) / cap.
 template <int HD>
-__device__ __forceinline__ void load_query(const Attn& a, const float* q, bf16* dst, int lane) {
+__device__ __forceinline__ void load_query(const Attn& a, const float* q, int pos, bf16* dst, int lane) {
   float v[HD / 32], ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < HD / 32; ++i) {
@@ -82,25 +117,27 @@ __device__ __forceinline__ void load_query(const Attn& a, const float* q, bf16* 
     ss += v[i] * v[i];
   }
   ss = warp_sum(ss);
-  const float f = a.scale * kLog2e / sqrtf(ss / (float)a.dim + a.eps);
+  const float f = a.scale * temperature(a, pos) * (a.softcap > 0.0f ? 2.0f * kLog2e / a.softcap : kLog2e) / sqrtf(ss / (float)a.dim + a.eps);
 #pragma unroll
   for (int i = 0; i < HD / 32; ++i) {
     const int d = lane + 32 * i;
-    dst[d] = __float2bfloat16_rn(d < a.dim ? v[i] * f * a.q_norm[d] * a.k_norm[d] : 0.0f);
+    const float w = d < a.dim && a.q_norm != nullptr ? a.q_norm[d] * a.k_norm[d] : 1.0f;
+    dst[d] = __float2bfloat16_rn(v[i] * f * w);
   }
 }
 
 // ---- portions of prompts ------------------------------------------------------------------------------------------------------
 // entries[e] = {first row, tokens, slot, first position}; tiles[i] = {entry, first token of the tile}.  A tile holds
 // 64 / G tokens x the G query heads of one kv head.
-template <int HD>
+template <int HD, bool SEP>
 __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries, const int2* tiles) {
   constexpr int LD = HD + 8;
   constexpr bool kQReg = HD <= 128;   // query fragments stay in registers (else they are re-read from shared memory)
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16* sQ = reinterpret_cast<bf16*>(smem_raw);
   bf16* sK = sQ + 64 * LD;            // two stages of [64][LD]
-  float* sR = reinterpret_cast<float*>(sK + 2 * 64 * LD);   // two stages of 64 key factors
+  bf16* sV = sK + 2 * 64 * LD;        // SEP: two stages of [64][LD]
+  float* sR = reinterpret_cast<float*>(sK + 2 * 64 * LD);   // otherwise two stages of 64 key factors
   const int kvh = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int G = a.heads / a.kv_heads, tpt = 64 / G;
   pdl_wait();
@@ -119,9 +156,11 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
     for (int i = threadIdx.x; i < 64 * (HD / 8); i += 128) {
       const int r = i / (HD / 8), c = (i % (HD / 8)) * 8, t = kb + r;
       const bool ok = t < hi;
-      cp_async16(dst + r * LD + c, pool + (ok ? cache_row(a, bt, kvh, t) * HD + c : 0), ok);
+      const size_t at = ok ? cache_row(a, bt, kvh, t) * HD + c : 0;
+      cp_async16(dst + r * LD + c, pool + at, ok);
+      if (SEP) cp_async16(sV + st * 64 * LD + r * LD + c, static_cast<const bf16*>(a.vpool) + at, ok);
     }
-    if (threadIdx.x < 64) sR[st * 64 + threadIdx.x] = kb + threadIdx.x < hi ? a.krms[cache_row(a, bt, kvh, kb + threadIdx.x)] : 0.0f;
+    if (!SEP && threadIdx.x < 64) sR[st * 64 + threadIdx.x] = kb + threadIdx.x < hi ? a.krms[cache_row(a, bt, kvh, kb + threadIdx.x)] : 0.0f;
   };
   // key tiles: those that hold kept tokens, then those of the window's range
   auto next = [&](int kb) {
@@ -134,7 +173,7 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
   cp_async_commit();
   for (int r = warp * 16; r < warp * 16 + 16; ++r) {
     if (r < rows) {
-      load_query<HD>(a, a.proj + (size_t)(en.x + q0 + r / G) * a.ld + a.q_col + (kvh * G + r % G) * a.dim, sQ + r * LD, lane);
+      load_query<HD>(a, a.proj + (size_t)(en.x + q0 + r / G) * a.ld + a.q_col + (kvh * G + r % G) * a.dim, pfirst + r / G, sQ + r * LD, lane);
     } else {
       for (int d = lane; d < HD; d += 32) sQ[r * LD + d] = __float2bfloat16_rn(0.0f);
     }
@@ -156,10 +195,11 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
     row[e] = warp * 16 + (lane >> 2) + 8 * e;
     qpos[e] = row[e] < rows ? pfirst + row[e] / G : -1;      // rows past the tile see nothing
     head[e] = kvh * G + row[e] % G;
-    slope[e] = a.slopes[head[e]] * kLog2e;
+    slope[e] = a.slopes == nullptr ? 0.0f : a.slopes[head[e]] * kLog2e;
   }
   const int wfirst = pfirst + warp * 16 / G, wlast = min(plast, pfirst + (warp * 16 + 15) / G);   // positions of this warp's rows
   const bool wlive = warp * 16 + 15 < rows;
+  const float cap = a.softcap * kLog2e;
   for (int it = 0; kb < hi; ++it) {
     const int nx = next(kb);
     if (nx < hi) fetch(nx, (it + 1) & 1);
@@ -167,6 +207,7 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
     cp_async_wait<1>();
     __syncthreads();
     const bf16* k = sK + (it & 1) * 64 * LD;
+    const bf16* v = SEP ? sV + (it & 1) * 64 * LD : k;
     const float* kr = sR + (it & 1) * 64;
     float s[8][4];
 #pragma unroll
@@ -188,11 +229,13 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) {
       const int c = nt * 8 + (lane & 3) * 2;
-      const float2 f = *reinterpret_cast<const float2*>(kr + c);
+      const float2 f = SEP ? make_float2(1.0f, 1.0f) : *reinterpret_cast<const float2*>(kr + c);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = e >> 1, j = kb + c + (e & 1);
-        s[nt][e] = s[nt][e] * ((e & 1) ? f.y : f.x) - slope[r] * (float)(qpos[r] - j);
+        if (!SEP) s[nt][e] *= (e & 1) ? f.y : f.x;
+        if (a.softcap > 0.0f) s[nt][e] = cap_score(s[nt][e], cap);
+        s[nt][e] -= slope[r] * (float)(qpos[r] - j);
         if (!whole && !sees(a, qpos[r], j)) s[nt][e] = -INFINITY;
         nm[r] = fmaxf(nm[r], s[nt][e]);
       }
@@ -230,7 +273,7 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
 #pragma unroll
       for (int np = 0; np < HD / 16; ++np) {
         uint32_t b[4];
-        ldsm4_t(b, frag_b_cols(k, LD, ks * 16, np * 16, lane));
+        ldsm4_t(b, frag_b_cols(v, LD, ks * 16, np * 16, lane));
         mma_bf16(o[2 * np], pa, b[0], b[1]);
         mma_bf16(o[2 * np + 1], pa, b[2], b[3]);
       }
@@ -245,13 +288,13 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
     if (row[r] >= rows) continue;
     const size_t t = en.x + q0 + row[r] / G;
-    const float f = sigmoid(a.proj[t * a.ld + a.g_col + head[r]]) / l[r];   // the query's own position is always visible
-    bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + head[r] * a.dim;
+    const float f = gate(a, t, head[r]) / l[r];   // the query's own position is always visible
+    bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + head[r] * a.vdim;
 #pragma unroll
     for (int nt = 0; nt < HD / 8; ++nt) {
       const int d = nt * 8 + (lane & 3) * 2;
-      if (d < a.dim) dst[d] = __float2bfloat16_rn(o[nt][2 * r] * f);
-      if (d + 1 < a.dim) dst[d + 1] = __float2bfloat16_rn(o[nt][2 * r + 1] * f);
+      if (d < a.vdim) dst[d] = __float2bfloat16_rn(o[nt][2 * r] * f);
+      if (d + 1 < a.vdim) dst[d + 1] = __float2bfloat16_rn(o[nt][2 * r + 1] * f);
     }
   }
 }
@@ -260,16 +303,19 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
 // grid (kv heads x groups of 16 query heads, splits, rows); the splits of one row form a cluster and meet in distributed
 // shared memory.  A warp walks 16-token tiles of the visible range; the split that holds the row's own position appends its
 // key before it reads it.
-constexpr int decode_stages(int hd) { return hd <= 128 ? 4 : 2; }   // key tiles a warp keeps in flight, one of them in use
+// tiles a warp keeps in flight, one of them in use; warps of a CTA
+constexpr int decode_stages(int hd, bool sep) { return sep ? (hd <= 64 ? 4 : (hd <= 192 ? 3 : 2)) : (hd <= 128 ? 4 : 2); }
+constexpr int decode_warps(int hd, bool sep) { return sep && hd > 128 ? 4 : 8; }
 
-template <int HD>
-__global__ void __launch_bounds__(256) decode_kernel(Attn a) {
-  constexpr int LD = HD + 8, NW = 8, NST = decode_stages(HD);
+template <int HD, bool SEP>
+__global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn a) {
+  constexpr int LD = HD + 8, NW = decode_warps(HD, SEP), NTH = 32 * NW, NST = decode_stages(HD, SEP);
   constexpr int kTile = 16 * LD;      // elements of a tile
+  constexpr int kStage = SEP ? 2 * kTile : kTile;   // keys, then values
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                    // [16][LD]
   float* res = reinterpret_cast<float*>(sQ + kTile);               // this CTA's merged rows [16][HD + 2]
-  bf16* tiles = reinterpret_cast<bf16*>(res + 16 * (HD + 2));      // [warp][stage][16][LD], later the warps' partial rows
+  bf16* tiles = reinterpret_cast<bf16*>(res + 16 * (HD + 2));      // [warp][stage][tile], later the warps' partial rows
   float* part = reinterpret_cast<float*>(tiles);                   // [warp][16][HD + 2]
   namespace cg = cooperative_groups;
   cg::cluster_group cluster = cg::this_cluster();
@@ -293,8 +339,8 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
   const int per = (ntiles + nsplit - 1) / nsplit;
   const int b0 = split * per, b1 = min(ntiles, b0 + per);
   const bool owner = b1 == ntiles && b0 < b1;                            // holds the last tile: the row's own position
-  bf16* wt = tiles + warp * NST * kTile;
-  float* wf = reinterpret_cast<float*>(tiles + NW * NST * kTile) + warp * NST * 16;   // key factors of the tiles
+  bf16* wt = tiles + warp * NST * kStage;
+  float* wf = reinterpret_cast<float*>(tiles + NW * NST * kStage) + warp * NST * 16;   // key factors of the tiles
   auto first_token = [&](int j) { return (j < nkeep ? j : lo16 + j - nkeep) << 4; };
   auto issue = [&](int j, int st) {     // a tile lies in one page: its rows and factors are contiguous
     const int tb = first_token(j);
@@ -302,9 +348,10 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
 #pragma unroll
     for (int i = 0; i < 16 * (HD / 8) / 32; ++i) {
       const int idx = lane + 32 * i, r = idx / (HD / 8), c = (idx % (HD / 8)) * 8;
-      cp_async16(wt + st * kTile + r * LD + c, pool + (row + r) * HD + c, tb + r <= pos);
+      cp_async16(wt + st * kStage + r * LD + c, pool + (row + r) * HD + c, tb + r <= pos);
+      if (SEP) cp_async16(wt + st * kStage + kTile + r * LD + c, static_cast<const bf16*>(a.vpool) + (row + r) * HD + c, tb + r <= pos);
     }
-    if (lane < 4) cp_async16(wf + st * 16 + lane * 4, a.krms + row + lane * 4, true);
+    if (!SEP && lane < 4) cp_async16(wf + st * 16 + lane * 4, a.krms + row + lane * 4, true);
   };
   const int j0 = b0 + warp;
   auto is_new = [&](int j) { return owner && j == b1 - 1; };              // the tile that receives the row's own key
@@ -315,11 +362,11 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
   pdl_trigger();
   const float* prow = a.proj + (size_t)t * a.ld;
   for (int r = warp; r < 16 + (owner ? 1 : 0); r += NW) {
-    if (r < nh) load_query<HD>(a, prow + a.q_col + (kvh * G + h0 + r) * a.dim, sQ + r * LD, lane);
+    if (r < nh) load_query<HD>(a, prow + a.q_col + (kvh * G + h0 + r) * a.dim, pos, sQ + r * LD, lane);
     else if (r < 16)
       for (int d = lane; d < HD; d += 32) sQ[r * LD + d] = __float2bfloat16_rn(0.0f);
     else {
-      append_row<HD, bf16>(a, prow + a.k_col + kvh * a.dim, cache_row(a, bt, kvh, pos), lane);
+      append_row<HD, SEP, bf16>(a, prow, kvh, cache_row(a, bt, kvh, pos), lane);
       __threadfence();
     }
   }
@@ -331,7 +378,8 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
   const int g = lane >> 2;
   float slope[2];
 #pragma unroll
-  for (int r = 0; r < 2; ++r) slope[r] = a.slopes[kvh * G + h0 + min(g + 8 * r, nh - 1)] * kLog2e;
+  for (int r = 0; r < 2; ++r) slope[r] = a.slopes == nullptr ? 0.0f : a.slopes[kvh * G + h0 + min(g + 8 * r, nh - 1)] * kLog2e;
+  const float cap = a.softcap * kLog2e;
 #pragma unroll
   for (int st = 0; st < NST - 1; ++st) {
     if (j0 + st * NW < b1 && is_new(j0 + st * NW)) issue(j0 + st * NW, st);
@@ -349,7 +397,8 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
     __syncwarp();
     if (j + (NST - 1) * NW < b1) issue(j + (NST - 1) * NW, (it + NST - 1) % NST);
     cp_async_commit();
-    const bf16* k = wt + (it % NST) * kTile;
+    const bf16* k = wt + (it % NST) * kStage;
+    const bf16* v = SEP ? k + kTile : k;
     const float* kf = wf + (it % NST) * 16;
     const int tb = first_token(j);
     float s[2][4] = {};
@@ -367,7 +416,9 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int c = nt * 8 + (lane & 3) * 2 + (e & 1), j1 = tb + c;
-        s[nt][e] = s[nt][e] * kf[c] - slope[e >> 1] * (float)(pos - j1);
+        if (!SEP) s[nt][e] *= kf[c];
+        if (a.softcap > 0.0f) s[nt][e] = cap_score(s[nt][e], cap);
+        s[nt][e] -= slope[e >> 1] * (float)(pos - j1);
         if (!sees(a, pos, j1)) s[nt][e] = -INFINITY;
         nm[e >> 1] = fmaxf(nm[e >> 1], s[nt][e]);
       }
@@ -400,7 +451,7 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
 #pragma unroll
     for (int np = 0; np < HD / 16; ++np) {
       uint32_t b[4];
-      ldsm4_t(b, frag_b_cols(k, LD, 0, np * 16, lane));
+      ldsm4_t(b, frag_b_cols(v, LD, 0, np * 16, lane));
       mma_bf16(o[2 * np], pa, b[0], b[1]);
       mma_bf16(o[2 * np + 1], pa, b[2], b[3]);
     }
@@ -426,7 +477,7 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < nh * HD; i += 256) {
+  for (int i = threadIdx.x; i < nh * HD; i += NTH) {
     const int r = i / HD, d = i % HD;
     float M = -INFINITY, acc = 0.0f, L = 0.0f;
 #pragma unroll
@@ -447,8 +498,8 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
   if (nsplit > 1) cluster.sync();
   else __syncthreads();
   // every CTA of the cluster finishes its share of the outputs
-  for (int i = split * 256 + threadIdx.x; i < nh * a.dim; i += nsplit * 256) {
-    const int r = i / a.dim, d = i % a.dim;
+  for (int i = split * NTH + threadIdx.x; i < nh * a.vdim; i += nsplit * NTH) {
+    const int r = i / a.vdim, d = i % a.vdim;
     float M = -INFINITY, acc = 0.0f, L = 0.0f;
     for (int s = 0; s < nsplit; ++s) M = fmaxf(M, (nsplit > 1 ? cluster.map_shared_rank(res, s) : res)[r * ST + HD]);
     for (int s = 0; s < nsplit; ++s) {
@@ -458,14 +509,14 @@ __global__ void __launch_bounds__(256) decode_kernel(Attn a) {
       L += f * src[HD + 1];
     }
     const int h = kvh * G + h0 + r;
-    static_cast<bf16*>(a.out)[(size_t)t * a.ldo + h * a.dim + d] = __float2bfloat16_rn(acc / L * sigmoid(prow[a.g_col + h]));
+    static_cast<bf16*>(a.out)[(size_t)t * a.ldo + h * a.vdim + d] = __float2bfloat16_rn(acc / L * gate(a, t, h));
   }
   if (nsplit > 1) cluster.sync();   // nobody leaves while its rows are being read
 }
 
 // ---- 32-bit mode ------------------------------------------------------------------------------------------------------------------
 // grid (heads, rows): four warps take the visible keys in turn, exact f32 products and exponentials
-template <int HD>
+template <int HD, bool SEP>
 __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
   __shared__ float sm[4][HD + 2];
   pdl_wait();
@@ -489,9 +540,10 @@ __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
 #pragma unroll
   for (int i = 0; i < HD / 32; ++i) {
     const int d = lane + 32 * i;
-    q[i] = d < a.dim ? q[i] * rq * a.q_norm[d] * a.k_norm[d] : 0.0f;
+    const float w = d < a.dim && a.q_norm != nullptr ? a.q_norm[d] * a.k_norm[d] : 1.0f;
+    q[i] *= rq * w;
   }
-  const float slope = a.slopes[h];
+  const float slope = a.slopes == nullptr ? 0.0f : a.slopes[h], scale = a.scale * temperature(a, pos);
   float m = -INFINITY, l = 0.0f;
   const int lo = window_lo(a, pos), nkeep = min(a.window > 0 ? a.keep : 0, lo);
   for (int i = warp; i < nkeep + pos + 1 - lo; i += 4) {
@@ -503,12 +555,14 @@ __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
       k[c] = pool[row * HD + lane + 32 * c];
       s = fmaf(q[c], k[c], s);
     }
-    s = warp_sum(s) * a.krms[row] * a.scale - slope * (float)(pos - j);
+    s = warp_sum(s) * scale * (SEP ? 1.0f : a.krms[row]);
+    if (a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
+    s -= slope * (float)(pos - j);
     const float nm = fmaxf(m, s), f = expf(m - nm), p = expf(s - nm);
     m = nm;
     l = l * f + p;
 #pragma unroll
-    for (int c = 0; c < HD / 32; ++c) o[c] = o[c] * f + p * k[c];
+    for (int c = 0; c < HD / 32; ++c) o[c] = o[c] * f + p * (SEP ? static_cast<const float*>(a.vpool)[row * HD + lane + 32 * c] : k[c]);
   }
 #pragma unroll
   for (int c = 0; c < HD / 32; ++c) sm[warp][lane + 32 * c] = o[c];
@@ -520,36 +574,38 @@ __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
   float M = -INFINITY, L = 0.0f;
   for (int w = 0; w < 4; ++w) M = fmaxf(M, sm[w][HD]);
   for (int w = 0; w < 4; ++w) L += expf(sm[w][HD] - M) * sm[w][HD + 1];
-  const float f = sigmoid(a.proj[(size_t)t * a.ld + a.g_col + h]) / L;
-  for (int d = threadIdx.x; d < a.dim; d += 128) {
+  const float f = gate(a, t, h) / L;
+  for (int d = threadIdx.x; d < a.vdim; d += 128) {
     float acc = 0.0f;
     for (int w = 0; w < 4; ++w) acc += expf(sm[w][HD] - M) * sm[w][d];
-    static_cast<float*>(a.out)[(size_t)t * a.ldo + h * a.dim + d] = acc * f;
+    static_cast<float*>(a.out)[(size_t)t * a.ldo + h * a.vdim + d] = acc * f;
   }
 }
 
-template <int HD>
+template <int HD, bool SEP>
 static int run_append(const Attn& a, int first, int count, int f32, cudaStream_t stream) {
   const dim3 grid((count + 3) / 4, a.kv_heads);
-  return f32 ? launch(append_kernel<HD, float>, grid, 128, 0, stream, 1, 0, a, first, count)
-             : launch(append_kernel<HD, bf16>, grid, 128, 0, stream, 1, 0, a, first, count);
+  return f32 ? launch(append_kernel<HD, SEP, float>, grid, 128, 0, stream, 1, 0, a, first, count)
+             : launch(append_kernel<HD, SEP, bf16>, grid, 128, 0, stream, 1, 0, a, first, count);
 }
-template <int HD>
+template <int HD, bool SEP>
 static int run_prompt(const Attn& a, const int* entries, const int* tiles, int ntiles, cudaStream_t stream) {
-  const size_t smem = (size_t)3 * 64 * (HD + 8) * sizeof(bf16) + 128 * sizeof(float);
-  cudaFuncSetAttribute(prompt_kernel<HD>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
-  return launch(prompt_kernel<HD>, dim3(a.kv_heads, ntiles), 128, smem, stream, 1, 0, a, (const int4*)entries, (const int2*)tiles);
+  const size_t smem = (size_t)(SEP ? 5 : 3) * 64 * (HD + 8) * sizeof(bf16) + (SEP ? 0 : 128 * sizeof(float));
+  cudaFuncSetAttribute(prompt_kernel<HD, SEP>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
+  return launch(prompt_kernel<HD, SEP>, dim3(a.kv_heads, ntiles), 128, smem, stream, 1, 0, a, (const int4*)entries, (const int2*)tiles);
 }
-template <int HD>
+template <int HD, bool SEP>
 static int run_decode(const Attn& a, int nrows, int nsplit, cudaStream_t stream) {
   const int mg = (a.heads / a.kv_heads + 15) / 16;
-  const size_t smem = (size_t)16 * (HD + 8) * sizeof(bf16) * (1 + 8 * decode_stages(HD)) + (size_t)16 * (HD + 2) * sizeof(float) +
-                      (size_t)8 * decode_stages(HD) * 16 * sizeof(float);
-  return launch(decode_kernel<HD>, dim3(a.kv_heads * mg, nsplit, nrows), 256, smem, stream, nsplit, 1, a);
+  constexpr int NW = decode_warps(HD, SEP), NST = decode_stages(HD, SEP);
+  constexpr size_t smem = (size_t)16 * (HD + 8) * sizeof(bf16) * (1 + NW * NST * (SEP ? 2 : 1)) + (size_t)16 * (HD + 2) * sizeof(float) +
+                          (SEP ? 0 : (size_t)NW * NST * 16 * sizeof(float));
+  static_assert(smem <= 227 * 1024, "shared memory of a CTA");
+  return launch(decode_kernel<HD, SEP>, dim3(a.kv_heads * mg, nsplit, nrows), 32 * NW, smem, stream, nsplit, 1, a);
 }
-template <int HD>
+template <int HD, bool SEP>
 static int run_f32(const Attn& a, int T, cudaStream_t stream) {
-  return launch(f32_kernel<HD>, dim3(a.heads, T), 128, 0, stream, 1, 0, a);
+  return launch(f32_kernel<HD, SEP>, dim3(a.heads, T), 128, 0, stream, 1, 0, a);
 }
 
 static int padded_dim(int dim) {
@@ -562,24 +618,32 @@ static int padded_dim(int dim) {
 static bool fill(Attn& a, const void* const* ptrs, const int* ints, const float* floats) {
   a.proj = (const float*)ptrs[0]; a.q_norm = (const float*)ptrs[1]; a.k_norm = (const float*)ptrs[2]; a.slopes = (const float*)ptrs[3];
   a.pos = (const int*)ptrs[4]; a.slots = (const int*)ptrs[5]; a.block_table = (const int*)ptrs[6]; a.pool = const_cast<void*>(ptrs[7]);
-  a.krms = (float*)ptrs[8]; a.out = const_cast<void*>(ptrs[9]);
-  a.ld = ints[0]; a.q_col = ints[1]; a.k_col = ints[2]; a.g_col = ints[3]; a.ldo = ints[4]; a.heads = ints[5]; a.kv_heads = ints[6];
-  a.dim = ints[7]; a.max_pages = ints[8];
-  for (a.pshift = 0; (2 << a.pshift) <= ints[9]; ++a.pshift) {} a.window = ints[10]; a.keep = ints[11];
-  a.eps = floats[0]; a.scale = floats[1];
-  return a.heads >= 1 && a.kv_heads >= 1 && a.heads % a.kv_heads == 0 && a.heads / a.kv_heads <= 64 && a.dim >= 1 && padded_dim(a.dim) > 0 &&
-         a.pshift >= 4 && (1 << a.pshift) == ints[9] && a.keep >= 0;
+  a.krms = (float*)ptrs[8]; a.vpool = const_cast<void*>(ptrs[9]); a.out = const_cast<void*>(ptrs[10]);
+  a.ld = ints[0]; a.q_col = ints[1]; a.k_col = ints[2]; a.v_col = ints[3]; a.g_col = ints[4]; a.ldo = ints[5]; a.heads = ints[6];
+  a.kv_heads = ints[7]; a.dim = ints[8]; a.vdim = ints[9]; a.max_pages = ints[10];
+  for (a.pshift = 0; (2 << a.pshift) <= ints[11]; ++a.pshift) {}
+  a.window = ints[12]; a.keep = ints[13];
+  a.eps = floats[0]; a.scale = floats[1]; a.out_scale = floats[2]; a.softcap = floats[3]; a.temp_coef = floats[4]; a.temp_every = floats[5];
+  if (a.vpool == nullptr ? a.krms == nullptr || a.vdim != a.dim : a.vdim < 1) return false;
+  return a.heads >= 1 && a.kv_heads >= 1 && a.heads % a.kv_heads == 0 && a.heads / a.kv_heads <= 64 && a.dim >= 1 &&
+         padded_dim(a.dim > a.vdim ? a.dim : a.vdim) > 0 && a.pshift >= 4 && (1 << a.pshift) == ints[11] && a.keep >= 0 &&
+         (a.temp_coef == 0.0f || a.temp_every > 0.0f) && (a.q_norm == nullptr) == (a.k_norm == nullptr);
 }
 
-#define BONSAI_BY_DIM(CALL)                                  \
-  switch (padded_dim(a.dim)) {                               \
-    case 32: { constexpr int HD = 32; return CALL; }         \
-    case 64: { constexpr int HD = 64; return CALL; }         \
-    case 96: { constexpr int HD = 96; return CALL; }         \
-    case 128: { constexpr int HD = 128; return CALL; }       \
-    case 192: { constexpr int HD = 192; return CALL; }       \
-    case 256: { constexpr int HD = 256; return CALL; }       \
-    default: return BONSAI_CUDA_BAD_ARG;                     \
+#define BONSAI_ONE_DIM(D, CALL)                                                                            \
+  case D: {                                                                                                \
+    constexpr int HD = D;                                                                                  \
+    if (a.vpool != nullptr) { constexpr bool SEP = true; return CALL; } else { constexpr bool SEP = false; return CALL; } \
+  }
+#define BONSAI_BY_DIM(CALL)                                 \
+  switch (padded_dim(a.dim > a.vdim ? a.dim : a.vdim)) {    \
+    BONSAI_ONE_DIM(32, CALL)                                \
+    BONSAI_ONE_DIM(64, CALL)                                \
+    BONSAI_ONE_DIM(96, CALL)                                \
+    BONSAI_ONE_DIM(128, CALL)                               \
+    BONSAI_ONE_DIM(192, CALL)                               \
+    BONSAI_ONE_DIM(256, CALL)                               \
+    default: return BONSAI_CUDA_BAD_ARG;                    \
   }
 
 }  // namespace lay
@@ -590,15 +654,16 @@ extern "C" {
 // elements of a cache row for a head size (0: not supported)
 int bonsai_lay_attn_row(int dim) { return dim < 1 ? 0 : bonsai::lay::padded_dim(dim); }
 
-// Arguments of all launches: ptrs = {proj, q_norm, k_norm, slopes, pos, slots, block_table, pool, krms, out}, ints = {ld,
-// q_col, k_col, g_col, ldo, heads, kv_heads, dim, max_pages, page_size, window, keep}, floats = {eps, scale}.
+// Arguments of all launches: ptrs = {proj, q_norm, k_norm, slopes, pos, slots, block_table, pool, krms, vpool, out} (null where
+// a design has none; vpool null: rows are key and value), ints = {ld, q_col, k_col, v_col, g_col, ldo, heads, kv_heads, dim,
+// vdim, max_pages, page_size, window, keep}, floats = {eps, scale, out_scale, softcap, temp_coef, temp_every}.
 
 // Writes the keys of rows first .. first + count - 1.
 int bonsai_lay_attn_append(const void* const* ptrs, const int* ints, const float* floats, int first, int count, int f32, cudaStream_t stream) {
   using namespace bonsai::lay;
   Attn a;
   if (!fill(a, ptrs, ints, floats) || count < 1 || first < 0) return BONSAI_CUDA_BAD_ARG;
-  BONSAI_BY_DIM((run_append<HD>(a, first, count, f32, stream)))
+  BONSAI_BY_DIM((run_append<HD, SEP>(a, first, count, f32, stream)))
 }
 
 // entries int4 [..] {first row, tokens, slot, first position}, tiles int2 [ntiles] {entry, first token}; a tile has
@@ -608,7 +673,7 @@ int bonsai_lay_attn_prompt(const void* const* ptrs, const int* ints, const float
   using namespace bonsai::lay;
   Attn a;
   if (!fill(a, ptrs, ints, floats) || ntiles < 1 || ntiles > 65535) return BONSAI_CUDA_BAD_ARG;
-  BONSAI_BY_DIM((run_prompt<HD>(a, entries, tiles, ntiles, stream)))
+  BONSAI_BY_DIM((run_prompt<HD, SEP>(a, entries, tiles, ntiles, stream)))
 }
 
 // One token in each of the rows 0 .. nrows - 1, its key appended here.
@@ -616,7 +681,7 @@ int bonsai_lay_attn_decode(const void* const* ptrs, const int* ints, const float
   using namespace bonsai::lay;
   Attn a;
   if (!fill(a, ptrs, ints, floats) || nrows < 1 || nrows > 65535 || (nsplit != 1 && nsplit != 2 && nsplit != 4 && nsplit != 8)) return BONSAI_CUDA_BAD_ARG;
-  BONSAI_BY_DIM((run_decode<HD>(a, nrows, nsplit, stream)))
+  BONSAI_BY_DIM((run_decode<HD, SEP>(a, nrows, nsplit, stream)))
 }
 
 // All T rows, 32-bit throughout; the rows' keys must have been appended.
@@ -624,7 +689,7 @@ int bonsai_lay_attn_f32(const void* const* ptrs, const int* ints, const float* f
   using namespace bonsai::lay;
   Attn a;
   if (!fill(a, ptrs, ints, floats) || T < 1 || T > 65535) return BONSAI_CUDA_BAD_ARG;
-  BONSAI_BY_DIM((run_f32<HD>(a, T, stream)))
+  BONSAI_BY_DIM((run_f32<HD, SEP>(a, T, stream)))
 }
 
 }  // extern "C"

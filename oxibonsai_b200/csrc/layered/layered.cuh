@@ -79,6 +79,13 @@ __device__ __forceinline__ float load_act(const float* p) { return *p; }
 
 constexpr float kLog2e = 1.4426950408889634f;
 
+// chunked recurrences: tokens per chunk, value columns per CTA, row length of a staged value tile
+constexpr int kL = 64;
+constexpr int kVT = 64;
+constexpr int kVLD = kVT + 8;
+// a portion as a whole, the local states of its segments, the segments from the states they start from
+enum ChunkMode { kWhole, kLocal, kResume };
+
 // One launch with programmatic dependent launch and, for cluster > 1, thread-block clusters of that many CTAs along
 // dimension `dim` (0 = x, 1 = y) of the grid.
 template <typename Kern, typename... Args>

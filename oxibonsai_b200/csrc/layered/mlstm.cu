@@ -174,10 +174,6 @@ __global__ void __launch_bounds__(16 * DG) step_kernel(Mlstm a, const int4* entr
 }
 
 // ---- portions of prompts ------------------------------------------------------------------------------------------------------------
-constexpr int kL = 64;      // tokens per chunk
-constexpr int kVT = 64;     // value columns per CTA
-constexpr int kVLD = kVT + 8;
-
 constexpr int chunk_warps(int dim) { return dim >= 256 ? 16 : 8; }
 
 template <int DIM>
@@ -199,8 +195,6 @@ struct ChunkSmem {
   float rows[NCH][kL];  // row sums of p over the warps' key columns
   float nq[kL];         // q_t . n_0
 };
-
-enum ChunkMode { kWhole, kLocal, kResume };
 
 // grid (vp / 64, heads, entries).  Warp w: rows (w & 3) * 16 .. + 15 of the chunk and group w >> 2 of the columns (keys and
 // values); of the state two 16-row tiles and WN 8-column tiles.

@@ -1,38 +1,64 @@
 // Row-wise steps of the layer-list decoders: embedding lookup, norm-of-the-output residual add, final norm of selected rows,
-// and the per-head norm with output gate of the recurrent mixers.  The residual stream is f32; every kernel that changes it
-// also leaves the bf16 copy that the next projection reads (null in the f32 mode, where projections read the stream).
+// and the gated norms of the recurrent mixers.  The residual stream is f32; every kernel that changes it also leaves the input
+// of the next projection: the stream itself, or, in designs with a norm ahead of each sublayer, its norm.
 #include "layered/layered.cuh"
 
 namespace bonsai {
 namespace lay {
 
-__global__ void embed_kernel(const bf16* __restrict__ table, int ld_table, const int* tokens, int width, float* x,
-                             bf16* x16, int ld16) {
+constexpr int kKeep = 4;   // float4 chunks of a row that a thread keeps in registers
+
+__device__ __forceinline__ void store_act4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+__device__ __forceinline__ void store_act4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+
+// x[t] = table[tokens[t]] * scale; h[t] = x[t], or its norm when `next` (the norm's weight) is given.  h may be null.
+template <typename H>
+__global__ void embed_kernel(const bf16* __restrict__ table, int ld_table, const int* tokens, float scale, int width, float* x, H* h, int ldh,
+                             const float* __restrict__ next, float eps) {
+  __shared__ float s32[32];
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
   const bf16* src = table + (size_t)tokens[t] * ld_table;
+  float inv = 1.0f;
+  if (next != nullptr) {
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      const float v = __bfloat162float(src[c]) * scale;
+      ss += v * v;
+    }
+    inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+  }
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const bf16 v = src[c];
-    x[(size_t)t * width + c] = __bfloat162float(v);
-    if (x16 != nullptr) x16[(size_t)t * ld16 + c] = v;
+    const float v = __bfloat162float(src[c]) * scale;
+    x[(size_t)t * width + c] = v;
+    if (h != nullptr) store_act(h + (size_t)t * ldh + c, next != nullptr ? v * inv * next[c] : v);
   }
 }
 
-constexpr int kKeep = 4;   // float4 chunks of a row that a thread keeps in registers
-
-// x += y / sqrt(mean(y^2) + eps) * w
-__global__ void norm_add_kernel(float* x, const float* y, int ldy, const float* __restrict__ w, float eps, int width,
-                                bf16* x16, int ld16) {
+// x += y / sqrt(mean(y^2) + eps) * w; h = x, or its norm with weight `next`
+template <typename H>
+__global__ void norm_add_kernel(float* x, const float* y, int ldy, const float* __restrict__ w, float eps, int width, H* h, int ldh,
+                                const float* __restrict__ next) {
   __shared__ float s32[32];
+  // weights depend on no earlier kernel
+  const bool vec = (width & 3) == 0 && width <= 4 * kKeep * (int)blockDim.x;
+  const int nch = width >> 2;
+  float4 wv[kKeep];
+  if (vec) {
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nch) wv[i] = reinterpret_cast<const float4*>(w)[c];
+    }
+  }
   pdl_wait();
   pdl_trigger();
   float* xr = x + (size_t)blockIdx.x * width;
   const float* yr = y + (size_t)blockIdx.x * ldy;
-  bf16* hr = x16 == nullptr ? nullptr : x16 + (size_t)blockIdx.x * ld16;
+  H* hr = h == nullptr ? nullptr : h + (size_t)blockIdx.x * ldh;
   float ss = 0.0f;
-  if ((width & 3) == 0 && width <= 4 * kKeep * (int)blockDim.x) {
-    const int nch = width >> 2;
+  if (vec) {
     float4 v[kKeep], r[kKeep];
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
@@ -42,28 +68,44 @@ __global__ void norm_add_kernel(float* x, const float* y, int ldy, const float* 
       ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+    float sx = 0.0f;
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
       const int c = threadIdx.x + i * blockDim.x;
       if (c < nch) {
-        const float4 g = reinterpret_cast<const float4*>(w)[c];
-        r[i].x += v[i].x * inv * g.x;
-        r[i].y += v[i].y * inv * g.y;
-        r[i].z += v[i].z * inv * g.z;
-        r[i].w += v[i].w * inv * g.w;
+        r[i].x += v[i].x * inv * wv[i].x;
+        r[i].y += v[i].y * inv * wv[i].y;
+        r[i].z += v[i].z * inv * wv[i].z;
+        r[i].w += v[i].w * inv * wv[i].w;
         reinterpret_cast<float4*>(xr)[c] = r[i];
-        if (hr != nullptr) reinterpret_cast<uint2*>(hr)[c] = make_uint2(pack_bf16(r[i].x, r[i].y), pack_bf16(r[i].z, r[i].w));
+        sx += r[i].x * r[i].x + r[i].y * r[i].y + r[i].z * r[i].z + r[i].w * r[i].w;
       }
+    }
+    if (hr == nullptr) return;
+    const float nx = next == nullptr ? 1.0f : 1.0f / sqrtf(block_sum(sx, s32) / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c >= nch) continue;
+      if (next != nullptr) {
+        const float4 g = reinterpret_cast<const float4*>(next)[c];
+        r[i] = make_float4(r[i].x * nx * g.x, r[i].y * nx * g.y, r[i].z * nx * g.z, r[i].w * nx * g.w);
+      }
+      store_act4(hr + 4 * c, r[i]);
     }
     return;
   }
   for (int c = threadIdx.x; c < width; c += blockDim.x) ss += yr[c] * yr[c];
   const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+  float sx = 0.0f;
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     const float v = xr[c] + yr[c] * inv * w[c];
     xr[c] = v;
-    if (hr != nullptr) hr[c] = __float2bfloat16_rn(v);
+    sx += v * v;
   }
+  if (hr == nullptr) return;
+  const float nx = next == nullptr ? 1.0f : 1.0f / sqrtf(block_sum(sx, s32) / (float)width + eps);
+  for (int c = threadIdx.x; c < width; c += blockDim.x) store_act(hr + c, next == nullptr ? xr[c] : xr[c] * nx * next[c]);
 }
 
 // out[i] = norm(x[rows[i]]) * w; rows == null: row i
@@ -81,48 +123,93 @@ __global__ void norm_rows_kernel(const float* x, const int* rows, const float* _
   for (int c = threadIdx.x; c < width; c += blockDim.x) store_act(out + (size_t)blockIdx.x * ld + c, xr[c] * inv * w[c]);
 }
 
-// One warp per (row, head): o / rms(o over the head) * w * sigmoid(gate)
-template <typename OUT>
-__global__ void __launch_bounds__(256) gated_head_norm_kernel(const float* o, int ldo, const float* gate, int ldg, const float* __restrict__ w,
-                                                              float eps, int T, int heads, int vdim, OUT* out, int ld, int vec) {
+// Norm of a recurrent mixer's output in parts of `width` columns (a head, a group of heads, or all of them), with a gate before
+// or after it:
+//   after:  out = o / rms(o) [* w] * act(gate) * scale          before:  u = o * act(gate), out = u / rms(u) [* w] * scale
+// act: sigmoid, or silu.  GT threads per (row, part).
+struct GatedNorm {
+  const float* o;
+  const float* gate;
+  const float* w;           // null: no weight
+  int ldo, ldg, T, parts, width, ld, vec, silu, before;
+  float eps, scale;
+};
+
+__device__ __forceinline__ float gate_act(const GatedNorm& a, float g) {
+  const float s = sigmoid(g);
+  return a.silu ? g * s : s;
+}
+
+template <int GT, typename OUT>
+__global__ void __launch_bounds__(256) gated_norm_kernel(GatedNorm a, OUT* out) {
+  __shared__ float s32[32];
   pdl_wait();
   pdl_trigger();
-  const int lane = threadIdx.x & 31, item = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (item >= T * heads) return;
-  const int t = item / heads, c0 = (item % heads) * vdim;
-  const float* orow = o + (size_t)t * ldo + c0;
-  const float* grow = gate + (size_t)t * ldg + c0;
-  OUT* dst = out + (size_t)t * ld + c0;
-  w += c0;
-  if (vec) {                 // rows of float4, up to kKeep per lane
-    const int nch = vdim >> 2;
+  constexpr int PER = 256 / GT;
+  const int lane = threadIdx.x % GT, item = blockIdx.x * PER + threadIdx.x / GT;
+  if (item >= a.T * a.parts) return;       // with GT = 256 the whole CTA
+  const int t = item / a.parts, c0 = (item % a.parts) * a.width;
+  const float* orow = a.o + (size_t)t * a.ldo + c0;
+  const float* grow = a.gate + (size_t)t * a.ldg + c0;
+  OUT* dst = out + (size_t)t * a.ld + c0;
+  const float* w = a.w == nullptr ? nullptr : a.w + c0;
+  auto sum = [&](float v) { return GT == 32 ? warp_sum(v) : block_sum(v, s32); };
+  if (a.vec) {                 // rows of float4, up to kKeep per thread
+    const int nch = a.width >> 2;
     float4 v[kKeep], g[kKeep];
     float ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
-      const int c = lane + 32 * i;
+      const int c = lane + GT * i;
       v[i] = c < nch ? reinterpret_cast<const float4*>(orow)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
       g[i] = c < nch ? reinterpret_cast<const float4*>(grow)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
-      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
     }
-    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
-      const int c = lane + 32 * i;
-      if (c < nch) {
-        const float4 ww = reinterpret_cast<const float4*>(w)[c];
-        const float y[4] = {v[i].x * inv * ww.x * sigmoid(g[i].x), v[i].y * inv * ww.y * sigmoid(g[i].y), v[i].z * inv * ww.z * sigmoid(g[i].z),
-                            v[i].w * inv * ww.w * sigmoid(g[i].w)};
-        if constexpr (sizeof(OUT) == 2) reinterpret_cast<uint2*>(dst)[c] = make_uint2(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]));
-        else reinterpret_cast<float4*>(dst)[c] = make_float4(y[0], y[1], y[2], y[3]);
+      g[i] = make_float4(gate_act(a, g[i].x), gate_act(a, g[i].y), gate_act(a, g[i].z), gate_act(a, g[i].w));
+      if (a.before) {
+        v[i].x *= g[i].x; v[i].y *= g[i].y; v[i].z *= g[i].z; v[i].w *= g[i].w;
       }
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float inv = a.scale / sqrtf(sum(ss) / (float)a.width + a.eps);
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int c = lane + GT * i;
+      if (c >= nch) continue;
+      float4 y = make_float4(v[i].x * inv, v[i].y * inv, v[i].z * inv, v[i].w * inv);
+      if (!a.before) {
+        y.x *= g[i].x; y.y *= g[i].y; y.z *= g[i].z; y.w *= g[i].w;
+      }
+      if (w != nullptr) {
+        const float4 ww = reinterpret_cast<const float4*>(w)[c];
+        y.x *= ww.x; y.y *= ww.y; y.z *= ww.z; y.w *= ww.w;
+      }
+      store_act4(dst + 4 * c, y);
     }
     return;
   }
+  auto value = [&](int c) { return a.before ? orow[c] * gate_act(a, grow[c]) : orow[c]; };
   float ss = 0.0f;
-  for (int c = lane; c < vdim; c += 32) ss += orow[c] * orow[c];
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
-  for (int c = lane; c < vdim; c += 32) store_act(dst + c, orow[c] * inv * w[c] * sigmoid(grow[c]));
+  for (int c = lane; c < a.width; c += GT) {
+    const float v = value(c);
+    ss += v * v;
+  }
+  const float inv = a.scale / sqrtf(sum(ss) / (float)a.width + a.eps);
+  for (int c = lane; c < a.width; c += GT) {
+    float y = value(c) * inv;
+    if (!a.before) y *= gate_act(a, grow[c]);
+    store_act(dst + c, w == nullptr ? y : y * w[c]);
+  }
+}
+
+template <typename OUT>
+static int run_gated_norm(GatedNorm a, OUT* out, cudaStream_t stream) {
+  const uintptr_t at = reinterpret_cast<uintptr_t>(a.o) | reinterpret_cast<uintptr_t>(a.gate) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(out);
+  const bool wide = a.width > 128 * kKeep;
+  a.vec = a.width % 4 == 0 && a.width <= (wide ? 1024 : 128) * kKeep && a.ldo % 4 == 0 && a.ldg % 4 == 0 && a.ld % 4 == 0 && at % 16 == 0;
+  if (wide) return launch(gated_norm_kernel<256, OUT>, dim3(a.T * a.parts), 256, 0, stream, 1, 0, a, out);
+  return launch(gated_norm_kernel<32, OUT>, dim3((a.T * a.parts + 7) / 8), 256, 0, stream, 1, 0, a, out);
 }
 
 static int row_threads(int width) {
@@ -136,17 +223,25 @@ static int row_threads(int width) {
 
 extern "C" {
 
-// x f32 [T][width] = table[tokens[t]] (bf16 rows of ld_table elements); x16 (may be null) bf16 [T][ld16]
-int bonsai_lay_embed(const void* table, int ld_table, const int* tokens, int T, int width, float* x, void* x16, int ld16, cudaStream_t stream) {
+// x f32 [T][width] = table[tokens[t]] * scale (bf16 rows of ld_table elements); h (may be null) [T][ldh], bf16 or f32 = x or, with
+// `next`, its norm
+int bonsai_lay_embed(const void* table, int ld_table, const int* tokens, float scale, int T, int width, float* x, void* h, int ldh, int h_f32,
+                     const float* next, float eps, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (T < 1 || width < 1 || ld_table < width) return BONSAI_CUDA_BAD_ARG;
-  return launch(embed_kernel, dim3(T), 256, 0, stream, 1, 0, (const bf16*)table, ld_table, tokens, width, x, (bf16*)x16, ld16);
+  if (T < 1 || width < 1 || ld_table < width || (h != nullptr && ldh < width)) return BONSAI_CUDA_BAD_ARG;
+  if (h_f32)
+    return launch(embed_kernel<float>, dim3(T), 256, 0, stream, 1, 0, (const bf16*)table, ld_table, tokens, scale, width, x, (float*)h, ldh, next, eps);
+  return launch(embed_kernel<bf16>, dim3(T), 256, 0, stream, 1, 0, (const bf16*)table, ld_table, tokens, scale, width, x, (bf16*)h, ldh, next, eps);
 }
 
-int bonsai_lay_norm_add(float* x, const float* y, int ldy, const float* w, float eps, int T, int width, void* x16, int ld16, cudaStream_t stream) {
+// x += norm(y) * w; h (may be null) = x or, with `next`, its norm
+int bonsai_lay_norm_add(float* x, const float* y, int ldy, const float* w, float eps, int T, int width, void* h, int ldh, int h_f32, const float* next,
+                        cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (T < 1 || width < 1 || ldy < width || (ldy & 3) != 0 || (ld16 & 3) != 0) return BONSAI_CUDA_BAD_ARG;
-  return launch(norm_add_kernel, dim3(T), row_threads(width), 0, stream, 1, 0, x, y, ldy, w, eps, width, (bf16*)x16, ld16);
+  if (T < 1 || width < 1 || ldy < width || (ldy & 3) != 0 || (h != nullptr && (ldh < width || (ldh & 3) != 0))) return BONSAI_CUDA_BAD_ARG;
+  const int th = row_threads(width);
+  if (h_f32) return launch(norm_add_kernel<float>, dim3(T), th, 0, stream, 1, 0, x, y, ldy, w, eps, width, (float*)h, ldh, next);
+  return launch(norm_add_kernel<bf16>, dim3(T), th, 0, stream, 1, 0, x, y, ldy, w, eps, width, (bf16*)h, ldh, next);
 }
 
 // out: bf16 when f32_out == 0, f32 otherwise
@@ -159,16 +254,14 @@ int bonsai_lay_norm_rows(const float* x, const int* rows, const float* w, float 
   return launch(norm_rows_kernel<bf16>, dim3(R), th, 0, stream, 1, 0, x, rows, w, eps, width, (bf16*)out, ld);
 }
 
-int bonsai_lay_gated_head_norm(const float* o, int ldo, const float* gate, int ldg, const float* w, float eps, int T, int heads, int vdim, void* out,
-                               int ld, int f32_out, cudaStream_t stream) {
+// Gated norm: o and gate f32 [T][ld..] with `parts` parts of `width` columns, w [parts * width] or null; act 0 =
+// sigmoid, 1 = silu; before: the gate comes before the norm
+int bonsai_lay_gated_norm(const float* o, int ldo, const float* gate, int ldg, const float* w, float eps, int T, int parts, int width, int act, int before,
+                          float scale, void* out, int ld, int f32_out, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (T < 1 || heads < 1 || vdim < 1 || ld < heads * vdim || (long long)T * heads >= (1ll << 30)) return BONSAI_CUDA_BAD_ARG;
-  const dim3 grid((T * heads + 7) / 8);
-  const uintptr_t at = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out);
-  const int vec = vdim % 4 == 0 && vdim <= 128 * kKeep && ldo % 4 == 0 && ldg % 4 == 0 && ld % 4 == 0 && at % 16 == 0;
-  if (f32_out)
-    return launch(gated_head_norm_kernel<float>, grid, 256, 0, stream, 1, 0, o, ldo, gate, ldg, w, eps, T, heads, vdim, (float*)out, ld, vec);
-  return launch(gated_head_norm_kernel<bf16>, grid, 256, 0, stream, 1, 0, o, ldo, gate, ldg, w, eps, T, heads, vdim, (bf16*)out, ld, vec);
+  if (T < 1 || parts < 1 || width < 1 || ld < parts * width || (long long)T * parts >= (1ll << 30)) return BONSAI_CUDA_BAD_ARG;
+  const GatedNorm a{o, gate, w, ldo, ldg, T, parts, width, ld, 0, act, before, eps, scale};
+  return f32_out ? run_gated_norm(a, (float*)out, stream) : run_gated_norm(a, (bf16*)out, stream);
 }
 
 }  // extern "C"

@@ -2,7 +2,8 @@
 
 A step is a batch of rows (tokens).  Rows of single tokens (decode) come first, portions of prompts follow, each portion
 contiguous; every projection runs over all rows, a mixer runs its single-token kernel over the first group and its prompt
-kernel over the second.  A row carries its position and its slot; the slot's block-table row names the pages of its sequence
+kernel over the second.  Mixers that stand side by side in a layer share one projection and one output projection over their
+joined outputs.  A row carries its position and its slot; the slot's block-table row names the pages of its sequence
 and the state table its recurrent state row, so which pages, rows and companions a token has does not enter its arithmetic.
 
 Two modes: bf16 (tensor-core projections and attention, f32 residual stream, norms, scores, gates and recurrent state) and
@@ -21,8 +22,8 @@ import torch
 from ..ops import cuda_ops as K
 from ..ops import layered_ops as L
 from ..ops import nvtx
-from .layered_config import AttentionSpec, LayeredConfig, MlstmSpec
-from .paged import SharedRowCache, StatePool
+from .layered_config import AttentionSpec, Branch, GatedMlpSpec, LayeredConfig, LinearRecurrenceSpec, MlstmSpec, SquaredReluMlpSpec
+from .paged import RowCache, StatePool
 from .rope_scaling import geometric_slopes
 from .slot_state import SlotState
 
@@ -36,18 +37,38 @@ def _tensor(t) -> torch.Tensor:
 
 @dataclass
 class MlpWeights:
+    pre_norm: torch.Tensor | None
     norm: torch.Tensor
-    gate_up: L.DenseWeight
+    up: L.DenseWeight                # gated blocks: gate and up rows interleaved
     down: L.DenseWeight
+    act: L.Glu | str
+
+
+@dataclass
+class BranchWeights:
+    columns: list[int]               # first output of each section in the layer's projection
+    vectors: dict[str, torch.Tensor]
+    offset: int                      # first column in the input of the output projection
 
 
 @dataclass
 class LayerWeights:
+    pre_norm: torch.Tensor | None
     norm: torch.Tensor
-    proj: L.DenseWeight              # every projection that reads the mixer's input, one matrix
-    out: L.DenseWeight
-    vectors: dict[str, torch.Tensor]
+    proj: L.DenseWeight              # every projection that reads the mixers' input, one matrix
+    out: L.DenseWeight               # the branches' output projections side by side
+    branches: list[BranchWeights]
     mlp: MlpWeights | None
+
+
+def branch_offsets(widths: Sequence[int]) -> tuple[list[int], int]:
+    """First columns of the branches' outputs in their joined buffer (16-byte boundaries in either mode), and its width."""
+    at, offsets = 0, []
+    for w in widths:
+        at = L.round_up(at, 8)
+        offsets.append(at)
+        at += w
+    return offsets, at
 
 
 class LayeredWeights:
@@ -62,22 +83,35 @@ class LayeredWeights:
                 raise ValueError(f"tensor {n} is {list(tensors[n].shape)}, expected {list(s)}")
         self.cfg, self.device = cfg, torch.device(device)
         m = lambda n: tensors[n].to(torch.bfloat16)
-        v = lambda n: tensors[n].float().to(self.device)
+        v = lambda n: None if n is None else tensors[n].float().to(self.device)
         self.embed = L.DenseWeight([m("embed")], self.device)      # also the output head
         self.final_norm = v("final.norm")
         self.layers: list[LayerWeights] = []
         for i, spec in enumerate(cfg.layer_specs):
-            p, x = f"l{i}.", f"l{i}.mix."
-            if spec.mixer.kind == "attention":
-                proj, vec = ["q", "k", "g"], ["q.norm", "k.norm"]
-            else:
-                proj, vec = ["q", "k", "v", "g", "i", "f"], ["i.b", "f.b", "norm"]
+            norms, p, parts, counts = cfg.norm_names(i), f"l{i}.mlp.", [], []
+            for b in spec.mixer.branches:
+                first: dict[str, int] = {}
+                for name, rows in b.spec.sections:
+                    at = first.get(name, 0)
+                    parts.append(m(f"l{i}.mix.{b.prefix}{name}")[at:at + rows])
+                    first[name] = at + rows
+                counts.append(len(b.spec.sections))
+            proj = L.DenseWeight(parts, self.device)
+            offsets, width = branch_offsets([b.spec.out_width for b in spec.mixer.branches])
+            out = torch.zeros((cfg.width, width), dtype=torch.bfloat16)
+            branches, at = [], 0
+            for b, off, count in zip(spec.mixer.branches, offsets, counts):
+                x = f"l{i}.mix.{b.prefix}"
+                out[:, off:off + b.spec.out_width] = m(x + "o")
+                branches.append(BranchWeights(proj.columns[at:at + count], {n: v(x + n) for n in b.spec.vectors}, off))
+                at += count
             mlp = None
-            if spec.mlp is not None:
-                mlp = MlpWeights(v(p + "norm2"), L.DenseWeight([m(p + "mlp.gate"), m(p + "mlp.up")], self.device, interleave=True),
-                                 L.DenseWeight([m(p + "mlp.down")], self.device))
-            self.layers.append(LayerWeights(v(p + "norm1"), L.DenseWeight([m(x + n) for n in proj], self.device),
-                                            L.DenseWeight([m(x + "o")], self.device), {n: v(x + n) for n in vec}, mlp))
+            if isinstance(spec.mlp, GatedMlpSpec):
+                up = L.DenseWeight([m(p + "gate"), m(p + "up")], self.device, interleave=True)
+                mlp = MlpWeights(*map(v, norms[1]), up, L.DenseWeight([m(p + "down")], self.device), L.Glu(spec.mlp.limit, spec.mlp.alpha, spec.mlp.offset))
+            elif isinstance(spec.mlp, SquaredReluMlpSpec):
+                mlp = MlpWeights(*map(v, norms[1]), L.DenseWeight([m(p + "up")], self.device), L.DenseWeight([m(p + "down")], self.device), L.SQUARED_RELU)
+            self.layers.append(LayerWeights(*map(v, norms[0]), proj, L.DenseWeight([out], self.device), branches, mlp))
         torch.cuda.synchronize(self.device)
 
     @classmethod
@@ -90,21 +124,39 @@ class LayeredWeights:
         """Bytes a decode step must stream."""
         n = self.embed.nbytes
         for l in self.layers:
-            n += l.proj.nbytes + l.out.nbytes + (0 if l.mlp is None else l.mlp.gate_up.nbytes + l.mlp.down.nbytes)
+            n += l.proj.nbytes + l.out.nbytes + (0 if l.mlp is None else l.mlp.up.nbytes + l.mlp.down.nbytes)
         return n
 
 
-def new_row_cache(cfg: LayeredConfig, num_pages: int, page_size: int, exact: bool, device) -> SharedRowCache:
-    layers = {i: (cfg.layer_specs[i].mixer.kv_heads, L.lib().bonsai_lay_attn_row(cfg.layer_specs[i].mixer.dim)) for i in cfg.attention_layers}
-    return SharedRowCache(layers, num_pages, page_size, K.KV_F32 if exact else K.KV_BF16, torch.float32 if exact else torch.bfloat16, device)
+def new_row_cache(cfg: LayeredConfig, num_pages: int, page_size: int, exact: bool, device) -> RowCache:
+    specs = {i: cfg.attention(i) for i in cfg.attention_layers}
+    layers = {i: (s.kv_heads, L.lib().bonsai_lay_attn_row(max(s.dim, s.value_dim)), s.vdim is not None) for i, s in specs.items()}
+    return RowCache(layers, num_pages, page_size, K.KV_F32 if exact else K.KV_BF16, torch.float32 if exact else torch.bfloat16, device)
+
+
+def state_dims(m: MlstmSpec | LinearRecurrenceSpec) -> tuple[int, int]:
+    """Padded rows and columns of a head's state."""
+    l = L.lib()
+    if isinstance(m, MlstmSpec):
+        return l.bonsai_lay_mlstm_dim(m.dim), l.bonsai_lay_mlstm_vdim(m.vdim)
+    return l.bonsai_lay_rec_dim(m.dim), l.bonsai_lay_rec_vdim(m.vdim)
+
+
+def runs_chunked(m: MlstmSpec | LinearRecurrenceSpec) -> bool:
+    """Whether portions of prompts go to the tensor cores (longer keys take the token-by-token kernel)."""
+    return m.dim <= (L.lib().bonsai_lay_mlstm_chunk_dim() if isinstance(m, MlstmSpec) else L.lib().bonsai_lay_rec_chunk_dim())
 
 
 def new_state_pool(cfg: LayeredConfig, num_rows: int, device) -> StatePool:
     layers = {}
     for i in cfg.recurrent_layers:
-        m: MlstmSpec = cfg.layer_specs[i].mixer
-        d, e = L.lib().bonsai_lay_mlstm_dim(m.dim), L.lib().bonsai_lay_mlstm_vdim(m.vdim)
-        layers[i] = {"S": (m.heads, d, e), "n": (m.heads, e // 64, d), "m": (m.heads, e // 64)}
+        m = cfg.recurrence(i)
+        d, e = state_dims(m)
+        layers[i] = {"S": (m.heads, d, e)}
+        if isinstance(m, MlstmSpec):
+            layers[i].update({"n": (m.heads, e // 64, d), "m": (m.heads, e // 64)})
+        elif m.conv:
+            layers[i]["conv"] = (m.conv, m.conv_channels)
     return StatePool(layers, num_rows, device)
 
 
@@ -151,17 +203,17 @@ def plan_segments(lengths: Sequence[int], ctas: int, sms: int) -> int:
 
 
 class AttentionMixer:
-    def __init__(self, r: "LayeredRunner", index: int, spec: AttentionSpec):
-        self.r, self.spec, self.w, cfg = r, spec, r.w.layers[index], r.cfg
+    def __init__(self, r: "LayeredRunner", index: int, branch: Branch, w: BranchWeights, out: torch.Tensor):
+        self.r, self.spec, self.out = r, branch.spec, out
+        spec, cols = self.spec, dict(zip((n for n, _ in branch.spec.sections), w.columns))
         self.tile = 64 // spec.group
-        self.slopes = geometric_slopes(spec.heads, spec.slope_exponent).to(r.device)
-        self.out = r.act_buffer(spec.out_width)
-        q, k, g = self.w.proj.columns
-        ints = [r.proj.stride(0), q, k, g, self.out.stride(0), spec.heads, spec.kv_heads, spec.dim, r.max_pages, r.kv.page_size, spec.window,
-                spec.keep_first]
-        cache, factors = r.kv.rows[index], r.kv.factors[index]
-        self.call = {id(rows): L.MixerCall([r.proj, self.w.vectors["q.norm"], self.w.vectors["k.norm"], self.slopes, rows.positions, rows.slots,
-                                            r.block_table, cache, factors, self.out], ints, [cfg.eps, spec.scale]) for rows in (r.slot_rows, r.batch_rows)}
+        slopes = None if spec.slope_exponent is None else geometric_slopes(spec.heads, spec.slope_exponent).to(r.device)
+        ints = [r.proj.stride(0), cols["q"], cols["k"], cols.get("v", 0), cols.get("g", -1), out.stride(0), spec.heads, spec.kv_heads, spec.dim,
+                spec.value_dim, r.max_pages, r.kv.page_size, spec.window, spec.keep_first]
+        floats = [r.cfg.eps, spec.scale, branch.scale, spec.softcap, spec.temp_coef, spec.temp_every]
+        self.call = {id(rows): L.MixerCall([r.proj, w.vectors.get("q.norm"), w.vectors.get("k.norm"), slopes, rows.positions, rows.slots, r.block_table,
+                                            r.kv.rows[index], r.kv.factors.get(index), r.kv.values.get(index), out], ints, floats)
+                     for rows in (r.slot_rows, r.batch_rows)}
 
     def splits(self, batch: int) -> int:
         """KV splits of one row's decode attention: about a CTA per SM, and no more than there are 16-token tiles per warp."""
@@ -172,31 +224,30 @@ class AttentionMixer:
             n *= 2
         return n
 
-    def __call__(self, rows: Rows, st: StepShape, stream: int) -> torch.Tensor:
+    def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
         lib, a = L.lib(), self.call[id(rows)].args
         if self.r.exact:
             K.check(lib.bonsai_lay_attn_append(*a, 0, st.rows, 1, stream), "attn_append")
             K.check(lib.bonsai_lay_attn_f32(*a, st.rows, stream), "attn_f32")
-            return self.out
+            return
         if st.singles:
             K.check(lib.bonsai_lay_attn_decode(*a, st.singles, self.splits(st.singles), stream), "attn_decode")
         if st.portions:
             tiles, n = st.tiles[self.tile]
             K.check(lib.bonsai_lay_attn_append(*a, st.singles, st.rows - st.singles, 0, stream), "attn_append")
             K.check(lib.bonsai_lay_attn_prompt(*a, st.entries, tiles, n, stream), "attn_prompt")
-        return self.out
 
     def launches(self) -> int:
         return 2 if self.r.exact else 1
 
 
 class MlstmMixer:
-    def __init__(self, r: "LayeredRunner", index: int, spec: MlstmSpec):
-        self.r, self.spec, self.w, cfg = r, spec, r.w.layers[index], r.cfg
-        self.out = r.act_buffer(spec.out_width)
-        q, k, v, self.g_col, i, f = self.w.proj.columns
-        s = r.states.tensors[index]
-        self.chunked = not r.exact and spec.dim <= L.lib().bonsai_lay_mlstm_chunk_dim()
+    def __init__(self, r: "LayeredRunner", index: int, branch: Branch, w: BranchWeights, out: torch.Tensor):
+        self.r, self.spec, self.w, self.out, cfg = r, branch.spec, w, out, r.cfg
+        spec, s = self.spec, r.states.tensors[index]
+        assert branch.scale == 1.0, "an mLSTM output is not scaled"
+        q, k, v, self.g_col, i, f = w.columns
+        self.chunked = not r.exact and runs_chunked(spec)
         self.fused = spec.vdim <= L.lib().bonsai_lay_mlstm_fused_vdim()
         floats = [spec.gate_cap, cfg.eps, spec.den_eps, spec.dim ** -0.5]
 
@@ -210,9 +261,9 @@ class MlstmMixer:
 
     def _finish(self, row0: int, count: int) -> None:
         s = self.spec
-        L.gated_head_norm(self.r.head_out, row0, self.r.proj, self.g_col, self.w.vectors["norm"], self.r.cfg.eps, count, s.heads, s.vdim, self.out)
+        L.gated_norm(self.r.head_out, row0, self.r.proj, self.g_col, self.w.vectors["norm"], self.r.cfg.eps, count, s.heads, s.vdim, self.out)
 
-    def __call__(self, rows: Rows, st: StepShape, stream: int) -> torch.Tensor:
+    def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
         lib = L.lib()
         if st.singles and self.fused:
             K.check(lib.bonsai_lay_mlstm_step(*self.done[id(rows)].args, None, st.singles, 2 if self.r.exact else 1, stream), "mlstm_step")
@@ -226,13 +277,72 @@ class MlstmMixer:
             else:
                 K.check(lib.bonsai_lay_mlstm_step(*a, st.entries, st.portions, 0, stream), "mlstm_step")
             self._finish(st.singles, st.rows - st.singles)
-        return self.out
 
     def launches(self) -> int:
         return 1 if self.fused else 2
 
 
-MIXERS = {"attention": AttentionMixer, "mlstm": MlstmMixer}
+class LinearRecurrenceMixer:
+    def __init__(self, r: "LayeredRunner", index: int, branch: Branch, w: BranchWeights, out: torch.Tensor):
+        self.r, self.spec, self.scale, self.out, cfg = r, branch.spec, branch.scale, out, r.cfg
+        spec, s, lib, vec = self.spec, r.states.tensors[index], L.lib(), w.vectors
+        self.norm = vec.get("norm")
+        self.chunked = not r.exact and runs_chunked(spec)
+        # the single-token step finishes its outputs itself when the norm is per head
+        self.fused = spec.norm_parts == spec.heads and not spec.gate_first and spec.vdim <= lib.bonsai_lay_rec_fused_vdim()
+        decay = rate = conv_w = freq = None
+        if spec.decay is None:
+            self.g_col, conv, dt = w.columns
+            v, k, q = conv, conv + spec.out_width, conv + spec.out_width + spec.groups * spec.dim
+            rate = torch.exp(vec["A_log"])
+        else:
+            q, k, v, self.g_col = w.columns
+            conv = dt = 0
+            decay = torch.tensor(spec.decay, dtype=torch.float32, device=r.device)
+        if spec.conv:
+            conv_w = vec["conv"].flip(1).t().contiguous()              # [taps][channels], the current token's tap first
+        if spec.rotary is not None:
+            freq = torch.tensor(spec.rotary.frequencies, dtype=torch.float64, device=r.device)
+        floats = [cfg.eps, spec.key_scale, self.scale]
+
+        def call(rows, dst):
+            return L.MixerCall([r.proj, decay, rate, vec.get("dt_bias"), vec.get("D"), self.norm, conv_w, vec.get("conv.b"), s.get("conv"), freq, s["S"],
+                                rows.positions, rows.slots, r.state_table, dst, r.features, r.segment_scratch[0], r.segment_scratch[3]],
+                               [r.proj.stride(0), q, k, v, self.g_col, dt, conv, dst.stride(0), r.features.stride(0), spec.heads, spec.groups, spec.dim,
+                                spec.vdim, int(spec.activation), spec.conv, spec.conv_channels if spec.conv else 0,
+                                spec.rotary.dims if spec.rotary else 0, int(spec.gate == "silu")], floats)
+        # o f32 for the gated norm, and the finished activations of the fused single-token step
+        self.raw = {id(rows): call(rows, r.head_out) for rows in (r.slot_rows, r.batch_rows)}
+        self.done = {id(rows): call(rows, out) for rows in (r.slot_rows, r.batch_rows)}
+
+    def _finish(self, row0: int, count: int) -> None:
+        s = self.spec
+        L.gated_norm(self.r.head_out, row0, self.r.proj, self.g_col, self.norm, self.r.cfg.eps, count, s.norm_parts, s.out_width // s.norm_parts, self.out,
+                     s.gate, s.gate_first, self.scale)
+
+    def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
+        lib, exact = L.lib(), int(self.r.exact)
+        if st.singles and self.fused:
+            K.check(lib.bonsai_lay_rec_step(*self.done[id(rows)].args, None, st.singles, 2, exact, int(early), stream), "rec_step")
+        elif st.singles:
+            K.check(lib.bonsai_lay_rec_step(*self.raw[id(rows)].args, None, st.singles, 1, exact, int(early), stream), "rec_step")
+            self._finish(0, st.singles)
+        if st.portions:
+            a = self.raw[id(rows)].args
+            K.check(lib.bonsai_lay_rec_features(*a, st.singles, st.rows - st.singles, exact, stream), "rec_features")
+            if self.spec.conv:
+                K.check(lib.bonsai_lay_rec_ring(*a, st.entries, st.portions, stream), "rec_ring")
+            if self.chunked:
+                K.check(lib.bonsai_lay_rec_chunk(*a, st.entries, st.portions, st.segment_list, st.segments, st.prompt_list, stream), "rec_chunk")
+            else:
+                K.check(lib.bonsai_lay_rec_step(*a, st.entries, st.portions, 0, exact, 0, stream), "rec_step")
+            self._finish(st.singles, st.rows - st.singles)
+
+    def launches(self) -> int:
+        return 1 if self.fused else 2
+
+
+MIXERS = {"attention": AttentionMixer, "mlstm": MlstmMixer, "recurrence": LinearRecurrenceMixer}
 
 
 class LayeredRunner(SlotState):
@@ -241,7 +351,7 @@ class LayeredRunner(SlotState):
 
     sample_fn = staticmethod(L.sample)
 
-    def __init__(self, weights: LayeredWeights, kv: SharedRowCache, states: StatePool, max_batch: int, max_seq: int, exact: bool = False,
+    def __init__(self, weights: LayeredWeights, kv: RowCache, states: StatePool, max_batch: int, max_seq: int, exact: bool = False,
                  prefill_chunk: int = 4096):
         self.w, self.kv, self.states, self.exact = weights, kv, states, exact
         self.cfg, self.device = weights.cfg, weights.device
@@ -261,39 +371,49 @@ class LayeredRunner(SlotState):
         # activations; the padding columns of the bf16 buffers stay zero for the projections that read them
         self._acts: dict[int, torch.Tensor] = {}
         self.x = torch.zeros((cap, cfg.width), **f32)
-        self.x16 = None if exact else self.act_buffer(cfg.width, shared=False)
+        # input of the next projection; without a norm in between, that of the exact mode is the stream itself
+        self.h = self.x if exact and not cfg.pre_norm else self.act_buffer(cfg.width, shared=False)
         self.normed = self.act_buffer(cfg.width, shared=False)
         self.y = torch.zeros((cap, L.round_up(cfg.width, 4)), **f32)
         self.proj = torch.zeros((cap, max(L.round_up(l.proj.n, 4) for l in weights.layers)), **f32)
-        widths = [cfg.layer_specs[i].mixer.out_width for i in cfg.recurrent_layers]
-        self.head_out = torch.zeros((cap, L.round_up(max(widths, default=4), 4)), **f32)
+        recurrent = [cfg.recurrence(i) for i in cfg.recurrent_layers]
+        self.head_out = torch.zeros((cap, L.round_up(max((m.out_width for m in recurrent), default=4), 4)), **f32)
+        # prepared queries, keys and values of prompt rows
+        linear = [m for m in recurrent if isinstance(m, LinearRecurrenceSpec)]
+        width = max((L.lib().bonsai_lay_rec_features_width(m.heads, m.groups, m.dim, m.vdim) for m in linear), default=8)
+        self.features = torch.zeros((cap if linear else 1, width), dtype=torch.float32 if exact else torch.bfloat16, device=dev)
         # states of the segments a long prompt is cut into (layers run one after another and share them)
-        chunked = [] if exact else [m for m in (cfg.layer_specs[i].mixer for i in cfg.recurrent_layers) if m.dim <= L.lib().bonsai_lay_mlstm_chunk_dim()]
-        self._segment_ctas = min((m.heads * L.lib().bonsai_lay_mlstm_vdim(m.vdim) // 64 for m in chunked), default=0)
-        shapes = [(m.heads, L.lib().bonsai_lay_mlstm_dim(m.dim), L.lib().bonsai_lay_mlstm_vdim(m.vdim)) for m in chunked]
+        chunked = [] if exact else [m for m in recurrent if runs_chunked(m)]
+        shapes = [(m.heads, *state_dims(m)) for m in chunked]
+        self._segment_ctas = min((h * e // 64 for h, _, e in shapes), default=0)
         segs = min(MAX_SEGMENTS, cap // CHUNK) if shapes else 0
         self.segment_scratch = [torch.empty(max(1, segs * max((f(*s) for s in shapes), default=0)), **f32) for f in
                                 (lambda h, d, e: h * d * e, lambda h, d, e: h * d * e // 64, lambda h, d, e: h * e // 64, lambda h, d, e: h * e // 32)]
         # row metadata: decode steps use the slot tensors as they are; a mixed batch uploads [tokens | positions | slots | lists]
         self.slot_rows = Rows(self.tokens, self.positions, torch.arange(max_batch, **i32))
-        self._tile_sizes = sorted({64 // cfg.layer_specs[i].mixer.group for i in cfg.attention_layers})
+        self._tile_sizes = sorted({64 // cfg.attention(i).group for i in cfg.attention_layers})
         self._meta = torch.zeros(3 * cap + 4 * cap + 8 * MAX_SEGMENTS + 2 * cap * len(self._tile_sizes) + cap + 16, **i32)
         self.batch_rows = Rows(*(self._meta[i * cap:(i + 1) * cap] for i in range(3)))
         self._host = [torch.zeros(self._meta.numel(), dtype=torch.int32).pin_memory() for _ in range(2)]
         self._host_free = [torch.cuda.Event() for _ in range(2)]
         self._turn = 0
-        self.mixers = [MIXERS[s.mixer.kind](self, i, s.mixer) for i, s in enumerate(cfg.layer_specs)]
+        self.mixers, self.mixer_out = [], []           # per layer: the branches' mixers and the buffer they write
+        for i, (spec, w) in enumerate(zip(cfg.layer_specs, weights.layers)):
+            widths = tuple(b.spec.out_width for b in spec.mixer.branches)
+            out = self.act_buffer(*widths)
+            self.mixer_out.append(out)
+            self.mixers.append([MIXERS[b.spec.kind](self, i, b, bw, out[:, bw.offset:]) for b, bw in zip(spec.mixer.branches, w.branches)])
         self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
 
-    def act_buffer(self, width: int, shared: bool = True) -> torch.Tensor:
-        """Input buffer of a projection with ``width`` inputs: f32 in the exact mode, else bf16 padded to the tensor-core width.
-        One per width, so that the padding of a narrower layer never holds another layer's values."""
-        if shared and width in self._acts:
-            return self._acts[width]
-        ld = L.round_up(width, 4 if self.exact else L.K_ALIGN)
+    def act_buffer(self, *widths: int, shared: bool = True) -> torch.Tensor:
+        """Input buffer of a projection that reads blocks of ``widths`` columns (:func:`branch_offsets`): f32 in the exact mode, else
+        bf16 padded to the tensor-core width.  One per layout, so that the padding never holds another layer's values."""
+        if shared and widths in self._acts:
+            return self._acts[widths]
+        ld = L.round_up(branch_offsets(widths)[1], 4 if self.exact else L.K_ALIGN)
         t = torch.zeros((self.capacity, ld), dtype=torch.float32 if self.exact else torch.bfloat16, device=self.device)
         if shared:
-            self._acts[width] = t
+            self._acts[widths] = t
         return t
 
     # ---- slots ------------------------------------------------------------------------------------------------------------------
@@ -320,18 +440,21 @@ class LayeredRunner(SlotState):
     # ---- one step ------------------------------------------------------------------------------------------------------------------
     def _layers(self, rows: Rows, st: StepShape) -> None:
         cfg, T, s = self.cfg, st.rows, K.stream()
-        x, x16 = self.x, self.x16
-        h = x if self.exact else x16
-        L.embed(self.w.embed.data, rows.tokens, T, cfg.width, x, x16)
-        for spec, w, mixer in zip(cfg.layer_specs, self.w.layers, self.mixers):
+        x, h, layers = self.x, self.h, self.w.layers
+        copy = None if h is x else h
+        L.embed(self.w.embed.data, rows.tokens, cfg.embed_scale, T, cfg.width, x, copy, layers[0].pre_norm, cfg.eps)
+        for i, (spec, w) in enumerate(zip(cfg.layer_specs, layers)):
+            following = layers[i + 1].pre_norm if i + 1 < len(layers) else None
             L.linear(w.proj, h, T, self.proj, self.scratch)
-            L.linear(w.out, mixer(rows, st, s), T, self.y, self.scratch)
-            L.norm_add(x, self.y, w.norm, cfg.eps, T, x16)
-            if spec.mlp is not None:
+            for n, mixer in enumerate(self.mixers[i]):
+                mixer(rows, st, s, early=n > 0)            # only the first one follows the projection directly
+            L.linear(w.out, self.mixer_out[i], T, self.y, self.scratch)
+            L.norm_add(x, self.y, w.norm, cfg.eps, T, copy, following if w.mlp is None else w.mlp.pre_norm)
+            if w.mlp is not None:
                 act = self.act_buffer(spec.mlp.ff)
-                L.linear(w.mlp.gate_up, h, T, act, self.scratch, (spec.mlp.limit, spec.mlp.alpha, spec.mlp.offset))
+                L.linear(w.mlp.up, h, T, act, self.scratch, w.mlp.act)
                 L.linear(w.mlp.down, act, T, self.y, self.scratch)
-                L.norm_add(x, self.y, w.mlp.norm, cfg.eps, T, x16)
+                L.norm_add(x, self.y, w.mlp.norm, cfg.eps, T, copy, following)
 
     def _head(self, row_list: int | None, count: int, out: torch.Tensor) -> None:
         """Logits of ``count`` rows (device address of their indices, None = the first ones) into ``out`` [count, vocab]."""
@@ -449,6 +572,6 @@ class LayeredRunner(SlotState):
     def kernel_launches(self, batch: int, sample: bool = True) -> int:
         """Launches of one decode step (each is one of this library's kernels)."""
         n = 1 + 2 + int(sample)
-        for spec, mixer in zip(self.cfg.layer_specs, self.mixers):
-            n += 3 + mixer.launches() + (3 if spec.mlp is not None else 0)
+        for spec, mixers in zip(self.cfg.layer_specs, self.mixers):
+            n += 3 + sum(m.launches() for m in mixers) + (3 if spec.mlp is not None else 0)
         return n

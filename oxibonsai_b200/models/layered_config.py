@@ -1,9 +1,12 @@
 """Configuration of decoders that are described layer by layer in a ``config.json``.
 
 A model directory holds ``config.json`` and ``model.safetensors``.  The configuration lists the layers; each entry names its
-mixer (a kind of attention or a recurrence) with its sizes and its feed-forward block.  The specs below are the mechanisms
-with their constants as fields; a *design* (``models.registry.ARCHITECTURES``) is a function that reads a ``config.json`` into
-a :class:`LayeredConfig` and fixes the constants the file does not carry.
+mixer (a kind of attention, a recurrence, or several side by side) with its sizes and its feed-forward block.  The specs below
+are the mechanisms with their constants as fields; a *design* (``models.registry.ARCHITECTURES``) is a function that reads a
+``config.json`` into a :class:`LayeredConfig` and fixes the constants the file does not carry.
+
+Every mixer spec names its tensors: ``sections`` (the matrices that read the mixer's input, as row ranges), ``vectors``, and the
+output matrix "o" with ``out_width`` inputs.
 """
 from __future__ import annotations
 
@@ -18,30 +21,66 @@ class LayeredConfigError(ValueError):
     """A ``config.json`` that is incomplete or describes something the kernels do not cover."""
 
 
+class MixerSpec:
+    """What all mixers have in common: the branches of a layer (one, unless mixers stand side by side)."""
+
+    @property
+    def branches(self) -> tuple["Branch", ...]:
+        return (Branch("", self, 1.0),)
+
+
 @dataclass(frozen=True)
-class AttentionSpec:
-    """Softmax attention over rows that are key and value at once (the values are the un-normalised keys), with query / key norm,
-    a linear distance bias, a sliding window that keeps the first tokens, and one sigmoid gate per head."""
+class Branch:
+    """A mixer of a layer: the prefix of its tensors and the factor of its output in the layer's sum."""
+    prefix: str
+    spec: "AttentionSpec | MlstmSpec | LinearRecurrenceSpec"
+    scale: float
+
+
+@dataclass(frozen=True)
+class AttentionSpec(MixerSpec):
+    """Softmax attention with normalised queries and keys; everything from ``vdim`` on is optional."""
     heads: int
     kv_heads: int
     dim: int
     scale: float
-    window: int                 # positions a query sees, its own included; 0 = all
-    keep_first: int             # first positions that stay visible
-    slope_exponent: float = 8.0
+    vdim: int | None = None     # None: the values are the un-normalised keys (cache rows that are key and value)
+    window: int = 0             # positions a query sees, its own included; 0 = all
+    keep_first: int = 0         # first positions that stay visible
+    slope_exponent: float | None = None    # geometric slopes of a linear distance bias
+    norm_weights: bool = False  # weights of the query and key norms
+    gated: bool = False         # one sigmoid gate per head on the output
+    softcap: float = 0.0        # scores become softcap * tanh(score / softcap); 0 = as they are
+    temp_coef: float = 0.0      # queries are multiplied by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)
+    temp_every: float = 1.0
     kind = "attention"
 
     @property
+    def value_dim(self) -> int:
+        return self.dim if self.vdim is None else self.vdim
+
+    @property
     def out_width(self) -> int:
-        return self.heads * self.dim
+        return self.heads * self.value_dim
 
     @property
     def group(self) -> int:
         return self.heads // self.kv_heads
 
+    @property
+    def sections(self) -> list[tuple[str, int]]:
+        s = [("q", self.heads * self.dim), ("k", self.kv_heads * self.dim)]
+        if self.vdim is not None:
+            s.append(("v", self.kv_heads * self.vdim))
+        return s + ([("g", self.heads)] if self.gated else [])
+
+    @property
+    def vectors(self) -> dict[str, tuple[int, ...]]:
+        return {"q.norm": (self.dim,), "k.norm": (self.dim,)} if self.norm_weights else {}
+
 
 @dataclass(frozen=True)
-class MlstmSpec:
+class MlstmSpec(MixerSpec):
     """Matrix-memory recurrence with capped exponential gates (mLSTM)."""
     heads: int
     dim: int
@@ -54,6 +93,84 @@ class MlstmSpec:
     def out_width(self) -> int:
         return self.heads * self.vdim
 
+    @property
+    def sections(self) -> list[tuple[str, int]]:
+        qk = self.heads * self.dim
+        return [("q", qk), ("k", qk), ("v", self.out_width), ("g", self.out_width), ("i", self.heads), ("f", self.heads)]
+
+    @property
+    def vectors(self) -> dict[str, tuple[int, ...]]:
+        return {"i.b": (self.heads,), "f.b": (self.heads,), "norm": (self.out_width,)}
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first ``dims`` dimensions of a head, dimension i paired with i + dims / 2."""
+    base: float
+    dims: int
+
+    @property
+    def frequencies(self) -> list[float]:
+        return [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+
+
+@dataclass(frozen=True)
+class LinearRecurrenceSpec(MixerSpec):
+    """``S <- a S + b k v^T, o = S^T q`` with one decay per head and token, then a gated norm in ``norm_parts`` equal parts.
+
+    ``decay`` lists fixed decays (b = 1); without it they come from the input (state-space duality): dt = softplus(raw + bias),
+    a = exp(-exp(A_log) dt), b = dt, a skip D per head, and one matrix "in" for all projections.  ``conv`` > 0: a causal
+    convolution of that many taps on values, keys and queries."""
+    heads: int
+    dim: int
+    vdim: int
+    groups: int                         # heads / groups heads share queries and keys
+    norm_parts: int
+    gate: str                           # "silu" or "sigmoid"
+    decay: tuple[float, ...] | None = None
+    activation: bool = False            # silu on queries, keys and values (after the convolution)
+    rotary: RotarySpec | None = None
+    key_scale: float = 1.0
+    conv: int = 0
+    gate_first: bool = False            # the gate comes before the norm
+    norm_weight: bool = False
+    kind = "recurrence"
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_channels(self) -> int:
+        return self.out_width + 2 * self.groups * self.dim
+
+    @property
+    def sections(self) -> list[tuple[str, int]]:
+        if self.decay is None:          # z, then x, B, C (values, keys, queries), then dt
+            return [("in", self.out_width), ("in", self.conv_channels), ("in", self.heads)]
+        qk = self.groups * self.dim
+        return [("q", qk), ("k", qk), ("v", self.out_width), ("g", self.out_width)]
+
+    @property
+    def vectors(self) -> dict[str, tuple[int, ...]]:
+        v: dict[str, tuple[int, ...]] = {"norm": (self.out_width,)} if self.norm_weight else {}
+        if self.conv:
+            v.update({"conv": (self.conv_channels, self.conv), "conv.b": (self.conv_channels,)})
+        if self.decay is None:
+            v.update({"dt_bias": (self.heads,), "A_log": (self.heads,), "D": (self.heads,)})
+        return v
+
+
+@dataclass(frozen=True)
+class ParallelSpec(MixerSpec):
+    """Mixers side by side that read the same input; the scaled sum of their outputs is the layer's."""
+    parts: tuple[Branch, ...]
+    kind = "parallel"
+
+    @property
+    def branches(self) -> tuple[Branch, ...]:
+        return self.parts
+
 
 @dataclass(frozen=True)
 class GatedMlpSpec:
@@ -62,12 +179,20 @@ class GatedMlpSpec:
     limit: float
     alpha: float
     offset: float
+    matrices = ("gate", "up")
+
+
+@dataclass(frozen=True)
+class SquaredReluMlpSpec:
+    """``W_down relu(W_up h)^2``."""
+    ff: int
+    matrices = ("up",)
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | MlstmSpec
-    mlp: GatedMlpSpec | None
+    mixer: MixerSpec
+    mlp: GatedMlpSpec | SquaredReluMlpSpec | None
 
 
 @dataclass(frozen=True)
@@ -78,6 +203,8 @@ class LayeredConfig:
     vocab: int
     eps: float
     layer_specs: tuple[LayerSpec, ...] = field(repr=False)
+    embed_scale: float = 1.0
+    pre_norm: bool = False      # a norm ahead of each sublayer too ("norm1", "norm2"; those on the outputs are then "norm1b", "norm2b")
 
     @property
     def layers(self) -> int:
@@ -87,37 +214,52 @@ class LayeredConfig:
     def hidden(self) -> int:
         return self.width
 
+    def branches(self, i: int, *kinds: str) -> list[Branch]:
+        """The mixers of layer ``i`` of the given kinds."""
+        return [b for b in self.layer_specs[i].mixer.branches if b.spec.kind in kinds]
+
     @property
     def attention_layers(self) -> list[int]:
-        return [i for i, l in enumerate(self.layer_specs) if l.mixer.kind == "attention"]
+        return [i for i in range(self.layers) if self.branches(i, "attention")]
 
     @property
     def recurrent_layers(self) -> list[int]:
-        return [i for i, l in enumerate(self.layer_specs) if l.mixer.kind == "mlstm"]
+        return [i for i in range(self.layers) if self.branches(i, "mlstm", "recurrence")]
+
+    def attention(self, i: int) -> AttentionSpec:
+        return self.branches(i, "attention")[0].spec
+
+    def recurrence(self, i: int) -> MlstmSpec | LinearRecurrenceSpec:
+        return self.branches(i, "mlstm", "recurrence")[0].spec
 
     @property
     def max_visible(self) -> int | None:
         """Most cached tokens a query of any attention layer can see (None: no bound, or no attention layer)."""
-        seen = [self.layer_specs[i].mixer for i in self.attention_layers]
+        seen = [self.attention(i) for i in self.attention_layers]
         return None if not seen or any(m.window <= 0 for m in seen) else max(m.window + m.keep_first for m in seen)
+
+    def norm_names(self, i: int) -> list[tuple[str | None, str]]:
+        """Per sublayer of layer ``i`` the names of the norms of its input (None: none) and of its output."""
+        p = f"l{i}."
+        names = [(p + f"norm{n}", p + f"norm{n}b") if self.pre_norm else (None, p + f"norm{n}") for n in (1, 2)]
+        return names if self.layer_specs[i].mlp is not None else names[:1]
 
     def tensor_shapes(self) -> dict[str, tuple[int, ...]]:
         """Name and shape of every tensor of the checkpoint."""
         w = self.width
         s: dict[str, tuple[int, ...]] = {"embed": (self.vocab, w), "final.norm": (w,)}
         for i, layer in enumerate(self.layer_specs):
-            p, m = f"l{i}.", layer.mixer
-            x = p + "mix."
-            s[p + "norm1"] = (w,)
-            s[x + "q"], s[x + "o"] = (m.heads * m.dim, w), (w, m.out_width)
-            if m.kind == "attention":
-                s.update({x + "k": (m.kv_heads * m.dim, w), x + "q.norm": (m.dim,), x + "k.norm": (m.dim,), x + "g": (m.heads, w)})
-            else:
-                s.update({x + "k": (m.heads * m.dim, w), x + "v": (m.out_width, w), x + "g": (m.out_width, w), x + "norm": (m.out_width,),
-                          x + "i": (m.heads, w), x + "i.b": (m.heads,), x + "f": (m.heads, w), x + "f.b": (m.heads,)})
+            s.update({n: (w,) for pair in self.norm_names(i) for n in pair if n is not None})
+            for b in layer.mixer.branches:
+                x = f"l{i}.mix.{b.prefix}"
+                for name, rows in b.spec.sections:
+                    s[x + name] = (s.get(x + name, (0, w))[0] + rows, w)
+                s.update({x + n: shape for n, shape in b.spec.vectors.items()})
+                s[x + "o"] = (w, b.spec.out_width)
             if layer.mlp is not None:
                 f = layer.mlp.ff
-                s.update({p + "norm2": (w,), p + "mlp.gate": (f, w), p + "mlp.up": (f, w), p + "mlp.down": (w, f)})
+                s.update({f"l{i}.mlp.{n}": (f, w) for n in layer.mlp.matrices})
+                s[f"l{i}.mlp.down"] = (w, f)
         return s
 
     def param_count(self) -> int:
@@ -150,44 +292,122 @@ def _number(d: dict, key: str, where: str) -> float:
     return float(v)
 
 
-def _attention(m: dict, where: str) -> AttentionSpec:
+def _positive(d: dict, key: str, where: str) -> float:
+    v = _number(d, key, where)
+    if not v > 0:
+        raise LayeredConfigError(f"config.json: {where}.{key} must be positive, got {v!r}")
+    return v
+
+
+def _attention_sizes(m: dict, where: str) -> tuple[int, int, int, int]:
     heads, kv, dim, vdim = (_size(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim"))
-    mask = _get(m, "mask", where)
-    if vdim != dim:
-        raise LayeredConfigError(f"config.json: {where}: the values are the keys, so vdim ({vdim}) must equal dim ({dim})")
     if heads % kv or heads // kv > MAX_GROUP:
         raise LayeredConfigError(f"config.json: {where}: {heads} heads over {kv} key/value heads")
-    if dim > MAX_HEAD_DIM:
-        raise LayeredConfigError(f"config.json: {where}: head size {dim} exceeds {MAX_HEAD_DIM}")
-    return AttentionSpec(heads, kv, dim, _number(m, "scale", where), _size(mask, "size", where + ".mask"), _size(mask, "keep_first", where + ".mask", 0))
+    if max(dim, vdim) > MAX_HEAD_DIM:
+        raise LayeredConfigError(f"config.json: {where}: head size {max(dim, vdim)} exceeds {MAX_HEAD_DIM}")
+    return heads, kv, dim, vdim
 
 
-def _mlstm(m: dict, where: str) -> MlstmSpec:
-    heads, dim, vdim = (_size(m, k, where) for k in ("heads", "dim", "vdim"))
+def _state_dim(dim: int, where: str) -> int:
     if dim > MAX_STATE_DIM:
         raise LayeredConfigError(f"config.json: {where}: key size {dim} exceeds {MAX_STATE_DIM}")
-    return MlstmSpec(heads, dim, vdim, _number(m, "gate_cap", where))
+    return dim
 
 
-def keripel_config(raw: dict, name: str = "") -> LayeredConfig:
-    """The Keripel design: mLSTM and windowed-attention mixers in the order the file lists, output norms, gated feed-forward
-    blocks where a layer has one, and a head tied to the embedding."""
-    mixers = {"attention": _attention, "mlstm": _mlstm}
+def _layers(raw: dict, mixers: dict, mlp) -> tuple[LayerSpec, ...]:
+    """The layer list: ``mixers`` reads a mixer by its type, ``mlp`` a dense feed-forward block."""
     layers = []
     for i, entry in enumerate(_get(raw, "layers", "the model")):
         where = f"layers[{i}]"
         kind = _get(entry, "type", where)
         if kind not in mixers:
             raise LayeredConfigError(f"config.json: {where}: unknown mixer type {kind!r}")
-        mixer = mixers[kind](_get(entry, "mixer", where), where + ".mixer")
-        mlp = _get(entry, "mlp", where)
-        if mlp is not None:
-            if _get(mlp, "kind", where + ".mlp") != "dense":
-                raise LayeredConfigError(f"config.json: {where}.mlp: unknown kind {mlp['kind']!r}")
-            mlp = GatedMlpSpec(_size(mlp, "ff", where + ".mlp"), _number(mlp, "limit", where + ".mlp"), alpha=1.702, offset=1.0)
-        layers.append(LayerSpec(mixer, mlp))
+        ff = _get(entry, "mlp", where)
+        if ff is not None and _get(ff, "kind", where + ".mlp") != "dense":
+            raise LayeredConfigError(f"config.json: {where}.mlp: unknown kind {ff['kind']!r}")
+        layers.append(LayerSpec(mixers[kind](_get(entry, "mixer", where), where + ".mixer"), None if ff is None else mlp(ff, where + ".mlp")))
     if not layers:
         raise LayeredConfigError("config.json: the model has no layers")
-    arch = raw.get("architecture", "Keripel")
+    return tuple(layers)
+
+
+def _model(raw: dict, design: str, name: str, layers: tuple[LayerSpec, ...], **extra) -> LayeredConfig:
+    arch = raw.get("architecture", design)
     return LayeredConfig(arch, name or arch, _size(raw, "width", "the model"), _size(raw, "vocab", "the model"),
-                         _number(_get(raw, "norm", "the model"), "eps", "norm"), tuple(layers))
+                         _number(_get(raw, "norm", "the model"), "eps", "norm"), layers, **extra)
+
+
+# ---- Keripel ----------------------------------------------------------------------------------------------------------------------
+def _windowed_attention(m: dict, where: str) -> AttentionSpec:
+    heads, kv, dim, vdim = _attention_sizes(m, where)
+    mask = _get(m, "mask", where)
+    if vdim != dim:
+        raise LayeredConfigError(f"config.json: {where}: the values are the keys, so vdim ({vdim}) must equal dim ({dim})")
+    return AttentionSpec(heads, kv, dim, _number(m, "scale", where), window=_size(mask, "size", where + ".mask"),
+                         keep_first=_size(mask, "keep_first", where + ".mask", 0), slope_exponent=8.0, norm_weights=True, gated=True)
+
+
+def _mlstm(m: dict, where: str) -> MlstmSpec:
+    heads, dim, vdim = (_size(m, k, where) for k in ("heads", "dim", "vdim"))
+    return MlstmSpec(heads, _state_dim(dim, where), vdim, _number(m, "gate_cap", where))
+
+
+def keripel_config(raw: dict, name: str = "") -> LayeredConfig:
+    """The Keripel design: mLSTM and windowed-attention mixers in the order the file lists, output norms, gated feed-forward
+    blocks where a layer has one, and a head tied to the embedding."""
+    mlp = lambda m, where: GatedMlpSpec(_size(m, "ff", where), _number(m, "limit", where), alpha=1.702, offset=1.0)
+    return _model(raw, "Keripel", name, _layers(raw, {"attention": _windowed_attention, "mlstm": _mlstm}, mlp))
+
+
+# ---- Kekevik ----------------------------------------------------------------------------------------------------------------------
+def _decays(m: dict, heads: int, where: str) -> tuple[float, ...]:
+    d = _get(m, "decay", where)
+    if not isinstance(d, list) or len(d) != heads or any(isinstance(x, bool) or not isinstance(x, (int, float)) or not 0 <= x <= 1 for x in d):
+        raise LayeredConfigError(f"config.json: {where}.decay must list {heads} numbers from 0 to 1")
+    return tuple(float(x) for x in d)
+
+
+def _retention(m: dict, where: str) -> LinearRecurrenceSpec:
+    heads, dim, vdim = (_size(m, k, where) for k in ("heads", "dim", "vdim"))
+    rot = _get(m, "rot", where)
+    dims = _size(rot, "dims", where + ".rot", 0)
+    if dims % 2 or dims > dim:
+        raise LayeredConfigError(f"config.json: {where}.rot.dims must be even and at most {dim}, got {dims}")
+    rotary = RotarySpec(_positive(rot, "base", where + ".rot"), dims) if dims else None
+    return LinearRecurrenceSpec(heads, _state_dim(dim, where), vdim, groups=heads, norm_parts=heads, gate="silu", decay=_decays(m, heads, where),
+                                rotary=rotary, key_scale=dim ** -0.5)
+
+
+def _lightning(m: dict, where: str) -> LinearRecurrenceSpec:
+    heads, dim, vdim = (_size(m, k, where) for k in ("heads", "dim", "vdim"))
+    return LinearRecurrenceSpec(heads, _state_dim(dim, where), vdim, groups=heads, norm_parts=1, gate="sigmoid", decay=_decays(m, heads, where),
+                                activation=True, norm_weight=True)
+
+
+def _capped_attention(m: dict, where: str) -> AttentionSpec:
+    heads, kv, dim, vdim = _attention_sizes(m, where)
+    temp = _get(m, "q_temp", where)
+    return AttentionSpec(heads, kv, dim, _number(m, "scale", where), vdim=vdim, softcap=_positive(m, "softcap", where),
+                         temp_coef=_number(temp, "coef", where + ".q_temp"), temp_every=_positive(temp, "every", where + ".q_temp"))
+
+
+def _mamba2(m: dict, where: str) -> LinearRecurrenceSpec:
+    heads, vdim, state, groups, parts, taps = (_size(m, k, where) for k in ("heads", "vdim", "state", "groups", "norm_groups", "conv"))
+    if heads % groups or heads * vdim % parts:
+        raise LayeredConfigError(f"config.json: {where}: {heads} heads of {vdim} values over {groups} groups and {parts} norm groups")
+    return LinearRecurrenceSpec(heads, _state_dim(state, where), vdim, groups=groups, norm_parts=parts, gate="silu", activation=True, conv=taps,
+                                gate_first=True, norm_weight=True)
+
+
+def _side_by_side(m: dict, where: str) -> ParallelSpec:
+    return ParallelSpec((Branch("left.", _capped_attention(_get(m, "left", where), where + ".left"), _number(m, "left_scale", where)),
+                         Branch("right.", _mamba2(_get(m, "right", where), where + ".right"), _number(m, "right_scale", where))))
+
+
+def kekevik_config(raw: dict, name: str = "") -> LayeredConfig:
+    """The Kekevik design: retention, lightning attention, and capped attention beside a state-space mixer, in the order the
+    file lists; norms before and after each sublayer, squared-relu feed-forward blocks, a scaled embedding tied to the head."""
+    layers = _layers(raw, {"retention": _retention, "lightning": _lightning, "parallel": _side_by_side},
+                     lambda m, where: SquaredReluMlpSpec(_size(m, "ff", where)))
+    scale = _number(_get(raw, "embedding", "the model"), "scale", "embedding")
+    return _model(raw, "Kekevik", name, layers, embed_scale=scale, pre_norm=True)

@@ -2,7 +2,7 @@
 
 Reference: ``BlockPool`` / ``BlockTable`` (crates/oxibonsai-model/src/paged_kv_cache.rs:33-557) for the pages; recurrent state
 has no counterpart there.  ``PagePool`` hands out reference-counted pages; the caches (``PagedKvCache`` in ``qwen3``,
-``SharedRowCache`` here) own the tensors the pages index.  ``StatePool`` hands out one state row per sequence.
+``RowCache`` here) own the tensors the pages index.  ``StatePool`` hands out one state row per sequence.
 """
 from __future__ import annotations
 
@@ -44,20 +44,27 @@ class PagePool:
         return 1.0 - len(self.free_pages) / max(1, self.num_pages)
 
 
-class SharedRowCache(PagePool):
-    """Paged cache of attention layers whose rows serve as key and value: per layer ``rows`` [pages, kv_heads, page_size, row]
-    and one float per row (the key's reciprocal root mean square).  ``layers``: {layer index: (kv heads, row elements)};
-    layers may differ, they share the page numbering."""
+class RowCache(PagePool):
+    """Paged cache of attention layers: per layer ``rows`` [pages, kv_heads, page_size, row], the keys, and beside them either
+    ``values`` of the same shape, or, where the rows serve as key and value, one float per row (``factors``: the key's
+    reciprocal root mean square).  ``layers``: {layer index: (kv heads, row elements, separate values)}; layers may differ, they
+    share the page numbering."""
 
-    def __init__(self, layers: dict[int, tuple[int, int]], num_pages: int, page_size: int, kvt: int, dtype: torch.dtype, device):
+    def __init__(self, layers: dict[int, tuple[int, int, bool]], num_pages: int, page_size: int, kvt: int, dtype: torch.dtype, device):
         super().__init__(num_pages, page_size)
         self.kvt = kvt
-        self.rows = {l: torch.zeros((num_pages, h, page_size, row), dtype=dtype, device=device) for l, (h, row) in layers.items()}
-        self.factors = {l: torch.zeros((num_pages, h, page_size), dtype=torch.float32, device=device) for l, (h, _) in layers.items()}
+        self.rows, self.values, self.factors = {}, {}, {}
+        for l, (h, row, separate) in layers.items():
+            new = lambda *shape, dtype=dtype: torch.zeros((num_pages, h, page_size, *shape), dtype=dtype, device=device)
+            self.rows[l] = new(row)
+            if separate:
+                self.values[l] = new(row)
+            else:
+                self.factors[l] = new(dtype=torch.float32)
 
     @property
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.rows, self.factors) for t in d.values())
+        return sum(t.numel() * t.element_size() for d in (self.rows, self.values, self.factors) for t in d.values())
 
 
 class StatePool:

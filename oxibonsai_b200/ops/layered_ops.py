@@ -3,6 +3,7 @@ tcgen05 GEMM).  Every function launches on torch's current stream; there is no P
 from __future__ import annotations
 
 import ctypes as C
+from dataclasses import dataclass
 
 import torch
 
@@ -11,10 +12,10 @@ from . import cuda_ops as K
 
 _vp, _i, _f = C.c_void_p, C.c_int, C.c_float
 _SIG = {
-    "bonsai_lay_embed": [_vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp],
-    "bonsai_lay_norm_add": [_vp, _vp, _i, _vp, _f, _i, _i, _vp, _i, _vp],
+    "bonsai_lay_embed": [_vp, _i, _vp, _f, _i, _i, _vp, _vp, _i, _i, _vp, _f, _vp],
+    "bonsai_lay_norm_add": [_vp, _vp, _i, _vp, _f, _i, _i, _vp, _i, _i, _vp, _vp],
     "bonsai_lay_norm_rows": [_vp, _vp, _vp, _f, _i, _i, _vp, _i, _i, _vp],
-    "bonsai_lay_gated_head_norm": [_vp, _i, _vp, _i, _vp, _f, _i, _i, _i, _vp, _i, _i, _vp],
+    "bonsai_lay_gated_norm": [_vp, _i, _vp, _i, _vp, _f, _i, _i, _i, _i, _i, _f, _vp, _i, _i, _vp],
     "bonsai_lay_linear_few": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _vp],
     "bonsai_lay_linear_f32": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
     "bonsai_dense_gemm_bf16": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _vp, _vp, C.c_size_t, _i, _vp],
@@ -31,6 +32,15 @@ _SIG = {
     "bonsai_lay_mlstm_step": [_vp, _vp, _vp, _vp, _i, _i, _vp],
     "bonsai_lay_mlstm_chunk_tokens": [],
     "bonsai_lay_mlstm_chunk": [_vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _vp],
+    "bonsai_lay_rec_dim": [_i],
+    "bonsai_lay_rec_vdim": [_i],
+    "bonsai_lay_rec_features_width": [_i, _i, _i, _i],
+    "bonsai_lay_rec_chunk_dim": [],
+    "bonsai_lay_rec_fused_vdim": [],
+    "bonsai_lay_rec_features": [_vp, _vp, _vp, _i, _i, _i, _vp],
+    "bonsai_lay_rec_ring": [_vp, _vp, _vp, _vp, _i, _vp],
+    "bonsai_lay_rec_step": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "bonsai_lay_rec_chunk": [_vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _vp],
     "bonsai_sample": K._SIG["bonsai_sample"],
 }
 _lib = None
@@ -92,35 +102,54 @@ class GemmScratch:
         self.sms = torch.cuda.get_device_properties(device).multi_processor_count
 
 
-def linear(w: DenseWeight, x: torch.Tensor, T: int, out: torch.Tensor, scratch: GemmScratch, glu: tuple[float, float, float] | None = None) -> None:
-    """out[:T] = x[:T] W^T.  bf16 ``x`` (row stride >= kp, finite in the padding): tensor cores, f32 ``out`` (bf16 with
-    ``glu``); f32 ``x``: 32-bit throughout.  ``glu`` = (limit, alpha, offset): gated unit over interleaved rows."""
+@dataclass(frozen=True)
+class Glu:
+    """Clamped gated unit over interleaved gate / up rows."""
+    limit: float
+    alpha: float
+    offset: float
+
+
+SQUARED_RELU = "squared_relu"
+_NO_GLU = Glu(0.0, 0.0, 0.0)
+
+
+def linear(w: DenseWeight, x: torch.Tensor, T: int, out: torch.Tensor, scratch: GemmScratch, act: Glu | str | None = None) -> None:
+    """out[:T] = act(x[:T] W^T).  bf16 ``x`` (row stride >= kp, finite in the padding): tensor cores, f32 ``out`` (bf16 with
+    ``act``); f32 ``x``: 32-bit throughout.  ``act``: none, :class:`Glu`, or ``SQUARED_RELU``."""
     l, s = lib(), K.stream()
-    lim, alpha, off = glu if glu is not None else (0.0, 0.0, 0.0)
+    glu = act if isinstance(act, Glu) else _NO_GLU
+    epi = 0 if act is None else (1 if isinstance(act, Glu) else 2)
     if x.dtype == torch.float32:
         K.check(l.bonsai_lay_linear_f32(w.data.data_ptr(), w.n, w.k, w.kp, x.data_ptr(), x.stride(0), T, out.data_ptr(), out.stride(0),
-                                        int(glu is not None), lim, alpha, off, s), "linear_f32")
+                                        epi, glu.limit, glu.alpha, glu.offset, s), "linear_f32")
         return
-    assert x.dtype == torch.bfloat16 and out.dtype == (torch.float32 if glu is None else torch.bfloat16)
-    f32, b16 = (out.data_ptr(), None) if glu is None else (None, out.data_ptr())
+    assert x.dtype == torch.bfloat16 and out.dtype == (torch.float32 if act is None else torch.bfloat16)
+    f32, b16 = (out.data_ptr(), None) if act is None else (None, out.data_ptr())
     if T <= FEW_ROWS:
-        K.check(l.bonsai_lay_linear_few(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), int(glu is not None),
-                                        lim, alpha, off, s), "linear_few")
+        K.check(l.bonsai_lay_linear_few(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), epi,
+                                        glu.limit, glu.alpha, glu.offset, s), "linear_few")
     else:
         K.check(l.bonsai_dense_gemm_bf16(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0),
-                                         0 if glu is None else 4, lim, alpha, off, scratch.status.data_ptr(), scratch.ws.data_ptr(),
+                                         (0, 4, 5)[epi], glu.limit, glu.alpha, glu.offset, scratch.status.data_ptr(), scratch.ws.data_ptr(),
                                          scratch.ws.numel(), scratch.sms, s), "dense_gemm_bf16")
 
 
-def embed(table: torch.Tensor, tokens: torch.Tensor, T: int, width: int, x: torch.Tensor, x16: torch.Tensor | None) -> None:
-    K.check(lib().bonsai_lay_embed(table.data_ptr(), table.stride(0), tokens.data_ptr(), T, width, x.data_ptr(), K.ptr(x16),
-                                   0 if x16 is None else x16.stride(0), K.stream()), "embed")
+def _row_out(t: torch.Tensor | None) -> tuple[int | None, int, int]:
+    return (None, 0, 0) if t is None else (t.data_ptr(), t.stride(0), int(t.dtype == torch.float32))
 
 
-def norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, T: int, x16: torch.Tensor | None) -> None:
-    """x += rmsnorm(y) * w over the first T rows; ``x16`` receives the bf16 copy."""
-    K.check(lib().bonsai_lay_norm_add(x.data_ptr(), y.data_ptr(), y.stride(0), w.data_ptr(), eps, T, x.shape[1], K.ptr(x16),
-                                      0 if x16 is None else x16.stride(0), K.stream()), "norm_add")
+def embed(table: torch.Tensor, tokens: torch.Tensor, scale: float, T: int, width: int, x: torch.Tensor, h: torch.Tensor | None,
+          next_norm: torch.Tensor | None, eps: float) -> None:
+    """x = table[tokens] * scale; ``h`` receives x, or its norm with weight ``next_norm``."""
+    K.check(lib().bonsai_lay_embed(table.data_ptr(), table.stride(0), tokens.data_ptr(), scale, T, width, x.data_ptr(), *_row_out(h), K.ptr(next_norm), eps,
+                                   K.stream()), "embed")
+
+
+def norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, T: int, h: torch.Tensor | None, next_norm: torch.Tensor | None = None) -> None:
+    """x += rmsnorm(y) * w over the first T rows; ``h`` receives x, or its norm with weight ``next_norm``."""
+    K.check(lib().bonsai_lay_norm_add(x.data_ptr(), y.data_ptr(), y.stride(0), w.data_ptr(), eps, T, x.shape[1], *_row_out(h), K.ptr(next_norm), K.stream()),
+            "norm_add")
 
 
 def norm_rows(x: torch.Tensor, rows: int | None, count: int, w: torch.Tensor, eps: float, out: torch.Tensor) -> None:
@@ -129,21 +158,22 @@ def norm_rows(x: torch.Tensor, rows: int | None, count: int, w: torch.Tensor, ep
                                        int(out.dtype == torch.float32), K.stream()), "norm_rows")
 
 
-def gated_head_norm(o: torch.Tensor, row0: int, gate: torch.Tensor, gate_col: int, w: torch.Tensor, eps: float, T: int, heads: int, vdim: int,
-                    out: torch.Tensor) -> None:
-    """out[row] = o / rms(o per head) * w * sigmoid(gate) for rows row0 .. row0 + T - 1 of all three."""
-    K.check(lib().bonsai_lay_gated_head_norm(o.data_ptr() + 4 * row0 * o.stride(0), o.stride(0), gate.data_ptr() + 4 * (row0 * gate.stride(0) + gate_col),
-                                             gate.stride(0), w.data_ptr(), eps, T, heads, vdim,
-                                             out.data_ptr() + out.element_size() * row0 * out.stride(0), out.stride(0),
-                                             int(out.dtype == torch.float32), K.stream()), "gated_head_norm")
+def gated_norm(o: torch.Tensor, row0: int, gate: torch.Tensor, gate_col: int, w: torch.Tensor | None, eps: float, T: int, parts: int, width: int,
+               out: torch.Tensor, act: str = "sigmoid", gate_first: bool = False, scale: float = 1.0) -> None:
+    """Rows row0 .. row0 + T - 1 of all three, in ``parts`` parts of ``width`` columns with their own root mean square:
+    out = o / rms(o) * w * act(gate) * scale, or with ``gate_first`` the same of o * act(gate) without a gate behind."""
+    K.check(lib().bonsai_lay_gated_norm(o.data_ptr() + 4 * row0 * o.stride(0), o.stride(0), gate.data_ptr() + 4 * (row0 * gate.stride(0) + gate_col),
+                                        gate.stride(0), K.ptr(w), eps, T, parts, width, {"sigmoid": 0, "silu": 1}[act], int(gate_first), scale,
+                                        out.data_ptr() + out.element_size() * row0 * out.stride(0), out.stride(0), int(out.dtype == torch.float32),
+                                        K.stream()), "gated_norm")
 
 
 class MixerCall:
     """The argument blocks (pointers, sizes, constants) of one mixer's launches; the tensors must outlive it."""
 
-    def __init__(self, ptrs: list[torch.Tensor], ints: list[int], floats: list[float]):
+    def __init__(self, ptrs: list[torch.Tensor | None], ints: list[int], floats: list[float]):
         self._keep = ptrs
-        self.ptrs = (_vp * len(ptrs))(*[t.data_ptr() for t in ptrs])
+        self.ptrs = (_vp * len(ptrs))(*[K.ptr(t) for t in ptrs])
         self.ints = (_i * len(ints))(*ints)
         self.floats = (_f * len(floats))(*floats)
 

@@ -109,19 +109,140 @@ def dense_ff(x, w, p, limit):
     return linear(clamped_glu(linear(x, w[p + "gate"]), linear(x, w[p + "up"]), limit), w[p + "down"])
 
 
-MIXERS = {"attention": attention_mixer, "mlstm": mlstm_mixer}
+# ---- recurrences with a decay and no normaliser ----------------------------------------------------------------------------------
+def silu(x):
+    return x * torch.sigmoid(x)
+
+
+def rotate_half(x, first_position, base, dims):
+    """x [n, heads, d]: dimension i pairs with i + dims / 2; dimensions from ``dims`` on pass."""
+    n, half = x.shape[0], dims // 2
+    pos = torch.arange(first_position, first_position + n, dtype=x.dtype)
+    freq = torch.tensor([base ** (-2.0 * i / dims) for i in range(half)], dtype=x.dtype)
+    a = pos[:, None] * freq[None, :]
+    c, s = torch.cos(a)[:, None, :], torch.sin(a)[:, None, :]
+    u, v = x[..., :half], x[..., half:dims]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], dim=-1)
+
+
+def decayed_memory(q, k, v, a, b, state=None):
+    """One head, token by token: S <- a_t S + b_t k_t v_t^T, o_t = S^T q_t.  q, k [n, d], v [n, e], a, b [n].  Returns (o, S)."""
+    S = torch.zeros(q.shape[1], v.shape[1], dtype=q.dtype) if state is None else state
+    out = []
+    for t in range(q.shape[0]):
+        S = a[t] * S + b[t] * torch.outer(k[t], v[t])
+        out.append(S.T @ q[t])
+    return torch.stack(out), S
+
+
+def fixed_decay_heads(q, k, v, decay):
+    """q, k [n, H, d], v [n, H, e] -> o [n, H, e]."""
+    one = torch.ones(q.shape[0], dtype=q.dtype)
+    return torch.stack([decayed_memory(q[:, h], k[:, h], v[:, h], decay[h] * one, one)[0] for h in range(q.shape[1])], dim=1)
+
+
+def retention_mixer(h, w, p, m, eps):
+    n, H, d, e = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    rot = lambda x: rotate_half(x.view(n, H, d), 0, m["rot"]["base"], m["rot"]["dims"])
+    q, k = rot(linear(h, w[p + "q"])), rot(linear(h, w[p + "k"])) * d ** -0.5
+    o = fixed_decay_heads(q, k, linear(h, w[p + "v"]).view(n, H, e), m["decay"])
+    return linear(rms(o, eps).reshape(n, H * e) * silu(linear(h, w[p + "g"])), w[p + "o"])
+
+
+def lightning_mixer(h, w, p, m, eps):
+    n, H, d, e = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    q, k, v = (silu(linear(h, w[p + c])) for c in "qkv")
+    o = fixed_decay_heads(q.view(n, H, d), k.view(n, H, d), v.view(n, H, e), m["decay"]).reshape(n, H * e)
+    return linear(rms_norm(o, w[p + "norm"], eps) * torch.sigmoid(linear(h, w[p + "g"])), w[p + "o"])
+
+
+def causal_conv(x, weight, bias):
+    """x [n, C], weight [C, taps]: the last column is the current token's; zeros before the start."""
+    taps = weight.shape[1]
+    out = bias.expand_as(x).clone()
+    for j in range(taps):
+        back = taps - 1 - j
+        if back < x.shape[0]:
+            out[back:] += x[: x.shape[0] - back] * weight[:, j]
+    return out
+
+
+def grouped_rms(x, parts, eps):
+    return rms(x.reshape(x.shape[0], parts, -1), eps).reshape(x.shape)
+
+
+def mamba2_mixer(h, w, p, m, eps):
+    n, H, e, N, G = h.shape[0], m["heads"], m["vdim"], m["state"], m["groups"]
+    inner = H * e
+    z, xbc, dt = torch.split(linear(h, w[p + "in"]), [inner, inner + 2 * G * N, H], dim=-1)
+    xbc = silu(causal_conv(xbc, w[p + "conv"], w[p + "conv.b"]))
+    x, B, C = torch.split(xbc, [inner, G * N, G * N], dim=-1)
+    x, B, C = x.reshape(n, H, e), B.reshape(n, G, N), C.reshape(n, G, N)
+    dt = torch.nn.functional.softplus(dt + w[p + "dt_bias"])
+    a = torch.exp(-torch.exp(w[p + "A_log"]) * dt)
+    y = torch.stack([decayed_memory(C[:, i // (H // G)], B[:, i // (H // G)], x[:, i], a[:, i], dt[:, i])[0] + w[p + "D"][i] * x[:, i] for i in range(H)], dim=1)
+    y = grouped_rms(y.reshape(n, inner) * silu(z), m["norm_groups"], eps) * w[p + "norm"]
+    return linear(y, w[p + "o"])
+
+
+# ---- softmax attention with normalised heads, a query temperature and capped scores -------------------------------------------------
+def query_temperature(n, coef, every):
+    return torch.tensor([1.0 + coef * math.log(math.floor((p + 1) / every) + 1) for p in range(n)], dtype=torch.float64)
+
+
+def capped_attention(q, k, v, scale, softcap):
+    """One head over all earlier positions."""
+    n = q.shape[0]
+    s = soft_cap((q @ k.T) * scale, softcap)
+    return torch.softmax(s.masked_fill(torch.ones(n, n).triu(1).bool(), float("-inf")), dim=-1) @ v
+
+
+def capped_attention_mixer(h, w, p, m, eps):
+    n, H, G, d, e = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q, k = rms(linear(h, w[p + "q"]).view(n, H, d), eps), rms(linear(h, w[p + "k"]).view(n, G, d), eps)
+    v = linear(h, w[p + "v"]).view(n, G, e)
+    q = q * query_temperature(n, m["q_temp"]["coef"], m["q_temp"]["every"]).to(q.dtype)[:, None, None]
+    o = torch.stack([capped_attention(q[:, a], k[:, a // (H // G)], v[:, a // (H // G)], m["scale"], m["softcap"]) for a in range(H)], dim=1)
+    return linear(o.reshape(n, H * e), w[p + "o"])
+
+
+def parallel_mixer(h, w, p, m, eps):
+    return m["left_scale"] * capped_attention_mixer(h, w, p + "left.", m["left"], eps) + m["right_scale"] * mamba2_mixer(h, w, p + "right.", m["right"], eps)
+
+
+def squared_relu_ff(x, w, p):
+    return linear(torch.relu(linear(x, w[p + "up"])) ** 2, w[p + "down"])
+
+
+# ---- whole models -----------------------------------------------------------------------------------------------------------------
+MIXERS = {"attention": attention_mixer, "mlstm": mlstm_mixer, "retention": retention_mixer, "lightning": lightning_mixer, "parallel": parallel_mixer}
+
+
+def keripel_layer(x, w, p, layer, eps):
+    """Norms on the sublayers' outputs only."""
+    x = x + rms_norm(MIXERS[layer["type"]](x, w, p + "mix.", layer["mixer"], eps), w[p + "norm1"], eps)
+    if layer["mlp"] is not None:
+        x = x + rms_norm(dense_ff(x, w, p + "mlp.", layer["mlp"]["limit"]), w[p + "norm2"], eps)
+    return x
+
+
+def kekevik_layer(x, w, p, layer, eps):
+    """A norm before and a norm after each sublayer."""
+    y = MIXERS[layer["type"]](rms_norm(x, w[p + "norm1"], eps), w, p + "mix.", layer["mixer"], eps)
+    x = x + rms_norm(y, w[p + "norm1b"], eps)
+    if layer["mlp"] is not None:
+        x = x + rms_norm(squared_relu_ff(rms_norm(x, w[p + "norm2"], eps), w, p + "mlp."), w[p + "norm2b"], eps)
+    return x
 
 
 def forward(cfg, w, tokens, keep_layers=False):
     """Logits [n, vocab] of every position (and the residual stream after every layer)."""
     eps = cfg["norm"]["eps"]
-    x = w["embed"][torch.as_tensor(list(tokens), dtype=torch.long)]
+    run = {"Keripel": keripel_layer, "Kekevik": kekevik_layer}[cfg["architecture"]]
+    x = w["embed"][torch.as_tensor(list(tokens), dtype=torch.long)] * cfg.get("embedding", {}).get("scale", 1.0)
     kept = []
     for l, layer in enumerate(cfg["layers"]):
-        p = f"l{l}."
-        x = x + rms_norm(MIXERS[layer["type"]](x, w, p + "mix.", layer["mixer"], eps), w[p + "norm1"], eps)
-        if layer["mlp"] is not None:
-            x = x + rms_norm(dense_ff(x, w, p + "mlp.", layer["mlp"]["limit"]), w[p + "norm2"], eps)
+        x = run(x, w, f"l{l}.", layer, eps)
         kept.append(x)
     logits = linear(rms_norm(x, w["final.norm"], eps), w["embed"])
     return (logits, torch.stack(kept)) if keep_layers else logits
