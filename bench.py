@@ -58,8 +58,8 @@ def parse_args():
     ap.add_argument("--no-replicas", action="store_true", help="skip the independent-replica measurement at N > 1")
     ap.add_argument("--no-gate", action="store_true", help="skip the correctness gate")
     ap.add_argument("--no-extras", action="store_true", help="skip the exact-f32 and NCCL-baseline measurements")
-    ap.add_argument("--design", choices=["keripel"], help="instead of the headline: prefill and decode throughput of a layer-list design beside "
-                    "the generic-format engine at equal parameter count (1 GPU)")
+    ap.add_argument("--design", choices=["keripel", "kekevik"], help="instead of the headline: prefill and decode throughput of a layer-list "
+                    "design beside the closest existing model (keripel: the generic-format engine; kekevik: keripel) at equal parameter count (1 GPU)")
     ap.add_argument("--design-sizes", default="s,m,l", help="--design: model sizes (benchmarks/layered.py)")
     ap.add_argument("--model-dir", default=os.environ.get("BONSAI_BENCH_DIR", "/tmp/oxibonsai_b200_bench"))
     return ap.parse_args()
@@ -262,15 +262,16 @@ def run_gate(args, world: int, rank: int, local_rank: int) -> dict:
 
 
 def design_bench(args) -> None:
-    """One JSON line: the layer-list design and the generic-format f16 engine at the same sizes, random weights."""
+    """One JSON line: the layer-list design and the closest existing model at the same sizes, random weights."""
     sys.path.insert(0, os.path.join(HERE, "benchmarks"))
     import layered
     import torch
     torch.cuda.set_device(0)
     clocks = ClockSampler(0)
     clocks.start()
-    rows = layered.run_models(args.design_sizes.split(","), steps=args.steps, warmup=max(3, args.warmup), log=sys.stderr)
-    print(json.dumps({"metric": f"prefill and decode tokens/s, {args.design} design beside the generic-format f16 engine", "unit": "tokens/s", "n_gpus": 1,
+    run, like = {"keripel": (layered.run_models, "the generic-format f16 engine"), "kekevik": (layered.run_kekevik, "the keripel design")}[args.design]
+    rows = run(args.design_sizes.split(","), steps=args.steps, warmup=max(3, args.warmup), log=sys.stderr)
+    print(json.dumps({"metric": f"prefill and decode tokens/s, {args.design} design beside {like}", "unit": "tokens/s", "n_gpus": 1,
                       "steps": args.steps, "warmup": max(3, args.warmup), "higher_is_better": True, "dtype": "bf16", "data": "synthetic (random weights and tokens)",
                       "config": {"prompt_len": 2048, "l2": "no flush between steps; weights and caches of a step exceed L2 except for size s at batch 1"},
                       "clocks": clocks.stop(), "sizes": rows}))

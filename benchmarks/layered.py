@@ -1,8 +1,9 @@
 #!/usr/bin/env python
-"""Layer-list decoders (Keripel) beside the closest existing model, the generic-format Qwen3 engine with f16 weights.
+"""Layer-list decoders beside the closest existing model: Keripel beside the generic-format Qwen3 engine with f16 weights,
+Kekevik beside Keripel.
 
-    python benchmarks/layered.py kernels [--width 4096]     every kernel of the design and its counterpart, with roofline fractions
-    python benchmarks/layered.py models  [--sizes s,m]      prefill and decode throughput at equal parameter count
+    python benchmarks/layered.py kernels [--width 4096] [--only ..]     the kernels and their counterparts, with roofline fractions
+    python benchmarks/layered.py models --design kekevik [--sizes s,m]  prefill and decode throughput at equal parameter count
 
 Random weights, random tokens.  Kernels: CUDA events around a CUDA graph of repeated launches that walks through enough copies
 of its inputs to exceed L2; the roofline is the slower of bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate.
@@ -25,7 +26,7 @@ from kernels import peaks, time_us
 F16 = 1
 
 
-def design(width: int, repeats: int, vocab: int = 32000, window: int = 1024) -> dict:
+def keripel(width: int, repeats: int, vocab: int = 32000, window: int = 1024) -> dict:
     """``repeats`` times three recurrent layers and one attention layer with a feed-forward block."""
     m = {"type": "mlstm", "mixer": {"heads": max(2, width // 512), "dim": 256, "vdim": 512, "gate_cap": 15.0}, "mlp": None}
     a = {"type": "attention", "mixer": {"heads": width // 128, "kv_heads": max(1, width // 512), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
@@ -34,21 +35,38 @@ def design(width: int, repeats: int, vocab: int = 32000, window: int = 1024) -> 
     return {"architecture": "Keripel", "layers": [m, m, m, a] * repeats, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width}
 
 
+def kekevik(width: int, repeats: int, vocab: int = 32000) -> dict:
+    """``repeats`` times a lightning layer, two layers of attention beside a state-space mixer, and a retention layer."""
+    H = width // 128
+    decay = lambda n: [1.0 - 2.0 ** (-5.0 - 6.0 * i / max(1, n - 1)) for i in range(n)]
+    ff = {"kind": "dense", "ff": 4 * width}
+    light = {"type": "lightning", "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": decay(H)}, "mlp": ff}
+    both = {"type": "parallel", "mlp": ff, "mixer": {
+        "left": {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0, "q_temp": {"coef": 0.1, "every": 4096}},
+        "right": {"heads": width // 64, "vdim": 64, "state": 128, "groups": max(1, H // 4), "norm_groups": max(1, H // 4), "conv": 4},
+        "left_scale": 0.5, "right_scale": 0.5}}
+    n = max(1, width // 256)
+    ret = {"type": "retention", "mlp": ff, "mixer": {"heads": n, "dim": 256, "vdim": 256, "decay": decay(n), "rot": {"base": 10000.0, "dims": 256}}}
+    return {"architecture": "Kekevik", "layers": [light, both, both, ret] * repeats, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width,
+            "embedding": {"scale": float(width ** 0.5)}}
+
+
 def write_design(path: str, cfg: dict) -> int:
     """A model directory with random bf16 weights; returns the parameter count."""
     from oxibonsai_b200.convert import write_safetensors
-    from oxibonsai_b200.models.layered_config import keripel_config
+    from oxibonsai_b200.models.registry import ARCHITECTURES
+    config = ARCHITECTURES[cfg["architecture"]](cfg, "")
     os.makedirs(path, exist_ok=True)
     with open(os.path.join(path, "config.json"), "w") as f:
         json.dump(cfg, f)
     g = torch.Generator(device="cuda").manual_seed(0)
     t = {}
-    for n, s in keripel_config(cfg).tensor_shapes().items():
+    for n, s in config.tensor_shapes().items():
         x = torch.randn(s, generator=g, device="cuda")
         x = 1 + 0.1 * x if "norm" in n else (x if len(s) == 1 else x * s[-1] ** -0.5)
         t[n] = x.bfloat16().cpu()
     write_safetensors(os.path.join(path, "model.safetensors"), t)
-    return keripel_config(cfg).param_count()
+    return config.param_count()
 
 
 class Report:
@@ -79,6 +97,13 @@ def bench_linear(rep: Report, width: int, iters: int, profile: bool) -> None:
             ws.append(w)
         for T in (1, 8, 32, 64, 256, 4096):
             x = torch.randn(T, k, device=dev).bfloat16()
+            if name == "gate_up":                # an ungated block's up projection of the same bytes
+                sq, turn = torch.empty(T, n, dtype=torch.bfloat16, device=dev), [0]
+
+                def relu2():
+                    turn[0] += 1
+                    L.linear(ws[turn[0] % copies], x, T, sq, scratch, L.SQUARED_RELU)
+                rep.add("linear, squared relu", f"up {n}x{k} T={T}", time_us(relu2, iters, profile), 2 * n * k + 2 * T * k + 2 * T * n, 2.0 * T * n * k)
             glu = L.Glu(7.0, 1.702, 1.0) if name == "gate_up" else None
             out = torch.empty(T, n // 2 if glu else n, dtype=torch.bfloat16 if glu else torch.float32, device=dev)
             it = [0]
@@ -164,6 +189,114 @@ def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
     kp, vp = torch.randn(npages, nkv, page, hd, device=dev).half(), torch.randn(npages, nkv, page, hd, device=dev).half()
     rep.add("attn_prefill", f"T={T} heads={nq}/{nkv}", time_us(lambda: K.attn_prefill(q, 0, bt[0], nq, nkv, hd, K.KV_F16, page, kp, vp, out=o16), 10, profile),
             4 * T * nq * hd + 4 * T * nkv * hd + 2 * T * nq * hd, 4.0 * T * (T + 1) / 2 * nq * hd, "attn_prompt")
+
+
+def bench_capped_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
+    """Attention with separate values, capped scores and a query temperature; the like kernels are those of bench_attention."""
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    nq, nkv, hd, page = width // 128, max(1, width // 512), 128, 64
+    i32 = dict(dtype=torch.int32, device=dev)
+    ld = (nq + 2 * nkv) * hd
+
+    def call(proj, pos, slots, bt, k, v, out, cap=50.0):
+        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out],
+                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0], [1e-6, hd ** -0.5, 0.5, cap, 0.1, 4096.0])
+    for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
+        npages = ctx // page
+        copies = max(2, int(300e6 / (4 * B * ctx * nkv * hd)) + 1)
+        pools = [[torch.randn(B * npages, nkv, page, hd, device=dev).bfloat16() for _ in range(2)] for _ in range(copies)]
+        bt = torch.arange(B * npages, **i32).view(B, npages)
+        pos, slots, proj = torch.full((B,), ctx - 1, **i32), torch.arange(B, **i32), torch.randn(B, ld, device=dev)
+        out = torch.zeros(B, nq * hd, dtype=torch.bfloat16, device=dev)
+        calls = [call(proj, pos, slots, bt, *p, out) for p in pools]
+        it, split = [0], 1
+        while split < 8 and B * nkv * split * 2 <= 160:
+            split *= 2
+
+        def ours():
+            it[0] += 1
+            K.check(L.lib().bonsai_lay_attn_decode(*calls[it[0] % copies].args, B, split, K.stream()), "attn_decode")
+        rep.add("attn_decode, capped, K and V", f"B={B} ctx={ctx} heads={nq}/{nkv}", time_us(ours, iters, profile), 4 * B * ctx * nkv * hd, 4.0 * B * ctx * nq * hd)
+    T, npages = 4096, 64
+    k, v = (torch.randn(npages, nkv, page, hd, device=dev).bfloat16() for _ in range(2))
+    bt, pos, slots = torch.arange(npages, **i32).view(1, -1), torch.arange(T, **i32), torch.zeros(T, **i32)
+    proj, out = torch.randn(T, ld, device=dev), torch.zeros(T, nq * hd, dtype=torch.bfloat16, device=dev)
+    entries = torch.tensor([0, T, 0, 0], **i32)
+    tiles = torch.tensor([[0, t] for t in range(0, T, 64 // (nq // nkv))], **i32)
+    for cap in (50.0, 0.0):
+        c = call(proj, pos, slots, bt, k, v, out, cap)
+        fn = lambda: K.check(L.lib().bonsai_lay_attn_prompt(*c.args, entries.data_ptr(), tiles.data_ptr(), len(tiles), K.stream()), "attn_prompt")
+        rep.add("attn_prompt, K and V", f"T={T} heads={nq}/{nkv} cap={cap}", time_us(fn, 10, profile), 4 * T * ld + 4 * T * nkv * hd + 2 * T * nq * hd,
+                4.0 * T * (T + 1) / 2 * nq * hd)
+    fn = lambda: K.check(L.lib().bonsai_lay_attn_append(*c.args, 0, T, 0, K.stream()), "attn_append")
+    rep.add("attn_append, K and V", f"T={T}", time_us(fn, iters, profile), 12 * T * nkv * hd)
+
+
+def bench_recurrence(rep: Report, width: int, iters: int, profile: bool) -> None:
+    """The linear recurrences; the like kernels are those of bench_mlstm."""
+    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, plan_segments
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    i32, lib = dict(dtype=torch.int32, device=dev), L.lib()
+    H = width // 128
+    kinds = {"lightning": dict(h=H, g=H, d=128, e=128, act=1), "retention": dict(h=max(1, width // 256), g=max(1, width // 256), d=256, e=256, rot=256),
+             "ssd": dict(h=width // 64, g=max(1, H // 4), d=128, e=64, act=1, taps=4)}
+    for name, c in kinds.items():
+        h, g, d, e, taps, rot = c["h"], c["g"], c["d"], c["e"], c.get("taps", 0), c.get("rot", 0)
+        inner, ch = h * e, h * e + 2 * g * d
+        v, k, q, gate, dt = 0, inner, inner + g * d, ch, ch + inner
+        ld, ldf = ch + inner + L.round_up(h, 4), lib.bonsai_lay_rec_features_width(h, g, d, e)
+        vec = torch.full((h,), 0.99, device=dev)
+        conv = (torch.randn(taps, ch, device=dev), torch.randn(ch, device=dev)) if taps else (None, None)
+        freq = torch.rand(rot // 2, dtype=torch.float64, device=dev) if rot else None
+        scratch = [torch.empty(MAX_SEGMENTS * n, device=dev) for n in (h * d * e, h)]
+
+        def call(T, rows, out, pos, slots):
+            S, ring = torch.zeros(rows, h, d, e, device=dev), (torch.zeros(rows, taps, ch, device=dev) if taps else None)
+            proj, feat = torch.randn(T, ld, device=dev), torch.zeros(T, ldf, dtype=torch.bfloat16, device=dev)
+            return L.MixerCall([proj, None if taps else vec, vec, vec, vec if taps else None, None, *conv, ring, freq, S, pos, slots, torch.arange(rows, **i32), out,
+                                feat, *scratch],
+                               [ld, q, k, v, gate, dt, 0, out.stride(0), ldf, h, g, d, e, c.get("act", 0), taps, ch if taps else 0, rot, int(name != "lightning")],
+                               [1e-6, 1.0, 1.0])
+        for B in (1, 8, 64):
+            copies = max(2, int(400e6 / (4 * B * h * d * e)) + 1)
+            done = name == "retention"
+            out = torch.zeros(B, inner, dtype=torch.bfloat16 if done else torch.float32, device=dev)
+            calls = [call(B, B, out, torch.full((B,), 5, **i32), torch.arange(B, **i32)) for _ in range(copies)]
+            it = [0]
+
+            def step():
+                it[0] += 1
+                K.check(lib.bonsai_lay_rec_step(*calls[it[0] % copies].args, None, B, 2 if done else 1, 0, 0, K.stream()), "rec_step")
+            rep.add("rec_step", f"{name} B={B} heads={h} {d}x{e}", time_us(step, iters, profile), 8.0 * B * h * d * e, 4.0 * B * h * d * e)
+            del calls
+        for nseq, T in ((1, 4096), (1, 512), (8, 512)):
+            rows = nseq * T
+            out = torch.zeros(rows, inner, device=dev)
+            cl = call(rows, nseq, out, torch.arange(T, **i32).repeat(nseq), torch.arange(nseq, **i32).repeat_interleave(T))
+            entries = torch.tensor([[s * T, T, s, 0] for s in range(nseq)], **i32)
+            size = plan_segments([T] * nseq, h * e // 64, torch.cuda.get_device_properties(dev).multi_processor_count) * CHUNK
+            segs = [(s * T + x, min(size, T - x), s, int(x + size >= T)) for s in range(nseq) for x in range(0, T, size)] if size else []
+            per = len(segs) // nseq
+            sl, pl = torch.tensor(segs or [[0] * 4], **i32), torch.tensor([(s, 0, s * per, per) for s in range(nseq)], **i32)
+            case = f"{name} {nseq} x {T} tokens heads={h}/{g} {d}x{e}"
+            fn = lambda: K.check(lib.bonsai_lay_rec_features(*cl.args, 0, rows, 0, K.stream()), "rec_features")
+            rep.add("rec_features", case, time_us(fn, 10, profile), 6.0 * rows * ch)
+            fn = lambda: K.check(lib.bonsai_lay_rec_chunk(*cl.args, entries.data_ptr(), nseq, sl.data_ptr(), len(segs), pl.data_ptr(), K.stream()), "rec_chunk")
+            rep.add("rec_chunk", f"{case} segments={len(segs)}", time_us(fn, 10, profile), rows * (2.0 * ch + 4.0 * inner), 4.0 * rows * h * d * e)
+            if nseq == 1 and T == 512:
+                continue
+            act, gates = torch.zeros(rows, inner, dtype=torch.bfloat16, device=dev), torch.randn(rows, ld, device=dev)
+            parts = {"lightning": 1, "retention": h, "ssd": g}[name]
+            fn = lambda: L.gated_norm(out, 0, gates, gate, None, 1e-6, rows, parts, inner // parts, act, "silu", name == "ssd")
+            rep.add("gated_norm", f"{name} T={rows} parts={parts}", time_us(fn, iters, profile), 10.0 * rows * inner)
+    for T in (1, 64, 4096):
+        x, y, w = torch.randn(T, width, device=dev), torch.randn(T, width, device=dev), torch.ones(width, device=dev)
+        x16 = torch.zeros(T, width, dtype=torch.bfloat16, device=dev)
+        rep.add("norm_add, next norm", f"T={T} width={width}", time_us(lambda: L.norm_add(x, y, w, 1e-6, T, x16, w), iters, profile), 14.0 * T * width)
 
 
 def bench_mlstm(rep: Report, width: int, iters: int, profile: bool) -> None:
@@ -281,12 +414,34 @@ def measure_generic(path: str, steps: int, warmup: int, prompt: int, batches) ->
     return res
 
 
+def run_kekevik(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64), log=sys.stdout) -> list[dict]:
+    """Kekevik beside Keripel of the same width with as many layers as bring it to the same parameter count."""
+    rows = []
+    for size in sizes:
+        width, repeats = SIZES[size]["width"], max(1, SIZES[size]["repeats"] // 2)
+        row = {"size": size, "width": width}
+        for name, make in (("kekevik", kekevik), ("keripel", keripel)):
+            with tempfile.TemporaryDirectory() as d:
+                if name == "keripel":
+                    count = lambda n: write_design(os.path.join(d, "m"), keripel(width, n))
+                    one, two = count(1), count(2)
+                    repeats = max(1, round((row["kekevik_params_M"] * 1e6 - one) / (two - one)) + 1)
+                cfg = make(width, repeats)
+                params = write_design(os.path.join(d, "m"), cfg)
+                row[f"{name}_layers"], row[f"{name}_params_M"] = len(cfg["layers"]), round(params / 1e6)
+                row[name] = measure_layered(os.path.join(d, "m"), steps, warmup, prompt, batches)
+            torch.cuda.empty_cache()
+        rows.append(row)
+        print(json.dumps(row), file=log, flush=True)
+    return rows
+
+
 def run_models(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64), log=sys.stdout) -> list[dict]:
     from oxibonsai_b200.cli import requantize_gguf
     from oxibonsai_b200.core import Qwen3Config, write_synthetic_gguf
     rows = []
     for size in sizes:
-        cfg = design(**SIZES[size])
+        cfg = keripel(**SIZES[size])
         width = cfg["width"]
         with tempfile.TemporaryDirectory() as d:
             params = write_design(os.path.join(d, "design"), cfg)
@@ -313,17 +468,19 @@ def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("case", choices=["kernels", "models"])
     ap.add_argument("--width", type=int, default=4096)
-    ap.add_argument("--only", default="linear,attention,mlstm")
+    ap.add_argument("--only", default="linear,attention,mlstm,capped,recurrence")
+    ap.add_argument("--design", choices=["keripel", "kekevik"], default="kekevik")
     ap.add_argument("--iters", type=int, default=40)
     ap.add_argument("--sizes", default="s,m,l")
     ap.add_argument("--profile", action="store_true", help="a few eager launches per case, for captures under a profiler")
     a = ap.parse_args()
     torch.cuda.set_device(0)
     if a.case == "models":
-        run_models(a.sizes.split(","))
+        (run_kekevik if a.design == "kekevik" else run_models)(a.sizes.split(","))
         return
     rep = Report()
-    for name, fn in (("linear", bench_linear), ("attention", bench_attention), ("mlstm", bench_mlstm)):
+    for name, fn in (("linear", bench_linear), ("attention", bench_attention), ("mlstm", bench_mlstm), ("capped", bench_capped_attention),
+                     ("recurrence", bench_recurrence)):
         if name in a.only.split(","):
             fn(rep, a.width, a.iters, a.profile)
 

@@ -29,6 +29,47 @@ def mixed_config():
                    mlstm(heads=1, dim=100, vdim=136, cap=4.0, ff=90)])
 
 
+# ---- Kekevik ----------------------------------------------------------------------------------------------------------------------
+def relu2(ff):
+    return None if ff is None else {"kind": "dense", "ff": ff}
+
+
+def decays(heads):
+    """From a few tokens to a few hundred."""
+    return [1.0 - 0.4 * 0.3 ** (4.5 * h / max(1, heads - 1)) for h in range(heads)]
+
+
+def retention(heads=3, dim=24, vdim=40, base=5000.0, dims=None, decay=None, ff=None):
+    return {"type": "retention", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay or decays(heads),
+                                           "rot": {"base": base, "dims": dim if dims is None else dims}}, "mlp": relu2(ff)}
+
+
+def lightning(heads=5, dim=20, vdim=36, decay=None, ff=None):
+    return {"type": "lightning", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay or decays(heads)}, "mlp": relu2(ff)}
+
+
+def capped(heads=6, kv_heads=2, dim=40, vdim=24, scale=0.3, cap=6.0, coef=0.7, every=19):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "softcap": cap, "q_temp": {"coef": coef, "every": every}}
+
+
+def ssd(heads=6, vdim=20, state=28, groups=2, parts=3, conv=4):
+    return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "norm_groups": parts, "conv": conv}
+
+
+def parallel(left=None, right=None, scales=(0.7, 1.3), ff=None):
+    return {"type": "parallel", "mixer": {"left": left or capped(), "right": right or ssd(), "left_scale": scales[0], "right_scale": scales[1]}, "mlp": relu2(ff)}
+
+
+def kekevik(layers, width=152, vocab=331, eps=1e-5, scale=3.5):
+    return {"architecture": "Kekevik", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "embedding": {"scale": scale}}
+
+
+# every branch in one model: the three mixers with and without a feed-forward, shared and own queries and keys, odd sizes
+def kekevik_mixed():
+    return kekevik([parallel(ff=200), retention(), lightning(ff=90), parallel(capped(4, 4, 32, 72, 0.2, 20.0, -0.1, 7), ssd(4, 33, 70, 1, 2, 3)),
+                    retention(2, 50, 66, 100.0, 30, ff=70), lightning(1, 70, 130)])
+
+
 def write(path, cfg, weights):
     from oxibonsai_b200.convert import write_safetensors
     os.makedirs(path, exist_ok=True)

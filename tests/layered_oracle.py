@@ -249,24 +249,48 @@ def forward(cfg, w, tokens, keep_layers=False):
 
 
 # ---- seeded small models -----------------------------------------------------------------------------------------------------
+def keripel_mixer_shapes(layer, p, W):
+    m = layer["mixer"]
+    H, d, e = m["heads"], m["dim"], m["vdim"]
+    s = {p + "q": (H * d, W), p + "o": (W, H * e)}
+    if layer["type"] == "attention":
+        s.update({p + "k": (m["kv_heads"] * d, W), p + "q.norm": (d,), p + "k.norm": (d,), p + "g": (H, W)})
+    else:
+        s.update({p + "k": (H * d, W), p + "v": (H * e, W), p + "g": (H * e, W), p + "norm": (H * e,),
+                  p + "i": (H, W), p + "i.b": (H,), p + "f": (H, W), p + "f.b": (H,)})
+    return s
+
+
+def kekevik_mixer_shapes(layer, p, W):
+    m = layer["mixer"]
+    if layer["type"] == "parallel":
+        a, b = m["left"], m["right"]
+        G, inner = a["kv_heads"], b["heads"] * b["vdim"]
+        C = inner + 2 * b["groups"] * b["state"]
+        l, r = p + "left.", p + "right."
+        return {l + "q": (a["heads"] * a["dim"], W), l + "k": (G * a["dim"], W), l + "v": (G * a["vdim"], W), l + "o": (W, a["heads"] * a["vdim"]),
+                r + "in": (inner + C + b["heads"], W), r + "conv": (C, b["conv"]), r + "conv.b": (C,), r + "dt_bias": (b["heads"],),
+                r + "A_log": (b["heads"],), r + "D": (b["heads"],), r + "norm": (inner,), r + "o": (W, inner)}
+    H, d, e = m["heads"], m["dim"], m["vdim"]
+    s = {p + "q": (H * d, W), p + "k": (H * d, W), p + "v": (H * e, W), p + "g": (H * e, W), p + "o": (W, H * e)}
+    if layer["type"] == "lightning":
+        s[p + "norm"] = (H * e,)
+    return s
+
+
 def tensor_shapes(cfg):
     """Name -> shape of every tensor of a model."""
-    W = cfg["width"]
+    W, keripel = cfg["width"], cfg["architecture"] == "Keripel"
     s = {"embed": (cfg["vocab"], W), "final.norm": (W,)}
     for l, layer in enumerate(cfg["layers"]):
-        p, m = f"l{l}.", layer["mixer"]
-        H, d, e = m["heads"], m["dim"], m["vdim"]
-        s[p + "norm1"] = (W,)
-        s[p + "mix.q"] = (H * d, W)
-        s[p + "mix.o"] = (W, H * e)
-        if layer["type"] == "attention":
-            s.update({p + "mix.k": (m["kv_heads"] * d, W), p + "mix.q.norm": (d,), p + "mix.k.norm": (d,), p + "mix.g": (H, W)})
-        else:
-            s.update({p + "mix.k": (H * d, W), p + "mix.v": (H * e, W), p + "mix.g": (H * e, W), p + "mix.norm": (H * e,),
-                      p + "mix.i": (H, W), p + "mix.i.b": (H,), p + "mix.f": (H, W), p + "mix.f.b": (H,)})
+        p, tail = f"l{l}.", [""] if keripel else ["", "b"]
+        s.update({p + "norm1" + t: (W,) for t in tail})
+        s.update((keripel_mixer_shapes if keripel else kekevik_mixer_shapes)(layer, p + "mix.", W))
         if layer["mlp"] is not None:
             F = layer["mlp"]["ff"]
-            s.update({p + "norm2": (W,), p + "mlp.gate": (F, W), p + "mlp.up": (F, W), p + "mlp.down": (W, F)})
+            s.update({p + "norm2" + t: (W,) for t in tail})
+            s.update({p + "mlp." + n: (F, W) for n in (["gate", "up"] if keripel else ["up"])})
+            s[p + "mlp.down"] = (W, F)
     return s
 
 
@@ -284,6 +308,14 @@ def random_weights(cfg, seed=0, scale=1.0):
             t = 0.5 * t - 1.0
         elif name.endswith(".f.b"):
             t = 2.0 + 1.5 * t                      # from strong forgetting to almost none
+        elif name.endswith("dt_bias"):
+            t = t - 1.0
+        elif name.endswith("A_log"):
+            t = 1.5 * t - 2.0                      # from forgetting in a few tokens to hardly at all
+        elif name.endswith(".D"):
+            t = 1.0 + 0.3 * t
+        elif name.endswith("conv.b"):
+            t = 0.2 * t
         elif name.endswith((".i", ".f")):
             t = t * 0.5 * scale * shape[-1] ** -0.5
         else:

@@ -10,7 +10,7 @@ import layered_oracle as O
 import numpy as np
 import pytest
 import torch
-from layered_gpu import check, engine, feed, poison
+from layered_gpu import check, engine, feed, poison, run_unequal_requests
 
 pytestmark = pytest.mark.gpu
 
@@ -74,32 +74,7 @@ def test_batches_match_single_requests(mixed, mixed_engine):
     """Unequal requests share steps: portions beside decoded tokens, left out now and then, ending at different times; their
     pages and slots go to new requests, over a pool that starts full of NaN."""
     kv, eng = mixed_engine
-    poison(eng)
-    rng = np.random.default_rng(7)
-    reqs = [mixed.tokens(n, seed=20 + n) for n in (3, 130, 1, 77, 201, 64, 40, 65)]
-    want = [mixed.logits(t) for t in reqs]
-    queue, live, free, got = list(range(len(reqs))), {}, [2, 0, 3, 1], {i: [] for i in range(len(reqs))}
-    while queue or live:
-        while queue and free and len(live) < 4:
-            live[queue.pop(0)] = [free.pop(0), 0]
-        chosen = [i for i in live if rng.random() < 0.8] or list(live)
-        entries, wants, lens = [], [], []
-        for i in chosen:
-            slot, at = live[i]
-            n = min(int(rng.choice([1, 1, 2, 3, 17, 60])), len(reqs[i]) - at)
-            eng.reserve(slot, at + n)
-            entries.append((slot, reqs[i][at:at + n], at))
-            wants.append(list(range(n)))
-            lens.append(n)
-        out = eng.feed(entries, wants).clone()
-        for i, part in zip(chosen, out.split(lens)):
-            got[i].append(part)
-            live[i][1] += len(part)
-            if live[i][1] == len(reqs[i]):
-                eng.close_sequence(live[i][0])
-                free.append(live.pop(i)[0])
-    for i in got:
-        check(torch.cat(got[i]), want[i], kv, what=f"request {i}")
+    run_unequal_requests(mixed, eng, kv)
 
 
 def test_wanted_places(mixed, mixed_engine):
