@@ -236,7 +236,7 @@ def bench_capped_attention(rep: Report, width: int, iters: int, profile: bool) -
 
 def bench_recurrence(rep: Report, width: int, iters: int, profile: bool) -> None:
     """The linear recurrences; the like kernels are those of bench_mlstm."""
-    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, plan_segments
+    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, RECURRENCE_COST, WIDE_RECURRENCE_COST, SegmentPlan, plan_segments
     from oxibonsai_b200.ops import cuda_ops as K
     from oxibonsai_b200.ops import layered_ops as L
     dev = torch.device("cuda")
@@ -278,7 +278,8 @@ def bench_recurrence(rep: Report, width: int, iters: int, profile: bool) -> None
             out = torch.zeros(rows, inner, device=dev)
             cl = call(rows, nseq, out, torch.arange(T, **i32).repeat(nseq), torch.arange(nseq, **i32).repeat_interleave(T))
             entries = torch.tensor([[s * T, T, s, 0] for s in range(nseq)], **i32)
-            size = plan_segments([T] * nseq, h * e // 64, torch.cuda.get_device_properties(dev).multi_processor_count) * CHUNK
+            plan = SegmentPlan(h * e // 64, RECURRENCE_COST if d <= 128 else WIDE_RECURRENCE_COST)
+            size = plan_segments([T] * nseq, plan, torch.cuda.get_device_properties(dev).multi_processor_count) * CHUNK
             segs = [(s * T + x, min(size, T - x), s, int(x + size >= T)) for s in range(nseq) for x in range(0, T, size)] if size else []
             per = len(segs) // nseq
             sl, pl = torch.tensor(segs or [[0] * 4], **i32), torch.tensor([(s, 0, s * per, per) for s in range(nseq)], **i32)
@@ -309,7 +310,7 @@ def bench_mlstm(rep: Report, width: int, iters: int, profile: bool) -> None:
     i32 = dict(dtype=torch.int32, device=dev)
     bias, norm = torch.zeros(H + 4, device=dev), torch.ones(H * e, device=dev)
 
-    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, plan_segments
+    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, MLSTM_COST, SegmentPlan, plan_segments
     scratch = [torch.empty(MAX_SEGMENTS * n, device=dev) for n in (H * d * e, H * d * e // 64, H * e // 64, H * e // 32)]
 
     def call(T, rows, out, states, pos):
@@ -334,7 +335,7 @@ def bench_mlstm(rep: Report, width: int, iters: int, profile: bool) -> None:
         out = torch.zeros(rows, H * e, device=dev)
         c = call(rows, nseq, out, state(nseq), torch.zeros(nseq, **i32))
         entries = torch.tensor([[s * T, T, s, 0] for s in range(nseq)], **i32)
-        size = plan_segments([T] * nseq, H * e // 64, torch.cuda.get_device_properties(dev).multi_processor_count) * CHUNK
+        size = plan_segments([T] * nseq, SegmentPlan(H * e // 64, MLSTM_COST), torch.cuda.get_device_properties(dev).multi_processor_count) * CHUNK
         segs = [(s * T + x, min(size, T - x), s, int(x + size >= T)) for s in range(nseq) for x in range(0, T, size)] if size else []
         per = len(segs) // nseq
         sl = torch.tensor(segs or [[0] * 4], **i32)

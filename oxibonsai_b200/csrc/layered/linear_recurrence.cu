@@ -69,12 +69,22 @@ __device__ __forceinline__ float2 rotation(int pos, double freq) {
 }
 
 // Column `col` of a single token's row p, convolved with the ring's inputs where the design has a convolution, and activated.
-__device__ __forceinline__ float single_feature(const LinRec& a, const float* p, const float* ring, int pos, int col) {
+// here: pos % taps.
+__device__ __forceinline__ float single_feature(const LinRec& a, const float* p, const float* ring, int pos, int here, int col) {
   float v = p[col];
   if (a.taps > 0) {
     const int c = col - a.conv_col;
+    float x[3], w[3];                                // the first three inputs back, loaded at once
+#pragma unroll
+    for (int j = 1; j <= 3; ++j) {
+      const bool ok = j < a.taps && j <= pos;
+      x[j - 1] = ok ? ring[(here >= j ? here - j : here - j + a.taps) * a.conv_n + c] : 0.0f;
+      w[j - 1] = ok ? a.conv_w[j * a.conv_n + c] : 0.0f;
+    }
     v = fmaf(v, a.conv_w[c], a.conv_b[c]);
-    for (int j = 1; j < a.taps && j <= pos; ++j) v = fmaf(a.conv_w[j * a.conv_n + c], ring[((pos - j) % a.taps) * a.conv_n + c], v);
+#pragma unroll
+    for (int j = 0; j < 3; ++j) v = fmaf(w[j], x[j], v);
+    for (int j = 4; j < a.taps && j <= pos; ++j) v = fmaf(a.conv_w[j * a.conv_n + c], ring[(here >= j ? here - j : here - j + a.taps) * a.conv_n + c], v);
   }
   return a.act ? silu(v) : v;
 }
@@ -123,30 +133,31 @@ __global__ void __launch_bounds__(16 * DG) step_kernel(LinRec a, const int4* ent
     pdl_trigger();
   }
   const float skip = a.skip == nullptr ? 0.0f : a.skip[h];
+  const int here = ONE && a.taps > 0 ? pos0 % a.taps : 0;
   for (int tt = 0; tt < count; ++tt) {
     const float* p = a.proj + (size_t)(t0 + tt) * a.ld;
     if (ONE) {
       const int qc = a.q_col + grp * a.dim, kc = a.k_col + grp * a.dim, half = a.rot_dims >> 1;
       for (int i = tid; i < half; i += NTH) {
         const float2 cs = rotation(pos0, a.freq[i]);
-        const float qu = single_feature(a, p, ring, pos0, qc + i), qv = single_feature(a, p, ring, pos0, qc + half + i);
-        const float ku = single_feature(a, p, ring, pos0, kc + i), kv = single_feature(a, p, ring, pos0, kc + half + i);
+        const float qu = single_feature(a, p, ring, pos0, here, qc + i), qv = single_feature(a, p, ring, pos0, here, qc + half + i);
+        const float ku = single_feature(a, p, ring, pos0, here, kc + i), kv = single_feature(a, p, ring, pos0, here, kc + half + i);
         sq[i] = qu * cs.x - qv * cs.y;
         sq[half + i] = qv * cs.x + qu * cs.y;
         sk[i] = (ku * cs.x - kv * cs.y) * a.key_scale;
         sk[half + i] = (kv * cs.x + ku * cs.y) * a.key_scale;
       }
       for (int d = a.rot_dims + tid; d < DIM; d += NTH) {
-        sq[d] = d < a.dim ? single_feature(a, p, ring, pos0, qc + d) : 0.0f;
-        sk[d] = d < a.dim ? single_feature(a, p, ring, pos0, kc + d) * a.key_scale : 0.0f;
+        sq[d] = d < a.dim ? single_feature(a, p, ring, pos0, here, qc + d) : 0.0f;
+        sk[d] = d < a.dim ? single_feature(a, p, ring, pos0, here, kc + d) * a.key_scale : 0.0f;
       }
       const int vt = NTH - 1 - tid;                  // the last threads: the first ones have a rotation to do
       if (vt < kVT) {
         const int c = tile * kVT + vt;
-        sv[vt] = c < a.vdim ? single_feature(a, p, ring, pos0, a.v_col + h * a.vdim + c) : 0.0f;
+        sv[vt] = c < a.vdim ? single_feature(a, p, ring, pos0, here, a.v_col + h * a.vdim + c) : 0.0f;
       }
       if (a.taps > 0) {                              // this token's inputs join the ring, every channel from one CTA
-        float* dst = ring + (pos0 % a.taps) * a.conv_n;
+        float* dst = ring + here * a.conv_n;
         for (int i = tid; i < min(kVT, a.vdim - tile * kVT); i += NTH) {
           const int cc = a.v_col + h * a.vdim + tile * kVT + i;
           dst[cc - a.conv_col] = p[cc];
@@ -228,15 +239,16 @@ __global__ void __launch_bounds__(16 * DG) step_kernel(LinRec a, const int4* ent
 // Rows first .. first + count - 1, kFR per CTA; a thread has VEC feature columns.  Rows of one portion are neighbours; an input
 // from before the portion comes from the ring.
 constexpr int kFR = 8;
+enum FeatureKind { kPlain, kRotary, kConv4, kConv };     // kConv4: up to four taps, the inputs back in registers
 
-template <int VEC, typename X>
+template <int VEC, int KIND, typename X>
 __global__ void __launch_bounds__(128) features_kernel(LinRec a, int first, int count) {
   extern __shared__ float2 cs[];                     // [kFR][rot_dims / 2]
   pdl_wait();
   pdl_trigger();
   const int r0 = first + blockIdx.y * kFR, rows = min(kFR, first + count - r0), half = a.rot_dims >> 1;
   const int qk = a.groups * a.dp, f0 = (blockIdx.x * 128 + threadIdx.x) * VEC;
-  if (half > 0) {
+  if (KIND == kRotary) {
     if (blockIdx.x * 128 * VEC < 2 * qk)
       for (int i = threadIdx.x; i < rows * half; i += 128) cs[i] = rotation(a.pos[r0 + i / half], a.freq[i % half]);
     __syncthreads();
@@ -255,64 +267,109 @@ __global__ void __launch_bounds__(128) features_kernel(LinRec a, int first, int 
     size = a.vdim;
     col = a.v_col + h * a.vdim + d;
   }
-  const bool in = d < size, rot = what < 2 && d < a.rot_dims;
-  const int partner = d < half ? half : -half;
-  auto load = [&](const float* p, float* v) {
+  const bool in = d < size, rot = KIND == kRotary && what < 2 && d < a.rot_dims;
+  auto load = [&](const float* p, float* v, bool ok) {
     if constexpr (VEC == 4) {
-      const float4 q = *reinterpret_cast<const float4*>(p);
+      const float4 q = ok ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
       v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
     } else {
-      v[0] = *p;
+      v[0] = ok ? *p : 0.0f;
     }
   };
-  for (int r = 0; r < rows; ++r) {
+  float v[kFR][VEC], u[KIND == kRotary ? kFR : 1][VEC];
+  const float* src = a.proj + (size_t)r0 * a.ld + col;
+  const int partner = d < half ? half : -half;
+#pragma unroll
+  for (int r = 0; r < kFR; ++r) {
+    load(src + (size_t)r * a.ld, v[r], in && r < rows);
+    if (KIND == kRotary) load(src + (size_t)r * a.ld + partner, u[KIND == kRotary ? r : 0], rot && r < rows);
+  }
+  const int c = col - a.conv_col;
+  bool same = false;                                 // all of these rows and the three before them belong to one portion
+  float w[KIND == kConv4 ? 4 : 1][VEC], back[KIND == kConv4 ? 3 : 1][VEC], bias[VEC];   // back[j]: the input j + 1 rows back
+  if (KIND == kConv4) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) load(a.conv_w + (size_t)j * a.conv_n + c, w[KIND == kConv4 ? j : 0], in && j < a.taps);
+    if (r0 - 3 >= first) {
+#pragma unroll
+      for (int j = 1; j <= 3; ++j) load(src - (size_t)j * a.ld, back[KIND == kConv4 ? j - 1 : 0], in);
+      same = a.slots[r0 - 3] == a.slots[r0 + rows - 1];
+    }
+  }
+  if (KIND >= kConv4) load(a.conv_b + c, bias, in);
+  // the input j rows before row t, a zero before the sequence's start
+  auto earlier = [&](int t, int slot, int pos, int j, float* x) {
+    bool here = t - j >= first;                      // the rows back to t - j belong to the same portion
+    for (int i = 1; i <= j && here; ++i) here = a.slots[t - i] == slot;
+    const float* ring = a.ring + ((size_t)a.state_rows[slot] * a.taps + (pos - j + a.taps * j) % a.taps) * a.conv_n + c;
+    load(here ? a.proj + (size_t)(t - j) * a.ld + col : ring, x, in && j < a.taps && j <= pos);
+  };
+  int last = -1;                                     // slot of the row before
+#pragma unroll
+  for (int r = 0; r < kFR; ++r) {
+    if (r >= rows) break;
     const int t = r0 + r;
-    float v[VEC] = {};
-    if (in) {
-      load(a.proj + (size_t)t * a.ld + col, v);
-      if (a.taps > 0) {
-        const int c = col - a.conv_col, slot = a.slots[t], pos = a.pos[t];
-        const float* ring = a.ring + (size_t)a.state_rows[slot] * a.taps * a.conv_n + c;
-        float w[VEC], acc[VEC], x[VEC];
-        load(a.conv_w + c, w);
-        load(a.conv_b + c, acc);
+    float y[VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) acc[e] = fmaf(v[e], w[e], acc[e]);
-        bool here = true;                            // the rows back to t - j belong to the same portion
-        for (int j = 1; j < a.taps && j <= pos; ++j) {
-          here = here && t - j >= first && a.slots[t - j] == slot;
-          load(here ? a.proj + (size_t)(t - j) * a.ld + col : ring + (size_t)((pos - j) % a.taps) * a.conv_n, x);
-          load(a.conv_w + (size_t)j * a.conv_n + c, w);
+    for (int e = 0; e < VEC; ++e) y[e] = v[r][e];
+    if constexpr (KIND == kConv4) {
+      if (!same) {
+        const int slot = a.slots[t];
+        if (slot != last) {
+          const int pos = a.pos[t];
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) acc[e] = fmaf(x[e], w[e], acc[e]);
+          for (int j = 1; j <= 3; ++j) earlier(t, slot, pos, j, back[j - 1]);
+          last = slot;
         }
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) v[e] = acc[e];
       }
 #pragma unroll
-      for (int e = 0; e < VEC; ++e)
-        if (a.act) v[e] = silu(v[e]);
+      for (int e = 0; e < VEC; ++e) {
+        y[e] = fmaf(v[r][e], w[0][e], bias[e]);
+        y[e] = fmaf(back[0][e], w[1][e], y[e]);
+        y[e] = fmaf(back[1][e], w[2][e], y[e]);
+        y[e] = fmaf(back[2][e], w[3][e], y[e]);
+        back[2][e] = back[1][e];
+        back[1][e] = back[0][e];
+        back[0][e] = v[r][e];
+      }
+    }
+    if constexpr (KIND == kConv) {
+      const int slot = a.slots[t], pos = a.pos[t];
+      float x[VEC], k[VEC];
+      load(a.conv_w + c, k, in);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = fmaf(v[r][e], k[e], bias[e]);
+      for (int j = 1; j < a.taps && j <= pos; ++j) {
+        earlier(t, slot, pos, j, x);
+        load(a.conv_w + (size_t)j * a.conv_n + c, k, in);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = fmaf(x[e], k[e], y[e]);
+      }
+    }
+    if (a.act) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = silu(y[e]);
+    }
+    if constexpr (KIND == kRotary) {
       if (rot) {
-        float u[VEC];
-        load(a.proj + (size_t)t * a.ld + col + partner, u);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-          if (a.act) u[e] = silu(u[e]);
+          const float z = a.act ? silu(u[r][e]) : u[r][e];
           const float2 k = cs[r * half + (d < half ? d : d - half) + e];
-          v[e] = d < half ? v[e] * k.x - u[e] * k.y : v[e] * k.x + u[e] * k.y;
+          y[e] = d < half ? y[e] * k.x - z * k.y : y[e] * k.x + z * k.y;
         }
       }
-      if (what == 1) {
+    }
+    if (what == 1) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) v[e] *= a.key_scale;
-      }
+      for (int e = 0; e < VEC; ++e) y[e] *= a.key_scale;
     }
     X* dst = static_cast<X*>(a.feat) + (size_t)t * a.ldf + f0;
     if constexpr (VEC == 4 && sizeof(X) == 2) {
-      *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+      *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]));
     } else {
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) store_act(dst + e, v[e]);
+      for (int e = 0; e < VEC; ++e) store_act(dst + e, in ? y[e] : 0.0f);
     }
   }
 }
@@ -750,10 +807,14 @@ int bonsai_lay_rec_features(const void* const* ptrs, const int* ints, const floa
   const int quads = (2 * a.groups * a.dp + a.heads * a.ep) / (vec ? 4 : 1);
   const dim3 grid((quads + 127) / 128, (count + kFR - 1) / kFR);
   const size_t smem = (size_t)kFR * (a.rot_dims / 2) * sizeof(float2);
-  if (f32) return vec ? launch(features_kernel<4, float>, grid, 128, smem, stream, 1, 0, a, first, count)
-                      : launch(features_kernel<1, float>, grid, 128, smem, stream, 1, 0, a, first, count);
-  return vec ? launch(features_kernel<4, bf16>, grid, 128, smem, stream, 1, 0, a, first, count)
-             : launch(features_kernel<1, bf16>, grid, 128, smem, stream, 1, 0, a, first, count);
+#define BONSAI_FEATURES(KIND)                                                                                     \
+  (f32 ? (vec ? launch(features_kernel<4, KIND, float>, grid, 128, smem, stream, 1, 0, a, first, count)           \
+              : launch(features_kernel<1, KIND, float>, grid, 128, smem, stream, 1, 0, a, first, count))          \
+       : (vec ? launch(features_kernel<4, KIND, bf16>, grid, 128, smem, stream, 1, 0, a, first, count)            \
+              : launch(features_kernel<1, KIND, bf16>, grid, 128, smem, stream, 1, 0, a, first, count)))
+  if (a.taps > 0) return a.taps <= 4 ? BONSAI_FEATURES(kConv4) : BONSAI_FEATURES(kConv);
+  return a.rot_dims > 0 ? BONSAI_FEATURES(kRotary) : BONSAI_FEATURES(kPlain);
+#undef BONSAI_FEATURES
 }
 
 // The portions' last inputs join the convolution's ring; after the features.

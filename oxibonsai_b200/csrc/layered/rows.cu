@@ -6,77 +6,98 @@
 namespace bonsai {
 namespace lay {
 
-constexpr int kKeep = 4;   // float4 chunks of a row that a thread keeps in registers
-
 __device__ __forceinline__ void store_act4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
 __device__ __forceinline__ void store_act4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 
+__device__ __forceinline__ float sum_sq(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// KEEP in the kernels below: float4 of a row that a thread keeps in registers (0: rows of any width, read again instead).
+
 // x[t] = table[tokens[t]] * scale; h[t] = x[t], or its norm when `next` (the norm's weight) is given.  h may be null.
-template <typename H>
-__global__ void embed_kernel(const bf16* __restrict__ table, int ld_table, const int* tokens, float scale, int width, float* x, H* h, int ldh,
-                             const float* __restrict__ next, float eps) {
+template <int KEEP, typename H>
+__global__ void __launch_bounds__(1024) embed_kernel(const bf16* __restrict__ table, int ld_table, const int* tokens, float scale, int width, float* x,
+                                                     H* h, int ldh, const float* __restrict__ next, float eps) {
   __shared__ float s32[32];
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
   const bf16* src = table + (size_t)tokens[t] * ld_table;
-  float inv = 1.0f;
-  if (next != nullptr) {
+  float* xr = x + (size_t)t * width;
+  H* hr = h == nullptr ? nullptr : h + (size_t)t * ldh;
+  if constexpr (KEEP > 0) {
+    const int nch = width >> 2;
+    float4 v[KEEP];
     float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      const uint2 q = c < nch ? reinterpret_cast<const uint2*>(src)[c] : make_uint2(0u, 0u);
+      const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+      v[i] = make_float4(lo.x * scale, lo.y * scale, hi.x * scale, hi.y * scale);
+      if (c < nch) reinterpret_cast<float4*>(xr)[c] = v[i];
+      ss += sum_sq(v[i]);
+    }
+    if (hr == nullptr) return;
+    const float inv = next == nullptr ? 1.0f : 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c >= nch) continue;
+      if (next != nullptr) {
+        const float4 g = reinterpret_cast<const float4*>(next)[c];
+        v[i] = make_float4(v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w);
+      }
+      store_act4(hr + 4 * c, v[i]);
+    }
+  } else {
+    float inv = 1.0f;
+    if (next != nullptr) {
+      float ss = 0.0f;
+      for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const float v = __bfloat162float(src[c]) * scale;
+        ss += v * v;
+      }
+      inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+    }
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
       const float v = __bfloat162float(src[c]) * scale;
-      ss += v * v;
+      xr[c] = v;
+      if (hr != nullptr) store_act(hr + c, next != nullptr ? v * inv * next[c] : v);
     }
-    inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
-  }
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float v = __bfloat162float(src[c]) * scale;
-    x[(size_t)t * width + c] = v;
-    if (h != nullptr) store_act(h + (size_t)t * ldh + c, next != nullptr ? v * inv * next[c] : v);
   }
 }
 
 // x += y / sqrt(mean(y^2) + eps) * w; h = x, or its norm with weight `next`
-template <typename H>
-__global__ void norm_add_kernel(float* x, const float* y, int ldy, const float* __restrict__ w, float eps, int width, H* h, int ldh,
-                                const float* __restrict__ next) {
+template <int KEEP, typename H>
+__global__ void __launch_bounds__(1024) norm_add_kernel(float* x, const float* y, int ldy, const float* __restrict__ w, float eps, int width, H* h, int ldh,
+                                                        const float* __restrict__ next) {
   __shared__ float s32[32];
-  // weights depend on no earlier kernel
-  const bool vec = (width & 3) == 0 && width <= 4 * kKeep * (int)blockDim.x;
-  const int nch = width >> 2;
-  float4 wv[kKeep];
-  if (vec) {
-#pragma unroll
-    for (int i = 0; i < kKeep; ++i) {
-      const int c = threadIdx.x + i * blockDim.x;
-      if (c < nch) wv[i] = reinterpret_cast<const float4*>(w)[c];
-    }
-  }
   pdl_wait();
   pdl_trigger();
   float* xr = x + (size_t)blockIdx.x * width;
   const float* yr = y + (size_t)blockIdx.x * ldy;
   H* hr = h == nullptr ? nullptr : h + (size_t)blockIdx.x * ldh;
-  float ss = 0.0f;
-  if (vec) {
-    float4 v[kKeep], r[kKeep];
+  float ss = 0.0f, sx = 0.0f;
+  if constexpr (KEEP > 0) {
+    const int nch = width >> 2;
+    float4 v[KEEP], r[KEEP];
 #pragma unroll
-    for (int i = 0; i < kKeep; ++i) {
+    for (int i = 0; i < KEEP; ++i) {
       const int c = threadIdx.x + i * blockDim.x;
       v[i] = c < nch ? reinterpret_cast<const float4*>(yr)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
       r[i] = c < nch ? reinterpret_cast<const float4*>(xr)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
       ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
-    float sx = 0.0f;
 #pragma unroll
-    for (int i = 0; i < kKeep; ++i) {
+    for (int i = 0; i < KEEP; ++i) {
       const int c = threadIdx.x + i * blockDim.x;
       if (c < nch) {
-        r[i].x += v[i].x * inv * wv[i].x;
-        r[i].y += v[i].y * inv * wv[i].y;
-        r[i].z += v[i].z * inv * wv[i].z;
-        r[i].w += v[i].w * inv * wv[i].w;
+        const float4 g = reinterpret_cast<const float4*>(w)[c];
+        r[i].x += v[i].x * inv * g.x;
+        r[i].y += v[i].y * inv * g.y;
+        r[i].z += v[i].z * inv * g.z;
+        r[i].w += v[i].w * inv * g.w;
         reinterpret_cast<float4*>(xr)[c] = r[i];
         sx += r[i].x * r[i].x + r[i].y * r[i].y + r[i].z * r[i].z + r[i].w * r[i].w;
       }
@@ -84,7 +105,7 @@ __global__ void norm_add_kernel(float* x, const float* y, int ldy, const float* 
     if (hr == nullptr) return;
     const float nx = next == nullptr ? 1.0f : 1.0f / sqrtf(block_sum(sx, s32) / (float)width + eps);
 #pragma unroll
-    for (int i = 0; i < kKeep; ++i) {
+    for (int i = 0; i < KEEP; ++i) {
       const int c = threadIdx.x + i * blockDim.x;
       if (c >= nch) continue;
       if (next != nullptr) {
@@ -93,45 +114,63 @@ __global__ void norm_add_kernel(float* x, const float* y, int ldy, const float* 
       }
       store_act4(hr + 4 * c, r[i]);
     }
-    return;
+  } else {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) ss += yr[c] * yr[c];
+    const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      const float v = xr[c] + yr[c] * inv * w[c];
+      xr[c] = v;
+      sx += v * v;
+    }
+    if (hr == nullptr) return;
+    const float nx = next == nullptr ? 1.0f : 1.0f / sqrtf(block_sum(sx, s32) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) store_act(hr + c, next == nullptr ? xr[c] : xr[c] * nx * next[c]);
   }
-  for (int c = threadIdx.x; c < width; c += blockDim.x) ss += yr[c] * yr[c];
-  const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
-  float sx = 0.0f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float v = xr[c] + yr[c] * inv * w[c];
-    xr[c] = v;
-    sx += v * v;
-  }
-  if (hr == nullptr) return;
-  const float nx = next == nullptr ? 1.0f : 1.0f / sqrtf(block_sum(sx, s32) / (float)width + eps);
-  for (int c = threadIdx.x; c < width; c += blockDim.x) store_act(hr + c, next == nullptr ? xr[c] : xr[c] * nx * next[c]);
 }
 
 // out[i] = norm(x[rows[i]]) * w; rows == null: row i
-template <typename OUT>
-__global__ void norm_rows_kernel(const float* x, const int* rows, const float* __restrict__ w, float eps, int width,
-                                 OUT* out, int ld) {
+template <int KEEP, typename OUT>
+__global__ void __launch_bounds__(1024) norm_rows_kernel(const float* x, const int* rows, const float* __restrict__ w, float eps, int width, OUT* out, int ld) {
   __shared__ float s32[32];
   pdl_wait();
   pdl_trigger();
   const int row = rows == nullptr ? blockIdx.x : rows[blockIdx.x];
   const float* xr = x + (size_t)row * width;
+  OUT* dst = out + (size_t)blockIdx.x * ld;
   float ss = 0.0f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) ss += xr[c] * xr[c];
-  const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
-  for (int c = threadIdx.x; c < width; c += blockDim.x) store_act(out + (size_t)blockIdx.x * ld + c, xr[c] * inv * w[c]);
+  if constexpr (KEEP > 0) {
+    const int nch = width >> 2;
+    float4 v[KEEP];
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      v[i] = c < nch ? reinterpret_cast<const float4*>(xr)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += sum_sq(v[i]);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c >= nch) continue;
+      const float4 g = reinterpret_cast<const float4*>(w)[c];
+      store_act4(dst + 4 * c, make_float4(v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w));
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) ss += xr[c] * xr[c];
+    const float inv = 1.0f / sqrtf(block_sum(ss, s32) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) store_act(dst + c, xr[c] * inv * w[c]);
+  }
 }
 
 // Norm of a recurrent mixer's output in parts of `width` columns (a head, a group of heads, or all of them), with a gate before
 // or after it:
 //   after:  out = o / rms(o) [* w] * act(gate) * scale          before:  u = o * act(gate), out = u / rms(u) [* w] * scale
-// act: sigmoid, or silu.  GT threads per (row, part).
+// act: sigmoid, or silu.  GT threads per (row, part); KEEP: float4 a thread keeps in registers (0: any width and alignment).
 struct GatedNorm {
   const float* o;
   const float* gate;
   const float* w;           // null: no weight
-  int ldo, ldg, T, parts, width, ld, vec, silu, before;
+  int ldo, ldg, T, parts, width, ld, silu, before;
   float eps, scale;
 };
 
@@ -140,7 +179,7 @@ __device__ __forceinline__ float gate_act(const GatedNorm& a, float g) {
   return a.silu ? g * s : s;
 }
 
-template <int GT, typename OUT>
+template <int GT, int KEEP, typename OUT>
 __global__ void __launch_bounds__(256) gated_norm_kernel(GatedNorm a, OUT* out) {
   __shared__ float s32[32];
   pdl_wait();
@@ -154,18 +193,18 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(GatedNorm a, OUT* out) 
   OUT* dst = out + (size_t)t * a.ld + c0;
   const float* w = a.w == nullptr ? nullptr : a.w + c0;
   auto sum = [&](float v) { return GT == 32 ? warp_sum(v) : block_sum(v, s32); };
-  if (a.vec) {                 // rows of float4, up to kKeep per thread
+  if constexpr (KEEP > 0) {
     const int nch = a.width >> 2;
-    float4 v[kKeep], g[kKeep];
+    float4 v[KEEP], g[KEEP];
     float ss = 0.0f;
 #pragma unroll
-    for (int i = 0; i < kKeep; ++i) {
+    for (int i = 0; i < KEEP; ++i) {
       const int c = lane + GT * i;
       v[i] = c < nch ? reinterpret_cast<const float4*>(orow)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
       g[i] = c < nch ? reinterpret_cast<const float4*>(grow)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
 #pragma unroll
-    for (int i = 0; i < kKeep; ++i) {
+    for (int i = 0; i < KEEP; ++i) {
       g[i] = make_float4(gate_act(a, g[i].x), gate_act(a, g[i].y), gate_act(a, g[i].z), gate_act(a, g[i].w));
       if (a.before) {
         v[i].x *= g[i].x; v[i].y *= g[i].y; v[i].z *= g[i].z; v[i].w *= g[i].w;
@@ -174,7 +213,7 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(GatedNorm a, OUT* out) 
     }
     const float inv = a.scale / sqrtf(sum(ss) / (float)a.width + a.eps);
 #pragma unroll
-    for (int i = 0; i < kKeep; ++i) {
+    for (int i = 0; i < KEEP; ++i) {
       const int c = lane + GT * i;
       if (c >= nch) continue;
       float4 y = make_float4(v[i].x * inv, v[i].y * inv, v[i].z * inv, v[i].w * inv);
@@ -204,19 +243,37 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(GatedNorm a, OUT* out) 
 }
 
 template <typename OUT>
-static int run_gated_norm(GatedNorm a, OUT* out, cudaStream_t stream) {
+static int run_gated_norm(const GatedNorm& a, OUT* out, cudaStream_t stream) {
   const uintptr_t at = reinterpret_cast<uintptr_t>(a.o) | reinterpret_cast<uintptr_t>(a.gate) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(out);
-  const bool wide = a.width > 128 * kKeep;
-  a.vec = a.width % 4 == 0 && a.width <= (wide ? 1024 : 128) * kKeep && a.ldo % 4 == 0 && a.ldg % 4 == 0 && a.ld % 4 == 0 && at % 16 == 0;
-  if (wide) return launch(gated_norm_kernel<256, OUT>, dim3(a.T * a.parts), 256, 0, stream, 1, 0, a, out);
-  return launch(gated_norm_kernel<32, OUT>, dim3((a.T * a.parts + 7) / 8), 256, 0, stream, 1, 0, a, out);
+  const bool vec = a.width % 4 == 0 && a.ldo % 4 == 0 && a.ldg % 4 == 0 && a.ld % 4 == 0 && at % 16 == 0;
+  const int items = a.T * a.parts;
+#define BONSAI_GATED(GT, KEEP) launch(gated_norm_kernel<GT, KEEP, OUT>, dim3((items + 256 / GT - 1) / (256 / GT)), 256, 0, stream, 1, 0, a, out)
+  if (a.width <= 512) {
+    if (!vec) return BONSAI_GATED(32, 0);
+    return a.width <= 128 ? BONSAI_GATED(32, 1) : (a.width <= 256 ? BONSAI_GATED(32, 2) : BONSAI_GATED(32, 4));
+  }
+  if (!vec || a.width > 4096) return BONSAI_GATED(256, 0);
+  return a.width <= 1024 ? BONSAI_GATED(256, 1) : (a.width <= 2048 ? BONSAI_GATED(256, 2) : BONSAI_GATED(256, 4));
+#undef BONSAI_GATED
 }
 
 static int row_threads(int width) {
-  const int want = (width + 15) / 16;   // kKeep float4 per thread
-  const int t = (want + 31) / 32 * 32;
-  return t < 64 ? 64 : (t > 1024 ? 1024 : (width >= 2048 && t < 512 ? 512 : t));
+  const int t = ((width + 7) / 8 + 31) / 32 * 32;   // two float4 per thread
+  return t < 64 ? 64 : (t > 1024 ? 1024 : t);
 }
+
+// float4 a thread keeps for rows of `width`, 0 where rows or pointers (or-ed together) are not made of float4
+static int row_keep(int width, int ld, uintptr_t pointers) {
+  const int th = row_threads(width);
+  return width % 4 != 0 || ld % 4 != 0 || pointers % 16 != 0 ? 0 : (width <= 8 * th ? 2 : (width <= 16 * th ? 4 : 0));
+}
+template <typename... P>
+static uintptr_t bits(const P*... p) { return (reinterpret_cast<uintptr_t>(p) | ...); }
+
+#define BONSAI_ROWS(KEEP, KERNEL, H, GRID, ...)                                                       \
+  (KEEP == 2 ? launch(KERNEL<2, H>, dim3(GRID), th, 0, stream, 1, 0, __VA_ARGS__)                     \
+             : (KEEP == 4 ? launch(KERNEL<4, H>, dim3(GRID), th, 0, stream, 1, 0, __VA_ARGS__)        \
+                          : launch(KERNEL<0, H>, dim3(GRID), th, 0, stream, 1, 0, __VA_ARGS__)))
 
 }  // namespace lay
 }  // namespace bonsai
@@ -229,9 +286,9 @@ int bonsai_lay_embed(const void* table, int ld_table, const int* tokens, float s
                      const float* next, float eps, cudaStream_t stream) {
   using namespace bonsai::lay;
   if (T < 1 || width < 1 || ld_table < width || (h != nullptr && ldh < width)) return BONSAI_CUDA_BAD_ARG;
-  if (h_f32)
-    return launch(embed_kernel<float>, dim3(T), 256, 0, stream, 1, 0, (const bf16*)table, ld_table, tokens, scale, width, x, (float*)h, ldh, next, eps);
-  return launch(embed_kernel<bf16>, dim3(T), 256, 0, stream, 1, 0, (const bf16*)table, ld_table, tokens, scale, width, x, (bf16*)h, ldh, next, eps);
+  const int th = row_threads(width), keep = row_keep(width, ld_table | ldh, bits((const char*)table, x, (const char*)h, next));
+  return h_f32 ? BONSAI_ROWS(keep, embed_kernel, float, T, (const bf16*)table, ld_table, tokens, scale, width, x, (float*)h, ldh, next, eps)
+               : BONSAI_ROWS(keep, embed_kernel, bf16, T, (const bf16*)table, ld_table, tokens, scale, width, x, (bf16*)h, ldh, next, eps);
 }
 
 // x += norm(y) * w; h (may be null) = x or, with `next`, its norm
@@ -239,9 +296,9 @@ int bonsai_lay_norm_add(float* x, const float* y, int ldy, const float* w, float
                         cudaStream_t stream) {
   using namespace bonsai::lay;
   if (T < 1 || width < 1 || ldy < width || (ldy & 3) != 0 || (h != nullptr && (ldh < width || (ldh & 3) != 0))) return BONSAI_CUDA_BAD_ARG;
-  const int th = row_threads(width);
-  if (h_f32) return launch(norm_add_kernel<float>, dim3(T), th, 0, stream, 1, 0, x, y, ldy, w, eps, width, (float*)h, ldh, next);
-  return launch(norm_add_kernel<bf16>, dim3(T), th, 0, stream, 1, 0, x, y, ldy, w, eps, width, (bf16*)h, ldh, next);
+  const int th = row_threads(width), keep = row_keep(width, ldy | ldh, bits(x, y, w, (const char*)h, next));
+  return h_f32 ? BONSAI_ROWS(keep, norm_add_kernel, float, T, x, y, ldy, w, eps, width, (float*)h, ldh, next)
+               : BONSAI_ROWS(keep, norm_add_kernel, bf16, T, x, y, ldy, w, eps, width, (bf16*)h, ldh, next);
 }
 
 // out: bf16 when f32_out == 0, f32 otherwise
@@ -249,9 +306,9 @@ int bonsai_lay_norm_rows(const float* x, const int* rows, const float* w, float 
                          cudaStream_t stream) {
   using namespace bonsai::lay;
   if (R < 1 || width < 1 || ld < width) return BONSAI_CUDA_BAD_ARG;
-  const int th = row_threads(width);
-  if (f32_out) return launch(norm_rows_kernel<float>, dim3(R), th, 0, stream, 1, 0, x, rows, w, eps, width, (float*)out, ld);
-  return launch(norm_rows_kernel<bf16>, dim3(R), th, 0, stream, 1, 0, x, rows, w, eps, width, (bf16*)out, ld);
+  const int th = row_threads(width), keep = row_keep(width, ld, bits(x, w, (const char*)out));
+  return f32_out ? BONSAI_ROWS(keep, norm_rows_kernel, float, R, x, rows, w, eps, width, (float*)out, ld)
+                 : BONSAI_ROWS(keep, norm_rows_kernel, bf16, R, x, rows, w, eps, width, (bf16*)out, ld);
 }
 
 // Gated norm: o and gate f32 [T][ld..] with `parts` parts of `width` columns, w [parts * width] or null; act 0 =
@@ -260,7 +317,7 @@ int bonsai_lay_gated_norm(const float* o, int ldo, const float* gate, int ldg, c
                           float scale, void* out, int ld, int f32_out, cudaStream_t stream) {
   using namespace bonsai::lay;
   if (T < 1 || parts < 1 || width < 1 || ld < parts * width || (long long)T * parts >= (1ll << 30)) return BONSAI_CUDA_BAD_ARG;
-  const GatedNorm a{o, gate, w, ldo, ldg, T, parts, width, ld, 0, act, before, eps, scale};
+  const GatedNorm a{o, gate, w, ldo, ldg, T, parts, width, ld, act, before, eps, scale};
   return f32_out ? run_gated_norm(a, (float*)out, stream) : run_gated_norm(a, (bf16*)out, stream);
 }
 

@@ -177,26 +177,66 @@ class StepShape:
     portions: int = 0
     entries: int = 0
     tiles: dict[int, tuple[int, int]] | None = None      # tokens per tile -> (device address, tiles)
-    segments: int = 0                                    # recurrences run the portions cut into this many segments (0: whole)
-    segment_list: int = 0
-    prompt_list: int = 0
+    segments: dict["SegmentPlan", tuple[int, int, int]] | None = None    # recurrences that cut the portions: segments, device addresses of the two lists
+
+    def cut(self, plan: "SegmentPlan | None") -> tuple[int, int, int]:
+        """Segment list, segments (0: portions as a whole) and prompt list of a recurrence."""
+        n, segs, prompts = (self.segments or {}).get(plan, (0, 0, 0))
+        return segs, n, prompts
 
 
 MAX_SEGMENTS = 24           # segment states the scratch of the recurrent layers holds
 CHUNK = 64                  # tokens per chunk of the recurrences
 
 
-def plan_segments(lengths: Sequence[int], ctas: int, sms: int) -> int:
-    """Chunks per segment for portions of ``lengths`` tokens when one segment occupies ``ctas`` CTAs, one per SM; 0 = do not
-    cut.  Segments run side by side, but their state products run twice; the constants are fitted to measured times (8 heads of
-    256 x 512: 4096 tokens 600 us whole, 443 us in 2 segments, 451 in 4, 548 in 16; 512 tokens 76 us whole, 64 us in 2)."""
+@dataclass(frozen=True)
+class SegmentCost:
+    """What running a recurrence in segments costs, in times of one chunk of a lone CTA.  Segments run side by side, but their
+    state products run twice.  Fitted to measured times."""
+    resident: int           # CTAs an SM holds
+    crowded: float          # time of a chunk when an SM is full
+    twice: float            # both passes of a segment over one pass
+    fixed: float
+    each: float             # per segment
+    shortest: int           # chunks
+
+    def waves(self, ctas: int, sms: int) -> float:
+        if self.resident > 1 and ctas <= 0.6 * sms:        # more of them do not spread evenly
+            return 1.0
+        return self.crowded * -(-ctas // (self.resident * sms))
+
+
+# mLSTM, 8 heads of 256 x 512: 4096 tokens 600 us whole, 443 us in 2 segments, 451 in 4, 548 in 16; 512 tokens 76 us whole, 64 us in 2.
+# Linear recurrence, 32 heads of 128 x 128: 4096 tokens 306 us whole, 166 in 4, 174 in 8, 210 in 32; 512 tokens 38 whole, 30 in 4.
+# 16 heads of 256 x 256: 4096 tokens 424 us whole, 315 in 2, 324 in 4; 512 tokens 55 whole, 49 in 2.
+MLSTM_COST = SegmentCost(1, 1.0, 1.5, 0.5, 0.6, 4)
+RECURRENCE_COST = SegmentCost(2, 1.55, 1.45, 2.0, 0.08, 2)
+WIDE_RECURRENCE_COST = SegmentCost(1, 1.0, 1.35, 1.2, 0.1, 2)
+
+
+@dataclass(frozen=True)
+class SegmentPlan:
+    """Layers with as many CTAs per portion and the same costs cut a step's portions alike."""
+    ctas: int
+    cost: SegmentCost
+
+
+def segment_plan(m: MlstmSpec | LinearRecurrenceSpec) -> SegmentPlan:
+    d, e = state_dims(m)
+    cost = MLSTM_COST if isinstance(m, MlstmSpec) else (RECURRENCE_COST if d <= 128 else WIDE_RECURRENCE_COST)
+    return SegmentPlan(m.heads * e // 64, cost)
+
+
+def plan_segments(lengths: Sequence[int], plan: SegmentPlan, sms: int) -> int:
+    """Chunks per segment for portions of ``lengths`` tokens; 0 = do not cut."""
+    c = plan.cost
     chunks = [-(-n // CHUNK) for n in lengths]
-    best, best_cost = 0, max(chunks) * -(-ctas * len(chunks) // sms)
-    for size in range(4, max(chunks)):
-        segs = sum(-(-c // size) for c in chunks)
+    best, best_cost = 0, max(chunks) * c.waves(plan.ctas * len(chunks), sms)
+    for size in range(c.shortest, max(chunks)):
+        segs = sum(-(-n // size) for n in chunks)
         if segs > MAX_SEGMENTS:
             continue
-        cost = 1.5 * size * -(-ctas * segs // sms) + 0.5 + 0.6 * segs
+        cost = c.twice * size * c.waves(plan.ctas * segs, sms) + c.fixed + c.each * segs
         if cost < best_cost:
             best, best_cost = size, cost
     return best
@@ -248,6 +288,7 @@ class MlstmMixer:
         assert branch.scale == 1.0, "an mLSTM output is not scaled"
         q, k, v, self.g_col, i, f = w.columns
         self.chunked = not r.exact and runs_chunked(spec)
+        self.plan = segment_plan(spec)
         self.fused = spec.vdim <= L.lib().bonsai_lay_mlstm_fused_vdim()
         floats = [spec.gate_cap, cfg.eps, spec.den_eps, spec.dim ** -0.5]
 
@@ -273,7 +314,7 @@ class MlstmMixer:
         if st.portions:
             a = self.raw[id(rows)].args
             if self.chunked:
-                K.check(lib.bonsai_lay_mlstm_chunk(*a, st.entries, st.portions, st.segment_list, st.segments, st.prompt_list, stream), "mlstm_chunk")
+                K.check(lib.bonsai_lay_mlstm_chunk(*a, st.entries, st.portions, *st.cut(self.plan), stream), "mlstm_chunk")
             else:
                 K.check(lib.bonsai_lay_mlstm_step(*a, st.entries, st.portions, 0, stream), "mlstm_step")
             self._finish(st.singles, st.rows - st.singles)
@@ -288,6 +329,7 @@ class LinearRecurrenceMixer:
         spec, s, lib, vec = self.spec, r.states.tensors[index], L.lib(), w.vectors
         self.norm = vec.get("norm")
         self.chunked = not r.exact and runs_chunked(spec)
+        self.plan = segment_plan(spec)
         # the single-token step finishes its outputs itself when the norm is per head
         self.fused = spec.norm_parts == spec.heads and not spec.gate_first and spec.vdim <= lib.bonsai_lay_rec_fused_vdim()
         decay = rate = conv_w = freq = None
@@ -333,7 +375,7 @@ class LinearRecurrenceMixer:
             if self.spec.conv:
                 K.check(lib.bonsai_lay_rec_ring(*a, st.entries, st.portions, stream), "rec_ring")
             if self.chunked:
-                K.check(lib.bonsai_lay_rec_chunk(*a, st.entries, st.portions, st.segment_list, st.segments, st.prompt_list, stream), "rec_chunk")
+                K.check(lib.bonsai_lay_rec_chunk(*a, st.entries, st.portions, *st.cut(self.plan), stream), "rec_chunk")
             else:
                 K.check(lib.bonsai_lay_rec_step(*a, st.entries, st.portions, 0, exact, 0, stream), "rec_step")
             self._finish(st.singles, st.rows - st.singles)
@@ -385,14 +427,14 @@ class LayeredRunner(SlotState):
         # states of the segments a long prompt is cut into (layers run one after another and share them)
         chunked = [] if exact else [m for m in recurrent if runs_chunked(m)]
         shapes = [(m.heads, *state_dims(m)) for m in chunked]
-        self._segment_ctas = min((h * e // 64 for h, _, e in shapes), default=0)
-        segs = min(MAX_SEGMENTS, cap // CHUNK) if shapes else 0
+        self.segment_plans = sorted({segment_plan(m) for m in chunked}, key=lambda p: p.ctas)
+        segs = MAX_SEGMENTS if shapes else 0
         self.segment_scratch = [torch.empty(max(1, segs * max((f(*s) for s in shapes), default=0)), **f32) for f in
                                 (lambda h, d, e: h * d * e, lambda h, d, e: h * d * e // 64, lambda h, d, e: h * e // 64, lambda h, d, e: h * e // 32)]
         # row metadata: decode steps use the slot tensors as they are; a mixed batch uploads [tokens | positions | slots | lists]
         self.slot_rows = Rows(self.tokens, self.positions, torch.arange(max_batch, **i32))
         self._tile_sizes = sorted({64 // cfg.attention(i).group for i in cfg.attention_layers})
-        self._meta = torch.zeros(3 * cap + 4 * cap + 8 * MAX_SEGMENTS + 2 * cap * len(self._tile_sizes) + cap + 16, **i32)
+        self._meta = torch.zeros(3 * cap + 4 * cap + 8 * MAX_SEGMENTS * len(self.segment_plans) + 2 * cap * len(self._tile_sizes) + cap + 16, **i32)
         self.batch_rows = Rows(*(self._meta[i * cap:(i + 1) * cap] for i in range(3)))
         self._host = [torch.zeros(self._meta.numel(), dtype=torch.int32).pin_memory() for _ in range(2)]
         self._host_free = [torch.cuda.Event() for _ in range(2)]
@@ -438,34 +480,38 @@ class LayeredRunner(SlotState):
             raise ValueError("the layer-list decoders have one cache format per engine")
 
     # ---- one step ------------------------------------------------------------------------------------------------------------------
-    def _layers(self, rows: Rows, st: StepShape) -> None:
+    def _layers(self, rows: Rows, st: StepShape, final: bool = False) -> None:
+        """Embedding and layers.  ``final``: the last residual step leaves the final norm of all rows in ``normed``."""
         cfg, T, s = self.cfg, st.rows, K.stream()
         x, h, layers = self.x, self.h, self.w.layers
         copy = None if h is x else h
         L.embed(self.w.embed.data, rows.tokens, cfg.embed_scale, T, cfg.width, x, copy, layers[0].pre_norm, cfg.eps)
         for i, (spec, w) in enumerate(zip(cfg.layer_specs, layers)):
-            following = layers[i + 1].pre_norm if i + 1 < len(layers) else None
+            last = i + 1 == len(layers)
+            after, following = (self.normed, self.w.final_norm) if last and final else (copy, None if last else layers[i + 1].pre_norm)
             L.linear(w.proj, h, T, self.proj, self.scratch)
             for n, mixer in enumerate(self.mixers[i]):
                 mixer(rows, st, s, early=n > 0)            # only the first one follows the projection directly
             L.linear(w.out, self.mixer_out[i], T, self.y, self.scratch)
-            L.norm_add(x, self.y, w.norm, cfg.eps, T, copy, following if w.mlp is None else w.mlp.pre_norm)
-            if w.mlp is not None:
+            if w.mlp is None:
+                L.norm_add(x, self.y, w.norm, cfg.eps, T, after, following)
+            else:
+                L.norm_add(x, self.y, w.norm, cfg.eps, T, copy, w.mlp.pre_norm)
                 act = self.act_buffer(spec.mlp.ff)
                 L.linear(w.mlp.up, h, T, act, self.scratch, w.mlp.act)
                 L.linear(w.mlp.down, act, T, self.y, self.scratch)
-                L.norm_add(x, self.y, w.mlp.norm, cfg.eps, T, copy, following)
+                L.norm_add(x, self.y, w.mlp.norm, cfg.eps, T, after, following)
 
-    def _head(self, row_list: int | None, count: int, out: torch.Tensor) -> None:
-        """Logits of ``count`` rows (device address of their indices, None = the first ones) into ``out`` [count, vocab]."""
+    def _head(self, row_list: int, count: int, out: torch.Tensor) -> None:
+        """Logits of ``count`` rows (device address of their indices) into ``out`` [count, vocab]."""
         L.norm_rows(self.x, row_list, count, self.w.final_norm, self.cfg.eps, self.normed)
         L.linear(self.w.embed, self.normed, count, out, self.scratch)
 
     def step_eager(self, batch: int, sample: bool = True, lm_head: bool = True, masked: bool = False) -> None:
         """One token for each of the slots 0 .. batch-1 (tokens and positions are read from the slot tensors)."""
-        self._layers(self.slot_rows, StepShape(batch, batch))
+        self._layers(self.slot_rows, StepShape(batch, batch), final=lm_head)
         if lm_head:
-            self._head(None, batch, self.logits)
+            L.linear(self.w.embed, self.normed, batch, self.logits, self.scratch)
         if sample:
             self.sample_rows(0, batch, masked, advance=True)
 
@@ -516,15 +562,17 @@ class LayeredRunner(SlotState):
         end = -(-3 * cap // 4) * 4
         put = lambda a: (end, end + a.size)
         base = self._meta.data_ptr()
-        st = StepShape(T, singles, len(lists), base + 4 * end, {})
+        st = StepShape(T, singles, len(lists), base + 4 * end, {}, {})
         if lists:
             a = np.asarray(lists, dtype=np.int32).reshape(-1)
             lo, hi = put(a)
             host[lo:hi] = a
             end = hi
             lengths = [n for _, n, _, _ in lists]
-            size = plan_segments(lengths, self._segment_ctas, self.scratch.sms) if self._segment_ctas else 0
-            if size:
+            for plan in self.segment_plans:
+                size = plan_segments(lengths, plan, self.scratch.sms)
+                if not size:
+                    continue
                 segs, prompts = [], []
                 for first, n, slot, pos0 in lists:
                     cuts = range(0, n, size * CHUNK)
@@ -533,7 +581,7 @@ class LayeredRunner(SlotState):
                 a = np.asarray(segs + prompts, dtype=np.int32).reshape(-1)
                 lo, hi = put(a)
                 host[lo:hi] = a
-                st.segments, st.segment_list, st.prompt_list = len(segs), base + 4 * lo, base + 4 * (lo + 4 * len(segs))
+                st.segments[plan] = (len(segs), base + 4 * lo, base + 4 * (lo + 4 * len(segs)))
                 end = hi
             for size in self._tile_sizes:
                 a = np.asarray([(e, t) for e, (_, n, _, _) in enumerate(lists) for t in range(0, n, size)], dtype=np.int32).reshape(-1)
@@ -571,7 +619,7 @@ class LayeredRunner(SlotState):
 
     def kernel_launches(self, batch: int, sample: bool = True) -> int:
         """Launches of one decode step (each is one of this library's kernels)."""
-        n = 1 + 2 + int(sample)
+        n = 2 + int(sample)
         for spec, mixers in zip(self.cfg.layer_specs, self.mixers):
             n += 3 + sum(m.launches() for m in mixers) + (3 if spec.mlp is not None else 0)
         return n

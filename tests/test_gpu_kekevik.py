@@ -289,7 +289,7 @@ def test_long_prompts_in_segments(tmp_path, d, e):
     poison(eng)
     tokens = m.tokens(900)
     want = m.logits(tokens)
-    assert plan_segments([900], eng.runner._segment_ctas, 148) and plan_segments([600, 700], eng.runner._segment_ctas, 148)
+    assert eng.runner.segment_plans and all(plan_segments(n, p, 148) for p in eng.runner.segment_plans for n in ([900], [600, 700]))
     check(feed(eng, tokens, []), want, "bf16", "whole")
     check(feed(eng, tokens, [77, 700, 2]), want, "bf16", "resumed")
     for s, n in ((0, 601), (1, 1), (2, 901)):

@@ -170,7 +170,8 @@ def test_long_prompts_in_segments(tmp_path, d, e):
     poison(eng)
     tokens = m.tokens(900)
     want = m.logits(tokens)
-    assert plan_segments([900], eng.runner._segment_ctas, 148) and plan_segments([600, 700], eng.runner._segment_ctas, 148)
+    (plan,) = eng.runner.segment_plans
+    assert plan_segments([900], plan, 148) and plan_segments([600, 700], plan, 148)
     check(feed(eng, tokens, []), want, "bf16", "whole")
     check(feed(eng, tokens, [77, 700, 2]), want, "bf16", "resumed")
     for s, n in ((0, 600), (1, 1), (2, 900)):

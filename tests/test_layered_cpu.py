@@ -216,10 +216,12 @@ def test_scheduler_cancel_pending_mixed():
 
 
 def test_segment_plan():
-    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, plan_segments
-    assert plan_segments([100], 64, 148) == 0 and plan_segments([512] * 8, 64, 148) == 0 and plan_segments([2], 1, 148) == 0
-    for lengths, ctas in (([4096], 64), ([4096], 2), ([100_000], 1), ([900, 2, 700], 4), ([64 * 9 + 1], 3), ([2000] * 30, 1)):
-        size = plan_segments(lengths, ctas, 148)
-        segs = sum(-(-n // (size * CHUNK)) for n in lengths) if size else 0
-        assert segs <= MAX_SEGMENTS and (size == 0 or size >= 4)
-        assert size > 0 or len(lengths) > MAX_SEGMENTS
+    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, MLSTM_COST, RECURRENCE_COST, WIDE_RECURRENCE_COST, SegmentPlan, plan_segments
+    for cost in (MLSTM_COST, RECURRENCE_COST, WIDE_RECURRENCE_COST):
+        plan = lambda ctas: SegmentPlan(ctas, cost)
+        assert plan_segments([100], plan(64), 148) == 0 and plan_segments([512] * 8, plan(64), 148) == 0 and plan_segments([2], plan(1), 148) == 0
+        for lengths, ctas in (([4096], 64), ([4096], 2), ([100_000], 1), ([900, 2, 700], 4), ([64 * 9 + 1], 3), ([2000] * 30, 1)):
+            size = plan_segments(lengths, plan(ctas), 148)
+            segs = sum(-(-n // (size * CHUNK)) for n in lengths) if size else 0
+            assert segs <= MAX_SEGMENTS and (size == 0 or size >= cost.shortest)
+            assert size > 0 or len(lengths) > MAX_SEGMENTS
