@@ -10,7 +10,7 @@
 //  * one row per token that is both key and value (designs whose values are the un-normalised keys): the row holds the projected
 //    key, a float beside it the reciprocal root mean square, which multiplies the scores of its column.  Half the cache traffic
 //    of separate rows, and a tile is staged once for S = Q K^T and O = P K;
-//  * SEP: a row of normalised keys and a row of values, both padded to the same row length.
+//  * SEP: a row of normalised keys and a row of values, both padded to the same row length.  Scores are capped only here.
 //
 // Rows of a batch are tokens: a row has a position and a slot (its sequence's block-table row).  `append_kernel` writes the
 // rows' keys; `prompt_kernel` handles portions of prompts (tiles of 64 query rows = tokens x heads of one kv group);
@@ -115,15 +115,12 @@ __device__ __forceinline__ void load_query(const Attn& a, const float* q, int po
     const int d = lane + 32 * i;
     v[i] = d < a.dim ? q[d] : 0.0f;
     ss += v[i] * v[i];
+    if (a.q_norm != nullptr && d < a.dim) v[i] *= a.q_norm[d] * a.k_norm[d];
   }
   ss = warp_sum(ss);
   const float f = a.scale * temperature(a, pos) * (a.softcap > 0.0f ? 2.0f * kLog2e / a.softcap : kLog2e) / sqrtf(ss / (float)a.dim + a.eps);
 #pragma unroll
-  for (int i = 0; i < HD / 32; ++i) {
-    const int d = lane + 32 * i;
-    const float w = d < a.dim && a.q_norm != nullptr ? a.q_norm[d] * a.k_norm[d] : 1.0f;
-    dst[d] = __float2bfloat16_rn(v[i] * f * w);
-  }
+  for (int i = 0; i < HD / 32; ++i) dst[lane + 32 * i] = __float2bfloat16_rn(v[i] * f);
 }
 
 // ---- portions of prompts ------------------------------------------------------------------------------------------------------
@@ -234,7 +231,7 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
       for (int e = 0; e < 4; ++e) {
         const int r = e >> 1, j = kb + c + (e & 1);
         if (!SEP) s[nt][e] *= (e & 1) ? f.y : f.x;
-        if (a.softcap > 0.0f) s[nt][e] = cap_score(s[nt][e], cap);
+        if (SEP && a.softcap > 0.0f) s[nt][e] = cap_score(s[nt][e], cap);
         s[nt][e] -= slope[r] * (float)(qpos[r] - j);
         if (!whole && !sees(a, qpos[r], j)) s[nt][e] = -INFINITY;
         nm[r] = fmaxf(nm[r], s[nt][e]);
@@ -417,7 +414,7 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
       for (int e = 0; e < 4; ++e) {
         const int c = nt * 8 + (lane & 3) * 2 + (e & 1), j1 = tb + c;
         if (!SEP) s[nt][e] *= kf[c];
-        if (a.softcap > 0.0f) s[nt][e] = cap_score(s[nt][e], cap);
+        if (SEP && a.softcap > 0.0f) s[nt][e] = cap_score(s[nt][e], cap);
         s[nt][e] -= slope[e >> 1] * (float)(pos - j1);
         if (!sees(a, pos, j1)) s[nt][e] = -INFINITY;
         nm[e >> 1] = fmaxf(nm[e >> 1], s[nt][e]);
@@ -556,7 +553,7 @@ __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
       s = fmaf(q[c], k[c], s);
     }
     s = warp_sum(s) * scale * (SEP ? 1.0f : a.krms[row]);
-    if (a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
+    if (SEP && a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
     s -= slope * (float)(pos - j);
     const float nm = fmaxf(m, s), f = expf(m - nm), p = expf(s - nm);
     m = nm;
@@ -624,7 +621,7 @@ static bool fill(Attn& a, const void* const* ptrs, const int* ints, const float*
   for (a.pshift = 0; (2 << a.pshift) <= ints[11]; ++a.pshift) {}
   a.window = ints[12]; a.keep = ints[13];
   a.eps = floats[0]; a.scale = floats[1]; a.out_scale = floats[2]; a.softcap = floats[3]; a.temp_coef = floats[4]; a.temp_every = floats[5];
-  if (a.vpool == nullptr ? a.krms == nullptr || a.vdim != a.dim : a.vdim < 1) return false;
+  if (a.vpool == nullptr ? a.krms == nullptr || a.vdim != a.dim || a.softcap > 0.0f : a.vdim < 1) return false;
   return a.heads >= 1 && a.kv_heads >= 1 && a.heads % a.kv_heads == 0 && a.heads / a.kv_heads <= 64 && a.dim >= 1 &&
          padded_dim(a.dim > a.vdim ? a.dim : a.vdim) > 0 && a.pshift >= 4 && (1 << a.pshift) == ints[11] && a.keep >= 0 &&
          (a.temp_coef == 0.0f || a.temp_every > 0.0f) && (a.q_norm == nullptr) == (a.k_norm == nullptr);

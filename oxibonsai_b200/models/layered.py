@@ -210,8 +210,8 @@ class SegmentCost:
 # Linear recurrence, 32 heads of 128 x 128: 4096 tokens 306 us whole, 166 in 4, 174 in 8, 210 in 32; 512 tokens 38 whole, 30 in 4.
 # 16 heads of 256 x 256: 4096 tokens 424 us whole, 315 in 2, 324 in 4; 512 tokens 55 whole, 49 in 2.
 MLSTM_COST = SegmentCost(1, 1.0, 1.5, 0.5, 0.6, 4)
-RECURRENCE_COST = SegmentCost(2, 1.55, 1.45, 2.0, 0.08, 2)
-WIDE_RECURRENCE_COST = SegmentCost(1, 1.0, 1.35, 1.2, 0.1, 2)
+RECURRENCE_COST = SegmentCost(2, 1.55, 1.45, 2.0, 0.3, 2)
+WIDE_RECURRENCE_COST = SegmentCost(1, 1.0, 1.35, 1.2, 0.6, 2)
 
 
 @dataclass(frozen=True)

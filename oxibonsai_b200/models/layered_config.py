@@ -50,7 +50,7 @@ class AttentionSpec(MixerSpec):
     slope_exponent: float | None = None    # geometric slopes of a linear distance bias
     norm_weights: bool = False  # weights of the query and key norms
     gated: bool = False         # one sigmoid gate per head on the output
-    softcap: float = 0.0        # scores become softcap * tanh(score / softcap); 0 = as they are
+    softcap: float = 0.0        # scores become softcap * tanh(score / softcap), with separate values; 0 = as they are
     temp_coef: float = 0.0      # queries are multiplied by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)
     temp_every: float = 1.0
     kind = "attention"
