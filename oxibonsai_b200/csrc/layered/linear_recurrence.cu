@@ -11,7 +11,7 @@
 // `step_kernel` runs the recurrence as written, a column tile of 64 values of one head per CTA, the state in registers.  For
 // single tokens it makes the features itself and, where the norm is per head, finishes the outputs (the column tiles of a head
 // form a cluster and exchange their sums of squares).  For several tokens (32-bit mode, long keys) it reads prepared features.
-// `features_kernel` prepares the features of prompt rows; `chunk_kernel` runs portions of prompts on the tensor cores, 64 tokens
+// `features_kernel` prepares the features of prompt rows; `rec_chunk_kernel` runs portions of prompts on the tensor cores, 64 tokens
 // at a time.  With F the running sum of log2 a inside the chunk, token t sees token s <= t with weight b_s 2^(F_t - F_s) and the
 // chunk's initial state with weight 2^F_t, so no exponent is positive for decays up to 1:
 //   o_t = sum_s b_s 2^(F_t - F_s) (q_t . k_s) v_s + 2^F_t S_0^T q_t,    S' = 2^F_L S_0 + sum_s b_s 2^(F_L - F_s) k_s v_s^T
