@@ -146,8 +146,8 @@ def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
         proj = torch.randn(B, ld, device=dev)
         w1, slopes = torch.ones(hd, device=dev), torch.full((nq,), 0.01, device=dev)
         out = torch.zeros(B, nq * hd, dtype=torch.bfloat16, device=dev)
-        calls = [L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, p, rk, None, out],
-                             [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, 0, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0]) for p in pools]
+        calls = [L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, p, rk, None, out, None, None],
+                             [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, 0, 0, 1, 0, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0]) for p in pools]
         it = [0]
         split = 1
         while split < 8 and B * nkv * split * 2 <= 160:
@@ -173,8 +173,8 @@ def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
     entries = torch.tensor([0, T, 0, 0], **i32)
     tiles = torch.tensor([[0, t] for t in range(0, T, tpt)], **i32)
     for window in (0, 1024):
-        call = L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, pool, rk, None, out],
-                           [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, window, 4], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0])
+        call = L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, pool, rk, None, out, None, None],
+                           [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, window, 4, 1, 0, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0])
 
         def ours():
             K.check(L.lib().bonsai_lay_attn_prompt(*call.args, entries.data_ptr(), tiles.data_ptr(), len(tiles), K.stream()), "attn_prompt")
@@ -201,8 +201,8 @@ def bench_capped_attention(rep: Report, width: int, iters: int, profile: bool) -
     ld = (nq + 2 * nkv) * hd
 
     def call(proj, pos, slots, bt, k, v, out, cap=50.0):
-        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out],
-                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0], [1e-6, hd ** -0.5, 0.5, cap, 0.1, 4096.0])
+        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out, None, None],
+                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0, 1, 0, 0], [1e-6, hd ** -0.5, 0.5, cap, 0.1, 4096.0])
     for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
         npages = ctx // page
         copies = max(2, int(300e6 / (4 * B * ctx * nkv * hd)) + 1)

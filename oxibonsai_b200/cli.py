@@ -7,7 +7,9 @@ model, :420-625 run / chat loops, :604-621 the summary line ``"{p} prompt + {g} 
 from __future__ import annotations
 
 import argparse
+import dataclasses
 import json
+import math
 import os
 import re
 import sys
@@ -156,11 +158,12 @@ def model_dir_info(path: str) -> dict:
     cfg = load_model_dir_config(path)
     v = validate_model_dir(path)
     weights = Path(path) / "model.safetensors"
-    fields = lambda spec: {k: vars(x) if k == "rotary" and x is not None else x for k, x in vars(spec).items() if k != "parts"}
+    plain = lambda v: {k: plain(x) for k, x in v.items()} if isinstance(v, dict) else (None if v in (math.inf, -math.inf) else v)
+    fields = lambda spec: {k: x for k, x in plain(dataclasses.asdict(spec)).items() if k != "parts"}
     layers = []
     for s in cfg.layer_specs:
         parts = [{"prefix": b.prefix, "output_scale": b.scale, "mixer": b.spec.kind, **fields(b.spec)} for b in s.mixer.branches if b.prefix]
-        layers.append({"mixer": s.mixer.kind, **fields(s.mixer), **({"parts": parts} if parts else {}), "mlp": None if s.mlp is None else dict(vars(s.mlp))})
+        layers.append({"mixer": s.mixer.kind, **fields(s.mixer), **({"parts": parts} if parts else {}), "mlp": None if s.mlp is None else fields(s.mlp)})
     return {"path": path, "gpu_engine": "layer-list engine", "architecture": cfg.arch, "name": cfg.name, "quantization": "BF16",
             "tensors": len(cfg.tensor_shapes()), "estimated_parameters": cfg.param_count(),
             "file_size_bytes": os.path.getsize(weights) if weights.exists() else 0,
@@ -202,7 +205,9 @@ def cmd_info(args) -> int:
         print(f"# {info['name']}\narchitecture: {info['architecture']} ({c['layers']} layers x {c['hidden']}, vocab {c['vocab']}, "
               f"{info['estimated_parameters'] / 1e6:.1f} M parameters, {info['quantization']})\nGPU engine: {info['gpu_engine']}")
         for i, l in enumerate(c["layer_list"]):
-            print(f"  layer {i}: " + ", ".join(f"{k} {v}" for k, v in l.items() if k != "mlp") + (", no feed-forward" if l["mlp"] is None else f", feed-forward {l['mlp']['ff']}"))
+            m = l["mlp"]
+            ff = ", no feed-forward" if m is None else f", feed-forward {m['ff']}" + (f" x {m['router']['top']} of {m['router']['experts']}" if "router" in m else "")
+            print(f"  layer {i}: " + ", ".join(f"{k} {v}" for k, v in l.items() if k != "mlp") + ff)
     else:
         from .core import GgufFile
         from .core.compat import extract_model_card

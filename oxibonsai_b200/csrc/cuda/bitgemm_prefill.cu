@@ -23,6 +23,10 @@
 // the CTA that observes the final count adds the partials in CTA order (a fixed order: results do not depend on
 // timing) and applies the epilogue.  Without a workspace every CTA gets whole tiles.
 //
+// Grouped form (dense operands): the rows of X belong to groups (the experts of a mixture), group g to the rows offsets[g] ..
+// offsets[g + 1] - 1, and each group has its own weight matrix, one below the other.  The offsets are made on the device, so every
+// CTA derives the tile list (groups in order, 128 weight rows x TOK rows of one group) from them and takes an equal share of it.
+//
 // K order: the expansion naturally yields the weights of a 16-input word in the order
 // [0,4,1,5,2,6,3,7, 8,12,9,13,10,14,11,15]; instead of un-shuffling them the activation operand is
 // kept in the same order ("paired-K" layout), which every producer of a prefill activation writes
@@ -65,6 +69,9 @@ struct PfParams {
   int dense;               // 1: A is a dense f16 / bf16 matrix fetched by TMA (natural K order), no expansion
   int bf16;                // dense operands are bf16 (both) instead of f16
   float glu_limit, glu_alpha, glu_offset;   // epi 4
+  const float* row_scale;  // epi 4, grouped: factor of a row's outputs
+  const int* offsets;      // grouped: [groups + 1] first row of every group (device memory)
+  int groups;
   int streamk;             // 1: ranges cut anywhere in (tile, pair) space, partial tiles meet in the workspace
   float* ws_part;          // [2 * grid][TOK][128] partial accumulators
   int* ws_count;           // [tiles] arrival counters, zero between launches
@@ -124,17 +131,19 @@ __device__ __forceinline__ float pf_residual(const PfParams& p, int tok, int row
   return p.epi == 1 && row_ok && tok < p.T ? p.residual[(size_t)tok * p.out_ld + row] : 0.0f;
 }
 
-// epilogue for one accumulator value; every lane of the warp calls it (epi 2 exchanges gate / up between lanes)
-__device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, int tok, int row, int a, bool row_ok) {
+// epilogue for one accumulator value; every lane of the warp calls it (epi 2 exchanges gate / up between lanes); tend: the rows of X
+// that belong to the tile end there
+__device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, int tok, int tend, int row, int a, bool row_ok) {
   if (p.epi == 2) {
     float other = __shfl_xor_sync(0xffffffffu, v, 1);
-    if (row_ok && tok < p.T && (a & 1) == 0)
+    if (row_ok && tok < tend && (a & 1) == 0)
       p.out_f16[(size_t)tok * p.out_ld + paired_k(row >> 1)] = __float2half_rn(v / (1.0f + __expf(-v)) * other);
-  } else if (row_ok && tok < p.T) {
+  } else if (row_ok && tok < tend) {
     const size_t o = (size_t)tok * p.out_ld + row;
     if (p.epi == 0) p.out_f32[o] = v;
     else if (p.epi == 1) p.out_f32[o] = res + v;
     else if (p.epi == 5) reinterpret_cast<__nv_bfloat16*>(p.out_f16)[o] = __float2bfloat16_rn(fmaxf(v, 0.0f) * fmaxf(v, 0.0f));
+    else if (p.epi == 6) reinterpret_cast<__nv_bfloat16*>(p.out_f16)[o] = __float2bfloat16_rn(v);
     else p.out_f16[o] = __float2half_rn(v);
   }
 }
@@ -143,8 +152,8 @@ __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, 
 // and up (odd) rows, min(g, limit) * sigmoid(alpha g) * (clamp(u, -limit, limit) + offset), stored as bf16.  The two lanes of a
 // pair split the columns: the even lane finishes even ones, the odd lane odd ones, so every lane has CB / 2 outputs and one
 // shuffle per output.
-template <int CB>
-__device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, int tok0, int row, int a, bool row_ok) {
+template <int CB, bool SCALED = false>
+__device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, int tok0, int tend, int row, int a, bool row_ok) {
   const bool odd = a & 1;
   float o[CB / 2];
 #pragma unroll
@@ -159,14 +168,32 @@ __device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, 
 #pragma unroll
   for (int j = 0; j < CB / 2; ++j) {
     const int tok = tok0 + 2 * j + (odd ? 1 : 0);
-    if (row_ok && tok < p.T) dst[(size_t)tok * p.out_ld] = __float2bfloat16_rn(o[j]);
+    if (row_ok && tok < tend) dst[(size_t)tok * p.out_ld] = __float2bfloat16_rn(SCALED ? o[j] * p.row_scale[tok] : o[j]);
   }
 }
 
 __device__ __forceinline__ void pf_epi_barrier() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
+constexpr int kPfMaxGroups = 512;
+
+struct PfTile {
+  int arow, row0, tok0, tend;   // first weight row in the matrix and in its group, first row of X, end of the rows that count
+};
+
+// tile number `tile` of a grouped product; first[g]: number of the group's first tile
+__device__ __forceinline__ PfTile pf_group_tile(const PfParams& p, const int* first, const int* off, int tile, int row_tiles, int tok_per_tile) {
+  int lo = 0, hi = p.groups - 1;   // last group whose first tile is not behind this one
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (first[mid] <= tile) lo = mid;
+    else hi = mid - 1;
+  }
+  const int in = tile - first[lo], row0 = (in % row_tiles) * 128;
+  return PfTile{lo * p.n_rows + row0, row0, off[lo] + (in / row_tiles) * tok_per_tile, off[lo + 1]};
+}
+
 // TOK = tokens per tile (MMA N): 256 for prompt chunks, 64 for batched decode / verification.
-template <int TOK>
+template <int TOK, bool GROUPED = false>
 __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __grid_constant__ CUtensorMap xmap,
                                                                      const __grid_constant__ CUtensorMap amap, PfParams p) {
   constexpr int S = TOK == 64 ? 8 : 4;   // pipeline stages (one 64-input k-block each)
@@ -189,11 +216,39 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
   __shared__ int s_info[4];
   __shared__ int s_slots[kPfMaxCtas];
   __shared__ uint64_t red_bar;   // completion of the bulk copies that bring partial tiles in for the final reduction
+  __shared__ int s_first[GROUPED ? kPfMaxGroups + 1 : 1], s_off[GROUPED ? kPfMaxGroups + 1 : 1];
   const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
   const int npairs = p.K >> 7;
   const int row_tiles = (p.n_rows + 127) >> 7, tok_tiles = (p.T + TOK - 1) / TOK;
-  const int ntiles = row_tiles * tok_tiles;
+  int ntiles = row_tiles * tok_tiles;
   const int grid = gridDim.x;
+  if (GROUPED) {
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    for (int g = t; g <= p.groups; g += kPfThreads) s_off[g] = min(p.offsets[g], p.T);
+    __syncthreads();
+    if (warp == 0) {
+      int total = 0;
+      for (int g0 = 0; g0 < p.groups; g0 += 32) {
+        const int g = g0 + lane, n = g < p.groups ? (max(s_off[g + 1] - s_off[g], 0) + TOK - 1) / TOK * row_tiles : 0;
+        int v = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const int u = __shfl_up_sync(0xffffffffu, v, o);
+          if (lane >= o) v += u;
+        }
+        if (g < p.groups) s_first[g] = total + v - n;
+        total += __shfl_sync(0xffffffffu, v, 31);
+      }
+      if (lane == 0) s_first[p.groups] = total;
+    }
+    __syncthreads();
+    ntiles = s_first[p.groups];
+  }
+  auto tile_at = [&](int tile) {
+    if (GROUPED) return pf_group_tile(p, s_first, s_off, tile, row_tiles, TOK);
+    const int row0 = (tile % row_tiles) * 128;
+    return PfTile{row0, row0, (tile / row_tiles) * TOK, p.T};
+  };
   const long long I0 = pf_range_start(p.streamk, blockIdx.x, grid, ntiles, npairs);
   const int n = (int)(pf_range_start(p.streamk, blockIdx.x + 1, grid, ntiles, npairs) - I0);   // pairs of this CTA
   const int tile0 = (int)(I0 / npairs), pair0 = (int)(I0 - (long long)tile0 * npairs);
@@ -240,9 +295,11 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const int tw = warp - kPfTmaWarp;
     int tile = tile0, pair = pair0;
+    PfTile tl{0, 0, 0, 0};
     for (int q = 0; q < n && !failed; ++q) {
       if (NISS == 1 || (q % NISS) == tw) {
-        const int tok0 = (tile / row_tiles) * TOK, row0 = (tile % row_tiles) * 128;
+        if (GROUPED ? (q == 0 || pair < NISS) : true) tl = tile_at(tile);     // grouped: an issuer's first pair of a tile
+        const int tok0 = tl.tok0, row0 = tl.arow;
         for (int g0 = 0; g0 < 2 && !failed; g0 += GK) {   // one barrier per GK k-blocks
           const int it = 2 * q + g0, bs = (it / GK) % NBS;
           if (!__all_sync(0xffffffffu, tc::mbar_wait(&empty_bar[bs], (((it / GK) / NBS) & 1) ^ 1))) { failed = true; break; }
@@ -386,10 +443,10 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
       const int len = min(n - q, npairs - pair_b);
       const bool whole = len == npairs;
       const int ab = seg & 1;
-      const int row = (tile % row_tiles) * 128 + a;
-      const int tok0 = (tile / row_tiles) * TOK;
+      const PfTile tl = tile_at(tile);
+      const int row = tl.row0 + a, tok0 = tl.tok0, tend = tl.tend;
       const bool row_ok = row < p.n_rows;
-      const int ncols = min(TOK, p.T - tok0);
+      const int ncols = min(TOK, tend - tok0);
       float* part = p.ws_part + (size_t)(2 * blockIdx.x + (q == 0 ? 0 : 1)) * (128 * TOK);
       if (!tc::mbar_wait_warp<64>(&accf_bar[ab], (seg >> 1) & 1, lane)) { failed = true; break; }
       tc::tc_fence_after();
@@ -419,13 +476,13 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
           float v[CB];
 #pragma unroll
           for (int j = 0; j < CB; ++j) v[j] = __uint_as_float(rr[j]);
-          pf_store_glu<CB>(p, v, tok0 + c0, row, a, row_ok);
+          pf_store_glu<CB, GROUPED>(p, v, tok0 + c0, tend, row, a, row_ok);
         } else if (whole) {
           float res[CB];
 #pragma unroll
           for (int j = 0; j < CB; ++j) res[j] = pf_residual(p, tok0 + c0 + j, row, row_ok);
 #pragma unroll
-          for (int j = 0; j < CB; ++j) pf_store(p, __uint_as_float(rr[j]), res[j], tok0 + c0 + j, row, a, row_ok);
+          for (int j = 0; j < CB; ++j) pf_store(p, __uint_as_float(rr[j]), res[j], tok0 + c0 + j, tend, row, a, row_ok);
         } else {
           // a slot is [TOK columns][128 rows]: a warp's store and the reducer's reads run along the rows
 #pragma unroll
@@ -497,12 +554,12 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
                   for (int i = 0; i < 5; ++i) v[j] += i < cnt ? x[i] : 0.0f;
                 }
                 if (last && p.epi == 4) {
-                  pf_store_glu<8>(p, v, tok0 + cb, row, a, row_ok);      // columns past the last token are dropped there
+                  pf_store_glu<8>(p, v, tok0 + cb, tend, row, a, row_ok);      // columns past the last token are dropped there
                   continue;
                 }
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
-                  if (last) pf_store(p, v[j], res[j], tok0 + cb + j, row, a, row_ok && cb + j < ncols);
+                  if (last) pf_store(p, v[j], res[j], tok0 + cb + j, tend, row, a, row_ok && cb + j < ncols);
                   else if (cb + j < ncols) carry[(cb + j) * 128 + a] = v[j];
                 }
               }
@@ -516,12 +573,12 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
                   if (c + j < ncols) v[j] += __ldcg(p.ws_part + (size_t)s_slots[i] * (128 * TOK) + (c + j) * 128 + a);
-              pf_store_glu<2>(p, v, tok0 + c, row, a, row_ok);
+              pf_store_glu<2>(p, v, tok0 + c, tend, row, a, row_ok);
             }
             for (int c = 0; c < ncols && p.epi != 4; ++c) {
               float v = 0.0f;
               for (int i = 0; i < nc; ++i) v += __ldcg(p.ws_part + (size_t)s_slots[i] * (128 * TOK) + c * 128 + a);
-              pf_store(p, v, pf_residual(p, tok0 + c, row, row_ok), tok0 + c, row, a, row_ok);
+              pf_store(p, v, pf_residual(p, tok0 + c, row, row_ok), tok0 + c, tend, row, a, row_ok);
             }
           }
           if (a == 0) p.ws_count[tile] = 0;
@@ -638,26 +695,51 @@ int bonsai_bitgemm_prefill_ws(const void* codes, const void* scales, const void*
     amap = xmap;
   }
   PfParams p{(const uint32_t*)codes, (const __half*)scales, out_f32, residual, (__half*)out_f16, status, n_rows, K, T, epi, out_ld,
-             dense_w != nullptr ? 1 : 0, 0, 0.0f, 0.0f, 0.0f, 0, nullptr, nullptr};
+             dense_w != nullptr ? 1 : 0, 0, 0.0f, 0.0f, 0.0f, nullptr, nullptr, 0, 0, nullptr, nullptr};
   return tok == 64 ? launch_prefill<64>(xmap, amap, p, sms, ws, ws_bytes, balance, stream)
                    : launch_prefill<256>(xmap, amap, p, sms, ws, ws_bytes, balance, stream);
 }
 
 // Dense bf16 operands: W [n_rows][K] (K a multiple of 128), x [T][x_ld], f32 accumulation.  epi 0: out_f32 = W x; 4: out_bf16 =
-// clamped gated unit over interleaved gate / up rows (n_rows / 2 columns); 5: out_bf16 = relu(W x)^2.  Workspace and status as above.
+// clamped gated unit over interleaved gate / up rows (n_rows / 2 columns); 5: out_bf16 = relu(W x)^2; 6: out_bf16 = W x.  Workspace and
+// status as above.
 int bonsai_dense_gemm_bf16(const void* w, int n_rows, int K, const void* x, int x_ld, int T, float* out_f32, void* out_bf16, int out_ld, int epi,
                            float limit, float alpha, float offset, int* status, void* ws, size_t ws_bytes, int sms, cudaStream_t stream) {
   using namespace bonsai;
-  if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && epi != 4 && epi != 5)) return BONSAI_CUDA_BAD_ARG;
+  if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && epi != 4 && epi != 5 && epi != 6)) return BONSAI_CUDA_BAD_ARG;
   if ((epi == 0 && out_f32 == nullptr) || (epi != 0 && out_bf16 == nullptr) || (epi == 4 && n_rows % 2 != 0) || status == nullptr) return BONSAI_CUDA_BAD_ARG;
   const int tok = T <= 64 ? 64 : 256;
   CUtensorMap xmap, amap;
   if (!make_map_f16(&xmap, x, K, T, x_ld, tok, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
       !make_map_f16(&amap, w, K, n_rows, K, 128, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
     return BONSAI_CUDA_BAD_ARG;
-  PfParams p{nullptr, nullptr, out_f32, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, 1, limit, alpha, offset, 0, nullptr, nullptr};
+  PfParams p{nullptr, nullptr, out_f32, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, 1, limit, alpha, offset, nullptr, nullptr, 0, 0, nullptr, nullptr};
   return tok == 64 ? launch_prefill<64>(xmap, amap, p, sms, ws, ws_bytes, 1, stream)
                    : launch_prefill<256>(xmap, amap, p, sms, ws, ws_bytes, 1, stream);
+}
+
+// Grouped dense bf16 product: W [groups][n_rows][K] (K a multiple of 128), x [T][x_ld] whose rows offsets[g] .. offsets[g + 1] - 1
+// (device memory, ascending, at most T) belong to group g.  epi 4: out_bf16 = clamped gated unit over interleaved gate / up rows times
+// row_scale[row]; 6: out_bf16 = W x.  wide: tiles of 256 rows of x instead of 64.
+int bonsai_grouped_gemm_bf16(const void* w, int groups, int n_rows, int K, const void* x, int x_ld, int T, const int* offsets, const float* row_scale,
+                             void* out_bf16, int out_ld, int epi, float limit, float alpha, float offset, int wide, int* status, int sms, cudaStream_t stream) {
+  using namespace bonsai;
+  if (groups < 1 || groups > kPfMaxGroups || K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 4 && epi != 6))
+    return BONSAI_CUDA_BAD_ARG;
+  if (out_bf16 == nullptr || offsets == nullptr || status == nullptr || (epi == 4 && (n_rows % 2 != 0 || row_scale == nullptr))) return BONSAI_CUDA_BAD_ARG;
+  if ((long long)groups * n_rows >= (1ll << 31) || ((long long)groups + T / 64) * ((n_rows + 127) / 128) * (K >> 7) >= (1ll << 31)) return BONSAI_CUDA_BAD_ARG;
+  CUtensorMap xmap, amap;
+  if (!make_map_f16(&xmap, x, K, T, x_ld, wide ? 256 : 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
+      !make_map_f16(&amap, w, K, (uint64_t)groups * n_rows, K, 128, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
+    return BONSAI_CUDA_BAD_ARG;
+  const PfParams p{nullptr, nullptr, nullptr, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, 1, limit, alpha, offset, row_scale, offsets,
+                   groups, 0, nullptr, nullptr};
+  const int grid = sms > kPfMaxCtas ? kPfMaxCtas : (sms < 1 ? 1 : sms);
+  const size_t smem = 1024 + (wide ? 4 * (size_t)(kPfABytes + 256 * 128) : 8 * (size_t)(kPfABytes + 64 * 128));
+  const auto kernel = wide ? bitgemm_prefill_kernel<256, true> : bitgemm_prefill_kernel<64, true>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return BONSAI_CUDA_LAUNCH_FAILED;
+  const cudaError_t e = launch_pdl(kernel, dim3(grid), dim3(kPfThreads), smem, stream, xmap, amap, p);
+  return e == cudaSuccess ? BONSAI_CUDA_OK : BONSAI_CUDA_LAUNCH_FAILED;
 }
 
 int bonsai_bitgemm_prefill(const void* codes, const void* scales, const void* x_f16, int x_ld, float* out_f32,

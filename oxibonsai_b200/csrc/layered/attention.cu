@@ -1,16 +1,17 @@
-// Attention of the layer-list decoders over a paged cache.  Queries and keys are divided by their root mean square; everything
-// else is a parameter that a design may leave out:
+// Attention of the layer-list decoders over a paged cache.  Every part is a parameter that a design may leave out:
 //
 //   score(i, j) = cap(q'_i . k'_j) - slope_h (i - j)       j <= i and (i - j < window or j < keep)
-//   out         = softmax(score) V * sigmoid(gate_h) * out_scale
+//   out         = softmax(score) V * sigmoid(gate_h) * out_scale       [denominator + e^(sink_h)]
 //
-// with q' = norm(q) [* w_q * w_k] * scale [* (1 + coef ln(floor((i + 1) / every) + 1))] and cap(s) = s or c tanh(s / c).
+// with q' = rot(norm(q)) [* w_q * w_k] * scale [* (1 + coef ln(floor((i + 1) / every) + 1))], k' = rot(norm(k)) and
+// cap(s) = s or c tanh(s / c); norm divides by the root mean square, rot turns pairs of dimensions by angles of the position.
 //
 // Two kinds of cache rows (template parameter SEP):
 //  * one row per token that is both key and value (designs whose values are the un-normalised keys): the row holds the projected
 //    key, a float beside it the reciprocal root mean square, which multiplies the scores of its column.  Half the cache traffic
 //    of separate rows, and a tile is staged once for S = Q K^T and O = P K;
-//  * SEP: a row of normalised keys and a row of values, both padded to the same row length.  Scores are capped only here.
+//  * SEP: a row of finished keys and a row of values, both padded to the same row length.  Scores are capped, heads rotated and rows
+//    of another layer used (k_col < 0: nothing is appended) only here.
 //
 // Rows of a batch are tokens: a row has a position and a slot (its sequence's block-table row).  `append_kernel` writes the
 // rows' keys; `prompt_kernel` handles portions of prompts (tiles of 64 query rows = tokens x heads of one kv group);
@@ -28,6 +29,8 @@ struct Attn {
   const float* q_norm;      // [dim]; null: no norm weights
   const float* k_norm;      // [dim]
   const float* slopes;      // [heads]; null: no distance bias
+  const float* sinks;       // [heads]; null: no sink
+  const float2* rot;        // [positions][rot_dims / 2] cosines and sines; null: no rotation
   const int* pos;           // [T]
   const int* slots;         // [T]
   const int* block_table;   // [slots][max_pages]
@@ -35,9 +38,11 @@ struct Attn {
   float* krms;              // [pages][kv_heads][page_size]; SEP: unused
   void* vpool;              // SEP: value rows, laid out like the pool
   void* out;                // [T][ldo], head h at h * vdim
-  int ld, q_col, k_col, v_col, g_col, ldo;       // g_col < 0: no gate
+  int ld, q_col, k_col, v_col, g_col, ldo;       // g_col < 0: no gate; k_col < 0: another layer appends the rows
   int heads, kv_heads, dim, vdim, max_pages, pshift;   // page size 1 << pshift
   int window, keep;         // window <= 0: no window
+  int normed;               // queries and keys are divided by their root mean square
+  int rot_dims, rot_pairs;  // rotated dimensions; pairs (2i, 2i + 1) instead of (i, i + rot_dims / 2)
   float eps, scale, out_scale;
   float softcap;            // <= 0: scores are not capped
   float temp_coef, temp_every;   // query temperature; coef 0: none
@@ -49,6 +54,7 @@ __device__ __forceinline__ float temperature(const Attn& a, int pos) {
 __device__ __forceinline__ float gate(const Attn& a, size_t t, int head) {
   return a.g_col < 0 ? a.out_scale : a.out_scale * sigmoid(a.proj[t * a.ld + a.g_col + head]);
 }
+__device__ __forceinline__ const float2* angles(const Attn& a, int pos) { return a.rot == nullptr ? nullptr : a.rot + (size_t)pos * (a.rot_dims >> 1); }
 // Scores arrive as base-2 logarithms, or with a cap as x = 2 log2(e) score / cap: cap * tanh(score / cap) * log2(e) from one
 // exponential, tanh(y) = 1 - 2 / (e^2y + 1).
 __device__ __forceinline__ float cap_score(float x, float cap_log2e) { return cap_log2e - __fdividef(2.0f * cap_log2e, ex2(x) + 1.0f); }
@@ -62,21 +68,22 @@ __device__ __forceinline__ size_t cache_row(const Attn& a, const int* bt, int kv
 
 // A warp writes one token's row of kv head kvh: the key and its reciprocal root mean square, or the normalised key and the value.
 template <int HD, bool SEP, typename C>
-__device__ __forceinline__ void append_row(const Attn& a, const float* proj, int kvh, size_t row, int lane) {
+__device__ __forceinline__ void append_row(const Attn& a, const float* proj, int kvh, int pos, size_t row, int lane) {
   C* dst = static_cast<C*>(a.pool) + row * HD;
   const float* k = proj + a.k_col + kvh * a.dim;
   if constexpr (SEP) {
     const float* v = proj + a.v_col + kvh * a.vdim;
     C* vdst = static_cast<C*>(a.vpool) + row * HD;
+    const float2* rot = angles(a, pos);
     float x[HD / 32], ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < HD / 32; ++i) {
       const int d = lane + 32 * i;
-      x[i] = d < a.dim ? k[d] : 0.0f;
+      x[i] = d < a.dim ? rotated(k, d, rot, a.rot_dims, a.rot_pairs) : 0.0f;      // keeps the sum of squares
       store_act(vdst + d, d < a.vdim ? v[d] : 0.0f);
       ss += x[i] * x[i];
     }
-    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    const float inv = a.normed ? 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps) : 1.0f;
 #pragma unroll
     for (int i = 0; i < HD / 32; ++i) store_act(dst + lane + 32 * i, x[i] * inv);
     return;
@@ -102,23 +109,24 @@ __global__ void append_kernel(Attn a, int first, int count) {
   const int t = first + i;
   if (a.pos[t] >= (a.max_pages << a.pshift)) return;
   const int* bt = a.block_table + (size_t)a.slots[t] * a.max_pages;
-  append_row<HD, SEP, C>(a, a.proj + (size_t)t * a.ld, kvh, cache_row(a, bt, kvh, a.pos[t]), lane);
+  append_row<HD, SEP, C>(a, a.proj + (size_t)t * a.ld, kvh, a.pos[t], cache_row(a, bt, kvh, a.pos[t]), lane);
 }
 
 // A warp normalises one query head and leaves q' * log2(e) in dst (columns past dim zero): scores are base-2 logarithms; with
 // a cap, q' * 2 log2(e) / cap.
 template <int HD>
 __device__ __forceinline__ void load_query(const Attn& a, const float* q, int pos, bf16* dst, int lane) {
+  const float2* rot = angles(a, pos);
   float v[HD / 32], ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < HD / 32; ++i) {
     const int d = lane + 32 * i;
-    v[i] = d < a.dim ? q[d] : 0.0f;
+    v[i] = d < a.dim ? rotated(q, d, rot, a.rot_dims, a.rot_pairs) : 0.0f;
     ss += v[i] * v[i];
     if (a.q_norm != nullptr && d < a.dim) v[i] *= a.q_norm[d] * a.k_norm[d];
   }
   ss = warp_sum(ss);
-  const float f = a.scale * temperature(a, pos) * (a.softcap > 0.0f ? 2.0f * kLog2e / a.softcap : kLog2e) / sqrtf(ss / (float)a.dim + a.eps);
+  const float f = a.scale * temperature(a, pos) * (a.softcap > 0.0f ? 2.0f * kLog2e / a.softcap : kLog2e) / (a.normed ? sqrtf(ss / (float)a.dim + a.eps) : 1.0f);
 #pragma unroll
   for (int i = 0; i < HD / 32; ++i) dst[lane + 32 * i] = __float2bfloat16_rn(v[i] * f);
 }
@@ -285,7 +293,13 @@ __global__ void __launch_bounds__(128) prompt_kernel(Attn a, const int4* entries
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
     if (row[r] >= rows) continue;
     const size_t t = en.x + q0 + row[r] / G;
-    const float f = gate(a, t, head[r]) / l[r];   // the query's own position is always visible
+    float f = gate(a, t, head[r]);
+    if (a.sinks == nullptr) {
+      f /= l[r];   // the query's own position is always visible
+    } else {
+      const float sink = a.sinks[head[r]] * kLog2e, top = fmaxf(mx[r], sink), down = ex2(mx[r] - top);
+      f *= down / (l[r] * down + ex2(sink - top));
+    }
     bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + head[r] * a.vdim;
 #pragma unroll
     for (int nt = 0; nt < HD / 8; ++nt) {
@@ -335,7 +349,7 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
   const int ntiles = nkeep + end16 - lo16;
   const int per = (ntiles + nsplit - 1) / nsplit;
   const int b0 = split * per, b1 = min(ntiles, b0 + per);
-  const bool owner = b1 == ntiles && b0 < b1;                            // holds the last tile: the row's own position
+  const bool owner = a.k_col >= 0 && b1 == ntiles && b0 < b1;            // holds the last tile, the row's own position, and appends it
   bf16* wt = tiles + warp * NST * kStage;
   float* wf = reinterpret_cast<float*>(tiles + NW * NST * kStage) + warp * NST * 16;   // key factors of the tiles
   auto first_token = [&](int j) { return (j < nkeep ? j : lo16 + j - nkeep) << 4; };
@@ -363,7 +377,7 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
     else if (r < 16)
       for (int d = lane; d < HD; d += 32) sQ[r * LD + d] = __float2bfloat16_rn(0.0f);
     else {
-      append_row<HD, SEP, bf16>(a, prow, kvh, cache_row(a, bt, kvh, pos), lane);
+      append_row<HD, SEP, bf16>(a, prow, kvh, pos, cache_row(a, bt, kvh, pos), lane);
       __threadfence();
     }
   }
@@ -506,6 +520,11 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
       L += f * src[HD + 1];
     }
     const int h = kvh * G + h0 + r;
+    if (a.sinks != nullptr) {
+      const float sink = a.sinks[h] * kLog2e, top = fmaxf(M, sink), down = ex2(M - top);
+      acc *= down;
+      L = L * down + ex2(sink - top);
+    }
     static_cast<bf16*>(a.out)[(size_t)t * a.ldo + h * a.vdim + d] = __float2bfloat16_rn(acc / L * gate(a, t, h));
   }
   if (nsplit > 1) cluster.sync();   // nobody leaves while its rows are being read
@@ -525,15 +544,16 @@ __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
   const int* bt = a.block_table + (size_t)a.slots[t] * a.max_pages;
   const float* pool = static_cast<const float*>(a.pool);
   const float* qr = a.proj + (size_t)t * a.ld + a.q_col + h * a.dim;
+  const float2* rot = angles(a, pos);
   float q[HD / 32], o[HD / 32], ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < HD / 32; ++i) {
     const int d = lane + 32 * i;
-    q[i] = d < a.dim ? qr[d] : 0.0f;
+    q[i] = d < a.dim ? rotated(qr, d, rot, a.rot_dims, a.rot_pairs) : 0.0f;
     o[i] = 0.0f;
     ss += q[i] * q[i];
   }
-  const float rq = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+  const float rq = a.normed ? 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps) : 1.0f;
 #pragma unroll
   for (int i = 0; i < HD / 32; ++i) {
     const int d = lane + 32 * i;
@@ -570,6 +590,10 @@ __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
   __syncthreads();
   float M = -INFINITY, L = 0.0f;
   for (int w = 0; w < 4; ++w) M = fmaxf(M, sm[w][HD]);
+  if (a.sinks != nullptr) {
+    M = fmaxf(M, a.sinks[h]);
+    L = expf(a.sinks[h] - M);
+  }
   for (int w = 0; w < 4; ++w) L += expf(sm[w][HD] - M) * sm[w][HD + 1];
   const float f = gate(a, t, h) / L;
   for (int d = threadIdx.x; d < a.vdim; d += 128) {
@@ -615,13 +639,15 @@ static int padded_dim(int dim) {
 static bool fill(Attn& a, const void* const* ptrs, const int* ints, const float* floats) {
   a.proj = (const float*)ptrs[0]; a.q_norm = (const float*)ptrs[1]; a.k_norm = (const float*)ptrs[2]; a.slopes = (const float*)ptrs[3];
   a.pos = (const int*)ptrs[4]; a.slots = (const int*)ptrs[5]; a.block_table = (const int*)ptrs[6]; a.pool = const_cast<void*>(ptrs[7]);
-  a.krms = (float*)ptrs[8]; a.vpool = const_cast<void*>(ptrs[9]); a.out = const_cast<void*>(ptrs[10]);
+  a.krms = (float*)ptrs[8]; a.vpool = const_cast<void*>(ptrs[9]); a.out = const_cast<void*>(ptrs[10]); a.sinks = (const float*)ptrs[11];
+  a.rot = (const float2*)ptrs[12];
   a.ld = ints[0]; a.q_col = ints[1]; a.k_col = ints[2]; a.v_col = ints[3]; a.g_col = ints[4]; a.ldo = ints[5]; a.heads = ints[6];
   a.kv_heads = ints[7]; a.dim = ints[8]; a.vdim = ints[9]; a.max_pages = ints[10];
   for (a.pshift = 0; (2 << a.pshift) <= ints[11]; ++a.pshift) {}
-  a.window = ints[12]; a.keep = ints[13];
+  a.window = ints[12]; a.keep = ints[13]; a.normed = ints[14]; a.rot_dims = a.rot == nullptr ? 0 : ints[15]; a.rot_pairs = ints[16];
   a.eps = floats[0]; a.scale = floats[1]; a.out_scale = floats[2]; a.softcap = floats[3]; a.temp_coef = floats[4]; a.temp_every = floats[5];
-  if (a.vpool == nullptr ? a.krms == nullptr || a.vdim != a.dim || a.softcap > 0.0f : a.vdim < 1) return false;
+  if (a.vpool == nullptr ? a.krms == nullptr || a.vdim != a.dim || a.softcap > 0.0f || a.rot != nullptr || !a.normed || a.k_col < 0 : a.vdim < 1) return false;
+  if (a.rot != nullptr && (a.rot_dims < 2 || a.rot_dims % 2 != 0 || a.rot_dims > a.dim || a.q_norm != nullptr)) return false;
   return a.heads >= 1 && a.kv_heads >= 1 && a.heads % a.kv_heads == 0 && a.heads / a.kv_heads <= 64 && a.dim >= 1 &&
          padded_dim(a.dim > a.vdim ? a.dim : a.vdim) > 0 && a.pshift >= 4 && (1 << a.pshift) == ints[11] && a.keep >= 0 &&
          (a.temp_coef == 0.0f || a.temp_every > 0.0f) && (a.q_norm == nullptr) == (a.k_norm == nullptr);
@@ -651,15 +677,15 @@ extern "C" {
 // elements of a cache row for a head size (0: not supported)
 int bonsai_lay_attn_row(int dim) { return dim < 1 ? 0 : bonsai::lay::padded_dim(dim); }
 
-// Arguments of all launches: ptrs = {proj, q_norm, k_norm, slopes, pos, slots, block_table, pool, krms, vpool, out} (null where
-// a design has none; vpool null: rows are key and value), ints = {ld, q_col, k_col, v_col, g_col, ldo, heads, kv_heads, dim,
-// vdim, max_pages, page_size, window, keep}, floats = {eps, scale, out_scale, softcap, temp_coef, temp_every}.
+// Arguments of all launches: ptrs = {proj, q_norm, k_norm, slopes, pos, slots, block_table, pool, krms, vpool, out, sinks, rot} (null
+// where a design has none; vpool null: rows are key and value; rot has a row for every position the pages hold), ints = {ld,
+// q_col, k_col, v_col, g_col, ldo, heads, kv_heads, dim, vdim, max_pages, page_size, window, keep, normed, rot_dims, rot_pairs}, floats = {eps, scale, out_scale, softcap, temp_coef, temp_every}.
 
 // Writes the keys of rows first .. first + count - 1.
 int bonsai_lay_attn_append(const void* const* ptrs, const int* ints, const float* floats, int first, int count, int f32, cudaStream_t stream) {
   using namespace bonsai::lay;
   Attn a;
-  if (!fill(a, ptrs, ints, floats) || count < 1 || first < 0) return BONSAI_CUDA_BAD_ARG;
+  if (!fill(a, ptrs, ints, floats) || count < 1 || first < 0 || a.k_col < 0) return BONSAI_CUDA_BAD_ARG;
   BONSAI_BY_DIM((run_append<HD, SEP>(a, first, count, f32, stream)))
 }
 

@@ -77,6 +77,17 @@ __device__ __forceinline__ void store_act(float* p, float v) { *p = v; }
 __device__ __forceinline__ float load_act(const bf16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ float load_act(const float* p) { return *p; }
 
+// Element d of a head whose first `dims` dimensions are turned by the angles of `rot` (cosine, sine per pair; null: no rotation);
+// pairs are (2i, 2i + 1), or (i, i + dims / 2).
+__device__ __forceinline__ float rotated(const float* v, int d, const float2* rot, int dims, int pairs) {
+  if (d >= dims || rot == nullptr) return v[d];
+  const int half = dims >> 1;
+  const bool first = pairs ? (d & 1) == 0 : d < half;
+  const float2 cs = rot[pairs ? d >> 1 : (first ? d : d - half)];
+  const float other = v[pairs ? d ^ 1 : (first ? d + half : d - half)];
+  return first ? v[d] * cs.x - other * cs.y : v[d] * cs.x + other * cs.y;
+}
+
 constexpr float kLog2e = 1.4426950408889634f;
 
 // chunked recurrences: tokens per chunk, value columns per CTA, row length of a staged value tile
@@ -90,7 +101,7 @@ enum ChunkMode { kWhole, kLocal, kResume };
 // dimension `dim` (0 = x, 1 = y) of the grid.
 template <typename Kern, typename... Args>
 static inline int launch(Kern kernel, dim3 grid, int threads, size_t smem, cudaStream_t stream, int cluster, int dim, Args... args) {
-  if (smem > 48 * 1024 &&
+  if (smem > 24 * 1024 &&     // 48 KB with the static part
       cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     return BONSAI_CUDA_LAUNCH_FAILED;
   cudaLaunchConfig_t cfg = {};

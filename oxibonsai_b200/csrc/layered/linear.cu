@@ -11,7 +11,7 @@
 //
 // Epilogues: 0 = f32 store, 1 = clamped gated unit over interleaved gate / up rows:
 //   g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(alpha g) * (u + up_offset);
-// 2 = squared relu.
+// 2 = squared relu, 3 = the product itself in the activations' type.
 #include "layered/layered.cuh"
 
 namespace bonsai {
@@ -90,7 +90,7 @@ __global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __res
       for (int w = 0; w < kWarps; ++w) v += red[w][r][t];
       if (row0 + r >= n) continue;
       if (epi == 0) out[(size_t)t * ldo + row0 + r] = v;
-      else out16[(size_t)t * ldo + row0 + r] = __float2bfloat16_rn(squared_relu(v));
+      else out16[(size_t)t * ldo + row0 + r] = __float2bfloat16_rn(epi == 2 ? squared_relu(v) : v);
     }
   } else {
     for (int i = threadIdx.x; i < 8 * T; i += kWarps * 32) {
@@ -147,7 +147,7 @@ __global__ void __launch_bounds__(256) f32_kernel(const bf16* __restrict__ W, in
     for (int j = 0; j < 4; ++j) {
       const int r = n0 + tn * 4 + j;
       if (epi != 1) {
-        if (r < n) out[(size_t)t * ldo + r] = epi == 0 ? acc[i][j] : squared_relu(acc[i][j]);
+        if (r < n) out[(size_t)t * ldo + r] = epi == 2 ? squared_relu(acc[i][j]) : acc[i][j];
       } else if ((j & 1) == 0 && r + 1 < n) {
         out[(size_t)t * ldo + (r >> 1)] = glu(act, acc[i][j], acc[i][j + 1]);
       }
@@ -161,11 +161,11 @@ __global__ void __launch_bounds__(256) f32_kernel(const bf16* __restrict__ W, in
 extern "C" {
 
 // W bf16 [n][kp] (kp a multiple of 128, columns past the layer's width zero), x bf16 [T][ldx] (ldx >= kp, finite in the
-// padding), T <= 32.  epi 0: out f32 [T][ldo]; epi 1: out16 bf16 [T][ldo] of n / 2 columns; epi 2: out16 bf16 [T][ldo].
+// padding), T <= 32.  epi 0: out f32 [T][ldo]; epi 1: out16 bf16 [T][ldo] of n / 2 columns; epi 2 and 3: out16 bf16 [T][ldo].
 int bonsai_lay_linear_few(const void* W, int n, int kp, const void* x, int ldx, int T, float* out, void* out16, int ldo, int epi, float limit,
                           float alpha, float up_offset, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || T < 1 || T > 32 || epi < 0 || epi > 2) return BONSAI_CUDA_BAD_ARG;
+  if (n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || T < 1 || T > 32 || epi < 0 || epi > 3) return BONSAI_CUDA_BAD_ARG;
   if ((epi == 0 && out == nullptr) || (epi != 0 && out16 == nullptr) || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
   const Glu act{limit, alpha, up_offset};
   const dim3 grid((n + 15) / 16);
@@ -178,7 +178,7 @@ int bonsai_lay_linear_few(const void* W, int n, int kp, const void* x, int ldx, 
 int bonsai_lay_linear_f32(const void* W, int n, int k, int kp, const float* x, int ldx, int T, float* out, int ldo, int epi, float limit, float alpha,
                           float up_offset, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (n < 1 || k < 1 || kp < k || ldx < k || T < 1 || out == nullptr || epi < 0 || epi > 2 || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
+  if (n < 1 || k < 1 || kp < k || ldx < k || T < 1 || out == nullptr || epi < 0 || epi > 3 || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
   return launch(f32_kernel, dim3((n + 63) / 64, (T + 63) / 64), 256, 0, stream, 1, 0, (const bf16*)W, n, k, kp, x, ldx, T, out, ldo, epi,
                 Glu{limit, alpha, up_offset});
 }

@@ -1,9 +1,10 @@
 """Decoders described layer by layer (``layered_config``): weights, mixers and the step runner.
 
 A step is a batch of rows (tokens).  Rows of single tokens (decode) come first, portions of prompts follow, each portion
-contiguous; every projection runs over all rows, a mixer runs its single-token kernel over the first group and its prompt
-kernel over the second.  Mixers that stand side by side in a layer share one projection and one output projection over their
-joined outputs.  A row carries its position and its slot; the slot's block-table row names the pages of its sequence
+contiguous, short ones first; every projection runs over all rows, a mixer runs its single-token kernel over the first group and
+its prompt kernel over the second (latent attention takes short portions for single tokens).  Mixers that stand side by side in a
+layer share one projection and one output projection over their joined outputs; a feed-forward block beside the mixer shares the
+projection too.  A row carries its position and its slot; the slot's block-table row names the pages of its sequence
 and the state table its recurrent state row, so which pages, rows and companions a token has does not enter its arithmetic.
 
 Two modes: bf16 (tensor-core projections and attention, f32 residual stream, norms, scores, gates and recurrent state) and
@@ -12,7 +13,7 @@ eagerly with the same kernels.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from pathlib import Path
 from typing import Sequence
 
@@ -22,7 +23,8 @@ import torch
 from ..ops import cuda_ops as K
 from ..ops import layered_ops as L
 from ..ops import nvtx
-from .layered_config import AttentionSpec, Branch, GatedMlpSpec, LayeredConfig, LinearRecurrenceSpec, MlstmSpec, SquaredReluMlpSpec
+from .layered_config import (AttentionSpec, Branch, ExpertsSpec, GatedMlpSpec, LatentAttentionSpec, LayeredConfig, LinearRecurrenceSpec, MlstmSpec,
+                             RotarySpec, SquaredReluMlpSpec)
 from .paged import RowCache, StatePool
 from .rope_scaling import geometric_slopes
 from .slot_state import SlotState
@@ -45,20 +47,51 @@ class MlpWeights:
 
 
 @dataclass
+class ExpertWeights:
+    column: int                      # first router logit in the layer's projection
+    correction: torch.Tensor
+    up: L.DenseWeight                # all experts' gate and up rows, interleaved, one expert below the other
+    down: L.DenseWeight
+
+
+@dataclass
+class LatentWeights:
+    """The expansions of a latent in the forms the kernels read (sizes padded with zeros)."""
+    keys: torch.Tensor               # [heads, rank to 16, dim to 32]
+    values: torch.Tensor             # [heads, vdim, rank to 32]
+    expand: L.DenseWeight            # per head dim to 8 key rows, vdim to 8 value rows
+
+    @classmethod
+    def load(cls, m: LatentAttentionSpec, uk: torch.Tensor, uv: torch.Tensor, device) -> "LatentWeights":
+        H, R, up = m.heads, m.rank, L.round_up
+        uk, uv = uk.view(H, m.dim, R), uv.view(H, m.vdim, R)
+        pad = torch.nn.functional.pad
+        keys = pad(uk.transpose(1, 2), (0, up(m.dim, 32) - m.dim, 0, up(R, 16) - R))
+        both = torch.cat([pad(uk, (0, 0, 0, up(m.dim, 8) - m.dim)), pad(uv, (0, 0, 0, up(m.vdim, 8) - m.vdim))], dim=1)
+        return cls(keys.contiguous().to(device), pad(uv, (0, up(R, 32) - R)).contiguous().to(device), L.DenseWeight([both.reshape(-1, R)], device))
+
+    @property
+    def nbytes(self) -> int:
+        """Bytes a decode step must stream."""
+        return 2 * (self.keys.numel() + self.values.numel())
+
+
+@dataclass
 class BranchWeights:
     columns: list[int]               # first output of each section in the layer's projection
     vectors: dict[str, torch.Tensor]
     offset: int                      # first column in the input of the output projection
+    latent: LatentWeights | None = None
 
 
 @dataclass
 class LayerWeights:
     pre_norm: torch.Tensor | None
-    norm: torch.Tensor
+    norm: torch.Tensor | None
     proj: L.DenseWeight              # every projection that reads the mixers' input, one matrix
     out: L.DenseWeight               # the branches' output projections side by side
     branches: list[BranchWeights]
-    mlp: MlpWeights | None
+    mlp: MlpWeights | ExpertWeights | None
 
 
 def branch_offsets(widths: Sequence[int]) -> tuple[list[int], int]:
@@ -96,6 +129,8 @@ class LayeredWeights:
                     parts.append(m(f"l{i}.mix.{b.prefix}{name}")[at:at + rows])
                     first[name] = at + rows
                 counts.append(len(b.spec.sections))
+            if isinstance(spec.mlp, ExpertsSpec):
+                parts.append(m(p + "router"))
             proj = L.DenseWeight(parts, self.device)
             offsets, width = branch_offsets([b.spec.out_width for b in spec.mixer.branches])
             out = torch.zeros((cfg.width, width), dtype=torch.bfloat16)
@@ -103,10 +138,16 @@ class LayeredWeights:
             for b, off, count in zip(spec.mixer.branches, offsets, counts):
                 x = f"l{i}.mix.{b.prefix}"
                 out[:, off:off + b.spec.out_width] = m(x + "o")
-                branches.append(BranchWeights(proj.columns[at:at + count], {n: v(x + n) for n in b.spec.vectors}, off))
+                latent = LatentWeights.load(b.spec, m(x + "uk"), m(x + "uv"), self.device) if isinstance(b.spec, LatentAttentionSpec) else None
+                branches.append(BranchWeights(proj.columns[at:at + count], {n: v(x + n) for n in b.spec.vectors}, off, latent))
                 at += count
             mlp = None
-            if isinstance(spec.mlp, GatedMlpSpec):
+            assert cfg.side_by_side == isinstance(spec.mlp, ExpertsSpec) or spec.mlp is None, "experts stand beside the mixer, dense blocks behind it"
+            if isinstance(spec.mlp, ExpertsSpec):
+                names = [f"{p}e{e}." for e in range(spec.mlp.router.experts)]
+                up = L.DenseWeight([torch.cat([m(n + c) for n in names]) for c in ("gate", "up")], self.device, interleave=True)
+                mlp = ExpertWeights(proj.columns[at], v(p + "correction"), up, L.DenseWeight([torch.cat([m(n + "down") for n in names])], self.device))
+            elif isinstance(spec.mlp, GatedMlpSpec):
                 up = L.DenseWeight([m(p + "gate"), m(p + "up")], self.device, interleave=True)
                 mlp = MlpWeights(*map(v, norms[1]), up, L.DenseWeight([m(p + "down")], self.device), L.Glu(spec.mlp.limit, spec.mlp.alpha, spec.mlp.offset))
             elif isinstance(spec.mlp, SquaredReluMlpSpec):
@@ -123,14 +164,22 @@ class LayeredWeights:
     def packed_bytes(self) -> int:
         """Bytes a decode step must stream."""
         n = self.embed.nbytes
-        for l in self.layers:
-            n += l.proj.nbytes + l.out.nbytes + (0 if l.mlp is None else l.mlp.up.nbytes + l.mlp.down.nbytes)
+        for spec, l in zip(self.cfg.layer_specs, self.layers):
+            mlp = 0 if l.mlp is None else l.mlp.up.nbytes + l.mlp.down.nbytes
+            if isinstance(spec.mlp, ExpertsSpec):                # of one token
+                mlp = mlp * spec.mlp.router.top // spec.mlp.router.experts
+            n += l.proj.nbytes + l.out.nbytes + mlp + sum(b.latent.nbytes for b in l.branches if b.latent is not None)
         return n
 
 
 def new_row_cache(cfg: LayeredConfig, num_pages: int, page_size: int, exact: bool, device) -> RowCache:
-    specs = {i: cfg.attention(i) for i in cfg.attention_layers}
-    layers = {i: (s.kv_heads, L.lib().bonsai_lay_attn_row(max(s.dim, s.value_dim)), s.vdim is not None) for i, s in specs.items()}
+    layers = {}
+    for i in cfg.attention_layers:
+        s = cfg.attention(i)
+        if isinstance(s, LatentAttentionSpec):
+            layers[i] = (1, L.lib().bonsai_lay_latent_row(s.rank, s.rot_dim), "latent")
+        elif s.kv_from is None:
+            layers[i] = (s.kv_heads, L.lib().bonsai_lay_attn_row(max(s.dim, s.value_dim)), "shared" if s.vdim is None else "separate")
     return RowCache(layers, num_pages, page_size, K.KV_F32 if exact else K.KV_BF16, torch.float32 if exact else torch.bfloat16, device)
 
 
@@ -171,18 +220,52 @@ class Rows:
 @dataclass
 class StepShape:
     """How a step's rows split: ``singles`` single-token rows, then ``portions`` (device address of the int4 list and of the
-    query tiles per tokens-per-tile)."""
+    query tiles per tokens-per-tile).  ``short``: the rows up to the first portion of more than ``SHORT`` tokens."""
     rows: int
     singles: int
+    short: int
     portions: int = 0
     entries: int = 0
     tiles: dict[int, tuple[int, int]] | None = None      # tokens per tile -> (device address, tiles)
     segments: dict["SegmentPlan", tuple[int, int, int]] | None = None    # recurrences that cut the portions: segments, device addresses of the two lists
+    contexts: list["ContextGroup"] = field(default_factory=list)
 
     def cut(self, plan: "SegmentPlan | None") -> tuple[int, int, int]:
         """Segment list, segments (0: portions as a whole) and prompt list of a recurrence."""
         n, segs, prompts = (self.segments or {}).get(plan, (0, 0, 0))
         return segs, n, prompts
+
+
+SHORT = 32                  # tokens of a portion whose rows latent attention treats as single tokens
+SHORT_ROWS = 256            # such rows in a step, at least
+CONTEXT_TILE = 128          # query tokens per tile over expanded keys
+
+
+@dataclass
+class ContextGroup:
+    """Long portions whose cached latents are expanded together: device addresses of the portions, of {first scratch row, cached
+    tokens, slot, 0} for each, and of the query tiles."""
+    portions: int
+    contexts: int
+    count: int
+    tiles: int
+    n_tiles: int
+    rows: int                   # scratch rows in all
+    longest: int
+
+
+def group_contexts(lists: Sequence[tuple[int, int, int, int]], limit: int) -> list[list[tuple[int, int, int, int]]]:
+    """Cuts portions (first row, tokens, slot, first position) into runs whose cached tokens together stay within ``limit`` rows."""
+    groups: list[list[tuple[int, int, int, int]]] = []
+    rows = 0
+    for e in lists:
+        n = e[1] + e[3]
+        if not groups or rows + n > limit:
+            groups.append([])
+            rows = 0
+        groups[-1].append(e)
+        rows += n
+    return groups
 
 
 MAX_SEGMENTS = 24           # segment states the scratch of the recurrent layers holds
@@ -247,12 +330,16 @@ class AttentionMixer:
         self.r, self.spec, self.out = r, branch.spec, out
         spec, cols = self.spec, dict(zip((n for n, _ in branch.spec.sections), w.columns))
         self.tile = 64 // spec.group
+        source = index if spec.kv_from is None else spec.kv_from          # the layer whose rows are used
+        self.appends, rot = spec.kv_from is None, spec.rotary
         slopes = None if spec.slope_exponent is None else geometric_slopes(spec.heads, spec.slope_exponent).to(r.device)
-        ints = [r.proj.stride(0), cols["q"], cols["k"], cols.get("v", 0), cols.get("g", -1), out.stride(0), spec.heads, spec.kv_heads, spec.dim,
-                spec.value_dim, r.max_pages, r.kv.page_size, spec.window, spec.keep_first]
+        ints = [r.proj.stride(0), cols["q"], cols.get("k", -1), cols.get("v", 0), cols.get("g", -1), out.stride(0), spec.heads, spec.kv_heads, spec.dim,
+                spec.value_dim, r.max_pages, r.kv.page_size, spec.window, spec.keep_first, int(spec.normed), 0 if rot is None else rot.dims,
+                int(rot is not None and rot.interleaved)]
         floats = [r.cfg.eps, spec.scale, branch.scale, spec.softcap, spec.temp_coef, spec.temp_every]
         self.call = {id(rows): L.MixerCall([r.proj, w.vectors.get("q.norm"), w.vectors.get("k.norm"), slopes, rows.positions, rows.slots, r.block_table,
-                                            r.kv.rows[index], r.kv.factors.get(index), r.kv.values.get(index), out], ints, floats)
+                                            r.kv.rows[source], r.kv.factors.get(source), r.kv.values.get(source), out, w.vectors.get("sink"),
+                                            None if rot is None else r.angles(rot)], ints, floats)
                      for rows in (r.slot_rows, r.batch_rows)}
 
     def splits(self, batch: int) -> int:
@@ -267,18 +354,63 @@ class AttentionMixer:
     def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
         lib, a = L.lib(), self.call[id(rows)].args
         if self.r.exact:
-            K.check(lib.bonsai_lay_attn_append(*a, 0, st.rows, 1, stream), "attn_append")
+            if self.appends:
+                K.check(lib.bonsai_lay_attn_append(*a, 0, st.rows, 1, stream), "attn_append")
             K.check(lib.bonsai_lay_attn_f32(*a, st.rows, stream), "attn_f32")
             return
         if st.singles:
             K.check(lib.bonsai_lay_attn_decode(*a, st.singles, self.splits(st.singles), stream), "attn_decode")
         if st.portions:
             tiles, n = st.tiles[self.tile]
-            K.check(lib.bonsai_lay_attn_append(*a, st.singles, st.rows - st.singles, 0, stream), "attn_append")
+            if self.appends:
+                K.check(lib.bonsai_lay_attn_append(*a, st.singles, st.rows - st.singles, 0, stream), "attn_append")
             K.check(lib.bonsai_lay_attn_prompt(*a, st.entries, tiles, n, stream), "attn_prompt")
 
     def launches(self) -> int:
-        return 2 if self.r.exact else 1
+        return 1 + int(self.r.exact and self.appends)
+
+
+class LatentAttentionMixer:
+    """Single tokens and short portions attend to the latents themselves, longer portions to keys and values expanded from them."""
+
+    def __init__(self, r: "LayeredRunner", index: int, branch: Branch, w: BranchWeights, out: torch.Tensor):
+        self.r, self.spec, self.w, s = r, branch.spec, w, branch.spec
+        q, c, rot, g = w.columns
+        row = self.row = r.kv.rows[index].shape[-1]
+        self.groups = -(-s.heads // L.lib().bonsai_lay_latent_group(s.heads))
+        self.lat_ld, self.kv_ld = max(row, w.latent.expand.kp), w.latent.expand.n
+        absorbed, partial, sums = r.latent_scratch(row, self.lat_ld, s.heads, L.round_up(s.rank, 16), self.kv_ld)
+        ints = [r.proj.stride(0), q, c, rot, g, out.stride(0), s.heads, s.dim, s.rot_dim, s.vdim, s.rank, r.max_pages, r.kv.page_size]
+        self.call = {id(rows): L.MixerCall([r.proj, w.vectors["dkv.norm"], r.angles(s.rotary), rows.positions, rows.slots, r.block_table, r.kv.rows[index],
+                                            w.latent.keys, w.latent.values, absorbed, partial, sums, out], ints, [r.cfg.eps, s.scale, branch.scale])
+                     for rows in (r.slot_rows, r.batch_rows)}
+
+    def splits(self, rows: int) -> int:
+        """KV splits of the absorbed form: about a CTA per SM, and at least two tiles of 64 keys each at full length."""
+        return max(1, min(L.lib().bonsai_lay_latent_max_splits(), self.r.scratch.sms // (rows * self.groups), -(-self.r.max_seq // 128)))
+
+    def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
+        lib, a, r = L.lib(), self.call[id(rows)].args, self.r
+        if r.exact:
+            K.check(lib.bonsai_lay_latent_append(*a, 0, st.rows, 1, stream), "latent_append")
+            K.check(lib.bonsai_lay_latent_f32(*a, st.rows, stream), "latent_f32")
+            return
+        if st.short:
+            n = self.splits(st.short)
+            K.check(lib.bonsai_lay_latent_query(*a, st.short, stream), "latent_query")
+            K.check(lib.bonsai_lay_latent_decode(*a, st.short, n, stream), "latent_decode")
+            K.check(lib.bonsai_lay_latent_value(*a, st.short, n, stream), "latent_value")
+        if st.rows > st.short:
+            K.check(lib.bonsai_lay_latent_append(*a, st.short, st.rows - st.short, 0, stream), "latent_append")
+        for g in st.contexts:
+            lat, kv = r.latents[self.row, self.lat_ld], r.expanded[: r.context_rows * self.kv_ld].view(-1, self.kv_ld)
+            K.check(lib.bonsai_lay_latent_gather(*a, g.contexts, g.count, g.longest, lat.data_ptr(), self.lat_ld, stream), "latent_gather")
+            L.linear(self.w.latent.expand, lat, g.rows, kv, r.scratch)
+            K.check(lib.bonsai_lay_latent_prompt(*a, g.portions, g.contexts, g.tiles, g.n_tiles, kv.data_ptr(), self.kv_ld, lat.data_ptr(), self.lat_ld, stream),
+                    "latent_prompt")
+
+    def launches(self) -> int:
+        return 2 if self.r.exact else 3
 
 
 class MlstmMixer:
@@ -384,7 +516,7 @@ class LinearRecurrenceMixer:
         return 1 if self.fused else 2
 
 
-MIXERS = {"attention": AttentionMixer, "mlstm": MlstmMixer, "recurrence": LinearRecurrenceMixer}
+MIXERS = {"attention": AttentionMixer, "latent": LatentAttentionMixer, "mlstm": MlstmMixer, "recurrence": LinearRecurrenceMixer}
 
 
 class LayeredRunner(SlotState):
@@ -414,7 +546,7 @@ class LayeredRunner(SlotState):
         self._acts: dict[int, torch.Tensor] = {}
         self.x = torch.zeros((cap, cfg.width), **f32)
         # input of the next projection; without a norm in between, that of the exact mode is the stream itself
-        self.h = self.x if exact and not cfg.pre_norm else self.act_buffer(cfg.width, shared=False)
+        self.h = self.x if exact and not (cfg.pre_norm or cfg.side_by_side) else self.act_buffer(cfg.width, shared=False)
         self.normed = self.act_buffer(cfg.width, shared=False)
         self.y = torch.zeros((cap, L.round_up(cfg.width, 4)), **f32)
         self.proj = torch.zeros((cap, max(L.round_up(l.proj.n, 4) for l in weights.layers)), **f32)
@@ -431,10 +563,19 @@ class LayeredRunner(SlotState):
         segs = MAX_SEGMENTS if shapes else 0
         self.segment_scratch = [torch.empty(max(1, segs * max((f(*s) for s in shapes), default=0)), **f32) for f in
                                 (lambda h, d, e: h * d * e, lambda h, d, e: h * d * e // 64, lambda h, d, e: h * e // 64, lambda h, d, e: h * e // 32)]
+        # tables of rotations and the scratch of latent attention, filled by the mixers that need them
+        self._angles: dict[RotarySpec, torch.Tensor] = {}
+        self.short_rows = max(SHORT_ROWS, max_batch)
+        self.context_rows = max(cap, L.round_up(max_seq, kv.page_size))
+        self.latents: dict[tuple[int, int], torch.Tensor] = {}
+        self.expanded = torch.empty(0, dtype=torch.bfloat16, device=dev)
+        self._absorbed: dict[tuple, list[torch.Tensor]] = {}
         # row metadata: decode steps use the slot tensors as they are; a mixed batch uploads [tokens | positions | slots | lists]
         self.slot_rows = Rows(self.tokens, self.positions, torch.arange(max_batch, **i32))
-        self._tile_sizes = sorted({64 // cfg.attention(i).group for i in cfg.attention_layers})
-        self._meta = torch.zeros(3 * cap + 4 * cap + 8 * MAX_SEGMENTS * len(self.segment_plans) + 2 * cap * len(self._tile_sizes) + cap + 16, **i32)
+        attention = [cfg.attention(i) for i in cfg.attention_layers]
+        self._tile_sizes = sorted({64 // s.group for s in attention if isinstance(s, AttentionSpec)})
+        self._expands = not exact and any(isinstance(s, LatentAttentionSpec) for s in attention)
+        self._meta = torch.zeros(3 * cap + 4 * cap + 8 * MAX_SEGMENTS * len(self.segment_plans) + 2 * cap * len(self._tile_sizes) + 2 * cap + 12 * max_batch + 64, **i32)
         self.batch_rows = Rows(*(self._meta[i * cap:(i + 1) * cap] for i in range(3)))
         self._host = [torch.zeros(self._meta.numel(), dtype=torch.int32).pin_memory() for _ in range(2)]
         self._host_free = [torch.cuda.Event() for _ in range(2)]
@@ -445,7 +586,34 @@ class LayeredRunner(SlotState):
             out = self.act_buffer(*widths)
             self.mixer_out.append(out)
             self.mixers.append([MIXERS[b.spec.kind](self, i, b, bw, out[:, bw.offset:]) for b, bw in zip(spec.mixer.branches, w.branches)])
+        specs = [cfg.experts(i) for i in cfg.expert_layers]
+        shared = L.ExpertScratch(cap, cfg.width, specs, exact, dev) if specs else None
+        self.experts = {i: L.Routing(cfg.experts(i), w.mlp.up, w.mlp.down, w.mlp.correction, self.proj, w.mlp.column, shared)
+                        for i, w in enumerate(weights.layers) if i in cfg.expert_layers}
         self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
+
+    def angles(self, rot: RotarySpec) -> torch.Tensor:
+        """Cosines and sines of a rotation at every position the pages can hold, from angles in double precision."""
+        if rot not in self._angles:
+            f64 = dict(dtype=torch.float64, device=self.device)
+            a = torch.outer(torch.arange(self.max_pages * self.kv.page_size, **f64), torch.tensor(rot.frequencies, **f64))
+            self._angles[rot] = torch.stack([a.cos(), a.sin()], dim=-1).float().contiguous()
+        return self._angles[rot]
+
+    def latent_scratch(self, row: int, lat_ld: int, heads: int, rank: int, kv_ld: int) -> list[torch.Tensor]:
+        """Absorbed queries, partial sums and their maxima for rows of one latent attention layer (layers of equal sizes share them);
+        also makes room for its gathered and expanded rows."""
+        bf16, f32 = dict(dtype=torch.bfloat16, device=self.device), dict(dtype=torch.float32, device=self.device)
+        if not self.exact:
+            if (row, lat_ld) not in self.latents:
+                self.latents[row, lat_ld] = torch.zeros((self.context_rows, lat_ld), **bf16)
+            if self.expanded.numel() < self.context_rows * kv_ld:
+                self.expanded = torch.empty(self.context_rows * kv_ld, **bf16)
+        if (row, heads, rank) not in self._absorbed:
+            rows, parts = (1, 1) if self.exact else (self.short_rows, max(self.short_rows, self.scratch.sms))
+            self._absorbed[row, heads, rank] = [torch.zeros((rows, heads, row), **bf16), torch.empty((parts, heads, rank), **f32),
+                                                torch.empty((parts, heads, 2), **f32)]
+        return self._absorbed[row, heads, rank]
 
     def act_buffer(self, *widths: int, shared: bool = True) -> torch.Tensor:
         """Input buffer of a projection that reads blocks of ``widths`` columns (:func:`branch_offsets`): f32 in the exact mode, else
@@ -485,7 +653,7 @@ class LayeredRunner(SlotState):
         cfg, T, s = self.cfg, st.rows, K.stream()
         x, h, layers = self.x, self.h, self.w.layers
         copy = None if h is x else h
-        L.embed(self.w.embed.data, rows.tokens, cfg.embed_scale, T, cfg.width, x, copy, layers[0].pre_norm, cfg.eps)
+        L.embed(self.w.embed.data, rows.tokens, cfg.embed_scale, T, cfg.width, x, copy, layers[0].pre_norm, cfg.eps, cfg.layer_norm)
         for i, (spec, w) in enumerate(zip(cfg.layer_specs, layers)):
             last = i + 1 == len(layers)
             after, following = (self.normed, self.w.final_norm) if last and final else (copy, None if last else layers[i + 1].pre_norm)
@@ -493,7 +661,12 @@ class LayeredRunner(SlotState):
             for n, mixer in enumerate(self.mixers[i]):
                 mixer(rows, st, s, early=n > 0)            # only the first one follows the projection directly
             L.linear(w.out, self.mixer_out[i], T, self.y, self.scratch)
-            if w.mlp is None:
+            if cfg.side_by_side:
+                experts = self.experts.get(i)
+                if experts is not None:
+                    experts(h, T, self.scratch)
+                L.side_by_side(x, self.y, experts, cfg.residual_mult, T, after, following, cfg.eps, cfg.layer_norm)
+            elif w.mlp is None:
                 L.norm_add(x, self.y, w.norm, cfg.eps, T, after, following)
             else:
                 L.norm_add(x, self.y, w.norm, cfg.eps, T, copy, w.mlp.pre_norm)
@@ -504,12 +677,12 @@ class LayeredRunner(SlotState):
 
     def _head(self, row_list: int, count: int, out: torch.Tensor) -> None:
         """Logits of ``count`` rows (device address of their indices) into ``out`` [count, vocab]."""
-        L.norm_rows(self.x, row_list, count, self.w.final_norm, self.cfg.eps, self.normed)
+        L.norm_rows(self.x, row_list, count, self.w.final_norm, self.cfg.eps, self.normed, self.cfg.layer_norm)
         L.linear(self.w.embed, self.normed, count, out, self.scratch)
 
     def step_eager(self, batch: int, sample: bool = True, lm_head: bool = True, masked: bool = False) -> None:
         """One token for each of the slots 0 .. batch-1 (tokens and positions are read from the slot tensors)."""
-        self._layers(self.slot_rows, StepShape(batch, batch), final=lm_head)
+        self._layers(self.slot_rows, StepShape(batch, batch, batch), final=lm_head)
         if lm_head:
             L.linear(self.w.embed, self.normed, batch, self.logits, self.scratch)
         if sample:
@@ -520,7 +693,7 @@ class LayeredRunner(SlotState):
         key = (batch, sample, masked)
         g = self._graphs.get(key)
         if g is None:
-            for mlp in (s.mlp for s in self.cfg.layer_specs if s.mlp is not None):
+            for mlp in (s.mlp for s in self.cfg.layer_specs if isinstance(s.mlp, (GatedMlpSpec, SquaredReluMlpSpec))):
                 self.act_buffer(mlp.ff)                        # allocated outside the capture
             g = self._graphs[key] = K.capture_graph(self.device, lambda: self.step_eager(batch, sample, masked=masked))
         mark = nvtx.push(f"decode_step[batch={batch}]")
@@ -537,7 +710,8 @@ class LayeredRunner(SlotState):
             raise ValueError(f"a step takes 1 to {self.capacity} tokens, got {T}")
         if len({e[0] for e in entries}) != len(entries):
             raise ValueError("a step takes one entry per slot")
-        order = sorted(range(len(entries)), key=lambda i: (len(entries[i][1]) != 1, i))     # single tokens first
+        sizes = [len(e[1]) for e in entries]
+        order = sorted(range(len(entries)), key=lambda i: (sizes[i] != 1, sizes[i] > SHORT, i))     # single tokens, then short portions
         cap = self.capacity
         turn = self._turn = (self._turn + 1) % 2
         self._host_free[turn].synchronize()                    # the copy that read this buffer has finished
@@ -558,11 +732,15 @@ class LayeredRunner(SlotState):
                 lists.append((row, n, slot, pos0))
             row0[i] = row
             row += n
-        singles = sum(len(e[1]) == 1 for e in entries)
+        singles = short = sum(n == 1 for n in sizes)
+        for _, n, _, _ in lists:
+            if n > SHORT or short + n > self.short_rows:
+                break
+            short += n
         end = -(-3 * cap // 4) * 4
         put = lambda a: (end, end + a.size)
         base = self._meta.data_ptr()
-        st = StepShape(T, singles, len(lists), base + 4 * end, {}, {})
+        st = StepShape(T, singles, short, len(lists), base + 4 * end, {}, {})
         if lists:
             a = np.asarray(lists, dtype=np.int32).reshape(-1)
             lo, hi = put(a)
@@ -583,6 +761,20 @@ class LayeredRunner(SlotState):
                 host[lo:hi] = a
                 st.segments[plan] = (len(segs), base + 4 * lo, base + 4 * (lo + 4 * len(segs)))
                 end = hi
+            groups = group_contexts([e for e in lists if e[0] >= short], self.context_rows) if self._expands else []
+            for g in groups:                                      # blocks of four words, ahead of the lists of two
+                first = np.cumsum([0] + [n + pos0 for _, n, _, pos0 in g])
+                a = np.asarray(g + [(f, n + pos0, slot, 0) for f, (_, n, slot, pos0) in zip(first, g)], dtype=np.int32).reshape(-1)
+                lo, hi = put(a)
+                host[lo:hi] = a
+                at = base + 4 * lo
+                st.contexts.append(ContextGroup(at, at + 16 * len(g), len(g), 0, 0, int(first[-1]), max(n + pos0 for _, n, _, pos0 in g)))
+                end = hi
+            for c, g in zip(st.contexts, groups):
+                a = np.asarray([(e, t) for e, (_, n, _, _) in enumerate(g) for t in range(0, n, CONTEXT_TILE)], dtype=np.int32).reshape(-1)
+                lo, hi = put(a)
+                host[lo:hi] = a
+                c.tiles, c.n_tiles, end = base + 4 * lo, a.size // 2, hi
             for size in self._tile_sizes:
                 a = np.asarray([(e, t) for e, (_, n, _, _) in enumerate(lists) for t in range(0, n, size)], dtype=np.int32).reshape(-1)
                 lo, hi = put(a)
@@ -620,6 +812,7 @@ class LayeredRunner(SlotState):
     def kernel_launches(self, batch: int, sample: bool = True) -> int:
         """Launches of one decode step (each is one of this library's kernels)."""
         n = 2 + int(sample)
-        for spec, mixers in zip(self.cfg.layer_specs, self.mixers):
-            n += 3 + sum(m.launches() for m in mixers) + (3 if spec.mlp is not None else 0)
+        for i, (spec, mixers) in enumerate(zip(self.cfg.layer_specs, self.mixers)):
+            mlp = self.experts[i].launches(batch) if i in self.experts else (3 if spec.mlp is not None else 0)
+            n += 3 + sum(m.launches() for m in mixers) + mlp
         return n

@@ -5,16 +5,25 @@ mixer (a kind of attention, a recurrence, or several side by side) with its size
 are the mechanisms with their constants as fields; a *design* (``models.registry.ARCHITECTURES``) is a function that reads a
 ``config.json`` into a :class:`LayeredConfig` and fixes the constants the file does not carry.
 
-Every mixer spec names its tensors: ``sections`` (the matrices that read the mixer's input, as row ranges), ``vectors``, and the
-output matrix "o" with ``out_width`` inputs.
+Every mixer spec names its tensors: ``sections`` (the matrices that read the mixer's input, as row ranges), ``vectors``, ``inner``
+(matrices that read something else) and the output matrix "o" with ``out_width`` inputs.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
+
+import torch
+
+from .rope_scaling import llama31_frequencies
 
 MAX_HEAD_DIM = 256          # attention head sizes the kernels cover
 MAX_STATE_DIM = 512         # key sizes of a matrix memory
 MAX_GROUP = 64              # query heads per kv head
+MAX_RANK = 512              # latent size of a compressed cache
+MAX_LATENT_ROW = 640        # that and the shared key part, each padded to 16
+MAX_EXPERTS = 512
+MAX_CHOSEN = 32             # experts of a token
 
 
 class LayeredConfigError(ValueError):
@@ -28,18 +37,50 @@ class MixerSpec:
     def branches(self) -> tuple["Branch", ...]:
         return (Branch("", self, 1.0),)
 
+    @property
+    def inner(self) -> dict[str, tuple[int, int]]:
+        return {}
+
 
 @dataclass(frozen=True)
 class Branch:
     """A mixer of a layer: the prefix of its tensors and the factor of its output in the layer's sum."""
     prefix: str
-    spec: "AttentionSpec | MlstmSpec | LinearRecurrenceSpec"
+    spec: "AttentionSpec | LatentAttentionSpec | MlstmSpec | LinearRecurrenceSpec"
     scale: float
 
 
 @dataclass(frozen=True)
+class FrequencyScaling:
+    """Rotary frequencies for contexts longer than ``original``: wavelengths above original / low are stretched by ``factor``, those
+    below original / high are kept, with a linear ramp in between."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first ``dims`` dimensions of a head: dimension i paired with i + dims / 2, or with ``interleaved`` 2i
+    with 2i + 1."""
+    base: float
+    dims: int
+    interleaved: bool = False
+    scaling: FrequencyScaling | None = None
+
+    @property
+    def frequencies(self) -> list[float]:
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if self.scaling is None:
+            return f
+        s = self.scaling
+        return llama31_frequencies(torch.tensor(f, dtype=torch.float64), s.factor, s.low, s.high, s.original).tolist()
+
+
+@dataclass(frozen=True)
 class AttentionSpec(MixerSpec):
-    """Softmax attention with normalised queries and keys; everything from ``vdim`` on is optional."""
+    """Softmax attention; everything from ``vdim`` on is optional."""
     heads: int
     kv_heads: int
     dim: int
@@ -53,6 +94,10 @@ class AttentionSpec(MixerSpec):
     softcap: float = 0.0        # scores become softcap * tanh(score / softcap), with separate values; 0 = as they are
     temp_coef: float = 0.0      # queries are multiplied by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)
     temp_every: float = 1.0
+    normed: bool = True         # queries and keys are divided by their root mean square
+    rotary: RotarySpec | None = None
+    sink: bool = False          # a learned term per head in the softmax denominator, without a key and a value
+    kv_from: int | None = None  # the layer whose cached keys and values are used; None: this layer has its own
     kind = "attention"
 
     @property
@@ -69,14 +114,47 @@ class AttentionSpec(MixerSpec):
 
     @property
     def sections(self) -> list[tuple[str, int]]:
-        s = [("q", self.heads * self.dim), ("k", self.kv_heads * self.dim)]
-        if self.vdim is not None:
-            s.append(("v", self.kv_heads * self.vdim))
+        s = [("q", self.heads * self.dim)]
+        if self.kv_from is None:
+            s.append(("k", self.kv_heads * self.dim))
+            if self.vdim is not None:
+                s.append(("v", self.kv_heads * self.vdim))
         return s + ([("g", self.heads)] if self.gated else [])
 
     @property
     def vectors(self) -> dict[str, tuple[int, ...]]:
-        return {"q.norm": (self.dim,), "k.norm": (self.dim,)} if self.norm_weights else {}
+        v: dict[str, tuple[int, ...]] = {"q.norm": (self.dim,), "k.norm": (self.dim,)} if self.norm_weights else {}
+        return {**v, "sink": (self.heads,)} if self.sink else v
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec(MixerSpec):
+    """Softmax attention whose keys and values are linear in one normalised latent per token ("dkv", its first ``rank`` rows): the
+    cache holds the latent and one rotated key part that all heads share.  The output has one sigmoid gate per element."""
+    heads: int
+    dim: int                    # unrotated query / key dimensions of a head
+    rot_dim: int                # rotated ones, behind them
+    vdim: int
+    rank: int
+    scale: float
+    rotary: RotarySpec
+    kind = "latent"
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def sections(self) -> list[tuple[str, int]]:
+        return [("q", self.heads * (self.dim + self.rot_dim)), ("dkv", self.rank), ("dkv", self.rot_dim), ("g", self.out_width)]
+
+    @property
+    def vectors(self) -> dict[str, tuple[int, ...]]:
+        return {"dkv.norm": (self.rank,)}
+
+    @property
+    def inner(self) -> dict[str, tuple[int, int]]:
+        return {"uk": (self.heads * self.dim, self.rank), "uv": (self.out_width, self.rank)}
 
 
 @dataclass(frozen=True)
@@ -101,17 +179,6 @@ class MlstmSpec(MixerSpec):
     @property
     def vectors(self) -> dict[str, tuple[int, ...]]:
         return {"i.b": (self.heads,), "f.b": (self.heads,), "norm": (self.out_width,)}
-
-
-@dataclass(frozen=True)
-class RotarySpec:
-    """Rotary positions on the first ``dims`` dimensions of a head, dimension i paired with i + dims / 2."""
-    base: float
-    dims: int
-
-    @property
-    def frequencies(self) -> list[float]:
-        return [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
 
 
 @dataclass(frozen=True)
@@ -190,9 +257,32 @@ class SquaredReluMlpSpec:
 
 
 @dataclass(frozen=True)
+class RouterSpec:
+    """Chooses ``top`` of ``experts`` per token.  Scores are sigmoids; what is compared is score + correction.  Experts form
+    ``groups`` equal groups of neighbours, of which only the ``keep`` with the largest sums of their two best are eligible.  The
+    weights are the chosen scores over (their sum + ``den_eps``), times ``scale``."""
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    den_eps: float = 1e-20
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    """A weighted sum of the chosen experts; each is a gated block of ``ff`` hidden units as in :class:`GatedMlpSpec`."""
+    router: RouterSpec
+    ff: int
+    limit: float = math.inf
+    alpha: float = 1.0
+    offset: float = 0.0
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
-    mlp: GatedMlpSpec | SquaredReluMlpSpec | None
+    mlp: GatedMlpSpec | SquaredReluMlpSpec | ExpertsSpec | None
 
 
 @dataclass(frozen=True)
@@ -205,6 +295,9 @@ class LayeredConfig:
     layer_specs: tuple[LayerSpec, ...] = field(repr=False)
     embed_scale: float = 1.0
     pre_norm: bool = False      # a norm ahead of each sublayer too ("norm1", "norm2"; those on the outputs are then "norm1b", "norm2b")
+    side_by_side: bool = False  # mixer and feed-forward read the same norm ("norm1"); x grows by residual_mult times their sum
+    residual_mult: float = 1.0
+    layer_norm: bool = False    # norms take the mean off first
 
     @property
     def layers(self) -> int:
@@ -220,14 +313,14 @@ class LayeredConfig:
 
     @property
     def attention_layers(self) -> list[int]:
-        return [i for i in range(self.layers) if self.branches(i, "attention")]
+        return [i for i in range(self.layers) if self.branches(i, "attention", "latent")]
 
     @property
     def recurrent_layers(self) -> list[int]:
         return [i for i in range(self.layers) if self.branches(i, "mlstm", "recurrence")]
 
-    def attention(self, i: int) -> AttentionSpec:
-        return self.branches(i, "attention")[0].spec
+    def attention(self, i: int) -> AttentionSpec | LatentAttentionSpec:
+        return self.branches(i, "attention", "latent")[0].spec
 
     def recurrence(self, i: int) -> MlstmSpec | LinearRecurrenceSpec:
         return self.branches(i, "mlstm", "recurrence")[0].spec
@@ -236,11 +329,23 @@ class LayeredConfig:
     def max_visible(self) -> int | None:
         """Most cached tokens a query of any attention layer can see (None: no bound, or no attention layer)."""
         seen = [self.attention(i) for i in self.attention_layers]
-        return None if not seen or any(m.window <= 0 for m in seen) else max(m.window + m.keep_first for m in seen)
+        if not seen or any(isinstance(m, LatentAttentionSpec) or m.window <= 0 for m in seen):
+            return None
+        return max(m.window + m.keep_first for m in seen)
 
-    def norm_names(self, i: int) -> list[tuple[str | None, str]]:
-        """Per sublayer of layer ``i`` the names of the norms of its input (None: none) and of its output."""
+    @property
+    def expert_layers(self) -> list[int]:
+        return [i for i in range(self.layers) if isinstance(self.layer_specs[i].mlp, ExpertsSpec)]
+
+    def experts(self, i: int) -> ExpertsSpec:
+        return self.layer_specs[i].mlp
+
+    def norm_names(self, i: int) -> list[tuple[str | None, str | None]]:
+        """Per sublayer of layer ``i`` the names of the norms of its input and of its output (None: none).  Sublayers side by side
+        count as one."""
         p = f"l{i}."
+        if self.side_by_side:
+            return [(p + "norm1", None)]
         names = [(p + f"norm{n}", p + f"norm{n}b") if self.pre_norm else (None, p + f"norm{n}") for n in (1, 2)]
         return names if self.layer_specs[i].mlp is not None else names[:1]
 
@@ -254,9 +359,14 @@ class LayeredConfig:
                 x = f"l{i}.mix.{b.prefix}"
                 for name, rows in b.spec.sections:
                     s[x + name] = (s.get(x + name, (0, w))[0] + rows, w)
-                s.update({x + n: shape for n, shape in b.spec.vectors.items()})
+                s.update({x + n: shape for n, shape in {**b.spec.vectors, **b.spec.inner}.items()})
                 s[x + "o"] = (w, b.spec.out_width)
-            if layer.mlp is not None:
+            if isinstance(layer.mlp, ExpertsSpec):
+                f, n = layer.mlp.ff, layer.mlp.router.experts
+                s.update({f"l{i}.mlp.router": (n, w), f"l{i}.mlp.correction": (n,)})
+                for e in range(n):
+                    s.update({f"l{i}.mlp.e{e}.gate": (f, w), f"l{i}.mlp.e{e}.up": (f, w), f"l{i}.mlp.e{e}.down": (w, f)})
+            elif layer.mlp is not None:
                 f = layer.mlp.ff
                 s.update({f"l{i}.mlp.{n}": (f, w) for n in layer.mlp.matrices})
                 s[f"l{i}.mlp.down"] = (w, f)
@@ -308,14 +418,28 @@ def _attention_sizes(m: dict, where: str) -> tuple[int, int, int, int]:
     return heads, kv, dim, vdim
 
 
+def _rotary(m: dict, dim: int, where: str, interleaved: bool = False) -> RotarySpec | None:
+    """The rotation of heads of ``dim`` dimensions (None: nothing is rotated)."""
+    rot, where = _get(m, "rot", where), where + ".rot"
+    dims = _size(rot, "dims", where, 0)
+    if dims % 2 or dims > dim:
+        raise LayeredConfigError(f"config.json: {where}.dims must be even and at most {dim}, got {dims}")
+    scaling, raw = None, rot.get("scaling") if interleaved else None
+    if raw is not None:
+        scaling = FrequencyScaling(*(_positive(raw, k, where + ".scaling") for k in ("factor", "low", "high", "original")))
+        if scaling.low >= scaling.high:
+            raise LayeredConfigError(f"config.json: {where}.scaling: low ({scaling.low}) must be below high ({scaling.high})")
+    return RotarySpec(_positive(rot, "base", where), dims, interleaved, scaling) if dims else None
+
+
 def _state_dim(dim: int, where: str) -> int:
     if dim > MAX_STATE_DIM:
         raise LayeredConfigError(f"config.json: {where}: key size {dim} exceeds {MAX_STATE_DIM}")
     return dim
 
 
-def _layers(raw: dict, mixers: dict, mlp) -> tuple[LayerSpec, ...]:
-    """The layer list: ``mixers`` reads a mixer by its type, ``mlp`` a dense feed-forward block."""
+def _layers(raw: dict, mixers: dict, mlp, mlp_kind: str = "dense") -> tuple[LayerSpec, ...]:
+    """The layer list: ``mixers`` reads a mixer by its type, ``mlp`` a feed-forward block of the kind the design has."""
     layers = []
     for i, entry in enumerate(_get(raw, "layers", "the model")):
         where = f"layers[{i}]"
@@ -323,7 +447,7 @@ def _layers(raw: dict, mixers: dict, mlp) -> tuple[LayerSpec, ...]:
         if kind not in mixers:
             raise LayeredConfigError(f"config.json: {where}: unknown mixer type {kind!r}")
         ff = _get(entry, "mlp", where)
-        if ff is not None and _get(ff, "kind", where + ".mlp") != "dense":
+        if ff is not None and _get(ff, "kind", where + ".mlp") != mlp_kind:
             raise LayeredConfigError(f"config.json: {where}.mlp: unknown kind {ff['kind']!r}")
         layers.append(LayerSpec(mixers[kind](_get(entry, "mixer", where), where + ".mixer"), None if ff is None else mlp(ff, where + ".mlp")))
     if not layers:
@@ -369,13 +493,8 @@ def _decays(m: dict, heads: int, where: str) -> tuple[float, ...]:
 
 def _retention(m: dict, where: str) -> LinearRecurrenceSpec:
     heads, dim, vdim = (_size(m, k, where) for k in ("heads", "dim", "vdim"))
-    rot = _get(m, "rot", where)
-    dims = _size(rot, "dims", where + ".rot", 0)
-    if dims % 2 or dims > dim:
-        raise LayeredConfigError(f"config.json: {where}.rot.dims must be even and at most {dim}, got {dims}")
-    rotary = RotarySpec(_positive(rot, "base", where + ".rot"), dims) if dims else None
     return LinearRecurrenceSpec(heads, _state_dim(dim, where), vdim, groups=heads, norm_parts=heads, gate="silu", decay=_decays(m, heads, where),
-                                rotary=rotary, key_scale=dim ** -0.5)
+                                rotary=_rotary(m, dim, where), key_scale=dim ** -0.5)
 
 
 def _lightning(m: dict, where: str) -> LinearRecurrenceSpec:
@@ -411,3 +530,53 @@ def kekevik_config(raw: dict, name: str = "") -> LayeredConfig:
                      lambda m, where: SquaredReluMlpSpec(_size(m, "ff", where)))
     scale = _number(_get(raw, "embedding", "the model"), "scale", "embedding")
     return _model(raw, "Kekevik", name, layers, embed_scale=scale, pre_norm=True)
+
+
+# ---- Kutepel ----------------------------------------------------------------------------------------------------------------------
+def _rotary_attention(m: dict, where: str) -> AttentionSpec:
+    heads, kv, dim, vdim = _attention_sizes(m, where)
+    source = None if m.get("kv_from") is None else _size(m, "kv_from", where, 0)
+    return AttentionSpec(heads, kv, dim, _number(m, "scale", where), vdim=vdim, normed=False, rotary=_rotary(m, dim, where, interleaved=True), sink=True,
+                         kv_from=source)
+
+
+def _latent_attention(m: dict, where: str) -> LatentAttentionSpec:
+    heads, dim, rot_dim, vdim, rank = (_size(m, k, where) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+    rotary = _rotary(m, rot_dim, where, interleaved=True)
+    if rotary is None or rotary.dims != rot_dim:
+        raise LayeredConfigError(f"config.json: {where}: rot.dims must be rot_dim ({rot_dim}), which must be even")
+    up = lambda n, m: -(-n // m) * m
+    if up(dim, 8) + up(rot_dim, 8) > MAX_HEAD_DIM or vdim > MAX_HEAD_DIM:
+        raise LayeredConfigError(f"config.json: {where}: head sizes {dim} + {rot_dim} and {vdim} exceed {MAX_HEAD_DIM}")
+    if rank > MAX_RANK or up(rank, 16) + up(rot_dim, 16) > MAX_LATENT_ROW:
+        raise LayeredConfigError(f"config.json: {where}: a latent of {rank} + {rot_dim} exceeds {MAX_RANK} or {MAX_LATENT_ROW} together")
+    return LatentAttentionSpec(heads, dim, rot_dim, vdim, rank, _number(m, "scale", where), rotary)
+
+
+def _experts(m: dict, where: str) -> ExpertsSpec:
+    r, ff = _get(m, "router", where), _size(_get(m, "expert", where), "ff", where + ".expert")
+    where += ".router"
+    experts, top = _size(r, "experts", where), _size(r, "top", where)
+    g = r.get("groups")
+    count, keep = (1, 1) if g is None else (_size(g, "count", where + ".groups"), _size(g, "keep", where + ".groups"))
+    if experts > MAX_EXPERTS or top > MAX_CHOSEN:
+        raise LayeredConfigError(f"config.json: {where}: {top} of {experts} experts (at most {MAX_CHOSEN} of {MAX_EXPERTS})")
+    if experts % count or keep > count or top > keep * (experts // count):
+        raise LayeredConfigError(f"config.json: {where}: {top} of {experts} experts in {keep} of {count} groups")
+    return ExpertsSpec(RouterSpec(experts, top, count, keep, _number(r, "scale", where)), ff)
+
+
+def kutepel_config(raw: dict, name: str = "") -> LayeredConfig:
+    """The Kutepel design: latent attention and rotary attention with sinks (some layers on an earlier one's keys and values) in the
+    order the file lists, side by side with a mixture of experts behind one layer norm, and a head tied to the embedding."""
+    layers = _layers(raw, {"attention": _rotary_attention, "latent_attention": _latent_attention}, _experts, "moe")
+    for i, layer in enumerate(layers):
+        j = getattr(layer.mixer, "kv_from", None)
+        if j is None:
+            continue
+        source = layers[j].mixer if j < i else None
+        if not isinstance(source, AttentionSpec) or source.kv_from is not None:
+            raise LayeredConfigError(f"config.json: layers[{i}].mixer.kv_from: layer {j} is no earlier attention layer with keys and values of its own")
+        if (source.kv_heads, source.dim, source.vdim) != (layer.mixer.kv_heads, layer.mixer.dim, layer.mixer.vdim):
+            raise LayeredConfigError(f"config.json: layers[{i}].mixer.kv_from: layer {j} has other key/value heads")
+    return _model(raw, "Kutepel", name, layers, side_by_side=True, residual_mult=_number(raw, "residual_mult", "the model"), layer_norm=True)

@@ -45,21 +45,21 @@ class PagePool:
 
 
 class RowCache(PagePool):
-    """Paged cache of attention layers: per layer ``rows`` [pages, kv_heads, page_size, row], the keys, and beside them either
-    ``values`` of the same shape, or, where the rows serve as key and value, one float per row (``factors``: the key's
-    reciprocal root mean square).  ``layers``: {layer index: (kv heads, row elements, separate values)}; layers may differ, they
-    share the page numbering."""
+    """Paged cache of attention layers: per layer ``rows`` [pages, kv_heads, page_size, row] and, by what they hold, a companion:
+    "separate": keys, with ``values`` of the same shape; "shared": rows that serve as key and value, with one float per row
+    (``factors``: the key's reciprocal root mean square); "latent": rows that keys and values are expanded from, alone.
+    ``layers``: {layer index: (kv heads, row elements, kind)}; layers may differ, they share the page numbering."""
 
-    def __init__(self, layers: dict[int, tuple[int, int, bool]], num_pages: int, page_size: int, kvt: int, dtype: torch.dtype, device):
+    def __init__(self, layers: dict[int, tuple[int, int, str]], num_pages: int, page_size: int, kvt: int, dtype: torch.dtype, device):
         super().__init__(num_pages, page_size)
         self.kvt = kvt
         self.rows, self.values, self.factors = {}, {}, {}
-        for l, (h, row, separate) in layers.items():
+        for l, (h, row, kind) in layers.items():
             new = lambda *shape, dtype=dtype: torch.zeros((num_pages, h, page_size, *shape), dtype=dtype, device=device)
             self.rows[l] = new(row)
-            if separate:
+            if kind == "separate":
                 self.values[l] = new(row)
-            else:
+            elif kind == "shared":
                 self.factors[l] = new(dtype=torch.float32)
 
     @property

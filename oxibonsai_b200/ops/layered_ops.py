@@ -12,9 +12,10 @@ from . import cuda_ops as K
 
 _vp, _i, _f = C.c_void_p, C.c_int, C.c_float
 _SIG = {
-    "bonsai_lay_embed": [_vp, _i, _vp, _f, _i, _i, _vp, _vp, _i, _i, _vp, _f, _vp],
+    "bonsai_lay_embed": [_vp, _i, _vp, _f, _i, _i, _vp, _vp, _i, _i, _vp, _f, _i, _vp],
     "bonsai_lay_norm_add": [_vp, _vp, _i, _vp, _f, _i, _i, _vp, _i, _i, _vp, _vp],
-    "bonsai_lay_norm_rows": [_vp, _vp, _vp, _f, _i, _i, _vp, _i, _i, _vp],
+    "bonsai_lay_side_by_side": [_vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _f, _i, _i, _vp, _i, _i, _vp, _f, _i, _vp],
+    "bonsai_lay_norm_rows": [_vp, _vp, _vp, _f, _i, _i, _i, _vp, _i, _i, _vp],
     "bonsai_lay_gated_norm": [_vp, _i, _vp, _i, _vp, _f, _i, _i, _i, _i, _i, _f, _vp, _i, _i, _vp],
     "bonsai_lay_linear_few": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _vp],
     "bonsai_lay_linear_f32": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
@@ -25,6 +26,21 @@ _SIG = {
     "bonsai_lay_attn_prompt": [_vp, _vp, _vp, _vp, _vp, _i, _vp],
     "bonsai_lay_attn_decode": [_vp, _vp, _vp, _i, _i, _vp],
     "bonsai_lay_attn_f32": [_vp, _vp, _vp, _i, _vp],
+    "bonsai_lay_latent_row": [_i, _i],
+    "bonsai_lay_latent_max_splits": [],
+    "bonsai_lay_latent_group": [_i],
+    "bonsai_lay_latent_append": [_vp, _vp, _vp, _i, _i, _i, _vp],
+    "bonsai_lay_latent_query": [_vp, _vp, _vp, _i, _vp],
+    "bonsai_lay_latent_decode": [_vp, _vp, _vp, _i, _i, _vp],
+    "bonsai_lay_latent_value": [_vp, _vp, _vp, _i, _i, _vp],
+    "bonsai_lay_latent_gather": [_vp, _vp, _vp, _vp, _i, _i, _vp, _i, _vp],
+    "bonsai_lay_latent_prompt": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp],
+    "bonsai_lay_latent_f32": [_vp, _vp, _vp, _i, _vp],
+    "bonsai_lay_route_small": [_i],
+    "bonsai_lay_route": [_vp, _vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp],
+    "bonsai_lay_experts_few": [_vp, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
+    "bonsai_lay_experts_f32": [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
+    "bonsai_grouped_gemm_bf16": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _f, _f, _f, _i, _vp, _i, _vp],
     "bonsai_lay_mlstm_dim": [_i],
     "bonsai_lay_mlstm_vdim": [_i],
     "bonsai_lay_mlstm_chunk_dim": [],
@@ -115,23 +131,23 @@ _NO_GLU = Glu(0.0, 0.0, 0.0)
 
 
 def linear(w: DenseWeight, x: torch.Tensor, T: int, out: torch.Tensor, scratch: GemmScratch, act: Glu | str | None = None) -> None:
-    """out[:T] = act(x[:T] W^T).  bf16 ``x`` (row stride >= kp, finite in the padding): tensor cores, f32 ``out`` (bf16 with
+    """out[:T] = act(x[:T] W^T).  bf16 ``x`` (row stride >= kp, finite in the padding): tensor cores, f32 or bf16 ``out`` (bf16 with
     ``act``); f32 ``x``: 32-bit throughout.  ``act``: none, :class:`Glu`, or ``SQUARED_RELU``."""
     l, s = lib(), K.stream()
     glu = act if isinstance(act, Glu) else _NO_GLU
-    epi = 0 if act is None else (1 if isinstance(act, Glu) else 2)
+    epi = (3 if out.dtype == torch.bfloat16 else 0) if act is None else (1 if isinstance(act, Glu) else 2)
     if x.dtype == torch.float32:
         K.check(l.bonsai_lay_linear_f32(w.data.data_ptr(), w.n, w.k, w.kp, x.data_ptr(), x.stride(0), T, out.data_ptr(), out.stride(0),
                                         epi, glu.limit, glu.alpha, glu.offset, s), "linear_f32")
         return
-    assert x.dtype == torch.bfloat16 and out.dtype == (torch.float32 if act is None else torch.bfloat16)
-    f32, b16 = (out.data_ptr(), None) if act is None else (None, out.data_ptr())
+    assert x.dtype == torch.bfloat16 and (act is None or out.dtype == torch.bfloat16)
+    f32, b16 = (out.data_ptr(), None) if epi == 0 else (None, out.data_ptr())
     if T <= FEW_ROWS:
         K.check(l.bonsai_lay_linear_few(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), epi,
                                         glu.limit, glu.alpha, glu.offset, s), "linear_few")
     else:
         K.check(l.bonsai_dense_gemm_bf16(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0),
-                                         (0, 4, 5)[epi], glu.limit, glu.alpha, glu.offset, scratch.status.data_ptr(), scratch.ws.data_ptr(),
+                                         (0, 4, 5, 6)[epi], glu.limit, glu.alpha, glu.offset, scratch.status.data_ptr(), scratch.ws.data_ptr(),
                                          scratch.ws.numel(), scratch.sms, s), "dense_gemm_bf16")
 
 
@@ -140,10 +156,10 @@ def _row_out(t: torch.Tensor | None) -> tuple[int | None, int, int]:
 
 
 def embed(table: torch.Tensor, tokens: torch.Tensor, scale: float, T: int, width: int, x: torch.Tensor, h: torch.Tensor | None,
-          next_norm: torch.Tensor | None, eps: float) -> None:
-    """x = table[tokens] * scale; ``h`` receives x, or its norm with weight ``next_norm``."""
+          next_norm: torch.Tensor | None, eps: float, center: bool = False) -> None:
+    """x = table[tokens] * scale; ``h`` receives x, or its norm with weight ``next_norm`` (``center``: a layer norm)."""
     K.check(lib().bonsai_lay_embed(table.data_ptr(), table.stride(0), tokens.data_ptr(), scale, T, width, x.data_ptr(), *_row_out(h), K.ptr(next_norm), eps,
-                                   K.stream()), "embed")
+                                   int(center), K.stream()), "embed")
 
 
 def norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, T: int, h: torch.Tensor | None, next_norm: torch.Tensor | None = None) -> None:
@@ -152,9 +168,18 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, T: i
             "norm_add")
 
 
-def norm_rows(x: torch.Tensor, rows: int | None, count: int, w: torch.Tensor, eps: float, out: torch.Tensor) -> None:
-    """out[i] = rmsnorm(x[rows[i]]) * w (``rows``: device address of int32 indices, None = 0 .. count - 1)."""
-    K.check(lib().bonsai_lay_norm_rows(x.data_ptr(), rows, w.data_ptr(), eps, count, x.shape[1], out.data_ptr(), out.stride(0),
+def side_by_side(x: torch.Tensor, y: torch.Tensor, experts: "Routing | None", mult: float, T: int, h: torch.Tensor | None, next_norm: torch.Tensor | None,
+                 eps: float, center: bool) -> None:
+    """x += mult * (y + each row's expert outputs); ``h`` receives x, or its norm with weight ``next_norm``.  Leaves the router's
+    counters zero."""
+    e = (None, 0, 0, None, 0, None, 0) if experts is None else experts.outputs
+    K.check(lib().bonsai_lay_side_by_side(x.data_ptr(), y.data_ptr(), y.stride(0), *e, mult, T, x.shape[1], *_row_out(h), K.ptr(next_norm), eps, int(center),
+                                          K.stream()), "side_by_side")
+
+
+def norm_rows(x: torch.Tensor, rows: int | None, count: int, w: torch.Tensor, eps: float, out: torch.Tensor, center: bool = False) -> None:
+    """out[i] = rmsnorm(x[rows[i]]) * w (``rows``: device address of int32 indices, None = 0 .. count - 1); ``center``: a layer norm."""
+    K.check(lib().bonsai_lay_norm_rows(x.data_ptr(), rows, w.data_ptr(), eps, int(center), count, x.shape[1], out.data_ptr(), out.stride(0),
                                        int(out.dtype == torch.float32), K.stream()), "norm_rows")
 
 
@@ -180,6 +205,85 @@ class MixerCall:
     @property
     def args(self):
         return self.ptrs, self.ints, self.floats
+
+
+class ExpertScratch:
+    """Buffers the expert layers of a model share (they run one after another): the router's lists for ``rows`` tokens, and the sorted
+    rows, hidden units and outputs of all (token, chosen expert) pairs."""
+
+    def __init__(self, rows: int, width: int, specs, exact: bool, device):
+        self.rows, self.width, self.exact = rows, width, exact
+        top, experts = max(s.router.top for s in specs), max(s.router.experts for s in specs)
+        self.pairs = rows * top
+        i32, f32 = dict(dtype=torch.int32, device=device), dict(dtype=torch.float32, device=device)
+        act = dict(dtype=torch.float32 if exact else torch.bfloat16, device=device)
+        self.counts, self.lists = torch.zeros(experts, **i32), torch.zeros(2 * experts + 2, **i32)
+        self.pair, self.pair_weight = torch.zeros((self.pairs, 2), **i32), torch.zeros(self.pairs, **f32)
+        self.token, self.weight, self.at = torch.zeros(self.pairs, **i32), torch.zeros(self.pairs, **f32), torch.zeros(self.pairs, **i32)
+        # the padding columns stay zero for the projections that read them: one buffer per number of hidden units
+        self.sorted = None if exact else torch.zeros((self.pairs, round_up(width, K_ALIGN)), **act)
+        self.hidden = {ff: torch.zeros((self.pairs, round_up(ff, 4 if exact else K_ALIGN)), **act) for ff in {s.ff for s in specs}}
+        ld = round_up(width, 8)
+        self.out = torch.zeros((self.pairs, ld), **act)
+        # f32 outputs of steps with few pairs, in the same memory
+        self.out32 = self.out if exact else self.out.view(-1).view(torch.float32)[: self.pairs // 2 * ld].view(-1, ld)
+
+
+class Routing:
+    """One expert layer's calls: choice, sorting, the experts' projections.  ``logits``: the projections the router's are part of."""
+
+    def __init__(self, spec, up: DenseWeight, down: DenseWeight, correction: torch.Tensor, logits: torch.Tensor, column: int, scratch: ExpertScratch):
+        r = spec.router
+        self.spec, self.up, self.down, self.s = spec, up, down, scratch
+        self.glu = Glu(spec.limit, spec.alpha, spec.offset)
+        self.call = MixerCall([logits, correction, scratch.counts, scratch.pair, scratch.pair_weight, scratch.lists, scratch.token, scratch.weight, scratch.at],
+                              [logits.stride(0), column, r.experts, r.top, r.groups, r.keep], [r.scale, r.den_eps])
+        self.n_up, self.n_down = up.n // r.experts, down.n // r.experts
+        self.out = scratch.out
+
+    @property
+    def outputs(self) -> tuple:
+        """Expert rows and where a token finds its own, as :func:`side_by_side` takes them."""
+        o, r = self.out, self.spec.router
+        return (o.data_ptr(), o.stride(0), int(o.dtype == torch.float32), self.s.at.data_ptr(), r.top, self.s.counts.data_ptr(), r.experts)
+
+    def few(self, T: int) -> bool:
+        """Whether the experts' weights are streamed for a few rows each, rather than multiplied in tiles."""
+        r = self.spec.router
+        return T * r.top <= self.s.pairs // 2 and (T <= FEW_ROWS or T * r.top <= 12 * r.experts)
+
+    def launches(self, T: int) -> int:
+        return 2 + (1 if T <= lib().bonsai_lay_route_small(self.spec.router.top) and (self.s.exact or self.few(T)) else 2)
+
+    def __call__(self, h: torch.Tensor, T: int, scratch: GemmScratch) -> None:
+        l, s, st, r = lib(), self.s, K.stream(), self.spec.router
+        pairs, hid = T * r.top, s.hidden[self.spec.ff]
+        tile = not s.exact and not self.few(T)
+        xs, chunks = (s.sorted, round_up(s.width, 8) // 8) if tile else (None, 0)
+        K.check(l.bonsai_lay_route(*self.call.args, T, h.data_ptr(), h.stride(0), chunks, K.ptr(xs), 0 if xs is None else xs.stride(0), st), "route")
+        lists, token, weight = s.lists.data_ptr(), s.token.data_ptr(), s.weight.data_ptr()
+        up, down, g = self.up, self.down, self.glu
+        if s.exact:
+            self.out = s.out
+            K.check(l.bonsai_lay_experts_f32(up.data.data_ptr(), r.experts, self.n_up, up.k, up.kp, h.data_ptr(), h.stride(0), lists, token, weight, pairs, T,
+                                             hid.data_ptr(), hid.stride(0), 1, g.limit, g.alpha, g.offset, st), "experts_f32")
+            K.check(l.bonsai_lay_experts_f32(down.data.data_ptr(), r.experts, self.n_down, down.k, down.kp, hid.data_ptr(), hid.stride(0), lists, None, None,
+                                             pairs, T, s.out.data_ptr(), s.out.stride(0), 0, 0.0, 0.0, 0.0, st), "experts_f32")
+        elif not tile:
+            self.out = s.out32
+            slots, per = min(r.experts, pairs), min(T, 2 * pairs // r.experts + 8)
+            K.check(l.bonsai_lay_experts_few(up.data.data_ptr(), r.experts, self.n_up, up.kp, h.data_ptr(), h.stride(0), lists, token, weight, pairs, slots, per,
+                                             hid.data_ptr(), hid.stride(0), 1, g.limit, g.alpha, g.offset, st), "experts_few")
+            K.check(l.bonsai_lay_experts_few(down.data.data_ptr(), r.experts, self.n_down, down.kp, hid.data_ptr(), hid.stride(0), lists, None, None, pairs,
+                                             slots, per, s.out32.data_ptr(), s.out32.stride(0), 0, 0.0, 0.0, 0.0, st), "experts_few")
+        else:
+            self.out = s.out
+            wide = int(pairs > 96 * r.experts)
+            K.check(l.bonsai_grouped_gemm_bf16(up.data.data_ptr(), r.experts, self.n_up, up.kp, xs.data_ptr(), xs.stride(0), pairs, lists, weight, hid.data_ptr(),
+                                               hid.stride(0), 4, g.limit, g.alpha, g.offset, wide, scratch.status.data_ptr(), scratch.sms, st), "grouped_gemm")
+            K.check(l.bonsai_grouped_gemm_bf16(down.data.data_ptr(), r.experts, self.n_down, down.kp, hid.data_ptr(), hid.stride(0), pairs, lists, None,
+                                               s.out.data_ptr(), s.out.stride(0), 6, 0.0, 0.0, 0.0, wide, scratch.status.data_ptr(), scratch.sms, st),
+                    "grouped_gemm")
 
 
 def sample(logits: torch.Tensor, *a, **kw) -> torch.Tensor:

@@ -214,6 +214,104 @@ def squared_relu_ff(x, w, p):
     return linear(torch.relu(linear(x, w[p + "up"])) ** 2, w[p + "down"])
 
 
+# ---- interleaved rotation with scaled frequencies, attention with a sink, latent attention ----------------------------------------------
+def frequencies(rot):
+    """Angles per position of the ``dims`` / 2 pairs; long wavelengths are stretched by ``factor``, with a ramp in between."""
+    out = []
+    for i in range(rot["dims"] // 2):
+        f = rot["base"] ** (-2.0 * i / rot["dims"])
+        sc = rot.get("scaling")
+        if sc is not None:
+            turns = sc["original"] * f / (2.0 * math.pi)         # turns within the original context
+            if turns < sc["low"]:
+                f = f / sc["factor"]
+            elif turns <= sc["high"]:
+                s = (turns - sc["low"]) / (sc["high"] - sc["low"])
+                f = (1.0 - s) * f / sc["factor"] + s * f
+        out.append(f)
+    return out
+
+
+def rotate_pairs(x, first_position, rot):
+    """x [n, heads, d]: dimensions 2i and 2i + 1 are a pair; dimensions from ``dims`` on pass."""
+    dims = rot["dims"]
+    pos = torch.arange(first_position, first_position + x.shape[0], dtype=x.dtype)
+    a = pos[:, None] * torch.tensor(frequencies(rot), dtype=x.dtype)[None, :]
+    c, s = torch.cos(a)[:, None, :], torch.sin(a)[:, None, :]
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+    out = x.clone()
+    out[..., 0:dims:2] = u * c - v * s
+    out[..., 1:dims:2] = v * c + u * s
+    return out
+
+
+def sink_attention(q, k, v, scale, sink=None):
+    """One head over all earlier positions; the sink is one more term of the denominator (None: no sink)."""
+    n = q.shape[0]
+    s = ((q @ k.T) * scale).masked_fill(torch.ones(n, n).triu(1).bool(), float("-inf"))
+    if sink is None:
+        return torch.softmax(s, dim=-1) @ v
+    return torch.softmax(torch.cat([s, sink.expand(n, 1)], dim=-1), dim=-1)[:, :n] @ v
+
+
+def rotary_attention_mixer(h, w, p, m, shared):
+    """Grouped-query attention with rotated heads and sinks; ``shared``: the keys and values of each layer so far."""
+    n, H, G, d, e = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q = rotate_pairs(linear(h, w[p + "q"]).view(n, H, d), 0, m["rot"])
+    if "kv_from" in m:
+        k, v = shared[m["kv_from"]]
+    else:
+        k = rotate_pairs(linear(h, w[p + "k"]).view(n, G, d), 0, m["rot"])
+        v = linear(h, w[p + "v"]).view(n, G, e)
+    o = torch.stack([sink_attention(q[:, a], k[:, a // (H // G)], v[:, a // (H // G)], m["scale"], w[p + "sink"][a]) for a in range(H)], dim=1)
+    return linear(o.reshape(n, H * e), w[p + "o"]), (k, v)
+
+
+def latent_attention_mixer(h, w, p, m, eps):
+    """Keys and values are expanded from one normalised latent per token; one rotated key part serves all heads."""
+    n, H, d, r, e, R = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    q = linear(h, w[p + "q"]).view(n, H, d + r)
+    q = torch.cat([q[..., :d], rotate_pairs(q[..., d:], 0, m["rot"])], dim=-1)
+    ckr = linear(h, w[p + "dkv"])
+    c = rms_norm(ckr[:, :R], w[p + "dkv.norm"], eps)
+    kr = rotate_pairs(ckr[:, None, R:], 0, m["rot"])
+    k = torch.cat([linear(c, w[p + "uk"]).view(n, H, d), kr.expand(n, H, r)], dim=-1)
+    v = linear(c, w[p + "uv"]).view(n, H, e)
+    o = torch.stack([sink_attention(q[:, a], k[:, a], v[:, a], m["scale"]) for a in range(H)], dim=1).reshape(n, H * e)
+    return linear(o * torch.sigmoid(linear(h, w[p + "g"])), w[p + "o"])
+
+
+# ---- experts ---------------------------------------------------------------------------------------------------------------------
+def route(z, correction, top, groups, keep, scale):
+    """One token: chosen experts (best first) and their weights.  z [experts]: router logits."""
+    s = torch.sigmoid(z)
+    choice = s + correction
+    size = len(choice) // groups
+    best = sorted(range(groups), key=lambda g: -float(torch.sort(choice[g * size:(g + 1) * size], descending=True).values[:2].sum()))[:keep]
+    allowed = [e for e in range(len(choice)) if e // size in best]
+    chosen = sorted(allowed, key=lambda e: -float(choice[e]))[:top]
+    weights = torch.stack([s[e] for e in chosen])
+    return chosen, weights / (weights.sum() + 1e-20) * scale
+
+
+def expert(x, w, p):
+    return linear(silu(linear(x, w[p + "gate"])) * linear(x, w[p + "up"]), w[p + "down"])
+
+
+def experts_ff(h, w, p, mlp):
+    r, out = mlp["router"], []
+    z = linear(h, w[p + "router"])
+    for t in range(h.shape[0]):
+        chosen, weights = route(z[t], w[p + "correction"], r["top"], r["groups"]["count"], r["groups"]["keep"], r["scale"])
+        out.append(sum(g * expert(h[t], w, f"{p}e{e}.") for e, g in zip(chosen, weights)))
+    return torch.stack(out)
+
+
+def layer_norm(x, weight, eps):
+    d = x - x.mean(-1, keepdim=True)
+    return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * weight
+
+
 # ---- whole models -----------------------------------------------------------------------------------------------------------------
 MIXERS = {"attention": attention_mixer, "mlstm": mlstm_mixer, "retention": retention_mixer, "lightning": lightning_mixer, "parallel": parallel_mixer}
 
@@ -235,16 +333,32 @@ def kekevik_layer(x, w, p, layer, eps):
     return x
 
 
+def kutepel_layer(x, w, p, layer, eps, mult, shared):
+    """One layer norm, the mixer and the feed-forward side by side behind it.  Returns x and the layer's keys and values."""
+    h, m, kv = layer_norm(x, w[p + "norm1"], eps), layer["mixer"], None
+    if layer["type"] == "attention":
+        y, kv = rotary_attention_mixer(h, w, p + "mix.", m, shared)
+    else:
+        y = latent_attention_mixer(h, w, p + "mix.", m, eps)
+    if layer["mlp"] is not None:
+        y = y + experts_ff(h, w, p + "mlp.", layer["mlp"])
+    return x + mult * y, kv
+
+
 def forward(cfg, w, tokens, keep_layers=False):
     """Logits [n, vocab] of every position (and the residual stream after every layer)."""
-    eps = cfg["norm"]["eps"]
-    run = {"Keripel": keripel_layer, "Kekevik": kekevik_layer}[cfg["architecture"]]
+    eps, arch = cfg["norm"]["eps"], cfg["architecture"]
     x = w["embed"][torch.as_tensor(list(tokens), dtype=torch.long)] * cfg.get("embedding", {}).get("scale", 1.0)
-    kept = []
+    kept, shared = [], []
     for l, layer in enumerate(cfg["layers"]):
-        x = run(x, w, f"l{l}.", layer, eps)
+        if arch == "Kutepel":
+            x, kv = kutepel_layer(x, w, f"l{l}.", layer, eps, cfg["residual_mult"], shared)
+            shared.append(kv)
+        else:
+            x = {"Keripel": keripel_layer, "Kekevik": kekevik_layer}[arch](x, w, f"l{l}.", layer, eps)
         kept.append(x)
-    logits = linear(rms_norm(x, w["final.norm"], eps), w["embed"])
+    norm = layer_norm if arch == "Kutepel" else rms_norm
+    logits = linear(norm(x, w["final.norm"], eps), w["embed"])
     return (logits, torch.stack(kept)) if keep_layers else logits
 
 
@@ -278,8 +392,33 @@ def kekevik_mixer_shapes(layer, p, W):
     return s
 
 
+def kutepel_tensor_shapes(cfg):
+    W = cfg["width"]
+    s = {"embed": (cfg["vocab"], W), "final.norm": (W,)}
+    for l, layer in enumerate(cfg["layers"]):
+        m, p, f = layer["mixer"], f"l{l}.mix.", f"l{l}.mlp."
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        s[f"l{l}.norm1"] = (W,)
+        if layer["type"] == "attention":
+            s.update({p + "q": (H * d, W), p + "sink": (H,)})
+            if "kv_from" not in m:
+                s.update({p + "k": (m["kv_heads"] * d, W), p + "v": (m["kv_heads"] * e, W)})
+        else:
+            R, r = m["kv_rank"], m["rot_dim"]
+            s.update({p + "q": (H * (d + r), W), p + "dkv": (R + r, W), p + "dkv.norm": (R,), p + "uk": (H * d, R), p + "uv": (H * e, R), p + "g": (H * e, W)})
+        s[p + "o"] = (W, H * e)
+        if layer["mlp"] is not None:
+            E, F = layer["mlp"]["router"]["experts"], layer["mlp"]["expert"]["ff"]
+            s.update({f + "router": (E, W), f + "correction": (E,)})
+            for j in range(E):
+                s.update({f"{f}e{j}.gate": (F, W), f"{f}e{j}.up": (F, W), f"{f}e{j}.down": (W, F)})
+    return s
+
+
 def tensor_shapes(cfg):
     """Name -> shape of every tensor of a model."""
+    if cfg["architecture"] == "Kutepel":
+        return kutepel_tensor_shapes(cfg)
     W, keripel = cfg["width"], cfg["architecture"] == "Keripel"
     s = {"embed": (cfg["vocab"], W), "final.norm": (W,)}
     for l, layer in enumerate(cfg["layers"]):
@@ -310,6 +449,10 @@ def random_weights(cfg, seed=0, scale=1.0):
             t = 2.0 + 1.5 * t                      # from strong forgetting to almost none
         elif name.endswith("dt_bias"):
             t = t - 1.0
+        elif name.endswith(".sink"):
+            t = 1.0 + t
+        elif name.endswith(".correction"):
+            t = 0.3 * t - 0.2                      # some choice scores are negative
         elif name.endswith("A_log"):
             t = 1.5 * t - 2.0                      # from forgetting in a few tokens to hardly at all
         elif name.endswith(".D"):
