@@ -70,6 +70,39 @@ def kekevik_mixed():
                     retention(2, 50, 66, 100.0, 30, ff=70), lightning(1, 70, 130)])
 
 
+# ---- Kutepel ----------------------------------------------------------------------------------------------------------------------
+STRETCH = {"factor": 5.0, "low": 1.5, "high": 6.0, "original": 90}
+
+
+def experts(ff=40, n=12, top=3, groups=3, keep=2, scale=1.7):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": n, "groups": {"count": groups, "keep": keep}, "scale": scale, "top": top}}
+
+
+def rotation(dims, base, scaling):
+    return {"base": base, "dims": dims, **({} if scaling is None else {"scaling": scaling})}
+
+
+def rotary(heads=6, kv_heads=2, dim=40, vdim=24, scale=0.25, dims=None, base=2000.0, scaling=None, kv_from=None, mlp=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "rot": rotation(dim if dims is None else dims, base, scaling)}
+    return {"type": "attention", "mixer": m if kv_from is None else {**m, "kv_from": kv_from}, "mlp": mlp}
+
+
+def latent(heads=3, dim=20, rot_dim=12, vdim=28, rank=72, scale=0.3, base=700.0, scaling=None, mlp=None):
+    return {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank, "scale": scale,
+                                                  "rot": rotation(rot_dim, base, scaling)}, "mlp": mlp}
+
+
+def kutepel(layers, width=152, vocab=331, eps=1e-5, mult=0.4):
+    return {"architecture": "Kutepel", "layers": layers, "norm": {"eps": eps}, "residual_mult": mult, "vocab": vocab, "width": width}
+
+
+# every branch in one model: both mixers with and without experts, own and shared keys, with and without stretched frequencies
+def kutepel_mixed():
+    return kutepel([latent(mlp=experts()), rotary(scaling=STRETCH, mlp=experts(33, 10, 2, 5, 3, 0.8)), latent(5, 33, 30, 70, 130, 0.15, 1e4, STRETCH),
+                    rotary(kv_from=1, scaling=STRETCH, mlp=experts(24, 7, 1, 1, 1, 1.0)), rotary(4, 4, 32, 72, 0.2, 20), rotary(12, 2, kv_from=1, dims=10, mlp=experts()),
+                    latent(17, 16, 2, 8, 16, 0.3, 50.0, mlp=experts(64, 20, 4, 10, 2, 2.0))])
+
+
 def write(path, cfg, weights):
     from oxibonsai_b200.convert import write_safetensors
     os.makedirs(path, exist_ok=True)

@@ -294,6 +294,17 @@ def route(z, correction, top, groups, keep, scale):
     return chosen, weights / (weights.sum() + 1e-20) * scale
 
 
+def route_margin(z, correction, top, groups, keep):
+    """How far the choice is from another one: the smaller of the gaps behind the last kept group and behind the last chosen expert."""
+    choice = torch.sigmoid(z) + correction
+    size = len(choice) // groups
+    sums = torch.stack([torch.sort(choice[g * size:(g + 1) * size], descending=True).values[:2].sum() for g in range(groups)])
+    order = torch.argsort(sums, descending=True)
+    gap = float(sums[order[keep - 1]] - sums[order[keep]]) if keep < groups else math.inf
+    left = torch.sort(torch.cat([choice[g * size:(g + 1) * size] for g in order[:keep].tolist()]), descending=True).values
+    return min(gap, float(left[top - 1] - left[top])) if top < len(left) else gap
+
+
 def expert(x, w, p):
     return linear(silu(linear(x, w[p + "gate"])) * linear(x, w[p + "up"]), w[p + "down"])
 
@@ -464,4 +475,36 @@ def random_weights(cfg, seed=0, scale=1.0):
         else:
             t = t * scale * shape[-1] ** -0.5
         w[name] = t.bfloat16().float()
+    if cfg["architecture"] == "Kutepel":
+        settle_routers(cfg, w, g)
     return w
+
+
+CODES = 16
+
+
+def settle_routers(cfg, w, g, margin=0.016):
+    """Makes the choice of experts depend on the token alone, clearly: the last ``CODES`` dimensions of the stream hold a code of the token
+    that no sublayer changes, and router rows read only those.  The last code balances the rows, so that a mean does not enter."""
+    W, amp = cfg["width"], 6.0
+    code = torch.randint(0, CODES - 1, (cfg["vocab"],), generator=g)
+    w["embed"][:, -CODES:] = amp * torch.nn.functional.one_hot(code, CODES).float()
+    for l, layer in enumerate(cfg["layers"]):
+        p = f"l{l}."
+        w[p + "norm1"][-CODES:] = 1.0
+        w[p + "mix.o"][-CODES:] = 0.0
+        if layer["mlp"] is None:
+            continue
+        r, c = layer["mlp"]["router"], w[p + "mlp.correction"]
+        E, groups, keep = r["experts"], r["groups"]["count"], r["groups"]["keep"]
+        for e in range(E):
+            w[f"{p}mlp.e{e}.down"][-CODES:] = 0.0
+        rows = torch.zeros(E, W)
+        for i in range(CODES - 1):
+            for _ in range(400):
+                col = (torch.linspace(-0.7, 0.7, E)[torch.randperm(E, generator=g)] if E > 1 else torch.ones(1)).bfloat16().float()
+                if all(route_margin(col * amp / f, c, r["top"], groups, keep) > margin for f in torch.linspace(0.88, 1.6, 25).tolist()):
+                    break
+            rows[:, W - CODES + i] = col
+        rows[:, -1] = -rows.sum(1)
+        w[p + "mlp.router"] = rows.bfloat16().float()
