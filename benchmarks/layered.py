@@ -1,9 +1,9 @@
 #!/usr/bin/env python
 """Layer-list decoders beside the closest existing model: Keripel beside the generic-format Qwen3 engine with f16 weights,
-Kekevik beside Keripel.
+Kekevik beside Keripel, Kutepel beside Kekevik.
 
     python benchmarks/layered.py kernels [--width 4096] [--only ..]     the kernels and their counterparts, with roofline fractions
-    python benchmarks/layered.py models --design kekevik [--sizes s,m]  prefill and decode throughput at equal parameter count
+    python benchmarks/layered.py models --design kutepel [--sizes s,m]  prefill and decode throughput at equal parameter count
 
 Random weights, random tokens.  Kernels: CUDA events around a CUDA graph of repeated launches that walks through enough copies
 of its inputs to exceed L2; the roofline is the slower of bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate.
@@ -49,6 +49,21 @@ def kekevik(width: int, repeats: int, vocab: int = 32000) -> dict:
     ret = {"type": "retention", "mlp": ff, "mixer": {"heads": n, "dim": 256, "vdim": 256, "decay": decay(n), "rot": {"base": 10000.0, "dims": 256}}}
     return {"architecture": "Kekevik", "layers": [light, both, both, ret] * repeats, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width,
             "embedding": {"scale": float(width ** 0.5)}}
+
+
+def kutepel(width: int, repeats: int, vocab: int = 32000, n: int = 32, top: int = 4) -> dict:
+    """``repeats`` times two layers of latent attention, one of rotary attention with sinks and one on its keys and values, all with
+    ``n`` experts of a quarter of the width."""
+    H = width // 128
+    moe = {"kind": "moe", "expert": {"ff": width // 4}, "router": {"experts": n, "groups": {"count": 8, "keep": 4}, "scale": 2.5, "top": top}}
+    lat = {"type": "latent_attention", "mlp": moe, "mixer": {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+                                                             "rot": {"base": 10000.0, "dims": 64}}}
+    m = {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+         "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    layers = []
+    for r in range(repeats):
+        layers += [lat, lat, {"type": "attention", "mlp": moe, "mixer": m}, {"type": "attention", "mlp": moe, "mixer": {**m, "kv_from": 4 * r + 2}}]
+    return {"architecture": "Kutepel", "layers": layers, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "vocab": vocab, "width": width}
 
 
 def write_design(path: str, cfg: dict) -> int:
@@ -232,6 +247,199 @@ def bench_capped_attention(rep: Report, width: int, iters: int, profile: bool) -
                 4.0 * T * (T + 1) / 2 * nq * hd)
     fn = lambda: K.check(L.lib().bonsai_lay_attn_append(*c.args, 0, T, 0, K.stream()), "attn_append")
     rep.add("attn_append, K and V", f"T={T}", time_us(fn, iters, profile), 12 * T * nkv * hd)
+
+
+def bench_rotary(rep: Report, width: int, iters: int, profile: bool) -> None:
+    """Rotated heads with sinks; the like kernels are those of bench_capped_attention."""
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    nq, nkv, hd, page = width // 128, max(1, width // 512), 128, 64
+    i32 = dict(dtype=torch.int32, device=dev)
+    ld = (nq + 2 * nkv) * hd
+    rot, sinks = torch.randn(4096, hd // 2, 2, device=dev), torch.ones(nq, device=dev)
+
+    def call(proj, pos, slots, bt, k, v, out):
+        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out, sinks, rot],
+                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0, 0, hd, 1], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0])
+    for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
+        npages = ctx // page
+        copies = max(2, int(300e6 / (4 * B * ctx * nkv * hd)) + 1)
+        pools = [[torch.randn(B * npages, nkv, page, hd, device=dev).bfloat16() for _ in range(2)] for _ in range(copies)]
+        bt = torch.arange(B * npages, **i32).view(B, npages)
+        pos, slots, proj = torch.full((B,), ctx - 1, **i32), torch.arange(B, **i32), torch.randn(B, ld, device=dev)
+        out = torch.zeros(B, nq * hd, dtype=torch.bfloat16, device=dev)
+        calls = [call(proj, pos, slots, bt, *p, out) for p in pools]
+        it, split = [0], 1
+        while split < 8 and B * nkv * split * 2 <= 160:
+            split *= 2
+
+        def ours():
+            it[0] += 1
+            K.check(L.lib().bonsai_lay_attn_decode(*calls[it[0] % copies].args, B, split, K.stream()), "attn_decode")
+        rep.add("attn_decode, rotated, sinks", f"B={B} ctx={ctx} heads={nq}/{nkv}", time_us(ours, iters, profile), 4 * B * ctx * nkv * hd, 4.0 * B * ctx * nq * hd)
+    T, npages = 4096, 64
+    k, v = (torch.randn(npages, nkv, page, hd, device=dev).bfloat16() for _ in range(2))
+    bt, pos, slots = torch.arange(npages, **i32).view(1, -1), torch.arange(T, **i32), torch.zeros(T, **i32)
+    proj, out = torch.randn(T, ld, device=dev), torch.zeros(T, nq * hd, dtype=torch.bfloat16, device=dev)
+    entries = torch.tensor([0, T, 0, 0], **i32)
+    tiles = torch.tensor([[0, t] for t in range(0, T, 64 // (nq // nkv))], **i32)
+    c = call(proj, pos, slots, bt, k, v, out)
+    fn = lambda: K.check(L.lib().bonsai_lay_attn_prompt(*c.args, entries.data_ptr(), tiles.data_ptr(), len(tiles), K.stream()), "attn_prompt")
+    rep.add("attn_prompt, rotated, sinks", f"T={T} heads={nq}/{nkv}", time_us(fn, 10, profile), 4 * T * ld + 4 * T * nkv * hd + 2 * T * nq * hd, 4.0 * T * (T + 1) / 2 * nq * hd)
+    fn = lambda: K.check(L.lib().bonsai_lay_attn_append(*c.args, 0, T, 0, K.stream()), "attn_append")
+    rep.add("attn_append, rotated", f"T={T}", time_us(fn, iters, profile), 12 * T * nkv * hd)
+
+
+def bench_latent(rep: Report, width: int, iters: int, profile: bool, splits: int = 0, cluster: int = 0, prompts: bool = True) -> None:
+    """Latent attention; the like kernels are those of bench_capped_attention (and of bench_linear for the expansion)."""
+    from oxibonsai_b200.models.layered import CONTEXT_TILE
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev, lib = torch.device("cuda"), L.lib()
+    nq, dim, rot, vd, rank, page = width // 128, 128, 64, 128, 512, 64
+    row, i32, bf16 = lib.bonsai_lay_latent_row(rank, rot), dict(dtype=torch.int32, device=dev), dict(dtype=torch.bfloat16, device=dev)
+    q_w, g_w = nq * (dim + rot), nq * vd
+    ld = q_w + rank + rot + g_w
+    table, ones, sms = torch.randn(4096, rot // 2, 2, device=dev), torch.ones(rank, device=dev), torch.cuda.get_device_properties(dev).multi_processor_count
+
+    def call(T, pos, slots, bt, pool, keys, values, parts):
+        proj, out = torch.randn(T, ld, device=dev), torch.zeros(T, g_w, **bf16)
+        n = min(T, 256)
+        return L.MixerCall([proj, ones, table, pos, slots, bt, pool, keys, values, torch.randn(n, nq, row, device=dev).bfloat16() * 0.01,
+                            torch.zeros(parts, nq, rank, device=dev), torch.ones(parts, nq, 2, device=dev), torch.zeros(1, **i32), out],
+                           [ld, 0, q_w, q_w + rank, q_w + rank + rot, g_w, nq, dim, rot, vd, rank, bt.shape[1], page, n, parts, pool.shape[0]],
+                           [1e-6, 192 ** -0.5, 1.0])
+    for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
+        npages = ctx // page
+        copies = max(2, int(300e6 / (2 * B * ctx * row)) + 1)
+        bt = torch.arange(B * npages, **i32).view(B, npages)
+        pos, slots = torch.full((B,), ctx - 1, **i32), torch.arange(B, **i32)
+        wcopies = int(300e6 / (2 * nq * rank * dim)) + 1
+        ws = [[torch.randn(nq, rank, dim, device=dev).bfloat16() * 0.05, torch.randn(nq, vd, rank, device=dev).bfloat16() * 0.05] for _ in range(wcopies)]
+        groups = -(-nq // lib.bonsai_lay_latent_group(nq))
+        n = 1
+        while 2 * n <= min(lib.bonsai_lay_latent_max_splits(), sms // (B * groups), -(-ctx // 64)):
+            n *= 2
+        n, cl = splits or n, min(splits or n, cluster or (lib.bonsai_lay_latent_max_cluster() if B * groups * n <= 64 else 4))
+        calls = [call(B, pos, slots, bt, torch.randn(B * npages, page, row, device=dev).bfloat16(), *ws[i % wcopies], B * (n // cl)) for i in range(copies)]
+        wcalls = [call(B, pos, slots, bt, torch.zeros(B * npages, page, row, **bf16), *w, B * (n // cl)) for w in ws]
+        it = [0]
+
+        def turn(fn, among):
+            def run():
+                it[0] += 1
+                fn(among[it[0] % len(among)].args)
+            return run
+        query = turn(lambda a: K.check(lib.bonsai_lay_latent_query(*a, B, K.stream()), "latent_query"), wcalls)
+        decode = turn(lambda a: K.check(lib.bonsai_lay_latent_decode(*a, B, n, cl, K.stream()), "latent_decode"), calls)
+        value = turn(lambda a: K.check(lib.bonsai_lay_latent_value(*a, B, n // cl, K.stream()), "latent_value"), wcalls)
+        case = f"B={B} ctx={ctx} heads={nq} {rank}+{rot} splits={n}/{cl}"
+        rep.add("latent_query", case, time_us(query, iters, profile), 2 * nq * rank * dim + 4 * B * ld + 2 * B * nq * row, 2.0 * B * nq * rank * dim)
+        rep.add("latent_decode", case, time_us(decode, iters, profile), 2 * B * ctx * row, 2.0 * B * ctx * nq * (2 * rank + rot))
+        rep.add("latent_value", case, time_us(value, iters, profile), 2 * nq * rank * vd + 4 * B * (n // cl) * nq * rank, 2.0 * B * nq * rank * vd)
+
+        def both():
+            it[0] += 1
+            a, w = calls[it[0] % copies].args, wcalls[it[0] % wcopies].args
+            K.check(lib.bonsai_lay_latent_query(*w, B, K.stream()), "latent_query")
+            K.check(lib.bonsai_lay_latent_decode(*a, B, n, cl, K.stream()), "latent_decode")
+            K.check(lib.bonsai_lay_latent_value(*w, B, n // cl, K.stream()), "latent_value")
+        rep.add("latent, one step", case, time_us(both, iters, profile), 2 * B * ctx * row + 4 * nq * rank * dim, 2.0 * B * ctx * nq * (2 * rank + rot))
+        del calls, wcalls
+    if not prompts:
+        return
+    T, npages, ldkv = 4096, 64, nq * (dim + vd)
+    bt, pos, slots = torch.arange(npages, **i32).view(1, -1), torch.arange(T, **i32), torch.zeros(T, **i32)
+    c = call(T, pos, slots, bt, torch.randn(npages, page, row, device=dev).bfloat16(), *ws[0], 256)
+    entries, context = torch.tensor([0, T, 0, 0], **i32), torch.tensor([0, T, 0, 0], **i32)
+    tiles = torch.tensor([[0, t] for t in range(0, T, CONTEXT_TILE)], **i32)
+    lat, kv = torch.randn(T, row, device=dev).bfloat16(), torch.randn(T, ldkv, device=dev).bfloat16()
+    fn = lambda: K.check(lib.bonsai_lay_latent_append(*c.args, 0, T, 0, K.stream()), "latent_append")
+    rep.add("latent_append", f"T={T}", time_us(fn, iters, profile), 6 * T * (rank + rot))
+    fn = lambda: K.check(lib.bonsai_lay_latent_gather(*c.args, context.data_ptr(), 1, T, lat.data_ptr(), row, K.stream()), "latent_gather")
+    rep.add("latent_gather", f"T={T}", time_us(fn, iters, profile), 4 * T * row)
+    w, scratch = L.DenseWeight([torch.randn(ldkv, rank).bfloat16()], dev), L.GemmScratch(dev, torch.zeros(1, dtype=torch.int32, device=dev))
+    rep.add("linear, bf16 out", f"expand {ldkv}x{rank} T={T}", time_us(lambda: L.linear(w, lat, T, kv, scratch), 10, profile), 2 * T * ldkv + 2 * T * rank + 2 * ldkv * rank,
+            2.0 * T * ldkv * rank)
+    kv.normal_()
+    fn = lambda: K.check(lib.bonsai_lay_latent_prompt(*c.args, entries.data_ptr(), context.data_ptr(), tiles.data_ptr(), len(tiles), kv.data_ptr(), ldkv, lat.data_ptr(), row,
+                                                      K.stream()), "latent_prompt")
+    rep.add("latent_prompt", f"T={T} heads={nq} {dim}+{rot}, {vd}", time_us(fn, 10, profile), 4 * T * (q_w + g_w) + 2 * T * (ldkv + rot) + 2 * T * g_w,
+            2.0 * T * (T + 1) / 2 * nq * (dim + rot + vd))
+
+
+def bench_experts(rep: Report, width: int, iters: int, profile: bool) -> None:
+    """Router and experts; the like kernels are the gate/up, down and residual cases of bench_linear and bench_recurrence."""
+    from oxibonsai_b200.models.layered_config import ExpertsSpec, RouterSpec
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    scratch = L.GemmScratch(dev, torch.zeros(1, dtype=torch.int32, device=dev))
+    for E, top, ff in ((32, 4, width // 4), (128, 8, width // 4)):
+        spec = ExpertsSpec(RouterSpec(E, top, 8, 4, 2.5), ff)
+        s = L.ExpertScratch(4096, width, [spec], False, dev)
+        logits = torch.randn(4096, E, device=dev)
+
+        def matrix(n, k):
+            w = L.DenseWeight([torch.zeros(8, k, dtype=torch.bfloat16)], dev)
+            w.n, w.data = E * n, torch.empty(E * n, k, dtype=torch.bfloat16, device=dev).normal_(std=k ** -0.5)
+            return w
+        r = L.Routing(spec, matrix(2 * ff, width), matrix(width, ff), torch.zeros(E, device=dev), logits, 0, s)
+        h = torch.randn(4096, width, device=dev).bfloat16()
+        x, y, x16, norm = torch.zeros(4096, width, device=dev), torch.randn(4096, width, device=dev), torch.zeros(4096, width, dtype=torch.bfloat16, device=dev), torch.ones(width, device=dev)
+        lib, it = L.lib(), [0]
+        for T in (1, 8, 32, 64, 256, 1024, 4096):
+            if 8 * T * top < E and T > 8:
+                continue
+            pairs, few, st, hid = T * top, r.few(T), K.stream, s.hidden[ff]
+            xs = None if few else s.sorted
+
+            def route():
+                K.check(lib.bonsai_lay_route(*r.call.args, T, h.data_ptr(), h.stride(0), width // 8 if xs is not None else 0, K.ptr(xs), 0 if xs is None else xs.stride(0), st()),
+                        "route")
+                s.counts.zero_()
+            # distinct logits per turn, so that the chosen experts' weights are not in L2 from the turn before
+            lists = []
+            for _ in range(8):
+                logits.normal_()
+                route()
+                lists.append([t.clone() for t in (s.lists, s.token, s.weight)])
+            chosen = sum(int(l[0][E + 1]) for l in lists) / len(lists)
+            case, like = f"T={T} {top} of {E} experts, {ff} units, {'few' if few else 'tiles'}", 2 * ff * width
+
+            def route_only():
+                K.check(lib.bonsai_lay_route(*r.call.args, T, h.data_ptr(), h.stride(0), width // 8 if xs is not None else 0, K.ptr(xs), 0 if xs is None else xs.stride(0), st()),
+                        "route")
+                if xs is not None or T > lib.bonsai_lay_route_small(top):
+                    L.side_by_side(x, y, r, 0.0, 1, None, None, 1e-6, True)          # a row of it: leaves the counters zero
+            rep.add("route", case, time_us(route_only, iters, profile), 4 * T * E + (2 * (T + pairs) * width if xs is not None else 0))
+
+            def up():
+                it[0] += 1
+                li, tok, wt = lists[it[0] % 8]
+                if few:
+                    K.check(lib.bonsai_lay_experts_few(r.up.data.data_ptr(), E, 2 * ff, width, h.data_ptr(), width, li.data_ptr(), tok.data_ptr(), wt.data_ptr(), pairs,
+                                                       min(E, pairs), min(T, 2 * pairs // E + 8), hid.data_ptr(), ff, 1, float("inf"), 1.0, 0.0, st()), "experts_few")
+                else:
+                    K.check(lib.bonsai_grouped_gemm_bf16(r.up.data.data_ptr(), E, 2 * ff, width, xs.data_ptr(), width, pairs, li.data_ptr(), wt.data_ptr(), hid.data_ptr(), ff, 4,
+                                                         float("inf"), 1.0, 0.0, int(pairs > 96 * E), scratch.status.data_ptr(), scratch.sms, st()), "grouped_gemm")
+
+            def down():
+                it[0] += 1
+                li = lists[it[0] % 8][0]
+                if few:
+                    K.check(lib.bonsai_lay_experts_few(r.down.data.data_ptr(), E, width, ff, hid.data_ptr(), ff, li.data_ptr(), None, None, pairs, min(E, pairs),
+                                                       min(T, 2 * pairs // E + 8), s.out32.data_ptr(), s.out32.stride(0), 0, 0.0, 0.0, 0.0, st()), "experts_few")
+                else:
+                    K.check(lib.bonsai_grouped_gemm_bf16(r.down.data.data_ptr(), E, width, ff, hid.data_ptr(), ff, pairs, li.data_ptr(), None, s.out.data_ptr(), s.out.stride(0), 6,
+                                                         0.0, 0.0, 0.0, int(pairs > 96 * E), scratch.status.data_ptr(), scratch.sms, st()), "grouped_gemm")
+            rep.add("experts, gate/up", case, time_us(up, iters, profile), chosen * 2 * like + 2 * (T if few else pairs) * width + 2 * pairs * ff, 4.0 * pairs * ff * width)
+            rep.add("experts, down", case, time_us(down, iters, profile), chosen * like + 2 * pairs * ff + (4 if few else 2) * pairs * width, 2.0 * pairs * ff * width)
+            r.out = s.out32 if few else s.out
+            fn = lambda: L.side_by_side(x, y, r, 0.5, T, x16, norm, 1e-6, True)
+            rep.add("side_by_side", case, time_us(fn, iters, profile), (14.0 * T + (4 if few else 2) * pairs) * width)
+        del r, s
 
 
 def bench_recurrence(rep: Report, width: int, iters: int, profile: bool) -> None:
@@ -437,6 +645,40 @@ def run_kekevik(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, bat
     return rows
 
 
+def active_params(cfg: dict) -> int:
+    """Parameters a token uses: all but the experts that are not chosen."""
+    from oxibonsai_b200.models.registry import ARCHITECTURES
+    c = ARCHITECTURES[cfg["architecture"]](cfg, "")
+    idle = sum(3 * c.experts(i).ff * c.width * (c.experts(i).router.experts - c.experts(i).router.top) for i in c.expert_layers)
+    return c.param_count() - idle
+
+
+def run_kutepel(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64), log=sys.stdout) -> list[dict]:
+    """Kutepel beside Kekevik of the same width with as many layers as bring it to the same parameter count, and to the count that a
+    token of Kutepel uses."""
+    rows = []
+    for size in sizes:
+        width, repeats = SIZES[size]["width"], {"s": 1, "m": 1, "l": 1}[size]
+        cfg = kutepel(width, repeats)
+        row = {"size": size, "width": width, "kutepel_layers": len(cfg["layers"]), "active_params_M": round(active_params(cfg) / 1e6)}
+        with tempfile.TemporaryDirectory() as d:
+            row["params_M"] = round(write_design(os.path.join(d, "m"), cfg) / 1e6)
+            row["kutepel"] = measure_layered(os.path.join(d, "m"), steps, warmup, prompt, batches)
+        torch.cuda.empty_cache()
+        for name, target in (("kekevik", row["params_M"]), ("kekevik_active", row["active_params_M"])):
+            with tempfile.TemporaryDirectory() as d:
+                count = lambda n: write_design(os.path.join(d, "m"), kekevik(width, n))
+                one, two = count(1), count(2)
+                cfg = kekevik(width, max(1, round((target * 1e6 - one) / (two - one)) + 1))
+                params = write_design(os.path.join(d, "m"), cfg)
+                row[f"{name}_layers"], row[f"{name}_params_M"] = len(cfg["layers"]), round(params / 1e6)
+                row[name] = measure_layered(os.path.join(d, "m"), steps, warmup, prompt, batches)
+            torch.cuda.empty_cache()
+        rows.append(row)
+        print(json.dumps(row), file=log, flush=True)
+    return rows
+
+
 def run_models(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64), log=sys.stdout) -> list[dict]:
     from oxibonsai_b200.cli import requantize_gguf
     from oxibonsai_b200.core import Qwen3Config, write_synthetic_gguf
@@ -469,19 +711,19 @@ def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("case", choices=["kernels", "models"])
     ap.add_argument("--width", type=int, default=4096)
-    ap.add_argument("--only", default="linear,attention,mlstm,capped,recurrence")
-    ap.add_argument("--design", choices=["keripel", "kekevik"], default="kekevik")
+    ap.add_argument("--only", default="linear,attention,mlstm,capped,recurrence,rotary,latent,experts")
+    ap.add_argument("--design", choices=["keripel", "kekevik", "kutepel"], default="kutepel")
     ap.add_argument("--iters", type=int, default=40)
     ap.add_argument("--sizes", default="s,m,l")
     ap.add_argument("--profile", action="store_true", help="a few eager launches per case, for captures under a profiler")
     a = ap.parse_args()
     torch.cuda.set_device(0)
     if a.case == "models":
-        (run_kekevik if a.design == "kekevik" else run_models)(a.sizes.split(","))
+        {"keripel": run_models, "kekevik": run_kekevik, "kutepel": run_kutepel}[a.design](a.sizes.split(","))
         return
     rep = Report()
     for name, fn in (("linear", bench_linear), ("attention", bench_attention), ("mlstm", bench_mlstm), ("capped", bench_capped_attention),
-                     ("recurrence", bench_recurrence)):
+                     ("recurrence", bench_recurrence), ("rotary", bench_rotary), ("latent", bench_latent), ("experts", bench_experts)):
         if name in a.only.split(","):
             fn(rep, a.width, a.iters, a.profile)
 

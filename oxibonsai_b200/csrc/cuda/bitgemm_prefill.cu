@@ -14,7 +14,8 @@
 //   * tcgen05.mma kind::f16 accumulates in TMEM (double buffered so the epilogue of one segment overlaps the main
 //     loop of the next); 64-token tiles spread the MMA and TMA issue over four warps each, one per pipeline slot,
 //     every MMA issuer with its own accumulator (the comments at the issuer loops give the measurements behind it);
-//   * epilogue warps read TMEM back and store f32 (plain / residual add) or f16 (SwiGLU / plain) outputs.
+//   * epilogue warps read TMEM back and store f32 (plain / residual add) or f16 (SwiGLU / plain) outputs: four of them, or with dense
+//     weights and whole tiles up to sixteen, those that have nothing to expand.
 //
 // Work distribution ("stream-K"): the (tile, k-block pair) index space is cut into one contiguous, equally long
 // range per CTA, so every SM streams the same number of weight bytes whatever the tile count (32 row tiles of a
@@ -25,7 +26,10 @@
 //
 // Grouped form (dense operands): the rows of X belong to groups (the experts of a mixture), group g to the rows offsets[g] ..
 // offsets[g + 1] - 1, and each group has its own weight matrix, one below the other.  The offsets are made on the device, so every
-// CTA derives the tile list (groups in order, 128 weight rows x TOK rows of one group) from them and takes an equal share of it.
+// CTA derives the tile list (groups in order, 128 weight rows x TOK rows of one group) from them.
+//
+// Whole tiles of dense operands go round robin to the CTAs, those that share weight rows one after another: what the CTAs work on at
+// a time then stays in L2, where contiguous ranges per CTA read the operands many times from memory.
 //
 // K order: the expansion naturally yields the weights of a 16-input word in the order
 // [0,4,1,5,2,6,3,7, 8,12,9,13,10,14,11,15]; instead of un-shuffling them the activation operand is
@@ -66,12 +70,12 @@ struct PfParams {
   __half* out_f16;         // [T][out_ld]  (epi 2: SwiGLU, paired-K order; epi 3: plain f16 store)
   int* status;
   int n_rows, K, T, epi, out_ld;
-  int dense;               // 1: A is a dense f16 / bf16 matrix fetched by TMA (natural K order), no expansion
   int bf16;                // dense operands are bf16 (both) instead of f16
   float glu_limit, glu_alpha, glu_offset;   // epi 4
   const float* row_scale;  // epi 4, grouped: factor of a row's outputs
   const int* offsets;      // grouped: [groups + 1] first row of every group (device memory)
   int groups;
+  int quartets;            // dense, whole tiles: quartets of warps that share the epilogue (1, 2 or 4)
   int streamk;             // 1: ranges cut anywhere in (tile, pair) space, partial tiles meet in the workspace
   float* ws_part;          // [2 * grid][TOK][128] partial accumulators
   int* ws_count;           // [tiles] arrival counters, zero between launches
@@ -155,7 +159,12 @@ __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, 
 template <int CB, bool SCALED = false>
 __device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, int tok0, int tend, int row, int a, bool row_ok) {
   const bool odd = a & 1;
-  float o[CB / 2];
+  float o[CB / 2], scale[CB / 2];
+#pragma unroll
+  for (int j = 0; j < CB / 2; ++j) {
+    const int tok = tok0 + 2 * j + (odd ? 1 : 0);
+    scale[j] = SCALED && tok < tend ? p.row_scale[tok] : 1.0f;
+  }
 #pragma unroll
   for (int j = 0; j < CB / 2; ++j) {
     const float keep = odd ? v[2 * j + 1] : v[2 * j];
@@ -168,7 +177,30 @@ __device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, 
 #pragma unroll
   for (int j = 0; j < CB / 2; ++j) {
     const int tok = tok0 + 2 * j + (odd ? 1 : 0);
-    if (row_ok && tok < tend) dst[(size_t)tok * p.out_ld] = __float2bfloat16_rn(SCALED ? o[j] * p.row_scale[tok] : o[j]);
+    if (row_ok && tok < tend) dst[(size_t)tok * p.out_ld] = __float2bfloat16_rn(SCALED ? o[j] * scale[j] : o[j]);
+  }
+}
+
+// Epilogues 5 and 6: bf16 outputs.  The two lanes of a pair exchange columns, so that each stores two neighbouring rows of every
+// other column, at once where they are aligned.
+template <int CB>
+__device__ __forceinline__ void pf_store_bf16(const PfParams& p, const float* v, int tok0, int tend, int row, int a) {
+  const bool odd = a & 1;
+  const bool vec = ((p.out_ld & 1) | (int)(reinterpret_cast<uintptr_t>(p.out_f16) & 2)) == 0;
+  const int r0 = row & ~1;
+  __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out_f16) + (size_t)(tok0 + (odd ? 1 : 0)) * p.out_ld + r0;
+#pragma unroll
+  for (int j = 0; j < CB / 2; ++j) {
+    const float keep = odd ? v[2 * j + 1] : v[2 * j];
+    const float other = __shfl_xor_sync(0xffffffffu, odd ? v[2 * j] : v[2 * j + 1], 1);
+    const __nv_bfloat162 both = odd ? __floats2bfloat162_rn(other, keep) : __floats2bfloat162_rn(keep, other);
+    if (tok0 + 2 * j + (odd ? 1 : 0) >= tend) continue;
+    if (vec && r0 + 1 < p.n_rows) {
+      *reinterpret_cast<__nv_bfloat162*>(dst + (size_t)(2 * j) * p.out_ld) = both;
+    } else {
+      if (r0 < p.n_rows) dst[(size_t)(2 * j) * p.out_ld] = both.x;
+      if (r0 + 1 < p.n_rows) dst[(size_t)(2 * j) * p.out_ld + 1] = both.y;
+    }
   }
 }
 
@@ -188,12 +220,13 @@ __device__ __forceinline__ PfTile pf_group_tile(const PfParams& p, const int* fi
     if (first[mid] <= tile) lo = mid;
     else hi = mid - 1;
   }
-  const int in = tile - first[lo], row0 = (in % row_tiles) * 128;
-  return PfTile{lo * p.n_rows + row0, row0, off[lo] + (in / row_tiles) * tok_per_tile, off[lo + 1]};
+  const int in = tile - first[lo], tok_tiles = (first[lo + 1] - first[lo]) / row_tiles, row0 = (in / tok_tiles) * 128;
+  return PfTile{lo * p.n_rows + row0, row0, off[lo] + (in % tok_tiles) * tok_per_tile, off[lo + 1]};
 }
 
-// TOK = tokens per tile (MMA N): 256 for prompt chunks, 64 for batched decode / verification.
-template <int TOK, bool GROUPED = false>
+// TOK = tokens per tile (MMA N): 256 for prompt chunks, 64 for batched decode / verification.  DENSE: A is a dense f16 / bf16 matrix
+// fetched by TMA (natural K order), no expansion.
+template <int TOK, bool DENSE, bool GROUPED = false>
 __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __grid_constant__ CUtensorMap xmap,
                                                                      const __grid_constant__ CUtensorMap amap, PfParams p) {
   constexpr int S = TOK == 64 ? 8 : 4;   // pipeline stages (one 64-input k-block each)
@@ -211,6 +244,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
   uint8_t* base = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* sA = base;
   uint8_t* sB = base + S * kPfABytes;
+  const bool fan = DENSE && !p.streamk;     // the expander warps are the epilogue
   __shared__ uint64_t full_bar[S], empty_bar[S], accf_bar[2], acce_bar[2];
   __shared__ uint32_t tmem_slot;
   __shared__ int s_info[4];
@@ -246,12 +280,14 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
   }
   auto tile_at = [&](int tile) {
     if (GROUPED) return pf_group_tile(p, s_first, s_off, tile, row_tiles, TOK);
-    const int row0 = (tile % row_tiles) * 128;
-    return PfTile{row0, row0, (tile / row_tiles) * TOK, p.T};
+    const int row0 = (fan ? tile / tok_tiles : tile % row_tiles) * 128;
+    return PfTile{row0, row0, (fan ? tile % tok_tiles : tile / row_tiles) * TOK, p.T};
   };
   const long long I0 = pf_range_start(p.streamk, blockIdx.x, grid, ntiles, npairs);
-  const int n = (int)(pf_range_start(p.streamk, blockIdx.x + 1, grid, ntiles, npairs) - I0);   // pairs of this CTA
-  const int tile0 = (int)(I0 / npairs), pair0 = (int)(I0 - (long long)tile0 * npairs);
+  // pairs of this CTA, its first tile and pair, and the distance to its next tile
+  const int n = fan ? max(0, (ntiles - (int)blockIdx.x + grid - 1) / grid) * npairs
+                    : (int)(pf_range_start(p.streamk, blockIdx.x + 1, grid, ntiles, npairs) - I0);
+  const int tile0 = fan ? blockIdx.x : (int)(I0 / npairs), pair0 = fan ? 0 : (int)(I0 - (long long)tile0 * npairs), step = fan ? grid : 1;
 
   // Programmatic dependent launch: this CTA may start while the previous kernel of the stream is still running.  Set-up,
   // TMEM allocation and the expanders' first weight loads depend on nothing it writes; the warps that touch its outputs
@@ -263,12 +299,12 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
   }
   if (t == 0) {
     for (int i = 0; i < S; ++i) {
-      tc::mbar_init(&full_bar[i], p.dense ? 1 : 4 * GK + 1);   // four expander warps per k-block + the TMA issuer's expect_tx arrival
+      tc::mbar_init(&full_bar[i], DENSE ? 1 : 4 * GK + 1);   // four expander warps per k-block + the TMA issuer's expect_tx arrival
       tc::mbar_init(&empty_bar[i], 1);
     }
     for (int i = 0; i < 2; ++i) {
       tc::mbar_init(&accf_bar[i], NISS);
-      tc::mbar_init(&acce_bar[i], 4);
+      tc::mbar_init(&acce_bar[i], fan ? 4 * p.quartets : 4);
     }
     tc::mbar_init(&red_bar, 1);
     tc::mbar_fence_init();
@@ -304,18 +340,18 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
           const int it = 2 * q + g0, bs = (it / GK) % NBS;
           if (!__all_sync(0xffffffffu, tc::mbar_wait(&empty_bar[bs], (((it / GK) / NBS) & 1) ^ 1))) { failed = true; break; }
           if (lane == 0) {
-            tc::mbar_arrive_expect_tx(&full_bar[bs], GK * (kPfBBytes + (p.dense ? kPfABytes : 0)));
+            tc::mbar_arrive_expect_tx(&full_bar[bs], GK * (kPfBBytes + (DENSE ? kPfABytes : 0)));
 #pragma unroll
             for (int h = 0; h < GK; ++h) {
               const int s = (it + h) % S, kb = 2 * pair + g0 + h;
               tma_load_2d(sB + s * kPfBBytes, &xmap, kb * 64, tok0, &full_bar[bs]);
-              if (p.dense) tma_load_2d(sA + s * kPfABytes, &amap, kb * 64, row0, &full_bar[bs]);
+              if (DENSE) tma_load_2d(sA + s * kPfABytes, &amap, kb * 64, row0, &full_bar[bs]);
             }
           }
           __syncwarp();
         }
       }
-      if (++pair == npairs) { pair = 0; ++tile; }
+      if (++pair == npairs) { pair = 0; tile += step; }
     }
     if (failed && lane == 0) atomicExch(p.status, 1);
   } else if (warp >= kPfMmaWarp && warp < kPfMmaWarp + NISS) {
@@ -378,7 +414,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
     constexpr int NPG = 2;   // pair-groups
     constexpr int NV = 2 / KH;               // 16-byte code vectors per thread and pair
     static_assert((S / 2) % NPG == 0, "a pair of stages is always refilled by the same group");
-    if (!p.dense && warp < 4 * KH * NPG) {
+    if (!DENSE && warp < 4 * KH * NPG) {
       const int pg = warp / (4 * KH), hh0 = KH == 2 ? (warp >> 2) & 1 : 0, r = t & 127;
       // a thread's loads walk one weight row per tile: a dependent chain of cache misses unless several are in
       // flight, so the codes of kPfAhead of its pairs (NPG * kPfAhead pairs of the CTA) are requested ahead of use
@@ -430,7 +466,80 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
       }
       if (failed && lane == 0) atomicExch(p.status, 1);
     }
-  } else if (warp < kPfMmaWarp) {
+    if (DENSE && fan && warp < 4 * p.quartets) {
+      // ----------------------------- epilogue of whole tiles (thread = weight row, a quarter of the columns) ----
+      constexpr int CB = 16;
+      const int NC = TOK / p.quartets;
+      asm volatile("griddepcontrol.wait;" ::: "memory");
+      const int a = t & 127, cq = (warp >> 2) * NC;
+      const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
+      int seg = 0;
+      for (int q = 0; q < n && !failed; q += npairs, ++seg) {
+        const int ab = seg & 1;
+        const PfTile tl = tile_at(tile0 + seg * step);
+        const int row = tl.row0 + a, tok0 = tl.tok0, tend = tl.tend;
+        const bool row_ok = row < p.n_rows;
+        const int ncols = min(TOK, tend - tok0);
+        if (!tc::mbar_wait_warp<64>(&accf_bar[ab], (seg >> 1) & 1, lane)) { failed = true; break; }
+        tc::tc_fence_after();
+#pragma unroll 1
+        for (int c0 = cq; c0 < cq + NC && c0 < ncols; c0 += CB) {
+          float v[CB];
+          {
+            uint32_t rr[CB];
+            if (NACC == 1) {
+              tc::tmem_ld16(taddr + lane_base + ab * kAccCols + c0, rr);
+              tc::tmem_wait_ld();
+            } else {
+#pragma unroll
+              for (int j = 0; j < CB; ++j) rr[j] = 0u;
+            }
+#pragma unroll
+            for (int j = 0; j < CB; ++j) v[j] = __uint_as_float(rr[j]);
+          }
+#pragma unroll
+          for (int acc = 0; acc < (NACC == 1 ? 0 : NACC); ++acc) {
+            if (npairs < NACC && ((acc - q) & (NACC - 1)) >= npairs) continue;   // that issuer had no pair of this tile
+            uint32_t r2[CB];
+            tc::tmem_ld16(taddr + lane_base + ab * kAccCols + acc * TOK + c0, r2);
+            tc::tmem_wait_ld();
+#pragma unroll
+            for (int j = 0; j < CB; ++j) v[j] += __uint_as_float(r2[j]);
+          }
+          const int tok = tok0 + c0;
+          if (p.epi == 4) {
+            pf_store_glu<CB, GROUPED>(p, v, tok, tend, row, a, row_ok);
+          } else if (p.epi == 6 || p.epi == 5) {
+#pragma unroll
+            for (int j = 0; j < CB; ++j)
+              if (p.epi == 5) v[j] = fmaxf(v[j], 0.0f) * fmaxf(v[j], 0.0f);
+            pf_store_bf16<CB>(p, v, tok, tend, row, a);
+          } else if (p.epi == 0) {
+            float* dst = p.out_f32 + (size_t)tok * p.out_ld + row;
+            if (tok + CB <= tend) {
+#pragma unroll
+              for (int j = 0; j < CB; ++j)
+                if (row_ok) dst[(size_t)j * p.out_ld] = v[j];
+            } else {
+#pragma unroll
+              for (int j = 0; j < CB; ++j)
+                if (row_ok && tok + j < tend) dst[(size_t)j * p.out_ld] = v[j];
+            }
+          } else {
+            float res[CB];
+#pragma unroll
+            for (int j = 0; j < CB; ++j) res[j] = pf_residual(p, tok + j, row, row_ok);
+#pragma unroll
+            for (int j = 0; j < CB; ++j) pf_store(p, v[j], res[j], tok + j, tend, row, a, row_ok);
+          }
+        }
+        tc::tc_fence_before();
+        __syncwarp();
+        if (lane == 0) tc::mbar_arrive(&acce_bar[ab]);
+      }
+      if (failed && lane == 0) atomicExch(p.status, 1);
+    }
+  } else if (warp < kPfMmaWarp && !fan) {
     // ------------------------------- epilogue (thread = weight row) ------------------------------
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const int a = t - kPfExpThreads;
@@ -623,6 +732,11 @@ __global__ void norm_to_f16_paired_kernel(const float* __restrict__ x, int x_ld,
 
 }  // namespace bonsai
 
+// Quartets of warps that share the epilogue of dense whole tiles: while a long main loop hides it, more warps only take issue slots from
+// the issuers (4096-token gate/up GEMM, K = 4096: 666 us with one, 712 with two, 749 with four); behind a short one they pay (grouped
+// down projection, K = 1024: 186, 176, 164 us).
+static int epilogue_quartets(int K) { return K >= 4096 ? 1 : (K >= 2048 ? 2 : 4); }
+
 static bool make_map_f16(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer, uint64_t ld_elems, uint32_t box_rows,
                          CUtensorMapDataType type = CU_TENSOR_MAP_DATA_TYPE_FLOAT16) {
   cuuint64_t dims[2] = {(cuuint64_t)inner, (cuuint64_t)outer};
@@ -634,7 +748,7 @@ static bool make_map_f16(CUtensorMap* map, const void* base, uint64_t inner, uin
                                 CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int TOK>
+template <int TOK, bool DENSE>
 static int launch_prefill(const CUtensorMap& xmap, const CUtensorMap& amap, bonsai::PfParams p, int sms, void* ws, size_t ws_bytes,
                           int balance, cudaStream_t stream) {
   using namespace bonsai;
@@ -659,9 +773,9 @@ static int launch_prefill(const CUtensorMap& xmap, const CUtensorMap& amap, bons
   p.ws_count = static_cast<int*>(ws);
   p.ws_part = ws != nullptr ? reinterpret_cast<float*>(static_cast<char*>(ws) + kPfCounterBytes) : nullptr;
   size_t smem = 1024 + (size_t)S * (kPfABytes + TOK * 128);
-  cudaError_t e = cudaFuncSetAttribute(bitgemm_prefill_kernel<TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t e = cudaFuncSetAttribute(bitgemm_prefill_kernel<TOK, DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return BONSAI_CUDA_LAUNCH_FAILED;
-  e = launch_pdl(bitgemm_prefill_kernel<TOK>, dim3(grid), dim3(kPfThreads), smem, stream, xmap, amap, p);
+  e = launch_pdl(bitgemm_prefill_kernel<TOK, DENSE>, dim3(grid), dim3(kPfThreads), smem, stream, xmap, amap, p);
   return e == cudaSuccess ? BONSAI_CUDA_OK : BONSAI_CUDA_LAUNCH_FAILED;
 }
 
@@ -695,9 +809,12 @@ int bonsai_bitgemm_prefill_ws(const void* codes, const void* scales, const void*
     amap = xmap;
   }
   PfParams p{(const uint32_t*)codes, (const __half*)scales, out_f32, residual, (__half*)out_f16, status, n_rows, K, T, epi, out_ld,
-             dense_w != nullptr ? 1 : 0, 0, 0.0f, 0.0f, 0.0f, nullptr, nullptr, 0, 0, nullptr, nullptr};
-  return tok == 64 ? launch_prefill<64>(xmap, amap, p, sms, ws, ws_bytes, balance, stream)
-                   : launch_prefill<256>(xmap, amap, p, sms, ws, ws_bytes, balance, stream);
+             0, 0.0f, 0.0f, 0.0f, nullptr, nullptr, 0, epilogue_quartets(K), 0, nullptr, nullptr};
+  if (dense_w != nullptr)
+    return tok == 64 ? launch_prefill<64, true>(xmap, amap, p, sms, ws, ws_bytes, balance, stream)
+                     : launch_prefill<256, true>(xmap, amap, p, sms, ws, ws_bytes, balance, stream);
+  return tok == 64 ? launch_prefill<64, false>(xmap, amap, p, sms, ws, ws_bytes, balance, stream)
+                   : launch_prefill<256, false>(xmap, amap, p, sms, ws, ws_bytes, balance, stream);
 }
 
 // Dense bf16 operands: W [n_rows][K] (K a multiple of 128), x [T][x_ld], f32 accumulation.  epi 0: out_f32 = W x; 4: out_bf16 =
@@ -707,15 +824,16 @@ int bonsai_dense_gemm_bf16(const void* w, int n_rows, int K, const void* x, int 
                            float limit, float alpha, float offset, int* status, void* ws, size_t ws_bytes, int sms, cudaStream_t stream) {
   using namespace bonsai;
   if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && epi != 4 && epi != 5 && epi != 6)) return BONSAI_CUDA_BAD_ARG;
-  if ((epi == 0 && out_f32 == nullptr) || (epi != 0 && out_bf16 == nullptr) || (epi == 4 && n_rows % 2 != 0) || status == nullptr) return BONSAI_CUDA_BAD_ARG;
+  if ((epi == 0 && out_f32 == nullptr) || (epi != 0 && out_bf16 == nullptr) || (epi == 4 && n_rows % 2 != 0) || status == nullptr)
+    return BONSAI_CUDA_BAD_ARG;
   const int tok = T <= 64 ? 64 : 256;
   CUtensorMap xmap, amap;
   if (!make_map_f16(&xmap, x, K, T, x_ld, tok, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
       !make_map_f16(&amap, w, K, n_rows, K, 128, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
     return BONSAI_CUDA_BAD_ARG;
-  PfParams p{nullptr, nullptr, out_f32, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, 1, limit, alpha, offset, nullptr, nullptr, 0, 0, nullptr, nullptr};
-  return tok == 64 ? launch_prefill<64>(xmap, amap, p, sms, ws, ws_bytes, 1, stream)
-                   : launch_prefill<256>(xmap, amap, p, sms, ws, ws_bytes, 1, stream);
+  PfParams p{nullptr, nullptr, out_f32, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, limit, alpha, offset, nullptr, nullptr, 0, epilogue_quartets(K), 0, nullptr, nullptr};
+  return tok == 64 ? launch_prefill<64, true>(xmap, amap, p, sms, ws, ws_bytes, 1, stream)
+                   : launch_prefill<256, true>(xmap, amap, p, sms, ws, ws_bytes, 1, stream);
 }
 
 // Grouped dense bf16 product: W [groups][n_rows][K] (K a multiple of 128), x [T][x_ld] whose rows offsets[g] .. offsets[g + 1] - 1
@@ -726,17 +844,18 @@ int bonsai_grouped_gemm_bf16(const void* w, int groups, int n_rows, int K, const
   using namespace bonsai;
   if (groups < 1 || groups > kPfMaxGroups || K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 4 && epi != 6))
     return BONSAI_CUDA_BAD_ARG;
-  if (out_bf16 == nullptr || offsets == nullptr || status == nullptr || (epi == 4 && (n_rows % 2 != 0 || row_scale == nullptr))) return BONSAI_CUDA_BAD_ARG;
+  if (out_bf16 == nullptr || offsets == nullptr || status == nullptr || (epi == 4 && (n_rows % 2 != 0 || row_scale == nullptr)))
+    return BONSAI_CUDA_BAD_ARG;
   if ((long long)groups * n_rows >= (1ll << 31) || ((long long)groups + T / 64) * ((n_rows + 127) / 128) * (K >> 7) >= (1ll << 31)) return BONSAI_CUDA_BAD_ARG;
   CUtensorMap xmap, amap;
   if (!make_map_f16(&xmap, x, K, T, x_ld, wide ? 256 : 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
       !make_map_f16(&amap, w, K, (uint64_t)groups * n_rows, K, 128, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
     return BONSAI_CUDA_BAD_ARG;
-  const PfParams p{nullptr, nullptr, nullptr, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, 1, limit, alpha, offset, row_scale, offsets,
-                   groups, 0, nullptr, nullptr};
+  const PfParams p{nullptr, nullptr, nullptr, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, limit, alpha, offset, row_scale, offsets,
+                   groups, epilogue_quartets(K), 0, nullptr, nullptr};
   const int grid = sms > kPfMaxCtas ? kPfMaxCtas : (sms < 1 ? 1 : sms);
   const size_t smem = 1024 + (wide ? 4 * (size_t)(kPfABytes + 256 * 128) : 8 * (size_t)(kPfABytes + 64 * 128));
-  const auto kernel = wide ? bitgemm_prefill_kernel<256, true> : bitgemm_prefill_kernel<64, true>;
+  const auto kernel = wide ? bitgemm_prefill_kernel<256, true, true> : bitgemm_prefill_kernel<64, true, true>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return BONSAI_CUDA_LAUNCH_FAILED;
   const cudaError_t e = launch_pdl(kernel, dim3(grid), dim3(kPfThreads), smem, stream, xmap, amap, p);
   return e == cudaSuccess ? BONSAI_CUDA_OK : BONSAI_CUDA_LAUNCH_FAILED;

@@ -31,13 +31,14 @@ struct Router {
   float scale, den_eps;
 };
 
-// A warp chooses the experts of one token: lane k < top ends with the k-th one and its weight.  buf: [2 experts + groups] floats.
+// A warp chooses the experts of one token: lane k < top ends with the k-th one and its weight.  buf: [2 (experts + groups)] floats.
 template <int NE>
 __device__ __forceinline__ void choose(const Router& a, int t, float* buf, int lane, int& id, float& weight) {
   const float* z = a.z + (size_t)t * a.ld + a.col;
   float* choice = buf;
   float* score = buf + a.experts;
   float* sums = buf + 2 * a.experts;
+  float* kept = sums + a.groups;
   float c[NE];
 #pragma unroll
   for (int i = 0; i < NE; ++i) {
@@ -53,29 +54,35 @@ __device__ __forceinline__ void choose(const Router& a, int t, float* buf, int l
   __syncwarp();
   if (a.keep < a.groups) {
     const int size = a.experts / a.groups;
-    for (int g = lane; g < a.groups; g += 32) {
+    int lanes = 32;                              // lanes that share a group
+    while (lanes > 1 && lanes * a.groups > 32) lanes >>= 1;
+    for (int g0 = 0; g0 < a.groups; g0 += 32 / lanes) {
+      const int g = g0 + lane / lanes;
       float b1 = -INFINITY, b2 = -INFINITY;
-      for (int j = 0; j < size; ++j) {
-        const float v = choice[g * size + j];
-        if (v > b1) {
-          b2 = b1;
-          b1 = v;
-        } else {
-          b2 = fmaxf(b2, v);
+      if (g < a.groups)
+        for (int j = lane % lanes; j < size; j += lanes) {
+          const float v = choice[g * size + j];
+          b2 = fmaxf(b2, fminf(b1, v));
+          b1 = fmaxf(b1, v);
         }
+      for (int o = lanes >> 1; o > 0; o >>= 1) {
+        const float c1 = __shfl_xor_sync(0xffffffffu, b1, o), c2 = __shfl_xor_sync(0xffffffffu, b2, o);
+        b2 = fmaxf(fmaxf(b2, c2), fminf(b1, c1));
+        b1 = fmaxf(b1, c1);
       }
-      sums[g] = size > 1 ? b1 + b2 : b1;
+      if (g < a.groups && lane % lanes == 0) sums[g] = size > 1 ? b1 + b2 : b1;
+    }
+    __syncwarp();
+    for (int g = lane; g < a.groups; g += 32) {
+      int better = 0;
+      for (int j = 0; j < a.groups; ++j) better += sums[j] > sums[g] || (sums[j] == sums[g] && j < g);
+      kept[g] = better < a.keep ? 1.0f : 0.0f;
     }
     __syncwarp();
 #pragma unroll
     for (int i = 0; i < NE; ++i) {
       const int e = lane + 32 * i;
-      if (e >= a.experts) continue;
-      const int mine = e / size;
-      const float own = sums[mine];
-      int better = 0;
-      for (int g = 0; g < a.groups; ++g) better += sums[g] > own || (sums[g] == own && g < mine);
-      if (better >= a.keep) c[i] = -INFINITY;
+      if (e < a.experts && kept[e / size] == 0.0f) c[i] = -INFINITY;
     }
   }
   id = 0;
@@ -90,15 +97,9 @@ __device__ __forceinline__ void choose(const Router& a, int t, float* buf, int l
         v = c[i];
         e = lane + 32 * i;
       }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float v2 = __shfl_xor_sync(0xffffffffu, v, o);
-      const int e2 = __shfl_xor_sync(0xffffffffu, e, o);
-      if (v2 > v || (v2 == v && e2 < e)) {
-        v = v2;
-        e = e2;
-      }
-    }
+    const int bits = __float_as_int(v);          // as an unsigned number of the same order
+    const unsigned key = bits < 0 ? ~(unsigned)bits : (unsigned)bits | 0x80000000u;
+    e = (int)__reduce_min_sync(0xffffffffu, key == __reduce_max_sync(0xffffffffu, key) ? (unsigned)e : 0x7fffffffu);
     e = min(e, a.experts - 1);
 #pragma unroll
     for (int i = 0; i < NE; ++i)
@@ -144,19 +145,19 @@ __device__ __forceinline__ void prefix(const int* counts, int experts, int* offs
 }
 
 template <int NE>
-__global__ void __launch_bounds__(512) route_small_kernel(Router a) {
-  extern __shared__ float buf[];                 // [16 warps][2 experts + groups]
+__global__ void __launch_bounds__(1024) route_small_kernel(Router a, int warps) {
+  extern __shared__ float buf[];                 // [warps][2 (experts + groups)]
   __shared__ int s_id[kSmallPairs], s_place[kSmallPairs], s_count[kMaxExperts], s_off[kMaxExperts + 1];
   __shared__ float s_weight[kSmallPairs];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int e = threadIdx.x; e < a.experts; e += 512) s_count[e] = 0;
+  for (int e = threadIdx.x; e < a.experts; e += 1024) s_count[e] = 0;
   pdl_wait();
   pdl_trigger();
   __syncthreads();
-  for (int t = warp; t < a.T; t += 16) {
+  for (int t = warp; t < a.T && warp < warps; t += warps) {
     int id;
     float w;
-    choose<NE>(a, t, buf + warp * (2 * a.experts + a.groups), lane, id, w);
+    choose<NE>(a, t, buf + warp * 2 * (a.experts + a.groups), lane, id, w);
     if (lane < a.top) {
       const int p = t * a.top + lane;
       s_id[p] = id;
@@ -167,7 +168,7 @@ __global__ void __launch_bounds__(512) route_small_kernel(Router a) {
   __syncthreads();
   if (warp == 0) prefix(s_count, a.experts, s_off, a.lists, lane);
   __syncthreads();
-  for (int p = threadIdx.x; p < a.T * a.top; p += 512) {
+  for (int p = threadIdx.x; p < a.T * a.top; p += 1024) {
     const int row = s_off[s_id[p]] + s_place[p];
     a.at[p] = row;
     a.token[row] = p / a.top;
@@ -178,7 +179,7 @@ __global__ void __launch_bounds__(512) route_small_kernel(Router a) {
 // 32 tokens per CTA
 template <int NE>
 __global__ void __launch_bounds__(256) route_kernel(Router a) {
-  extern __shared__ float buf[];                 // [8 warps][2 experts + groups]
+  extern __shared__ float buf[];                 // [8 warps][2 (experts + groups)]
   __shared__ int s_count[kMaxExperts], s_base[kMaxExperts];
   __shared__ int s_id[32 * kMaxTop], s_place[32 * kMaxTop];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t0 = blockIdx.x * 32, n = min(32, a.T - t0);
@@ -189,7 +190,7 @@ __global__ void __launch_bounds__(256) route_kernel(Router a) {
   for (int i = warp; i < n; i += 8) {
     int id;
     float w;
-    choose<NE>(a, t0 + i, buf + warp * (2 * a.experts + a.groups), lane, id, w);
+    choose<NE>(a, t0 + i, buf + warp * 2 * (a.experts + a.groups), lane, id, w);
     if (lane < a.top) {
       s_id[i * a.top + lane] = id;
       s_place[i * a.top + lane] = atomicAdd(&s_count[id], 1);
@@ -421,9 +422,10 @@ int bonsai_lay_route(const void* const* ptrs, const int* ints, const float* floa
   using namespace bonsai::lay;
   Router a;
   if (!fill(a, ptrs, ints, floats, T)) return BONSAI_CUDA_BAD_ARG;
-  const size_t buf = (2 * a.experts + a.groups) * sizeof(float);
+  const size_t buf = 2 * (a.experts + a.groups) * sizeof(float);
   if (xs == nullptr && T <= bonsai_lay_route_small(a.top)) {
-#define BONSAI_SMALL(NE) launch(route_small_kernel<NE>, dim3(1), 512, 16 * buf, stream, 1, 0, a)
+    const int warps = min(min(T, 32), (int)(160 * 1024 / buf));
+#define BONSAI_SMALL(NE) launch(route_small_kernel<NE>, dim3(1), 1024, warps * buf, stream, 1, 0, a, warps)
     return BONSAI_BY_EXPERTS(BONSAI_SMALL);
 #undef BONSAI_SMALL
   }

@@ -74,6 +74,8 @@ __device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-
 
 __device__ __forceinline__ void store_act(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 __device__ __forceinline__ void store_act(float* p, float v) { *p = v; }
+__device__ __forceinline__ void store_act4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+__device__ __forceinline__ void store_act4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ float load_act(const bf16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ float load_act(const float* p) { return *p; }
 

@@ -7,8 +7,6 @@
 namespace bonsai {
 namespace lay {
 
-__device__ __forceinline__ void store_act4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
-__device__ __forceinline__ void store_act4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 
 __device__ __forceinline__ float4 load_act4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float4 load_act4(const bf16* p) {

@@ -380,14 +380,20 @@ class LatentAttentionMixer:
         self.groups = -(-s.heads // L.lib().bonsai_lay_latent_group(s.heads))
         self.lat_ld, self.kv_ld = max(row, w.latent.expand.kp), w.latent.expand.n
         absorbed, partial, sums = r.latent_scratch(row, self.lat_ld, s.heads, L.round_up(s.rank, 16), self.kv_ld)
-        ints = [r.proj.stride(0), q, c, rot, g, out.stride(0), s.heads, s.dim, s.rot_dim, s.vdim, s.rank, r.max_pages, r.kv.page_size]
+        ints = [r.proj.stride(0), q, c, rot, g, out.stride(0), s.heads, s.dim, s.rot_dim, s.vdim, s.rank, r.max_pages, r.kv.page_size,
+                absorbed.shape[0], partial.shape[0], r.kv.num_pages]
         self.call = {id(rows): L.MixerCall([r.proj, w.vectors["dkv.norm"], r.angles(s.rotary), rows.positions, rows.slots, r.block_table, r.kv.rows[index],
-                                            w.latent.keys, w.latent.values, absorbed, partial, sums, out], ints, [r.cfg.eps, s.scale, branch.scale])
+                                            w.latent.keys, w.latent.values, absorbed, partial, sums, r.status, out], ints, [r.cfg.eps, s.scale, branch.scale])
                      for rows in (r.slot_rows, r.batch_rows)}
 
-    def splits(self, rows: int) -> int:
-        """KV splits of the absorbed form: about a CTA per SM, and at least two tiles of 64 keys each at full length."""
-        return max(1, min(L.lib().bonsai_lay_latent_max_splits(), self.r.scratch.sms // (rows * self.groups), -(-self.r.max_seq // 128)))
+    def splits(self, rows: int) -> tuple[int, int]:
+        """KV splits of the absorbed form, a power of two, and how many of them share a sum: at most a CTA per SM (of those that clusters
+        reach), and no more than there are tiles of 64 keys at full length."""
+        lib, n = L.lib(), 1
+        while 2 * n <= min(lib.bonsai_lay_latent_max_splits(), self.r.scratch.sms // (rows * self.groups), -(-self.r.max_seq // 64)):
+            n *= 2
+        # large clusters do not fill the GPU: two of eight in a GPC of 16 to 20 SMs
+        return n, min(n, lib.bonsai_lay_latent_max_cluster() if rows * self.groups * n <= 64 else 4)
 
     def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
         lib, a, r = L.lib(), self.call[id(rows)].args, self.r
@@ -396,10 +402,10 @@ class LatentAttentionMixer:
             K.check(lib.bonsai_lay_latent_f32(*a, st.rows, stream), "latent_f32")
             return
         if st.short:
-            n = self.splits(st.short)
+            n, cluster = self.splits(st.short)
             K.check(lib.bonsai_lay_latent_query(*a, st.short, stream), "latent_query")
-            K.check(lib.bonsai_lay_latent_decode(*a, st.short, n, stream), "latent_decode")
-            K.check(lib.bonsai_lay_latent_value(*a, st.short, n, stream), "latent_value")
+            K.check(lib.bonsai_lay_latent_decode(*a, st.short, n, cluster, stream), "latent_decode")
+            K.check(lib.bonsai_lay_latent_value(*a, st.short, n // cluster, stream), "latent_value")
         if st.rows > st.short:
             K.check(lib.bonsai_lay_latent_append(*a, st.short, st.rows - st.short, 0, stream), "latent_append")
         for g in st.contexts:
@@ -590,6 +596,7 @@ class LayeredRunner(SlotState):
         shared = L.ExpertScratch(cap, cfg.width, specs, exact, dev) if specs else None
         self.experts = {i: L.Routing(cfg.experts(i), w.mlp.up, w.mlp.down, w.mlp.correction, self.proj, w.mlp.column, shared)
                         for i, w in enumerate(weights.layers) if i in cfg.expert_layers}
+        self._branch, self._forked = torch.cuda.Stream(dev), False
         self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
 
     def angles(self, rot: RotarySpec) -> torch.Tensor:
@@ -658,13 +665,15 @@ class LayeredRunner(SlotState):
             last = i + 1 == len(layers)
             after, following = (self.normed, self.w.final_norm) if last and final else (copy, None if last else layers[i + 1].pre_norm)
             L.linear(w.proj, h, T, self.proj, self.scratch)
+            experts = self.experts.get(i)
+            if experts is not None:
+                self._beside(experts, h, T)
             for n, mixer in enumerate(self.mixers[i]):
                 mixer(rows, st, s, early=n > 0)            # only the first one follows the projection directly
             L.linear(w.out, self.mixer_out[i], T, self.y, self.scratch)
             if cfg.side_by_side:
-                experts = self.experts.get(i)
                 if experts is not None:
-                    experts(h, T, self.scratch)
+                    self._join()
                 L.side_by_side(x, self.y, experts, cfg.residual_mult, T, after, following, cfg.eps, cfg.layer_norm)
             elif w.mlp is None:
                 L.norm_add(x, self.y, w.norm, cfg.eps, T, after, following)
@@ -674,6 +683,21 @@ class LayeredRunner(SlotState):
                 L.linear(w.mlp.up, h, T, act, self.scratch, w.mlp.act)
                 L.linear(w.mlp.down, act, T, self.y, self.scratch)
                 L.norm_add(x, self.y, w.mlp.norm, cfg.eps, T, after, following)
+
+    def _beside(self, experts: L.Routing, h: torch.Tensor, T: int) -> None:
+        """The experts of a layer, which need its projection only: in a captured decode step, a branch beside the mixer's kernels."""
+        main = torch.cuda.current_stream(self.device)
+        self._forked = torch.cuda.is_current_stream_capturing()
+        if not self._forked:
+            experts(h, T, self.scratch)
+            return
+        self._branch.wait_stream(main)
+        with torch.cuda.stream(self._branch):
+            experts(h, T, self.scratch)
+
+    def _join(self) -> None:
+        if self._forked:
+            torch.cuda.current_stream(self.device).wait_stream(self._branch)
 
     def _head(self, row_list: int, count: int, out: torch.Tensor) -> None:
         """Logits of ``count`` rows (device address of their indices) into ``out`` [count, vocab]."""

@@ -28,10 +28,11 @@ _SIG = {
     "bonsai_lay_attn_f32": [_vp, _vp, _vp, _i, _vp],
     "bonsai_lay_latent_row": [_i, _i],
     "bonsai_lay_latent_max_splits": [],
+    "bonsai_lay_latent_max_cluster": [],
     "bonsai_lay_latent_group": [_i],
     "bonsai_lay_latent_append": [_vp, _vp, _vp, _i, _i, _i, _vp],
     "bonsai_lay_latent_query": [_vp, _vp, _vp, _i, _vp],
-    "bonsai_lay_latent_decode": [_vp, _vp, _vp, _i, _i, _vp],
+    "bonsai_lay_latent_decode": [_vp, _vp, _vp, _i, _i, _i, _vp],
     "bonsai_lay_latent_value": [_vp, _vp, _vp, _i, _i, _vp],
     "bonsai_lay_latent_gather": [_vp, _vp, _vp, _vp, _i, _i, _vp, _i, _vp],
     "bonsai_lay_latent_prompt": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp],
@@ -250,7 +251,7 @@ class Routing:
     def few(self, T: int) -> bool:
         """Whether the experts' weights are streamed for a few rows each, rather than multiplied in tiles."""
         r = self.spec.router
-        return T * r.top <= self.s.pairs // 2 and (T <= FEW_ROWS or T * r.top <= 12 * r.experts)
+        return T * r.top <= self.s.pairs // 2 and (T <= FEW_ROWS or T * r.top <= 2 * r.experts)
 
     def launches(self, T: int) -> int:
         return 2 + (1 if T <= lib().bonsai_lay_route_small(self.spec.router.top) and (self.s.exact or self.few(T)) else 2)

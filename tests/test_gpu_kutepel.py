@@ -383,7 +383,7 @@ def test_long_context(tmp_path, kv):
     eng = engine(m, kv, max_batch=3, max_seq=1024, chunk=1024)
     tokens = m.tokens(900)
     want = m.logits(tokens)
-    assert kv == "f32" or eng.runner.mixers[0][0].splits(1) == 8
+    assert kv == "f32" or eng.runner.mixers[0][0].splits(1) == (16, 8)
     for cuts in ([], [77, 700, 2], [860] + [1] * 40, [500, 33, 32, 1, 200]):
         poison(eng)
         check(feed(eng, tokens, cuts), want, kv, str(cuts[:3]))
