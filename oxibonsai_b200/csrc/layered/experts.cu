@@ -176,25 +176,25 @@ __global__ void __launch_bounds__(1024) route_small_kernel(Router a, int warps) 
   }
 }
 
-// 32 tokens per CTA
+// 8 tokens per CTA
 template <int NE>
 __global__ void __launch_bounds__(256) route_kernel(Router a) {
   extern __shared__ float buf[];                 // [8 warps][2 (experts + groups)]
   __shared__ int s_count[kMaxExperts], s_base[kMaxExperts];
-  __shared__ int s_id[32 * kMaxTop], s_place[32 * kMaxTop];
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t0 = blockIdx.x * 32, n = min(32, a.T - t0);
+  __shared__ int s_id[8 * kMaxTop], s_place[8 * kMaxTop];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t0 = blockIdx.x * 8, n = min(8, a.T - t0);
   for (int e = threadIdx.x; e < a.experts; e += 256) s_count[e] = 0;
   pdl_wait();
   pdl_trigger();
   __syncthreads();
-  for (int i = warp; i < n; i += 8) {
+  if (warp < n) {
     int id;
     float w;
-    choose<NE>(a, t0 + i, buf + warp * 2 * (a.experts + a.groups), lane, id, w);
+    choose<NE>(a, t0 + warp, buf + warp * 2 * (a.experts + a.groups), lane, id, w);
     if (lane < a.top) {
-      s_id[i * a.top + lane] = id;
-      s_place[i * a.top + lane] = atomicAdd(&s_count[id], 1);
-      a.pair_weight[(size_t)(t0 + i) * a.top + lane] = w;
+      s_id[warp * a.top + lane] = id;
+      s_place[warp * a.top + lane] = atomicAdd(&s_count[id], 1);
+      a.pair_weight[(size_t)(t0 + warp) * a.top + lane] = w;
     }
   }
   __syncthreads();
@@ -430,7 +430,7 @@ int bonsai_lay_route(const void* const* ptrs, const int* ints, const float* floa
 #undef BONSAI_SMALL
   }
   if (xs != nullptr && (chunks < 1 || ldh % 8 != 0 || ldx % 8 != 0 || ldh < 8 * chunks || ldx < 8 * chunks)) return BONSAI_CUDA_BAD_ARG;
-#define BONSAI_LARGE(NE) launch(route_kernel<NE>, dim3((T + 31) / 32), 256, 8 * buf, stream, 1, 0, a)
+#define BONSAI_LARGE(NE) launch(route_kernel<NE>, dim3((T + 7) / 8), 256, 8 * buf, stream, 1, 0, a)
   const int st = BONSAI_BY_EXPERTS(BONSAI_LARGE);
 #undef BONSAI_LARGE
   if (st != BONSAI_CUDA_OK) return st;

@@ -34,7 +34,7 @@ struct Latent {
   void* pool;               // [pages][page_size][row], bf16 (f32 in the 32-bit mode)
   const bf16* wk;           // [heads][rp][dk]: key expansion, transposed, zero in the padding
   const bf16* wv;           // [heads][vdim][rk]: value expansion, zero in the padding
-  bf16* q;                  // [rows][heads][row]: absorbed queries times scale * log2(e)
+  bf16* q;                  // [rows][heads][row]: absorbed queries times scale * log2(e), columns in the order of `query_at`
   float* part;              // [rows][parts][heads][rp]: sums of ex2(score - max) c
   float2* ml;               // [rows][parts][heads]: maximum and sum of ex2(score - max)
   int* status;              // set to 1 when a copy does not arrive
@@ -129,6 +129,9 @@ struct WeightRows {
 };
 
 // ---- absorbed -----------------------------------------------------------------------------------------------------------------
+// Place of column c of an absorbed query: in every 32 columns the eight that a lane holds as A registers of two steps are neighbours.
+__device__ __forceinline__ int query_at(int c) { return (c & ~31) | ((c & 6) << 2) | ((c & 16) >> 2) | ((c & 8) >> 2) | (c & 1); }
+
 // One grid of three kinds of CTAs: cache entries (8 rows), the rotated parts of the queries (32 pairs of row and head), and the absorbed
 // parts (128 latent columns of one head for 8 NT rows).
 template <int NT, int NK>
@@ -150,10 +153,11 @@ __global__ void __launch_bounds__(256) query_kernel(Latent a, int T, int blocks)
       const int pair = (job - appends) * 32 + warp * 4 + i, t = pair / a.heads, head = pair - t * a.heads;
       if (t >= T) return;
       const float* q = a.proj + (size_t)t * a.ld + a.q_col + head * (a.dim + a.rot_dim) + a.dim;
-      bf16* dst = a.q + (size_t)pair * a.row + a.rp;
+      bf16* dst = a.q + (size_t)pair * a.row;
       const int pos = a.pos[t];
       const float2* rot = latent_angles(a, pos < (a.max_pages << a.pshift) ? pos : 0);
-      for (int d = lane; d < a.row - a.rp; d += 32) dst[d] = __float2bfloat16_rn(d < a.rot_dim ? rotated(q, d, rot, a.rot_dim, 1) * f : 0.0f);
+      for (int d = lane; d < a.row - a.rp; d += 32)
+        dst[query_at(a.rp + d)] = __float2bfloat16_rn(d < a.rot_dim ? rotated(q, d, rot, a.rot_dim, 1) * f : 0.0f);
     }
     return;
   }
@@ -180,7 +184,7 @@ __global__ void __launch_bounds__(256) query_kernel(Latent a, int T, int blocks)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int tok = t0 + 8 * j + 2 * t4 + (e & 1), r = r0 + g + 8 * (e >> 1);
-      if (tok < T) a.q[((size_t)tok * a.heads + head) * a.row + r] = __float2bfloat16_rn(acc[j][e] * a.scale * kLog2e);
+      if (tok < T) a.q[((size_t)tok * a.heads + head) * a.row + query_at(r)] = __float2bfloat16_rn(acc[j][e] * a.scale * kLog2e);
     }
 }
 
@@ -203,7 +207,7 @@ __device__ __forceinline__ const bf16* tile_at(const uint8_t* k, int r, int c) {
 
 template <int CB, int MT>
 __global__ void __launch_bounds__(512) latent_decode_kernel(const __grid_constant__ CUtensorMap rows_map, Latent a, int cl) {
-  constexpr int H = 16 * MT, LDS = 72, LDP = 72, NK = 10, NTH = 512;
+  constexpr int H = 16 * MT, LDS = 72, LDP = 72, NK = 5, NTH = 512;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __shared__ uint64_t full[2];
   __shared__ float2 s_ml[H];
@@ -224,46 +228,45 @@ __global__ void __launch_bounds__(512) latent_decode_kernel(const __grid_constan
   const int b0 = split * per, b1 = min(ntiles, b0 + per);
   const int* bt = a.block_table + (size_t)a.slots[t] * a.max_pages;
   if (threadIdx.x == 0) {
-    tc::mbar_init(&full[0], 1);
-    tc::mbar_init(&full[1], 1);
+    tc::mbar_init(&full[0], blocks);
+    tc::mbar_init(&full[1], blocks);
     tc::mbar_fence_init();
   }
   __syncthreads();
   const int box = min(64, 1 << a.pshift);                 // rows of a copy: they lie in one page
-  auto fetch = [&](int tile, int st) {                    // warp 0; pages past the last position are not touched
+  auto first_row = [&](int tile) { return tile < ntiles ? (int)latent_row(a, bt, tile * 64) : 0; };
+  auto fetch = [&](int tile, int st, int row) {           // one thread of `blocks` warps each; pages past the last position are not touched
     const int n = (min(64, pos + 1 - tile * 64) + box - 1) / box;
-    if (lane == 0) tc::mbar_arrive_expect_tx(&full[st], (uint32_t)(n * blocks * box * 128));
-    __syncwarp();
-    for (int i = lane; i < n * blocks; i += 32) {
-      const int b = i % blocks, r = (i / blocks) * box;
-      tma_rows(sK + st * stage + b * kBlockBytes + r * 128, &rows_map, b * 64, (int)latent_row(a, bt, tile * 64 + r), &full[st]);
-    }
+    tc::mbar_arrive_expect_tx(&full[st], (uint32_t)(n * box * 128));
+    for (int i = 0; i < n; ++i)
+      tma_rows(sK + st * stage + warp * kBlockBytes + i * box * 128, &rows_map, warp * 64, i == 0 ? row : (int)latent_row(a, bt, tile * 64 + i * box), &full[st]);
   };
+  const bool copies = lane == 0 && warp < blocks;
+  int next_row = copies ? first_row(b0) : 0;
   // rows of this batch are appended by the kernel before this one; a tile that ends 64 tokens before this one holds none of them
   const bool early = b0 < b1 && b0 * 64 + 64 <= pos - 63;
-  if (early && warp == 0) fetch(b0, 0);
+  if (early && copies) fetch(b0, 0, next_row);
   pdl_wait();
   pdl_trigger();
   float mx[MT], l[MT];                                    // heads warp * MT + i
 #pragma unroll
   for (int i = 0; i < MT; ++i) mx[i] = -INFINITY, l[i] = 0.0f;
   if (b0 < b1) {
-    if (!early && warp == 0) fetch(b0, 0);
-    // this warp's scores: 16 heads x 16 MT keys over steps kq, kq + 4, .. of 16 columns
-    const int mt = warp % MT, kq = (warp / MT) & 3, key0 = (warp / (4 * MT)) * 16 * MT, nk = ((a.row >> 4) - kq + 3) >> 2;
-    uint32_t qf[NK][4];                                   // the queries' share as A registers
+    if (!early && copies) fetch(b0, 0, next_row);
+    if (copies) next_row = first_row(b0 + 1);
+    // this warp's scores: 16 heads x 16 MT keys over blocks kq, kq + 4, .. of 32 columns
+    const int mt = warp % MT, kq = (warp / MT) & 3, key0 = (warp / (4 * MT)) * 16 * MT, nk = ((a.row >> 5) - kq + 3) >> 2;
+    uint4 q0[NK], q1[NK];                                 // the queries' share: A registers of two steps each
     {
       const int r0 = mt * 16 + g;
-      const bf16* q0 = a.q + ((size_t)t * a.heads + h0 + min(r0, nh - 1)) * a.row + 16 * kq + 2 * t4;
-      const bf16* q1 = a.q + ((size_t)t * a.heads + h0 + min(r0 + 8, nh - 1)) * a.row + 16 * kq + 2 * t4;
+      const bf16* p0 = a.q + ((size_t)t * a.heads + h0 + min(r0, nh - 1)) * a.row + 32 * kq + 8 * t4;
+      const bf16* p1 = a.q + ((size_t)t * a.heads + h0 + min(r0 + 8, nh - 1)) * a.row + 32 * kq + 8 * t4;
 #pragma unroll
-      for (int i = 0; i < NK; ++i) {
-        if (i >= nk) break;
-        qf[i][0] = *reinterpret_cast<const uint32_t*>(q0 + 64 * i);
-        qf[i][1] = *reinterpret_cast<const uint32_t*>(q1 + 64 * i);
-        qf[i][2] = *reinterpret_cast<const uint32_t*>(q0 + 64 * i + 8);
-        qf[i][3] = *reinterpret_cast<const uint32_t*>(q1 + 64 * i + 8);
-      }
+      for (int i = 0; i < NK; ++i)
+        if (i < nk) {
+          q0[i] = *reinterpret_cast<const uint4*>(p0 + 128 * i);
+          q1[i] = *reinterpret_cast<const uint4*>(p1 + 128 * i);
+        }
     }
     float o[MT][2 * CB][4];
 #pragma unroll
@@ -274,7 +277,10 @@ __global__ void __launch_bounds__(512) latent_decode_kernel(const __grid_constan
       const int st = (tile - b0) & 1;
       uint8_t* k = sK + st * stage;
       __syncthreads();     // everyone is done with the other stage
-      if (tile + 1 < b1 && warp == 0) fetch(tile + 1, st ^ 1);
+      if (tile + 1 < b1 && copies) {
+        fetch(tile + 1, st ^ 1, next_row);
+        next_row = first_row(tile + 2);                   // used a tile later
+      }
       if (!tc::mbar_wait(&full[st], ((tile - b0) >> 1) & 1) && lane == 0) atomicExch(a.status, 1);
       if (tile == ntiles - 1) {     // rows behind the last position may hold anything: their weights are zero, so they must be finite
         for (int i = threadIdx.x + (pos + 1 - tile * 64) * 8; i < 64 * 8; i += NTH)
@@ -286,14 +292,21 @@ __global__ void __launch_bounds__(512) latent_decode_kernel(const __grid_constan
       for (int i = 0; i < 2 * MT; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
 #pragma unroll
       for (int ks = 0; ks < NK; ++ks) {
-        if (ks >= nk) break;
+        if (ks >= nk) continue;
+        const uint32_t qa[2][4] = {{q0[ks].x, q1[ks].x, q0[ks].y, q1[ks].y}, {q0[ks].z, q1[ks].z, q0[ks].w, q1[ks].w}};
+        uint32_t b[2][MT][4];
 #pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          uint32_t b[4];
-          ldsm4(b, tile_at(k, key0 + 16 * i + (lane & 7) + ((lane >> 4) << 3), (kq + 4 * ks) * 16 + ((lane >> 3) & 1) * 8));
-          mma_bf16(s[2 * i], qf[ks], b[0], b[1]);
-          mma_bf16(s[2 * i + 1], qf[ks], b[2], b[3]);
-        }
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int i = 0; i < MT; ++i)
+            ldsm4(b[u][i], tile_at(k, key0 + 16 * i + (lane & 7) + ((lane >> 4) << 3), (kq + 4 * ks) * 32 + 16 * u + ((lane >> 3) & 1) * 8));
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int i = 0; i < MT; ++i) {
+            mma_bf16(s[2 * i], qa[u], b[u][i][0], b[u][i][1]);
+            mma_bf16(s[2 * i + 1], qa[u], b[u][i][2], b[u][i][3]);
+          }
       }
 #pragma unroll
       for (int i = 0; i < 2 * MT; ++i)
@@ -402,7 +415,10 @@ __global__ void __launch_bounds__(512) latent_decode_kernel(const __grid_constan
     }
     *reinterpret_cast<float4*>(a.part + (base + r) * a.rp + c) = acc;
   }
-  if (cl > 1) cluster.sync();   // nobody leaves while its sums are being read
+  if (cl > 1) {     // nobody leaves while its sums are being read; the reads are over when their values are stored
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+  }
 }
 
 // grid (heads x blocks of 16 RT value columns, groups of 8 NT rows): the partial sums become one latent per row, which is expanded

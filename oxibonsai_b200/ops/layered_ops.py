@@ -249,9 +249,12 @@ class Routing:
         return (o.data_ptr(), o.stride(0), int(o.dtype == torch.float32), self.s.at.data_ptr(), r.top, self.s.counts.data_ptr(), r.experts)
 
     def few(self, T: int) -> bool:
-        """Whether the experts' weights are streamed for a few rows each, rather than multiplied in tiles."""
+        """Whether the experts' weights are streamed for a few rows each, rather than multiplied in tiles behind a copy of the rows.
+        On their own the tiles win from eight tokens on (unless the experts are so small that the copy's launch counts), but their
+        CTAs take the SMs whole, and a decode step of that size does better with the mixer's kernels beside them."""
         r = self.spec.router
-        return T * r.top <= self.s.pairs // 2 and (T <= FEW_ROWS or T * r.top <= 2 * r.experts)
+        chosen = min(r.experts, T * r.top) * (self.up.nbytes + self.down.nbytes) // r.experts
+        return T * r.top <= self.s.pairs // 2 and (T <= 16 or (T <= FEW_ROWS and chosen < 48 << 20))
 
     def launches(self, T: int) -> int:
         return 2 + (1 if T <= lib().bonsai_lay_route_small(self.spec.router.top) and (self.s.exact or self.few(T)) else 2)
