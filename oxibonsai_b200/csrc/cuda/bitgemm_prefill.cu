@@ -71,7 +71,7 @@ struct PfParams {
   int* status;
   int n_rows, K, T, epi, out_ld;
   int bf16;                // dense operands are bf16 (both) instead of f16
-  float glu_limit, glu_alpha, glu_offset;   // epi 4
+  float glu_limit, glu_alpha, glu_offset, glu_cubic;   // epi 4 (epi 7: the limit)
   const float* row_scale;  // epi 4, grouped: factor of a row's outputs
   const int* offsets;      // grouped: [groups + 1] first row of every group (device memory)
   int groups;
@@ -145,6 +145,7 @@ __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, 
   } else if (row_ok && tok < tend) {
     const size_t o = (size_t)tok * p.out_ld + row;
     if (p.epi == 0) p.out_f32[o] = v;
+    else if (p.epi == 7) p.out_f32[o] = p.glu_limit * tanhf(v / p.glu_limit);
     else if (p.epi == 1) p.out_f32[o] = res + v;
     else if (p.epi == 5) reinterpret_cast<__nv_bfloat16*>(p.out_f16)[o] = __float2bfloat16_rn(fmaxf(v, 0.0f) * fmaxf(v, 0.0f));
     else if (p.epi == 6) reinterpret_cast<__nv_bfloat16*>(p.out_f16)[o] = __float2bfloat16_rn(v);
@@ -153,8 +154,8 @@ __device__ __forceinline__ void pf_store(const PfParams& p, float v, float res, 
 }
 
 // Epilogue 4 for CB accumulator values of one weight row, columns tok0 .. tok0 + CB - 1: the clamped gated unit over gate (even)
-// and up (odd) rows, min(g, limit) * sigmoid(alpha g) * (clamp(u, -limit, limit) + offset), stored as bf16.  The two lanes of a
-// pair split the columns: the even lane finishes even ones, the odd lane odd ones, so every lane has CB / 2 outputs and one
+// and up (odd) rows, g * sigmoid(alpha (g + cubic g^3)) * (clamp(u, -limit, limit) + offset) with the gate limited, g = min(g, limit),
+// stored as bf16.  The two lanes of a pair split the columns: the even lane finishes even ones, the odd lane odd ones, so every lane has CB / 2 outputs and one
 // shuffle per output.
 template <int CB, bool SCALED = false>
 __device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, int tok0, int tend, int row, int a, bool row_ok) {
@@ -171,7 +172,7 @@ __device__ __forceinline__ void pf_store_glu(const PfParams& p, const float* v, 
     const float other = __shfl_xor_sync(0xffffffffu, odd ? v[2 * j] : v[2 * j + 1], 1);
     const float g = fminf(odd ? other : keep, p.glu_limit);
     const float u = fminf(fmaxf(odd ? keep : other, -p.glu_limit), p.glu_limit);
-    o[j] = __fdividef(g, 1.0f + __expf(-p.glu_alpha * g)) * (u + p.glu_offset);
+    o[j] = __fdividef(g, 1.0f + __expf(-p.glu_alpha * fmaf(p.glu_cubic * g * g, g, g))) * (u + p.glu_offset);
   }
   __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out_f16) + (row >> 1);
 #pragma unroll
@@ -514,7 +515,11 @@ __global__ void __launch_bounds__(kPfThreads, 1) bitgemm_prefill_kernel(const __
             for (int j = 0; j < CB; ++j)
               if (p.epi == 5) v[j] = fmaxf(v[j], 0.0f) * fmaxf(v[j], 0.0f);
             pf_store_bf16<CB>(p, v, tok, tend, row, a);
-          } else if (p.epi == 0) {
+          } else if (p.epi == 0 || p.epi == 7) {
+            if (p.epi == 7) {
+#pragma unroll
+              for (int j = 0; j < CB; ++j) v[j] = p.glu_limit * tanhf(v[j] / p.glu_limit);
+            }
             float* dst = p.out_f32 + (size_t)tok * p.out_ld + row;
             if (tok + CB <= tend) {
 #pragma unroll
@@ -809,7 +814,7 @@ int bonsai_bitgemm_prefill_ws(const void* codes, const void* scales, const void*
     amap = xmap;
   }
   PfParams p{(const uint32_t*)codes, (const __half*)scales, out_f32, residual, (__half*)out_f16, status, n_rows, K, T, epi, out_ld,
-             0, 0.0f, 0.0f, 0.0f, nullptr, nullptr, 0, epilogue_quartets(K), 0, nullptr, nullptr};
+             0, 0.0f, 0.0f, 0.0f, 0.0f, nullptr, nullptr, 0, epilogue_quartets(K), 0, nullptr, nullptr};
   if (dense_w != nullptr)
     return tok == 64 ? launch_prefill<64, true>(xmap, amap, p, sms, ws, ws_bytes, balance, stream)
                      : launch_prefill<256, true>(xmap, amap, p, sms, ws, ws_bytes, balance, stream);
@@ -818,20 +823,21 @@ int bonsai_bitgemm_prefill_ws(const void* codes, const void* scales, const void*
 }
 
 // Dense bf16 operands: W [n_rows][K] (K a multiple of 128), x [T][x_ld], f32 accumulation.  epi 0: out_f32 = W x; 4: out_bf16 =
-// clamped gated unit over interleaved gate / up rows (n_rows / 2 columns); 5: out_bf16 = relu(W x)^2; 6: out_bf16 = W x.  Workspace and
-// status as above.
+// clamped gated unit over interleaved gate / up rows (n_rows / 2 columns); 5: out_bf16 = relu(W x)^2; 6: out_bf16 = W x;
+// 7: out_f32 = limit * tanh(W x / limit).  Workspace and status as above.
 int bonsai_dense_gemm_bf16(const void* w, int n_rows, int K, const void* x, int x_ld, int T, float* out_f32, void* out_bf16, int out_ld, int epi,
-                           float limit, float alpha, float offset, int* status, void* ws, size_t ws_bytes, int sms, cudaStream_t stream) {
+                           float limit, float alpha, float offset, float cubic, int* status, void* ws, size_t ws_bytes, int sms, cudaStream_t stream) {
   using namespace bonsai;
-  if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && epi != 4 && epi != 5 && epi != 6)) return BONSAI_CUDA_BAD_ARG;
-  if ((epi == 0 && out_f32 == nullptr) || (epi != 0 && out_bf16 == nullptr) || (epi == 4 && n_rows % 2 != 0) || status == nullptr)
+  if (K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 0 && (epi < 4 || epi > 7))) return BONSAI_CUDA_BAD_ARG;
+  const bool f32_out = epi == 0 || epi == 7;
+  if ((f32_out && out_f32 == nullptr) || (!f32_out && out_bf16 == nullptr) || (epi == 4 && n_rows % 2 != 0) || (epi == 7 && !(limit > 0.0f)) || status == nullptr)
     return BONSAI_CUDA_BAD_ARG;
   const int tok = T <= 64 ? 64 : 256;
   CUtensorMap xmap, amap;
   if (!make_map_f16(&xmap, x, K, T, x_ld, tok, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
       !make_map_f16(&amap, w, K, n_rows, K, 128, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
     return BONSAI_CUDA_BAD_ARG;
-  PfParams p{nullptr, nullptr, out_f32, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, limit, alpha, offset, nullptr, nullptr, 0, epilogue_quartets(K), 0, nullptr, nullptr};
+  PfParams p{nullptr, nullptr, out_f32, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, limit, alpha, offset, cubic, nullptr, nullptr, 0, epilogue_quartets(K), 0, nullptr, nullptr};
   return tok == 64 ? launch_prefill<64, true>(xmap, amap, p, sms, ws, ws_bytes, 1, stream)
                    : launch_prefill<256, true>(xmap, amap, p, sms, ws, ws_bytes, 1, stream);
 }
@@ -840,7 +846,7 @@ int bonsai_dense_gemm_bf16(const void* w, int n_rows, int K, const void* x, int 
 // (device memory, ascending, at most T) belong to group g.  epi 4: out_bf16 = clamped gated unit over interleaved gate / up rows times
 // row_scale[row]; 6: out_bf16 = W x.  wide: tiles of 256 rows of x instead of 64.
 int bonsai_grouped_gemm_bf16(const void* w, int groups, int n_rows, int K, const void* x, int x_ld, int T, const int* offsets, const float* row_scale,
-                             void* out_bf16, int out_ld, int epi, float limit, float alpha, float offset, int wide, int* status, int sms, cudaStream_t stream) {
+                             void* out_bf16, int out_ld, int epi, float limit, float alpha, float offset, float cubic, int wide, int* status, int sms, cudaStream_t stream) {
   using namespace bonsai;
   if (groups < 1 || groups > kPfMaxGroups || K < 128 || K % 128 != 0 || n_rows < 1 || T < 1 || x_ld < K || x_ld % 8 != 0 || (epi != 4 && epi != 6))
     return BONSAI_CUDA_BAD_ARG;
@@ -851,7 +857,7 @@ int bonsai_grouped_gemm_bf16(const void* w, int groups, int n_rows, int K, const
   if (!make_map_f16(&xmap, x, K, T, x_ld, wide ? 256 : 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) ||
       !make_map_f16(&amap, w, K, (uint64_t)groups * n_rows, K, 128, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16))
     return BONSAI_CUDA_BAD_ARG;
-  const PfParams p{nullptr, nullptr, nullptr, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, limit, alpha, offset, row_scale, offsets,
+  const PfParams p{nullptr, nullptr, nullptr, nullptr, (__half*)out_bf16, status, n_rows, K, T, epi, out_ld, 1, limit, alpha, offset, cubic, row_scale, offsets,
                    groups, epilogue_quartets(K), 0, nullptr, nullptr};
   const int grid = sms > kPfMaxCtas ? kPfMaxCtas : (sms < 1 ? 1 : sms);
   const size_t smem = 1024 + (wide ? 4 * (size_t)(kPfABytes + 256 * 128) : 8 * (size_t)(kPfABytes + 64 * 128));

@@ -1,7 +1,7 @@
 // Mixture of experts: the router's choice, and the experts' projections over the tokens that chose them.
 //
-//   s = sigmoid(z), choice = s + correction; only the experts of the `keep` groups with the largest sums of their two best choices
-//   are eligible; the `top` best of them get the weights s / (sum of the chosen s + den_eps) * scale.
+//   s = sigmoid(z) or softmax(z), choice = s [+ correction]; only the experts of the `keep` groups with the largest sums of their two
+//   best choices are eligible; the `top` best of them get the weights s [/ (sum of the chosen s + den_eps)] * scale.
 //
 // The pairs (token, chosen expert) are laid out expert by expert: expert e has the sorted rows offsets[e] .. offsets[e + 1] - 1, `token`
 // names the token of a sorted row, `weight` its weight and `at` the sorted row of each pair.  A step of few tokens is routed and sorted
@@ -19,7 +19,7 @@ constexpr int kMaxExperts = 512, kMaxTop = 32, kSmallPairs = 1024, kSmallTokens 
 
 struct Router {
   const float* z;           // [T][ld], logits at col
-  const float* correction;  // [experts]
+  const float* correction;  // [experts]; null: none
   int* counts;              // [experts], zero before a large step's routing
   int* pair;                // [T * top][2]: expert, place among its rows (large steps)
   float* pair_weight;       // [T * top]
@@ -28,6 +28,7 @@ struct Router {
   float* weight;            // [T * top] by sorted row
   int* at;                  // [T * top] by pair
   int ld, col, experts, top, groups, keep, T;
+  int softmax, divide;      // scores are a softmax over all experts; weights are divided by their sum
   float scale, den_eps;
 };
 
@@ -39,14 +40,29 @@ __device__ __forceinline__ void choose(const Router& a, int t, float* buf, int l
   float* score = buf + a.experts;
   float* sums = buf + 2 * a.experts;
   float* kept = sums + a.groups;
-  float c[NE];
+  float c[NE], most = 0.0f, sum_exp = 1.0f;
+  if (a.softmax) {
+    most = -INFINITY;
+    sum_exp = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NE; ++i) {
+      c[i] = lane + 32 * i < a.experts ? z[lane + 32 * i] : -INFINITY;
+      most = fmaxf(most, c[i]);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) most = fmaxf(most, __shfl_xor_sync(0xffffffffu, most, o));
+#pragma unroll
+    for (int i = 0; i < NE; ++i) sum_exp += expf(c[i] - most);
+    sum_exp = warp_sum(sum_exp);
+  }
 #pragma unroll
   for (int i = 0; i < NE; ++i) {
     const int e = lane + 32 * i;
     c[i] = -INFINITY;
     if (e < a.experts) {
-      const float s = sigmoid(z[e]);
-      c[i] = s + a.correction[e];
+      const float s = a.softmax ? expf(z[e] - most) / sum_exp : sigmoid(z[e]);
+      // without a correction or groups, logits choose as their softmax does, and never tie where it underflows
+      c[i] = a.correction != nullptr ? s + a.correction[e] : (a.softmax && a.keep == a.groups ? z[e] : s);
       score[e] = s;
       choice[e] = c[i];
     }
@@ -111,7 +127,7 @@ __device__ __forceinline__ void choose(const Router& a, int t, float* buf, int l
       weight = s;
     }
   }
-  weight = weight / (sum + a.den_eps) * a.scale;
+  weight = (a.divide ? weight / (sum + a.den_eps) : weight) * a.scale;
   __syncwarp();
 }
 
@@ -247,14 +263,8 @@ struct Grouped {
   const float* weight;      // gated epilogue: factor of a sorted row's outputs
   int n, k, kp, experts, rows;   // rows: sorted rows in all
   int ldx, ldo, glu;        // glu: the gated epilogue over interleaved gate / up rows
-  float limit, alpha, offset;
+  Glu unit;
 };
-
-__device__ __forceinline__ float gated_unit(const Grouped& a, float g, float u) {
-  g = fminf(g, a.limit);
-  u = fminf(fmaxf(u, -a.limit), a.limit);
-  return g * sigmoid(a.alpha * g) * (u + a.offset);
-}
 
 constexpr int kFewWarps = 8;
 
@@ -330,7 +340,7 @@ __global__ void __launch_bounds__(kFewWarps * 32) few_kernel(Grouped a, const bf
           gv += red[w][2 * r][t];
           uv += red[w][2 * r + 1][t];
         }
-        if (row0 + 2 * r + 1 < a.n) out16[(size_t)(s0 + t) * a.ldo + (row0 >> 1) + r] = __float2bfloat16_rn(gated_unit(a, gv, uv) * a.weight[s0 + t]);
+        if (row0 + 2 * r + 1 < a.n) out16[(size_t)(s0 + t) * a.ldo + (row0 >> 1) + r] = __float2bfloat16_rn(glu(a.unit, gv, uv) * a.weight[s0 + t]);
       }
     }
     __syncthreads();     // the partial sums are read before the next rows overwrite them
@@ -387,7 +397,7 @@ __global__ void __launch_bounds__(256) expert_f32_kernel(Grouped a, const float*
       if (!a.glu) {
         if (r < a.n) out[(size_t)s * a.ldo + r] = acc[i][j];
       } else if ((j & 1) == 0 && r + 1 < a.n) {
-        out[(size_t)s * a.ldo + (r >> 1)] = gated_unit(a, acc[i][j], acc[i][j + 1]) * a.weight[s];
+        out[(size_t)s * a.ldo + (r >> 1)] = glu(a.unit, acc[i][j], acc[i][j + 1]) * a.weight[s];
       }
     }
   }
@@ -397,7 +407,7 @@ static bool fill(Router& a, const void* const* ptrs, const int* ints, const floa
   a.z = (const float*)ptrs[0]; a.correction = (const float*)ptrs[1]; a.counts = (int*)ptrs[2]; a.pair = (int*)ptrs[3]; a.pair_weight = (float*)ptrs[4];
   a.lists = (int*)ptrs[5]; a.token = (int*)ptrs[6]; a.weight = (float*)ptrs[7]; a.at = (int*)ptrs[8];
   a.ld = ints[0]; a.col = ints[1]; a.experts = ints[2]; a.top = ints[3]; a.groups = ints[4]; a.keep = ints[5]; a.T = T;
-  a.scale = floats[0]; a.den_eps = floats[1];
+  a.softmax = ints[6]; a.divide = ints[7]; a.scale = floats[0]; a.den_eps = floats[1];
   return T >= 1 && a.experts >= 1 && a.experts <= kMaxExperts && a.top >= 1 && a.top <= kMaxTop && a.groups >= 1 && a.experts % a.groups == 0 && a.keep >= 1 &&
          a.keep <= a.groups && a.top <= a.keep * (a.experts / a.groups) && (long long)T * a.top < (1ll << 30);
 }
@@ -415,7 +425,7 @@ extern "C" {
 int bonsai_lay_route_small(int top) { return top < 1 || top > bonsai::lay::kMaxTop ? 0 : min(bonsai::lay::kSmallTokens, bonsai::lay::kSmallPairs / top); }
 
 // Chooses and sorts.  ptrs = {logits, correction, counts, pair, pair_weight, lists, token, weight, at}, ints = {ld, col, experts, top,
-// groups, keep}, floats = {scale, den_eps}.  h bf16 [T][ldh] -> xs [T * top][ldx] in sorted order, `chunks` blocks of 8 columns (xs
+// groups, keep, softmax, divide}, floats = {scale, den_eps}.  h bf16 [T][ldh] -> xs [T * top][ldx] in sorted order, `chunks` blocks of 8 columns (xs
 // null: no copy).  Steps above bonsai_lay_route_small tokens need counts at zero (bonsai_lay_side_by_side leaves them so).
 int bonsai_lay_route(const void* const* ptrs, const int* ints, const float* floats, int T, const void* h, int ldh, int chunks, void* xs, int ldx,
                      cudaStream_t stream) {
@@ -440,12 +450,12 @@ int bonsai_lay_route(const void* const* ptrs, const int* ints, const float* floa
 // Projection of the sorted rows by their experts' matrices W [experts][n][kp], few rows per expert.  x bf16 (row token[s], or s when
 // token is null); glu: out bf16 [rows][n / 2] = gated unit * weight[s]; otherwise out f32 [rows][n].  slots: most experts chosen.
 int bonsai_lay_experts_few(const void* W, int experts, int n, int kp, const void* x, int ldx, const int* lists, const int* token, const float* weight, int rows,
-                           int slots, int per_expert, void* out, int ldo, int glu, float limit, float alpha, float offset, cudaStream_t stream) {
+                           int slots, int per_expert, void* out, int ldo, int glu, float limit, float alpha, float offset, float cubic, cudaStream_t stream) {
   using namespace bonsai::lay;
   if (experts < 1 || experts > kMaxExperts || n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || rows < 1 || slots < 1 || slots > experts ||
       ldo < (glu ? n / 2 : n) || (glu && (n % 2 != 0 || weight == nullptr)))
     return BONSAI_CUDA_BAD_ARG;
-  const Grouped a{(const bf16*)W, lists, token, weight, n, kp, kp, experts, rows, ldx, ldo, glu, limit, alpha, offset};
+  const Grouped a{(const bf16*)W, lists, token, weight, n, kp, kp, experts, rows, ldx, ldo, glu, Glu{limit, alpha, offset, cubic}};
   const dim3 grid((n + 15) / 16, slots);
 #define BONSAI_FEW(NT) launch(few_kernel<NT>, grid, kFewWarps * 32, 0, stream, 1, 0, a, (const bf16*)x, (float*)out, (bf16*)out)
   return per_expert <= 8 ? BONSAI_FEW(1) : (per_expert <= 16 ? BONSAI_FEW(2) : BONSAI_FEW(4));
@@ -454,12 +464,12 @@ int bonsai_lay_experts_few(const void* W, int experts, int n, int kp, const void
 
 // The same in 32 bits: x and out f32, at most `tokens` rows per expert.
 int bonsai_lay_experts_f32(const void* W, int experts, int n, int k, int kp, const float* x, int ldx, const int* lists, const int* token, const float* weight,
-                           int rows, int tokens, float* out, int ldo, int glu, float limit, float alpha, float offset, cudaStream_t stream) {
+                           int rows, int tokens, float* out, int ldo, int glu, float limit, float alpha, float offset, float cubic, cudaStream_t stream) {
   using namespace bonsai::lay;
   if (experts < 1 || experts > kMaxExperts || n < 1 || k < 1 || kp < k || ldx < k || rows < 1 || tokens < 1 || tokens > 64 * 65535 ||
       ldo < (glu ? n / 2 : n) || (glu && (n % 2 != 0 || weight == nullptr)))
     return BONSAI_CUDA_BAD_ARG;
-  const Grouped a{(const bf16*)W, lists, token, weight, n, k, kp, experts, rows, ldx, ldo, glu, limit, alpha, offset};
+  const Grouped a{(const bf16*)W, lists, token, weight, n, k, kp, experts, rows, ldx, ldo, glu, Glu{limit, alpha, offset, cubic}};
   return launch(expert_f32_kernel, dim3((n + 63) / 64, (tokens + 63) / 64, experts), 256, 0, stream, 1, 0, a, x, out);
 }
 

@@ -79,15 +79,31 @@ __device__ __forceinline__ void store_act4(float* p, float4 v) { *reinterpret_ca
 __device__ __forceinline__ float load_act(const bf16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ float load_act(const float* p) { return *p; }
 
-// Element d of a head whose first `dims` dimensions are turned by the angles of `rot` (cosine, sine per pair; null: no rotation);
-// pairs are (2i, 2i + 1), or (i, i + dims / 2).
-__device__ __forceinline__ float rotated(const float* v, int d, const float2* rot, int dims, int pairs) {
-  if (d >= dims || rot == nullptr) return v[d];
+// Element d of a head v(0), v(1), ... whose first `dims` dimensions are turned by the angles of `rot` (cosine, sine per pair; null: no
+// rotation); pairs are (2i, 2i + 1), or (i, i + dims / 2).
+template <typename V>
+__device__ __forceinline__ float rotated(V v, int d, const float2* rot, int dims, int pairs) {
+  if (d >= dims || rot == nullptr) return v(d);
   const int half = dims >> 1;
   const bool first = pairs ? (d & 1) == 0 : d < half;
   const float2 cs = rot[pairs ? d >> 1 : (first ? d : d - half)];
-  const float other = v[pairs ? d ^ 1 : (first ? d + half : d - half)];
-  return first ? v[d] * cs.x - other * cs.y : v[d] * cs.x + other * cs.y;
+  const float own = v(d), other = v(pairs ? d ^ 1 : (first ? d + half : d - half));
+  return first ? own * cs.x - other * cs.y : own * cs.x + other * cs.y;
+}
+
+__device__ __forceinline__ float rotated(const float* v, int d, const float2* rot, int dims, int pairs) {
+  return rotated([&](int j) { return v[j]; }, d, rot, dims, pairs);
+}
+
+// Clamped gated unit: g * sigmoid(alpha (g + cubic g^3)) * (u + up_offset) with g = min(gate, limit), u = clamp(up, -limit, limit).  With
+// alpha = 2 sqrt(2 / pi) and cubic = 0.044715 the first two factors are the tanh form of gelu: (1 + tanh(y)) / 2 = sigmoid(2 y).
+struct Glu {
+  float limit, alpha, up_offset, cubic;
+};
+__device__ __forceinline__ float glu(const Glu& a, float g, float u) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return g * sigmoid(a.alpha * fmaf(a.cubic * g * g, g, g)) * (u + a.up_offset);
 }
 
 constexpr float kLog2e = 1.4426950408889634f;

@@ -9,28 +9,20 @@
 //
 // `f32_kernel` is the 32-bit mode: f32 activations, the same bf16 weights (exact in f32), f32 FMA throughout.
 //
-// Epilogues: 0 = f32 store, 1 = clamped gated unit over interleaved gate / up rows:
-//   g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(alpha g) * (u + up_offset);
-// 2 = squared relu, 3 = the product itself in the activations' type.
+// Epilogues: 0 = f32 store, 1 = clamped gated unit over interleaved gate / up rows, 2 = squared relu, 3 = the product itself in the
+// activations' type, 4 = f32 store of limit * tanh(product / limit).
 #include "layered/layered.cuh"
 
 namespace bonsai {
 namespace lay {
 
-struct Glu {
-  float limit, alpha, up_offset;
-};
-
-__device__ __forceinline__ float glu(const Glu& a, float g, float u) {
-  g = fminf(g, a.limit);
-  u = fminf(fmaxf(u, -a.limit), a.limit);
-  return g * sigmoid(a.alpha * g) * (u + a.up_offset);
-}
-
 __device__ __forceinline__ float squared_relu(float v) {
   v = fmaxf(v, 0.0f);
   return v * v;
 }
+
+// the f32 outputs of epilogues 0 and 4
+__device__ __forceinline__ float capped(float v, int epi, const Glu& a) { return epi == 4 ? a.limit * tanhf(v / a.limit) : v; }
 
 constexpr int kWarps = 8;
 
@@ -89,7 +81,7 @@ __global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __res
 #pragma unroll
       for (int w = 0; w < kWarps; ++w) v += red[w][r][t];
       if (row0 + r >= n) continue;
-      if (epi == 0) out[(size_t)t * ldo + row0 + r] = v;
+      if (epi == 0 || epi == 4) out[(size_t)t * ldo + row0 + r] = capped(v, epi, act);
       else out16[(size_t)t * ldo + row0 + r] = __float2bfloat16_rn(epi == 2 ? squared_relu(v) : v);
     }
   } else {
@@ -147,7 +139,7 @@ __global__ void __launch_bounds__(256) f32_kernel(const bf16* __restrict__ W, in
     for (int j = 0; j < 4; ++j) {
       const int r = n0 + tn * 4 + j;
       if (epi != 1) {
-        if (r < n) out[(size_t)t * ldo + r] = epi == 2 ? squared_relu(acc[i][j]) : acc[i][j];
+        if (r < n) out[(size_t)t * ldo + r] = epi == 2 ? squared_relu(acc[i][j]) : capped(acc[i][j], epi, act);
       } else if ((j & 1) == 0 && r + 1 < n) {
         out[(size_t)t * ldo + (r >> 1)] = glu(act, acc[i][j], acc[i][j + 1]);
       }
@@ -161,13 +153,14 @@ __global__ void __launch_bounds__(256) f32_kernel(const bf16* __restrict__ W, in
 extern "C" {
 
 // W bf16 [n][kp] (kp a multiple of 128, columns past the layer's width zero), x bf16 [T][ldx] (ldx >= kp, finite in the
-// padding), T <= 32.  epi 0: out f32 [T][ldo]; epi 1: out16 bf16 [T][ldo] of n / 2 columns; epi 2 and 3: out16 bf16 [T][ldo].
+// padding), T <= 32.  epi 0 and 4: out f32 [T][ldo]; epi 1: out16 bf16 [T][ldo] of n / 2 columns; epi 2 and 3: out16 bf16 [T][ldo].
 int bonsai_lay_linear_few(const void* W, int n, int kp, const void* x, int ldx, int T, float* out, void* out16, int ldo, int epi, float limit,
-                          float alpha, float up_offset, cudaStream_t stream) {
+                          float alpha, float up_offset, float cubic, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || T < 1 || T > 32 || epi < 0 || epi > 3) return BONSAI_CUDA_BAD_ARG;
-  if ((epi == 0 && out == nullptr) || (epi != 0 && out16 == nullptr) || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
-  const Glu act{limit, alpha, up_offset};
+  if (n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || T < 1 || T > 32 || epi < 0 || epi > 4) return BONSAI_CUDA_BAD_ARG;
+  const bool f32_out = epi == 0 || epi == 4;
+  if ((f32_out && out == nullptr) || (!f32_out && out16 == nullptr) || (epi == 4 && !(limit > 0.0f)) || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
+  const Glu act{limit, alpha, up_offset, cubic};
   const dim3 grid((n + 15) / 16);
 #define BONSAI_FEW(NT) \
   launch(few_rows_kernel<NT>, grid, kWarps * 32, 0, stream, 1, 0, (const bf16*)W, n, kp, (const bf16*)x, ldx, T, out, (bf16*)out16, ldo, epi, act)
@@ -176,11 +169,11 @@ int bonsai_lay_linear_few(const void* W, int n, int kp, const void* x, int ldx, 
 }
 
 int bonsai_lay_linear_f32(const void* W, int n, int k, int kp, const float* x, int ldx, int T, float* out, int ldo, int epi, float limit, float alpha,
-                          float up_offset, cudaStream_t stream) {
+                          float up_offset, float cubic, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (n < 1 || k < 1 || kp < k || ldx < k || T < 1 || out == nullptr || epi < 0 || epi > 3 || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
+  if (n < 1 || k < 1 || kp < k || ldx < k || T < 1 || out == nullptr || epi < 0 || epi > 4 || (epi == 1 && n % 2 != 0) || (epi == 4 && !(limit > 0.0f))) return BONSAI_CUDA_BAD_ARG;
   return launch(f32_kernel, dim3((n + 63) / 64, (T + 63) / 64), 256, 0, stream, 1, 0, (const bf16*)W, n, k, kp, x, ldx, T, out, ldo, epi,
-                Glu{limit, alpha, up_offset});
+                Glu{limit, alpha, up_offset, cubic});
 }
 
 }  // extern "C"

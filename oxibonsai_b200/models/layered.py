@@ -23,8 +23,8 @@ import torch
 from ..ops import cuda_ops as K
 from ..ops import layered_ops as L
 from ..ops import nvtx
-from .layered_config import (AttentionSpec, Branch, ExpertsSpec, GatedMlpSpec, LatentAttentionSpec, LayeredConfig, LinearRecurrenceSpec, MlstmSpec,
-                             RotarySpec, SquaredReluMlpSpec)
+from .layered_config import (AttentionSpec, Branch, ExpertsSpec, GatedMlpSpec, LatentAttentionSpec, LayeredConfig, LinearRecurrenceSpec, MinGruSpec,
+                             MlstmSpec, RotarySpec, SelectiveScanSpec, SquaredReluMlpSpec)
 from .paged import RowCache, StatePool
 from .rope_scaling import geometric_slopes
 from .slot_state import SlotState
@@ -40,18 +40,43 @@ def _tensor(t) -> torch.Tensor:
 @dataclass
 class MlpWeights:
     pre_norm: torch.Tensor | None
-    norm: torch.Tensor
+    norm: torch.Tensor | None
     up: L.DenseWeight                # gated blocks: gate and up rows interleaved
     down: L.DenseWeight
     act: L.Glu | str
+    ff: int
+
+    @classmethod
+    def gated(cls, spec: GatedMlpSpec, matrix, prefix: str, norms, device) -> "MlpWeights":
+        """``matrix``: a checkpoint matrix by its name."""
+        return cls(*norms, L.DenseWeight([matrix(prefix + "gate"), matrix(prefix + "up")], device, interleave=True), L.DenseWeight([matrix(prefix + "down")], device),
+                   L.Glu(spec.limit, spec.alpha, spec.offset, spec.cubic), spec.ff)
+
+    @property
+    def nbytes(self) -> int:
+        return self.up.nbytes + self.down.nbytes
 
 
 @dataclass
 class ExpertWeights:
-    column: int                      # first router logit in the layer's projection
-    correction: torch.Tensor
+    """A mixture of experts.  Beside the mixer its router is part of the layer's projection; behind it, ``router`` reads the
+    feed-forward's input: the router's rows and the shared block's gate."""
+    column: int                      # first router logit in that projection
+    correction: torch.Tensor | None
     up: L.DenseWeight                # all experts' gate and up rows, interleaved, one expert below the other
     down: L.DenseWeight
+    experts: int
+    top: int
+    pre_norm: torch.Tensor | None = None
+    norm: torch.Tensor | None = None
+    router: L.DenseWeight | None = None
+    shared: MlpWeights | None = None
+
+    @property
+    def nbytes(self) -> int:
+        """Bytes a decode step must stream for one token."""
+        n = (self.up.nbytes + self.down.nbytes) * self.top // self.experts
+        return n + (0 if self.router is None else self.router.nbytes) + (0 if self.shared is None else self.shared.nbytes)
 
 
 @dataclass
@@ -77,11 +102,26 @@ class LatentWeights:
 
 
 @dataclass
+class ScanWeights:
+    """The projections inside a selective scan."""
+    read: L.DenseWeight              # three parts: step sizes (low rank), inputs, outputs
+    step: L.DenseWeight
+
+    @classmethod
+    def load(cls, m: SelectiveScanSpec, x: torch.Tensor, dt: torch.Tensor, device) -> "ScanWeights":
+        return cls(L.DenseWeight(list(torch.split(x, [m.rank, m.states, m.states])), device), L.DenseWeight([dt], device))
+
+    @property
+    def nbytes(self) -> int:
+        return self.read.nbytes + self.step.nbytes
+
+
+@dataclass
 class BranchWeights:
     columns: list[int]               # first output of each section in the layer's projection
     vectors: dict[str, torch.Tensor]
     offset: int                      # first column in the input of the output projection
-    latent: LatentWeights | None = None
+    inner: LatentWeights | ScanWeights | None = None
 
 
 @dataclass
@@ -92,6 +132,8 @@ class LayerWeights:
     out: L.DenseWeight               # the branches' output projections side by side
     branches: list[BranchWeights]
     mlp: MlpWeights | ExpertWeights | None
+    convs: list[torch.Tensor]        # per sublayer: the convolution of its input [taps, width], the current token's tap first
+    out_bias: torch.Tensor | None = None
 
 
 def branch_offsets(widths: Sequence[int]) -> tuple[list[int], int]:
@@ -117,8 +159,10 @@ class LayeredWeights:
         self.cfg, self.device = cfg, torch.device(device)
         m = lambda n: tensors[n].to(torch.bfloat16)
         v = lambda n: None if n is None else tensors[n].float().to(self.device)
-        self.embed = L.DenseWeight([m("embed")], self.device)      # also the output head
+        self.embed = L.DenseWeight([m("embed")], self.device)
+        self.head = L.DenseWeight([m("head")], self.device) if cfg.own_head else self.embed
         self.final_norm = v("final.norm")
+        self.loop_step = v("loop.step") if cfg.loop is not None else None
         self.layers: list[LayerWeights] = []
         for i, spec in enumerate(cfg.layer_specs):
             norms, p, parts, counts = cfg.norm_names(i), f"l{i}.mlp.", [], []
@@ -129,7 +173,8 @@ class LayeredWeights:
                     parts.append(m(f"l{i}.mix.{b.prefix}{name}")[at:at + rows])
                     first[name] = at + rows
                 counts.append(len(b.spec.sections))
-            if isinstance(spec.mlp, ExpertsSpec):
+            moe = spec.mlp if isinstance(spec.mlp, ExpertsSpec) else None
+            if moe is not None and cfg.side_by_side:
                 parts.append(m(p + "router"))
             proj = L.DenseWeight(parts, self.device)
             offsets, width = branch_offsets([b.spec.out_width for b in spec.mixer.branches])
@@ -138,21 +183,33 @@ class LayeredWeights:
             for b, off, count in zip(spec.mixer.branches, offsets, counts):
                 x = f"l{i}.mix.{b.prefix}"
                 out[:, off:off + b.spec.out_width] = m(x + "o")
-                latent = LatentWeights.load(b.spec, m(x + "uk"), m(x + "uv"), self.device) if isinstance(b.spec, LatentAttentionSpec) else None
-                branches.append(BranchWeights(proj.columns[at:at + count], {n: v(x + n) for n in b.spec.vectors}, off, latent))
+                inner = None
+                if isinstance(b.spec, LatentAttentionSpec):
+                    inner = LatentWeights.load(b.spec, m(x + "uk"), m(x + "uv"), self.device)
+                elif isinstance(b.spec, SelectiveScanSpec):
+                    inner = ScanWeights.load(b.spec, m(x + "x"), m(x + "dt"), self.device)
+                branches.append(BranchWeights(proj.columns[at:at + count], {n: v(x + n) for n in b.spec.vectors}, off, inner))
                 at += count
             mlp = None
-            assert cfg.side_by_side == isinstance(spec.mlp, ExpertsSpec) or spec.mlp is None, "experts stand beside the mixer, dense blocks behind it"
-            if isinstance(spec.mlp, ExpertsSpec):
-                names = [f"{p}e{e}." for e in range(spec.mlp.router.experts)]
+            assert moe is not None or not cfg.side_by_side or spec.mlp is None, "dense blocks stand behind the mixer"
+            if moe is not None:
+                r, names = moe.router, [f"{p}e{e}." for e in range(moe.router.experts)]
                 up = L.DenseWeight([torch.cat([m(n + c) for n in names]) for c in ("gate", "up")], self.device, interleave=True)
-                mlp = ExpertWeights(proj.columns[at], v(p + "correction"), up, L.DenseWeight([torch.cat([m(n + "down") for n in names])], self.device))
+                mlp = ExpertWeights(proj.columns[at] if cfg.side_by_side else 0, v(p + "correction") if r.corrected else None, up,
+                                    L.DenseWeight([torch.cat([m(n + "down") for n in names])], self.device), r.experts, r.top)
+                if not cfg.side_by_side:
+                    mlp.pre_norm, mlp.norm = map(v, norms[1])
+                    mlp.router = L.DenseWeight([m(p + "router")] + ([m(p + "shared.sg")] if moe.shared is not None else []), self.device)
+                if moe.shared is not None:
+                    mlp.shared = MlpWeights.gated(moe.shared, m, p + "shared.", (None, None), self.device)
             elif isinstance(spec.mlp, GatedMlpSpec):
-                up = L.DenseWeight([m(p + "gate"), m(p + "up")], self.device, interleave=True)
-                mlp = MlpWeights(*map(v, norms[1]), up, L.DenseWeight([m(p + "down")], self.device), L.Glu(spec.mlp.limit, spec.mlp.alpha, spec.mlp.offset))
+                mlp = MlpWeights.gated(spec.mlp, m, p, map(v, norms[1]), self.device)
             elif isinstance(spec.mlp, SquaredReluMlpSpec):
-                mlp = MlpWeights(*map(v, norms[1]), L.DenseWeight([m(p + "up")], self.device), L.DenseWeight([m(p + "down")], self.device), L.SQUARED_RELU)
-            self.layers.append(LayerWeights(*map(v, norms[0]), proj, L.DenseWeight([out], self.device), branches, mlp))
+                mlp = MlpWeights(*map(v, norms[1]), L.DenseWeight([m(p + "up")], self.device), L.DenseWeight([m(p + "down")], self.device), L.SQUARED_RELU, spec.mlp.ff)
+            convs = [L.conv_weight(v(f"l{i}.canon{n + 1}")) for n in range(len(norms))] if cfg.input_taps else []
+            biased = [b.prefix for b in spec.mixer.branches if b.spec.out_bias]
+            bias = sum(v(f"l{i}.mix.{x}o.b") for x in biased) if biased else None
+            self.layers.append(LayerWeights(*map(v, norms[0]), proj, L.DenseWeight([out], self.device), branches, mlp, convs, bias))
         torch.cuda.synchronize(self.device)
 
     @classmethod
@@ -163,23 +220,22 @@ class LayeredWeights:
     @property
     def packed_bytes(self) -> int:
         """Bytes a decode step must stream."""
-        n = self.embed.nbytes
-        for spec, l in zip(self.cfg.layer_specs, self.layers):
-            mlp = 0 if l.mlp is None else l.mlp.up.nbytes + l.mlp.down.nbytes
-            if isinstance(spec.mlp, ExpertsSpec):                # of one token
-                mlp = mlp * spec.mlp.router.top // spec.mlp.router.experts
-            n += l.proj.nbytes + l.out.nbytes + mlp + sum(b.latent.nbytes for b in l.branches if b.latent is not None)
-        return n
+        layer = [l.proj.nbytes + l.out.nbytes + (0 if l.mlp is None else l.mlp.nbytes) + sum(b.inner.nbytes for b in l.branches if b.inner is not None)
+                 for l in self.layers]
+        return self.head.nbytes + sum(layer[r.layer] for r in self.cfg.runs)
 
 
 def new_row_cache(cfg: LayeredConfig, num_pages: int, page_size: int, exact: bool, device) -> RowCache:
+    """Rows by the number of a layer's run."""
     layers = {}
-    for i in cfg.attention_layers:
-        s = cfg.attention(i)
+    for n, run in enumerate(cfg.runs):
+        if run.layer not in cfg.attention_layers:
+            continue
+        s = cfg.attention(run.layer)
         if isinstance(s, LatentAttentionSpec):
-            layers[i] = (1, L.lib().bonsai_lay_latent_row(s.rank, s.rot_dim), "latent")
+            layers[n] = (1, L.lib().bonsai_lay_latent_row(s.rank, s.rot_dim), "latent")
         elif s.kv_from is None:
-            layers[i] = (s.kv_heads, L.lib().bonsai_lay_attn_row(max(s.dim, s.value_dim)), "shared" if s.vdim is None else "separate")
+            layers[n] = (s.kv_heads, L.lib().bonsai_lay_attn_row(s.row_dim), "shared" if s.vdim is None else "separate")
     return RowCache(layers, num_pages, page_size, K.KV_F32 if exact else K.KV_BF16, torch.float32 if exact else torch.bfloat16, device)
 
 
@@ -191,21 +247,33 @@ def state_dims(m: MlstmSpec | LinearRecurrenceSpec) -> tuple[int, int]:
     return l.bonsai_lay_rec_dim(m.dim), l.bonsai_lay_rec_vdim(m.vdim)
 
 
-def runs_chunked(m: MlstmSpec | LinearRecurrenceSpec) -> bool:
+def runs_chunked(m) -> bool:
     """Whether portions of prompts go to the tensor cores (longer keys take the token-by-token kernel)."""
+    if not isinstance(m, (MlstmSpec, LinearRecurrenceSpec)):
+        return False
     return m.dim <= (L.lib().bonsai_lay_mlstm_chunk_dim() if isinstance(m, MlstmSpec) else L.lib().bonsai_lay_rec_chunk_dim())
 
 
 def new_state_pool(cfg: LayeredConfig, num_rows: int, device) -> StatePool:
+    """State by the number of a layer's run."""
     layers = {}
-    for i in cfg.recurrent_layers:
-        m = cfg.recurrence(i)
-        d, e = state_dims(m)
-        layers[i] = {"S": (m.heads, d, e)}
-        if isinstance(m, MlstmSpec):
-            layers[i].update({"n": (m.heads, e // 64, d), "m": (m.heads, e // 64)})
-        elif m.conv:
-            layers[i]["conv"] = (m.conv, m.conv_channels)
+    for n, run in enumerate(cfg.runs):
+        state = {f"canon{i + 1}": (cfg.input_taps, cfg.width) for i in range(len(cfg.norm_names(run.layer)))} if cfg.input_taps else {}
+        if run.layer in cfg.recurrent_layers:
+            m = cfg.recurrence(run.layer)
+            if isinstance(m, MinGruSpec):
+                state["S"] = (m.width,)
+            elif isinstance(m, SelectiveScanSpec):
+                state.update({"S": (m.channels, L.lib().bonsai_lay_scan_states(m.states)), "conv": (m.conv, m.channels)})
+            else:
+                d, e = state_dims(m)
+                state["S"] = (m.heads, d, e)
+                if isinstance(m, MlstmSpec):
+                    state.update({"n": (m.heads, e // 64, d), "m": (m.heads, e // 64)})
+                elif m.conv:
+                    state["conv"] = (m.conv, m.conv_channels)
+        if state:
+            layers[n] = state
     return StatePool(layers, num_rows, device)
 
 
@@ -295,6 +363,7 @@ class SegmentCost:
 MLSTM_COST = SegmentCost(1, 1.0, 1.5, 0.5, 0.6, 4)
 RECURRENCE_COST = SegmentCost(2, 1.55, 1.45, 2.0, 0.3, 2)
 WIDE_RECURRENCE_COST = SegmentCost(1, 1.0, 1.35, 1.2, 0.6, 2)
+SCAN_COST = SegmentCost(4, 1.0, 1.9, 2.0, 0.1, 2)
 
 
 @dataclass(frozen=True)
@@ -304,7 +373,9 @@ class SegmentPlan:
     cost: SegmentCost
 
 
-def segment_plan(m: MlstmSpec | LinearRecurrenceSpec) -> SegmentPlan:
+def segment_plan(m: MlstmSpec | LinearRecurrenceSpec | SelectiveScanSpec) -> SegmentPlan:
+    if isinstance(m, SelectiveScanSpec):
+        return SegmentPlan(-(-m.channels // L.lib().bonsai_lay_scan_channels(m.states)), SCAN_COST)
     d, e = state_dims(m)
     cost = MLSTM_COST if isinstance(m, MlstmSpec) else (RECURRENCE_COST if d <= 128 else WIDE_RECURRENCE_COST)
     return SegmentPlan(m.heads * e // 64, cost)
@@ -326,6 +397,8 @@ def plan_segments(lengths: Sequence[int], plan: SegmentPlan, sms: int) -> int:
 
 
 class AttentionMixer:
+    """``index``: the number of the layer's run, here and below."""
+
     def __init__(self, r: "LayeredRunner", index: int, branch: Branch, w: BranchWeights, out: torch.Tensor):
         self.r, self.spec, self.out = r, branch.spec, out
         spec, cols = self.spec, dict(zip((n for n, _ in branch.spec.sections), w.columns))
@@ -335,18 +408,22 @@ class AttentionMixer:
         slopes = None if spec.slope_exponent is None else geometric_slopes(spec.heads, spec.slope_exponent).to(r.device)
         ints = [r.proj.stride(0), cols["q"], cols.get("k", -1), cols.get("v", 0), cols.get("g", -1), out.stride(0), spec.heads, spec.kv_heads, spec.dim,
                 spec.value_dim, r.max_pages, r.kv.page_size, spec.window, spec.keep_first, int(spec.normed), 0 if rot is None else rot.dims,
-                int(rot is not None and rot.interleaved)]
-        floats = [r.cfg.eps, spec.scale, branch.scale, spec.softcap, spec.temp_coef, spec.temp_every]
-        self.call = {id(rows): L.MixerCall([r.proj, w.vectors.get("q.norm"), w.vectors.get("k.norm"), slopes, rows.positions, rows.slots, r.block_table,
-                                            r.kv.rows[source], r.kv.factors.get(source), r.kv.values.get(source), out, w.vectors.get("sink"),
-                                            None if rot is None else r.angles(rot)], ints, floats)
+                int(rot is not None and rot.interleaved), spec.chunk, spec.maps, int(spec.element_gate)]
+        vec, lam, left = w.vectors, 0.0, 1.0
+        if spec.difference is not None:
+            dot = lambda i: float(torch.exp((vec[f"lq{i}"].double() * vec[f"lk{i}"].double()).sum()))
+            lam, left = dot(1) - dot(2) + spec.difference, 1.0 - spec.difference
+        floats = [r.cfg.eps, spec.scale, branch.scale, spec.softcap, spec.temp_coef, spec.temp_every, lam, left]
+        self.call = {id(rows): L.MixerCall([r.proj, vec.get("q.norm"), vec.get("k.norm"), slopes, rows.positions, rows.slots, r.block_table,
+                                            r.kv.rows[source], r.kv.factors.get(source), r.kv.values.get(source), out, vec.get("sink"),
+                                            None if rot is None else r.angles(rot), vec.get("q.b"), vec.get("k.b"), vec.get("v.b")], ints, floats)
                      for rows in (r.slot_rows, r.batch_rows)}
 
     def splits(self, batch: int) -> int:
         """KV splits of one row's decode attention: about a CTA per SM, and no more than there are 16-token tiles per warp."""
         s = self.spec
-        seen = self.r.max_seq if s.window <= 0 else min(self.r.max_seq, s.window + s.keep_first + 32)
-        n, ctas = 1, batch * s.kv_heads * (-(-s.group // 16))
+        seen = self.r.max_seq if s.visible <= 0 else min(self.r.max_seq, s.visible + 32)
+        n, ctas = 1, batch * s.kv_heads * (-(-s.maps * s.group // 16))
         while n < 8 and ctas * n * 2 <= 160 and n * 2 * 128 <= seen + 127:
             n *= 2
         return n
@@ -378,12 +455,12 @@ class LatentAttentionMixer:
         q, c, rot, g = w.columns
         row = self.row = r.kv.rows[index].shape[-1]
         self.groups = -(-s.heads // L.lib().bonsai_lay_latent_group(s.heads))
-        self.lat_ld, self.kv_ld = max(row, w.latent.expand.kp), w.latent.expand.n
+        self.lat_ld, self.kv_ld = max(row, w.inner.expand.kp), w.inner.expand.n
         absorbed, partial, sums = r.latent_scratch(row, self.lat_ld, s.heads, L.round_up(s.rank, 16), self.kv_ld)
         ints = [r.proj.stride(0), q, c, rot, g, out.stride(0), s.heads, s.dim, s.rot_dim, s.vdim, s.rank, r.max_pages, r.kv.page_size,
                 absorbed.shape[0], partial.shape[0], r.kv.num_pages]
         self.call = {id(rows): L.MixerCall([r.proj, w.vectors["dkv.norm"], r.angles(s.rotary), rows.positions, rows.slots, r.block_table, r.kv.rows[index],
-                                            w.latent.keys, w.latent.values, absorbed, partial, sums, r.status, out], ints, [r.cfg.eps, s.scale, branch.scale])
+                                            w.inner.keys, w.inner.values, absorbed, partial, sums, r.status, out], ints, [r.cfg.eps, s.scale, branch.scale])
                      for rows in (r.slot_rows, r.batch_rows)}
 
     def splits(self, rows: int) -> tuple[int, int]:
@@ -411,7 +488,7 @@ class LatentAttentionMixer:
         for g in st.contexts:
             lat, kv = r.latents[self.row, self.lat_ld], r.expanded[: r.context_rows * self.kv_ld].view(-1, self.kv_ld)
             K.check(lib.bonsai_lay_latent_gather(*a, g.contexts, g.count, g.longest, lat.data_ptr(), self.lat_ld, stream), "latent_gather")
-            L.linear(self.w.latent.expand, lat, g.rows, kv, r.scratch)
+            L.linear(self.w.inner.expand, lat, g.rows, kv, r.scratch)
             K.check(lib.bonsai_lay_latent_prompt(*a, g.portions, g.contexts, g.tiles, g.n_tiles, kv.data_ptr(), self.kv_ld, lat.data_ptr(), self.lat_ld, stream),
                     "latent_prompt")
 
@@ -522,7 +599,70 @@ class LinearRecurrenceMixer:
         return 1 if self.fused else 2
 
 
-MIXERS = {"attention": AttentionMixer, "latent": LatentAttentionMixer, "mlstm": MlstmMixer, "recurrence": LinearRecurrenceMixer}
+class MinGruMixer:
+    def __init__(self, r: "LayeredRunner", index: int, branch: Branch, w: BranchWeights, out: torch.Tensor):
+        self.r, self.spec, vec = r, branch.spec, w.vectors
+        assert branch.scale == 1.0, "a minGRU output is not scaled"
+        self.call = {id(rows): L.MixerCall([r.proj, vec["z.b"], vec["x.b"], r.states.tensors[index]["S"], rows.positions, rows.slots, r.state_table, out],
+                                           [r.proj.stride(0), *w.columns, out.stride(0), self.spec.width], [])
+                     for rows in (r.slot_rows, r.batch_rows)}
+
+    def cluster(self, portions: int, tokens: int) -> int:
+        """CTAs that share a portion: about two per SM, and no more than have tokens in one round."""
+        n, ctas = 1, portions * -(-self.spec.width // 32)
+        while n < 8 and 2 * n * ctas <= 2 * self.r.scratch.sms and 2 * n * L.lib().bonsai_lay_gru_tokens() <= tokens:
+            n *= 2
+        return n
+
+    def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
+        lib, a, exact = L.lib(), self.call[id(rows)].args, int(self.r.exact)
+        if st.singles:
+            K.check(lib.bonsai_lay_gru_step(*a, st.singles, exact, stream), "gru_step")
+        if st.portions:
+            n = self.cluster(st.portions, (st.rows - st.singles) // st.portions)
+            K.check(lib.bonsai_lay_gru_scan(*a, st.entries, st.portions, n, exact, stream), "gru_scan")
+
+    def launches(self) -> int:
+        return 1
+
+
+class SelectiveScanMixer:
+    def __init__(self, r: "LayeredRunner", index: int, branch: Branch, w: BranchWeights, out: torch.Tensor):
+        self.r, self.spec, self.w, s, vec = r, branch.spec, w.inner, branch.spec, w.vectors
+        assert branch.scale == 1.0, "a selective scan's output is not scaled"
+        self.plan = segment_plan(s)
+        state, (x_col, z_col), (dt_col, b_col, c_col) = r.states.tensors[index], w.columns, w.inner.read.columns
+        self.x, self.bc, self.dt, self.low = r.scan_buffers(s, w.inner)
+        A = torch.zeros((s.channels, state["S"].shape[-1]), dtype=torch.float32, device=r.device)
+        A[:, : s.states] = -torch.exp(vec["A_log"])
+        taps = L.conv_weight(vec["conv"])
+        ints = [r.proj.stride(0), z_col, self.bc.stride(0), b_col, c_col, self.dt.stride(0), self.x.stride(0), out.stride(0), s.channels, s.states]
+        self.call, self.conv = {}, {}
+        for rows in (r.slot_rows, r.batch_rows):
+            self.call[id(rows)] = L.MixerCall([r.proj, self.bc, self.dt, self.x, vec["dt.b"], A, vec["D"], state["S"], rows.positions, rows.slots, r.state_table, out,
+                                               *r.scan_scratch], ints, [])
+            self.conv[id(rows)] = L.Conv(r.proj, x_col, s.channels, taps, vec["conv.b"], state["conv"], rows, r.state_table, self.x, silu=True)
+
+    def __call__(self, rows: Rows, st: StepShape, stream: int, early: bool) -> None:
+        lib, a, r, s, T = L.lib(), self.call[id(rows)].args, self.r, self.spec, st.rows
+        exact = int(r.exact)
+        self.conv[id(rows)](st)
+        L.linear(self.w.read, self.x, T, self.bc, r.scratch)
+        if not r.exact:
+            L.narrow(self.bc, 0, s.rank, T, self.low)
+        L.linear(self.w.step, self.bc if r.exact else self.low, T, self.dt, r.scratch)
+        if st.singles:
+            K.check(lib.bonsai_lay_scan_step(*a, st.singles, exact, stream), "scan_step")
+        if st.portions:
+            segs, n, prompts = (0, 0, 0) if r.exact else st.cut(self.plan)
+            K.check(lib.bonsai_lay_scan(*a, st.entries, st.portions, segs, n, prompts, exact, stream), "scan")
+
+    def launches(self) -> int:
+        return 4 if self.r.exact else 5
+
+
+MIXERS = {"attention": AttentionMixer, "latent": LatentAttentionMixer, "mlstm": MlstmMixer, "recurrence": LinearRecurrenceMixer, "mingru": MinGruMixer,
+          "selective": SelectiveScanMixer}
 
 
 class LayeredRunner(SlotState):
@@ -553,11 +693,13 @@ class LayeredRunner(SlotState):
         self.x = torch.zeros((cap, cfg.width), **f32)
         # input of the next projection; without a norm in between, that of the exact mode is the stream itself
         self.h = self.x if exact and not (cfg.pre_norm or cfg.side_by_side) else self.act_buffer(cfg.width, shared=False)
+        self.n32 = torch.zeros((cap if cfg.input_taps else 1, L.round_up(cfg.width, 4)), **f32)     # what a convolution reads
         self.normed = self.act_buffer(cfg.width, shared=False)
         self.y = torch.zeros((cap, L.round_up(cfg.width, 4)), **f32)
         self.proj = torch.zeros((cap, max(L.round_up(l.proj.n, 4) for l in weights.layers)), **f32)
         recurrent = [cfg.recurrence(i) for i in cfg.recurrent_layers]
-        self.head_out = torch.zeros((cap, L.round_up(max((m.out_width for m in recurrent), default=4), 4)), **f32)
+        heads = [m.out_width for m in recurrent if isinstance(m, (MlstmSpec, LinearRecurrenceSpec))]
+        self.head_out = torch.zeros((cap if heads else 1, L.round_up(max(heads, default=4), 4)), **f32)
         # prepared queries, keys and values of prompt rows
         linear = [m for m in recurrent if isinstance(m, LinearRecurrenceSpec)]
         width = max((L.lib().bonsai_lay_rec_features_width(m.heads, m.groups, m.dim, m.vdim) for m in linear), default=8)
@@ -565,7 +707,12 @@ class LayeredRunner(SlotState):
         # states of the segments a long prompt is cut into (layers run one after another and share them)
         chunked = [] if exact else [m for m in recurrent if runs_chunked(m)]
         shapes = [(m.heads, *state_dims(m)) for m in chunked]
-        self.segment_plans = sorted({segment_plan(m) for m in chunked}, key=lambda p: p.ctas)
+        scans = [m for m in recurrent if isinstance(m, SelectiveScanSpec)]
+        self.segment_plans = sorted({segment_plan(m) for m in chunked + ([] if exact else scans)}, key=lambda p: p.ctas)
+        parts = 0 if exact else MAX_SEGMENTS
+        self.scan_scratch = [torch.empty(max(1, parts * max((m.channels * n(m) for m in scans), default=0)), **f32) for n in
+                             (lambda m: L.lib().bonsai_lay_scan_states(m.states), lambda m: 1)]
+        self._scan_buffers: dict[tuple, list[torch.Tensor]] = {}
         segs = MAX_SEGMENTS if shapes else 0
         self.segment_scratch = [torch.empty(max(1, segs * max((f(*s) for s in shapes), default=0)), **f32) for f in
                                 (lambda h, d, e: h * d * e, lambda h, d, e: h * d * e // 64, lambda h, d, e: h * e // 64, lambda h, d, e: h * e // 32)]
@@ -579,23 +726,29 @@ class LayeredRunner(SlotState):
         # row metadata: decode steps use the slot tensors as they are; a mixed batch uploads [tokens | positions | slots | lists]
         self.slot_rows = Rows(self.tokens, self.positions, torch.arange(max_batch, **i32))
         attention = [cfg.attention(i) for i in cfg.attention_layers]
-        self._tile_sizes = sorted({64 // s.group for s in attention if isinstance(s, AttentionSpec)})
+        conv = {L.lib().bonsai_lay_conv_rows()} if cfg.input_taps or scans else set()
+        self._tile_sizes = sorted({64 // s.group for s in attention if isinstance(s, AttentionSpec)} | conv)
         self._expands = not exact and any(isinstance(s, LatentAttentionSpec) for s in attention)
         self._meta = torch.zeros(3 * cap + 4 * cap + 8 * MAX_SEGMENTS * len(self.segment_plans) + 2 * cap * len(self._tile_sizes) + 2 * cap + 12 * max_batch + 64, **i32)
         self.batch_rows = Rows(*(self._meta[i * cap:(i + 1) * cap] for i in range(3)))
         self._host = [torch.zeros(self._meta.numel(), dtype=torch.int32).pin_memory() for _ in range(2)]
         self._host_free = [torch.cuda.Event() for _ in range(2)]
         self._turn = 0
-        self.mixers, self.mixer_out = [], []           # per layer: the branches' mixers and the buffer they write
-        for i, (spec, w) in enumerate(zip(cfg.layer_specs, weights.layers)):
+        self.runs = cfg.runs
+        self.mixers, self.mixer_out = [], []           # per run: the branches' mixers and the buffer they write
+        for n, run in enumerate(self.runs):
+            spec, w = cfg.layer_specs[run.layer], weights.layers[run.layer]
             widths = tuple(b.spec.out_width for b in spec.mixer.branches)
             out = self.act_buffer(*widths)
             self.mixer_out.append(out)
-            self.mixers.append([MIXERS[b.spec.kind](self, i, b, bw, out[:, bw.offset:]) for b, bw in zip(spec.mixer.branches, w.branches)])
+            self.mixers.append([MIXERS[b.spec.kind](self, n, b, bw, out[:, bw.offset:]) for b, bw in zip(spec.mixer.branches, w.branches)])
         specs = [cfg.experts(i) for i in cfg.expert_layers]
         shared = L.ExpertScratch(cap, cfg.width, specs, exact, dev) if specs else None
-        self.experts = {i: L.Routing(cfg.experts(i), w.mlp.up, w.mlp.down, w.mlp.correction, self.proj, w.mlp.column, shared)
+        routers = [weights.layers[i].mlp.router for i in cfg.expert_layers]
+        self.router_out = torch.zeros((cap, max((L.round_up(w.n, 4) for w in routers if w is not None), default=4)), **f32) if routers and not cfg.side_by_side else self.proj
+        self.experts = {i: L.Routing(cfg.experts(i), w.mlp.up, w.mlp.down, w.mlp.correction, self.router_out, w.mlp.column, shared)
                         for i, w in enumerate(weights.layers) if i in cfg.expert_layers}
+        self.row_steps = {id(rows): self._row_steps(rows) for rows in (self.slot_rows, self.batch_rows)} if cfg.row_steps else None
         self._branch, self._forked = torch.cuda.Stream(dev), False
         self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
 
@@ -622,6 +775,17 @@ class LayeredRunner(SlotState):
                                                 torch.empty((parts, heads, 2), **f32)]
         return self._absorbed[row, heads, rank]
 
+    def scan_buffers(self, m: SelectiveScanSpec, w: ScanWeights) -> list[torch.Tensor]:
+        """Convolved channels, their projection, step sizes, and the 16-bit low-rank part of one selective-scan layer (layers of equal
+        sizes share them; the padding of what projections read stays zero)."""
+        key = (m.channels, m.states, m.rank)
+        if key not in self._scan_buffers:
+            new = lambda n, ld, dtype: torch.zeros((n, ld), dtype=dtype, device=self.device)
+            act, cap = torch.float32 if self.exact else torch.bfloat16, self.capacity
+            self._scan_buffers[key] = [new(cap, L.round_up(m.channels, 4) if self.exact else w.read.kp, act), new(cap, L.round_up(w.read.n, 4), torch.float32),
+                                       new(cap, L.round_up(m.channels, 4), torch.float32), new(1 if self.exact else cap, w.step.kp, torch.bfloat16)]
+        return self._scan_buffers[key]
+
     def act_buffer(self, *widths: int, shared: bool = True) -> torch.Tensor:
         """Input buffer of a projection that reads blocks of ``widths`` columns (:func:`branch_offsets`): f32 in the exact mode, else
         bf16 padded to the tensor-core width.  One per layout, so that the padding never holds another layer's values."""
@@ -635,7 +799,7 @@ class LayeredRunner(SlotState):
 
     # ---- slots ------------------------------------------------------------------------------------------------------------------
     def bind_state(self, slot: int) -> None:
-        if self.cfg.recurrent_layers and slot not in self._state_row:
+        if self.cfg.has_state and slot not in self._state_row:
             row = self._state_row[slot] = self.states.alloc()
             self.state_table[slot] = row
 
@@ -655,8 +819,75 @@ class LayeredRunner(SlotState):
             raise ValueError("the layer-list decoders have one cache format per engine")
 
     # ---- one step ------------------------------------------------------------------------------------------------------------------
+    def _row_steps(self, rows: Rows) -> list[L.RowStep]:
+        """The row steps of designs that take the general kernel: the start, one behind each sublayer of each run, and the final norm of
+        listed rows.  Each leaves the next sublayer's input; the last one behind a sublayer the final norm of all rows."""
+        cfg, w = self.cfg, self.w
+        common = dict(eps=cfg.eps, groups=cfg.norm_groups or 1)
+        subs = [(n, run, j) for n, run in enumerate(self.runs) for j in range(len(cfg.norm_names(run.layer)))]
+
+        def following(k: int) -> dict:
+            """What comes between sublayer ``k`` - 1 and sublayer ``k``."""
+            if k == len(subs):
+                return dict(h=self.normed, next_norm=w.final_norm)
+            n, run, j = subs[k]
+            l = w.layers[run.layer]
+            a = dict(h=self.h, next_norm=l.pre_norm if j == 0 else l.mlp.pre_norm)
+            if cfg.input_taps:
+                a.update(conv=(l.convs[j], self.states.tensors[n][f"canon{j + 1}"]), n32=self.n32)
+            if j == 0 and run.begins is not None:
+                a["step"] = w.loop_step[run.begins]
+                if run.begins > 0:
+                    a.update(table=w.embed.data, scale=cfg.embed_scale)
+            return a
+        new = lambda **a: L.RowStep(self.x, a.pop("h"), rows, self.state_table, **common, **a)
+        steps = [new(fresh=True, **{**following(0), "table": w.embed.data, "scale": cfg.embed_scale})]
+        for k, (n, run, j) in enumerate(subs):
+            l, a = w.layers[run.layer], following(k + 1)
+            if j == 0:
+                a.update(y=self.y, bias=l.out_bias, w=l.norm)
+            else:
+                moe = isinstance(l.mlp, ExpertWeights)
+                a["w"] = l.mlp.norm
+                if not moe or l.mlp.shared is not None:
+                    a["y"] = self.y
+                if moe and l.mlp.shared is not None:
+                    a["gate"] = self.router_out[:, l.mlp.router.columns[1]:]
+            steps.append(new(mult=cfg.residual_mult, **a))
+        steps.append(new(h=self.normed, next_norm=w.final_norm))
+        return steps
+
+    def _looped_layers(self, rows: Rows, st: StepShape) -> None:
+        """:meth:`_layers` of designs whose row steps take the general kernel."""
+        T, s, steps = st.rows, K.stream(), iter(self.row_steps[id(rows)])
+        next(steps)(T, st)
+        for n, run in enumerate(self.runs):
+            w = self.w.layers[run.layer]
+            L.linear(w.proj, self.h, T, self.proj, self.scratch)
+            for k, mixer in enumerate(self.mixers[n]):
+                mixer(rows, st, s, early=k > 0)
+            L.linear(w.out, self.mixer_out[n], T, self.y, self.scratch)
+            next(steps)(T, st)
+            if w.mlp is None:
+                continue
+            experts = self.experts.get(run.layer)
+            block = w.mlp
+            if experts is not None:
+                L.linear(w.mlp.router, self.h, T, self.router_out, self.scratch)
+                self._beside(experts, self.h, T)
+                block = w.mlp.shared
+            if block is not None:
+                act = self.act_buffer(block.ff)
+                L.linear(block.up, self.h, T, act, self.scratch, block.act)
+                L.linear(block.down, act, T, self.y, self.scratch)
+            if experts is not None:
+                self._join()
+            next(steps)(T, st, experts)
+
     def _layers(self, rows: Rows, st: StepShape, final: bool = False) -> None:
         """Embedding and layers.  ``final``: the last residual step leaves the final norm of all rows in ``normed``."""
+        if self.row_steps is not None:
+            return self._looped_layers(rows, st)
         cfg, T, s = self.cfg, st.rows, K.stream()
         x, h, layers = self.x, self.h, self.w.layers
         copy = None if h is x else h
@@ -685,7 +916,8 @@ class LayeredRunner(SlotState):
                 L.norm_add(x, self.y, w.mlp.norm, cfg.eps, T, after, following)
 
     def _beside(self, experts: L.Routing, h: torch.Tensor, T: int) -> None:
-        """The experts of a layer, which need its projection only: in a captured decode step, a branch beside the mixer's kernels."""
+        """The experts of a layer, which need the router's projection only: in a captured decode step, a branch beside the mixer's kernels
+        or the shared block."""
         main = torch.cuda.current_stream(self.device)
         self._forked = torch.cuda.is_current_stream_capturing()
         if not self._forked:
@@ -701,14 +933,21 @@ class LayeredRunner(SlotState):
 
     def _head(self, row_list: int, count: int, out: torch.Tensor) -> None:
         """Logits of ``count`` rows (device address of their indices) into ``out`` [count, vocab]."""
-        L.norm_rows(self.x, row_list, count, self.w.final_norm, self.cfg.eps, self.normed, self.cfg.layer_norm)
-        L.linear(self.w.embed, self.normed, count, out, self.scratch)
+        if self.row_steps is None:
+            L.norm_rows(self.x, row_list, count, self.w.final_norm, self.cfg.eps, self.normed, self.cfg.layer_norm)
+        else:
+            self.row_steps[id(self.batch_rows)][-1](count, None, norm_of=row_list)
+        self._logits(count, out)
+
+    def _logits(self, count: int, out: torch.Tensor) -> None:
+        """The head over the first rows of ``normed``."""
+        L.linear(self.w.head, self.normed, count, out, self.scratch, L.SoftCap(self.cfg.logit_cap) if self.cfg.logit_cap > 0 else None)
 
     def step_eager(self, batch: int, sample: bool = True, lm_head: bool = True, masked: bool = False) -> None:
         """One token for each of the slots 0 .. batch-1 (tokens and positions are read from the slot tensors)."""
         self._layers(self.slot_rows, StepShape(batch, batch, batch), final=lm_head)
         if lm_head:
-            L.linear(self.w.embed, self.normed, batch, self.logits, self.scratch)
+            self._logits(batch, self.logits)
         if sample:
             self.sample_rows(0, batch, masked, advance=True)
 
@@ -717,8 +956,10 @@ class LayeredRunner(SlotState):
         key = (batch, sample, masked)
         g = self._graphs.get(key)
         if g is None:
-            for mlp in (s.mlp for s in self.cfg.layer_specs if isinstance(s.mlp, (GatedMlpSpec, SquaredReluMlpSpec))):
-                self.act_buffer(mlp.ff)                        # allocated outside the capture
+            for w in self.w.layers:                            # allocated outside the capture
+                block = w.mlp.shared if isinstance(w.mlp, ExpertWeights) else w.mlp
+                if block is not None:
+                    self.act_buffer(block.ff)
             g = self._graphs[key] = K.capture_graph(self.device, lambda: self.step_eager(batch, sample, masked=masked))
         mark = nvtx.push(f"decode_step[batch={batch}]")
         g.replay()
@@ -836,7 +1077,13 @@ class LayeredRunner(SlotState):
     def kernel_launches(self, batch: int, sample: bool = True) -> int:
         """Launches of one decode step (each is one of this library's kernels)."""
         n = 2 + int(sample)
-        for i, (spec, mixers) in enumerate(zip(self.cfg.layer_specs, self.mixers)):
-            mlp = self.experts[i].launches(batch) if i in self.experts else (3 if spec.mlp is not None else 0)
-            n += 3 + sum(m.launches() for m in mixers) + mlp
+        for run, mixers in zip(self.runs, self.mixers):
+            mlp = self.w.layers[run.layer].mlp
+            if mlp is None:
+                k = 0
+            elif isinstance(mlp, ExpertWeights):       # behind the mixer: its own projection and row step, and the shared block
+                k = self.experts[run.layer].launches(batch) + (0 if self.cfg.side_by_side else 2) + (0 if mlp.shared is None else 2)
+            else:
+                k = 3
+            n += 3 + sum(m.launches() for m in mixers) + k
         return n

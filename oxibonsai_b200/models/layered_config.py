@@ -24,6 +24,8 @@ MAX_RANK = 512              # latent size of a compressed cache
 MAX_LATENT_ROW = 640        # that and the shared key part, each padded to 16
 MAX_EXPERTS = 512
 MAX_CHOSEN = 32             # experts of a token
+MAX_TAPS = 16               # of a convolution over tokens
+MAX_SCAN_STATES = 256       # per channel
 
 
 class LayeredConfigError(ValueError):
@@ -41,12 +43,17 @@ class MixerSpec:
     def inner(self) -> dict[str, tuple[int, int]]:
         return {}
 
+    @property
+    def out_bias(self) -> bool:
+        """Whether the output projection has a bias ("o.b")."""
+        return False
+
 
 @dataclass(frozen=True)
 class Branch:
     """A mixer of a layer: the prefix of its tensors and the factor of its output in the layer's sum."""
     prefix: str
-    spec: "AttentionSpec | LatentAttentionSpec | MlstmSpec | LinearRecurrenceSpec"
+    spec: "AttentionSpec | LatentAttentionSpec | MlstmSpec | LinearRecurrenceSpec | MinGruSpec | SelectiveScanSpec"
     scale: float
 
 
@@ -87,10 +94,12 @@ class AttentionSpec(MixerSpec):
     scale: float
     vdim: int | None = None     # None: the values are the un-normalised keys (cache rows that are key and value)
     window: int = 0             # positions a query sees, its own included; 0 = all
+    chunk: int = 0              # a query sees its own chunk of that many positions only, counted from position 0
     keep_first: int = 0         # first positions that stay visible
     slope_exponent: float | None = None    # geometric slopes of a linear distance bias
     norm_weights: bool = False  # weights of the query and key norms
     gated: bool = False         # one sigmoid gate per head on the output
+    element_gate: bool = False  # one sigmoid gate per output element instead
     softcap: float = 0.0        # scores become softcap * tanh(score / softcap), with separate values; 0 = as they are
     temp_coef: float = 0.0      # queries are multiplied by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)
     temp_every: float = 1.0
@@ -98,7 +107,28 @@ class AttentionSpec(MixerSpec):
     rotary: RotarySpec | None = None
     sink: bool = False          # a learned term per head in the softmax denominator, without a key and a value
     kv_from: int | None = None  # the layer whose cached keys and values are used; None: this layer has its own
+    biases: bool = False        # projections with biases
+    difference: float | None = None    # two softmax maps per head: o = a1 - lambda a2 over its root mean square, times 1 - difference,
+    #                             with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + difference
     kind = "attention"
+
+    @property
+    def maps(self) -> int:
+        return 1 if self.difference is None else 2
+
+    @property
+    def row_dim(self) -> int:
+        """Elements a cache row must hold: the keys of all maps, or the value."""
+        return max(self.maps * self.dim, self.value_dim)
+
+    @property
+    def visible(self) -> int:
+        """Most cached tokens a query sees (0: no bound)."""
+        return self.window + self.keep_first if self.window > 0 else self.chunk
+
+    @property
+    def out_bias(self) -> bool:
+        return self.biases
 
     @property
     def value_dim(self) -> int:
@@ -114,17 +144,23 @@ class AttentionSpec(MixerSpec):
 
     @property
     def sections(self) -> list[tuple[str, int]]:
-        s = [("q", self.heads * self.dim)]
+        s = [("q", self.heads * self.maps * self.dim)]
         if self.kv_from is None:
-            s.append(("k", self.kv_heads * self.dim))
+            s.append(("k", self.kv_heads * self.maps * self.dim))
             if self.vdim is not None:
                 s.append(("v", self.kv_heads * self.vdim))
-        return s + ([("g", self.heads)] if self.gated else [])
+        return s + ([("g", self.out_width if self.element_gate else self.heads)] if self.gated or self.element_gate else [])
 
     @property
     def vectors(self) -> dict[str, tuple[int, ...]]:
         v: dict[str, tuple[int, ...]] = {"q.norm": (self.dim,), "k.norm": (self.dim,)} if self.norm_weights else {}
-        return {**v, "sink": (self.heads,)} if self.sink else v
+        if self.sink:
+            v["sink"] = (self.heads,)
+        if self.biases:
+            v.update({n + ".b": (rows,) for n, rows in self.sections if n != "g"})
+        if self.difference is not None:
+            v.update({n: (self.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        return v
 
 
 @dataclass(frozen=True)
@@ -229,6 +265,56 @@ class LinearRecurrenceSpec(MixerSpec):
 
 
 @dataclass(frozen=True)
+class MinGruSpec(MixerSpec):
+    """An element-wise gated recurrence whose gates read the current token only (minGRU), with a silu gate on the output."""
+    width: int
+    kind = "mingru"
+
+    @property
+    def out_width(self) -> int:
+        return self.width
+
+    @property
+    def sections(self) -> list[tuple[str, int]]:
+        return [("z", self.width), ("x", self.width), ("g", self.width)]
+
+    @property
+    def vectors(self) -> dict[str, tuple[int, ...]]:
+        return {"z.b": (self.width,), "x.b": (self.width,)}
+
+
+@dataclass(frozen=True)
+class SelectiveScanSpec(MixerSpec):
+    """A state-space recurrence with ``states`` decays per channel, whose step sizes (through a product of rank ``rank``), inputs and
+    outputs are read from the convolved channels (Mamba)."""
+    channels: int
+    states: int
+    rank: int
+    conv: int
+    kind = "selective"
+
+    @property
+    def out_width(self) -> int:
+        return self.channels
+
+    @property
+    def sections(self) -> list[tuple[str, int]]:
+        return [("in", self.channels), ("in", self.channels)]      # the channels, then their gates
+
+    @property
+    def vectors(self) -> dict[str, tuple[int, ...]]:
+        c = self.channels
+        return {"conv": (c, self.conv), "conv.b": (c,), "dt.b": (c,), "A_log": (c, self.states), "D": (c,)}
+
+    @property
+    def inner(self) -> dict[str, tuple[int, int]]:
+        return {"x": (self.rank + 2 * self.states, self.channels), "dt": (self.channels, self.rank)}
+
+
+RECURRENT = ("mlstm", "recurrence", "mingru", "selective")
+
+
+@dataclass(frozen=True)
 class ParallelSpec(MixerSpec):
     """Mixers side by side that read the same input; the scaled sum of their outputs is the layer's."""
     parts: tuple[Branch, ...]
@@ -241,12 +327,19 @@ class ParallelSpec(MixerSpec):
 
 @dataclass(frozen=True)
 class GatedMlpSpec:
-    """``W_down [g * sigmoid(alpha g) * (u + offset)]`` with ``g = min(W_gate h, limit)``, ``u = clamp(W_up h, -limit, limit)``."""
+    """``W_down [g * sigmoid(alpha (g + cubic g^3)) * (u + offset)]`` with ``g = min(W_gate h, limit)``, ``u = clamp(W_up h, -limit,
+    limit)``."""
     ff: int
     limit: float
     alpha: float
     offset: float
+    cubic: float = 0.0
     matrices = ("gate", "up")
+
+
+def gelu_mlp(ff: int) -> GatedMlpSpec:
+    """A gate through the tanh form of gelu: (1 + tanh(y)) / 2 = sigmoid(2 y)."""
+    return GatedMlpSpec(ff, math.inf, alpha=2.0 * math.sqrt(2.0 / math.pi), offset=0.0, cubic=0.044715)
 
 
 @dataclass(frozen=True)
@@ -258,31 +351,53 @@ class SquaredReluMlpSpec:
 
 @dataclass(frozen=True)
 class RouterSpec:
-    """Chooses ``top`` of ``experts`` per token.  Scores are sigmoids; what is compared is score + correction.  Experts form
-    ``groups`` equal groups of neighbours, of which only the ``keep`` with the largest sums of their two best are eligible.  The
-    weights are the chosen scores over (their sum + ``den_eps``), times ``scale``."""
+    """Chooses ``top`` of ``experts`` per token.  Scores are sigmoids, or with ``softmax`` that of all logits; what is compared is the
+    score, plus a learned correction where the router has one.  Experts form ``groups`` equal groups of neighbours, of which only the
+    ``keep`` with the largest sums of their two best are eligible.  The weights are the chosen scores, over (their sum + ``den_eps``)
+    if ``normalized``, times ``scale``."""
     experts: int
     top: int
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
     den_eps: float = 1e-20
+    softmax: bool = False
+    normalized: bool = True
+    corrected: bool = True
 
 
 @dataclass(frozen=True)
 class ExpertsSpec:
-    """A weighted sum of the chosen experts; each is a gated block of ``ff`` hidden units as in :class:`GatedMlpSpec`."""
+    """A weighted sum of the chosen experts; each is a gated block of ``ff`` hidden units as in :class:`GatedMlpSpec`.  ``shared``: one more
+    block that every token runs, times the sigmoid of one number per token ("shared.sg")."""
     router: RouterSpec
     ff: int
     limit: float = math.inf
     alpha: float = 1.0
     offset: float = 0.0
+    shared: GatedMlpSpec | None = None
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
     mlp: GatedMlpSpec | SquaredReluMlpSpec | ExpertsSpec | None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start`` .. ``stop`` - 1 run ``times`` times in a row with the same weights and a cache or state per pass.  Ahead of pass t
+    x grows by row t of "loop.step" and, from the second pass on, by the embedding."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class Run:
+    """One run of a layer; ``begins``: the pass it is the first run of (None: it begins none)."""
+    layer: int
+    begins: int | None = None
 
 
 @dataclass(frozen=True)
@@ -298,6 +413,11 @@ class LayeredConfig:
     side_by_side: bool = False  # mixer and feed-forward read the same norm ("norm1"); x grows by residual_mult times their sum
     residual_mult: float = 1.0
     layer_norm: bool = False    # norms take the mean off first
+    norm_groups: int | None = None     # norms divide that many equal parts by their own root mean square (None: one part)
+    input_taps: int = 0         # what a sublayer reads, h, becomes h + conv(h), a convolution over that many tokens ("canon1", "canon2"); 0: no
+    loop: LoopSpec | None = None
+    own_head: bool = False      # the head is a tensor of its own ("head")
+    logit_cap: float = 0.0      # logits become cap * tanh(logits / cap); 0: as they are
 
     @property
     def layers(self) -> int:
@@ -306,6 +426,25 @@ class LayeredConfig:
     @property
     def hidden(self) -> int:
         return self.width
+
+    @property
+    def runs(self) -> tuple[Run, ...]:
+        """The layers in the order they run; caches and states belong to runs."""
+        lo = self.loop
+        if lo is None:
+            return tuple(Run(i) for i in range(self.layers))
+        body = [Run(i, t if i == lo.start else None) for t in range(lo.times) for i in range(lo.start, lo.stop)]
+        return tuple([Run(i) for i in range(lo.start)] + body + [Run(i) for i in range(lo.stop, self.layers)])
+
+    @property
+    def row_steps(self) -> bool:
+        """Whether what happens between sublayers takes the general row kernel."""
+        return self.norm_groups is not None or self.input_taps > 0 or self.loop is not None
+
+    @property
+    def has_state(self) -> bool:
+        """Whether a sequence has state besides the pages of attention layers."""
+        return bool(self.recurrent_layers) or self.input_taps > 0
 
     def branches(self, i: int, *kinds: str) -> list[Branch]:
         """The mixers of layer ``i`` of the given kinds."""
@@ -317,21 +456,21 @@ class LayeredConfig:
 
     @property
     def recurrent_layers(self) -> list[int]:
-        return [i for i in range(self.layers) if self.branches(i, "mlstm", "recurrence")]
+        return [i for i in range(self.layers) if self.branches(i, *RECURRENT)]
 
     def attention(self, i: int) -> AttentionSpec | LatentAttentionSpec:
         return self.branches(i, "attention", "latent")[0].spec
 
-    def recurrence(self, i: int) -> MlstmSpec | LinearRecurrenceSpec:
-        return self.branches(i, "mlstm", "recurrence")[0].spec
+    def recurrence(self, i: int) -> "MlstmSpec | LinearRecurrenceSpec | MinGruSpec | SelectiveScanSpec":
+        return self.branches(i, *RECURRENT)[0].spec
 
     @property
     def max_visible(self) -> int | None:
         """Most cached tokens a query of any attention layer can see (None: no bound, or no attention layer)."""
         seen = [self.attention(i) for i in self.attention_layers]
-        if not seen or any(isinstance(m, LatentAttentionSpec) or m.window <= 0 for m in seen):
+        if not seen or any(isinstance(m, LatentAttentionSpec) or m.visible <= 0 for m in seen):
             return None
-        return max(m.window + m.keep_first for m in seen)
+        return max(m.visible for m in seen)
 
     @property
     def expert_layers(self) -> list[int]:
@@ -353,7 +492,13 @@ class LayeredConfig:
         """Name and shape of every tensor of the checkpoint."""
         w = self.width
         s: dict[str, tuple[int, ...]] = {"embed": (self.vocab, w), "final.norm": (w,)}
+        if self.own_head:
+            s["head"] = (self.vocab, w)
+        if self.loop is not None:
+            s["loop.step"] = (self.loop.times, w)
         for i, layer in enumerate(self.layer_specs):
+            if self.input_taps:
+                s.update({f"l{i}.canon{n + 1}": (w, self.input_taps) for n in range(len(self.norm_names(i)))})
             s.update({n: (w,) for pair in self.norm_names(i) for n in pair if n is not None})
             for b in layer.mixer.branches:
                 x = f"l{i}.mix.{b.prefix}"
@@ -361,9 +506,16 @@ class LayeredConfig:
                     s[x + name] = (s.get(x + name, (0, w))[0] + rows, w)
                 s.update({x + n: shape for n, shape in {**b.spec.vectors, **b.spec.inner}.items()})
                 s[x + "o"] = (w, b.spec.out_width)
+                if b.spec.out_bias:
+                    s[x + "o.b"] = (w,)
             if isinstance(layer.mlp, ExpertsSpec):
                 f, n = layer.mlp.ff, layer.mlp.router.experts
-                s.update({f"l{i}.mlp.router": (n, w), f"l{i}.mlp.correction": (n,)})
+                s[f"l{i}.mlp.router"] = (n, w)
+                if layer.mlp.router.corrected:
+                    s[f"l{i}.mlp.correction"] = (n,)
+                if layer.mlp.shared is not None:
+                    sf, sp = layer.mlp.shared.ff, f"l{i}.mlp.shared."
+                    s.update({sp + "gate": (sf, w), sp + "up": (sf, w), sp + "down": (w, sf), sp + "sg": (1, w)})
                 for e in range(n):
                     s.update({f"l{i}.mlp.e{e}.gate": (f, w), f"l{i}.mlp.e{e}.up": (f, w), f"l{i}.mlp.e{e}.down": (w, f)})
             elif layer.mlp is not None:
@@ -438,8 +590,8 @@ def _state_dim(dim: int, where: str) -> int:
     return dim
 
 
-def _layers(raw: dict, mixers: dict, mlp, mlp_kind: str = "dense") -> tuple[LayerSpec, ...]:
-    """The layer list: ``mixers`` reads a mixer by its type, ``mlp`` a feed-forward block of the kind the design has."""
+def _layers(raw: dict, mixers: dict, mlps: dict) -> tuple[LayerSpec, ...]:
+    """The layer list: ``mixers`` reads a mixer by its type, ``mlps`` a feed-forward block by its kind."""
     layers = []
     for i, entry in enumerate(_get(raw, "layers", "the model")):
         where = f"layers[{i}]"
@@ -447,9 +599,9 @@ def _layers(raw: dict, mixers: dict, mlp, mlp_kind: str = "dense") -> tuple[Laye
         if kind not in mixers:
             raise LayeredConfigError(f"config.json: {where}: unknown mixer type {kind!r}")
         ff = _get(entry, "mlp", where)
-        if ff is not None and _get(ff, "kind", where + ".mlp") != mlp_kind:
+        if ff is not None and _get(ff, "kind", where + ".mlp") not in mlps:
             raise LayeredConfigError(f"config.json: {where}.mlp: unknown kind {ff['kind']!r}")
-        layers.append(LayerSpec(mixers[kind](_get(entry, "mixer", where), where + ".mixer"), None if ff is None else mlp(ff, where + ".mlp")))
+        layers.append(LayerSpec(mixers[kind](_get(entry, "mixer", where), where + ".mixer"), None if ff is None else mlps[ff["kind"]](ff, where + ".mlp")))
     if not layers:
         raise LayeredConfigError("config.json: the model has no layers")
     return tuple(layers)
@@ -480,7 +632,7 @@ def keripel_config(raw: dict, name: str = "") -> LayeredConfig:
     """The Keripel design: mLSTM and windowed-attention mixers in the order the file lists, output norms, gated feed-forward
     blocks where a layer has one, and a head tied to the embedding."""
     mlp = lambda m, where: GatedMlpSpec(_size(m, "ff", where), _number(m, "limit", where), alpha=1.702, offset=1.0)
-    return _model(raw, "Keripel", name, _layers(raw, {"attention": _windowed_attention, "mlstm": _mlstm}, mlp))
+    return _model(raw, "Keripel", name, _layers(raw, {"attention": _windowed_attention, "mlstm": _mlstm}, {"dense": mlp}))
 
 
 # ---- Kekevik ----------------------------------------------------------------------------------------------------------------------
@@ -527,7 +679,7 @@ def kekevik_config(raw: dict, name: str = "") -> LayeredConfig:
     """The Kekevik design: retention, lightning attention, and capped attention beside a state-space mixer, in the order the
     file lists; norms before and after each sublayer, squared-relu feed-forward blocks, a scaled embedding tied to the head."""
     layers = _layers(raw, {"retention": _retention, "lightning": _lightning, "parallel": _side_by_side},
-                     lambda m, where: SquaredReluMlpSpec(_size(m, "ff", where)))
+                     {"dense": lambda m, where: SquaredReluMlpSpec(_size(m, "ff", where))})
     scale = _number(_get(raw, "embedding", "the model"), "scale", "embedding")
     return _model(raw, "Kekevik", name, layers, embed_scale=scale, pre_norm=True)
 
@@ -553,14 +705,20 @@ def _latent_attention(m: dict, where: str) -> LatentAttentionSpec:
     return LatentAttentionSpec(heads, dim, rot_dim, vdim, rank, _number(m, "scale", where), rotary)
 
 
+def _choice(r: dict, where: str) -> tuple[int, int]:
+    """Experts, and how many of them a token uses."""
+    experts, top = _size(r, "experts", where), _size(r, "top", where)
+    if experts > MAX_EXPERTS or top > min(MAX_CHOSEN, experts):
+        raise LayeredConfigError(f"config.json: {where}: {top} of {experts} experts (at most {MAX_CHOSEN} of {MAX_EXPERTS})")
+    return experts, top
+
+
 def _experts(m: dict, where: str) -> ExpertsSpec:
     r, ff = _get(m, "router", where), _size(_get(m, "expert", where), "ff", where + ".expert")
+    experts, top = _choice(r, where + ".router")
     where += ".router"
-    experts, top = _size(r, "experts", where), _size(r, "top", where)
     g = r.get("groups")
     count, keep = (1, 1) if g is None else (_size(g, "count", where + ".groups"), _size(g, "keep", where + ".groups"))
-    if experts > MAX_EXPERTS or top > MAX_CHOSEN:
-        raise LayeredConfigError(f"config.json: {where}: {top} of {experts} experts (at most {MAX_CHOSEN} of {MAX_EXPERTS})")
     if experts % count or keep > count or top > keep * (experts // count):
         raise LayeredConfigError(f"config.json: {where}: {top} of {experts} experts in {keep} of {count} groups")
     return ExpertsSpec(RouterSpec(experts, top, count, keep, _number(r, "scale", where)), ff)
@@ -569,7 +727,7 @@ def _experts(m: dict, where: str) -> ExpertsSpec:
 def kutepel_config(raw: dict, name: str = "") -> LayeredConfig:
     """The Kutepel design: latent attention and rotary attention with sinks (some layers on an earlier one's keys and values) in the
     order the file lists, side by side with a mixture of experts behind one layer norm, and a head tied to the embedding."""
-    layers = _layers(raw, {"attention": _rotary_attention, "latent_attention": _latent_attention}, _experts, "moe")
+    layers = _layers(raw, {"attention": _rotary_attention, "latent_attention": _latent_attention}, {"moe": _experts})
     for i, layer in enumerate(layers):
         j = getattr(layer.mixer, "kv_from", None)
         if j is None:
@@ -580,3 +738,67 @@ def kutepel_config(raw: dict, name: str = "") -> LayeredConfig:
         if (source.kv_heads, source.dim, source.vdim) != (layer.mixer.kv_heads, layer.mixer.dim, layer.mixer.vdim):
             raise LayeredConfigError(f"config.json: layers[{i}].mixer.kv_from: layer {j} has other key/value heads")
     return _model(raw, "Kutepel", name, layers, side_by_side=True, residual_mult=_number(raw, "residual_mult", "the model"), layer_norm=True)
+
+
+# ---- Naforax ----------------------------------------------------------------------------------------------------------------------
+SWISH_ALPHA = 1.702         # of the clamped units
+
+
+def _differential_attention(m: dict, where: str) -> AttentionSpec:
+    heads, kv, dim, vdim = _attention_sizes(m, where)
+    if 2 * dim > MAX_HEAD_DIM:
+        raise LayeredConfigError(f"config.json: {where}: two maps of {dim} dimensions exceed {MAX_HEAD_DIM}")
+    return AttentionSpec(heads, kv, dim, _number(m, "scale", where), vdim=vdim, chunk=_size(_get(m, "mask", where), "size", where + ".mask"), norm_weights=True,
+                         element_gate=True, rotary=_rotary(m, dim, where, interleaved=True), biases=True, difference=_number(m, "diff", where))
+
+
+def _taps(d: dict, key: str, where: str) -> int:
+    taps = _size(d, key, where)
+    if taps > MAX_TAPS:
+        raise LayeredConfigError(f"config.json: {where}.{key}: a convolution over {taps} tokens exceeds {MAX_TAPS}")
+    return taps
+
+
+def _mingru(m: dict, where: str) -> MinGruSpec:
+    return MinGruSpec(_size(m, "width", where))
+
+
+def _mamba1(m: dict, where: str) -> SelectiveScanSpec:
+    states = _size(m, "state", where)
+    if states > MAX_SCAN_STATES:
+        raise LayeredConfigError(f"config.json: {where}: {states} states per channel exceed {MAX_SCAN_STATES}")
+    return SelectiveScanSpec(_size(m, "inner", where), states, _size(m, "dt_rank", where), _taps(m, "conv", where))
+
+
+def _clamped_unit(m: dict, where: str) -> GatedMlpSpec:
+    return GatedMlpSpec(_size(m, "ff", where), _positive(m, "limit", where), alpha=SWISH_ALPHA, offset=1.0)
+
+
+def _softmax_experts(m: dict, where: str) -> ExpertsSpec:
+    experts, top = _choice(_get(m, "router", where), where + ".router")
+    e, shared = _clamped_unit(_get(m, "expert", where), where + ".expert"), m.get("shared")
+    return ExpertsSpec(RouterSpec(experts, top, softmax=True, normalized=False, corrected=False), e.ff, e.limit, e.alpha, e.offset,
+                       None if shared is None else _clamped_unit(shared, where + ".shared"))
+
+
+def _loop(raw: dict, layers: int) -> LoopSpec | None:
+    if raw.get("loop") is None:
+        return None
+    lo = LoopSpec(*(_size(raw["loop"], k, "loop", least) for k, least in (("start", 0), ("stop", 1), ("times", 1))))
+    if not lo.start < lo.stop <= layers:
+        raise LayeredConfigError(f"config.json: loop: layers {lo.start} .. {lo.stop - 1} of {layers}")
+    return lo
+
+
+def naforax_config(raw: dict, name: str = "") -> LayeredConfig:
+    """The Naforax design: differential attention in chunks, minGRU and selective-scan mixers in the order the file lists, a loop over some
+    of the layers, grouped norms before and after each sublayer, a convolution ahead of each, dense blocks and experts with a shared
+    one, and a capped head of its own."""
+    layers = _layers(raw, {"attention": _differential_attention, "mingru": _mingru, "mamba1": _mamba1},
+                     {"dense": lambda m, where: gelu_mlp(_size(m, "ff", where)), "moe": _softmax_experts})
+    groups, width = _size(_get(raw, "norm", "the model"), "groups", "norm"), _size(raw, "width", "the model")
+    if width % groups or groups << max(0, -(-(width // groups) // 16) - 1).bit_length() > 1024:     # a power of two of threads per part, 16 columns each
+        raise LayeredConfigError(f"config.json: norm.groups: {groups} equal parts of {width}")
+    return _model(raw, "Naforax", name, layers, pre_norm=True, residual_mult=_number(raw, "residual_mult", "the model"), norm_groups=groups,
+                  input_taps=_taps(_get(raw, "canon", "the model"), "taps", "canon"), loop=_loop(raw, len(layers)), own_head=True,
+                  logit_cap=_positive(raw, "logit_softcap", "the model"))

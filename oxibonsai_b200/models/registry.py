@@ -19,7 +19,7 @@ from typing import Callable, Iterator
 
 from ..core import gguf as G
 from ..core.gguf import GgufFile, Qwen3Config
-from .layered_config import LayeredConfig, LayeredConfigError, kekevik_config, keripel_config, kutepel_config
+from .layered_config import LayeredConfig, LayeredConfigError, kekevik_config, keripel_config, kutepel_config, naforax_config
 
 
 class ModelVariant(Enum):
@@ -237,7 +237,8 @@ def memory_budget_check(f: GgufFile, available_bytes: int, context: int = 4096, 
 
 # ---- designs described by a config.json ------------------------------------------------------------------------------------------
 # "architecture" of a model directory's config.json -> reader of that design's configuration
-ARCHITECTURES: dict[str, Callable[[dict, str], LayeredConfig]] = {"Keripel": keripel_config, "Kekevik": kekevik_config, "Kutepel": kutepel_config}
+ARCHITECTURES: dict[str, Callable[[dict, str], LayeredConfig]] = {"Keripel": keripel_config, "Kekevik": kekevik_config, "Kutepel": kutepel_config,
+                                                                      "Naforax": naforax_config}
 
 
 def is_model_dir(path) -> bool:

@@ -17,9 +17,9 @@ _SIG = {
     "bonsai_lay_side_by_side": [_vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _f, _i, _i, _vp, _i, _i, _vp, _f, _i, _vp],
     "bonsai_lay_norm_rows": [_vp, _vp, _vp, _f, _i, _i, _i, _vp, _i, _i, _vp],
     "bonsai_lay_gated_norm": [_vp, _i, _vp, _i, _vp, _f, _i, _i, _i, _i, _i, _f, _vp, _i, _i, _vp],
-    "bonsai_lay_linear_few": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _vp],
-    "bonsai_lay_linear_f32": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
-    "bonsai_dense_gemm_bf16": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _vp, _vp, C.c_size_t, _i, _vp],
+    "bonsai_lay_linear_few": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _f, _vp],
+    "bonsai_lay_linear_f32": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _f, _vp],
+    "bonsai_dense_gemm_bf16": [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _f, _f, _f, _f, _vp, _vp, C.c_size_t, _i, _vp],
     "bonsai_bitgemm_prefill_ws_bytes": [],
     "bonsai_lay_attn_row": [_i],
     "bonsai_lay_attn_append": [_vp, _vp, _vp, _i, _i, _i, _vp],
@@ -39,9 +39,9 @@ _SIG = {
     "bonsai_lay_latent_f32": [_vp, _vp, _vp, _i, _vp],
     "bonsai_lay_route_small": [_i],
     "bonsai_lay_route": [_vp, _vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp],
-    "bonsai_lay_experts_few": [_vp, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
-    "bonsai_lay_experts_f32": [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _vp],
-    "bonsai_grouped_gemm_bf16": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _f, _f, _f, _i, _vp, _i, _vp],
+    "bonsai_lay_experts_few": [_vp, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _f, _f, _f, _f, _vp],
+    "bonsai_lay_experts_f32": [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _f, _f, _f, _f, _vp],
+    "bonsai_grouped_gemm_bf16": [_vp, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _f, _f, _f, _f, _i, _vp, _i, _vp],
     "bonsai_lay_mlstm_dim": [_i],
     "bonsai_lay_mlstm_vdim": [_i],
     "bonsai_lay_mlstm_chunk_dim": [],
@@ -58,6 +58,18 @@ _SIG = {
     "bonsai_lay_rec_ring": [_vp, _vp, _vp, _vp, _i, _vp],
     "bonsai_lay_rec_step": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "bonsai_lay_rec_chunk": [_vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _vp],
+    "bonsai_lay_row_step": [_vp, _vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _vp, _i, _vp],
+    "bonsai_lay_conv": [_vp, _vp, _vp, _i, _vp, _vp, _i, _vp],
+    "bonsai_lay_conv_rows": [],
+    "bonsai_lay_conv_taps": [],
+    "bonsai_lay_gru_step": [_vp, _vp, _vp, _i, _i, _vp],
+    "bonsai_lay_gru_scan": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "bonsai_lay_gru_tokens": [],
+    "bonsai_lay_scan_states": [_i],
+    "bonsai_lay_scan_channels": [_i],
+    "bonsai_lay_scan_step": [_vp, _vp, _vp, _i, _i, _vp],
+    "bonsai_lay_scan": [_vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp],
+    "bonsai_lay_narrow": [_vp, _i, _i, _i, _i, _vp, _i, _vp],
     "bonsai_sample": K._SIG["bonsai_sample"],
 }
 _lib = None
@@ -121,35 +133,48 @@ class GemmScratch:
 
 @dataclass(frozen=True)
 class Glu:
-    """Clamped gated unit over interleaved gate / up rows."""
+    """Clamped gated unit over interleaved gate / up rows: g * sigmoid(alpha (g + cubic g^3)) * (u + offset)."""
     limit: float
     alpha: float
     offset: float
+    cubic: float = 0.0
+
+    @property
+    def args(self) -> tuple[float, float, float, float]:
+        return self.limit, self.alpha, self.offset, self.cubic
+
+
+@dataclass(frozen=True)
+class SoftCap:
+    """f32 outputs become cap * tanh(output / cap)."""
+    cap: float
 
 
 SQUARED_RELU = "squared_relu"
 _NO_GLU = Glu(0.0, 0.0, 0.0)
 
 
-def linear(w: DenseWeight, x: torch.Tensor, T: int, out: torch.Tensor, scratch: GemmScratch, act: Glu | str | None = None) -> None:
+def linear(w: DenseWeight, x: torch.Tensor, T: int, out: torch.Tensor, scratch: GemmScratch, act: Glu | SoftCap | str | None = None) -> None:
     """out[:T] = act(x[:T] W^T).  bf16 ``x`` (row stride >= kp, finite in the padding): tensor cores, f32 or bf16 ``out`` (bf16 with
-    ``act``); f32 ``x``: 32-bit throughout.  ``act``: none, :class:`Glu`, or ``SQUARED_RELU``."""
+    a :class:`Glu` or ``SQUARED_RELU``, f32 with a :class:`SoftCap`); f32 ``x``: 32-bit throughout."""
     l, s = lib(), K.stream()
-    glu = act if isinstance(act, Glu) else _NO_GLU
-    epi = (3 if out.dtype == torch.bfloat16 else 0) if act is None else (1 if isinstance(act, Glu) else 2)
-    if x.dtype == torch.float32:
-        K.check(l.bonsai_lay_linear_f32(w.data.data_ptr(), w.n, w.k, w.kp, x.data_ptr(), x.stride(0), T, out.data_ptr(), out.stride(0),
-                                        epi, glu.limit, glu.alpha, glu.offset, s), "linear_f32")
-        return
-    assert x.dtype == torch.bfloat16 and (act is None or out.dtype == torch.bfloat16)
-    f32, b16 = (out.data_ptr(), None) if epi == 0 else (None, out.data_ptr())
-    if T <= FEW_ROWS:
-        K.check(l.bonsai_lay_linear_few(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), epi,
-                                        glu.limit, glu.alpha, glu.offset, s), "linear_few")
+    if act is None:
+        epi, glu = (3 if out.dtype == torch.bfloat16 else 0), _NO_GLU
+    elif isinstance(act, SoftCap):
+        epi, glu = 4, Glu(act.cap, 0.0, 0.0)
     else:
-        K.check(l.bonsai_dense_gemm_bf16(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0),
-                                         (0, 4, 5, 6)[epi], glu.limit, glu.alpha, glu.offset, scratch.status.data_ptr(), scratch.ws.data_ptr(),
-                                         scratch.ws.numel(), scratch.sms, s), "dense_gemm_bf16")
+        epi, glu = (1, act) if isinstance(act, Glu) else (2, _NO_GLU)
+    if x.dtype == torch.float32:
+        K.check(l.bonsai_lay_linear_f32(w.data.data_ptr(), w.n, w.k, w.kp, x.data_ptr(), x.stride(0), T, out.data_ptr(), out.stride(0), epi, *glu.args, s),
+                "linear_f32")
+        return
+    assert x.dtype == torch.bfloat16 and (out.dtype == torch.float32 if epi in (0, 4) else out.dtype == torch.bfloat16)
+    f32, b16 = (out.data_ptr(), None) if epi in (0, 4) else (None, out.data_ptr())
+    if T <= FEW_ROWS:
+        K.check(l.bonsai_lay_linear_few(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), epi, *glu.args, s), "linear_few")
+    else:
+        K.check(l.bonsai_dense_gemm_bf16(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), (0, 4, 5, 6, 7)[epi], *glu.args,
+                                         scratch.status.data_ptr(), scratch.ws.data_ptr(), scratch.ws.numel(), scratch.sms, s), "dense_gemm_bf16")
 
 
 def _row_out(t: torch.Tensor | None) -> tuple[int | None, int, int]:
@@ -178,6 +203,58 @@ def side_by_side(x: torch.Tensor, y: torch.Tensor, experts: "Routing | None", mu
                                           K.stream()), "side_by_side")
 
 
+class RowStep:
+    """What happens between two sublayers, in one launch:
+    ``x += mult * norm(sigmoid(gate) (y + bias) + expert rows) * w``, then ``x += scale * table[token] + step``, then ``n = norm(x) * next``
+    and ``h = n + conv(n)``.  Every part may be left out; ``fresh``: x starts here.  ``rows``: positions, slots and tokens of the rows;
+    ``conv``: weights [taps, width] (the current token's first) and the ring of earlier inputs.  Norms have ``groups`` parts."""
+
+    def __init__(self, x: torch.Tensor, h: torch.Tensor | None, rows, state_table: torch.Tensor, *, eps: float, groups: int, mult: float = 1.0,
+                 y: torch.Tensor | None = None, bias: torch.Tensor | None = None, gate: torch.Tensor | None = None, w: torch.Tensor | None = None,
+                 table: torch.Tensor | None = None, scale: float = 1.0, step: torch.Tensor | None = None, next_norm: torch.Tensor | None = None,
+                 conv: tuple[torch.Tensor, torch.Tensor] | None = None, n32: torch.Tensor | None = None, fresh: bool = False):
+        ld = lambda t: 0 if t is None else t.stride(0)
+        weight, ring = conv if conv is not None else (None, None)
+        h_f32 = h is not None and h.dtype == torch.float32
+        self.call = MixerCall([x, y, bias, gate, w, table, rows.tokens, step, next_norm, n32, h, weight, ring, rows.positions, rows.slots, state_table],
+                              [ld(y), ld(gate), x.shape[1], groups, ld(table), ld(n32), ld(h), int(h_f32), 0 if weight is None else weight.shape[0], int(fresh)],
+                              [eps, mult, scale])
+        self.conv = None
+        if conv is not None and n32 is not None:
+            self.conv = Conv(n32, 0, x.shape[1], weight, None, ring, rows, state_table, h, add=True)
+
+    def __call__(self, T: int, st, experts: "Routing | None" = None, norm_of: int | None = None) -> None:
+        """``st``: the step's rows (single tokens and portions); ``norm_of``: device address of the rows whose norm alone is asked for."""
+        e = (None, 0, 0, None, 0, None, 0) if experts is None else experts.outputs
+        here = self.conv is None or not st.portions
+        K.check(lib().bonsai_lay_row_step(*self.call.args, T, *e, norm_of, int(here), K.stream()), "row_step")
+        if not here:
+            self.conv(st)
+
+
+class Conv:
+    """Causal convolution over tokens, a row of ``channels`` columns per token: out = [x +] [silu] (conv(x) + bias)."""
+
+    def __init__(self, x: torch.Tensor, col: int, channels: int, weight: torch.Tensor, bias: torch.Tensor | None, ring: torch.Tensor, rows,
+                 state_table: torch.Tensor, out: torch.Tensor, add: bool = False, silu: bool = False):
+        self.call = MixerCall([x, weight, bias, ring, rows.positions, rows.slots, state_table, out],
+                              [x.stride(0), col, channels, weight.shape[0], out.stride(0), int(out.dtype == torch.float32), int(add), int(silu)], [])
+
+    def __call__(self, st) -> None:
+        tiles, n = st.tiles[lib().bonsai_lay_conv_rows()] if st.portions else (None, 0)
+        K.check(lib().bonsai_lay_conv(*self.call.args, st.singles, st.entries if n else None, tiles, n, K.stream()), "conv")
+
+
+def conv_weight(w: torch.Tensor) -> torch.Tensor:
+    """[channels, taps] with the current token's tap last -> [taps, channels] with it first."""
+    return w.flip(1).t().contiguous()
+
+
+def narrow(x: torch.Tensor, col: int, n: int, T: int, out: torch.Tensor) -> None:
+    """f32 columns ``col`` .. ``col + n - 1`` of the first T rows as bf16."""
+    K.check(lib().bonsai_lay_narrow(x.data_ptr(), x.stride(0), col, n, T, out.data_ptr(), out.stride(0), K.stream()), "narrow")
+
+
 def norm_rows(x: torch.Tensor, rows: int | None, count: int, w: torch.Tensor, eps: float, out: torch.Tensor, center: bool = False) -> None:
     """out[i] = rmsnorm(x[rows[i]]) * w (``rows``: device address of int32 indices, None = 0 .. count - 1); ``center``: a layer norm."""
     K.check(lib().bonsai_lay_norm_rows(x.data_ptr(), rows, w.data_ptr(), eps, int(center), count, x.shape[1], out.data_ptr(), out.stride(0),
@@ -195,7 +272,7 @@ def gated_norm(o: torch.Tensor, row0: int, gate: torch.Tensor, gate_col: int, w:
 
 
 class MixerCall:
-    """The argument blocks (pointers, sizes, constants) of one mixer's launches; the tensors must outlive it."""
+    """The argument blocks (pointers, sizes, constants) of the launches of one mixer or step; the tensors must outlive it."""
 
     def __init__(self, ptrs: list[torch.Tensor | None], ints: list[int], floats: list[float]):
         self._keep = ptrs
@@ -233,12 +310,12 @@ class ExpertScratch:
 class Routing:
     """One expert layer's calls: choice, sorting, the experts' projections.  ``logits``: the projections the router's are part of."""
 
-    def __init__(self, spec, up: DenseWeight, down: DenseWeight, correction: torch.Tensor, logits: torch.Tensor, column: int, scratch: ExpertScratch):
+    def __init__(self, spec, up: DenseWeight, down: DenseWeight, correction: torch.Tensor | None, logits: torch.Tensor, column: int, scratch: ExpertScratch):
         r = spec.router
         self.spec, self.up, self.down, self.s = spec, up, down, scratch
         self.glu = Glu(spec.limit, spec.alpha, spec.offset)
         self.call = MixerCall([logits, correction, scratch.counts, scratch.pair, scratch.pair_weight, scratch.lists, scratch.token, scratch.weight, scratch.at],
-                              [logits.stride(0), column, r.experts, r.top, r.groups, r.keep], [r.scale, r.den_eps])
+                              [logits.stride(0), column, r.experts, r.top, r.groups, r.keep, int(r.softmax), int(r.normalized)], [r.scale, r.den_eps])
         self.n_up, self.n_down = up.n // r.experts, down.n // r.experts
         self.out = scratch.out
 
@@ -270,23 +347,23 @@ class Routing:
         if s.exact:
             self.out = s.out
             K.check(l.bonsai_lay_experts_f32(up.data.data_ptr(), r.experts, self.n_up, up.k, up.kp, h.data_ptr(), h.stride(0), lists, token, weight, pairs, T,
-                                             hid.data_ptr(), hid.stride(0), 1, g.limit, g.alpha, g.offset, st), "experts_f32")
+                                             hid.data_ptr(), hid.stride(0), 1, *g.args, st), "experts_f32")
             K.check(l.bonsai_lay_experts_f32(down.data.data_ptr(), r.experts, self.n_down, down.k, down.kp, hid.data_ptr(), hid.stride(0), lists, None, None,
-                                             pairs, T, s.out.data_ptr(), s.out.stride(0), 0, 0.0, 0.0, 0.0, st), "experts_f32")
+                                             pairs, T, s.out.data_ptr(), s.out.stride(0), 0, *_NO_GLU.args, st), "experts_f32")
         elif not tile:
             self.out = s.out32
             slots, per = min(r.experts, pairs), min(T, 2 * pairs // r.experts + 8)
             K.check(l.bonsai_lay_experts_few(up.data.data_ptr(), r.experts, self.n_up, up.kp, h.data_ptr(), h.stride(0), lists, token, weight, pairs, slots, per,
-                                             hid.data_ptr(), hid.stride(0), 1, g.limit, g.alpha, g.offset, st), "experts_few")
+                                             hid.data_ptr(), hid.stride(0), 1, *g.args, st), "experts_few")
             K.check(l.bonsai_lay_experts_few(down.data.data_ptr(), r.experts, self.n_down, down.kp, hid.data_ptr(), hid.stride(0), lists, None, None, pairs,
-                                             slots, per, s.out32.data_ptr(), s.out32.stride(0), 0, 0.0, 0.0, 0.0, st), "experts_few")
+                                             slots, per, s.out32.data_ptr(), s.out32.stride(0), 0, *_NO_GLU.args, st), "experts_few")
         else:
             self.out = s.out
             wide = int(pairs > 96 * r.experts)
             K.check(l.bonsai_grouped_gemm_bf16(up.data.data_ptr(), r.experts, self.n_up, up.kp, xs.data_ptr(), xs.stride(0), pairs, lists, weight, hid.data_ptr(),
-                                               hid.stride(0), 4, g.limit, g.alpha, g.offset, wide, scratch.status.data_ptr(), scratch.sms, st), "grouped_gemm")
+                                               hid.stride(0), 4, *g.args, wide, scratch.status.data_ptr(), scratch.sms, st), "grouped_gemm")
             K.check(l.bonsai_grouped_gemm_bf16(down.data.data_ptr(), r.experts, self.n_down, down.kp, hid.data_ptr(), hid.stride(0), pairs, lists, None,
-                                               s.out.data_ptr(), s.out.stride(0), 6, 0.0, 0.0, 0.0, wide, scratch.status.data_ptr(), scratch.sms, st),
+                                               s.out.data_ptr(), s.out.stride(0), 6, *_NO_GLU.args, wide, scratch.status.data_ptr(), scratch.sms, st),
                     "grouped_gemm")
 
 

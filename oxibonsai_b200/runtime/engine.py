@@ -563,11 +563,11 @@ class LayeredEngine(InferenceEngine):
 
     @property
     def supports_prefix_cache(self) -> bool:
-        return not self.config.recurrent_layers            # cached pages do not bring the recurrent state back
+        return not self.config.has_state            # cached pages do not bring the recurrent state back
 
     def enable_prefix_cache(self, max_pages: int | None = None):
         if not self.supports_prefix_cache:
-            raise ValueError("a model with recurrent layers cannot resume from cached prompt pages")
+            raise ValueError("a model with recurrent layers or convolutions over tokens cannot resume from cached prompt pages")
         return super().enable_prefix_cache(max_pages)
 
     def enable_kv_formats(self, formats: Sequence[str] = ("q8", "q4"), pages: int | None = None) -> list[str]:

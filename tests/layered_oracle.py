@@ -323,6 +323,143 @@ def layer_norm(x, weight, eps):
     return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * weight
 
 
+# ---- differential attention in chunks, element-wise recurrences, experts with a shared one, loops ----------------------------------------
+def chunk_mask(n, size):
+    """Position i sees j <= i of its own chunk of ``size`` positions."""
+    i, j = torch.arange(n)[:, None], torch.arange(n)[None, :]
+    return (j <= i) & (i // size == j // size)
+
+
+def masked_attention(q, k, v, scale, mask):
+    """One head (one map): q, k [n, d], v [n, e]."""
+    return torch.softmax(((q @ k.T) * scale).masked_fill(~mask, float("-inf")), dim=-1) @ v
+
+
+def difference_factor(w, p, diff):
+    return torch.exp((w[p + "lq1"] * w[p + "lk1"]).sum()) - torch.exp((w[p + "lq2"] * w[p + "lk2"]).sum()) + diff
+
+
+def differential_mixer(h, w, p, m, eps):
+    """Two softmax maps per head over the same values; the second is taken off, the difference normalised per head, then gated."""
+    n, H, G, d, e = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    project = lambda c: linear(h, w[p + c]) + w[p + c + ".b"]
+    q = rms_norm(project("q").view(n, 2 * H, d), w[p + "q.norm"], eps)
+    k = rms_norm(project("k").view(n, 2 * G, d), w[p + "k.norm"], eps)
+    q, k = (rotate_pairs(x, 0, m["rot"]) if m["rot"]["dims"] else x for x in (q, k))
+    v = project("v").view(n, G, e)
+    mask, lam = chunk_mask(n, m["mask"]["size"]), difference_factor(w, p, m["diff"])
+    out = []
+    for a in range(H):
+        g = a // (H // G)
+        a1, a2 = (masked_attention(q[:, 2 * a + i], k[:, 2 * g + i], v[:, g], m["scale"], mask) for i in (0, 1))
+        out.append(rms(a1 - lam * a2, eps) * (1.0 - m["diff"]))
+    o = torch.stack(out, dim=1).reshape(n, H * e) * torch.sigmoid(linear(h, w[p + "g"]))
+    return linear(o, w[p + "o"]) + w[p + "o.b"]
+
+
+def mingru_candidate(u):
+    return torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+
+
+def mingru_scan(z, c, state=None):
+    """S <- (1 - z) S + z c for z, c [n, width]; every state, [n, width]."""
+    S, out = torch.zeros(z.shape[1], dtype=z.dtype) if state is None else state, []
+    for t in range(z.shape[0]):
+        S = (1.0 - z[t]) * S + z[t] * c[t]
+        out.append(S)
+    return torch.stack(out)
+
+
+def mingru_mixer(h, w, p, m, eps):
+    z = torch.sigmoid(linear(h, w[p + "z"]) + w[p + "z.b"])
+    S = mingru_scan(z, mingru_candidate(linear(h, w[p + "x"]) + w[p + "x.b"]))
+    return linear(S * silu(linear(h, w[p + "g"])), w[p + "o"])
+
+
+def selective_scan(x, dt, A, B, C, D, state=None):
+    """x, dt [n, channels], A [channels, N], B, C [n, N], D [channels]: y [n, channels] and the last state."""
+    S, out = torch.zeros_like(A) if state is None else state, []
+    for t in range(x.shape[0]):
+        S = torch.exp(dt[t][:, None] * A) * S + (dt[t] * x[t])[:, None] * B[t][None, :]
+        out.append(S @ C[t] + D * x[t])
+    return torch.stack(out), S
+
+
+def mamba1_mixer(h, w, p, m, eps):
+    inner, R, N = m["inner"], m["dt_rank"], m["state"]
+    x, z = torch.split(linear(h, w[p + "in"]), [inner, inner], dim=-1)
+    x = silu(causal_conv(x, w[p + "conv"], w[p + "conv.b"]))
+    dt, B, C = torch.split(linear(x, w[p + "x"]), [R, N, N], dim=-1)
+    dt = torch.nn.functional.softplus(linear(dt, w[p + "dt"]) + w[p + "dt.b"])
+    y, _ = selective_scan(x, dt, -torch.exp(w[p + "A_log"]), B, C, w[p + "D"])
+    return linear(y * silu(z), w[p + "o"])
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def gelu_ff(h, w, p):
+    return linear(gelu_tanh(linear(h, w[p + "gate"])) * linear(h, w[p + "up"]), w[p + "down"])
+
+
+def softmax_route(z, top):
+    """One token: the experts with the largest scores (best first) and these scores."""
+    s = torch.softmax(z, dim=-1)
+    chosen = sorted(range(len(s)), key=lambda e: -float(s[e]))[:top]
+    return chosen, torch.stack([s[e] for e in chosen])
+
+
+def shared_experts_ff(h, w, p, mlp):
+    """Chosen experts, weighted by their softmax scores, and one expert for every token behind a sigmoid."""
+    z, limit, out = linear(h, w[p + "router"]), mlp["expert"]["limit"], []
+    for t in range(h.shape[0]):
+        chosen, weights = softmax_route(z[t], mlp["router"]["top"])
+        out.append(sum(g * dense_ff(h[t], w, f"{p}e{e}.", limit) for e, g in zip(chosen, weights)))
+    out = torch.stack(out)
+    if mlp.get("shared") is not None:
+        out = out + torch.sigmoid(linear(h, w[p + "shared.sg"])) * dense_ff(h, w, p + "shared.", mlp["shared"]["limit"])
+    return out
+
+
+def grouped_norm(x, weight, groups, eps):
+    return grouped_rms(x, groups, eps) * weight
+
+
+def plus_conv(h, weight):
+    return h + causal_conv(h, weight, torch.zeros(h.shape[1], dtype=h.dtype))
+
+
+def naforax_layer(x, w, p, layer, norm, mult):
+    mixer = {"attention": differential_mixer, "mingru": mingru_mixer, "mamba1": mamba1_mixer}[layer["type"]]
+    groups, eps = norm["groups"], norm["eps"]
+    h = plus_conv(grouped_norm(x, w[p + "norm1"], groups, eps), w[p + "canon1"])
+    x = x + mult * grouped_norm(mixer(h, w, p + "mix.", layer["mixer"], eps), w[p + "norm1b"], groups, eps)
+    if layer["mlp"] is not None:
+        h = plus_conv(grouped_norm(x, w[p + "norm2"], groups, eps), w[p + "canon2"])
+        y = gelu_ff(h, w, p + "mlp.") if layer["mlp"]["kind"] == "dense" else shared_experts_ff(h, w, p + "mlp.", layer["mlp"])
+        x = x + mult * grouped_norm(y, w[p + "norm2b"], groups, eps)
+    return x
+
+
+def loop_runs(layers, loop):
+    """(layer, pass; None outside the loop) in the order they run."""
+    start, stop, times = loop["start"], loop["stop"], loop["times"]
+    return [(i, None) for i in range(start)] + [(i, t) for t in range(times) for i in range(start, stop)] + [(i, None) for i in range(stop, layers)]
+
+
+def naforax_forward(cfg, w, tokens, keep_layers=False):
+    first = w["embed"][torch.as_tensor(list(tokens), dtype=torch.long)]
+    x, kept, norm, cap = first, [], cfg["norm"], cfg["logit_softcap"]
+    for i, t in loop_runs(len(cfg["layers"]), cfg["loop"]):
+        if t is not None and i == cfg["loop"]["start"]:
+            x = x + w["loop.step"][t] + (first if t > 0 else 0.0)
+        x = naforax_layer(x, w, f"l{i}.", cfg["layers"][i], norm, cfg["residual_mult"])
+        kept.append(x)
+    logits = soft_cap(linear(grouped_norm(x, w["final.norm"], norm["groups"], norm["eps"]), w["head"]), cap)
+    return (logits, torch.stack(kept)) if keep_layers else logits
+
+
 # ---- whole models -----------------------------------------------------------------------------------------------------------------
 MIXERS = {"attention": attention_mixer, "mlstm": mlstm_mixer, "retention": retention_mixer, "lightning": lightning_mixer, "parallel": parallel_mixer}
 
@@ -359,6 +496,8 @@ def kutepel_layer(x, w, p, layer, eps, mult, shared):
 def forward(cfg, w, tokens, keep_layers=False):
     """Logits [n, vocab] of every position (and the residual stream after every layer)."""
     eps, arch = cfg["norm"]["eps"], cfg["architecture"]
+    if arch == "Naforax":
+        return naforax_forward(cfg, w, tokens, keep_layers)
     x = w["embed"][torch.as_tensor(list(tokens), dtype=torch.long)] * cfg.get("embedding", {}).get("scale", 1.0)
     kept, shared = [], []
     for l, layer in enumerate(cfg["layers"]):
