@@ -168,7 +168,7 @@ def model_dir_info(path: str) -> dict:
             "tensors": len(cfg.tensor_shapes()), "estimated_parameters": cfg.param_count(),
             "file_size_bytes": os.path.getsize(weights) if weights.exists() else 0,
             "config": {"layers": cfg.layers, "hidden": cfg.width, "vocab": cfg.vocab, "rms_eps": cfg.eps, "attention_layers": cfg.attention_layers,
-                       "recurrent_layers": cfg.recurrent_layers, "layer_list": layers},
+                       "recurrent_layers": cfg.recurrent_layers, "loop": None if cfg.loop is None else dataclasses.asdict(cfg.loop), "layer_list": layers},
             "valid": v.ok, "errors": v.errors, "warnings": v.warnings}
 
 
@@ -208,6 +208,9 @@ def cmd_info(args) -> int:
             m = l["mlp"]
             ff = ", no feed-forward" if m is None else f", feed-forward {m['ff']}" + (f" x {m['router']['top']} of {m['router']['experts']}" if "router" in m else "")
             print(f"  layer {i}: " + ", ".join(f"{k} {v}" for k, v in l.items() if k != "mlp") + ff)
+        lo = c["loop"]
+        if lo is not None:
+            print(f"  layers {lo['start']}-{lo['stop'] - 1} run {lo['times']} times")
     else:
         from .core import GgufFile
         from .core.compat import extract_model_card

@@ -103,6 +103,40 @@ def kutepel_mixed():
                     latent(17, 16, 2, 8, 16, 0.3, 50.0, mlp=experts(64, 20, 4, 10, 2, 2.0))])
 
 
+# ---- Naforax ----------------------------------------------------------------------------------------------------------------------
+def gelu(ff=70):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(ff=40, n=11, top=3, limit=0.9, shared=(56, 1.3)):
+    m = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": n, "top": top}}
+    return m if shared is None else {**m, "shared": {"ff": shared[0], "limit": shared[1]}}
+
+
+def differential(heads=6, kv_heads=2, dim=20, vdim=28, scale=0.3, size=70, dims=12, base=900.0, diff=0.4, mlp=None):
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": size},
+                                           "rot": {"base": base, "dims": dims}, "diff": diff}, "mlp": mlp}
+
+
+def mingru(width=100, mlp=None):
+    return {"type": "mingru", "mixer": {"width": width}, "mlp": mlp}
+
+
+def mamba1(inner=90, state=12, rank=9, conv=4, mlp=None):
+    return {"type": "mamba1", "mixer": {"inner": inner, "state": state, "dt_rank": rank, "conv": conv}, "mlp": mlp}
+
+
+def naforax(layers, loop=(0, 1, 1), width=152, vocab=331, eps=1e-5, groups=4, taps=3, mult=0.6, cap=9.0):
+    return {"architecture": "Naforax", "layers": layers, "loop": dict(zip(("start", "stop", "times"), loop)), "norm": {"eps": eps, "groups": groups},
+            "canon": {"taps": taps}, "residual_mult": mult, "logit_softcap": cap, "vocab": vocab, "width": width}
+
+
+# every branch in one model: all mixers inside and outside the loop, dense blocks, experts with and without a shared one, no block
+def naforax_mixed():
+    return naforax([mingru(mlp=moe()), differential(mlp=gelu()), mamba1(mlp=moe(24, 5, 1, 2.0, None)), differential(4, 4, 33, 40, 0.2, 100, 6, 50.0, 0.1, mlp=moe(33, 7, 7, 0.5)),
+                    mamba1(77, 20, 3, 2), mingru(64, mlp=gelu(45)), differential(8, 1, 16, 72, 0.4, 37, 16, 2e4, 0.7)], loop=(1, 4, 3))
+
+
 def write(path, cfg, weights):
     from oxibonsai_b200.convert import write_safetensors
     os.makedirs(path, exist_ok=True)

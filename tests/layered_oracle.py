@@ -565,8 +565,42 @@ def kutepel_tensor_shapes(cfg):
     return s
 
 
+def naforax_tensor_shapes(cfg):
+    W, V, taps = cfg["width"], cfg["vocab"], cfg["canon"]["taps"]
+    s = {"embed": (V, W), "head": (V, W), "final.norm": (W,), "loop.step": (cfg["loop"]["times"], W)}
+    for l, layer in enumerate(cfg["layers"]):
+        m, p, f, mlp = layer["mixer"], f"l{l}.mix.", f"l{l}.mlp.", layer["mlp"]
+        for n in ("1", "2") if mlp is not None else ("1",):
+            s.update({f"l{l}.norm{n}": (W,), f"l{l}.norm{n}b": (W,), f"l{l}.canon{n}": (W, taps)})
+        if layer["type"] == "attention":
+            H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            for n, rows in (("q", 2 * H * d), ("k", 2 * G * d), ("v", G * e)):
+                s.update({p + n: (rows, W), p + n + ".b": (rows,)})
+            s.update({p + n: (d,) for n in ("q.norm", "k.norm", "lq1", "lk1", "lq2", "lk2")})
+            s.update({p + "g": (H * e, W), p + "o": (W, H * e), p + "o.b": (W,)})
+        elif layer["type"] == "mingru":
+            E = m["width"]
+            s.update({p + "z": (E, W), p + "z.b": (E,), p + "x": (E, W), p + "x.b": (E,), p + "g": (E, W), p + "o": (W, E)})
+        else:
+            C, N, R = m["inner"], m["state"], m["dt_rank"]
+            s.update({p + "in": (2 * C, W), p + "conv": (C, m["conv"]), p + "conv.b": (C,), p + "x": (R + 2 * N, C), p + "dt": (C, R), p + "dt.b": (C,),
+                      p + "A_log": (C, N), p + "D": (C,), p + "o": (W, C)})
+        block = lambda q, F: {q + "gate": (F, W), q + "up": (F, W), q + "down": (W, F)}
+        if mlp is not None and mlp["kind"] == "dense":
+            s.update(block(f, mlp["ff"]))
+        elif mlp is not None:
+            s[f + "router"] = (mlp["router"]["experts"], W)
+            for j in range(mlp["router"]["experts"]):
+                s.update(block(f"{f}e{j}.", mlp["expert"]["ff"]))
+            if mlp.get("shared") is not None:
+                s.update({**block(f + "shared.", mlp["shared"]["ff"]), f + "shared.sg": (1, W)})
+    return s
+
+
 def tensor_shapes(cfg):
     """Name -> shape of every tensor of a model."""
+    if cfg["architecture"] == "Naforax":
+        return naforax_tensor_shapes(cfg)
     if cfg["architecture"] == "Kutepel":
         return kutepel_tensor_shapes(cfg)
     W, keripel = cfg["width"], cfg["architecture"] == "Keripel"
@@ -603,6 +637,16 @@ def random_weights(cfg, seed=0, scale=1.0):
             t = 1.0 + t
         elif name.endswith(".correction"):
             t = 0.3 * t - 0.2                      # some choice scores are negative
+        elif name.endswith(".dt.b"):
+            t = t - 2.0                            # step sizes around an eighth
+        elif name.endswith((".q.b", ".k.b", ".v.b", ".o.b", ".z.b", ".x.b")):
+            t = 0.4 * t
+        elif name.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
+            t = 1.2 * t * shape[0] ** -0.5
+        elif ".canon" in name:
+            t = 0.35 * t
+        elif name == "loop.step":
+            t = 0.3 * t
         elif name.endswith("A_log"):
             t = 1.5 * t - 2.0                      # from forgetting in a few tokens to hardly at all
         elif name.endswith(".D"):
@@ -616,6 +660,8 @@ def random_weights(cfg, seed=0, scale=1.0):
         w[name] = t.bfloat16().float()
     if cfg["architecture"] == "Kutepel":
         settle_routers(cfg, w, g)
+    elif cfg["architecture"] == "Naforax":
+        settle_softmax_routers(cfg, w, g)
     return w
 
 
@@ -647,3 +693,27 @@ def settle_routers(cfg, w, g, margin=0.016):
             rows[:, W - CODES + i] = col
         rows[:, -1] = -rows.sum(1)
         w[p + "mlp.router"] = rows.bfloat16().float()
+
+
+def settle_softmax_routers(cfg, w, g):
+    """The same for routers that compare logits behind a norm without a mean, in a stream that a loop adds the embedding to: sublayers,
+    convolutions and the loop's steps leave the code's dimensions alone, so that router logits are a positive multiple of well-spread ones."""
+    layers = [l for l, layer in enumerate(cfg["layers"]) if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe"]
+    if not layers:
+        return
+    W = cfg["width"]
+    code = torch.randint(0, CODES, (cfg["vocab"],), generator=g)
+    w["embed"][:, -CODES:] = 6.0 * torch.nn.functional.one_hot(code, CODES).float()
+    w["loop.step"][:, -CODES:] = 0.0
+    for l, layer in enumerate(cfg["layers"]):
+        p = f"l{l}."
+        for n in ("1", "2") if layer["mlp"] is not None else ("1",):
+            w[p + f"norm{n}"][-CODES:] = 1.0
+            w[p + f"norm{n}b"][-CODES:] = 0.0
+            w[p + f"canon{n}"][-CODES:] = 0.0
+    for l in layers:
+        E = cfg["layers"][l]["mlp"]["router"]["experts"]
+        rows = torch.zeros(E, W)
+        for i in range(CODES):
+            rows[:, W - CODES + i] = torch.linspace(-0.6, 0.6, E)[torch.randperm(E, generator=g)] if E > 1 else torch.ones(1)
+        w[f"l{l}.mlp.router"] = rows.bfloat16().float()
