@@ -58,8 +58,8 @@ def parse_args():
     ap.add_argument("--no-replicas", action="store_true", help="skip the independent-replica measurement at N > 1")
     ap.add_argument("--no-gate", action="store_true", help="skip the correctness gate")
     ap.add_argument("--no-extras", action="store_true", help="skip the exact-f32 and NCCL-baseline measurements")
-    ap.add_argument("--design", choices=["keripel", "kekevik", "kutepel"], help="instead of the headline: prefill and decode throughput of a layer-list "
-                    "design beside the closest existing model (keripel: the generic-format engine; kekevik: keripel; kutepel: kekevik) at equal parameter count (1 GPU)")
+    ap.add_argument("--design", choices=["keripel", "kekevik", "kutepel", "naforax"], help="instead of the headline: prefill and decode throughput of a layer-list "
+                    "design beside the closest existing model (keripel: the generic-format engine; kekevik: keripel; kutepel and naforax: kekevik) at equal parameter count (1 GPU)")
     ap.add_argument("--design-sizes", default="s,m,l", help="--design: model sizes (benchmarks/layered.py)")
     ap.add_argument("--model-dir", default=os.environ.get("BONSAI_BENCH_DIR", "/tmp/oxibonsai_b200_bench"))
     return ap.parse_args()
@@ -270,7 +270,7 @@ def design_bench(args) -> None:
     clocks = ClockSampler(0)
     clocks.start()
     run, like = {"keripel": (layered.run_models, "the generic-format f16 engine"), "kekevik": (layered.run_kekevik, "the keripel design"),
-                 "kutepel": (layered.run_kutepel, "the kekevik design")}[args.design]
+                 "kutepel": (layered.run_kutepel, "the kekevik design"), "naforax": (layered.run_naforax, "the kekevik design")}[args.design]
     rows = run(args.design_sizes.split(","), steps=args.steps, warmup=max(3, args.warmup), log=sys.stderr)
     print(json.dumps({"metric": f"prefill and decode tokens/s, {args.design} design beside {like}", "unit": "tokens/s", "n_gpus": 1,
                       "steps": args.steps, "warmup": max(3, args.warmup), "higher_is_better": True, "dtype": "bf16", "data": "synthetic (random weights and tokens)",

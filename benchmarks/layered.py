@@ -1,6 +1,6 @@
 #!/usr/bin/env python
 """Layer-list decoders beside the closest existing model: Keripel beside the generic-format Qwen3 engine with f16 weights,
-Kekevik beside Keripel, Kutepel beside Kekevik.
+Kekevik beside Keripel, Kutepel and Naforax beside Kekevik.
 
     python benchmarks/layered.py kernels [--width 4096] [--only ..]     the kernels and their counterparts, with roofline fractions
     python benchmarks/layered.py models --design kutepel [--sizes s,m]  prefill and decode throughput at equal parameter count
@@ -66,6 +66,18 @@ def kutepel(width: int, repeats: int, vocab: int = 32000, n: int = 32, top: int 
     return {"architecture": "Kutepel", "layers": layers, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "vocab": vocab, "width": width}
 
 
+def naforax(width: int, repeats: int, vocab: int = 32000, n: int = 32, top: int = 4, times: int = 2) -> dict:
+    """``repeats`` times a layer of differential attention with a dense block, a minGRU, a selective scan, and attention again, those with
+    ``n`` experts of a quarter of the width and a shared one; the recurrent layers of the first repeat run ``times`` times."""
+    H = width // 128
+    moe = {"kind": "moe", "expert": {"ff": width // 4, "limit": 7.0}, "router": {"experts": n, "top": top}, "shared": {"ff": width // 2, "limit": 7.0}}
+    a = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "mask": {"size": 8192}, "rot": {"base": 500000.0, "dims": 64}, "diff": 0.5}
+    layers = [{"type": "attention", "mlp": {"kind": "dense", "ff": 3 * width}, "mixer": a}, {"type": "mingru", "mlp": moe, "mixer": {"width": width}},
+              {"type": "mamba1", "mlp": moe, "mixer": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}}, {"type": "attention", "mlp": moe, "mixer": a}]
+    return {"architecture": "Naforax", "layers": layers * repeats, "loop": {"start": 1, "stop": 3, "times": times}, "norm": {"eps": 1e-6, "groups": 4},
+            "canon": {"taps": 4}, "residual_mult": 0.5, "logit_softcap": 30.0, "vocab": vocab, "width": width}
+
+
 def write_design(path: str, cfg: dict) -> int:
     """A model directory with random bf16 weights; returns the parameter count."""
     from oxibonsai_b200.convert import write_safetensors
@@ -78,7 +90,7 @@ def write_design(path: str, cfg: dict) -> int:
     t = {}
     for n, s in config.tensor_shapes().items():
         x = torch.randn(s, generator=g, device="cuda")
-        x = 1 + 0.1 * x if "norm" in n else (x if len(s) == 1 else x * s[-1] ** -0.5)
+        x = 1 + 0.1 * x if "norm" in n else (0.3 * x if len(s) == 1 else x * s[-1] ** -0.5)
         t[n] = x.bfloat16().cpu()
     write_safetensors(os.path.join(path, "model.safetensors"), t)
     return config.param_count()
@@ -161,8 +173,8 @@ def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
         proj = torch.randn(B, ld, device=dev)
         w1, slopes = torch.ones(hd, device=dev), torch.full((nq,), 0.01, device=dev)
         out = torch.zeros(B, nq * hd, dtype=torch.bfloat16, device=dev)
-        calls = [L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, p, rk, None, out, None, None],
-                             [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, 0, 0, 1, 0, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0]) for p in pools]
+        calls = [L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, p, rk, None, out, *[None] * 5],
+                             [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, 0, 0, 1, 0, 0, 0, 1, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0, 0.0, 1.0]) for p in pools]
         it = [0]
         split = 1
         while split < 8 and B * nkv * split * 2 <= 160:
@@ -188,8 +200,8 @@ def bench_attention(rep: Report, width: int, iters: int, profile: bool) -> None:
     entries = torch.tensor([0, T, 0, 0], **i32)
     tiles = torch.tensor([[0, t] for t in range(0, T, tpt)], **i32)
     for window in (0, 1024):
-        call = L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, pool, rk, None, out, None, None],
-                           [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, window, 4, 1, 0, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0])
+        call = L.MixerCall([proj, w1, w1, slopes, pos, slots, bt, pool, rk, None, out, *[None] * 5],
+                           [ld, 0, nq * hd, 0, (nq + nkv) * hd, nq * hd, nq, nkv, hd, hd, npages, page, window, 4, 1, 0, 0, 0, 1, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0, 0.0, 1.0])
 
         def ours():
             K.check(L.lib().bonsai_lay_attn_prompt(*call.args, entries.data_ptr(), tiles.data_ptr(), len(tiles), K.stream()), "attn_prompt")
@@ -216,8 +228,8 @@ def bench_capped_attention(rep: Report, width: int, iters: int, profile: bool) -
     ld = (nq + 2 * nkv) * hd
 
     def call(proj, pos, slots, bt, k, v, out, cap=50.0):
-        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out, None, None],
-                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0, 1, 0, 0], [1e-6, hd ** -0.5, 0.5, cap, 0.1, 4096.0])
+        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out, *[None] * 5],
+                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0, 1, 0, 0, 0, 1, 0], [1e-6, hd ** -0.5, 0.5, cap, 0.1, 4096.0, 0.0, 1.0])
     for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
         npages = ctx // page
         copies = max(2, int(300e6 / (4 * B * ctx * nkv * hd)) + 1)
@@ -260,8 +272,8 @@ def bench_rotary(rep: Report, width: int, iters: int, profile: bool) -> None:
     rot, sinks = torch.randn(4096, hd // 2, 2, device=dev), torch.ones(nq, device=dev)
 
     def call(proj, pos, slots, bt, k, v, out):
-        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out, sinks, rot],
-                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0, 0, hd, 1], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0])
+        return L.MixerCall([proj, None, None, None, pos, slots, bt, k, None, v, out, sinks, rot, None, None, None],
+                           [ld, 0, nq * hd, (nq + nkv) * hd, -1, nq * hd, nq, nkv, hd, hd, bt.shape[1], page, 0, 0, 0, hd, 1, 0, 1, 0], [1e-6, hd ** -0.5, 1.0, 0.0, 0.0, 1.0, 0.0, 1.0])
     for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
         npages = ctx // page
         copies = max(2, int(300e6 / (4 * B * ctx * nkv * hd)) + 1)
@@ -420,20 +432,20 @@ def bench_experts(rep: Report, width: int, iters: int, profile: bool) -> None:
                 li, tok, wt = lists[it[0] % 8]
                 if few:
                     K.check(lib.bonsai_lay_experts_few(r.up.data.data_ptr(), E, 2 * ff, width, h.data_ptr(), width, li.data_ptr(), tok.data_ptr(), wt.data_ptr(), pairs,
-                                                       min(E, pairs), min(T, 2 * pairs // E + 8), hid.data_ptr(), ff, 1, float("inf"), 1.0, 0.0, st()), "experts_few")
+                                                       min(E, pairs), min(T, 2 * pairs // E + 8), hid.data_ptr(), ff, 1, float("inf"), 1.0, 0.0, 0.0, st()), "experts_few")
                 else:
                     K.check(lib.bonsai_grouped_gemm_bf16(r.up.data.data_ptr(), E, 2 * ff, width, xs.data_ptr(), width, pairs, li.data_ptr(), wt.data_ptr(), hid.data_ptr(), ff, 4,
-                                                         float("inf"), 1.0, 0.0, int(pairs > 96 * E), scratch.status.data_ptr(), scratch.sms, st()), "grouped_gemm")
+                                                         float("inf"), 1.0, 0.0, 0.0, int(pairs > 96 * E), scratch.status.data_ptr(), scratch.sms, st()), "grouped_gemm")
 
             def down():
                 it[0] += 1
                 li = lists[it[0] % 8][0]
                 if few:
                     K.check(lib.bonsai_lay_experts_few(r.down.data.data_ptr(), E, width, ff, hid.data_ptr(), ff, li.data_ptr(), None, None, pairs, min(E, pairs),
-                                                       min(T, 2 * pairs // E + 8), s.out32.data_ptr(), s.out32.stride(0), 0, 0.0, 0.0, 0.0, st()), "experts_few")
+                                                       min(T, 2 * pairs // E + 8), s.out32.data_ptr(), s.out32.stride(0), 0, 0.0, 0.0, 0.0, 0.0, st()), "experts_few")
                 else:
                     K.check(lib.bonsai_grouped_gemm_bf16(r.down.data.data_ptr(), E, width, ff, hid.data_ptr(), ff, pairs, li.data_ptr(), None, s.out.data_ptr(), s.out.stride(0), 6,
-                                                         0.0, 0.0, 0.0, int(pairs > 96 * E), scratch.status.data_ptr(), scratch.sms, st()), "grouped_gemm")
+                                                         0.0, 0.0, 0.0, 0.0, int(pairs > 96 * E), scratch.status.data_ptr(), scratch.sms, st()), "grouped_gemm")
             rep.add("experts, gate/up", case, time_us(up, iters, profile), chosen * 2 * like + 2 * (T if few else pairs) * width + 2 * pairs * ff, 4.0 * pairs * ff * width)
             rep.add("experts, down", case, time_us(down, iters, profile), chosen * like + 2 * pairs * ff + (4 if few else 2) * pairs * width, 2.0 * pairs * ff * width)
             r.out = s.out32 if few else s.out
@@ -560,6 +572,186 @@ def bench_mlstm(rep: Report, width: int, iters: int, profile: bool) -> None:
         rep.add("norm_add", f"T={T} width={width}", time_us(lambda: L.norm_add(x, y, w, 1e-6, T, x16), iters, profile), 14.0 * T * width)
 
 
+class BenchRows:
+    """Rows of ``nseq`` sequences, single tokens at position ``pos`` or portions of ``T`` tokens, with the lists of a step."""
+
+    def __init__(self, nseq: int, T: int, pos: int = 0):
+        from oxibonsai_b200.models.layered import StepShape
+        from oxibonsai_b200.ops import layered_ops as L
+        i32, rows, tile = dict(dtype=torch.int32, device="cuda"), nseq * T, L.lib().bonsai_lay_conv_rows()
+        self.tokens, self.rows = torch.zeros(rows, **i32), rows
+        self.positions = torch.arange(T, **i32).repeat(nseq) + pos
+        self.slots, self.state = torch.arange(nseq, **i32).repeat_interleave(T), torch.arange(nseq, **i32)
+        if T == 1:
+            self.shape = StepShape(rows, rows, rows)
+            return
+        self.entries = torch.tensor([[s * T, T, s, pos] for s in range(nseq)], **i32)
+        self.tiles = torch.tensor([[s, t] for s in range(nseq) for t in range(0, T, tile)], **i32)
+        self.shape = StepShape(rows, 0, 0, nseq, self.entries.data_ptr(), {tile: (self.tiles.data_ptr(), len(self.tiles))})
+
+
+def bench_differential(rep: Report, width: int, iters: int, profile: bool) -> None:
+    """Two maps of 64 dimensions over values of 128; the like kernels are those of bench_capped_attention and bench_rotary."""
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev = torch.device("cuda")
+    nq, nkv, hd, page = width // 128, max(1, width // 512), 128, 64
+    i32 = dict(dtype=torch.int32, device=dev)
+    ld = (2 * nq + 2 * nkv) * hd
+    rot, norm, bias = torch.randn(4096, 32, 2, device=dev), torch.ones(64, device=dev), torch.zeros(nq * hd, device=dev)
+
+    def call(proj, pos, slots, bt, k, v, out):
+        return L.MixerCall([proj, norm, norm, None, pos, slots, bt, k, None, v, out, None, rot, bias, bias, bias],
+                           [ld, 0, nq * hd, (nq + nkv) * hd, (nq + 2 * nkv) * hd, nq * hd, nq, nkv, 64, hd, bt.shape[1], page, 0, 0, 1, 64, 1, 8192, 2, 1],
+                           [1e-6, 0.125, 1.0, 0.0, 0.0, 1.0, 0.6, 0.5])
+    per_pair = 2.0 * nq * (2 * 64 + 2 * hd)
+    for B, ctx in ((1, 4096), (8, 4096), (64, 1024)):
+        npages = ctx // page
+        copies = max(2, int(300e6 / (4 * B * ctx * nkv * hd)) + 1)
+        pools = [[torch.randn(B * npages, nkv, page, hd, device=dev).bfloat16() for _ in range(2)] for _ in range(copies)]
+        bt = torch.arange(B * npages, **i32).view(B, npages)
+        pos, slots, proj = torch.full((B,), ctx - 1, **i32), torch.arange(B, **i32), torch.randn(B, ld, device=dev)
+        out = torch.zeros(B, nq * hd, dtype=torch.bfloat16, device=dev)
+        calls = [call(proj, pos, slots, bt, *p, out) for p in pools]
+        it, split = [0], 1
+        while split < 8 and B * nkv * split * 2 <= 160:
+            split *= 2
+
+        def ours():
+            it[0] += 1
+            K.check(L.lib().bonsai_lay_attn_decode(*calls[it[0] % copies].args, B, split, K.stream()), "attn_decode")
+        rep.add("attn_decode, two maps", f"B={B} ctx={ctx} heads={nq}/{nkv}", time_us(ours, iters, profile), 4 * B * ctx * nkv * hd, per_pair * B * ctx)
+    T, npages = 4096, 64
+    k, v = (torch.randn(npages, nkv, page, hd, device=dev).bfloat16() for _ in range(2))
+    bt, pos, slots = torch.arange(npages, **i32).view(1, -1), torch.arange(T, **i32), torch.zeros(T, **i32)
+    proj, out = torch.randn(T, ld, device=dev), torch.zeros(T, nq * hd, dtype=torch.bfloat16, device=dev)
+    entries = torch.tensor([0, T, 0, 0], **i32)
+    tiles = torch.tensor([[0, t] for t in range(0, T, 64 // (nq // nkv))], **i32)
+    c = call(proj, pos, slots, bt, k, v, out)
+    fn = lambda: K.check(L.lib().bonsai_lay_attn_prompt(*c.args, entries.data_ptr(), tiles.data_ptr(), len(tiles), K.stream()), "attn_prompt")
+    rep.add("attn_prompt, two maps", f"T={T} heads={nq}/{nkv}", time_us(fn, 10, profile), 4 * T * ld + 4 * T * nkv * hd + 2 * T * nq * hd, per_pair * T * (T + 1) / 2)
+    fn = lambda: K.check(L.lib().bonsai_lay_attn_append(*c.args, 0, T, 0, K.stream()), "attn_append")
+    rep.add("attn_append, two maps", f"T={T}", time_us(fn, iters, profile), 12 * T * nkv * hd)
+
+
+def bench_scans(rep: Report, width: int, iters: int, profile: bool) -> None:
+    """minGRU, the selective scan and the convolutions; the like kernels are those of bench_recurrence."""
+    from oxibonsai_b200.models.layered import CHUNK, MAX_SEGMENTS, SCAN_COST, SegmentPlan, plan_segments
+    from oxibonsai_b200.ops import cuda_ops as K
+    from oxibonsai_b200.ops import layered_ops as L
+    dev, lib = torch.device("cuda"), L.lib()
+    sms, W, N, R = torch.cuda.get_device_properties(dev).multi_processor_count, width, 16, width // 16
+    inner, i32, it = 2 * width, dict(dtype=torch.int32, device=dev), [0]
+    vec = torch.zeros(inner, device=dev)
+
+    def turn(calls, fn):
+        def run():
+            it[0] += 1
+            fn(calls[it[0] % len(calls)].args)
+        return run
+
+    def gru(rows):
+        proj, out = torch.randn(rows.rows, 3 * W, device=dev), torch.zeros(rows.rows, W, dtype=torch.bfloat16, device=dev)
+        return L.MixerCall([proj, vec, vec, torch.zeros(len(rows.state), W, device=dev), rows.positions, rows.slots, rows.state, out], [3 * W, 0, W, 2 * W, W, W], [])
+    scratch = [torch.empty(MAX_SEGMENTS * inner * n, device=dev) for n in (N, 1)]
+    A = -torch.rand(inner, N, device=dev)
+
+    def scan(rows):
+        T = rows.rows
+        proj, bc, dt = torch.randn(T, 2 * inner, device=dev), torch.randn(T, R + 2 * N, device=dev), torch.randn(T, inner, device=dev)
+        x, out = (torch.randn(T, inner, device=dev).bfloat16() for _ in range(2))
+        return L.MixerCall([proj, bc, dt, x, vec, A, vec, torch.zeros(len(rows.state), inner, N, device=dev), rows.positions, rows.slots, rows.state, out, *scratch],
+                           [2 * inner, inner, R + 2 * N, R, R + N, inner, inner, inner, inner, N], [])
+    for B in (1, 8, 64):
+        rows, copies = BenchRows(B, 1, 5), 2 + int(300e6 / (B * inner * (8 * N + 14)))
+        rep.add("gru_step", f"B={B} width={W}", time_us(turn([gru(rows) for _ in range(copies)], lambda a: K.check(lib.bonsai_lay_gru_step(*a, B, 0, K.stream()), "gru_step")),
+                                                        iters, profile), 22.0 * B * W)
+        rep.add("scan_step", f"B={B} {inner} x {N}", time_us(turn([scan(rows) for _ in range(copies)], lambda a: K.check(lib.bonsai_lay_scan_step(*a, B, 0, K.stream()), "scan_step")),
+                                                             iters, profile), B * inner * (8.0 * N + 12) + 4.0 * inner * N)
+        conv = lambda c: L.Conv(torch.randn(B, c, device=dev), 0, c, torch.randn(4, c, device=dev), vec, torch.zeros(B, 4, c, device=dev), rows, rows.state,
+                                torch.zeros(B, c, dtype=torch.bfloat16, device=dev), silu=True)
+        convs = [conv(inner) for _ in range(copies)]
+
+        def run_conv():
+            it[0] += 1
+            convs[it[0] % copies](rows.shape)
+        rep.add("conv, silu", f"B={B} channels={inner}", time_us(run_conv, iters, profile), 22.0 * B * inner)
+    for nseq, T in ((1, 4096), (1, 512), (8, 512)):
+        rows, n = BenchRows(nseq, T), nseq * T
+        copies = 1 + int(300e6 / (14.0 * n * W))
+        cluster, ctas = 1, nseq * -(-W // 32)
+        while cluster < 8 and 2 * cluster * ctas <= 2 * sms and 2 * cluster * lib.bonsai_lay_gru_tokens() <= T:
+            cluster *= 2
+        fn = lambda a: K.check(lib.bonsai_lay_gru_scan(*a, rows.shape.entries, nseq, cluster, 0, K.stream()), "gru_scan")
+        rep.add("gru_scan", f"{nseq} x {T} tokens width={W} cluster={cluster}", time_us(turn([gru(rows) for _ in range(copies)], fn), 10, profile), 14.0 * n * W)
+        plan = SegmentPlan(-(-inner // lib.bonsai_lay_scan_channels(N)), SCAN_COST)
+        size = plan_segments([T] * nseq, plan, sms) * CHUNK
+        for size in sorted({0, size, 1024, 512}):
+            if size and nseq * -(-T // size) > MAX_SEGMENTS or size >= T:
+                continue
+            segs = [(s * T + x, min(size, T - x), s, int(x + size >= T)) for s in range(nseq) for x in range(0, T, size)] if size else []
+            per = len(segs) // nseq
+            sl, pl = torch.tensor(segs or [[0] * 4], **i32), torch.tensor([(s, 0, s * per, per) for s in range(nseq)], **i32)
+            fn = lambda a: K.check(lib.bonsai_lay_scan(*a, rows.shape.entries, nseq, sl.data_ptr(), len(segs), pl.data_ptr(), 0, K.stream()), "scan")
+            rep.add("scan", f"{nseq} x {T} tokens {inner} x {N} segments={len(segs)}", time_us(turn([scan(rows)], fn), 10, profile), n * (12.0 * inner + 8 * N))
+        if n < 4096 or nseq > 1:
+            continue
+        for c, silu in ((W, False), (inner, True)):
+            x, out = torch.randn(n, c, device=dev), torch.zeros(n, c, dtype=torch.bfloat16, device=dev)
+            conv = L.Conv(x, 0, c, torch.randn(4, c, device=dev), vec if silu else None, torch.zeros(nseq, 4, c, device=dev), rows, rows.state, out, add=not silu, silu=silu)
+            rep.add("conv" + (", silu" if silu else ", added"), f"T={n} channels={c}", time_us(lambda: conv(rows.shape), iters, profile), 6.0 * n * c)
+        bc, low = torch.randn(n, R + 2 * N, device=dev), torch.zeros(n, L.round_up(R, 128), dtype=torch.bfloat16, device=dev)
+        rep.add("narrow", f"T={n} columns={R}", time_us(lambda: L.narrow(bc, 0, R, n, low), iters, profile), 6.0 * n * R)
+        scratch2 = L.GemmScratch(dev, torch.zeros(1, dtype=torch.int32, device=dev))
+        for rows_, k in ((R + 2 * N, inner), (inner, R)):
+            for T2 in (1, 64, n):
+                w = L.DenseWeight([torch.randn(rows_, k).bfloat16()], dev)
+                x, out = torch.randn(n, w.kp, device=dev).bfloat16(), torch.zeros(n, rows_, device=dev)
+                rep.add("linear", f"{rows_}x{k} T={T2}", time_us(lambda: L.linear(w, x, T2, out, scratch2), iters, profile), 2.0 * rows_ * k + T2 * (2.0 * k + 4 * rows_), 2.0 * T2 * rows_ * k)
+
+
+def bench_row_steps(rep: Report, width: int, iters: int, profile: bool) -> None:
+    """The general row step, the gelu gate, the capped head and the softmax router; the like kernels are norm_add, side_by_side, the gated
+    and the plain projections and the sigmoid router."""
+    from oxibonsai_b200.models.layered_config import ExpertsSpec, RouterSpec, gelu_mlp
+    from oxibonsai_b200.ops import layered_ops as L
+    dev, W = torch.device("cuda"), width
+    scratch = L.GemmScratch(dev, torch.zeros(1, dtype=torch.int32, device=dev))
+    w = torch.ones(W, device=dev)
+    for T in (1, 8, 64, 4096):
+        rows = BenchRows(T, 1, 9) if T < 4096 else BenchRows(1, T)
+        x, y, h = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev), torch.zeros(T, W, dtype=torch.bfloat16, device=dev)
+        conv, n32 = (torch.randn(4, W, device=dev), torch.zeros(len(rows.state), 4, W, device=dev)), torch.zeros(T, W, device=dev)
+        common = dict(eps=1e-6, groups=4, mult=0.5, y=y, w=w, next_norm=w)
+        plain = L.RowStep(x, h, rows, rows.state, **common)
+        rep.add("row_step", f"T={T} width={W}", time_us(lambda: plain(T, rows.shape), iters, profile), 14.0 * T * W)
+        full = L.RowStep(x, h, rows, rows.state, conv=conv, n32=n32, **common)
+        rep.add("row_step, convolution", f"T={T} width={W}", time_us(lambda: full(T, rows.shape), iters, profile), (14.0 + (16 if T < 4096 else 0)) * T * W)
+        spec = ExpertsSpec(RouterSpec(32, 4, softmax=True, normalized=False, corrected=False), 64)
+        s, logits = L.ExpertScratch(T, W, [spec], False, dev), torch.randn(T, 36, device=dev)
+        r = L.Routing(spec, L.DenseWeight([torch.zeros(64 * 32, 128).bfloat16()] * 2, dev, interleave=True), L.DenseWeight([torch.zeros(8, 128).bfloat16()], dev), None, logits, 0, s)
+        s.at.copy_(torch.randperm(4 * T, device=dev).int())
+        step = L.RowStep(x, h, rows, rows.state, gate=logits[:, 32:], **common)
+        rep.add("row_step, experts", f"T={T} width={W}", time_us(lambda: step(T, rows.shape, r), iters, profile), 22.0 * T * W)
+    g = gelu_mlp(3 * W)
+    for T in (1, 64, 4096):
+        for name, n, act in (("gate_up, gelu", 6 * W, L.Glu(g.limit, g.alpha, g.offset, g.cubic)), ("head, capped", 32000, L.SoftCap(30.0))):
+            copies = 3
+            ws = []
+            for _ in range(copies):
+                m = L.DenseWeight([torch.zeros(8, W, dtype=torch.bfloat16)], dev)
+                m.n, m.data = n, torch.randn(n, W, device=dev).bfloat16()
+                ws.append(m)
+            h = torch.randn(T, W, device=dev).bfloat16()
+            out = torch.empty(T, n // 2, dtype=torch.bfloat16, device=dev) if "gate" in name else torch.empty(T, n, device=dev)
+            it = [0]
+
+            def run():
+                it[0] += 1
+                L.linear(ws[it[0] % copies], h, T, out, scratch, act)
+            rep.add("linear", f"{name} {n}x{W} T={T}", time_us(run, iters, profile), 2.0 * n * W + 2.0 * T * W + out.numel() * out.element_size(), 2.0 * T * n * W)
+
+
 # ---- whole models ---------------------------------------------------------------------------------------------------------------------
 SIZES = {"s": dict(width=1024, repeats=3), "m": dict(width=2048, repeats=4), "l": dict(width=4096, repeats=4)}
 
@@ -679,6 +871,41 @@ def run_kutepel(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, bat
     return rows
 
 
+def used_params(cfg: dict) -> int:
+    """Parameters a token uses, those of a loop as often as it runs."""
+    from oxibonsai_b200.models.registry import ARCHITECTURES
+    c = ARCHITECTURES[cfg["architecture"]](cfg, "")
+    size = lambda prefix: sum(torch.Size(s).numel() for n, s in c.tensor_shapes().items() if n.startswith(prefix))
+    idle = lambda i: 3 * c.experts(i).ff * c.width * (c.experts(i).router.experts - c.experts(i).router.top) if i in c.expert_layers else 0
+    return size("head") + sum(size(f"l{r.layer}.") - idle(r.layer) for r in c.runs)
+
+
+def run_naforax(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64), log=sys.stdout) -> list[dict]:
+    """Naforax beside Kekevik of the same width with as many layers as bring it to the same parameter count, and to the count that a
+    token of Naforax uses (its loop counted as often as it runs)."""
+    rows = []
+    for size in sizes:
+        width = SIZES[size]["width"]
+        cfg = naforax(width, 1)
+        row = {"size": size, "width": width, "naforax_layers": len(cfg["layers"]), "used_params_M": round(used_params(cfg) / 1e6)}
+        with tempfile.TemporaryDirectory() as d:
+            row["params_M"] = round(write_design(os.path.join(d, "m"), cfg) / 1e6)
+            row["naforax"] = measure_layered(os.path.join(d, "m"), steps, warmup, prompt, batches)
+        torch.cuda.empty_cache()
+        for name, target in (("kekevik", row["params_M"]), ("kekevik_used", row["used_params_M"])):
+            with tempfile.TemporaryDirectory() as d:
+                count = lambda n: write_design(os.path.join(d, "m"), kekevik(width, n))
+                one, two = count(1), count(2)
+                other = kekevik(width, max(1, round((target * 1e6 - one) / (two - one)) + 1))
+                params = write_design(os.path.join(d, "m"), other)
+                row[f"{name}_layers"], row[f"{name}_params_M"] = len(other["layers"]), round(params / 1e6)
+                row[name] = measure_layered(os.path.join(d, "m"), steps, warmup, prompt, batches)
+            torch.cuda.empty_cache()
+        rows.append(row)
+        print(json.dumps(row), file=log, flush=True)
+    return rows
+
+
 def run_models(sizes, steps: int = 64, warmup: int = 5, prompt: int = 2048, batches=(1, 8, 64), log=sys.stdout) -> list[dict]:
     from oxibonsai_b200.cli import requantize_gguf
     from oxibonsai_b200.core import Qwen3Config, write_synthetic_gguf
@@ -711,19 +938,20 @@ def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("case", choices=["kernels", "models"])
     ap.add_argument("--width", type=int, default=4096)
-    ap.add_argument("--only", default="linear,attention,mlstm,capped,recurrence,rotary,latent,experts")
-    ap.add_argument("--design", choices=["keripel", "kekevik", "kutepel"], default="kutepel")
+    ap.add_argument("--only", default="linear,attention,mlstm,capped,recurrence,rotary,latent,experts,differential,scans,rows")
+    ap.add_argument("--design", choices=["keripel", "kekevik", "kutepel", "naforax"], default="naforax")
     ap.add_argument("--iters", type=int, default=40)
     ap.add_argument("--sizes", default="s,m,l")
     ap.add_argument("--profile", action="store_true", help="a few eager launches per case, for captures under a profiler")
     a = ap.parse_args()
     torch.cuda.set_device(0)
     if a.case == "models":
-        {"keripel": run_models, "kekevik": run_kekevik, "kutepel": run_kutepel}[a.design](a.sizes.split(","))
+        {"keripel": run_models, "kekevik": run_kekevik, "kutepel": run_kutepel, "naforax": run_naforax}[a.design](a.sizes.split(","))
         return
     rep = Report()
     for name, fn in (("linear", bench_linear), ("attention", bench_attention), ("mlstm", bench_mlstm), ("capped", bench_capped_attention),
-                     ("recurrence", bench_recurrence), ("rotary", bench_rotary), ("latent", bench_latent), ("experts", bench_experts)):
+                     ("recurrence", bench_recurrence), ("rotary", bench_rotary), ("latent", bench_latent), ("experts", bench_experts),
+                     ("differential", bench_differential), ("scans", bench_scans), ("rows", bench_row_steps)):
         if name in a.only.split(","):
             fn(rep, a.width, a.iters, a.profile)
 

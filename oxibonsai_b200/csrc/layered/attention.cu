@@ -26,6 +26,7 @@
 // query row of its own, zero in the other map's half); `f32_kernel` is the 32-bit mode for both.
 // Only the page tiles that a window or a chunk can see are visited: the kept first tokens and the range behind its first position.
 #include <cooperative_groups.h>
+#include <type_traits>
 
 #include "layered/layered.cuh"
 
@@ -61,6 +62,26 @@ struct Attn {
   float lambda, diff_scale; // two maps
 };
 
+// Calls f with "biases" and "norm weights" as types: code whose loads depend on neither at run time (a branch around a load keeps it
+// from being issued with the others).  Two maps have both, shared rows no biases.
+template <bool SEP, int MAPS, typename F>
+__device__ __forceinline__ void with_flags(bool bias, bool norm, F f) {
+  using Y = std::true_type;
+  using N = std::false_type;
+  if constexpr (MAPS == 2) {
+    f(Y(), Y());
+  } else {
+    if constexpr (SEP) {
+      if (bias) {
+        if (norm) f(Y(), Y());
+        else f(Y(), N());
+        return;
+      }
+    }
+    if (norm) f(N(), Y());
+    else f(N(), N());
+  }
+}
 __device__ __forceinline__ float biased(const float* p, const float* b, int i) { return b == nullptr ? p[i] : p[i] + b[i]; }
 
 __device__ __forceinline__ float temperature(const Attn& a, int pos) {
@@ -95,33 +116,40 @@ __device__ __forceinline__ void append_row(const Attn& a, const float* proj, int
   C* dst = static_cast<C*>(a.pool) + row * HD;
   const float* k = proj + a.k_col + kvh * MAPS * a.dim;
   if constexpr (SEP) {
-    const float* v = proj + a.v_col + kvh * a.vdim;
-    const float* vb = a.v_bias == nullptr ? nullptr : a.v_bias + kvh * a.vdim;
-    C* vdst = static_cast<C*>(a.vpool) + row * HD;
-    const float2* rot = angles(a, pos);
-    float x[HD / 32], ss[MAPS];
+    with_flags<SEP, MAPS>(a.k_bias != nullptr, a.k_norm != nullptr, [&](auto bias, auto norm) {
+      constexpr bool BIAS = decltype(bias)::value, NORM = decltype(norm)::value;
+      const float* v = proj + a.v_col + kvh * a.vdim;
+      const float* vb = a.v_bias + kvh * a.vdim;
+      C* vdst = static_cast<C*>(a.vpool) + row * HD;
+      const float2* rot = angles(a, pos);
+      float x[HD / 32], y[HD / 32], ss[MAPS];
 #pragma unroll
-    for (int m = 0; m < MAPS; ++m) ss[m] = 0.0f;
+      for (int m = 0; m < MAPS; ++m) ss[m] = 0.0f;
 #pragma unroll
-    for (int i = 0; i < HD / 32; ++i) {
-      const int c = lane + 32 * i, m = c / KD, d = c % KD;
-      const float* km = k + m * a.dim;
-      const float* kb = a.k_bias == nullptr ? nullptr : a.k_bias + (kvh * MAPS + m) * a.dim;
-      float raw = 0.0f;
-      x[i] = 0.0f;
-      if (d < a.dim) {
-        raw = biased(km, kb, d);
-        x[i] = rotated([&](int j) { return biased(km, kb, j) * (a.k_norm == nullptr ? 1.0f : a.k_norm[j]); }, d, rot, a.rot_dims, a.rot_pairs);
+      for (int i = 0; i < HD / 32; ++i) {            // every load ahead of the first store
+        const int c = lane + 32 * i, m = c / KD, d = c % KD;
+        const float* km = k + m * a.dim;
+        const float* kb = a.k_bias + (kvh * MAPS + m) * a.dim;
+        auto raw = [&](int j) { return BIAS ? km[j] + kb[j] : km[j]; };
+        float r = 0.0f;
+        x[i] = 0.0f;
+        if (d < a.dim) {
+          r = raw(d);
+          x[i] = rotated([&](int j) { return NORM ? raw(j) * a.k_norm[j] : raw(j); }, d, rot, a.rot_dims, a.rot_pairs);
+        }
+        y[i] = c < a.vdim ? (BIAS ? v[c] + vb[c] : v[c]) : 0.0f;
+#pragma unroll
+        for (int j = 0; j < MAPS; ++j) ss[j] += MAPS == 1 || m == j ? r * r : 0.0f;
       }
-      store_act(vdst + c, c < a.vdim ? biased(v, vb, c) : 0.0f);
+      float inv[MAPS];
 #pragma unroll
-      for (int j = 0; j < MAPS; ++j) ss[j] += MAPS == 1 || m == j ? raw * raw : 0.0f;
-    }
-    float inv[MAPS];
+      for (int m = 0; m < MAPS; ++m) inv[m] = a.normed ? 1.0f / sqrtf(warp_sum(ss[m]) / (float)a.dim + a.eps) : 1.0f;
 #pragma unroll
-    for (int m = 0; m < MAPS; ++m) inv[m] = a.normed ? 1.0f / sqrtf(warp_sum(ss[m]) / (float)a.dim + a.eps) : 1.0f;
-#pragma unroll
-    for (int i = 0; i < HD / 32; ++i) store_act(dst + lane + 32 * i, x[i] * (MAPS == 1 || lane + 32 * i < KD ? inv[0] : inv[MAPS - 1]));
+      for (int i = 0; i < HD / 32; ++i) {
+        store_act(dst + lane + 32 * i, x[i] * (MAPS == 1 || lane + 32 * i < KD ? inv[0] : inv[MAPS - 1]));
+        store_act(vdst + lane + 32 * i, y[i]);
+      }
+    });
     return;
   }
   float ss = 0.0f;
@@ -151,31 +179,89 @@ __global__ void append_kernel(Attn a, int first, int count) {
 // weight of a query dimension: its own, and with shared rows the key's too
 template <bool SEP>
 __device__ __forceinline__ float query_weight(const Attn& a, int d) {
-  return a.q_norm == nullptr ? 1.0f : (SEP ? a.q_norm[d] : a.q_norm[d] * a.k_norm[d]);
+  return SEP ? a.q_norm[d] : a.q_norm[d] * a.k_norm[d];
 }
 
-// A warp normalises the query of head h and map m of a token (prow: its projections) and leaves q' * log2(e) in dst[0 .. KD - 1]
-// (columns past dim zero): scores are base-2 logarithms; with a cap, q' * 2 log2(e) / cap.
-template <int KD, bool SEP, int MAPS>
-__device__ __forceinline__ void load_query(const Attn& a, const float* prow, int h, int m, int pos, bf16* dst, int lane) {
-  const float2* rot = angles(a, pos);
-  const float* q = prow + a.q_col + (h * MAPS + m) * a.dim;
-  const float* qb = a.q_bias == nullptr ? nullptr : a.q_bias + (h * MAPS + m) * a.dim;
-  constexpr int N = (KD + 31) / 32;
-  float v[N], ss = 0.0f;
+// A warp normalises queries of a kv head and leaves q' * log2(e) in rows of dst (columns past dim zero): scores are base-2 logarithms; with
+// a cap, q' * 2 log2(e) / cap.  place(r) names row r's projections, head, map, position and destination; rows r0, r0 + step, ..
+// below r1, UN of them at a time.
+struct QueryRow {
+  const float* proj;
+  int head, map, pos;
+  bf16* dst;
+};
+template <int KD, bool SEP, int MAPS, int UN, typename P>
+__device__ __forceinline__ void load_queries(const Attn& a, int r0, int r1, int step, P place, int lane) {
+  with_flags<SEP, MAPS>(a.q_bias != nullptr, a.q_norm != nullptr, [&](auto bias, auto norm) {
+    constexpr bool BIAS = decltype(bias)::value, NORM = decltype(norm)::value;
+    constexpr int N = (KD + 31) / 32;
+    for (int r = r0; r < r1; r += UN * step) {
+      float v[UN][N], ss[UN];
 #pragma unroll
-  for (int i = 0; i < N; ++i) {
-    const int d = lane + 32 * i;
-    const bool in = d < KD && d < a.dim;
-    const float raw = in ? biased(q, qb, d) : 0.0f;
-    v[i] = in ? rotated([&](int j) { return biased(q, qb, j) * query_weight<SEP>(a, j); }, d, rot, a.rot_dims, a.rot_pairs) : 0.0f;
-    ss += raw * raw;
+      for (int u = 0; u < UN; ++u) {
+        const QueryRow row = place(min(r + u * step, r1 - 1));
+        const float2* rot = angles(a, row.pos);
+        const float* q = row.proj + a.q_col + (row.head * MAPS + row.map) * a.dim;
+        const float* qb = a.q_bias + (row.head * MAPS + row.map) * a.dim;
+        auto raw = [&](int j) { return BIAS ? q[j] + qb[j] : q[j]; };
+        ss[u] = 0.0f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          const int d = lane + 32 * i;
+          float x = 0.0f;
+          v[u][i] = 0.0f;
+          if (d < KD && d < a.dim) {
+            x = raw(d);
+            v[u][i] = rotated([&](int j) { return NORM ? raw(j) * query_weight<SEP>(a, j) : raw(j); }, d, rot, a.rot_dims, a.rot_pairs);
+          }
+          ss[u] += x * x;
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < UN; ++u) {
+        if (r + u * step >= r1) break;
+        const QueryRow row = place(r + u * step);
+        const float f = a.scale * temperature(a, row.pos) * (a.softcap > 0.0f ? 2.0f * kLog2e / a.softcap : kLog2e) /
+                        (a.normed ? sqrtf(warp_sum(ss[u]) / (float)a.dim + a.eps) : 1.0f);
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+          if (KD % 32 == 0 || lane + 32 * i < KD) row.dst[lane + 32 * i] = __float2bfloat16_rn(v[u][i] * f);
+      }
+    }
+  });
+}
+
+// Row r (0 or 1) of a thread's accumulators times f and the gates of its head: out[t] for columns nt * 8 + 2 (lane & 3) and the next.
+template <int HD>
+__device__ __forceinline__ void store_row(const Attn& a, const float (&o)[HD / 8][4], int r, float f, size_t t, int head, int lane) {
+  bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + head * a.vdim + (lane & 3) * 2;
+  const bool pairs = ((a.vdim | a.ldo | (int)(reinterpret_cast<uintptr_t>(a.out) >> 1)) & 1) == 0;
+  const int left = a.vdim - (lane & 3) * 2;
+  auto store = [&](int nt, float x, float y) {
+    if (pairs) {
+      if (nt * 8 < left) *reinterpret_cast<uint32_t*>(dst + nt * 8) = pack_bf16(x, y);
+    } else {
+      if (nt * 8 < left) dst[nt * 8] = __float2bfloat16_rn(x);
+      if (nt * 8 + 1 < left) dst[nt * 8 + 1] = __float2bfloat16_rn(y);
+    }
+  };
+  if (!a.gate_wide) {
+#pragma unroll
+    for (int nt = 0; nt < HD / 8; ++nt) store(nt, o[nt][2 * r] * f, o[nt][2 * r + 1] * f);
+    return;
   }
-  ss = warp_sum(ss);
-  const float f = a.scale * temperature(a, pos) * (a.softcap > 0.0f ? 2.0f * kLog2e / a.softcap : kLog2e) / (a.normed ? sqrtf(ss / (float)a.dim + a.eps) : 1.0f);
+  const float* g = a.proj + t * a.ld + a.g_col + head * a.vdim + (lane & 3) * 2;
 #pragma unroll
-  for (int i = 0; i < N; ++i)
-    if (KD % 32 == 0 || lane + 32 * i < KD) dst[lane + 32 * i] = __float2bfloat16_rn(v[i] * f);
+  for (int n0 = 0; n0 < HD / 8; n0 += 4) {
+    float gv[4][2];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      gv[i][0] = (n0 + i) * 8 < left ? g[(n0 + i) * 8] : 0.0f;
+      gv[i][1] = (n0 + i) * 8 + 1 < left ? g[(n0 + i) * 8 + 1] : 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) store(n0 + i, o[n0 + i][2 * r] * f * sigmoid(gv[i][0]), o[n0 + i][2 * r + 1] * f * sigmoid(gv[i][1]));
+  }
 }
 
 // ---- portions of prompts ------------------------------------------------------------------------------------------------------
@@ -223,13 +309,12 @@ __global__ void __launch_bounds__(128 * MAPS) prompt_kernel(Attn a, const int4* 
   int kb = next(-64);
   fetch(kb, 0);
   cp_async_commit();
-  for (int r = warp * 16; r < warp * 16 + 16; ++r) {     // a warp loads its own rows and map
-    if (r < rows) {
-      load_query<KD, SEP, MAPS>(a, a.proj + (size_t)(en.x + q0 + r / G) * a.ld, kvh * G + r % G, map, pfirst + r / G, sQ + r * LD + map * KD, lane);
-    } else {
-      for (int d = lane; d < KD; d += 32) sQ[r * LD + map * KD + d] = __float2bfloat16_rn(0.0f);
-    }
-  }
+  const int r0 = warp * 16, r1 = min(rows, r0 + 16);     // a warp loads its own rows and map
+  load_queries<KD, SEP, MAPS, 4>(a, r0, r1, 1, [&](int r) {
+    return QueryRow{a.proj + (size_t)(en.x + q0 + r / G) * a.ld, kvh * G + r % G, map, pfirst + r / G, sQ + r * LD + map * KD};
+  }, lane);
+  for (int r = max(r0, r1); r < r0 + 16; ++r)
+    for (int d = lane; d < KD; d += 32) sQ[r * LD + map * KD + d] = __float2bfloat16_rn(0.0f);
   __syncwarp();
   uint32_t qf[kQReg ? KD / 16 : 1][4];
   if (kQReg) {
@@ -367,14 +452,7 @@ __global__ void __launch_bounds__(128 * MAPS) prompt_kernel(Attn a, const int4* 
       ss += __shfl_xor_sync(0xffffffffu, ss, 2);
       if (!live) continue;
       const size_t t = en.x + q0 + row[r] / G;
-      const float g = a.diff_scale * gate(a, t, head[r]) / sqrtf(ss / (float)a.vdim + a.eps);
-      bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + head[r] * a.vdim;
-#pragma unroll
-      for (int nt = 0; nt < HD / 8; ++nt) {
-        const int d = nt * 8 + (lane & 3) * 2;
-        if (d < a.vdim) dst[d] = __float2bfloat16_rn(o[nt][2 * r] * g * wide_gate(a, t, head[r], d));
-        if (d + 1 < a.vdim) dst[d + 1] = __float2bfloat16_rn(o[nt][2 * r + 1] * g * wide_gate(a, t, head[r], d + 1));
-      }
+      store_row<HD>(a, o, r, a.diff_scale * gate(a, t, head[r]) / sqrtf(ss / (float)a.vdim + a.eps), t, head[r], lane);
     }
     return;
   }
@@ -391,13 +469,7 @@ __global__ void __launch_bounds__(128 * MAPS) prompt_kernel(Attn a, const int4* 
       const float sink = a.sinks[head[r]] * kLog2e, top = fmaxf(mx[r], sink), down = ex2(mx[r] - top);
       f *= down / (l[r] * down + ex2(sink - top));
     }
-    bf16* dst = static_cast<bf16*>(a.out) + t * a.ldo + head[r] * a.vdim;
-#pragma unroll
-    for (int nt = 0; nt < HD / 8; ++nt) {
-      const int d = nt * 8 + (lane & 3) * 2;
-      if (d < a.vdim) dst[d] = __float2bfloat16_rn(o[nt][2 * r] * f * wide_gate(a, t, head[r], d));
-      if (d + 1 < a.vdim) dst[d + 1] = __float2bfloat16_rn(o[nt][2 * r + 1] * f * wide_gate(a, t, head[r], d + 1));
-    }
+    store_row<HD>(a, o, r, f, t, head[r], lane);
   }
 }
 
@@ -465,18 +537,16 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
   pdl_wait();
   pdl_trigger();
   const float* prow = a.proj + (size_t)t * a.ld;
-  for (int r = warp; r < 16 + (owner ? 1 : 0); r += NW) {
-    if (r < nh) {
-      const int m = (h0 + r) % MAPS;
-      load_query<KD, SEP, MAPS>(a, prow, head_of(r), m, pos, sQ + r * LD + m * KD, lane);
-      if (MAPS == 2)
-        for (int d = lane; d < KD; d += 32) sQ[r * LD + (1 - m) * KD + d] = __float2bfloat16_rn(0.0f);
-    } else if (r < 16)
-      for (int d = lane; d < HD; d += 32) sQ[r * LD + d] = __float2bfloat16_rn(0.0f);
-    else {
-      append_row<HD, SEP, MAPS, bf16>(a, prow, kvh, pos, cache_row(a, bt, kvh, pos), lane);
-      __threadfence();
-    }
+  load_queries<KD, SEP, MAPS, 16 / NW>(a, warp, nh, NW, [&](int r) {
+    const int m = (h0 + r) % MAPS;
+    return QueryRow{prow, head_of(r), m, pos, sQ + r * LD + m * KD};
+  }, lane);
+  for (int r = warp; r < 16; r += NW)
+    for (int d = lane; d < HD; d += 32)
+      if (r >= nh || (MAPS == 2 && d / KD != (h0 + r) % MAPS)) sQ[r * LD + d] = __float2bfloat16_rn(0.0f);
+  if (owner && warp == NW - 1) {
+    append_row<HD, SEP, MAPS, bf16>(a, prow, kvh, pos, cache_row(a, bt, kvh, pos), lane);
+    __threadfence();
   }
   __syncthreads();
   float o[HD / 8][4];
@@ -492,6 +562,13 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
   for (int st = 0; st < NST - 1; ++st) {
     if (j0 + st * NW < b1 && is_new(j0 + st * NW)) issue(j0 + st * NW, st);
     cp_async_commit();
+  }
+  float ahead[MAPS == 2 ? HD / 32 : 1];       // two maps: the gates of this warp's head
+  if (MAPS == 2) {
+    const int hh = split * NW + warp;
+#pragma unroll
+    for (int i = 0; i < HD / 32; ++i)
+      ahead[MAPS == 2 ? i : 0] = hh < nh / 2 && lane + 32 * i < a.vdim ? wide_gate(a, t, head_of(2 * hh), lane + 32 * i) : 1.0f;
   }
   constexpr bool kQReg = HD <= 128;
   uint32_t qf[kQReg ? HD / 16 : 1][4];
@@ -585,23 +662,33 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
     }
   }
   __syncthreads();
+  // the warps' factors, once per row
+  float own = -INFINITY, most, sum = 0.0f;
+  const int fr = threadIdx.x / NW, fw = threadIdx.x % NW;
+  static_assert(16 * NW <= NTH && (NW & (NW - 1)) == 0 && NW <= 32, "a thread per row and warp");
+  if (fr < nh) own = part[(fw * 16 + fr) * ST + HD];
+  most = own;
+#pragma unroll
+  for (int o = NW / 2; o > 0; o >>= 1) most = fmaxf(most, __shfl_xor_sync(0xffffffffu, most, o));
+  if (fr < nh) {
+    const float f = own == -INFINITY ? 0.0f : ex2(own - most);
+    float* src = part + (fw * 16 + fr) * ST;
+    src[HD] = f;
+    sum = f * src[HD + 1];
+  }
+#pragma unroll
+  for (int o = NW / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  if (fr < nh && fw == 0) {
+    res[fr * ST + HD] = most;
+    res[fr * ST + HD + 1] = sum;
+  }
+  __syncthreads();
   for (int i = threadIdx.x; i < nh * HD; i += NTH) {
     const int r = i / HD, d = i % HD;
-    float M = -INFINITY, acc = 0.0f, L = 0.0f;
+    float acc = 0.0f;
 #pragma unroll
-    for (int w = 0; w < NW; ++w) M = fmaxf(M, part[(w * 16 + r) * ST + HD]);
-#pragma unroll
-    for (int w = 0; w < NW; ++w) {
-      const float* src = part + (w * 16 + r) * ST;
-      const float f = src[HD] == -INFINITY ? 0.0f : ex2(src[HD] - M);
-      acc += f * src[d];
-      L += f * src[HD + 1];
-    }
+    for (int w = 0; w < NW; ++w) acc = fmaf(part[(w * 16 + r) * ST + HD], part[(w * 16 + r) * ST + d], acc);
     res[r * ST + d] = acc;
-    if (d == 0) {
-      res[r * ST + HD] = M;
-      res[r * ST + HD + 1] = L;
-    }
   }
   if (nsplit > 1) cluster.sync();
   else __syncthreads();
@@ -642,7 +729,7 @@ __global__ void __launch_bounds__(32 * decode_warps(HD, SEP)) decode_kernel(Attn
 #pragma unroll
       for (int i = 0; i < HD / 32; ++i) {
         const int d = lane + 32 * i;
-        if (d < a.vdim) static_cast<bf16*>(a.out)[(size_t)t * a.ldo + h * a.vdim + d] = __float2bfloat16_rn(o2[i] * g2 * wide_gate(a, t, h, d));
+        if (d < a.vdim) static_cast<bf16*>(a.out)[(size_t)t * a.ldo + h * a.vdim + d] = __float2bfloat16_rn(o2[i] * g2 * (hh == split * NW + warp ? ahead[MAPS == 2 ? i : 0] : wide_gate(a, t, h, d)));
       }
     }
     if (nsplit > 1) cluster.sync();
@@ -697,7 +784,7 @@ __global__ void __launch_bounds__(128) f32_kernel(Attn a) {
       const int d = lane + 32 * i;
       const bool in = d < KD && d < a.dim;
       const float raw = in ? biased(qr, qb, d) : 0.0f;
-      q[i] = in ? rotated([&](int j) { return biased(qr, qb, j) * query_weight<SEP>(a, j); }, d, rot, a.rot_dims, a.rot_pairs) : 0.0f;
+      q[i] = in ? rotated([&](int j) { return biased(qr, qb, j) * (a.q_norm == nullptr ? 1.0f : query_weight<SEP>(a, j)); }, d, rot, a.rot_dims, a.rot_pairs) : 0.0f;
       ss += raw * raw;
     }
 #pragma unroll
@@ -814,7 +901,8 @@ static bool fill(Attn& a, const void* const* ptrs, const int* ints, const float*
                               a.q_bias != nullptr || a.k_bias != nullptr || a.v_bias != nullptr
                         : a.vdim < 1) return false;
   if (a.rot != nullptr && (a.rot_dims < 2 || a.rot_dims % 2 != 0 || a.rot_dims > a.dim)) return false;
-  if (a.maps != 1 && (a.maps != 2 || a.sinks != nullptr)) return false;
+  if (a.maps != 1 && (a.maps != 2 || a.sinks != nullptr || a.q_norm == nullptr || a.q_bias == nullptr)) return false;
+  if ((a.q_bias == nullptr) != (a.v_bias == nullptr) || (a.k_col >= 0 && (a.q_bias == nullptr) != (a.k_bias == nullptr))) return false;
   if (a.window > 0 && a.chunk > 0) return false;
   return a.heads >= 1 && a.kv_heads >= 1 && a.heads % a.kv_heads == 0 && a.heads / a.kv_heads <= 64 && a.dim >= 1 &&
          row_dim(a) > 0 && a.pshift >= 4 && (1 << a.pshift) == ints[11] && a.keep >= 0 &&
@@ -850,7 +938,7 @@ extern "C" {
 int bonsai_lay_attn_row(int dim) { return dim < 1 ? 0 : bonsai::lay::padded_dim(dim); }
 
 // Arguments of all launches: ptrs = {proj, q_norm, k_norm, slopes, pos, slots, block_table, pool, krms, vpool, out, sinks, rot, q_bias,
-// k_bias, v_bias} (null where a design has none; vpool null: rows are key and value; rot has a row for every position the pages
+// k_bias, v_bias} (null where a design has none, the biases together; two maps have biases and norm weights; vpool null: rows are key and value; rot has a row for every position the pages
 // hold), ints = {ld, q_col, k_col, v_col, g_col, ldo, heads, kv_heads, dim, vdim, max_pages, page_size, window, keep, normed, rot_dims,
 // rot_pairs, chunk, maps, gate_wide}, floats = {eps, scale, out_scale, softcap, temp_coef, temp_every, lambda, diff_scale}.
 

@@ -409,10 +409,15 @@ class AttentionMixer:
         ints = [r.proj.stride(0), cols["q"], cols.get("k", -1), cols.get("v", 0), cols.get("g", -1), out.stride(0), spec.heads, spec.kv_heads, spec.dim,
                 spec.value_dim, r.max_pages, r.kv.page_size, spec.window, spec.keep_first, int(spec.normed), 0 if rot is None else rot.dims,
                 int(rot is not None and rot.interleaved), spec.chunk, spec.maps, int(spec.element_gate)]
-        vec, lam, left = w.vectors, 0.0, 1.0
+        vec, lam, left = dict(w.vectors), 0.0, 1.0
         if spec.difference is not None:
             dot = lambda i: float(torch.exp((vec[f"lq{i}"].double() * vec[f"lk{i}"].double()).sum()))
             lam, left = dot(1) - dot(2) + spec.difference, 1.0 - spec.difference
+            for n, rows in spec.sections:                    # the kernels have both here
+                if n != "g" and not spec.biases:
+                    vec[n + ".b"] = torch.zeros(rows, dtype=torch.float32, device=r.device)
+            if not spec.norm_weights:
+                vec["q.norm"] = vec["k.norm"] = torch.ones(spec.dim, dtype=torch.float32, device=r.device)
         floats = [r.cfg.eps, spec.scale, branch.scale, spec.softcap, spec.temp_coef, spec.temp_every, lam, left]
         self.call = {id(rows): L.MixerCall([r.proj, vec.get("q.norm"), vec.get("k.norm"), slopes, rows.positions, rows.slots, r.block_table,
                                             r.kv.rows[source], r.kv.factors.get(source), r.kv.values.get(source), out, vec.get("sink"),
