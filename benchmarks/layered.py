@@ -680,13 +680,13 @@ def bench_scans(rep: Report, width: int, iters: int, profile: bool) -> None:
         rows, n = BenchRows(nseq, T), nseq * T
         copies = 1 + int(300e6 / (14.0 * n * W))
         cluster, ctas = 1, nseq * -(-W // 32)
-        while cluster < 8 and 2 * cluster * ctas <= 2 * sms and 2 * cluster * lib.bonsai_lay_gru_tokens() <= T:
+        while cluster < 8 and 2 * cluster * ctas <= 4 * sms and 2 * cluster * lib.bonsai_lay_gru_tokens() <= T:
             cluster *= 2
         fn = lambda a: K.check(lib.bonsai_lay_gru_scan(*a, rows.shape.entries, nseq, cluster, 0, K.stream()), "gru_scan")
         rep.add("gru_scan", f"{nseq} x {T} tokens width={W} cluster={cluster}", time_us(turn([gru(rows) for _ in range(copies)], fn), 10, profile), 14.0 * n * W)
         plan = SegmentPlan(-(-inner // lib.bonsai_lay_scan_channels(N)), SCAN_COST)
         size = plan_segments([T] * nseq, plan, sms) * CHUNK
-        for size in sorted({0, size, 1024, 512}):
+        for size in sorted({0, size}):
             if size and nseq * -(-T // size) > MAX_SEGMENTS or size >= T:
                 continue
             segs = [(s * T + x, min(size, T - x), s, int(x + size >= T)) for s in range(nseq) for x in range(0, T, size)] if size else []

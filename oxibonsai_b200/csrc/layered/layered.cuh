@@ -72,6 +72,27 @@ __device__ __forceinline__ float ex2(float x) {
 }
 __device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 
+constexpr float kLog2e = 1.4426950408889634f;
+
+// The same with the approximate exponential and division (some 2^-22 of the result), for kernels that would wait for the accurate ones.
+template <bool EXACT>
+__device__ __forceinline__ float sigmoid_as(float x) {
+  return EXACT ? sigmoid(x) : __fdividef(1.0f, 1.0f + ex2(-x * kLog2e));
+}
+template <bool EXACT>
+__device__ __forceinline__ float silu_as(float x) {
+  return x * sigmoid_as<EXACT>(x);
+}
+// max(x, 0) + log(1 + e) with e = exp(-|x|); the approximate form sums the series of log(1 + e) where e is small, so that small results
+// keep their digits
+template <bool EXACT>
+__device__ __forceinline__ float softplus_as(float x) {
+  if (EXACT) return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x)));
+  const float e = ex2(-fabsf(x) * kLog2e);
+  const float series = e * (1.0f - e * (1.0f / 2 - e * (1.0f / 3 - e * (1.0f / 4 - e * (1.0f / 5 - e * (1.0f / 6))))));
+  return fmaxf(x, 0.0f) + (e < 0.0625f ? series : __logf(1.0f + e));
+}
+
 __device__ __forceinline__ void store_act(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 __device__ __forceinline__ void store_act(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_act4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
@@ -105,8 +126,6 @@ __device__ __forceinline__ float glu(const Glu& a, float g, float u) {
   u = fminf(fmaxf(u, -a.limit), a.limit);
   return g * sigmoid(a.alpha * fmaf(a.cubic * g * g, g, g)) * (u + a.up_offset);
 }
-
-constexpr float kLog2e = 1.4426950408889634f;
 
 // chunked recurrences: tokens per chunk, value columns per CTA, row length of a staged value tile
 constexpr int kL = 64;

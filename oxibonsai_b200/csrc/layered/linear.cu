@@ -1,16 +1,19 @@
 // Projections with dense bf16 weights: out[t][n] = sum_k x[t][k] W[n][k].
 //
-// `few_rows_kernel` serves decode batches and short portions (up to 32 rows): the weights are streamed once, a warp's lane
+// `few_rows_kernel` serves decode batches and short portions (up to 64 rows): the weights are streamed once, a warp's lane
 // loads 16 contiguous bytes of a weight row and uses them directly as `mma.sync.m16n8k16` A registers.  That is the
 // fragment layout up to a permutation of k inside every 32 inputs, and the activations are loaded through the same
 // permutation (16 contiguous bytes of an activation row as the B registers), so neither operand passes through shared
-// memory.  The eight warps of a CTA split K and meet in shared memory once.  More rows go to the tcgen05 GEMM
+// memory.  The eight warps of a CTA split K and meet in shared memory once; matrices of few rows are split further, over the CTAs of a
+// cluster, which meet in distributed shared memory.  More activation rows go to the tcgen05 GEMM
 // (cuda/bitgemm_prefill.cu, dense bf16 operands).
 //
 // `f32_kernel` is the 32-bit mode: f32 activations, the same bf16 weights (exact in f32), f32 FMA throughout.
 //
 // Epilogues: 0 = f32 store, 1 = clamped gated unit over interleaved gate / up rows, 2 = squared relu, 3 = the product itself in the
 // activations' type, 4 = f32 store of limit * tanh(product / limit).
+#include <cooperative_groups.h>
+
 #include "layered/layered.cuh"
 
 namespace bonsai {
@@ -26,16 +29,19 @@ __device__ __forceinline__ float capped(float v, int epi, const Glu& a) { return
 
 constexpr int kWarps = 8;
 
-template <int NT>   // 8-row groups of activations
+// NT: 8-row groups of activations; grid (16 weight rows, CTAs that split K, a cluster)
+template <int NT, bool SPLIT>
 __global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __restrict__ W, int n, int kp, const bf16* x, int ldx, int T,
                                                               float* out, bf16* out16, int ldo, int epi, Glu act) {
   constexpr int LD = 8 * NT + 1;
   __shared__ float red[kWarps][16][LD];
+  namespace cg = cooperative_groups;
+  cg::cluster_group cluster = cg::this_cluster();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t4 = lane & 3;
-  const int row0 = blockIdx.x * 16;
+  const int row0 = blockIdx.x * 16, split = SPLIT ? gridDim.y : 1, rank = SPLIT ? blockIdx.y : 0;
   const bf16* w0 = W + (size_t)min(row0 + g, n - 1) * kp + 8 * t4;
   const bf16* w1 = W + (size_t)min(row0 + g + 8, n - 1) * kp + 8 * t4;
-  const int chunks = kp >> 7;   // 128 inputs each
+  const int chunks = kp >> 7, first = rank * kWarps + warp, step = split * kWarps;   // 128 inputs each
   uint4 a[4], b[4];
   auto load_w = [&](int c) {
 #pragma unroll
@@ -44,7 +50,7 @@ __global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __res
       b[i] = __ldcs(reinterpret_cast<const uint4*>(w1 + c * 128 + i * 32));
     }
   };
-  if (warp < chunks) load_w(warp);   // weights depend on no earlier kernel
+  if (first < chunks) load_w(first);   // weights depend on no earlier kernel
   pdl_wait();
   pdl_trigger();
   const bf16* xr[NT];
@@ -53,7 +59,7 @@ __global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __res
   float acc[NT][4];
 #pragma unroll
   for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
-  for (int c = warp; c < chunks; c += kWarps) {
+  for (int c = first; c < chunks; c += step) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const uint32_t lo[4] = {a[i].x, b[i].x, a[i].y, b[i].y}, hi[4] = {a[i].z, b[i].z, a[i].w, b[i].w};
@@ -64,7 +70,7 @@ __global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __res
         mma_bf16(acc[j], hi, v.z, v.w);
       }
     }
-    if (c + kWarps < chunks) load_w(c + kWarps);
+    if (c + step < chunks) load_w(c + step);
   }
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
@@ -74,28 +80,50 @@ __global__ void __launch_bounds__(kWarps * 32) few_rows_kernel(const bf16* __res
     red[warp][g + 8][8 * j + 2 * t4 + 1] = acc[j][3];
   }
   __syncthreads();
-  if (epi != 1) {
-    for (int i = threadIdx.x; i < 16 * T; i += kWarps * 32) {
-      const int r = i & 15, t = i >> 4;
-      float v = 0.0f;
+  auto warps_sum = [&](int r, int t) {
+    float v = 0.0f;
 #pragma unroll
-      for (int w = 0; w < kWarps; ++w) v += red[w][r][t];
+    for (int w = 0; w < kWarps; ++w) v += red[w][r][t];
+    return v;
+  };
+  if constexpr (SPLIT) {               // this CTA's sums, where the others find them
+    constexpr int PER = 16 * 8 * NT / (kWarps * 32) > 0 ? 16 * 8 * NT / (kWarps * 32) : 1;
+    float own[PER];
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+      const int i = threadIdx.x + p * kWarps * 32;
+      own[p] = i < 16 * T ? warps_sum(i & 15, i >> 4) : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+      const int i = threadIdx.x + p * kWarps * 32;
+      if (i < 16 * T) red[0][i & 15][i >> 4] = own[p];
+    }
+    cluster.sync();
+  }
+  auto total = [&](int r, int t) {
+    if (!SPLIT) return warps_sum(r, t);
+    float v = 0.0f;
+    for (int s = 0; s < split; ++s) v += *cluster.map_shared_rank(&red[0][r][t], s);
+    return v;
+  };
+  if (epi != 1) {
+    for (int i = rank * kWarps * 32 + threadIdx.x; i < 16 * T; i += step * 32) {
+      const int r = i & 15, t = i >> 4;
+      const float v = total(r, t);
       if (row0 + r >= n) continue;
       if (epi == 0 || epi == 4) out[(size_t)t * ldo + row0 + r] = capped(v, epi, act);
       else out16[(size_t)t * ldo + row0 + r] = __float2bfloat16_rn(epi == 2 ? squared_relu(v) : v);
     }
   } else {
-    for (int i = threadIdx.x; i < 8 * T; i += kWarps * 32) {
+    for (int i = rank * kWarps * 32 + threadIdx.x; i < 8 * T; i += step * 32) {
       const int r = i & 7, t = i >> 3;
-      float gv = 0.0f, uv = 0.0f;
-#pragma unroll
-      for (int w = 0; w < kWarps; ++w) {
-        gv += red[w][2 * r][t];
-        uv += red[w][2 * r + 1][t];
-      }
+      const float gv = total(2 * r, t), uv = total(2 * r + 1, t);
       if (row0 + 2 * r + 1 < n) out16[(size_t)t * ldo + (row0 >> 1) + r] = __float2bfloat16_rn(glu(act, gv, uv));
     }
   }
+  if (SPLIT) cluster.sync();           // nobody leaves while its sums are being read
 }
 
 // 64 weight rows x 64 activation rows per CTA, 256 threads with 4 x 4 outputs each
@@ -153,18 +181,24 @@ __global__ void __launch_bounds__(256) f32_kernel(const bf16* __restrict__ W, in
 extern "C" {
 
 // W bf16 [n][kp] (kp a multiple of 128, columns past the layer's width zero), x bf16 [T][ldx] (ldx >= kp, finite in the
-// padding), T <= 32.  epi 0 and 4: out f32 [T][ldo]; epi 1: out16 bf16 [T][ldo] of n / 2 columns; epi 2 and 3: out16 bf16 [T][ldo].
+// padding), T <= 64.  epi 0 and 4: out f32 [T][ldo]; epi 1: out16 bf16 [T][ldo] of n / 2 columns; epi 2 and 3: out16 bf16 [T][ldo].
 int bonsai_lay_linear_few(const void* W, int n, int kp, const void* x, int ldx, int T, float* out, void* out16, int ldo, int epi, float limit,
                           float alpha, float up_offset, float cubic, cudaStream_t stream) {
   using namespace bonsai::lay;
-  if (n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || T < 1 || T > 32 || epi < 0 || epi > 4) return BONSAI_CUDA_BAD_ARG;
+  if (n < 1 || kp < 128 || kp % 128 != 0 || ldx < kp || ldx % 8 != 0 || T < 1 || T > 64 || epi < 0 || epi > 4) return BONSAI_CUDA_BAD_ARG;
   const bool f32_out = epi == 0 || epi == 4;
   if ((f32_out && out == nullptr) || (!f32_out && out16 == nullptr) || (epi == 4 && !(limit > 0.0f)) || (epi == 1 && n % 2 != 0)) return BONSAI_CUDA_BAD_ARG;
   const Glu act{limit, alpha, up_offset, cubic};
-  const dim3 grid((n + 15) / 16);
-#define BONSAI_FEW(NT) \
-  launch(few_rows_kernel<NT>, grid, kWarps * 32, 0, stream, 1, 0, (const bf16*)W, n, kp, (const bf16*)x, ldx, T, out, (bf16*)out16, ldo, epi, act)
-  return T <= 8 ? BONSAI_FEW(1) : (T <= 16 ? BONSAI_FEW(2) : BONSAI_FEW(4));
+  // few CTAs: K is split until they cover the GPU, or a warp has one chunk
+  int split = 1;
+  while (split < 8 && (n + 15) / 16 * split * 2 <= 148 && split * 2 * kWarps <= kp / 128) split *= 2;
+  const dim3 grid((n + 15) / 16, split);
+#define BONSAI_FEW(NT)                                                                                                                                  \
+  (split > 1 ? launch(few_rows_kernel<NT, true>, grid, kWarps * 32, 0, stream, split, 1, (const bf16*)W, n, kp, (const bf16*)x, ldx, T, out,            \
+                      (bf16*)out16, ldo, epi, act)                                                                                                      \
+             : launch(few_rows_kernel<NT, false>, grid, kWarps * 32, 0, stream, 1, 0, (const bf16*)W, n, kp, (const bf16*)x, ldx, T, out, (bf16*)out16, \
+                      ldo, epi, act))
+  return T <= 8 ? BONSAI_FEW(1) : (T <= 16 ? BONSAI_FEW(2) : (T <= 32 ? BONSAI_FEW(4) : BONSAI_FEW(8)));
 #undef BONSAI_FEW
 }
 

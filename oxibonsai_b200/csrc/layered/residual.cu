@@ -48,7 +48,7 @@ struct RowStep {
 
 // KEEP chunks of VEC columns per thread, tg = 2^tshift threads per group
 template <int VEC, int KEEP, bool CONV>
-__global__ void __launch_bounds__(KEEP * VEC > 8 ? 1024 : 512) row_step_kernel(RowStep a, int tshift) {
+__global__ void __launch_bounds__(KEEP * VEC > 8 ? 1024 : 512, KEEP * VEC > 8 || CONV ? 1 : 3) row_step_kernel(RowStep a, int tshift) {
   __shared__ float sums[2][32];
   const int tg = 1 << tshift, grp = threadIdx.x >> tshift, l = threadIdx.x & (tg - 1), gw = a.width / a.groups;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -94,6 +94,7 @@ __global__ void __launch_bounds__(KEEP * VEC > 8 ? 1024 : 512) row_step_kernel(R
     }
     return 1.0f / sqrtf(ss / (float)gw + a.eps);
   };
+  constexpr bool kEarly = KEEP * VEC <= 8;         // registers for weights ahead of the sums they follow
   // inputs of earlier tokens, older than the kernel before this one unless this is a step's first
   constexpr int kBack = CONV && KEEP * VEC <= 8 ? 3 : 0;
   float back[KEEP][kBack > 0 ? kBack : 1][VEC];
@@ -118,75 +119,105 @@ __global__ void __launch_bounds__(KEEP * VEC > 8 ? 1024 : 512) row_step_kernel(R
   pdl_trigger();
   if (t == 0 && a.counts != nullptr)
     for (int i = threadIdx.x; i < a.experts; i += blockDim.x) a.counts[i] = 0;
+  // columns that are off read column 0 and count as zero: no branch stands between the loads
+  auto off = [&](int i, float (&v)[VEC]) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = on[i] ? v[e] : 0.0f;
+  };
   float x[KEEP][VEC];
   float* xr = a.x + (size_t)row * a.width;
+  if (!a.fresh) {
 #pragma unroll
-  for (int i = 0; i < KEEP; ++i) {
+    for (int i = 0; i < KEEP; ++i) load(xr + col[i], x[i]);
+  } else {
 #pragma unroll
-    for (int v = 0; v < VEC; ++v) x[i][v] = 0.0f;
-    if (on[i] && !a.fresh) load(xr + col[i], x[i]);
+    for (int i = 0; i < KEEP; ++i)
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) x[i][v] = 0.0f;
   }
   if (a.y != nullptr || a.top > 0) {
-    float u[KEEP][VEC], ss = 0.0f;
-    const float g = a.y_gate == nullptr ? 1.0f : sigmoid(a.y_gate[(size_t)t * a.ldg]);
+    float u[KEEP][VEC], w[kEarly ? KEEP : 1][VEC], ss = 0.0f;
+    if (a.y != nullptr) {
+      const float* yr = a.y + (size_t)t * a.ldy;
 #pragma unroll
-    for (int i = 0; i < KEEP; ++i) {
-#pragma unroll
-      for (int v = 0; v < VEC; ++v) u[i][v] = 0.0f;
-      if (!on[i]) continue;
-      if (a.y != nullptr) load(a.y + (size_t)t * a.ldy + col[i], u[i]);
+      for (int i = 0; i < KEEP; ++i) load(yr + col[i], u[i]);
       if (a.y_bias != nullptr) {
-        float b[VEC];
-        load(a.y_bias + col[i], b);
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) u[i][v] += b[v];
+        for (int i = 0; i < KEEP; ++i) {
+          float b[VEC];
+          load(a.y_bias + col[i], b);
+#pragma unroll
+          for (int v = 0; v < VEC; ++v) u[i][v] += b[v];
+        }
       }
+      if (a.y_gate != nullptr) {
+        const float g = sigmoid(a.y_gate[(size_t)t * a.ldg]);
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) u[i][v] *= g;
+        for (int i = 0; i < KEEP; ++i)
+#pragma unroll
+          for (int v = 0; v < VEC; ++v) u[i][v] *= g;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i)
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) u[i][v] = 0.0f;
     }
-    for (int k = 0; k < a.top; ++k) {
+    auto add_expert = [&](int k, auto load_row) {
       const size_t er = (size_t)a.at[t * a.top + k] * a.lde;
 #pragma unroll
       for (int i = 0; i < KEEP; ++i) {
-        if (!on[i]) continue;
         float b[VEC];
-        if (a.e_f32) load(static_cast<const float*>(a.e) + er + col[i], b);
-        else load16(static_cast<const bf16*>(a.e) + er + col[i], b);
+        load_row(er + col[i], b);
 #pragma unroll
         for (int v = 0; v < VEC; ++v) u[i][v] += b[v];
       }
+    };
+    if (a.e_f32) {
+#pragma unroll(kEarly ? 2 : 1)
+      for (int k = 0; k < a.top; ++k) add_expert(k, [&](size_t at, float (&b)[VEC]) { load(static_cast<const float*>(a.e) + at, b); });
+    } else {
+#pragma unroll(kEarly ? 4 : 1)
+      for (int k = 0; k < a.top; ++k) add_expert(k, [&](size_t at, float (&b)[VEC]) { load16(static_cast<const bf16*>(a.e) + at, b); });
     }
     float f = a.mult;
     if (a.w != nullptr) {
 #pragma unroll
-      for (int i = 0; i < KEEP; ++i)
+      for (int i = 0; i < KEEP; ++i) {
+        if (kEarly) load(a.w + col[i], w[kEarly ? i : 0]);
+        off(i, u[i]);
 #pragma unroll
         for (int v = 0; v < VEC; ++v) ss += u[i][v] * u[i][v];
+      }
       f *= inverse(ss, sums[0]);
-    }
 #pragma unroll
-    for (int i = 0; i < KEEP; ++i) {
-      if (!on[i]) continue;
-      float w[VEC];
+      for (int i = 0; i < KEEP; ++i) {
+        if (!kEarly) load(a.w + col[i], w[0]);
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) w[v] = 1.0f;
-      if (a.w != nullptr) load(a.w + col[i], w);
+        for (int v = 0; v < VEC; ++v) x[i][v] = fmaf(u[i][v] * f, w[kEarly ? i : 0][v], x[i][v]);
+      }
+    } else {
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) x[i][v] = fmaf(u[i][v] * f, w[v], x[i][v]);
+      for (int i = 0; i < KEEP; ++i)
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) x[i][v] = fmaf(u[i][v], f, x[i][v]);
     }
   }
   if (a.table != nullptr || a.step != nullptr) {
     const bf16* tr = a.table == nullptr ? nullptr : a.table + (size_t)a.tokens[t] * a.ld_table;
+    if (tr != nullptr) {
 #pragma unroll
-    for (int i = 0; i < KEEP; ++i) {
-      if (!on[i]) continue;
-      float b[VEC];
-      if (tr != nullptr) {
+      for (int i = 0; i < KEEP; ++i) {
+        float b[VEC];
         load16(tr + col[i], b);
 #pragma unroll
         for (int v = 0; v < VEC; ++v) x[i][v] = fmaf(b[v], a.scale, x[i][v]);
       }
-      if (a.step != nullptr) {
+    }
+    if (a.step != nullptr) {
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {
+        float b[VEC];
         load(a.step + col[i], b);
 #pragma unroll
         for (int v = 0; v < VEC; ++v) x[i][v] += b[v];
@@ -200,19 +231,20 @@ __global__ void __launch_bounds__(KEEP * VEC > 8 ? 1024 : 512) row_step_kernel(R
   }
   if (a.h == nullptr) return;
   if (a.next != nullptr) {
-    float ss = 0.0f;
+    float ss = 0.0f, w[kEarly ? KEEP : 1][VEC];
 #pragma unroll
-    for (int i = 0; i < KEEP; ++i)
+    for (int i = 0; i < KEEP; ++i) {
+      if (kEarly) load(a.next + col[i], w[kEarly ? i : 0]);
+      off(i, x[i]);
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) ss += x[i][v] * x[i][v];        // columns that are off hold zeros
+      for (int v = 0; v < VEC; ++v) ss += x[i][v] * x[i][v];
+    }
     const float f = inverse(ss, sums[1]);
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
-      if (!on[i]) continue;
-      float w[VEC];
-      load(a.next + col[i], w);
+      if (!kEarly) load(a.next + col[i], w[0]);
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) x[i][v] *= f * w[v];
+      for (int v = 0; v < VEC; ++v) x[i][v] *= f * w[kEarly ? i : 0][v];
     }
   }
 #pragma unroll
@@ -311,7 +343,7 @@ __global__ void __launch_bounds__(128) conv_kernel(Conv a, int singles, const in
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
       if (a.add) y[e] += x[e];
-      if (a.silu) y[e] *= sigmoid(y[e]);
+      if (a.silu) y[e] = a.out_f32 ? silu_as<true>(y[e]) : silu_as<false>(y[e]);
     }
     const size_t at = (size_t)(first + q0 + i) * a.ldo + c;
     if constexpr (VEC == 4) {

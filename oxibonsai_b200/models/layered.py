@@ -350,8 +350,11 @@ class SegmentCost:
     fixed: float
     each: float             # per segment
     shortest: int           # chunks
+    share: float = 0.0      # > 0: CTAs share an SM evenly, and a chunk takes so long per CTA on it, but no less than alone
 
     def waves(self, ctas: int, sms: int) -> float:
+        if self.share > 0:
+            return max(1.0, self.share * ctas / sms)
         if self.resident > 1 and ctas <= 0.6 * sms:        # more of them do not spread evenly
             return 1.0
         return self.crowded * -(-ctas // (self.resident * sms))
@@ -363,7 +366,9 @@ class SegmentCost:
 MLSTM_COST = SegmentCost(1, 1.0, 1.5, 0.5, 0.6, 4)
 RECURRENCE_COST = SegmentCost(2, 1.55, 1.45, 2.0, 0.3, 2)
 WIDE_RECURRENCE_COST = SegmentCost(1, 1.0, 1.35, 1.2, 0.6, 2)
-SCAN_COST = SegmentCost(4, 1.0, 1.9, 2.0, 0.1, 2)
+# Selective scan, 16 states: 4096 tokens of 512 channels 252 us whole, 122 in 4 segments, 63 in 16; of 2048 channels 253, 209, 131; of 8192
+# channels 392 whole, 472 in 4.
+SCAN_COST = SegmentCost(8, 1.0, 1.68, 1.5, 0.4, 2, share=0.38)
 
 
 @dataclass(frozen=True)
@@ -613,9 +618,9 @@ class MinGruMixer:
                      for rows in (r.slot_rows, r.batch_rows)}
 
     def cluster(self, portions: int, tokens: int) -> int:
-        """CTAs that share a portion: about two per SM, and no more than have tokens in one round."""
+        """CTAs that share a portion: about four per SM, and no more than have tokens in one round."""
         n, ctas = 1, portions * -(-self.spec.width // 32)
-        while n < 8 and 2 * n * ctas <= 2 * self.r.scratch.sms and 2 * n * L.lib().bonsai_lay_gru_tokens() <= tokens:
+        while n < 8 and 2 * n * ctas <= 4 * self.r.scratch.sms and 2 * n * L.lib().bonsai_lay_gru_tokens() <= tokens:
             n *= 2
         return n
 

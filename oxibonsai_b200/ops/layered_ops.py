@@ -74,6 +74,7 @@ _SIG = {
 }
 _lib = None
 FEW_ROWS = 32               # rows up to which a projection goes to the weight-streaming kernel
+FEW_MORE = (64, 2368)       # and that, where the matrix has at most so many outputs (16 per SM)
 K_ALIGN = 128               # inputs of a bf16 projection are padded to a multiple of this
 
 
@@ -170,7 +171,7 @@ def linear(w: DenseWeight, x: torch.Tensor, T: int, out: torch.Tensor, scratch: 
         return
     assert x.dtype == torch.bfloat16 and (out.dtype == torch.float32 if epi in (0, 4) else out.dtype == torch.bfloat16)
     f32, b16 = (out.data_ptr(), None) if epi in (0, 4) else (None, out.data_ptr())
-    if T <= FEW_ROWS:
+    if T <= FEW_ROWS or (T <= FEW_MORE[0] and w.n <= FEW_MORE[1]):
         K.check(l.bonsai_lay_linear_few(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), epi, *glu.args, s), "linear_few")
     else:
         K.check(l.bonsai_dense_gemm_bf16(w.data.data_ptr(), w.n, w.kp, x.data_ptr(), x.stride(0), T, f32, b16, out.stride(0), (0, 4, 5, 6, 7)[epi], *glu.args,
