@@ -954,6 +954,7 @@ def main() -> None:
                      ("differential", bench_differential), ("scans", bench_scans), ("rows", bench_row_steps)):
         if name in a.only.split(","):
             fn(rep, a.width, a.iters, a.profile)
+            torch.cuda.empty_cache()             # buffers cut out of a former bench's blocks were slower to read by a quarter
 
 
 if __name__ == "__main__":
