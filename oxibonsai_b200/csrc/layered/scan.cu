@@ -80,12 +80,12 @@ __global__ void __launch_bounds__(32 * kGruWarps, 4) gru_scan_kernel(Gru a, cons
   pdl_trigger();
   const int4 en = entries[blockIdx.y];
   float* S = a.S + (size_t)a.state_rows[en.z] * a.width + c;
-  float state = on && en.w > 0 ? *S : 0.0f;                // of the tokens before this round's
+  float state = on && en.w > 0 ? *S : 0.0f;                // of the tokens ahead of these
   const float zb = on ? a.z_bias[c] : 0.0f, ub = on ? a.u_bias[c] : 0.0f;
   const float* base = a.proj + (size_t)en.x * a.ld + c;
-  const int per_round = ctas * kGruWarps * kGruTokens, mine = (rank * kGruWarps + warp) * kGruTokens;
+  const int per_turn = ctas * kGruWarps * kGruTokens, mine = (rank * kGruWarps + warp) * kGruTokens;
   int par = 0;
-  for (int r0 = 0; r0 < en.y; r0 += per_round, par ^= 1) {
+  for (int r0 = 0; r0 < en.y; r0 += per_turn, par ^= 1) {
     const int t0 = r0 + mine, n = on ? min(kGruTokens, en.y - t0) : 0;
     float keep[kGruTokens], add[kGruTokens], gate[kGruTokens];
 #pragma unroll
@@ -118,7 +118,7 @@ __global__ void __launch_bounds__(32 * kGruWarps, 4) gru_scan_kernel(Gru a, cons
         }
         whole[par][lane] = make_float2(A, B);
       }
-      cluster.sync();        // the other buffer is free again: everyone is past the reads of the round before the last
+      cluster.sync();        // the other buffer is free again: everyone is past the reads of two turns ago
     }
     float s = state;
     if (ctas > 1) {

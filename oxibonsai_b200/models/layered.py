@@ -618,7 +618,7 @@ class MinGruMixer:
                      for rows in (r.slot_rows, r.batch_rows)}
 
     def cluster(self, portions: int, tokens: int) -> int:
-        """CTAs that share a portion: about four per SM, and no more than have tokens in one round."""
+        """CTAs that share a portion: about four per SM, and no more than have tokens at a time."""
         n, ctas = 1, portions * -(-self.spec.width // 32)
         while n < 8 and 2 * n * ctas <= 4 * self.r.scratch.sms and 2 * n * L.lib().bonsai_lay_gru_tokens() <= tokens:
             n *= 2
